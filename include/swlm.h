@@ -87,6 +87,9 @@ int swlm_weights_add_dense_bf16(swlm_ctx* ctx, const char* name, int64_t rows, i
 /* Dense fp32 tensor, replicated: the recurrent layers' norm weight and A_log, which the reference keeps in fp32
  * whatever the bundle's dtype (STAF/STAFConversionPlanner.swift:117-127). */
 int swlm_weights_add_dense_f32(swlm_ctx* ctx, const char* name, int64_t count, const float* data);
+/* Dense bf16 matrix [n][k] of a SWLM_STEP_PRODUCT or latent-attention step, replicated. Rows are padded to a multiple of
+ * 8 columns on the device. */
+int swlm_weights_add_matrix_bf16(swlm_ctx* ctx, const char* name, int n, int k, const uint16_t* data);
 /* Total bytes of weights resident on the device for this context. */
 int64_t swlm_weights_bytes(const swlm_ctx* ctx);
 
@@ -189,6 +192,25 @@ int swlm_get_positions(const swlm_state* state, int32_t* positions);      /* [ma
 int swlm_prefill_seq(swlm_state* state, int seq, const int32_t* tokens, int n, int32_t* first_token);
 /* Position 0 and a cleared short-conv state for one sequence. */
 int swlm_state_reset_seq(swlm_state* state, int seq);
+/* ---- one batch of unequal portions (fp32-stream plans) ----------------------------------------------------------
+ * Runs counts[e] tokens of sequence seqs[e] for every entry e together, each from where its sequence stands: portions of
+ * prompts beside single decoded tokens. `tokens` holds the entries' tokens one after the other. Of entry e the places
+ * wants[...] (want_counts[e] of them, ascending or not, counted from the entry's first token) get logits and a greedy
+ * token: logits_out is [sum of want_counts][vocab] fp32, tokens_out [sum of want_counts] (either may be NULL). A sequence
+ * may appear once. Pages are taken from the pool before anything runs; when it has too few, nothing is changed and
+ * SWLM_ERR_STATE is returned. Steps of one token per entry, its logits wanted, replay a CUDA graph. */
+int swlm_run_batch(swlm_state* state, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens,
+                   const int32_t* want_counts, const int32_t* wants, float* logits_out, int32_t* tokens_out);
+/* Pages of 64 tokens that no sequence holds (fp32-stream plans; -1 otherwise). */
+int swlm_pool_free_pages(const swlm_state* state);
+/* fp32 forms of the probes for fp32-stream plans: the last decode step's logits [max_batch][vocab], and the first `rows` rows
+ * x count_per_row entries of a logical buffer as the last batch or step left it (bf16 buffers are converted). Writing
+ * addresses the buffers of decode steps and swlm_run_step. */
+int swlm_read_logits_f32(swlm_state* state, float* dst, size_t count);
+int swlm_read_buffer_f32(swlm_state* state, int buf, int rows, int count_per_row, float* dst);
+int swlm_write_buffer_f32(swlm_state* state, int buf, int rows, int count_per_row, const float* src);
+/* Cached rows of one latent layer and sequence as fp32: [count][rank + rotated entries]. */
+int swlm_read_latent(swlm_state* state, int layer, int seq, int count, float* dst);
 /* Execute one plan step on the current buffers (kernel-level parity tests). */
 int swlm_run_step(swlm_state* state, const swlm_step* step, const int32_t* token_in, int32_t* token_out);
 /* Kernel launches issued by this state since creation. */

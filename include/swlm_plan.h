@@ -88,7 +88,24 @@ enum {
        RMS norm over value_dim with `weight2` and the gate z * sigmoid(z).
        weight = conv taps [conv_dim][conv_kernel] bf16, weight2 = norm weight [value_dim] fp32, weight3 = dt_bias
        [heads] bf16, weight4 = A_log [heads] fp32 (the two fp32 tensors: swlm_weights_add_dense_f32). */
-    SWLM_STEP_SSM_RECURRENCE = 12
+    SWLM_STEP_SSM_RECURRENCE = 12,
+    /* ---- steps of fp32-stream plans (swlm_buffers_desc.stream_dtype != 0); no counterpart in the reference ----
+       Such plans also use EMBED (times `scale` when it is not 0), the three norm steps, SWIGLU / GEGLU and ARGMAX. */
+    /* out[n] = sum_k W[n][k] in[k], W a dense bf16 matrix (swlm_weights_add_matrix_bf16), fp32 accumulation. */
+    SWLM_STEP_PRODUCT = 13,
+    /* Sandwich norm: t = in * rsqrt(mean(in^2)+eps) * (weight + weight_bias); residual += t;
+       out = residual * rsqrt(mean(residual^2)+eps) * (weight2 + weight_bias). */
+    SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM = 14,
+    /* the same in front of the output head: the sum is not stored */
+    SWLM_STEP_POSTNORM_RESADD_RMSNORM = 15,
+    /* Latent attention. in_buf = q (heads * (head_dim + key_dim): per head head_dim plain, then key_dim rotated entries),
+       in2_buf = n latent entries followed by key_dim entries of the key part that all heads share, in3_buf = gate (heads,
+       before the sigmoid; SWLM_BUF_NONE: no gate), out_buf = heads * value_dim.
+       The latent c is RMS-normed (`weight`, eps, weight_bias); rotate-half rotary positions act on the first rope_dim of
+       the key_dim entries of q and of the shared key part. Cached per token: c and the rotated key part. Per head the
+       plain key is weight2 [heads * head_dim][n] c, the value weight3 [heads * value_dim][n] c; score = (q . k over both
+       parts) * scale, softmax over all positions up to the token's own; out = sigmoid(gate) * value sum. */
+    SWLM_STEP_LATENT_ATTN = 16
 };
 
 typedef struct swlm_step {
@@ -121,6 +138,13 @@ typedef struct swlm_step {
     int32_t value_dim;
     char    weight3[SWLM_NAME_MAX];
     char    weight4[SWLM_NAME_MAX];
+    /* SWLM_STEP_LATENT_ATTN: rotary frequencies interpolated by parts (YaRN). rope_factor 0 = plain frequencies; else pairs
+       that turn fewer than rope_slow times over rope_original positions are divided by rope_factor, pairs that turn more
+       than rope_fast times stay, a linear ramp in between, and cos and sin are multiplied by 0.1 ln(rope_factor) + 1. */
+    float   rope_factor;
+    float   rope_original;
+    float   rope_fast;
+    float   rope_slow;
 } swlm_step;
 
 /* Sizes of the runtime buffer set; mirrors the inputs of
@@ -164,7 +188,18 @@ typedef struct swlm_buffers_desc {
        (Phi . q_rotated) . (that row's values) (qjl_compute_residual, qjl_project_query, qjl_score_correction,
        :1983-2048). */
     int32_t kv_qjl_dim;
+    /* fp32-stream plans: hidden, residual and logits are kept in fp32 (as are scratch slots 3 and 4), the other scratch
+       slots and the cache in bf16 (SWLM_STREAM_F32) or everything in fp32 with true fp32 products (SWLM_STREAM_ALL_F32).
+       0 = the bf16 buffers of the reference. Buffer widths follow from the steps (slot_dim is not used). */
+    int32_t stream_dtype;
+    int32_t latent_layers;   /* number of latent-attention layers (page pools) */
+    /* tokens the page pool of the latent rows holds over all sequences, rounded up to pages of 64;
+       0 = max_batch * max_seq. Sequences take pages as they grow and give them back when they are reset. */
+    int32_t kv_pool_tokens;
 } swlm_buffers_desc;
+
+enum { SWLM_STREAM_BF16 = 0, SWLM_STREAM_F32 = 1, SWLM_STREAM_ALL_F32 = 2 };
+#define SWLM_PAGE_TOKENS 64
 
 enum {
     SWLM_KV_BF16 = 0x01,

@@ -7,7 +7,7 @@ relative imports are used throughout.
 Nothing here computes: every numeric path goes through the C ABI declared in include/swlm.h,
 and loading fails loudly when the CUDA library has not been built.
 """
-from .lib import Library, SwlmError, load_library  # noqa: F401
+from .lib import Library, SwlmError, build_library, load_library  # noqa: F401
 from .formats import (  # noqa: F401
     AffineQ4Group64Format,
     AffineQ4Group128Format,
@@ -24,7 +24,9 @@ from .plan import (  # noqa: F401
     llama3_8b_config,
     lfm2_like_config,
 )
-from .model import InferenceModel, WeightStore, bundle_tensors, load_model, load_model_from_staf  # noqa: F401
-from . import bundle, formats, plan, staf, tp  # noqa: F401
-from .bundle import load_bundle, prepare_bundle  # noqa: F401
+from .model import InferenceModel, WeightStore, bundle_tensors, load_model, load_model_from_staf, upload_weights  # noqa: F401
+from . import bundle, formats, plan, staf, tp, vuzunex  # noqa: F401
+from .bundle import load_bundle, prepare_bundle, prepare_dense_bundle  # noqa: F401
+from .scheduler import BatchScheduler, Request, SequenceSlots  # noqa: F401
+from .vuzunex import VuzunexConfig, VuzunexPlanBuilder  # noqa: F401
 from .synth import synth_model_weights, synth_q4  # noqa: F401

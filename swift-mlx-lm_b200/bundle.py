@@ -17,6 +17,7 @@ import os
 from typing import Dict, Optional, Tuple
 
 from . import staf as _staf
+from . import vuzunex as _vuzunex
 from .plan import DispatchPlanBuilder, ModelConfig
 
 # model_type values ModelGraphResolver.resolveModelGraph sends to the plain Transformer recipe (:9-13), without the
@@ -24,6 +25,9 @@ from .plan import DispatchPlanBuilder, ModelConfig
 TRANSFORMER_MODEL_TYPES = ("llama", "qwen2", "qwen3", "mistral", "phi", "phi3", "starcoder2", "gpt_neox", "internlm2",
                            "deepseek", "yi", "baichuan", "chatglm")
 LFM2_MODEL_TYPES = ("lfm2",)
+
+# config.json `architecture` values of dense bf16 checkpoints: name -> (config decoder, plan builder)
+ARCHITECTURES = {_vuzunex.ARCHITECTURE: (_vuzunex.decode_config, _vuzunex.VuzunexPlanBuilder)}
 
 # KVCachePolicy of InferencePolicy.default (Sources/MetalCompiler/InferencePolicy.swift:55-100)
 DEFAULT_MAXIMUM_SEQUENCE_LENGTH = 4096
@@ -166,8 +170,57 @@ def prepare_bundle(directory: str, max_seq: Optional[int] = None, max_batch: int
     return cfg, DispatchPlanBuilder(cfg), _staf.read_staf(out)
 
 
+def read_config(directory: str) -> Dict:
+    path = os.path.join(directory, "config.json")
+    if not os.path.exists(path):
+        raise BundleError(f"{directory}: no config.json")
+    with open(path, "rb") as f:
+        config = json.loads(f.read().decode())
+    if not isinstance(config, dict):
+        raise BundleError("config.json is not a JSON object")
+    return config
+
+
+def prepare_dense_bundle(directory: str, config: Optional[Dict] = None, **runtime):
+    """A dense bf16 checkpoint whose config.json names an `architecture` of the registry: decode the config, check every tensor
+    of the plan against the shards. Returns (builder, name -> bf16 bit patterns). `runtime`: dtype, max_seq, max_batch, pool_tokens."""
+    config = read_config(directory) if config is None else config
+    entry = ARCHITECTURES.get(config.get("architecture"))
+    if entry is None:
+        raise BundleError(f"Unsupported architecture: {config.get('architecture')}")
+    decode, make_builder = entry
+    try:
+        builder = make_builder(decode(config, **runtime))
+    except (KeyError, TypeError, ValueError) as e:
+        raise BundleError(f"{config['architecture']}: {e!r}") from e
+    shards = sorted(glob.glob(os.path.join(directory, "*.safetensors")))
+    if not shards:
+        raise BundleError(f"{directory}: no safetensors shard")
+    found = {}
+    for path in shards:
+        found.update(_staf.read_safetensors(path))
+    weights = {}
+    for name, _kind, shape, _shard in builder.tensors():
+        if name not in found:
+            raise BundleError(f"tensor {name} is missing")
+        dtype, got, data = found[name]
+        if tuple(got) != tuple(shape):
+            raise BundleError(f"tensor {name} is {tuple(got)}, the configuration says {tuple(shape)}")
+        if dtype != "BF16":
+            raise BundleError(f"tensor {name}: dtype {dtype}, bf16 expected")
+        weights[name] = data
+    return builder, weights
+
+
 def load_bundle(directory: str, store, **kw):
-    """prepare_bundle, then upload what the plan needs from the STAF file and build the plan (needs a GPU)."""
+    """A model directory into a running model (needs a GPU). config.json decides: an `architecture` of the registry is loaded
+    from its bf16 shards, anything else goes through prepare_bundle and the STAF file."""
+    config = read_config(directory)
+    if config.get("architecture") in ARCHITECTURES:
+        from .model import load_model
+
+        builder, weights = prepare_dense_bundle(directory, config, **kw)
+        return load_model(store, builder, weights)
     from .model import load_model_from_staf
 
     _cfg, builder, staf_file = prepare_bundle(directory, **kw)

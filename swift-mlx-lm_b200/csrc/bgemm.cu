@@ -1,0 +1,595 @@
+// Dense products of fp32-stream plans: Y[m][n] = X[m][k] . W[n][k]^T with bf16 weights and fp32 accumulation.
+//
+//   bgemv_kernel     1..kGemvRows activation rows: the weights are streamed once from HBM with 16-byte loads, four weight
+//                    rows per warp and K cut across the warps of a CTA; the norm in front of the product can run in the
+//                    prologue, gate and up in one launch with the gated activation in the epilogue. Activations bf16 or fp32
+//                    (with fp32 ones the product is a true fp32 product: a bf16 weight is exact in fp32).
+//   bgemm_tc_kernel  more rows, bf16 activations: tcgen05.mma with both operands staged by TMA (128-byte swizzle), two tiles
+//                    of 128 weight rows side by side in tensor memory, K cut across CTAs when there are few tiles. The two
+//                    tiles are 256 consecutive rows, or 128 rows of gate and the same rows of up.
+//   sgemm_kernel     more rows, fp32 activations: fp32 FMAs on 64 x 64 tiles.
+#include <algorithm>
+#include <cstdlib>
+
+#include "swlm_internal.h"
+#include "tc_device.cuh"
+
+namespace swlm {
+namespace {
+
+__device__ __forceinline__ float b_lo(unsigned w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float b_hi(unsigned w) { return __uint_as_float(w & 0xFFFF0000u); }
+__device__ __forceinline__ uint4 ldg_stream(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
+__device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
+    void* y = o.y[0];
+    int first = 0, stride = o.stride[0], f32 = o.f32[0];
+#pragma unroll
+    for (int q = 1; q < kMaxProductSegs; ++q)
+        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; }
+    const size_t at = (size_t)m * stride + (row - first);
+    if (f32) static_cast<float*>(y)[at] = val;
+    else static_cast<__nv_bfloat16*>(y)[at] = __float2bfloat16_rn(val);
+}
+
+// ---- few rows ---------------------------------------------------------------------------------------------------------
+constexpr int kGemvRows = 4;
+constexpr int kGemvThreads = 256, kGemvWarps = kGemvThreads / 32;
+constexpr int kGemvUnroll = 4;                       // 16-byte loads in flight per weight row and lane
+constexpr size_t kGemvMaxSmem = 200 * 1024;
+
+struct GemvParams {
+    const __nv_bfloat16* w; const __nv_bfloat16* w2;
+    int ld, n, k, m, act;
+    const void* x; int x_stride;
+    StreamNorm norm;
+    ProductOut out;
+};
+
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < kGemvWarps; ++i) total += red[i];
+    __syncthreads();
+    return total;
+}
+__device__ __forceinline__ void put_x(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put_x(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+// eight consecutive activations
+__device__ __forceinline__ void get_x8(const float* p, float (&f)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void get_x8(const __nv_bfloat16* p, float (&f)[8]) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    f[0] = b_lo(v.x); f[1] = b_hi(v.x); f[2] = b_lo(v.y); f[3] = b_hi(v.y); f[4] = b_lo(v.z); f[5] = b_hi(v.z); f[6] = b_lo(v.w); f[7] = b_hi(v.w);
+}
+
+// A warp takes groups of four weight rows (GATED: two of gate and the same two of up); WK warps share a group and cut K.
+template <typename T, int MR, int WK, bool GATED>
+__global__ void __launch_bounds__(kGemvThreads) bgemv_kernel(const GemvParams p) {
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) unsigned char gemv_raw[];
+    __shared__ float red[kGemvWarps];
+    __shared__ float part[kGemvWarps][4 * MR];
+    T* xs = reinterpret_cast<T*>(gemv_raw);                    // [MR][ld]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int kw = warp % WK, rg = warp / WK;
+    constexpr int ROWS = GATED ? 2 : 4;                         // output rows of a group
+    const int groups = (p.n + ROWS - 1) / ROWS, per_cta = kGemvWarps / WK;
+    const int chunks = p.ld >> 3;                               // 16-byte chunks per weight row
+    constexpr int STEP = 32 * WK;
+
+    auto row_ptr = [&](int group, int i) -> const __nv_bfloat16* {
+        const int r = min(group * ROWS + (GATED ? (i & 1) : i), p.n - 1);
+        return (GATED && i >= 2 ? p.w2 : p.w) + (size_t)r * p.ld;
+    };
+    uint4 wv[4][kGemvUnroll];
+    auto load = [&](int group, int c0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const __nv_bfloat16* row = row_ptr(group, i);
+#pragma unroll
+            for (int u = 0; u < kGemvUnroll; ++u) {
+                const int c = c0 + u * STEP;
+                wv[i][u] = c < chunks ? ldg_stream(row + 8 * c) : make_uint4(0, 0, 0, 0);
+            }
+        }
+    };
+    const int first_chunk = kw * 32 + lane;
+    int group = blockIdx.x * per_cta + rg;
+    // the first weights do not depend on the preceding kernel
+    if (group < groups) load(group, first_chunk);
+    pdl_wait();
+
+    // ---- activations to shared memory: plain rows, or the norm in front of the product (every CTA computes it; CTA 0 stores
+    // the new residual) ----
+    if (p.norm.mode) {
+        for (int m = 0; m < MR; ++m) {
+            T* xr = xs + (size_t)m * p.ld;
+            float* rowf = reinterpret_cast<float*>(gemv_raw + (size_t)MR * p.ld * sizeof(T));
+            const float* in = p.norm.in + (size_t)m * p.norm.in_stride;
+            const float* res = p.norm.res_in ? p.norm.res_in + (size_t)m * p.norm.res_stride : nullptr;
+            float post_scale = 1.f;
+            float ss = 0.f;
+            for (int i = tid; i < p.k; i += kGemvThreads) { const float v = in[i]; rowf[i] = v; ss = fmaf(v, v, ss); }
+            if (p.norm.w_post) post_scale = 1.0f / sqrtf(cta_sum(ss, red) / (float)p.k + p.norm.eps);
+            ss = 0.f;
+            for (int i = tid; i < p.k; i += kGemvThreads) {
+                float h = rowf[i];
+                if (p.norm.w_post) h = h * post_scale * (__bfloat162float(p.norm.w_post[i]) + p.norm.weight_bias);
+                if (res) h += res[i];
+                if (p.norm.res_out && blockIdx.x == 0) p.norm.res_out[(size_t)m * p.norm.res_stride + i] = h;
+                rowf[i] = h;
+                ss = fmaf(h, h, ss);
+            }
+            const float sc = 1.0f / sqrtf(cta_sum(ss, red) / (float)p.k + p.norm.eps);
+            for (int i = tid; i < p.ld; i += kGemvThreads)
+                put_x(xr + i, i < p.k ? rowf[i] * sc * (__bfloat162float(p.norm.w[i]) + p.norm.weight_bias) : 0.f);
+        }
+    } else {
+        for (int m = 0; m < MR; ++m) {
+            const T* src = static_cast<const T*>(p.x) + (size_t)m * p.x_stride;
+            for (int i = tid; i < p.ld; i += kGemvThreads) { T v = T(0.0f); if (i < p.k) v = src[i]; xs[(size_t)m * p.ld + i] = v; }
+        }
+    }
+    __syncthreads();
+
+    const int rounds = (groups + gridDim.x * per_cta - 1) / (gridDim.x * per_cta);
+    for (int it = 0; it < rounds; ++it) {
+        float acc[4][MR];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int m = 0; m < MR; ++m) acc[i][m] = 0.f;
+        const bool live = group < groups;
+        if (live) {
+            for (int c0 = first_chunk; c0 < chunks; c0 += STEP * kGemvUnroll) {
+                if (it > 0 || c0 != first_chunk) load(group, c0);
+#pragma unroll
+                for (int u = 0; u < kGemvUnroll; ++u) {
+                    const int c = c0 + u * STEP;
+                    if (c < chunks) {
+                        float wf[4][8];
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const uint4 v = wv[i][u];
+                            wf[i][0] = b_lo(v.x); wf[i][1] = b_hi(v.x); wf[i][2] = b_lo(v.y); wf[i][3] = b_hi(v.y);
+                            wf[i][4] = b_lo(v.z); wf[i][5] = b_hi(v.z); wf[i][6] = b_lo(v.w); wf[i][7] = b_hi(v.w);
+                        }
+#pragma unroll
+                        for (int m = 0; m < MR; ++m) {
+                            float xf[8];
+                            get_x8(xs + (size_t)m * p.ld + 8 * c, xf);
+#pragma unroll
+                            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                                for (int e = 0; e < 8; ++e) acc[i][m] = fmaf(wf[i][e], xf[e], acc[i][m]);
+                        }
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int m = 0; m < MR; ++m)
+                for (int o = 16; o > 0; o >>= 1) acc[i][m] += __shfl_xor_sync(0xffffffffu, acc[i][m], o);
+        if (WK > 1) {
+            if (lane == 0) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int m = 0; m < MR; ++m) part[warp][i * MR + m] = acc[i][m];
+            }
+            __syncthreads();
+            if (kw == 0) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int m = 0; m < MR; ++m) {
+                        float v = 0.f;
+#pragma unroll
+                        for (int q = 0; q < WK; ++q) v += part[rg * WK + q][i * MR + m];
+                        acc[i][m] = v;
+                    }
+            }
+            __syncthreads();
+        }
+        if (live && kw == 0) {
+            // lane (i * MR + m) stores one value
+#pragma unroll
+            for (int m = 0; m < MR; ++m) {
+                if (GATED) {
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        const int row = group * 2 + i;
+                        if (lane == i * MR + m && row < p.n) product_store(p.out, m, row, gated_activation(acc[i][m], acc[2 + i][m], p.act));
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int row = group * 4 + i;
+                        if (lane == i * MR + m && row < p.n) product_store(p.out, m, row, acc[i][m]);
+                    }
+                }
+            }
+        }
+        group += gridDim.x * per_cta;
+    }
+}
+
+// ---- many rows, bf16: tcgen05 -----------------------------------------------------------------------------------------
+constexpr int kTileRows = 128;       // weight rows of one accumulator = UMMA M
+constexpr int kTcK = 64;             // columns per stage = one 128-byte swizzle row
+constexpr int kTcWarps = 6;          // TMA, MMA, four epilogue warps
+constexpr int kTcBlock = kTcWarps * 32;
+
+struct TcParams {
+    int n, m, steps;                 // weight rows, activation rows, 64-column steps of K
+    int split_steps;                 // steps per K range (gridDim.z ranges); == steps when K is not cut
+    int act;
+    ProductOut out;
+    float* part;                     // [range][gated ? 2 : 1][m][n] when K is cut
+    int* status;
+};
+
+// kind::f16: D fp32, A = B = bf16, both K-major, M = 128
+__host__ __device__ constexpr unsigned tc_idesc(int bn) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(bn >> 3) << 17) | ((unsigned)(kTileRows >> 4) << 24);
+}
+__device__ __forceinline__ void umma_bf16(unsigned d_tmem, unsigned long long a_desc, unsigned long long b_desc, unsigned idesc, unsigned accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
+}
+
+template <int BN, int STAGES, bool GATED>
+__global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap xmap,
+                                                           const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap wmap2) {
+    extern __shared__ __align__(1024) unsigned char tc_raw[];
+    unsigned char* smem = tc_raw + ((1024 - (smem_u32(tc_raw) & 1023)) & 1023);   // swizzle atoms
+    constexpr int A_BYTES = kTileRows * 128, B_BYTES = BN * 128;
+    constexpr unsigned kCols = 2 * BN < 32 ? 32 : 2 * BN;
+    __shared__ __align__(8) unsigned long long full_bar[STAGES], empty_bar[STAGES], done_bar;
+    __shared__ unsigned tmem_base;
+    __shared__ int failed;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tok0 = blockIdx.x * BN;
+    const int row0 = blockIdx.y * (GATED ? kTileRows : 2 * kTileRows);
+    const int nt = !GATED && row0 + kTileRows >= p.n ? 1 : 2;                       // accumulators in use
+    const int stage_bytes = nt * A_BYTES + B_BYTES;
+    constexpr int STAGE = 2 * A_BYTES + B_BYTES;
+    const int step0 = blockIdx.z * p.split_steps;
+    const int steps = min(p.split_steps, p.steps - step0);
+    if (tid == 0) {
+        for (int s = 0; s < STAGES; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
+        mbar_init(&done_bar, 1);
+        failed = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        __syncwarp();
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base)), "r"(kCols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const unsigned tmem = tmem_base;
+    pdl_launch_dependents();   // behind the allocation: a successor that wants tensor memory cannot get in between
+
+    if (warp == 0) {
+        if (lane == 0) {
+            // the weights of the first stages do not depend on the preceding kernel; the activations do
+            const int ahead = min(STAGES, steps);
+            auto weights = [&](int kt, int s) {
+                const unsigned bar = smem_u32(&full_bar[s]), dst = smem_u32(smem + s * STAGE);
+                mbar_expect(bar, (unsigned)stage_bytes);
+                tma_load_2d(dst, &wmap, (step0 + kt) * kTcK, row0, bar);
+                if (nt == 2) tma_load_2d(dst + A_BYTES, GATED ? &wmap2 : &wmap, (step0 + kt) * kTcK, GATED ? row0 : row0 + kTileRows, bar);
+            };
+            auto activations = [&](int kt, int s) {
+                tma_load_2d(smem_u32(smem + s * STAGE) + 2 * A_BYTES, &xmap, (step0 + kt) * kTcK, tok0, smem_u32(&full_bar[s]));
+            };
+            for (int kt = 0; kt < ahead; ++kt) weights(kt, kt);
+            pdl_wait();
+            for (int kt = 0; kt < ahead; ++kt) activations(kt, kt);
+            int issued = ahead;
+            for (int kt = ahead; kt < steps; ++kt) {
+                const int s = kt % STAGES;
+                if (!mbar_wait(&empty_bar[s], (unsigned)((kt / STAGES - 1) & 1))) { atomicExch(p.status, 31); failed = 1; break; }
+                weights(kt, s);
+                activations(kt, s);
+                issued = kt + 1;
+            }
+            if (failed)   // copies already requested still write shared memory
+                for (int kt = issued > STAGES ? issued - STAGES : 0; kt < issued; ++kt) mbar_wait(&full_bar[kt % STAGES], (unsigned)((kt / STAGES) & 1));
+        }
+        __syncwarp();
+    } else if (warp == 1) {
+        if (lane == 0) {
+            constexpr unsigned idesc = tc_idesc(BN);
+            for (int kt = 0; kt < steps; ++kt) {
+                const int s = kt % STAGES;
+                if (!mbar_wait(&full_bar[s], (unsigned)((kt / STAGES) & 1))) { atomicExch(p.status, 32); failed = 1; break; }
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                const unsigned a = smem_u32(smem + s * STAGE), b = a + 2 * A_BYTES;
+#pragma unroll
+                for (int j = 0; j < kTcK / 16; ++j) {
+                    const unsigned acc = (kt > 0 || j > 0) ? 1u : 0u;
+                    umma_bf16(tmem, umma_desc(a + 32 * j), umma_desc(b + 32 * j), idesc, acc);
+                    if (nt == 2) umma_bf16(tmem + BN, umma_desc(a + A_BYTES + 32 * j), umma_desc(b + 32 * j), idesc, acc);
+                }
+                umma_commit(&empty_bar[s]);
+            }
+            umma_commit(&done_bar);   // also behind whatever was issued before a failure
+        }
+        __syncwarp();
+    } else {
+        // ---- epilogue: a warp reads the 32 accumulator lanes of its quarter (warp & 3), lane = weight row ----
+        pdl_wait();   // the outputs may still be read by the kernel before this one
+        const bool ok = mbar_wait(&done_bar, 0u);
+        if (!ok) { atomicExch(p.status, 33); }
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (ok && !failed) {
+            const int quarter = warp & 3;
+            const bool cut = gridDim.z > 1;
+#pragma unroll 1
+            for (int t = 0; t < (GATED && !cut ? 1 : nt); ++t) {
+                const int row = row0 + (GATED ? 0 : t * kTileRows) + quarter * 32 + lane;
+#pragma unroll 1
+                for (int c0 = 0; c0 < BN; c0 += 16) {
+                    if (tok0 + c0 >= p.m) break;   // uniform across the warp
+                    unsigned v[16], u[16];
+                    const unsigned at = tmem + ((unsigned)(quarter * 32) << 16) + (unsigned)(t * BN + c0);
+                    asm volatile(
+                        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+                        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
+                          "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+                        : "r"(at) : "memory");
+                    if (GATED && !cut)
+                        asm volatile(
+                            "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+                            : "=r"(u[0]), "=r"(u[1]), "=r"(u[2]), "=r"(u[3]), "=r"(u[4]), "=r"(u[5]), "=r"(u[6]), "=r"(u[7]),
+                              "=r"(u[8]), "=r"(u[9]), "=r"(u[10]), "=r"(u[11]), "=r"(u[12]), "=r"(u[13]), "=r"(u[14]), "=r"(u[15])
+                            : "r"(at + BN) : "memory");
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (row < p.n) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) {
+                            const int tok = tok0 + c0 + i;
+                            if (tok >= p.m) break;
+                            const float val = __uint_as_float(v[i]);
+                            if (cut) p.part[(((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m + tok) * p.n + row] = val;
+                            else product_store(p.out, tok, row, GATED ? gated_activation(val, __uint_as_float(u[i]), p.act) : val);
+                        }
+                    }
+                }
+            }
+        }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kCols) : "memory");
+}
+
+// Sum of the K ranges in order, then the store (GATED: activation(gate sum) * up sum).
+template <bool GATED>
+__global__ void __launch_bounds__(256) bgemm_sum_kernel(const float* part, int ranges, int m, int n, int act, const ProductOut out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t total = (size_t)m * n;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        float a = 0.f, b = 0.f;
+        for (int z = 0; z < ranges; ++z) {
+            const float* base = part + (size_t)z * (GATED ? 2 : 1) * total;
+            a += __ldcg(base + i);
+            if (GATED) b += __ldcg(base + total + i);
+        }
+        const int t = (int)(i / n), r = (int)(i - (size_t)t * n);
+        product_store(out, t, r, GATED ? gated_activation(a, b, act) : a);
+    }
+}
+
+// ---- many rows, fp32 --------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) sgemm_kernel(const __nv_bfloat16* w, int ld, int n, int k, int m, const float* x, int x_stride, const ProductOut out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float ws[16][68], xsm[16][68];
+    const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < k; k0 += 16) {
+        for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+            const int r = i >> 4, c = i & 15;
+            ws[c][r] = n0 + r < n && k0 + c < k ? __bfloat162float(w[(size_t)(n0 + r) * ld + k0 + c]) : 0.f;
+            xsm[c][r] = m0 + r < m && k0 + c < k ? x[(size_t)(m0 + r) * x_stride + k0 + c] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int c = 0; c < 16; ++c) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { a[i] = xsm[c][ty * 4 + i]; b[i] = ws[c][tx * 4 + i]; }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    for (int i = 0; i < 4; ++i)
+        for (int j = 0; j < 4; ++j) {
+            const int mm = m0 + ty * 4 + i, nn = n0 + tx * 4 + j;
+            if (mm < m && nn < n) product_store(out, mm, nn, acc[i][j]);
+        }
+}
+
+// ---- launches ---------------------------------------------------------------------------------------------------------
+template <typename T, int MR, int WK, bool GATED>
+int gemv_launch(const GemvParams& p, size_t smem, unsigned grid, cudaStream_t s) {
+    static const cudaError_t attr = cudaFuncSetAttribute(bgemv_kernel<T, MR, WK, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGemvMaxSmem);
+    if (attr != cudaSuccess) return cuda_fail(attr, "bgemv attributes");
+    const cudaError_t e = launch_k(bgemv_kernel<T, MR, WK, GATED>, dim3(grid), dim3(kGemvThreads), smem, s, p);
+    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "bgemv launch");
+}
+template <typename T, int MR>
+int gemv_pick(const GemvParams& p, bool gated, size_t smem, cudaStream_t s) {
+    const int groups = (p.n + (gated ? 1 : 3)) / (gated ? 2 : 4);
+    // warps that share a group: enough for 16 warps per SM, as long as each still has a full round of loads
+    int wk = 1;
+    while (wk < 8 && groups * wk < 148 * 16 && (p.ld >> 3) > 32 * wk * 2) wk *= 2;
+    const int per_cta = kGemvWarps / wk;
+    const unsigned grid = (unsigned)std::min((groups + per_cta - 1) / per_cta, 148 * (smem > 100 * 1024 ? 1 : smem > 64 * 1024 ? 2 : 3));
+    if (gated) {
+        switch (wk) {
+        case 1: return gemv_launch<T, MR, 1, true>(p, smem, grid, s);
+        case 2: return gemv_launch<T, MR, 2, true>(p, smem, grid, s);
+        case 4: return gemv_launch<T, MR, 4, true>(p, smem, grid, s);
+        default: return gemv_launch<T, MR, 8, true>(p, smem, grid, s);
+        }
+    }
+    switch (wk) {
+    case 1: return gemv_launch<T, MR, 1, false>(p, smem, grid, s);
+    case 2: return gemv_launch<T, MR, 2, false>(p, smem, grid, s);
+    case 4: return gemv_launch<T, MR, 4, false>(p, smem, grid, s);
+    default: return gemv_launch<T, MR, 8, false>(p, smem, grid, s);
+    }
+}
+template <typename T>
+int gemv_rows(const GemvParams& p, bool gated, size_t smem, cudaStream_t s) {
+    switch (p.m) {
+    case 1: return gemv_pick<T, 1>(p, gated, smem, s);
+    case 2: return gemv_pick<T, 2>(p, gated, smem, s);
+    case 3: return gemv_pick<T, 3>(p, gated, smem, s);
+    default: return gemv_pick<T, 4>(p, gated, smem, s);
+    }
+}
+size_t gemv_smem(int m, int ld, bool x_f32, bool norm) { return (size_t)m * ld * (x_f32 ? 4 : 2) + (norm ? (size_t)ld * 4 : 0); }
+
+// bf16 matrix [rows][ld] as a 2-D tensor, k columns valid (beyond: zeros); box = 64 columns x box_rows, 128-byte swizzle
+int bf16_map(const __nv_bfloat16* p, int ld, int rows, int k, int box_rows, CUtensorMap* map) {
+    TensorMapEncodeFn fn = tensor_map_encode_fn();
+    if (!fn) { set_error("dense product: cuTensorMapEncodeTiled is not available"); return SWLM_ERR_CUDA; }
+    const cuuint64_t dims[2] = {(cuuint64_t)k, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)kTcK, (cuuint32_t)box_rows};
+    const cuuint32_t estr[2] = {1, 1};
+    const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<__nv_bfloat16*>(p), dims, strides, box, estr,
+                          CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { set_error("dense product: cuTensorMapEncodeTiled failed (%d)", (int)r); return SWLM_ERR_CUDA; }
+    return SWLM_OK;
+}
+
+struct TcShape { int bn, ranges, split_steps, tiles_m, tiles_n; };
+TcShape tc_shape(int n, int k, int m, bool gated) {
+    TcShape t;
+    t.bn = m > 128 ? 256 : m > 64 ? 128 : m > 32 ? 64 : 32;
+    t.tiles_m = (m + t.bn - 1) / t.bn;
+    t.tiles_n = (n + (gated ? kTileRows : 2 * kTileRows) - 1) / (gated ? kTileRows : 2 * kTileRows);
+    const int steps = (k + kTcK - 1) / kTcK, tiles = t.tiles_m * t.tiles_n;
+    int ranges = tiles * 2 > 148 ? 1 : std::min(std::min(148 / tiles, std::max(1, steps / 4)), 16);
+    t.split_steps = (steps + ranges - 1) / ranges;
+    t.ranges = (steps + t.split_steps - 1) / t.split_steps;
+    return t;
+}
+
+template <int BN, int STAGES>
+constexpr size_t tc_smem() { return (size_t)STAGES * (2 * kTileRows * 128 + BN * 128) + 1024; }
+template <int BN, int STAGES, bool GATED>
+int tc_attr() {
+    SWLM_CUDA(cudaFuncSetAttribute(bgemm_tc_kernel<BN, STAGES, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tc_smem<BN, STAGES>()));
+    return SWLM_OK;
+}
+template <int BN, int STAGES>
+int tc_launch(const ProductLaunch& a, const TcShape& t, cudaStream_t s) {
+    const bool gated = a.w2 != nullptr;
+    TcParams p{};
+    p.n = a.w->n; p.m = a.m; p.steps = (a.w->k + kTcK - 1) / kTcK; p.split_steps = t.split_steps; p.act = a.act; p.out = a.out; p.part = a.part; p.status = a.status;
+    CUtensorMap xmap, wmap, wmap2;
+    int rc = bf16_map(static_cast<const __nv_bfloat16*>(a.x), a.x_stride, a.m, a.w->k, BN, &xmap);
+    if (!rc) rc = bf16_map(a.w->data, a.w->ld, a.w->n, a.w->k, kTileRows, &wmap);
+    wmap2 = wmap;
+    if (!rc && gated) rc = bf16_map(a.w2->data, a.w2->ld, a.w2->n, a.w2->k, kTileRows, &wmap2);
+    if (rc) return rc;
+    const dim3 grid((unsigned)t.tiles_m, (unsigned)t.tiles_n, (unsigned)t.ranges);
+    cudaError_t e = gated ? launch_k(bgemm_tc_kernel<BN, STAGES, true>, grid, dim3(kTcBlock), tc_smem<BN, STAGES>(), s, p, xmap, wmap, wmap2)
+                          : launch_k(bgemm_tc_kernel<BN, STAGES, false>, grid, dim3(kTcBlock), tc_smem<BN, STAGES>(), s, p, xmap, wmap, wmap2);
+    if (e != cudaSuccess) return cuda_fail(e, "bgemm launch");
+    if (t.ranges > 1) {
+        const unsigned g = (unsigned)std::min<size_t>(592, ((size_t)p.m * p.n + 255) / 256);
+        e = gated ? launch_k(bgemm_sum_kernel<true>, dim3(g), dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out)
+                  : launch_k(bgemm_sum_kernel<false>, dim3(g), dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out);
+        if (e != cudaSuccess) return cuda_fail(e, "bgemm sum launch");
+    }
+    return SWLM_OK;
+}
+
+bool gemv_fits(int m, int k, bool x_f32, bool norm) {
+    const int ld = (k + 7) / 8 * 8;
+    return m <= kGemvRows && gemv_smem(m, ld, x_f32, norm) <= kGemvMaxSmem;
+}
+
+}  // namespace
+
+int bgemm_init() {
+    int rc;
+    if ((rc = tc_attr<32, 4, false>()) || (rc = tc_attr<32, 4, true>()) || (rc = tc_attr<64, 4, false>()) || (rc = tc_attr<64, 4, true>()) ||
+        (rc = tc_attr<128, 4, false>()) || (rc = tc_attr<128, 4, true>()) || (rc = tc_attr<256, 3, false>()) || (rc = tc_attr<256, 3, true>())) return rc;
+    return SWLM_OK;
+}
+
+bool product_takes_norm(int m, int k) { return m <= 2 && k <= 16384 && gemv_fits(m, k, true, true); }
+// gate and up in one launch: always, except as true fp32 products over many rows
+bool product_takes_gate(int m, int k, bool x_f32) { return !x_f32 || gemv_fits(m, k, true, false); }
+
+size_t product_part_floats(int n, int k, int m, bool gated) {
+    if (gemv_fits(m, k, false, false)) return 0;
+    const TcShape t = tc_shape(n, k, m, gated);
+    return t.ranges > 1 ? (size_t)t.ranges * (gated ? 2 : 1) * m * n : 0;
+}
+
+int product_launch_count(const ProductLaunch& a) {
+    if (gemv_fits(a.m, a.w->k, a.x_f32, a.norm.mode != 0) || a.x_f32) return 1;
+    return tc_shape(a.w->n, a.w->k, a.m, a.w2 != nullptr).ranges > 1 ? 2 : 1;
+}
+
+int launch_product(const ProductLaunch& a, cudaStream_t s) {
+    if (a.m <= 0) return SWLM_OK;
+    const bool gated = a.w2 != nullptr;
+    if (gated && (a.w2->n != a.w->n || a.w2->k != a.w->k)) { set_error("gated product: the two matrices differ in shape"); return SWLM_ERR_INVALID; }
+    if (gemv_fits(a.m, a.w->k, a.x_f32, a.norm.mode != 0)) {
+        GemvParams p{};
+        p.w = a.w->data; p.w2 = gated ? a.w2->data : nullptr; p.ld = a.w->ld; p.n = a.w->n; p.k = a.w->k; p.m = a.m; p.act = a.act;
+        p.x = a.x; p.x_stride = a.x_stride; p.norm = a.norm; p.out = a.out;
+        const size_t smem = gemv_smem(a.m, a.w->ld, a.x_f32, a.norm.mode != 0);
+        return a.x_f32 ? gemv_rows<float>(p, gated, smem, s) : gemv_rows<__nv_bfloat16>(p, gated, smem, s);
+    }
+    if (a.norm.mode) { set_error("a norm in front of a product over %d rows runs on its own", a.m); return SWLM_ERR_INVALID; }
+    if (a.x_f32) {
+        if (gated) { set_error("gate and up of fp32 rows run one after the other"); return SWLM_ERR_INVALID; }
+        const cudaError_t e = launch_k(sgemm_kernel, dim3((a.w->n + 63) / 64, (a.m + 63) / 64), dim3(256), 0, s, (const __nv_bfloat16*)a.w->data,
+                                       a.w->ld, a.w->n, a.w->k, a.m, static_cast<const float*>(a.x), a.x_stride, a.out);
+        return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "sgemm launch");
+    }
+    if ((a.x_stride & 7) || (reinterpret_cast<uintptr_t>(a.x) & 15)) { set_error("dense product: activation rows must be 16-byte aligned"); return SWLM_ERR_INVALID; }
+    const TcShape t = tc_shape(a.w->n, a.w->k, a.m, gated);
+    if (t.ranges > 1 && (!a.part || a.part_floats < (size_t)t.ranges * (gated ? 2 : 1) * a.m * a.w->n)) { set_error("dense product: scratch too small"); return SWLM_ERR_INVALID; }
+    switch (t.bn) {
+    case 32: return tc_launch<32, 4>(a, t, s);
+    case 64: return tc_launch<64, 4>(a, t, s);
+    case 128: return tc_launch<128, 4>(a, t, s);
+    default: return tc_launch<256, 3>(a, t, s);
+    }
+}
+
+}  // namespace swlm

@@ -227,16 +227,20 @@ __device__ __forceinline__ void argmax_merge(float& v, int& i, float ov, int oi)
     if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
 }
 
-__global__ void __launch_bounds__(256) argmax_partial_kernel(int n, const __nv_bfloat16* logits, int stride,
+__device__ __forceinline__ float logit_value(float v) { return v; }
+__device__ __forceinline__ float logit_value(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+template <typename T>
+__global__ void __launch_bounds__(256) argmax_partial_kernel(int n, const T* logits, int stride,
                                                             float* pval, int32_t* pidx) {
     pdl_launch_dependents();
     pdl_wait();
     const int b = blockIdx.y;
-    const __nv_bfloat16* row = logits + (size_t)b * stride;
+    const T* row = logits + (size_t)b * stride;
     float best = -INFINITY;
     int bi = 0x7fffffff;
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
-        const float v = __bfloat162float(row[i]);
+        const float v = logit_value(row[i]);
         if (v > best) { best = v; bi = i; }   // i ascends within a thread: first maximum is kept
     }
     for (int o = 16; o > 0; o >>= 1) {
@@ -577,9 +581,21 @@ int launch_argmax(int m, int n, const __nv_bfloat16* logits, int stride, int32_t
                   int32_t* ring, int32_t* step_counter, int ring_cap, int32_t* position, int advance,
                   float* scratch_val, int32_t* scratch_idx, const TpParams& tp, int32_t* am_epoch, int shard_offset,
                   cudaStream_t s) {
-    launch_k(argmax_partial_kernel, dim3(kArgmaxBlocks, m), 256, 0, s, n, logits, stride, scratch_val, scratch_idx);
+    launch_k(argmax_partial_kernel<__nv_bfloat16>, dim3(kArgmaxBlocks, m), 256, 0, s, n, logits, stride, scratch_val, scratch_idx);
     launch_k(argmax_final_kernel, 1, 256, 0, s, m, scratch_val, scratch_idx, token_out, token_in_next, ring, step_counter,
                                           ring_cap, position, advance, tp, am_epoch, shard_offset);
+    return check_launch("argmax launch");
+}
+
+int launch_argmax_f32(int m, int n, const float* logits, int stride, int32_t* token_out, int32_t* token_in_next, int32_t* ring,
+                      int32_t* step_counter, int ring_cap, int32_t* position, int advance, float* scratch_val, int32_t* scratch_idx, cudaStream_t s) {
+    if (m > kMaxSequences && (advance || ring || token_in_next)) { set_error("argmax: %d rows cannot advance together", m); return SWLM_ERR_INVALID; }
+    for (int r0 = 0; r0 < m; r0 += kMaxSequences) {
+        const int c = std::min(kMaxSequences, m - r0);
+        launch_k(argmax_partial_kernel<float>, dim3(kArgmaxBlocks, c), 256, 0, s, n, logits + (size_t)r0 * stride, stride, scratch_val, scratch_idx);
+        launch_k(argmax_final_kernel, 1, 256, 0, s, c, scratch_val, scratch_idx, token_out + r0, token_in_next, ring, step_counter, ring_cap, position,
+                 advance, TpParams{}, (int32_t*)nullptr, 0);
+    }
     return check_launch("argmax launch");
 }
 

@@ -36,6 +36,7 @@
 #include <cstdlib>
 #include <cuda.h>
 #include "swlm_internal.h"
+#include "tc_device.cuh"
 
 namespace swlm {
 namespace {
@@ -44,7 +45,6 @@ constexpr int kTcThreads = 512;          // dequantising threads
 constexpr int kTcAllThreads = kTcThreads + 64;  // + the MMA warp and the activation (TMA) warp
 constexpr int kTcRows = 128;            // weight rows per CTA = UMMA M
 constexpr int kTcBK = 64;               // one quantisation group per pipeline stage
-constexpr int kTcSpinLimit = 1 << 22;
 
 struct QGemmTcParams {
     const uint32_t* w;        // [n][k/8] MLX words
@@ -64,46 +64,6 @@ struct QGemmTcParams {
     int split_steps;
 };
 
-__device__ __forceinline__ unsigned smem_u32(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
-
-__device__ __forceinline__ void mbar_init(unsigned long long* bar, unsigned count) {
-    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count) : "memory");
-}
-// Bounded wait on phase parity; returns false when the limit was reached. The loop is two instructions per
-// attempt (try_wait suspends the warp for a while by itself): waiting warps share their scheduler with warps
-// that still dequantise.
-__device__ __forceinline__ bool mbar_wait_addr(unsigned addr, unsigned parity) {
-    unsigned done;
-    asm volatile(
-        "{\n\t"
-        ".reg .pred p, q;\n\t"
-        ".reg .u32 n;\n\t"
-        "mov.u32 n, 0;\n\t"
-        "SWLM_TRY:\n\t"
-        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "@p bra SWLM_DONE;\n\t"
-        "add.u32 n, n, 1;\n\t"
-        "setp.lt.u32 q, n, %3;\n\t"
-        "@q bra SWLM_TRY;\n\t"
-        "SWLM_DONE:\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t"
-        "}"
-        : "=r"(done) : "r"(addr), "r"(parity), "r"((unsigned)kTcSpinLimit) : "memory");
-    return done != 0;
-}
-__device__ __forceinline__ bool mbar_wait(unsigned long long* bar, unsigned parity) { return mbar_wait_addr(smem_u32(bar), parity); }
-
-// Shared-memory matrix descriptor: K-major operand, 128-byte swizzle, rows of 128 bytes, 8-row groups 1024
-// bytes apart (stride byte offset); leading byte offset unused for this layout; descriptor version 1.
-__device__ __forceinline__ unsigned long long umma_desc(unsigned smem_addr) {
-    unsigned long long d = 0;
-    d |= (unsigned long long)((smem_addr & 0x3FFFFu) >> 4);
-    d |= (unsigned long long)(1024u >> 4) << 32;
-    d |= 1ull << 46;
-    d |= 2ull << 61;
-    return d;
-}
-
 // Instruction descriptor for kind::f16: D = fp32, A = B = fp16 (format 0), both K-major, M = 128, N = BN.
 __host__ __device__ constexpr unsigned umma_idesc(int bn) {
     return (1u << 4) | (0u << 7) | (0u << 10) | ((unsigned)(bn >> 3) << 17) | ((unsigned)(kTcRows >> 4) << 24);
@@ -118,10 +78,6 @@ __device__ __forceinline__ void umma_f16_ta(unsigned d_tmem, unsigned a_tmem, un
         "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
         ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
 }
-__device__ __forceinline__ void umma_commit(unsigned long long* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-
 // One result, rounded once to bf16, to the output its weight row belongs to.
 __device__ __forceinline__ void tc_store(const TcSegments& o, int token, int row, float val) {
     const int q = row < o.end[0] ? 0 : row < o.end[1] ? 1 : 2;
@@ -463,20 +419,6 @@ __global__ void __launch_bounds__(256) x_to_f16_kernel(const __nv_bfloat16* x, i
 
 template <int BN, int STAGES>
 constexpr size_t tc_smem_bytes() { return (size_t)STAGES * (BN * 128 + kTcRows * 32) + 1024; }
-
-// cuTensorMapEncodeTiled, looked up through the runtime so that the library does not link against the driver
-typedef CUresult (*TensorMapEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                      const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                      CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-TensorMapEncodeFn tensor_map_encode_fn() {
-    static TensorMapEncodeFn fn = [] {
-        void* f = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &f, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) f = nullptr;
-        return reinterpret_cast<TensorMapEncodeFn>(f);
-    }();
-    return fn;
-}
 
 // fp16 activations X[m][x_stride] as a 2-D tensor (k innermost); box = 64 columns x bn tokens, 128-byte swizzle
 int make_x_map(const __half* x, int x_stride, int m, int k, int bn, CUtensorMap* map) {

@@ -15,7 +15,7 @@
 #include <algorithm>
 #include <cmath>
 
-#include "swlm_internal.h"
+#include "swlm_runtime.h"
 
 namespace swlm {
 
@@ -38,32 +38,9 @@ int cuda_fail(cudaError_t e, const char* what) {
 
 }  // namespace swlm
 
-using namespace swlm;
-
 // =====================================================================================================
 // Context + weight store
 // =====================================================================================================
-struct swlm_ctx {
-    int device = 0, tp_rank = 0, tp_size = 1;
-    cudaStream_t stream = nullptr;
-    std::map<std::string, Q4Raw> raw;
-    std::map<std::string, Q4Tiled> tiled;  // plain and fused tensors, keyed by name ("a|b|c" for fused)
-    std::map<std::string, Q4Raw> raw_cat;  // source-layout tensors with the rows of several raw tensors one after the other ("a|b|c")
-    std::map<std::string, DenseTensor> dense;
-    std::map<std::string, DenseF32> densef;   // fp32 tensors (recurrent layers' norm weight and A_log)
-    int64_t bytes = 0;
-    float* op_partial = nullptr; size_t op_partial_floats = 0;
-    unsigned char* op_xh = nullptr; size_t op_xh_bytes = 0;   // scratch of the op-level tensor-core product
-    unsigned* op_attn_counters = nullptr; size_t op_attn_counter_count = 0;
-    unsigned* op_counters = nullptr; size_t op_counter_count = 0;
-    int* tc_status = nullptr;  // device word the tcgen05 GEMM sets when one of its bounded waits expired
-    // Lifetime: plans keep their context alive, states their plan. A destroy call on an object that still has
-    // users only marks it; the memory goes when the last user is destroyed (hosts with garbage-collected
-    // wrappers release objects in no particular order).
-    int users = 0;
-    bool destroy_requested = false;
-};
-
 namespace {
 
 int ensure_device(const swlm_ctx* ctx) {
@@ -71,22 +48,13 @@ int ensure_device(const swlm_ctx* ctx) {
     return SWLM_OK;
 }
 
-template <typename T>
-int dev_alloc(T** p, size_t count, swlm_ctx* ctx = nullptr) {
-    *p = nullptr;
-    if (count == 0) return SWLM_OK;
-    SWLM_CUDA(cudaMalloc((void**)p, count * sizeof(T)));
-    if (ctx) ctx->bytes += (int64_t)(count * sizeof(T));
-    return SWLM_OK;
-}
-
 int alloc_tiled(swlm_ctx* ctx, int n, int k, bool sb_f16, Q4Tiled* t) {
     t->n = n; t->k = k; t->sb_f16 = sb_f16;
     t->row_tiles = (n + 15) / 16;
     t->kt_pad = ((k / 64 + 3) / 4) * 4;
-    int rc = dev_alloc(&t->tiles, (size_t)t->row_tiles * t->kt_pad * 32, ctx);
+    int rc = dev_alloc(&t->tiles, (size_t)t->row_tiles * t->kt_pad * 32, &ctx->bytes);
     if (rc) return rc;
-    return dev_alloc(&t->sb, (size_t)t->row_tiles * (t->kt_pad / 4) * 16, ctx);
+    return dev_alloc(&t->sb, (size_t)t->row_tiles * (t->kt_pad / 4) * 16, &ctx->bytes);
 }
 
 // Rank-local slice of a [rows][cols] matrix given in `unit`-sized column units.
@@ -201,9 +169,9 @@ int add_q4_raw(swlm_ctx* ctx, const char* name, int n, int k, const uint32_t* w,
     Q4Raw r;
     r.n = sl.rows * sl.parts; r.k = sl.cols; r.sb_f16 = f16; r.shard_kind = shard_kind;
     const int wpr = k / 8, gpr = k / 64, lw = sl.cols / 8, lg = sl.cols / 64;
-    if ((rc = dev_alloc(&r.w, (size_t)r.n * lw, ctx))) return rc;
-    if ((rc = dev_alloc(&r.scales, (size_t)r.n * lg, ctx))) return rc;
-    if ((rc = dev_alloc(&r.biases, (size_t)r.n * lg, ctx))) return rc;
+    if ((rc = dev_alloc(&r.w, (size_t)r.n * lw, &ctx->bytes))) return rc;
+    if ((rc = dev_alloc(&r.scales, (size_t)r.n * lg, &ctx->bytes))) return rc;
+    if ((rc = dev_alloc(&r.biases, (size_t)r.n * lg, &ctx->bytes))) return rc;
     for (int part = 0; part < sl.parts; ++part) {
         const size_t src_row = (size_t)part * sl.part_stride + sl.row0, dst_row = (size_t)part * sl.rows;
         SWLM_CUDA(cudaMemcpy2D(r.w + dst_row * lw, (size_t)lw * 4, w + src_row * wpr + sl.col0 / 8, (size_t)wpr * 4, (size_t)lw * 4, sl.rows, cudaMemcpyHostToDevice));
@@ -219,62 +187,6 @@ int add_q4_raw(swlm_ctx* ctx, const char* name, int n, int k, const uint32_t* w,
 // =====================================================================================================
 // Plan
 // =====================================================================================================
-namespace {
-
-enum LaunchKind { L_EMBED, L_RMSNORM, L_QGEMV, L_QK_NORM, L_ATTN, L_SWIGLU, L_CONV, L_ARGMAX, L_SSM };
-
-struct Launch {
-    int kind = 0;
-    swlm_step st{};            // the (first) step this launch came from
-    const Q4Tiled* w = nullptr;
-    std::vector<std::string> w_names;
-    int w_mode = 0;
-    int epilogue = QGEMV_EPI_STORE;
-    int gated_act = GATED_ACT_SILU;
-    int n_seg = 1;
-    int seg_buf[3] = {-1, -1, -1};
-    int seg_end[3] = {0, 0, 0};
-    const DenseTensor* d1 = nullptr;
-    const DenseTensor* d2 = nullptr;
-    const Q4Raw* q_embed = nullptr;  // embedding step over a quantized table
-    const DenseF32* f1 = nullptr;    // recurrent step: norm weight, A_log (d1 = conv taps, d2 = dt_bias)
-    const DenseF32* f2 = nullptr;
-    int rope_table = -1;       // index into plan->rope_tables
-    std::string label;
-    int steps_covered = 1;
-    // residual add / copy / RMSNorm folded into this product's prologue (norm.kind == 0: none)
-    swlm_step norm{};
-    const DenseTensor* norm_w = nullptr;
-    int x_buf = -1;            // buffer the product reads (the norm's input when fused)
-    int push = 0, in_tp = 0;   // tensor parallel: partial rows pushed to all ranks / pushed partials consumed
-    int res_in = 0, res_out = 0;  // physical residual buffers (0 or 1) this launch reads / writes
-    int prefetch_launch = -1;     // index of the later product whose weights this launch pulls into L2
-    int kv_prefetch_attn = -1;    // index of the attention launch whose K/V rows this product pulls into L2
-};
-
-struct RopeTable { int rope_dim; float base; float* inv_freq; };
-
-}  // namespace
-
-struct swlm_plan {
-    swlm_ctx* ctx = nullptr;
-    swlm_buffers_desc desc{};
-    std::vector<swlm_step> steps;
-    std::vector<Launch> launches;
-    std::vector<RopeTable> rope_tables;
-    int attn_splits = 1;
-    size_t attn_scratch = 0, qgemv_partial = 0, qgemv_counters = 0;
-    int final_res = 0;  // physical residual buffer that holds the residual stream after a step
-    // Row-wise execution (prompt chunks, more than 16 sequences): consecutive products of one input run as one product
-    // over their concatenated rows. Per step: how many steps the product starting there covers (0: covered by an
-    // earlier one) and the tensor it multiplies.
-    struct RowsGroup { int count = 1; const Q4Raw* raw = nullptr; };
-    std::vector<RowsGroup> rows_groups;
-    bool rows_groups_ready = false;
-    int users = 0;
-    bool destroy_requested = false;
-};
-
 namespace {
 
 int buf_width(const swlm_buffers_desc& d, int buf) {
@@ -312,6 +224,7 @@ int compile_plan(swlm_plan* plan) {
     const std::vector<swlm_step>& st = plan->steps;
     const int m = d.max_batch;
     int rc;
+    if (plan->stream()) return stream_compile(plan);
     for (size_t i = 0; i < st.size();) {
         const swlm_step& s = st[i];
         Launch L;
@@ -609,58 +522,6 @@ int compile_plan(swlm_plan* plan) {
 // =====================================================================================================
 // State
 // =====================================================================================================
-struct swlm_state {
-    swlm_plan* plan = nullptr;
-    cudaStream_t own_stream = nullptr, stream = nullptr;
-    __nv_bfloat16* buf[SWLM_BUF_COUNT] = {};
-    int width[SWLM_BUF_COUNT] = {};
-    __nv_bfloat16* kcache = nullptr; __nv_bfloat16* vcache = nullptr; size_t kv_layer_elems = 0;
-    // rotated KV schemes: rotors [kv_layers][kv_heads][groups][4], projection matrix [head_dim][qjl_dim], projected K
-    // residuals [kv_layers][seq][kv_heads][max_seq][qjl_dim], all fp16
-    __half* rotors = nullptr; size_t rotor_layer_elems = 0;
-    __half* qjl_matrix = nullptr;
-    __half* qjl_res = nullptr; size_t qjl_layer_elems = 0;
-    std::vector<uint16_t> rotors_host, qjl_matrix_host;   // host copies for the cache probes
-    __nv_bfloat16* conv = nullptr; size_t conv_layer_elems = 0;
-    __nv_bfloat16* ssm_conv = nullptr; size_t ssm_conv_layer_elems = 0;   // [layer][seq][kernel][conv_dim]
-    float* ssm_state = nullptr; size_t ssm_state_layer_elems = 0;         // [layer][seq][heads][key_dim][value_dim]
-    int32_t* position = nullptr; int32_t* step_counter = nullptr;
-    int32_t* token_in = nullptr; int32_t* token_out = nullptr; int32_t* ring = nullptr;
-    int32_t* prompt = nullptr; size_t prompt_cap = 0;
-    int ring_cap = 4096;
-    float* attn_scratch = nullptr; float* qgemv_partial = nullptr; unsigned* qgemv_counters = nullptr;
-    size_t attn_scratch_cap = 0, qgemv_partial_cap = 0, qgemv_counters_cap = 0;
-    unsigned* attn_counters = nullptr;
-    float* argmax_val = nullptr; int32_t* argmax_idx = nullptr;
-    __nv_bfloat16* res2 = nullptr;  // second physical residual buffer (ping-pong partner of buf[RESIDUAL])
-    // tensor-parallel exchange (tp_size > 1): this rank's buffer, the peers' mappings, local counters
-    TpParams tp{};
-    bool tp_attached = false;
-    int32_t* tp_words = nullptr;  // [0] all-reduce epoch, [1] rows-done counter, [2] status, [3] argmax epoch, [4] CTAs done pushing a prompt chunk
-    int tp_rows_epoch = 0;        // prompt-chunk exchanges issued so far (the same count on every rank)
-    int32_t* h_tok = nullptr;  // pinned host staging, 2 * max_batch
-    std::vector<int> pos_host;   // host mirror of the per-sequence positions
-    long long steps_host = 0;
-    cudaGraphExec_t graph_full = nullptr, graph_body = nullptr;
-    int graph_full_launches = 0, graph_body_launches = 0;
-    int64_t launches = 0;
-    // prompt ingestion in chunks: activation rows for `pf_rows` tokens per logical buffer, attention scratch
-    __nv_bfloat16* pf_buf[SWLM_BUF_COUNT] = {};
-    int pf_rows = 0;
-    unsigned* pf_attn_counters = nullptr;
-    unsigned char* wide_xh = nullptr;  // the same for a decode step of more than kQGemvMaxRows sequences
-    unsigned char* pf_xh = nullptr;  // scratch of the tensor-core product: fp16 copy of a chunk's widest activations
-    int* pf_status = nullptr;      // device word: a bounded wait of the tensor-core product expired
-    int prefill_chunk = 2048;      // tokens per chunk; 0 = one token at a time through the decode graph
-    int* tc_status = nullptr;      // pinned host word (mapped): a bounded wait of a kernel expired
-};
-
-struct swlm_snap {
-    std::vector<void*> dev;
-    std::vector<size_t> bytes;
-    std::vector<int> pos_host;
-};
-
 namespace {
 
 // ---- rotated KV schemes on the host: parameters by the reference's rule, and the arithmetic of the cache probes ----
@@ -752,6 +613,7 @@ int enqueue_step(swlm_state* s, bool body_only, cudaStream_t stream, int only_ki
     const size_t n_launch = plan->launches.size();
     // the output head is the trailing [norm, lm_head, argmax] group
     (void)n_launch;
+    if (plan->stream()) return stream_enqueue_step(s, body_only, stream, only_kind);
     if (m > kQGemvMaxRows) {
         if (only_kind >= 0) { set_error("per-kind timing is for plans of up to %d sequences", kQGemvMaxRows); return SWLM_ERR_UNSUPPORTED; }
         return enqueue_rows(s, true, s->token_in, m, 0, 0, -1, body_only, stream);
@@ -907,6 +769,7 @@ int capture_graph(swlm_state* s, bool body_only, cudaGraphExec_t* out) {
 int launches_per_step(const swlm_plan* plan, bool body_only) {
     int n = 0;
     bool has_argmax = false;
+    if (plan->stream()) return stream_launches_per_step(plan);
     if (plan->desc.max_batch > kQGemvMaxRows) {
         // more than 16 sequences: the unfused steps, as enqueue_rows issues them
         int converted_buf = -1, converted_k = 0;
@@ -962,18 +825,20 @@ int run_graph(swlm_state* s, bool body_only) {
 void drop_graphs(swlm_state* s) {
     if (s->graph_full) { cudaGraphExecDestroy(s->graph_full); s->graph_full = nullptr; }
     if (s->graph_body) { cudaGraphExecDestroy(s->graph_body); s->graph_body = nullptr; }
+    stream_drop_graphs(s);
 }
 
 struct Region { void* p; size_t bytes; };
 std::vector<Region> state_regions(swlm_state* s) {
     const swlm_buffers_desc& d = s->plan->desc;
     std::vector<Region> r;
-    for (int i = 0; i < SWLM_BUF_COUNT; ++i) r.push_back({s->buf[i], (size_t)d.max_batch * s->width[i] * 2});
+    for (size_t l = 0; l < s->pool.size(); ++l) r.push_back({s->pool[l], s->pool_bytes[l]});
+    for (int i = 0; i < SWLM_BUF_COUNT && !s->plan->stream(); ++i) r.push_back({s->buf[i], (size_t)d.max_batch * s->width[i] * 2});
     r.push_back({s->kcache, (size_t)d.kv_layers * s->kv_layer_elems * 2});
     r.push_back({s->vcache, (size_t)d.kv_layers * s->kv_layer_elems * 2});
     r.push_back({s->qjl_res, (size_t)d.kv_layers * s->qjl_layer_elems * 2});
     r.push_back({s->conv, (size_t)d.conv_layers * s->conv_layer_elems * 2});
-    r.push_back({s->res2, (size_t)d.max_batch * s->width[SWLM_BUF_RESIDUAL] * 2});
+    if (!s->plan->stream()) r.push_back({s->res2, (size_t)d.max_batch * s->width[SWLM_BUF_RESIDUAL] * 2});
     r.push_back({s->ssm_conv, (size_t)d.ssm_layers * s->ssm_conv_layer_elems * 2});
     r.push_back({s->ssm_state, (size_t)d.ssm_layers * s->ssm_state_layer_elems * 4});
     r.push_back({s->position, (size_t)d.max_batch * 4});
@@ -1033,6 +898,12 @@ int check_position_room(swlm_state* s, int steps) {
         set_error("position %d + %d steps exceeds max_seq %d", furthest, steps, s->plan->desc.max_seq);
         return SWLM_ERR_STATE;
     }
+    if (s->plan->stream()) {   // every sequence decodes: all of them take the pages the steps will fill
+        int rc;
+        for (size_t b = 0; b < s->pos_host.size(); ++b)
+            if ((rc = stream_reserve(s, (int)b, s->pos_host[b] + steps))) return rc;
+        return stream_upload_pages(s);
+    }
     return SWLM_OK;
 }
 
@@ -1059,9 +930,9 @@ int get_raw_cat(swlm_ctx* ctx, const std::vector<std::string>& names, const Q4Ra
     for (const std::string& nm : names) cat.n += ctx->raw.at(nm).n;
     const size_t wpr = (size_t)cat.k / 8, gpr = (size_t)cat.k / 64;
     int rc;
-    if ((rc = dev_alloc(&cat.w, (size_t)cat.n * wpr, ctx))) return rc;
-    if ((rc = dev_alloc(&cat.scales, (size_t)cat.n * gpr, ctx))) return rc;
-    if ((rc = dev_alloc(&cat.biases, (size_t)cat.n * gpr, ctx))) return rc;
+    if ((rc = dev_alloc(&cat.w, (size_t)cat.n * wpr, &ctx->bytes))) return rc;
+    if ((rc = dev_alloc(&cat.scales, (size_t)cat.n * gpr, &ctx->bytes))) return rc;
+    if ((rc = dev_alloc(&cat.biases, (size_t)cat.n * gpr, &ctx->bytes))) return rc;
     size_t row = 0;
     for (const std::string& nm : names) {
         const Q4Raw& r = ctx->raw.at(nm);
@@ -1414,6 +1285,8 @@ int swlm_ctx_create(int device_id, int tp_rank, int tp_size, swlm_ctx** out) {
     int rc = qgemv_init();
     if (!rc) rc = attn_init();
     if (!rc) rc = qgemm_tc_init();
+    if (!rc) rc = bgemm_init();
+    if (!rc) rc = latent_init();
     if (rc) { cudaStreamDestroy(ctx->stream); delete ctx; return rc; }
     *out = ctx;
     return SWLM_OK;
@@ -1429,6 +1302,8 @@ void swlm_ctx_destroy(swlm_ctx* ctx) {
     for (auto& kv : ctx->raw_cat) { cudaFree(kv.second.w); cudaFree(kv.second.scales); cudaFree(kv.second.biases); }
     for (auto& kv : ctx->dense) cudaFree(kv.second.data);
     for (auto& kv : ctx->densef) cudaFree(kv.second.data);
+    for (auto& kv : ctx->matrices) if (!kv.second.view) cudaFree(kv.second.data);
+    for (auto& kv : ctx->matrix_cat) cudaFree(kv.second.data);
     cudaFree(ctx->op_partial);
     cudaFree(ctx->tc_status);
     cudaFree(ctx->op_xh);
@@ -1503,7 +1378,7 @@ int swlm_weights_add_dense_bf16(swlm_ctx* ctx, const char* name, int64_t rows, i
     }
     DenseTensor t;
     t.rows = sl.rows; t.cols = cols; t.shard_kind = shard_kind;
-    if ((rc = dev_alloc(&t.data, (size_t)t.rows * cols, ctx))) return rc;
+    if ((rc = dev_alloc(&t.data, (size_t)t.rows * cols, &ctx->bytes))) return rc;
     SWLM_CUDA(cudaMemcpy(t.data, data + (size_t)sl.row0 * cols, (size_t)t.rows * cols * 2, cudaMemcpyHostToDevice));
     ctx->dense[name] = t;
     return SWLM_OK;
@@ -1521,9 +1396,31 @@ int swlm_weights_add_dense_f32(swlm_ctx* ctx, const char* name, int64_t count, c
     }
     DenseF32 t;
     t.count = count;
-    if ((rc = dev_alloc(&t.data, (size_t)count, ctx))) return rc;
+    if ((rc = dev_alloc(&t.data, (size_t)count, &ctx->bytes))) return rc;
     SWLM_CUDA(cudaMemcpy(t.data, data, (size_t)count * 4, cudaMemcpyHostToDevice));
     ctx->densef[name] = t;
+    return SWLM_OK;
+}
+
+int swlm_weights_add_matrix_bf16(swlm_ctx* ctx, const char* name, int n, int k, const uint16_t* data) {
+    if (!ctx || !name || !data || n <= 0 || k <= 0) { set_error("bad matrix"); return SWLM_ERR_INVALID; }
+    int rc = ensure_device(ctx);
+    if (rc) return rc;
+    Matrix& m = ctx->matrices[name];
+    if (m.data && (m.n != n || m.k != k)) {
+        if (m.view) { set_error("matrix '%s' is part of a plan's concatenated matrix and cannot change its shape", name); return SWLM_ERR_STATE; }
+        SWLM_CUDA(cudaDeviceSynchronize());
+        cudaFree(m.data);
+        ctx->bytes -= (int64_t)m.n * m.ld * 2;
+        m = Matrix{};
+    }
+    if (!m.data) {
+        m.n = n; m.k = k; m.ld = (k + 7) / 8 * 8;
+        if ((rc = dev_alloc(&m.data, (size_t)n * m.ld, &ctx->bytes))) { ctx->matrices.erase(name); return rc; }
+        if (m.ld != k) SWLM_CUDA(cudaMemset(m.data, 0, (size_t)n * m.ld * 2));
+    }
+    SWLM_CUDA(cudaDeviceSynchronize());
+    SWLM_CUDA(cudaMemcpy2D(m.data, (size_t)m.ld * 2, data, (size_t)k * 2, (size_t)k * 2, n, cudaMemcpyHostToDevice));
     return SWLM_OK;
 }
 
@@ -1551,7 +1448,12 @@ int swlm_plan_build(swlm_ctx* ctx, const swlm_step* steps, int n_steps, const sw
     }
     if (desc->max_batch < 1 || desc->max_batch > kMaxSequences) { set_error("max_batch %d outside 1..%d", desc->max_batch, kMaxSequences); return SWLM_ERR_INVALID; }
     if (desc->max_batch > kQGemvMaxRows && ctx->tp_size > 1) { set_error("more than %d sequences per step are not supported under tensor parallelism", kQGemvMaxRows); return SWLM_ERR_UNSUPPORTED; }
-    if (desc->hidden % 8 || desc->slot_dim % 8 || desc->vocab % 8) { set_error("hidden, slot_dim and vocab must be multiples of 8"); return SWLM_ERR_INVALID; }
+    const bool stream = desc->stream_dtype != 0;
+    if (stream && (desc->max_seq < 1 || desc->hidden < 1 || desc->vocab < 1 || desc->latent_layers < 0 || desc->kv_pool_tokens < 0 || desc->kv_layers || desc->conv_layers || desc->ssm_layers)) {
+        set_error("fp32-stream plan: bad sizes, or layers with bf16 state");
+        return SWLM_ERR_INVALID;
+    }
+    if (!stream && (desc->hidden % 8 || desc->slot_dim % 8 || desc->vocab % 8)) { set_error("hidden, slot_dim and vocab must be multiples of 8"); return SWLM_ERR_INVALID; }
     int rc = ensure_device(ctx);
     if (rc) return rc;
     swlm_plan* plan = new swlm_plan();
@@ -1562,7 +1464,7 @@ int swlm_plan_build(swlm_ctx* ctx, const swlm_step* steps, int n_steps, const sw
     rc = compile_plan(plan);
     // Row-wise execution (prompt chunks; more than 16 sequences, inside a CUDA graph): build the concatenated tensors
     // now, not inside the first prompt's latency and not while a stream is capturing.
-    if (!rc && (desc->max_batch > kQGemvMaxRows || rows_capable(plan, true))) rc = ensure_rows_groups(plan);
+    if (!rc && !stream && (desc->max_batch > kQGemvMaxRows || rows_capable(plan, true))) rc = ensure_rows_groups(plan);
     if (rc) { swlm_plan_destroy(plan); return rc; }
     plan->attn_scratch = plan_attn_scratch(plan);
     *out = plan;
@@ -1612,7 +1514,7 @@ int swlm_state_create(swlm_plan* plan, swlm_state** out) {
     cudaError_t e = cudaStreamCreateWithFlags(&s->own_stream, cudaStreamNonBlocking);
     if (e != cudaSuccess) return fail(cuda_fail(e, "cudaStreamCreate"));
     s->stream = s->own_stream;
-    for (int i = 0; i < SWLM_BUF_COUNT; ++i) {
+    for (int i = 0; i < SWLM_BUF_COUNT && !plan->stream(); ++i) {
         s->width[i] = buf_width(d, i);
         if ((rc = dev_alloc(&s->buf[i], (size_t)d.max_batch * s->width[i]))) return fail(rc);
     }
@@ -1642,7 +1544,7 @@ int swlm_state_create(swlm_plan* plan, swlm_state** out) {
     }
     s->conv_layer_elems = (size_t)d.max_batch * d.conv_kernel * d.conv_dim;
     if ((rc = dev_alloc(&s->conv, (size_t)d.conv_layers * s->conv_layer_elems))) return fail(rc);
-    if ((rc = dev_alloc(&s->res2, (size_t)d.max_batch * s->width[SWLM_BUF_RESIDUAL]))) return fail(rc);
+    if (!plan->stream() && (rc = dev_alloc(&s->res2, (size_t)d.max_batch * s->width[SWLM_BUF_RESIDUAL]))) return fail(rc);
     if (d.ssm_layers > 0) {
         const size_t ssm_conv_dim = (size_t)2 * std::max(1, d.ssm_groups) * d.ssm_key_dim + (size_t)d.ssm_heads * d.ssm_value_dim;
         s->ssm_conv_layer_elems = (size_t)d.max_batch * d.ssm_conv_kernel * ssm_conv_dim;
@@ -1662,7 +1564,7 @@ int swlm_state_create(swlm_plan* plan, swlm_state** out) {
         cudaError_t ce = cudaMemset(s->attn_counters, 0, (size_t)d.max_batch * std::max(1, d.kv_heads) * sizeof(unsigned));
         if (ce != cudaSuccess) return fail(cuda_fail(ce, "cudaMemset"));
     }
-    if (d.max_batch > kQGemvMaxRows) {
+    if (d.max_batch > kQGemvMaxRows && !plan->stream()) {
         if ((rc = ensure_pf_status(s))) return fail(rc);
         if ((rc = dev_alloc(&s->wide_xh, qgemm_tc_scratch_bytes(d.max_batch, widest_activation(s))))) return fail(rc);
     }
@@ -1674,6 +1576,7 @@ int swlm_state_create(swlm_plan* plan, swlm_state** out) {
     e = cudaHostAlloc((void**)&s->tc_status, sizeof(int), cudaHostAllocMapped);
     if (e != cudaSuccess) return fail(cuda_fail(e, "cudaHostAlloc"));
     *s->tc_status = 0;
+    if (plan->stream() && (rc = stream_state_create(s))) return fail(rc);
     *out = s;
     rc = swlm_state_reset(s);
     if (rc) { *out = nullptr; return fail(rc); }
@@ -1685,6 +1588,7 @@ void swlm_state_destroy(swlm_state* s) {
     cudaSetDevice(s->plan->ctx->device);
     if (s->stream) cudaStreamSynchronize(s->stream);
     drop_graphs(s);
+    stream_state_free(s);
     for (int i = 0; i < SWLM_BUF_COUNT; ++i) cudaFree(s->buf[i]);
     cudaFree(s->kcache); cudaFree(s->vcache); cudaFree(s->conv); cudaFree(s->res2);
     cudaFree(s->rotors); cudaFree(s->qjl_matrix); cudaFree(s->qjl_res);
@@ -1726,6 +1630,7 @@ int swlm_state_reset(swlm_state* s) {
     SWLM_CUDA(cudaMemsetAsync(s->step_counter, 0, 4, s->stream));
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
     std::fill(s->pos_host.begin(), s->pos_host.end(), 0);
+    if (s->plan->stream()) stream_release_all(s);
     s->steps_host = 0;
     return SWLM_OK;
 }
@@ -1748,6 +1653,8 @@ int swlm_state_snapshot(swlm_state* s, swlm_snap** out) {
         snap->bytes.push_back(r.bytes);
     }
     snap->pos_host = s->pos_host;
+    snap->seq_pages = s->seq_pages;
+    snap->free_pages = s->free_pages;
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
     *out = snap;
     return SWLM_OK;
@@ -1763,6 +1670,11 @@ int swlm_state_restore(swlm_state* s, const swlm_snap* snap) {
     }
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
     s->pos_host = snap->pos_host;
+    s->seq_pages = snap->seq_pages;
+    s->free_pages = snap->free_pages;
+    for (size_t b = 0; b < s->seq_pages.size(); ++b)
+        std::copy(s->seq_pages[b].begin(), s->seq_pages[b].end(), s->page_table_host.begin() + b * s->pages_per_seq);
+    s->page_table_dirty = s->plan->stream();
     return SWLM_OK;
 }
 
@@ -1785,6 +1697,14 @@ int swlm_set_positions(swlm_state* s, const int32_t* positions) {
     const int m = s->plan->desc.max_batch;
     for (int b = 0; b < m; ++b)
         if (positions[b] < 0 || positions[b] > s->plan->desc.max_seq) { set_error("bad position %d of sequence %d", positions[b], b); return SWLM_ERR_INVALID; }
+    if (s->plan->stream()) {   // pages first given back, then taken
+        int rc;
+        for (int b = 0; b < m; ++b)
+            if (positions[b] < s->pos_host[b] && (rc = stream_reserve(s, b, positions[b], true))) return rc;
+        for (int b = 0; b < m; ++b)
+            if ((rc = stream_reserve(s, b, positions[b]))) return rc;
+        if ((rc = stream_upload_pages(s))) return rc;
+    }
     SWLM_CUDA(cudaMemcpyAsync(s->position, positions, sizeof(int32_t) * m, cudaMemcpyHostToDevice, s->stream));
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
     s->pos_host.assign(positions, positions + m);
@@ -1871,6 +1791,15 @@ int swlm_prefill(swlm_state* s, const int32_t* tokens, int n, int32_t* first_tok
     int rc = ensure_device(s->plan->ctx);
     if (!rc) rc = check_position_room(s, n);
     if (rc) return rc;
+    if (s->plan->stream()) {
+        if (n > s->plan->desc.max_seq) { set_error("a prompt of %d tokens exceeds max_seq", n); return SWLM_ERR_STATE; }
+        std::vector<int32_t> seqs(m), counts(m, n), ones(m, 1), last(m, n - 1);
+        for (int b = 0; b < m; ++b) seqs[b] = b;
+        rc = stream_run(s, m, seqs.data(), counts.data(), tokens, ones.data(), last.data(), nullptr, first_token, s->prefill_chunk > 0 ? s->prefill_chunk : 2048);
+        if (rc) { for (int b = 0; b < m; ++b) first_token[b] = -1; return rc; }
+        SWLM_CUDA(cudaMemcpy(s->token_in, first_token, sizeof(int32_t) * m, cudaMemcpyHostToDevice));
+        return SWLM_OK;
+    }
     // several sequences with prompts long enough for chunks: one sequence after the other through the row-wise path
     if (m > 1 && n >= kPrefillMinChunk && s->prefill_chunk >= kPrefillMinChunk && rows_capable(s->plan)) {
         for (int b = 0; b < m; ++b)
@@ -1929,6 +1858,14 @@ int swlm_prefill_seq(swlm_state* s, int seq, const int32_t* tokens, int n, int32
     *first_token = -1;
     const swlm_buffers_desc& d = s->plan->desc;
     if (seq < 0 || seq >= d.max_batch) { set_error("sequence %d outside 0..%d", seq, d.max_batch - 1); return SWLM_ERR_INVALID; }
+    if (s->plan->stream()) {
+        const int32_t q = seq, c = n, one = 1, last = n - 1;
+        int rc = ensure_device(s->plan->ctx);
+        if (!rc) rc = stream_run(s, 1, &q, &c, tokens, &one, &last, nullptr, first_token, s->prefill_chunk > 0 ? s->prefill_chunk : 2048);
+        if (rc) { *first_token = -1; return rc; }
+        SWLM_CUDA(cudaMemcpy(s->token_in + seq, first_token, sizeof(int32_t), cudaMemcpyHostToDevice));
+        return SWLM_OK;
+    }
     if (!rows_capable(s->plan)) { set_error("this plan cannot ingest a prompt into one sequence (tensor parallel, head_dim > 128 or an in-place product)"); return SWLM_ERR_UNSUPPORTED; }
     int rc = ensure_device(s->plan->ctx);
     if (rc) return rc;
@@ -1977,6 +1914,7 @@ int swlm_state_reset_seq(swlm_state* s, int seq) {
     }
     SWLM_CUDA(cudaMemsetAsync(s->position + seq, 0, 4, s->stream));
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    if (s->plan->stream() && (rc = stream_reserve(s, seq, 0, true))) return rc;   // its pages go back to the pool
     s->pos_host[seq] = 0;
     return SWLM_OK;
 }
@@ -1988,6 +1926,7 @@ int swlm_state_set_prefill_chunk(swlm_state* s, int tokens) {
 }
 
 int swlm_read_buffer(swlm_state* s, int buf, uint16_t* dst, int count_per_row) {
+    if (s && s->plan->stream()) { set_error("this plan keeps fp32 buffers: use the _f32 form"); return SWLM_ERR_UNSUPPORTED; }
     if (!s || !dst || !buf_ok(buf) || count_per_row > s->width[buf]) { set_error("bad buffer read"); return SWLM_ERR_INVALID; }
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
     // the residual stream ends a step in whichever of its two physical buffers the plan wrote last
@@ -1998,6 +1937,7 @@ int swlm_read_buffer(swlm_state* s, int buf, uint16_t* dst, int count_per_row) {
 }
 
 int swlm_write_buffer(swlm_state* s, int buf, const uint16_t* src, int count_per_row) {
+    if (s && s->plan->stream()) { set_error("this plan keeps fp32 buffers: use the _f32 form"); return SWLM_ERR_UNSUPPORTED; }
     if (!s || !src || !buf_ok(buf) || count_per_row > s->width[buf]) { set_error("bad buffer write"); return SWLM_ERR_INVALID; }
     SWLM_CUDA(cudaStreamSynchronize(s->stream));
     SWLM_CUDA(cudaMemcpy2D(s->buf[buf], (size_t)s->width[buf] * 2, src, (size_t)count_per_row * 2, (size_t)count_per_row * 2,
@@ -2174,6 +2114,7 @@ int swlm_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_in,
     const int m = s->plan->desc.max_batch;
     int rc = ensure_device(s->plan->ctx);
     if (rc) return rc;
+    if (s->plan->stream()) return stream_run_step(s, step, token_in, token_out);
     // compile a one-step plan against the same weight store and buffer set, run it eagerly
     swlm_plan tmp;
     tmp.ctx = s->plan->ctx;
@@ -2200,6 +2141,81 @@ int swlm_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_in,
     const int32_t saved_steps = (int32_t)s->steps_host;
     SWLM_CUDA(cudaMemcpy(s->step_counter, &saved_steps, 4, cudaMemcpyHostToDevice));
     if (token_out) SWLM_CUDA(cudaMemcpy(token_out, s->token_out, sizeof(int32_t) * m, cudaMemcpyDeviceToHost));
+    return SWLM_OK;
+}
+
+int swlm_run_batch(swlm_state* s, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens,
+                   const int32_t* want_counts, const int32_t* wants, float* logits_out, int32_t* tokens_out) {
+    if (!s || n_entries < 0 || (n_entries > 0 && (!seqs || !counts || !tokens)) || (want_counts && !wants)) { set_error("bad argument"); return SWLM_ERR_INVALID; }
+    if (!s->plan->stream()) { set_error("batches of unequal portions are for fp32-stream plans"); return SWLM_ERR_UNSUPPORTED; }
+    if (n_entries == 0) return SWLM_OK;
+    int rc = ensure_device(s->plan->ctx);
+    if (rc) return rc;
+    constexpr int kBatchRows = 8192;   // rows that run together; more are cut into several passes
+    return stream_run(s, n_entries, seqs, counts, tokens, want_counts, wants, logits_out, tokens_out, kBatchRows);
+}
+
+int swlm_pool_free_pages(const swlm_state* s) { return s && s->plan->stream() ? (int)s->free_pages.size() : -1; }
+
+static bool stream_buf_f32(const swlm_plan* plan, int buf) {
+    return plan->all_f32() || buf == SWLM_BUF_HIDDEN || buf == SWLM_BUF_RESIDUAL || buf == SWLM_BUF_SCRATCH3 || buf == SWLM_BUF_SCRATCH4 || buf == SWLM_BUF_LOGITS;
+}
+int swlm_read_buffer_f32(swlm_state* s, int buf, int rows, int count_per_row, float* dst) {
+    if (!s || !dst || !s->plan->stream()) { set_error("fp32 probes are for fp32-stream plans"); return SWLM_ERR_INVALID; }
+    const StreamBufs& b = *s->last_bufs;
+    if (!buf_ok(buf) || rows < 0 || rows > (buf == SWLM_BUF_LOGITS ? b.wants : b.rows) || count_per_row < 0 || count_per_row > s->width[buf]) { set_error("bad buffer read"); return SWLM_ERR_INVALID; }
+    SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    const void* src = buf == SWLM_BUF_RESIDUAL && s->last_res ? b.res2 : b.buf[buf];
+    if (stream_buf_f32(s->plan, buf)) {
+        SWLM_CUDA(cudaMemcpy2D(dst, (size_t)count_per_row * 4, src, (size_t)s->width[buf] * 4, (size_t)count_per_row * 4, rows, cudaMemcpyDeviceToHost));
+        return SWLM_OK;
+    }
+    std::vector<uint16_t> h((size_t)rows * count_per_row);
+    SWLM_CUDA(cudaMemcpy2D(h.data(), (size_t)count_per_row * 2, src, (size_t)s->width[buf] * 2, (size_t)count_per_row * 2, rows, cudaMemcpyDeviceToHost));
+    for (size_t i = 0; i < h.size(); ++i) dst[i] = bf16_bits_to_float(h[i]);
+    return SWLM_OK;
+}
+int swlm_write_buffer_f32(swlm_state* s, int buf, int rows, int count_per_row, const float* src) {
+    if (!s || !src || !s->plan->stream()) { set_error("fp32 probes are for fp32-stream plans"); return SWLM_ERR_INVALID; }
+    const StreamBufs& b = s->dec;
+    if (!buf_ok(buf) || rows < 0 || rows > (buf == SWLM_BUF_LOGITS ? b.wants : b.rows) || count_per_row < 0 || count_per_row > s->width[buf]) { set_error("bad buffer write"); return SWLM_ERR_INVALID; }
+    SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    const bool f32 = stream_buf_f32(s->plan, buf);
+    std::vector<uint16_t> h;
+    if (!f32) { h.resize((size_t)rows * count_per_row); for (size_t i = 0; i < h.size(); ++i) h[i] = float_to_bf16_bits(src[i]); }
+    const size_t e = f32 ? 4 : 2;
+    const void* from = f32 ? static_cast<const void*>(src) : h.data();
+    SWLM_CUDA(cudaMemcpy2D(b.buf[buf], (size_t)s->width[buf] * e, from, (size_t)count_per_row * e, (size_t)count_per_row * e, rows, cudaMemcpyHostToDevice));
+    if (buf == SWLM_BUF_RESIDUAL) SWLM_CUDA(cudaMemcpy2D(b.res2, (size_t)s->width[buf] * e, from, (size_t)count_per_row * e, (size_t)count_per_row * e, rows, cudaMemcpyHostToDevice));
+    return SWLM_OK;
+}
+int swlm_read_logits_f32(swlm_state* s, float* dst, size_t count) {
+    if (!s || !dst || !s->plan->stream() || count != (size_t)s->plan->desc.max_batch * s->plan->desc.vocab) { set_error("fp32 logits are [max_batch][vocab] of an fp32-stream plan"); return SWLM_ERR_INVALID; }
+    SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    const int v = s->plan->desc.vocab;
+    SWLM_CUDA(cudaMemcpy2D(dst, (size_t)v * 4, s->dec.buf[SWLM_BUF_LOGITS], (size_t)s->width[SWLM_BUF_LOGITS] * 4, (size_t)v * 4, s->plan->desc.max_batch, cudaMemcpyDeviceToHost));
+    return SWLM_OK;
+}
+int swlm_read_latent(swlm_state* s, int layer, int seq, int count, float* dst) {
+    if (!s || !dst || !s->plan->stream()) { set_error("latent rows belong to fp32-stream plans"); return SWLM_ERR_INVALID; }
+    const swlm_buffers_desc& d = s->plan->desc;
+    if (layer < 0 || layer >= d.latent_layers || seq < 0 || seq >= d.max_batch || count < 0 || (size_t)count > s->seq_pages[seq].size() * SWLM_PAGE_TOKENS) { set_error("bad latent address"); return SWLM_ERR_INVALID; }
+    SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    const LatentLayer& l = s->plan->latent[layer];
+    const size_t e = s->plan->all_f32() ? 4 : 2, row = (size_t)l.row.pitch * e;
+    std::vector<unsigned char> page(row * SWLM_PAGE_TOKENS);
+    for (int t = 0; t < count; ++t) {
+        if (t % SWLM_PAGE_TOKENS == 0)
+            SWLM_CUDA(cudaMemcpy(page.data(), static_cast<unsigned char*>(s->pool[layer]) + (size_t)s->seq_pages[seq][t / SWLM_PAGE_TOKENS] * page.size(), page.size(), cudaMemcpyDeviceToHost));
+        const unsigned char* r = page.data() + (size_t)(t % SWLM_PAGE_TOKENS) * row;
+        for (int i = 0; i < l.rank + l.rot; ++i) {
+            const int at = i < l.rank ? i : l.row.rp + i - l.rank;
+            float f;
+            if (e == 4) memcpy(&f, r + (size_t)at * 4, 4);
+            else { uint16_t h; memcpy(&h, r + (size_t)at * 2, 2); f = bf16_bits_to_float(h); }
+            dst[(size_t)t * (l.rank + l.rot) + i] = f;
+        }
+    }
     return SWLM_OK;
 }
 
@@ -2290,7 +2306,9 @@ int swlm_profile_kind(swlm_state* s, int step_kind, int repeats) {
     int kind;
     switch (step_kind) {
     case SWLM_STEP_QGEMV: kind = L_QGEMV; break;
-    case SWLM_STEP_ATTN_DECODE: kind = L_ATTN; break;
+    case SWLM_STEP_ATTN_DECODE: kind = L_ATTN; break;   // of a latent step: its attention kernel alone
+    case SWLM_STEP_PRODUCT: kind = L_PRODUCT; break;
+    case SWLM_STEP_LATENT_ATTN: kind = L_LATENT; break;
     case SWLM_STEP_RESADD_COPY_RMSNORM: kind = L_RMSNORM; break;
     default: set_error("profile: step kind %d has no per-kind loop", step_kind); return SWLM_ERR_UNSUPPORTED;
     }

@@ -1,0 +1,866 @@
+// Executor of fp32-stream plans: step list -> launches, the paged pool of latent rows, and one row executor that runs decode
+// steps, prompt chunks and mixed batches alike. A batch is a list of rows, each with its token, sequence and position; the
+// only step that looks beyond its own row is latent attention, which finds the cached rows through the page table.
+#include <cmath>
+#include <cstdio>
+#include <cstring>
+
+#include "swlm_runtime.h"
+
+namespace swlm {
+namespace {
+
+bool stored_f32(const swlm_plan* p, int buf) {
+    return p->all_f32() || buf == SWLM_BUF_HIDDEN || buf == SWLM_BUF_RESIDUAL || buf == SWLM_BUF_SCRATCH3 || buf == SWLM_BUF_SCRATCH4 || buf == SWLM_BUF_LOGITS;
+}
+size_t stored_bytes(const swlm_plan* p, int buf) { return stored_f32(p, buf) ? 4 : 2; }
+bool act_buf(const swlm_plan* p, int buf) { return buf >= SWLM_BUF_SCRATCH0 && buf <= SWLM_BUF_SCRATCH2; }   // buffers products read
+bool any_buf(int b) { return b >= 0 && b < SWLM_BUF_COUNT; }
+
+int find_matrix(swlm_ctx* ctx, const char* name, int n, int k, const Matrix** out) {
+    auto it = ctx->matrices.find(name);
+    if (it == ctx->matrices.end()) { set_error("matrix '%s' not in the weight store", name); return SWLM_ERR_NOT_FOUND; }
+    if (it->second.n != n || it->second.k != k) { set_error("matrix '%s' is %d x %d, the step wants %d x %d", name, it->second.n, it->second.k, n, k); return SWLM_ERR_INVALID; }
+    *out = &it->second;
+    return SWLM_OK;
+}
+int find_vector(swlm_ctx* ctx, const char* name, int count, const DenseTensor** out) {
+    auto it = ctx->dense.find(name);
+    if (it == ctx->dense.end()) { set_error("tensor '%s' not in the weight store", name); return SWLM_ERR_NOT_FOUND; }
+    if (it->second.rows * it->second.cols != count) { set_error("tensor '%s' holds %lld values, the step wants %d", name, (long long)(it->second.rows * it->second.cols), count); return SWLM_ERR_INVALID; }
+    *out = &it->second;
+    return SWLM_OK;
+}
+
+// The rows of several matrices one after the other; the parts become views of it, so nothing is stored twice.
+int concat_matrices(swlm_ctx* ctx, const std::vector<std::string>& names, const Matrix** out) {
+    std::string key = names[0];
+    for (size_t i = 1; i < names.size(); ++i) key += "|" + names[i];
+    auto hit = ctx->matrix_cat.find(key);
+    if (hit != ctx->matrix_cat.end()) { *out = &hit->second; return SWLM_OK; }
+    Matrix cat;
+    cat.k = ctx->matrices.at(names[0]).k; cat.ld = ctx->matrices.at(names[0]).ld;
+    for (const std::string& nm : names) cat.n += ctx->matrices.at(nm).n;
+    int rc = dev_alloc(&cat.data, (size_t)cat.n * cat.ld, &ctx->bytes);
+    if (rc) return rc;
+    size_t row = 0;
+    for (const std::string& nm : names) {
+        Matrix& m = ctx->matrices.at(nm);
+        SWLM_CUDA(cudaMemcpy(cat.data + row * cat.ld, m.data, (size_t)m.n * m.ld * 2, cudaMemcpyDeviceToDevice));
+        if (!m.view) {
+            // plans built earlier may hold the old address: their kernels are ordered before the free by the device
+            SWLM_CUDA(cudaDeviceSynchronize());
+            cudaFree(m.data);
+            ctx->bytes -= (int64_t)m.n * m.ld * 2;
+        }
+        m.data = cat.data + row * cat.ld;
+        m.view = true;
+        row += m.n;
+    }
+    ctx->matrix_cat[key] = cat;
+    *out = &ctx->matrix_cat[key];
+    return SWLM_OK;
+}
+
+// Angle per position of every pair, interpolated by parts when the step says so, in double precision on the host.
+int stream_rope_table(swlm_plan* plan, const swlm_step& st, int* index) {
+    for (size_t i = 0; i < plan->rope_tables.size(); ++i) {
+        const RopeTable& t = plan->rope_tables[i];
+        if (t.rope_dim == st.rope_dim && t.base == st.rope_base && t.factor == st.rope_factor && t.original == st.rope_original &&
+            t.fast == st.rope_fast && t.slow == st.rope_slow) { *index = (int)i; return SWLM_OK; }
+    }
+    const int half = st.rope_dim / 2;
+    std::vector<float> f(std::max(1, half));
+    const double base = st.rope_base, dims = st.rope_dim;
+    RopeTable t;
+    t.rope_dim = st.rope_dim; t.base = st.rope_base; t.factor = st.rope_factor; t.original = st.rope_original; t.fast = st.rope_fast; t.slow = st.rope_slow;
+    double lo = 0, hi = 0;
+    if (st.rope_factor > 0.f) {
+        auto dim_of = [&](double turns) { return dims * std::log((double)st.rope_original / (2.0 * M_PI * turns)) / (2.0 * std::log(base)); };
+        lo = std::max(std::floor(dim_of(st.rope_fast)), 0.0);
+        hi = std::min(std::ceil(dim_of(st.rope_slow)), dims - 1.0);
+        t.magnitude = (float)(0.1 * std::log((double)st.rope_factor) + 1.0);
+    }
+    for (int i = 0; i < half; ++i) {
+        const double plain = std::pow(base, -2.0 * i / dims);
+        const double ramp = st.rope_factor > 0.f ? std::min(1.0, std::max(0.0, (i - lo) / std::max(hi - lo, 0.001))) : 0.0;
+        f[i] = (float)(ramp > 0.0 ? plain / st.rope_factor * ramp + plain * (1.0 - ramp) : plain);
+    }
+    int rc = dev_alloc(&t.inv_freq, f.size());
+    if (rc) return rc;
+    SWLM_CUDA(cudaMemcpy(t.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice));
+    plan->rope_tables.push_back(t);
+    *index = (int)plan->rope_tables.size() - 1;
+    return SWLM_OK;
+}
+
+bool is_norm(int kind) {
+    return kind == SWLM_STEP_COPY_RMSNORM || kind == SWLM_STEP_RESADD_COPY_RMSNORM || kind == SWLM_STEP_RESADD_RMSNORM ||
+           kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_RMSNORM;
+}
+bool is_postnorm(int kind) { return kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_RMSNORM; }
+bool norm_stores(int kind) { return kind == SWLM_STEP_COPY_RMSNORM || kind == SWLM_STEP_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM; }
+bool reads(const swlm_step& s, int buf) { return s.in_buf == buf || (s.kind != SWLM_STEP_PRODUCT && !is_norm(s.kind) && (s.in2_buf == buf || s.in3_buf == buf)); }
+
+}  // namespace
+
+int stream_compile(swlm_plan* plan) {
+    swlm_ctx* ctx = plan->ctx;
+    const swlm_buffers_desc& d = plan->desc;
+    const std::vector<swlm_step>& st = plan->steps;
+    if (ctx->tp_size > 1) { set_error("fp32-stream plans run on one GPU"); return SWLM_ERR_UNSUPPORTED; }
+    if (d.stream_dtype < 0 || d.stream_dtype > SWLM_STREAM_ALL_F32) { set_error("stream_dtype %d", d.stream_dtype); return SWLM_ERR_INVALID; }
+    int rc;
+    auto widen = [&](int buf, int n) { plan->stream_width[buf] = std::max(plan->stream_width[buf], (n + 7) / 8 * 8); };
+    plan->latent.assign(std::max(0, d.latent_layers), LatentLayer{});
+    widen(SWLM_BUF_HIDDEN, d.hidden);
+    widen(SWLM_BUF_RESIDUAL, d.hidden);
+    widen(SWLM_BUF_LOGITS, d.vocab);
+    for (size_t i = 0; i < st.size();) {
+        const swlm_step& s = st[i];
+        Launch L;
+        L.st = s;
+        switch (s.kind) {
+        case SWLM_STEP_EMBED: {
+            L.kind = L_EMBED;
+            auto it = ctx->dense.find(s.weight);
+            if (it == ctx->dense.end()) { set_error("embedding table '%s' missing", s.weight); return SWLM_ERR_NOT_FOUND; }
+            L.d1 = &it->second;
+            if (s.out_buf != SWLM_BUF_HIDDEN || s.n != d.hidden || L.d1->cols != s.n || L.d1->rows != d.vocab) { set_error("embedding '%s': table %lld x %lld for vocabulary %d, width %d", s.weight, (long long)L.d1->rows, (long long)L.d1->cols, d.vocab, d.hidden); return SWLM_ERR_INVALID; }
+            L.label = std::string("embed ") + s.weight;
+            break;
+        }
+        case SWLM_STEP_COPY_RMSNORM: case SWLM_STEP_RESADD_COPY_RMSNORM: case SWLM_STEP_RESADD_RMSNORM:
+        case SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM: case SWLM_STEP_POSTNORM_RESADD_RMSNORM:
+            L.kind = L_RMSNORM;
+            if (s.in_buf != SWLM_BUF_HIDDEN || !act_buf(plan, s.out_buf) || s.n != d.hidden) { set_error("norm '%s': reads hidden, writes scratch 0..2, width %d", s.weight, d.hidden); return SWLM_ERR_INVALID; }
+            if ((rc = find_vector(ctx, is_postnorm(s.kind) ? s.weight2 : s.weight, s.n, &L.d1))) return rc;
+            if (is_postnorm(s.kind) && (rc = find_vector(ctx, s.weight, s.n, &L.norm_post))) return rc;
+            widen(s.out_buf, s.n);
+            L.label = std::string(is_postnorm(s.kind) ? "postnorm+rmsnorm " : "rmsnorm ") + (is_postnorm(s.kind) ? s.weight2 : s.weight);
+            break;
+        case SWLM_STEP_PRODUCT: {
+            L.kind = L_PRODUCT;
+            if (!act_buf(plan, s.in_buf) || !any_buf(s.out_buf) || s.out_buf == s.in_buf || s.out_buf == SWLM_BUF_RESIDUAL) { set_error("product '%s': bad buffers", s.weight); return SWLM_ERR_INVALID; }
+            if ((rc = find_matrix(ctx, s.weight, s.n, s.k, &L.m1))) return rc;
+            widen(s.in_buf, s.k);
+            widen(s.out_buf, s.n);
+            // gate, up, gated activation -> one launch
+            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && (st[i + 2].kind == SWLM_STEP_SWIGLU || st[i + 2].kind == SWLM_STEP_GEGLU) &&
+                st[i + 1].in_buf == s.in_buf && st[i + 1].k == s.k && st[i + 1].n == s.n && st[i + 2].in_buf == s.out_buf &&
+                st[i + 2].in2_buf == st[i + 1].out_buf && st[i + 2].n == s.n && act_buf(plan, st[i + 2].out_buf) && st[i + 2].out_buf != s.in_buf &&
+                act_buf(plan, s.out_buf) && act_buf(plan, st[i + 1].out_buf)) {
+                if ((rc = find_matrix(ctx, st[i + 1].weight, s.n, s.k, &L.m2))) return rc;
+                widen(st[i + 1].out_buf, s.n);
+                widen(st[i + 2].out_buf, s.n);
+                L.gated_act = st[i + 2].kind == SWLM_STEP_GEGLU ? GATED_ACT_GELU_TANH : GATED_ACT_SILU;
+                L.seg_buf[0] = st[i + 2].out_buf; L.seg_end[0] = s.n;
+                L.seg_buf[1] = s.out_buf; L.seg_buf[2] = st[i + 1].out_buf;   // where the halves go when they run apart
+                L.steps_covered = 3;
+                L.label = std::string("product+gate ") + s.weight + " ^ " + st[i + 1].weight;
+                break;
+            }
+            std::vector<std::string> names{s.weight};
+            L.seg_buf[0] = s.out_buf; L.seg_end[0] = s.n;
+            L.label = std::string("product ") + s.weight;
+            size_t j = i + 1;
+            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && st[j].in_buf == s.in_buf && st[j].k == s.k &&
+                   st[j].out_buf != s.in_buf && any_buf(st[j].out_buf) && st[j].out_buf != SWLM_BUF_LOGITS && s.out_buf != SWLM_BUF_LOGITS) {
+                bool clash = false;
+                for (size_t q = i; q < j; ++q) clash |= st[q].out_buf == st[j].out_buf || !strcmp(st[q].weight, st[j].weight);
+                // a gate / up pair that starts here keeps its own launch
+                if (clash || (j + 2 < st.size() && (st[j + 2].kind == SWLM_STEP_SWIGLU || st[j + 2].kind == SWLM_STEP_GEGLU) && st[j + 2].in_buf == st[j].out_buf)) break;
+                const Matrix* m;
+                if ((rc = find_matrix(ctx, st[j].weight, st[j].n, st[j].k, &m))) return rc;
+                widen(st[j].out_buf, st[j].n);
+                const int q = (int)names.size();
+                L.seg_buf[q] = st[j].out_buf; L.seg_end[q] = L.seg_end[q - 1] + st[j].n;
+                names.push_back(st[j].weight);
+                L.label += std::string(" ") + st[j].weight;
+                ++j;
+            }
+            L.n_seg = (int)names.size();
+            L.steps_covered = L.n_seg;
+            if (L.n_seg > 1 && (rc = concat_matrices(ctx, names, &L.m1))) return rc;
+            break;
+        }
+        case SWLM_STEP_SWIGLU: case SWLM_STEP_GEGLU:
+            L.kind = L_SWIGLU;
+            L.gated_act = s.kind == SWLM_STEP_GEGLU ? GATED_ACT_GELU_TANH : GATED_ACT_SILU;
+            if (!act_buf(plan, s.in_buf) || !act_buf(plan, s.in2_buf) || !act_buf(plan, s.out_buf) || s.n <= 0) { set_error("gated activation: bad buffers"); return SWLM_ERR_INVALID; }
+            widen(s.in_buf, s.n); widen(s.in2_buf, s.n); widen(s.out_buf, s.n);
+            L.label = L.gated_act ? "geglu" : "swiglu";
+            break;
+        case SWLM_STEP_LATENT_ATTN: {
+            L.kind = L_LATENT;
+            if (s.layer < 0 || s.layer >= d.latent_layers) { set_error("latent attention: layer %d outside the pool", s.layer); return SWLM_ERR_INVALID; }
+            if (s.heads <= 0 || s.head_dim <= 0 || s.key_dim < 0 || s.value_dim <= 0 || s.n <= 0 || s.rope_dim < 0 || s.rope_dim > s.key_dim || (s.rope_dim & 1)) { set_error("latent attention: bad sizes"); return SWLM_ERR_INVALID; }
+            if (!act_buf(plan, s.in_buf) || !stored_f32(plan, s.in2_buf) || !any_buf(s.in2_buf) || !act_buf(plan, s.out_buf) || s.out_buf == s.in_buf ||
+                (s.in3_buf != SWLM_BUF_NONE && (!any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf)))) { set_error("latent attention: q and the result in scratch 0..2, latent and gate in scratch 3 and 4"); return SWLM_ERR_INVALID; }
+            if ((rc = find_vector(ctx, s.weight, s.n, &L.d1))) return rc;
+            const Matrix *uk, *uv;
+            if ((rc = find_matrix(ctx, s.weight2, s.heads * s.head_dim, s.n, &uk)) || (rc = find_matrix(ctx, s.weight3, s.heads * s.value_dim, s.n, &uv))) return rc;
+            const Matrix* both;
+            const std::vector<std::string> pair{s.weight2, s.weight3};
+            if ((rc = concat_matrices(ctx, pair, &both))) return rc;
+            L.m1 = uk; L.m2 = uv;
+            if ((rc = stream_rope_table(plan, s, &L.rope_table))) return rc;
+            LatentLayer& ll = plan->latent[s.layer];
+            if (ll.rank && (ll.rank != s.n || ll.rot != s.key_dim)) { set_error("latent layer %d is used with two row sizes", s.layer); return SWLM_ERR_INVALID; }
+            ll.rank = s.n; ll.rot = s.key_dim; ll.row = latent_row(s.n, s.key_dim, plan->all_f32());
+            widen(s.in_buf, s.heads * (s.head_dim + s.key_dim));
+            widen(s.in2_buf, s.n + s.key_dim);
+            if (s.in3_buf != SWLM_BUF_NONE) widen(s.in3_buf, s.heads);
+            widen(s.out_buf, s.heads * s.value_dim);
+            plan->latent_heads_max = std::max(plan->latent_heads_max, s.heads);
+            plan->latent_q_floats = std::max(plan->latent_q_floats, (int)latent_qcat_floats(ll.row, s.heads));
+            plan->latent_part_floats = std::max(plan->latent_part_floats, (int)latent_partial_floats(ll.row, s.heads));
+            L.label = std::string("latent_attention ") + s.weight2;
+            break;
+        }
+        case SWLM_STEP_ARGMAX:
+            L.kind = L_ARGMAX;
+            if (s.in_buf != SWLM_BUF_LOGITS || s.n != d.vocab) { set_error("argmax: reads the logits"); return SWLM_ERR_INVALID; }
+            L.label = "argmax";
+            break;
+        default:
+            set_error("step %zu: kind %d cannot be part of an fp32-stream plan", i, s.kind);
+            return SWLM_ERR_UNSUPPORTED;
+        }
+        i += L.steps_covered;
+        plan->launches.push_back(L);
+    }
+    for (int l = 0; l < d.latent_layers; ++l)
+        if (!plan->latent[l].rank && st.size() > 1) { set_error("latent layer %d has no step", l); return SWLM_ERR_INVALID; }
+
+    // A norm rides with the product behind it when that is its only reader: few rows compute it in the product's prologue,
+    // more rows run it in front.
+    for (size_t i = 0; i + 1 < plan->launches.size(); ++i) {
+        const Launch A = plan->launches[i];
+        Launch& B = plan->launches[i + 1];
+        if (A.kind != L_RMSNORM || B.kind != L_PRODUCT || B.st.in_buf != A.st.out_buf) continue;
+        bool ok = true;
+        for (size_t j = i + 2; j < plan->launches.size(); ++j) {
+            const Launch& C = plan->launches[j];
+            if (reads(C.st, A.st.out_buf)) { ok = false; break; }
+            bool writes = C.st.out_buf == A.st.out_buf;
+            for (int q = 0; q < C.n_seg; ++q) writes |= C.seg_buf[q] == A.st.out_buf;
+            if (writes) break;
+        }
+        if (!ok) continue;
+        B.norm = A.st; B.norm_w = A.d1; B.norm_post = A.norm_post;
+        B.label = A.label + " + " + B.label;
+        B.steps_covered += 1;
+        plan->launches.erase(plan->launches.begin() + i);
+    }
+    // the residual stream alternates between two buffers, so that a norm computed by every CTA of a product can be stored by one
+    int cur = 0;
+    for (Launch& L : plan->launches) {
+        const int kind = L.kind == L_RMSNORM ? L.st.kind : L.kind == L_PRODUCT ? L.norm.kind : 0;
+        L.res_in = L.res_out = cur;
+        if (is_norm(kind) && norm_stores(kind)) { L.res_out = 1 - cur; cur = 1 - cur; }
+    }
+    plan->final_res = cur;
+    return SWLM_OK;
+}
+
+// ---- pages -----------------------------------------------------------------------------------------------------------
+int stream_reserve(swlm_state* s, int seq, int tokens, bool shrink) {
+    if (tokens > s->plan->desc.max_seq) { set_error("sequence %d: %d tokens exceed max_seq %d", seq, tokens, s->plan->desc.max_seq); return SWLM_ERR_STATE; }
+    std::vector<int>& have = s->seq_pages[seq];
+    const size_t need = (size_t)(tokens + SWLM_PAGE_TOKENS - 1) / SWLM_PAGE_TOKENS;
+    if (need > have.size() + s->free_pages.size()) {
+        set_error("sequence %d needs %zu pages, %zu held and %zu free", seq, need, have.size(), s->free_pages.size());
+        return SWLM_ERR_STATE;
+    }
+    while (have.size() < need) {
+        s->page_table_host[(size_t)seq * s->pages_per_seq + have.size()] = s->free_pages.back();
+        have.push_back(s->free_pages.back());
+        s->free_pages.pop_back();
+        s->page_table_dirty = true;
+    }
+    while (shrink && have.size() > need) {
+        s->free_pages.push_back(have.back());
+        have.pop_back();
+    }
+    return SWLM_OK;
+}
+
+void stream_release_all(swlm_state* s) {
+    for (std::vector<int>& pages : s->seq_pages) pages.clear();
+    s->free_pages.clear();
+    for (int p = s->pool_pages - 1; p >= 0; --p) s->free_pages.push_back(p);   // page 0 is handed out first
+}
+
+int stream_upload_pages(swlm_state* s) {
+    if (!s->page_table_dirty || s->page_table_host.empty()) return SWLM_OK;
+    SWLM_CUDA(cudaMemcpyAsync(s->page_table, s->page_table_host.data(), s->page_table_host.size() * 4, cudaMemcpyHostToDevice, s->stream));
+    s->page_table_dirty = false;
+    return SWLM_OK;
+}
+
+namespace {
+
+template <typename T>
+int grow(T** p, size_t* cap, size_t need, cudaStream_t stream) {
+    if (need <= *cap) return SWLM_OK;
+    SWLM_CUDA(cudaStreamSynchronize(stream));
+    cudaFree(*p);
+    *p = nullptr; *cap = 0;
+    const int rc = dev_alloc(p, need);
+    if (!rc) *cap = need;
+    return rc;
+}
+
+int bufs_rows(swlm_state* s, StreamBufs* b, int rows, int wants) {
+    const swlm_plan* plan = s->plan;
+    int rc;
+    if (rows > b->rows) {
+        SWLM_CUDA(cudaStreamSynchronize(s->stream));
+        for (int i = 0; i < SWLM_BUF_COUNT; ++i) {
+            if (i == SWLM_BUF_LOGITS) continue;
+            cudaFree(b->buf[i]);
+            b->buf[i] = nullptr;
+            const size_t bytes = (size_t)rows * s->width[i] * stored_bytes(plan, i);
+            unsigned char* p = nullptr;
+            if ((rc = dev_alloc(&p, bytes))) return rc;
+            b->buf[i] = p;
+            if (bytes) SWLM_CUDA(cudaMemsetAsync(p, 0, bytes, s->stream));
+        }
+        cudaFree(b->res2);
+        if ((rc = dev_alloc(&b->res2, (size_t)rows * s->width[SWLM_BUF_RESIDUAL]))) return rc;
+        SWLM_CUDA(cudaMemsetAsync(b->res2, 0, (size_t)rows * s->width[SWLM_BUF_RESIDUAL] * 4, s->stream));
+        b->rows = rows;
+    }
+    if (wants > b->wants) {
+        SWLM_CUDA(cudaStreamSynchronize(s->stream));
+        cudaFree(b->buf[SWLM_BUF_LOGITS]);
+        cudaFree(b->argmax_out);
+        b->buf[SWLM_BUF_LOGITS] = nullptr; b->argmax_out = nullptr; b->wants = 0;
+        float* p = nullptr;
+        if ((rc = dev_alloc(&p, (size_t)wants * s->width[SWLM_BUF_LOGITS]))) return rc;
+        b->buf[SWLM_BUF_LOGITS] = p;
+        if ((rc = dev_alloc(&b->argmax_out, wants))) return rc;
+        b->wants = wants;
+    }
+    if (!b->argmax_val) {
+        if ((rc = dev_alloc(&b->argmax_val, argmax_scratch_elems(kMaxSequences)))) return rc;
+        if ((rc = dev_alloc(&b->argmax_idx, argmax_scratch_elems(kMaxSequences)))) return rc;
+    }
+    return SWLM_OK;
+}
+
+size_t part_need(const swlm_plan* plan, int rows, int wants) {
+    size_t need = 0;
+    if (plan->all_f32()) return 0;
+    for (const Launch& L : plan->launches)
+        if (L.kind == L_PRODUCT) need = std::max(need, product_part_floats(L.m1->n, L.m1->k, L.seg_buf[0] == SWLM_BUF_LOGITS ? wants : rows, L.m2 != nullptr));
+    return need;
+}
+
+// scratch of a batch; r.splits_pages bounds the splits
+int bufs_scratch(swlm_state* s, StreamBufs* b, const RowBatch& r) {
+    const swlm_plan* plan = s->plan;
+    int rc;
+    size_t part = part_need(plan, r.rows, r.wants), expand = 0;
+    for (const Launch& L : plan->launches) {
+        if (L.kind != L_LATENT || r.n_long == 0) continue;
+        const LatentLayer& ll = plan->latent[L.st.layer];
+        expand = std::max(expand, latent_expand_bytes(ll.row, L.st.heads, L.st.head_dim, L.st.value_dim, r.total_ctx));
+        part = std::max(part, product_part_floats(L.st.heads * (L.st.head_dim + L.st.value_dim), ll.rank, r.total_ctx, false));
+    }
+    if ((rc = grow(&b->part, &b->part_cap, part, s->stream))) return rc;
+    if ((rc = grow(&b->expand, &b->expand_cap, expand, s->stream))) return rc;
+    if ((rc = grow(&b->qcat, &b->qcat_cap, (size_t)r.n_short * plan->latent_q_floats, s->stream))) return rc;
+    size_t partial = 0;
+    for (const Launch& L : plan->launches)
+        if (L.kind == L_LATENT)
+            partial = std::max(partial, (size_t)r.n_short * latent_pick_splits(r.n_short, L.st.heads, r.splits_pages) * latent_partial_floats(plan->latent[L.st.layer].row, L.st.heads));
+    return grow(&b->partial, &b->partial_cap, partial, s->stream);
+}
+
+void bufs_free(StreamBufs* b) {
+    for (void* p : b->buf) cudaFree(p);
+    cudaFree(b->res2); cudaFree(b->meta); cudaFree(b->argmax_out); cudaFree(b->qcat); cudaFree(b->partial); cudaFree(b->part);
+    cudaFree(b->expand); cudaFree(b->argmax_val); cudaFree(b->argmax_idx);
+    *b = StreamBufs{};
+}
+
+float* residual(StreamBufs* b, int phys) { return phys ? b->res2 : static_cast<float*>(b->buf[SWLM_BUF_RESIDUAL]); }
+
+StreamNorm norm_of(swlm_state* s, StreamBufs* b, const swlm_step& st, const DenseTensor* w, const DenseTensor* post, int res_in, int res_out) {
+    StreamNorm n;
+    n.mode = st.kind;
+    n.in = static_cast<const float*>(b->buf[st.in_buf]); n.in_stride = s->width[st.in_buf];
+    n.res_stride = s->width[SWLM_BUF_RESIDUAL];
+    if (st.kind != SWLM_STEP_COPY_RMSNORM) n.res_in = residual(b, res_in);
+    if (norm_stores(st.kind)) n.res_out = residual(b, res_out);
+    n.w = w->data; n.w_post = post ? post->data : nullptr;
+    n.eps = st.eps; n.weight_bias = st.weight_bias;
+    return n;
+}
+
+// The plan's launches over one batch of rows. only_kind >= 0: those launches alone (timing hook; L_ATTN stands for the
+// attention kernel of the latent steps).
+int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool body_only, cudaStream_t stream, int only_kind = -1) {
+    const swlm_plan* plan = s->plan;
+    const swlm_buffers_desc& d = plan->desc;
+    const bool f32 = plan->all_f32();
+    const int wants = body_only ? 0 : r.wants;
+    bool advanced = false;
+    int rc = SWLM_OK;
+    s->last_bufs = b;
+    s->last_res = plan->final_res;
+    for (const Launch& L : plan->launches) {
+        const swlm_step& st = L.st;
+        const bool latent_kernel = only_kind == L_ATTN && L.kind == L_LATENT;
+        if (only_kind >= 0 && L.kind != only_kind && !latent_kernel) continue;
+        switch (L.kind) {
+        case L_EMBED:
+            rc = launch_stream_embed(r.rows, st.n, r.tok, d.vocab, L.d1->data, st.scale != 0.f ? st.scale : 1.f, static_cast<float*>(b->buf[st.out_buf]), s->width[st.out_buf], stream);
+            s->launches += 1;
+            break;
+        case L_RMSNORM:
+            rc = launch_stream_norm(norm_of(s, b, st, L.d1, L.norm_post, L.res_in, L.res_out), r.rows, st.n, nullptr, b->buf[st.out_buf], s->width[st.out_buf], f32, stream);
+            s->launches += 1;
+            break;
+        case L_PRODUCT: {
+            const bool head = L.seg_buf[0] == SWLM_BUF_LOGITS;
+            const int m = head ? wants : r.rows;
+            if (m == 0) break;
+            const int32_t* idx = head ? r.wants_idx : nullptr;
+            ProductLaunch a;
+            a.w = L.m1; a.w2 = L.m2; a.act = L.gated_act; a.m = m; a.x_f32 = f32;
+            a.x = b->buf[st.in_buf]; a.x_stride = s->width[st.in_buf];
+            a.part = b->part; a.part_floats = b->part_cap; a.status = s->pf_status;
+            if (head && idx && !L.norm.kind) { set_error("the output head must follow a norm that nothing else reads"); return SWLM_ERR_UNSUPPORTED; }
+            if (L.norm.kind) {
+                const StreamNorm n = norm_of(s, b, L.norm, L.norm_w, L.norm_post, L.res_in, L.res_out);
+                if (!idx && product_takes_norm(m, L.m1->k)) a.norm = n;
+                else {
+                    rc = launch_stream_norm(n, m, L.norm.n, idx, b->buf[st.in_buf], s->width[st.in_buf], f32, stream);
+                    s->launches += 1;
+                    if (rc) return rc;
+                }
+            }
+            auto segment = [&](int q, int buf, int end) {
+                a.out.y[q] = b->buf[buf]; a.out.stride[q] = s->width[buf]; a.out.f32[q] = stored_f32(plan, buf) ? 1 : 0; a.out.end[q] = end;
+            };
+            if (L.m2 && !product_takes_gate(m, L.m1->k, f32)) {
+                // gate and up one after the other, then the activation
+                for (int h = 0; h < 2 && !rc; ++h) {
+                    ProductLaunch c = a;
+                    c.w = h ? L.m2 : L.m1; c.w2 = nullptr;
+                    c.out.count = 1;
+                    const int buf = L.seg_buf[1 + h];
+                    c.out.y[0] = b->buf[buf]; c.out.stride[0] = s->width[buf]; c.out.f32[0] = stored_f32(plan, buf) ? 1 : 0; c.out.end[0] = c.w->n;
+                    rc = launch_product(c, stream);
+                    s->launches += product_launch_count(c);
+                }
+                if (!rc) rc = launch_stream_gated(m, L.m1->n, b->buf[L.seg_buf[1]], s->width[L.seg_buf[1]], b->buf[L.seg_buf[2]], s->width[L.seg_buf[2]],
+                                                  b->buf[L.seg_buf[0]], s->width[L.seg_buf[0]], f32, L.gated_act, stream);
+                s->launches += 1;
+                break;
+            }
+            a.out.count = L.n_seg;
+            for (int q = 0; q < L.n_seg; ++q) segment(q, L.seg_buf[q], L.seg_end[q]);
+            for (int q = L.n_seg; q < kMaxProductSegs; ++q) a.out.end[q] = L.seg_end[L.n_seg - 1];
+            rc = launch_product(a, stream);
+            s->launches += product_launch_count(a);
+            break;
+        }
+        case L_SWIGLU:
+            rc = launch_stream_gated(r.rows, st.n, b->buf[st.in_buf], s->width[st.in_buf], b->buf[st.in2_buf], s->width[st.in2_buf], b->buf[st.out_buf],
+                                     s->width[st.out_buf], f32, L.gated_act, stream);
+            s->launches += 1;
+            break;
+        case L_LATENT: {
+            LatentLaunch a;
+            const RopeTable& rope = plan->rope_tables[L.rope_table];
+            a.row = plan->latent[st.layer].row;
+            a.heads = st.heads; a.dim = st.head_dim; a.vdim = st.value_dim; a.rot_dims = st.rope_dim;
+            a.scale = st.scale; a.eps = st.eps; a.weight_bias = st.weight_bias; a.magnitude = rope.magnitude; a.inv_freq = rope.inv_freq; a.f32 = f32;
+            a.q = b->buf[st.in_buf]; a.q_stride = s->width[st.in_buf];
+            a.kv = static_cast<const float*>(b->buf[st.in2_buf]); a.kv_stride = s->width[st.in2_buf];
+            if (st.in3_buf != SWLM_BUF_NONE) { a.gate = static_cast<const float*>(b->buf[st.in3_buf]); a.gate_stride = s->width[st.in3_buf]; }
+            a.norm_w = L.d1->data; a.uk = L.m1; a.uv = L.m2;
+            a.ukv = &plan->ctx->matrix_cat.at(std::string(st.weight2) + "|" + st.weight3);
+            a.pool = s->pool[st.layer]; a.page_table = s->page_table; a.pages_per_seq = s->pages_per_seq;
+            a.row_seq = r.seq; a.row_pos = r.pos;
+            a.out = b->buf[st.out_buf]; a.out_stride = s->width[st.out_buf];
+            a.n_short = r.n_short; a.short_rows = r.short_rows; a.splits = latent_pick_splits(r.n_short, st.heads, r.splits_pages);
+            a.qcat = b->qcat; a.partial = b->partial;
+            a.n_long = r.n_long; a.long_rows = r.long_rows; a.n_spans = r.n_spans; a.spans = r.spans; a.n_tiles = r.n_tiles; a.tiles = r.tiles; a.total_ctx = r.total_ctx;
+            a.expand = b->expand; a.part = b->part; a.part_floats = b->part_cap; a.status = s->pf_status;
+            a.only_attention = latent_kernel;
+            int n = 0;
+            rc = launch_latent(a, stream, &n);
+            s->launches += n;
+            break;
+        }
+        case L_ARGMAX:
+            if (wants == 0) break;
+            if (r.advance) {
+                rc = launch_argmax_f32(wants, st.n, static_cast<const float*>(b->buf[SWLM_BUF_LOGITS]), s->width[SWLM_BUF_LOGITS], s->token_out, s->token_in, s->ring,
+                                       s->step_counter, s->ring_cap, s->position, 1, b->argmax_val, b->argmax_idx, stream);
+                advanced = true;
+            } else {
+                rc = launch_argmax_f32(wants, st.n, static_cast<const float*>(b->buf[SWLM_BUF_LOGITS]), s->width[SWLM_BUF_LOGITS], b->argmax_out, nullptr, nullptr,
+                                       s->step_counter, s->ring_cap, s->position, 0, b->argmax_val, b->argmax_idx, stream);
+            }
+            s->launches += 2 * ((wants + kMaxSequences - 1) / kMaxSequences);
+            break;
+        }
+        if (rc) return rc;
+    }
+    if (r.advance && !advanced && only_kind < 0) {
+        rc = launch_advance(r.rows, s->position, nullptr, stream);
+        s->launches += 1;
+    }
+    return rc;
+}
+
+RowBatch identity_batch(const swlm_state* s) {
+    RowBatch r;
+    r.rows = r.wants = r.n_short = s->plan->desc.max_batch;
+    r.tok = s->token_in; r.seq = s->seq_identity; r.pos = s->position;
+    r.splits_pages = s->pages_per_seq;
+    r.advance = true;
+    return r;
+}
+
+// scratch of every decode step a graph may hold: 1 .. max_batch rows
+int decode_scratch(swlm_state* s) {
+    for (int n = 1; n <= s->plan->desc.max_batch; ++n) {
+        RowBatch r;
+        r.rows = r.wants = r.n_short = n;
+        r.splits_pages = s->pages_per_seq;
+        const int rc = bufs_scratch(s, &s->dec, r);
+        if (rc) return rc;
+    }
+    return SWLM_OK;
+}
+
+}  // namespace
+
+// ---- state -----------------------------------------------------------------------------------------------------------
+int stream_state_create(swlm_state* s) {
+    const swlm_plan* plan = s->plan;
+    const swlm_buffers_desc& d = plan->desc;
+    int rc;
+    for (int i = 0; i < SWLM_BUF_COUNT; ++i) s->width[i] = plan->stream_width[i];
+    s->pages_per_seq = (d.max_seq + SWLM_PAGE_TOKENS - 1) / SWLM_PAGE_TOKENS;
+    s->pool_pages = d.kv_pool_tokens > 0 ? (d.kv_pool_tokens + SWLM_PAGE_TOKENS - 1) / SWLM_PAGE_TOKENS : s->pages_per_seq * d.max_batch;
+    const size_t elem = plan->all_f32() ? 4 : 2;
+    for (const LatentLayer& l : plan->latent) {
+        const size_t bytes = (size_t)s->pool_pages * SWLM_PAGE_TOKENS * l.row.pitch * elem;
+        unsigned char* p = nullptr;
+        if ((rc = dev_alloc(&p, bytes))) return rc;
+        s->pool.push_back(p);
+        s->pool_bytes.push_back(bytes);
+        // a page is read whole: rows nobody has written must hold finite numbers
+        if (bytes) SWLM_CUDA(cudaMemset(p, 0, bytes));
+    }
+    s->seq_pages.assign(d.max_batch, {});
+    s->page_table_host.assign((size_t)d.max_batch * s->pages_per_seq, 0);
+    if ((rc = dev_alloc(&s->page_table, s->page_table_host.size()))) return rc;
+    s->page_table_dirty = true;
+    stream_release_all(s);
+    if ((rc = dev_alloc(&s->seq_identity, d.max_batch))) return rc;
+    std::vector<int32_t> ident(d.max_batch);
+    for (int i = 0; i < d.max_batch; ++i) ident[i] = i;
+    SWLM_CUDA(cudaMemcpy(s->seq_identity, ident.data(), ident.size() * 4, cudaMemcpyHostToDevice));
+    if (!s->pf_status) {
+        if ((rc = dev_alloc(&s->pf_status, 1))) return rc;
+        SWLM_CUDA(cudaMemset(s->pf_status, 0, sizeof(int)));
+    }
+    if ((rc = bufs_rows(s, &s->dec, d.max_batch, d.max_batch))) return rc;
+    if ((rc = grow(&s->dec.meta, &s->dec.meta_cap, (size_t)3 * d.max_batch, s->stream))) return rc;
+    s->last_bufs = &s->dec;
+    return decode_scratch(s);
+}
+
+void stream_drop_graphs(swlm_state* s) {
+    for (auto& g : s->row_graphs) cudaGraphExecDestroy(g.second);
+    s->row_graphs.clear();
+    s->row_graph_launches.clear();
+}
+
+void stream_state_free(swlm_state* s) {
+    stream_drop_graphs(s);
+    for (void* p : s->pool) cudaFree(p);
+    cudaFree(s->page_table);
+    cudaFree(s->seq_identity);
+    bufs_free(&s->dec);
+    bufs_free(&s->big);
+    if (s->h_rows) cudaFreeHost(s->h_rows);
+}
+
+int stream_enqueue_step(swlm_state* s, bool body_only, cudaStream_t stream, int only_kind) {
+    return enqueue_rows_stream(s, &s->dec, identity_batch(s), body_only, stream, only_kind);
+}
+
+int stream_launches_per_step(const swlm_plan* plan) {
+    const int m = plan->desc.max_batch;
+    int n = 0;
+    for (const Launch& L : plan->launches) {
+        if (L.kind == L_PRODUCT) {
+            ProductLaunch a;
+            a.w = L.m1; a.w2 = L.m2; a.m = m; a.x_f32 = plan->all_f32();
+            const bool fused = L.norm.kind && product_takes_norm(m, L.m1->k);
+            if (fused) a.norm.mode = L.norm.kind;
+            else if (L.norm.kind) n += 1;
+            if (L.m2 && !product_takes_gate(m, L.m1->k, a.x_f32)) { a.w2 = nullptr; n += 2 * product_launch_count(a) + 1; }
+            else n += product_launch_count(a);
+        } else n += L.kind == L_LATENT ? 3 : L.kind == L_ARGMAX ? 2 : 1;
+    }
+    return n;
+}
+
+int stream_check_status(swlm_state* s) {
+    int st = 0;
+    SWLM_CUDA(cudaMemcpy(&st, s->pf_status, sizeof(int), cudaMemcpyDeviceToHost));
+    if (!st) return SWLM_OK;
+    SWLM_CUDA(cudaMemset(s->pf_status, 0, sizeof(int)));
+    set_error("a bounded wait in a kernel expired (code %d)", st);
+    return SWLM_ERR_TIMEOUT;
+}
+
+// ---- batches ---------------------------------------------------------------------------------------------------------
+namespace {
+
+struct Piece { int seq, pos0, count; const int32_t* tokens; };
+
+int stage(swlm_state* s, StreamBufs* b, const std::vector<int32_t>& meta) {
+    int rc;
+    // (`dec` never grows: its capacity covers 3 * max_batch words from the start)
+    if ((rc = grow(&b->meta, &b->meta_cap, meta.size(), s->stream))) return rc;
+    if (meta.size() > s->h_rows_cap) {
+        SWLM_CUDA(cudaStreamSynchronize(s->stream));
+        if (s->h_rows) cudaFreeHost(s->h_rows);
+        s->h_rows = nullptr; s->h_rows_cap = 0;
+        const size_t cap = std::max<size_t>(4096, meta.size());
+        SWLM_CUDA(cudaMallocHost((void**)&s->h_rows, cap * 4));
+        s->h_rows_cap = cap;
+    }
+    memcpy(s->h_rows, meta.data(), meta.size() * 4);   // callers synchronise before the next batch is staged
+    SWLM_CUDA(cudaMemcpyAsync(b->meta, s->h_rows, meta.size() * 4, cudaMemcpyHostToDevice, s->stream));
+    return SWLM_OK;
+}
+
+// spans of at least this many rows are attended over expanded keys and values
+constexpr int kSpanMinRows = 64;
+static_assert(sizeof(LatentSpan) == 20, "spans are staged as five words");
+
+// Rows of `pieces` in one pass; `want_rows` get logits and tokens in b->buf[LOGITS] / b->argmax_out.
+int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<int32_t>& want_rows, StreamBufs** used) {
+    const swlm_plan* plan = s->plan;
+    int rows = 0;
+    bool single = true;
+    for (const Piece& p : pieces) { rows += p.count; single &= p.count == 1; }
+    bool every = (int)want_rows.size() == rows;
+    for (int i = 0; i < (int)want_rows.size() && every; ++i) every = want_rows[i] == i;
+    const bool graph = single && every && rows <= plan->desc.max_batch;
+    StreamBufs* b = graph ? &s->dec : &s->big;
+    *used = b;
+    int rc;
+    if ((rc = stream_upload_pages(s))) return rc;
+    std::vector<int32_t> meta((size_t)3 * rows);
+    int at = 0, longest = 0;
+    for (const Piece& p : pieces) {
+        longest = std::max(longest, p.pos0 + p.count);
+        for (int i = 0; i < p.count; ++i, ++at) { meta[at] = p.tokens[i]; meta[rows + at] = p.seq; meta[2 * rows + at] = p.pos0 + i; }
+    }
+    RowBatch r;
+    r.rows = rows;
+    r.wants = (int)want_rows.size();
+    if (graph) {
+        if ((rc = stage(s, b, meta))) return rc;
+        r.tok = b->meta; r.seq = b->meta + rows; r.pos = b->meta + 2 * rows;
+        r.n_short = rows; r.splits_pages = s->pages_per_seq;
+        auto it = s->row_graphs.find(rows);
+        if (it == s->row_graphs.end()) {
+            cudaGraph_t g = nullptr;
+            const int64_t before = s->launches;
+            SWLM_CUDA(cudaStreamBeginCapture(s->stream, cudaStreamCaptureModeThreadLocal));
+            rc = enqueue_rows_stream(s, b, r, false, s->stream);
+            cudaError_t e = cudaStreamEndCapture(s->stream, &g);
+            const int n = (int)(s->launches - before);
+            s->launches = before;   // capture does not execute
+            if (rc) { if (g) cudaGraphDestroy(g); return rc; }
+            if (e != cudaSuccess) return cuda_fail(e, "cudaStreamEndCapture");
+            cudaGraphExec_t x = nullptr;
+            e = cudaGraphInstantiate(&x, g, 0);
+            cudaGraphDestroy(g);
+            if (e != cudaSuccess) return cuda_fail(e, "cudaGraphInstantiate");
+            it = s->row_graphs.emplace(rows, x).first;
+            s->row_graph_launches[rows] = n;
+        }
+        SWLM_CUDA(cudaGraphLaunch(it->second, s->stream));
+        s->launches += s->row_graph_launches[rows];
+        s->last_bufs = b;
+        return SWLM_OK;
+    }
+
+    // which pieces are attended in spans: every latent layer must allow it
+    bool expands = true;
+    for (const Launch& L : plan->launches)
+        if (L.kind == L_LATENT) expands &= latent_expands(plan->latent[L.st.layer].row, L.st.head_dim, L.st.value_dim, plan->all_f32());
+    std::vector<int32_t> shorts, longs;
+    std::vector<LatentSpan> spans;
+    std::vector<std::pair<int, int2>> tiles;   // (context at the end of the tile, tile)
+    int row0 = 0, short_longest = 0;
+    for (const Piece& p : pieces) {
+        if (expands && p.count >= kSpanMinRows) {
+            const int sp = (int)spans.size();
+            spans.push_back(LatentSpan{row0, p.count, p.pos0, p.seq, r.total_ctx});
+            r.total_ctx += p.pos0 + p.count;
+            for (int i = 0; i < p.count; ++i) longs.push_back(row0 + i);
+            for (int q = 0; q * kLatentQueryTile < p.count; ++q)
+                tiles.push_back({p.pos0 + std::min(p.count, (q + 1) * kLatentQueryTile), int2{sp, q}});
+        } else {
+            for (int i = 0; i < p.count; ++i) shorts.push_back(row0 + i);
+            short_longest = std::max(short_longest, p.pos0 + p.count);
+        }
+        row0 += p.count;
+    }
+    std::stable_sort(tiles.begin(), tiles.end(), [](const std::pair<int, int2>& a, const std::pair<int, int2>& c) { return a.first > c.first; });   // the longest first
+    const size_t o_want = meta.size();
+    meta.insert(meta.end(), want_rows.begin(), want_rows.end());
+    const size_t o_short = meta.size();
+    meta.insert(meta.end(), shorts.begin(), shorts.end());
+    const size_t o_long = meta.size();
+    meta.insert(meta.end(), longs.begin(), longs.end());
+    if (meta.size() & 1) meta.push_back(0);
+    const size_t o_tiles = meta.size();
+    for (const auto& tl : tiles) { meta.push_back(tl.second.x); meta.push_back(tl.second.y); }
+    const size_t o_spans = meta.size();
+    for (const LatentSpan& sp : spans) { const int32_t w[5] = {sp.row0, sp.count, sp.pos0, sp.seq, sp.ctx0}; meta.insert(meta.end(), w, w + 5); }
+    r.n_short = (int)shorts.size();
+    r.n_long = (int)longs.size();
+    r.n_spans = (int)spans.size();
+    r.n_tiles = (int)tiles.size();
+    r.splits_pages = std::max(1, (short_longest + SWLM_PAGE_TOKENS - 1) / SWLM_PAGE_TOKENS);
+    if ((rc = bufs_rows(s, b, std::max(rows, r.wants), r.wants)) || (rc = bufs_scratch(s, b, r)) || (rc = stage(s, b, meta))) return rc;
+    r.tok = b->meta; r.seq = b->meta + rows; r.pos = b->meta + 2 * rows;
+    r.wants_idx = b->meta + o_want;
+    r.short_rows = b->meta + o_short; r.long_rows = b->meta + o_long;
+    r.tiles = reinterpret_cast<const int2*>(b->meta + o_tiles);
+    r.spans = reinterpret_cast<const LatentSpan*>(b->meta + o_spans);
+    return enqueue_rows_stream(s, b, r, false, s->stream);
+}
+
+}  // namespace
+
+int stream_run(swlm_state* s, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, const int32_t* want_counts,
+               const int32_t* wants, float* logits_out, int32_t* tokens_out, int row_cap) {
+    const swlm_buffers_desc& d = s->plan->desc;
+    int rc;
+    std::vector<char> seen(d.max_batch, 0);
+    size_t n_tok = 0, n_want = 0, new_pages = 0;
+    for (int e = 0; e < n_entries; ++e) {
+        const int q = seqs[e];
+        if (q < 0 || q >= d.max_batch || seen[q]) { set_error("entry %d: sequence %d outside 0..%d or named twice", e, q, d.max_batch - 1); return SWLM_ERR_INVALID; }
+        seen[q] = 1;
+        if (counts[e] <= 0 || (want_counts && want_counts[e] < 0)) { set_error("entry %d: no tokens", e); return SWLM_ERR_INVALID; }
+        if (s->pos_host[q] + counts[e] > d.max_seq) { set_error("sequence %d: position %d + %d tokens exceeds max_seq %d", q, s->pos_host[q], counts[e], d.max_seq); return SWLM_ERR_STATE; }
+        for (int i = 0; i < counts[e]; ++i)
+            if (tokens[n_tok + i] < 0 || tokens[n_tok + i] >= d.vocab) { set_error("entry %d: token %d outside the vocabulary of %d", e, tokens[n_tok + i], d.vocab); return SWLM_ERR_INVALID; }
+        for (int i = 0; want_counts && i < want_counts[e]; ++i)
+            if (wants[n_want + i] < 0 || wants[n_want + i] >= counts[e]) { set_error("entry %d: place %d outside its %d tokens", e, wants[n_want + i], counts[e]); return SWLM_ERR_INVALID; }
+        n_tok += counts[e];
+        n_want += want_counts ? want_counts[e] : 0;
+        const size_t need = (size_t)(s->pos_host[q] + counts[e] + SWLM_PAGE_TOKENS - 1) / SWLM_PAGE_TOKENS;
+        new_pages += need > s->seq_pages[q].size() ? need - s->seq_pages[q].size() : 0;
+    }
+    if (new_pages > s->free_pages.size()) { set_error("the batch needs %zu more pages, %zu are free", new_pages, s->free_pages.size()); return SWLM_ERR_STATE; }
+    for (int e = 0; e < n_entries; ++e)
+        if ((rc = stream_reserve(s, seqs[e], s->pos_host[seqs[e]] + counts[e]))) return rc;
+
+    const size_t vocab = d.vocab;
+    std::vector<float> row_logits;
+    std::vector<int32_t> row_tokens;
+    int e = 0, off = 0;                 // next entry and how many of its tokens have run
+    size_t tok0 = 0, want0 = 0;         // first token and first wanted place of entry e
+    while (e < n_entries) {
+        std::vector<Piece> pieces;
+        std::vector<int32_t> want_rows;
+        std::vector<size_t> slots;      // where a wanted row goes in the outputs
+        int rows = 0;
+        while (e < n_entries && rows < row_cap) {
+            const int take = std::min(row_cap - rows, counts[e] - off);
+            pieces.push_back(Piece{seqs[e], s->pos_host[seqs[e]] + off, take, tokens + tok0 + off});
+            const int nw = want_counts ? want_counts[e] : 0;
+            for (int i = 0; i < nw; ++i)
+                if (wants[want0 + i] >= off && wants[want0 + i] < off + take) { want_rows.push_back(rows + wants[want0 + i] - off); slots.push_back(want0 + i); }
+            rows += take;
+            off += take;
+            if (off == counts[e]) { tok0 += counts[e]; want0 += nw; off = 0; ++e; }
+        }
+        StreamBufs* b = nullptr;
+        if ((rc = run_rows(s, pieces, want_rows, &b))) return rc;
+        const size_t w = want_rows.size();
+        if (w && logits_out) {
+            const size_t pitch = (size_t)s->width[SWLM_BUF_LOGITS] * 4;
+            bool straight = true;
+            for (size_t i = 1; i < w; ++i) straight &= slots[i] == slots[i - 1] + 1;
+            float* dst = logits_out + slots[0] * vocab;
+            if (!straight) { row_logits.resize(w * vocab); dst = row_logits.data(); }
+            SWLM_CUDA(cudaMemcpy2DAsync(dst, vocab * 4, b->buf[SWLM_BUF_LOGITS], pitch, vocab * 4, w, cudaMemcpyDeviceToHost, s->stream));
+            SWLM_CUDA(cudaStreamSynchronize(s->stream));
+            if (!straight) for (size_t i = 0; i < w; ++i) memcpy(logits_out + slots[i] * vocab, row_logits.data() + i * vocab, vocab * 4);
+        }
+        if (w && tokens_out) {
+            row_tokens.resize(w);
+            SWLM_CUDA(cudaMemcpyAsync(row_tokens.data(), b->argmax_out, w * 4, cudaMemcpyDeviceToHost, s->stream));
+            SWLM_CUDA(cudaStreamSynchronize(s->stream));
+            for (size_t i = 0; i < w; ++i) tokens_out[slots[i]] = row_tokens[i];
+        }
+        SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    }
+    for (int q = 0; q < n_entries; ++q) s->pos_host[seqs[q]] += counts[q];
+    SWLM_CUDA(cudaMemcpyAsync(s->position, s->pos_host.data(), sizeof(int32_t) * d.max_batch, cudaMemcpyHostToDevice, s->stream));
+    SWLM_CUDA(cudaStreamSynchronize(s->stream));
+    return stream_check_status(s);
+}
+
+int stream_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_in, int32_t* token_out) {
+    const int m = s->plan->desc.max_batch;
+    swlm_plan tmp;
+    tmp.ctx = s->plan->ctx;
+    tmp.desc = s->plan->desc;
+    tmp.steps.assign(step, step + 1);
+    int rc = stream_compile(&tmp);
+    auto done = [&](int code) { stream_plan_free(&tmp); return code; };
+    if (rc) return done(rc);
+    for (int i = 0; i < SWLM_BUF_COUNT; ++i)
+        if (tmp.stream_width[i] > s->width[i]) { set_error("step: buffer %d is %d wide, the step needs %d", i, s->width[i], tmp.stream_width[i]); return done(SWLM_ERR_INVALID); }
+    for (size_t l = 0; l < tmp.latent.size(); ++l)
+        if (tmp.latent[l].rank && tmp.latent[l].row.pitch != s->plan->latent[l].row.pitch) { set_error("step: latent layer %zu has other rows", l); return done(SWLM_ERR_INVALID); }
+    for (int b = 0; b < m; ++b)
+        if ((rc = stream_reserve(s, b, s->pos_host[b] + 1))) return done(rc);
+    if ((rc = stream_upload_pages(s))) return done(rc);
+    if (token_in) SWLM_CUDA(cudaMemcpyAsync(s->token_in, token_in, sizeof(int32_t) * m, cudaMemcpyHostToDevice, s->stream));
+    stream_drop_graphs(s);   // the step may need more scratch than the graphs were captured with
+    if (s->graph_full) { cudaGraphExecDestroy(s->graph_full); s->graph_full = nullptr; }
+    if (s->graph_body) { cudaGraphExecDestroy(s->graph_body); s->graph_body = nullptr; }
+    swlm_plan* saved = s->plan;
+    RowBatch r = identity_batch(s);
+    r.advance = false;
+    s->plan = &tmp;
+    rc = bufs_scratch(s, &s->dec, r);
+    if (!rc) rc = enqueue_rows_stream(s, &s->dec, r, false, s->stream);
+    s->plan = saved;
+    const cudaError_t e = cudaStreamSynchronize(s->stream);
+    if (rc) return done(rc);
+    if (e != cudaSuccess) return done(cuda_fail(e, "run_step sync"));
+    if (token_out) SWLM_CUDA(cudaMemcpy(token_out, s->dec.argmax_out, sizeof(int32_t) * m, cudaMemcpyDeviceToHost));
+    return done(stream_check_status(s));
+}
+
+void stream_plan_free(swlm_plan* plan) {
+    for (RopeTable& t : plan->rope_tables) cudaFree(t.inv_freq);
+    plan->rope_tables.clear();
+}
+
+}  // namespace swlm

@@ -326,4 +326,112 @@ int launch_tp_rows_allreduce(const TpParams& tp, __nv_bfloat16* x, int x_stride,
 int launch_fill_u32(uint32_t* p, size_t n, uint32_t v, cudaStream_t s);
 int launch_advance(int m, int32_t* position, int32_t* step_counter, cudaStream_t s);
 
+// =====================================================================================================================
+// fp32-stream plans: dense bf16 products, sandwich norms, latent attention over a paged cache
+// =====================================================================================================================
+
+// Dense bf16 matrix [n][k], row pitch ld (k rounded up to 8, the padding is zero).
+struct Matrix {
+    int n = 0, k = 0, ld = 0;
+    __nv_bfloat16* data = nullptr;
+    bool view = false;   // rows of a concatenated matrix that owns the memory
+};
+constexpr int kMaxProductSegs = 4;
+
+// Where a product's rows go: rows [end[q-1], end[q]) to y[q], an fp32 or bf16 buffer [m][stride[q]].
+struct ProductOut {
+    int count = 1;
+    int end[kMaxProductSegs] = {0, 0, 0, 0};
+    void* y[kMaxProductSegs] = {nullptr, nullptr, nullptr, nullptr};
+    int stride[kMaxProductSegs] = {0, 0, 0, 0};
+    int f32[kMaxProductSegs] = {0, 0, 0, 0};
+};
+
+// A norm step over the fp32 stream. mode = its step kind (0: none).
+//   COPY_RMSNORM             h = in
+//   RESADD_*                 h = res_in + in
+//   POSTNORM_*               h = res_in + norm(in; w_post)
+// res_out (unless null) = h; the result is norm(h; w).
+struct StreamNorm {
+    int mode = 0;
+    const float* in = nullptr; int in_stride = 0;
+    const float* res_in = nullptr; float* res_out = nullptr; int res_stride = 0;
+    const __nv_bfloat16* w_post = nullptr;
+    const __nv_bfloat16* w = nullptr;
+    float eps = 0.f, weight_bias = 0.f;
+};
+// rows_idx (may be null): output row r is computed from input row rows_idx[r].
+int launch_stream_norm(const StreamNorm& a, int m, int dim, const int32_t* rows_idx, void* out, int out_stride, bool out_f32, cudaStream_t s);
+// out[r] = table[tok[r]] * scale, fp32
+int launch_stream_embed(int m, int dim, const int32_t* tokens, int vocab, const __nv_bfloat16* table, float scale, float* out, int out_stride, cudaStream_t s);
+int launch_stream_gated(int m, int n, const void* gate, int g_stride, const void* up, int u_stride, void* out, int o_stride, bool f32, int act, cudaStream_t s);
+// argmax over fp32 rows, any m (blocks of kMaxSequences rows); the advancing form of launch_argmax for m <= kMaxSequences
+int launch_argmax_f32(int m, int n, const float* logits, int stride, int32_t* token_out, int32_t* token_in_next, int32_t* ring,
+                      int32_t* step_counter, int ring_cap, int32_t* position, int advance, float* scratch_val, int32_t* scratch_idx, cudaStream_t s);
+
+struct ProductLaunch {
+    const Matrix* w = nullptr;
+    const Matrix* w2 = nullptr;     // gated form: out = act(w x) * (w2 x), rows of both side by side
+    int act = GATED_ACT_SILU;
+    int m = 0;
+    const void* x = nullptr; int x_stride = 0; bool x_f32 = false;   // x_f32: activations fp32, true fp32 products
+    StreamNorm norm;                // x = this norm's result (only when product_takes_norm)
+    ProductOut out;
+    float* part = nullptr; size_t part_floats = 0;   // split-K sums
+    int* status = nullptr;          // device word set when a bounded wait expired
+};
+int bgemm_init();
+int launch_product(const ProductLaunch& a, cudaStream_t s);
+bool product_takes_norm(int m, int k);
+bool product_takes_gate(int m, int k, bool x_f32);
+int product_launch_count(const ProductLaunch& a);
+size_t product_part_floats(int n, int k, int m, bool gated);
+
+// Geometry of one cached latent row: rank latent entries padded to rp, then rot rotated entries padded to rotp; `pitch`
+// entries from row to row (in bf16 pools an odd multiple of 16 bytes, so that eight consecutive rows of a page copied
+// to shared memory as they are lie in different bank groups). Padding entries are zero.
+struct LatentRow { int rank = 0, rot = 0, rp = 0, rotp = 0, pitch = 0; };
+LatentRow latent_row(int rank, int rot, bool f32);
+// Consecutive rows of one sequence inside a batch: rows row0 .. row0 + count - 1 at positions pos0 ..; ctx0 = first of the
+// pos0 + count gathered rows of this span.
+struct LatentSpan { int row0, count, pos0, seq, ctx0; };
+
+struct LatentLaunch {
+    LatentRow row;
+    int heads = 0, dim = 0, vdim = 0, rot_dims = 0;
+    float scale = 1.f, eps = 0.f, weight_bias = 0.f, magnitude = 1.f;
+    const float* inv_freq = nullptr;
+    bool f32 = false;
+    void* q = nullptr; int q_stride = 0;                   // [rows][heads * (dim + rot)]; rotated in place for span rows
+    const float* kv = nullptr; int kv_stride = 0;          // [rows][rank + rot]
+    const float* gate = nullptr; int gate_stride = 0;      // [rows][heads] or null
+    const __nv_bfloat16* norm_w = nullptr;
+    const Matrix* uk = nullptr; const Matrix* uv = nullptr;
+    const Matrix* ukv = nullptr;                           // uk's rows, then uv's
+    void* pool = nullptr;
+    const int32_t* page_table = nullptr; int pages_per_seq = 0;
+    const int32_t* row_seq = nullptr; const int32_t* row_pos = nullptr;
+    void* out = nullptr; int out_stride = 0;
+    // rows that are attended one by one in the latent space (row numbers; null: rows 0 .. n_short - 1)
+    int n_short = 0; const int32_t* short_rows = nullptr; int splits = 1;
+    float* qcat = nullptr; float* partial = nullptr;
+    // rows attended in spans over expanded keys and values: row numbers, the spans, (span, query tile) pairs
+    int n_long = 0; const int32_t* long_rows = nullptr;
+    int n_spans = 0; const LatentSpan* spans = nullptr; int n_tiles = 0; const int2* tiles = nullptr; int total_ctx = 0;
+    unsigned char* expand = nullptr;
+    float* part = nullptr; size_t part_floats = 0;
+    int* status = nullptr;
+    bool only_attention = false;   // timing hook: the attention kernel alone
+};
+int latent_init();
+int latent_pick_splits(int rows, int heads, int max_pages);
+size_t latent_qcat_floats(const LatentRow& r, int heads);              // per row
+size_t latent_partial_floats(const LatentRow& r, int heads);           // per row and split
+size_t latent_expand_bytes(const LatentRow& r, int heads, int dim, int vdim, int total_ctx);
+// can rows of this layer be attended in spans over expanded keys and values?
+bool latent_expands(const LatentRow& r, int dim, int vdim, bool f32);
+constexpr int kLatentQueryTile = 128;
+// launches (for the counters): short part 3, span part 4 or 5
+int launch_latent(const LatentLaunch& a, cudaStream_t s, int* launches);
+
 }  // namespace swlm

@@ -2,7 +2,10 @@
 from __future__ import annotations
 
 import ctypes as C
+import fcntl
 import os
+import subprocess
+import sys
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libswlm_cuda.so")
@@ -46,6 +49,10 @@ class Step(C.Structure):
         ("value_dim", C.c_int32),
         ("weight3", C.c_char * NAME_MAX),
         ("weight4", C.c_char * NAME_MAX),
+        ("rope_factor", C.c_float),
+        ("rope_original", C.c_float),
+        ("rope_fast", C.c_float),
+        ("rope_slow", C.c_float),
     ]
 
 
@@ -72,6 +79,9 @@ class BuffersDesc(C.Structure):
         ("ssm_conv_kernel", C.c_int32),
         ("kv_scheme", C.c_int32),
         ("kv_qjl_dim", C.c_int32),
+        ("stream_dtype", C.c_int32),
+        ("latent_layers", C.c_int32),
+        ("kv_pool_tokens", C.c_int32),
     ]
 
 
@@ -90,6 +100,13 @@ SIGNATURES = {
     "swlm_weights_add_q4g128_staf": (_I, [_P, C.c_char_p, _I, _I, _P, _I]),
     "swlm_weights_add_dense_bf16": (_I, [_P, C.c_char_p, C.c_int64, C.c_int64, _P, _I]),
     "swlm_weights_add_dense_f32": (_I, [_P, C.c_char_p, C.c_int64, _P]),
+    "swlm_weights_add_matrix_bf16": (_I, [_P, C.c_char_p, _I, _I, _P]),
+    "swlm_run_batch": (_I, [_P, _I, _P, _P, _P, _P, _P, _P, _P]),
+    "swlm_pool_free_pages": (_I, [_P]),
+    "swlm_read_logits_f32": (_I, [_P, _P, C.c_size_t]),
+    "swlm_read_buffer_f32": (_I, [_P, _I, _I, _I, _P]),
+    "swlm_write_buffer_f32": (_I, [_P, _I, _I, _I, _P]),
+    "swlm_read_latent": (_I, [_P, _I, _I, _I, _P]),
     "swlm_weights_bytes": (C.c_int64, [_P]),
     "swlm_plan_build": (_I, [_P, C.POINTER(Step), _I, C.POINTER(BuffersDesc), C.POINTER(_P)]),
     "swlm_plan_destroy": (None, [_P]),
@@ -142,6 +159,17 @@ SIGNATURES = {
     "swlm_op_flash_decode_noalloc_capacity": (C.c_size_t, []),
     "swlm_op_flash_decode_noalloc_dev": (_I, [_P, _I, _I, _I, _I, _I, _I, C.c_float, _P, _P, _P, _P, _P]),
 }
+
+
+def build_library() -> str:
+    """Compile libswlm_cuda.so when it is not there yet (make in csrc/, one process at a time) and return its path."""
+    if not os.path.exists(LIB_PATH):
+        csrc = os.path.join(_HERE, "csrc")
+        with open(os.path.join(csrc, ".build.lock"), "w") as lock:
+            fcntl.flock(lock, fcntl.LOCK_EX)
+            if not os.path.exists(LIB_PATH):
+                subprocess.run(["make", "-C", csrc, f"-j{os.cpu_count() or 4}"], check=True, stdout=sys.stderr)
+    return LIB_PATH
 
 
 class Library:

@@ -62,6 +62,13 @@ class WeightStore:
         d = np.ascontiguousarray(data, dtype=np.float32)
         self.lib.check(self.lib.swlm_weights_add_dense_f32(self.handle, name.encode(), d.size, _ptr(d)))
 
+    def add_matrix(self, name: str, data_bf16: np.ndarray) -> None:
+        """Dense bf16 matrix [n][k] of a product (fp32-stream plans)."""
+        d = np.ascontiguousarray(data_bf16, dtype=np.uint16)
+        if d.ndim != 2:
+            raise ValueError(f"{name}: a matrix has two dimensions, not {d.shape}")
+        self.lib.check(self.lib.swlm_weights_add_matrix_bf16(self.handle, name.encode(), d.shape[0], d.shape[1], _ptr(d)))
+
     def add_dense(self, name: str, data_bf16: np.ndarray, shard: int = 0) -> None:
         d = np.ascontiguousarray(data_bf16, dtype=np.uint16)
         rows = d.shape[0] if d.ndim == 2 else 1
@@ -175,6 +182,11 @@ class InferenceModel:
         self.lib.swlm_snap_destroy(snap)
 
     def logits(self) -> np.ndarray:
+        """[batch][vocab] of the last decode step: bf16 bit patterns, or fp32 for an fp32-stream plan."""
+        if self.desc.stream_dtype:
+            out = np.empty((self.batch, int(self.desc.vocab)), dtype=np.float32)
+            self.lib.check(self.lib.swlm_read_logits_f32(self.state, _ptr(out), out.size))
+            return out
         out = np.empty((self.batch, int(self.desc.vocab)), dtype=np.uint16)
         self.lib.check(self.lib.swlm_read_logits(self.state, _ptr(out), out.size))
         return out
@@ -249,6 +261,40 @@ class InferenceModel:
     def reset_sequence(self, seq: int) -> None:
         self.lib.check(self.lib.swlm_state_reset_seq(self.state, seq))
 
+    # -- fp32-stream plans: batches of unequal portions, paged cache -------------------------------------
+    def run_batch(self, entries, logits: bool = True):
+        """Run [(sequence, tokens, wanted places), ...] together (swlm_run_batch). Returns (logits [wanted, vocab] fp32 or None,
+        greedy tokens [wanted]), in the order of the entries and their places."""
+        seqs = np.array([e[0] for e in entries], dtype=np.int32)
+        counts = np.array([len(e[1]) for e in entries], dtype=np.int32)
+        tokens = np.array([t for e in entries for t in e[1]], dtype=np.int32)
+        want_counts = np.array([len(e[2]) for e in entries], dtype=np.int32)
+        wants = np.array([p for e in entries for p in e[2]] or [0], dtype=np.int32)
+        n = int(want_counts.sum())
+        out = np.empty((n, int(self.desc.vocab)), dtype=np.float32) if logits else None
+        greedy = np.empty(max(n, 1), dtype=np.int32)
+        self.lib.check(self.lib.swlm_run_batch(self.state, len(entries), _ptr(seqs), _ptr(counts), _ptr(tokens), _ptr(want_counts), _ptr(wants),
+                                               _ptr(out) if n and logits else None, _ptr(greedy) if n else None))
+        return out, greedy[:n]
+
+    @property
+    def free_pages(self) -> int:
+        return int(self.lib.swlm_pool_free_pages(self.state))
+
+    def read_buffer_f32(self, buf: int, rows: int, count: int) -> np.ndarray:
+        out = np.empty((rows, count), dtype=np.float32)
+        self.lib.check(self.lib.swlm_read_buffer_f32(self.state, buf, rows, count, _ptr(out)))
+        return out
+
+    def write_buffer_f32(self, buf: int, data: np.ndarray) -> None:
+        d = np.ascontiguousarray(data, dtype=np.float32)
+        self.lib.check(self.lib.swlm_write_buffer_f32(self.state, buf, d.shape[0], d.shape[1], _ptr(d)))
+
+    def read_latent(self, layer: int, seq: int, count: int, width: int) -> np.ndarray:
+        out = np.empty((count, width), dtype=np.float32)
+        self.lib.check(self.lib.swlm_read_latent(self.state, layer, seq, count, _ptr(out)))
+        return out
+
     def run_step(self, step: Step, token_in=None) -> np.ndarray:
         tin = None
         if token_in is not None:
@@ -276,16 +322,23 @@ class InferenceModel:
         return buf.value.decode()
 
 
-def load_model(store: WeightStore, builder, weights) -> InferenceModel:
-    """Upload `weights` (name -> arrays, see synth.synth_model_weights) and compile the decode plan."""
+def upload_weights(store: WeightStore, builder, weights) -> None:
+    """`weights` (name -> arrays, see synth.synth_model_weights) into the store."""
     for name, kind, _shape, shard in builder.tensors():
         entry = weights[name]
         if kind == "q4":
             store.add_q4_mlx(name, entry[0], entry[1], entry[2], shard)
         elif kind == "f32":
             store.add_dense_f32(name, entry)
+        elif kind == "matrix":
+            store.add_matrix(name, entry)
         else:
             store.add_dense(name, entry, shard if kind == "conv" else 0)
+
+
+def load_model(store: WeightStore, builder, weights) -> InferenceModel:
+    """Upload `weights` and compile the decode plan."""
+    upload_weights(store, builder, weights)
     return InferenceModel(store, builder.decode_steps(), builder.config.buffers_desc())
 
 

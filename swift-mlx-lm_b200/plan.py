@@ -31,6 +31,14 @@ STEP_CONV_STATE_UPDATE = 9
 STEP_ARGMAX = 10
 STEP_GEGLU = 11
 STEP_SSM_RECURRENCE = 12
+# fp32-stream plans
+STEP_PRODUCT = 13
+STEP_POSTNORM_RESADD_COPY_RMSNORM = 14
+STEP_POSTNORM_RESADD_RMSNORM = 15
+STEP_LATENT_ATTN = 16
+
+STREAM_BF16, STREAM_F32, STREAM_ALL_F32 = 0, 1, 2
+PAGE_TOKENS = 64
 
 SHARD_REPLICATE, SHARD_COLUMN, SHARD_ROW, SHARD_COLUMN3 = 0, 1, 2, 3
 

@@ -44,6 +44,10 @@ def synth_model_weights(builder, seed: int = 3, centered: bool = False, group: i
             out[name] = f32_to_bf16((1.0 + rng.normal(0.0, 0.02, size=shape)).astype(np.float32))
         elif kind == "f32":   # recurrent layers: norm weight ~ 1, A_log ~ U(-1, 1); kept in fp32
             out[name] = (rng.uniform(-1.0, 1.0, size=shape) if name.endswith("A_log") else 1.0 + rng.normal(0.0, 0.02, size=shape)).astype(np.float32)
+        elif kind == "norm0":     # norm weight stored around zero
+            out[name] = f32_to_bf16(rng.normal(0.0, 0.1, size=shape).astype(np.float32))
+        elif kind == "matrix":    # rows of about unit gain
+            out[name] = f32_to_bf16((rng.standard_normal(size=shape, dtype=np.float32) / np.float32(np.sqrt(shape[1]))))
         elif name.endswith("dt_bias"):
             out[name] = f32_to_bf16(rng.normal(0.0, 0.5, size=shape).astype(np.float32))
         elif name.endswith("conv1d.weight"):
