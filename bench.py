@@ -304,6 +304,136 @@ def run_op(args, pkg):
     store.close()
 
 
+VUZUNEX_SHAPES = {   # width, heads, feed-forward, layers: per-layer sizes of real models, fewer layers and a 32768-token vocabulary
+    "1b": (2048, 16, 8192, 16), "8b": (4096, 32, 14336, 8)}
+
+
+def block_weights(builder, seed=3):
+    """Random-init tensors of a builder. Large ones repeat one random block: the values do not matter for the timing, drawing
+    gigabytes of them on the host would take longer than the benchmark."""
+    rng = np.random.default_rng(seed)
+    block = rng.standard_normal(1 << 22, dtype=np.float32)
+    words, sb = rng.integers(0, 1 << 32, size=1 << 21, dtype=np.uint32), rng.uniform(0.005, 0.02, size=1 << 20).astype(np.float32)
+
+    def bf16(x):
+        return (np.ascontiguousarray(x, dtype=np.float32).view(np.uint32) >> 16).astype(np.uint16)
+
+    out = {}
+    for name, kind, shape, _shard in builder.tensors():
+        n = int(np.prod(shape))
+        if kind == "q4":
+            scales = np.resize(sb, n // 64)
+            out[name] = (np.resize(words, n // 8).reshape(shape[0], -1), bf16(scales).reshape(shape[0], -1), bf16(-7.5 * scales).reshape(shape[0], -1))
+        elif kind in ("norm", "norm0"):
+            out[name] = bf16((1.0 if kind == "norm" else 0.0) + 0.02 * block[:n])
+        else:
+            out[name] = bf16(np.resize(block, n) * np.float32(0.02 if kind == "dense" else shape[-1] ** -0.5)).reshape(shape)
+    return out
+
+
+def run_vuzunex(args, pkg):
+    """Prompt and decode throughput of the Vuzunex design (dense bf16 weights, latent attention, fp32 stream) beside the Llama
+    recipe (4-bit weights, grouped-query attention) at equal width, heads, feed-forward, layers and vocabulary. One JSON line."""
+    import torch
+
+    torch.cuda.set_device(0)
+    stream = torch.cuda.Stream()
+    torch.cuda.set_stream(stream)
+    width, heads, ff, layers = VUZUNEX_SHAPES[args.shape]
+    vocab, batch, ctx, P = 32768, args.batch, args.ctx, pkg.plan
+    dim, rot, vdim, rank = 128, 64, 128, 512
+    warm = max(3, args.warmup)
+    max_seq = ctx + 4 * (warm + args.steps) + 64
+    mixer = pkg.vuzunex.LatentAttention(heads, dim, rot, vdim, rank, (dim + rot) ** -0.5, 10000.0, rot, pkg.vuzunex.RotaryScaling(40.0, 4096.0, 32.0, 1.0))
+    vcfg = pkg.VuzunexConfig(vocab=vocab, width=width, layers=[pkg.vuzunex.Layer(mixer, ff, i) for i in range(layers)], max_seq=max_seq, max_batch=batch)
+    lcfg = pkg.ModelConfig("llama", width, ff, layers, heads, heads // 4, 128, vocab, max_seq=max_seq, max_batch=batch)
+    hbm, hbm_src = measured_peaks()
+    tensor, _ = measured_tensor_peak()
+
+    def timed(fn, reps):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record(stream)
+        for _ in range(reps):
+            fn()
+        e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps
+
+    def measure(builder, latent):
+        store = pkg.WeightStore(0)
+        model = pkg.load_model(store, builder, block_weights(builder))
+        model.set_stream(stream.cuda_stream)
+        prompt = np.random.default_rng(7).integers(0, vocab, size=(batch, ctx), dtype=np.int32)
+        seconds = []
+        for _ in range(4):
+            model.reset_state()
+            torch.cuda.synchronize()
+            t0 = time.perf_counter()
+            tok = model.prefill(prompt)
+            seconds.append(time.perf_counter() - t0)
+        sampler = ClockSampler(0)
+        sampler.start()
+        sampler.wait_first(3.0)
+        model.decode_n_async(tok, warm)
+        before = model.launches
+        step_ms = timed(lambda: model.decode_n_async(None, args.steps), 1) / args.steps
+        launches = model.launches - before
+        tok = model.read_tokens(args.steps)[-1]
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        for _ in range(args.steps):
+            tok = model.decode(tok)
+        e2e = batch * args.steps / (time.perf_counter() - t0)
+        clocks = sampler.stop()
+        out = {"prefill_tok_s": batch * ctx / min(seconds[1:]), "decode_tok_s": batch * 1e3 / step_ms, "ms_per_step": step_ms, "e2e_tok_s": e2e,
+               "launches_per_step": model.launches_per_step, "clocks": clocks, "gpu_launches": int(launches)}
+        pos = model.position
+        if batch <= 16 or latent:
+            kind = P.STEP_PRODUCT if latent else P.STEP_QGEMV
+            model.profile_kind(kind, 2)
+            ms = timed(lambda: model.profile_kind(kind, 1), 10)
+            weight_bytes = (vcfg.weight_elems() - layers * heads * (dim + vdim) * rank) * 2 if latent else lcfg.q4_weight_elems() * 0.5625
+            out["decode_products"] = {"ms": ms, "bytes": weight_bytes, "GBs": weight_bytes / ms / 1e6, "frac": weight_bytes / ms / 1e6 / hbm}
+            model.profile_kind(P.STEP_ATTN_DECODE, 2)
+            ms = timed(lambda: model.profile_kind(P.STEP_ATTN_DECODE, 1), 10)
+            kv = layers * batch * pos * (2 * (rank + rot) if latent else lcfg.kv_heads * 128 * 4)
+            out["decode_attention"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv, "GBs": kv / ms / 1e6, "frac": kv / ms / 1e6 / hbm}
+        if latent:
+            ms = timed(lambda: model.profile_kind(P.STEP_LATENT_ATTN, 1), 10)
+            small = layers * heads * (dim + vdim) * rank * 2
+            out["decode_latent_step"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv + small, "frac": (kv + small) / ms / 1e6 / hbm}
+            # one prompt chunk from position 0: products, and the attention kernel alone
+            n = min(ctx, 2048)
+            model.reset_state()
+            chunk = prompt[0, :n]
+            model.profile_batch(0, chunk, P.STEP_PRODUCT, 2)
+            ms = timed(lambda: model.profile_batch(0, chunk, P.STEP_PRODUCT, 5), 1) / 5
+            flops = 2.0 * n * (weight_bytes / 2 - vocab * width)
+            out["prefill_products"] = {"rows": n, "ms": ms, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
+            model.profile_batch(0, chunk, P.STEP_ATTN_DECODE, 2)
+            ms = timed(lambda: model.profile_batch(0, chunk, P.STEP_ATTN_DECODE, 5), 1) / 5
+            flops = layers * heads * n * (n + 1) / 2 * 2.0 * (dim + rot + vdim)
+            out["prefill_attention"] = {"rows": n, "us_per_layer": ms * 1e3 / layers, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
+            ms = timed(lambda: model.profile_batch(0, chunk, P.STEP_LATENT_ATTN, 5), 1) / 5
+            out["prefill_latent_step_us_per_layer"] = ms * 1e3 / layers
+        model.close()
+        store.close()
+        return out
+
+    ours = measure(pkg.VuzunexPlanBuilder(vcfg), True)
+    closest = measure(pkg.DispatchPlanBuilder(lcfg), False)
+    print(json.dumps({
+        "metric": f"decode tok/s, Vuzunex {args.shape} layers bs{batch}", "value": ours["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+        "warmup": warm, "ms_per_step": ours["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+        "dtype": "bf16 weights and activations, fp32 stream and accumulation", "data": "synthetic (random-init weights of the named shape)",
+        "config": {"workload": f"{layers} layers, width {width}, {heads} heads (128 + 64 / 128, latent 512), feed-forward {ff}, vocabulary {vocab}, context {ctx}, batch {batch}",
+                   "l2": "weights larger than L2 are streamed per step", "peak_source": hbm_src},
+        "clocks": ours["clocks"], "gpu_launches": ours["gpu_launches"],
+        "e2e": {"value": ours["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 * batch, "d2h_bytes_per_step": 4 * batch},
+        "vuzunex": ours, "llama_q4_equal_size": closest}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--op", choices=["qgemv", "flash"], default=None, help="op-level line instead of the decode benchmark")
@@ -319,7 +449,9 @@ def main():
     ap.add_argument("--prefill", choices=["real", "synthetic"], default="real",
                     help="how the KV cache gets its `ctx` tokens: by running the prompt, or random bf16 rows")
     ap.add_argument("--small", action="store_true")
-    ap.add_argument("--model", choices=["llama", "lfm2"], default="llama", help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape")
+    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex"], default="llama",
+                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size")
+    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex: which layer sizes")
     ap.add_argument("--batch", type=int, default=1, help="sequences decoded together (1..64), all at the same position")
     ap.add_argument("--kv", choices=["bf16", "q8", "rotor-q4", "rotor-q4-qjl16"], default="bf16",
                     help="KV cache elements: bf16, 8-bit groups of 32 (36-byte blocks), or the rotated 4-bit groups of 64 "
@@ -329,6 +461,9 @@ def main():
     args = ap.parse_args()
     pkg = load_package()
 
+    if args.model == "vuzunex":
+        run_vuzunex(args, pkg)
+        return
     if args.model == "lfm2" and args.ctx == 4096:
         args.ctx = 2048   # the hybrid configuration's prompt length
     if args.batch > 1 and args.prefill == "real":

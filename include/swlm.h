@@ -221,6 +221,10 @@ int64_t swlm_launches(const swlm_state* state);
  * (Sources/MetalCompiler/Execution/MetalDecodeExecutor.swift). */
 int swlm_profile_kind(swlm_state* state, int step_kind, int repeats);
 
+/* The same for a portion of n tokens of one sequence (fp32-stream plans): `repeats` times the launches of one step kind for
+ * these rows, from where the sequence stands, without advancing it (it takes the pages the portion would need). */
+int swlm_profile_batch(swlm_state* state, int seq, const int32_t* tokens, int n, int step_kind, int repeats);
+
 /* ---- tensor parallel: one process per GPU, tp_size of them ----------------------------------------------
  * No counterpart in the reference (single device). Each rank creates its context with (tp_rank, tp_size),
  * uploads the full tensors with a shard kind (the library keeps its slice), builds the same plan and state,

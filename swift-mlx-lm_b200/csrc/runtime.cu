@@ -2301,18 +2301,31 @@ int swlm_shard_range(int shard_kind, int n, int k, int tp_rank, int tp_size, int
     return SWLM_OK;
 }
 
-int swlm_profile_kind(swlm_state* s, int step_kind, int repeats) {
-    if (!s || repeats < 0) { set_error("bad argument"); return SWLM_ERR_INVALID; }
-    int kind;
+static int profiled_launch_kind(int step_kind, int* kind) {
     switch (step_kind) {
-    case SWLM_STEP_QGEMV: kind = L_QGEMV; break;
-    case SWLM_STEP_ATTN_DECODE: kind = L_ATTN; break;   // of a latent step: its attention kernel alone
-    case SWLM_STEP_PRODUCT: kind = L_PRODUCT; break;
-    case SWLM_STEP_LATENT_ATTN: kind = L_LATENT; break;
-    case SWLM_STEP_RESADD_COPY_RMSNORM: kind = L_RMSNORM; break;
+    case SWLM_STEP_QGEMV: *kind = L_QGEMV; break;
+    case SWLM_STEP_ATTN_DECODE: *kind = L_ATTN; break;   // of a latent step: its attention kernel alone
+    case SWLM_STEP_PRODUCT: *kind = L_PRODUCT; break;
+    case SWLM_STEP_LATENT_ATTN: *kind = L_LATENT; break;
+    case SWLM_STEP_RESADD_COPY_RMSNORM: *kind = L_RMSNORM; break;
     default: set_error("profile: step kind %d has no per-kind loop", step_kind); return SWLM_ERR_UNSUPPORTED;
     }
-    int rc = ensure_device(s->plan->ctx);
+    return SWLM_OK;
+}
+
+int swlm_profile_batch(swlm_state* s, int seq, const int32_t* tokens, int n, int step_kind, int repeats) {
+    if (!s || !tokens || n <= 0 || repeats < 0 || !s->plan->stream() || seq < 0 || seq >= s->plan->desc.max_batch) { set_error("bad argument"); return SWLM_ERR_INVALID; }
+    int kind = 0;
+    int rc = profiled_launch_kind(step_kind, &kind);
+    if (!rc) rc = ensure_device(s->plan->ctx);
+    return rc ? rc : stream_profile(s, seq, tokens, n, kind, repeats);
+}
+
+int swlm_profile_kind(swlm_state* s, int step_kind, int repeats) {
+    if (!s || repeats < 0) { set_error("bad argument"); return SWLM_ERR_INVALID; }
+    int kind = 0;
+    int rc = profiled_launch_kind(step_kind, &kind);
+    if (!rc) rc = ensure_device(s->plan->ctx);
     for (int i = 0; i < repeats && !rc; ++i) rc = enqueue_step(s, false, s->stream, kind);
     return rc;
 }

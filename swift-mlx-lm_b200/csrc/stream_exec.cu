@@ -653,14 +653,14 @@ constexpr int kSpanMinRows = 64;
 static_assert(sizeof(LatentSpan) == 20, "spans are staged as five words");
 
 // Rows of `pieces` in one pass; `want_rows` get logits and tokens in b->buf[LOGITS] / b->argmax_out.
-int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<int32_t>& want_rows, StreamBufs** used) {
+int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<int32_t>& want_rows, StreamBufs** used, int only_kind = -1, int repeats = 1) {
     const swlm_plan* plan = s->plan;
     int rows = 0;
     bool single = true;
     for (const Piece& p : pieces) { rows += p.count; single &= p.count == 1; }
     bool every = (int)want_rows.size() == rows;
     for (int i = 0; i < (int)want_rows.size() && every; ++i) every = want_rows[i] == i;
-    const bool graph = single && every && rows <= plan->desc.max_batch;
+    const bool graph = single && every && rows <= plan->desc.max_batch && only_kind < 0;
     StreamBufs* b = graph ? &s->dec : &s->big;
     *used = b;
     int rc;
@@ -747,10 +747,18 @@ int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<
     r.short_rows = b->meta + o_short; r.long_rows = b->meta + o_long;
     r.tiles = reinterpret_cast<const int2*>(b->meta + o_tiles);
     r.spans = reinterpret_cast<const LatentSpan*>(b->meta + o_spans);
-    return enqueue_rows_stream(s, b, r, false, s->stream);
+    for (int i = 0; i < repeats && !rc; ++i) rc = enqueue_rows_stream(s, b, r, false, s->stream, only_kind);
+    return rc;
 }
 
 }  // namespace
+
+int stream_profile(swlm_state* s, int seq, const int32_t* tokens, int n, int only_kind, int repeats) {
+    const int rc = stream_reserve(s, seq, s->pos_host[seq] + n);
+    if (rc) return rc;
+    StreamBufs* b = nullptr;
+    return run_rows(s, {Piece{seq, s->pos_host[seq], n, tokens}}, {}, &b, only_kind, repeats);
+}
 
 int stream_run(swlm_state* s, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, const int32_t* want_counts,
                const int32_t* wants, float* logits_out, int32_t* tokens_out, int row_cap) {

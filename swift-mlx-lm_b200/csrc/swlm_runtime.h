@@ -229,6 +229,7 @@ void stream_drop_graphs(swlm_state* s);
 // the entries of swlm_run_batch, at most row_cap rows at a time
 int stream_run(swlm_state* s, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, const int32_t* want_counts,
                const int32_t* wants, float* logits_out, int32_t* tokens_out, int row_cap);
+int stream_profile(swlm_state* s, int seq, const int32_t* tokens, int n, int only_kind, int repeats);
 int stream_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_in, int32_t* token_out);
 int stream_check_status(swlm_state* s);
 }  // namespace swlm

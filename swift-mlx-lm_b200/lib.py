@@ -145,6 +145,7 @@ SIGNATURES = {
     "swlm_state_reset_seq": (_I, [_P, _I]),
     "swlm_run_step": (_I, [_P, C.POINTER(Step), _P, _P]),
     "swlm_launches": (C.c_int64, [_P]),
+    "swlm_profile_batch": (_I, [_P, _I, _P, _I, _I, _I]),
     "swlm_profile_kind": (_I, [_P, _I, _I]),
     "swlm_tp_export": (_I, [_P, _P]),
     "swlm_tp_attach": (_I, [_P, _P]),

@@ -307,6 +307,10 @@ class InferenceModel:
     def profile_kind(self, step_kind: int, repeats: int) -> None:
         self.lib.check(self.lib.swlm_profile_kind(self.state, step_kind, repeats))
 
+    def profile_batch(self, seq: int, tokens, step_kind: int, repeats: int) -> None:
+        t = np.ascontiguousarray(np.asarray(tokens, dtype=np.int32))
+        self.lib.check(self.lib.swlm_profile_batch(self.state, seq, _ptr(t), t.size, step_kind, repeats))
+
     @property
     def launches_per_step(self) -> int:
         return int(self.lib.swlm_plan_launch_count(self.plan))
