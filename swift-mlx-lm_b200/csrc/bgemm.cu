@@ -389,14 +389,17 @@ __global__ void __launch_bounds__(256) bgemm_sum_kernel(const float* part, int r
     pdl_launch_dependents();
     pdl_wait();
     const size_t total = (size_t)m * n;
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const int r = blockIdx.x * blockDim.x + threadIdx.x;
+    if (r >= n) return;
+    for (int t = blockIdx.y; t < m; t += gridDim.y) {
+        const size_t i = (size_t)t * n + r;
         float a = 0.f, b = 0.f;
+#pragma unroll 4
         for (int z = 0; z < ranges; ++z) {
             const float* base = part + (size_t)z * (GATED ? 2 : 1) * total;
             a += __ldcg(base + i);
             if (GATED) b += __ldcg(base + total + i);
         }
-        const int t = (int)(i / n), r = (int)(i - (size_t)t * n);
         product_store(out, t, r, GATED ? gated_activation(a, b, act) : a);
     }
 }
@@ -494,6 +497,9 @@ struct TcShape { int bn, ranges, split_steps, tiles_m, tiles_n; };
 TcShape tc_shape(int n, int k, int m, bool gated) {
     TcShape t;
     t.bn = m > 128 ? 256 : m > 64 ? 128 : m > 32 ? 64 : 32;
+    // too few tiles to fill the GPU: half as many rows per tile before K is cut
+    const int rows_n = gated ? kTileRows : 2 * kTileRows;
+    if (t.bn == 256 && (m + 255) / 256 * ((n + rows_n - 1) / rows_n) < 100) t.bn = 128;
     t.tiles_m = (m + t.bn - 1) / t.bn;
     t.tiles_n = (n + (gated ? kTileRows : 2 * kTileRows) - 1) / (gated ? kTileRows : 2 * kTileRows);
     const int steps = (k + kTcK - 1) / kTcK, tiles = t.tiles_m * t.tiles_n;
@@ -526,9 +532,9 @@ int tc_launch(const ProductLaunch& a, const TcShape& t, cudaStream_t s) {
                           : launch_k(bgemm_tc_kernel<BN, STAGES, false>, grid, dim3(kTcBlock), tc_smem<BN, STAGES>(), s, p, xmap, wmap, wmap2);
     if (e != cudaSuccess) return cuda_fail(e, "bgemm launch");
     if (t.ranges > 1) {
-        const unsigned g = (unsigned)std::min<size_t>(592, ((size_t)p.m * p.n + 255) / 256);
-        e = gated ? launch_k(bgemm_sum_kernel<true>, dim3(g), dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out)
-                  : launch_k(bgemm_sum_kernel<false>, dim3(g), dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out);
+        const dim3 g((unsigned)((p.n + 255) / 256), (unsigned)std::min(p.m, 64));
+        e = gated ? launch_k(bgemm_sum_kernel<true>, g, dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out)
+                  : launch_k(bgemm_sum_kernel<false>, g, dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out);
         if (e != cudaSuccess) return cuda_fail(e, "bgemm sum launch");
     }
     return SWLM_OK;

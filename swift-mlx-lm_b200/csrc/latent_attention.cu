@@ -23,6 +23,7 @@ namespace swlm {
 namespace {
 
 constexpr int kPage = SWLM_PAGE_TOKENS;
+constexpr int kPartialTail = 4;   // behind a partial's rp sums: running maximum, sum of weights, padding to 16 bytes
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float lat_get(const float* p) { return *p; }
@@ -65,12 +66,26 @@ struct LatentParams {
     int n_rows; const int32_t* rows;     // the rows of this launch; null: 0 .. n_rows - 1
     int splits;
     float* qcat; float* partial;
+    int frag;                            // qcat holds bf16 hi + lo fragments of the tensor-core kernel instead of fp32 rows
     int* status;
     // spans
     const LatentSpan* spans; const int2* tiles; int n_spans, total_ctx;
     __nv_bfloat16* ctx_latent; __nv_bfloat16* ctx_rot; int ctx_ld, rot_ld;
     const __nv_bfloat16* ctx_k; const __nv_bfloat16* ctx_v;
 };
+
+// Entry (row of the launch, head, column) of the queries. As fragments: per 16 heads and 16 columns, lane (g, t) holds 8 words:
+// the four words of an m16n8k16 A fragment from the high bf16 halves, then the four from the low ones.
+__device__ __forceinline__ void store_query(const LatentParams& p, int rl, int h, int col, float v) {
+    const int qw = p.row.rp + p.row.rotp;
+    if (!p.frag) { p.qcat[((size_t)rl * p.heads + h) * qw + col] = v; return; }
+    const int tiles = (p.heads + 15) >> 4, hr = h & 15, k = col & 15;
+    const int lane = (hr & 7) * 4 + ((k & 7) >> 1), word = (hr >> 3) + 2 * (k >> 3);
+    __nv_bfloat16* d = reinterpret_cast<__nv_bfloat16*>(p.qcat) + ((((size_t)rl * tiles + (h >> 4)) * (qw >> 4) + (col >> 4)) * 32 + lane) * 16 + word * 2 + (k & 1);
+    const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+    d[0] = hi;
+    d[8] = __float2bfloat16_rn(v - __bfloat162float(hi));
+}
 
 __device__ __forceinline__ int batch_row(const LatentParams& p, int i) { return p.rows ? p.rows[i] : i; }
 template <typename T>
@@ -96,103 +111,164 @@ __device__ __forceinline__ float rotated(const LatentParams& p, const V& x, int 
 }
 
 // The row a warp appends: norm of the latent, rotation of the shared key part, zeros in the padding.
+constexpr int kAppendRegs = 16;   // latent entries per lane that are read once
 template <typename T>
 __device__ __forceinline__ void append_row(const LatentParams& p, int r, int lane) {
     const float* src = p.kv + (size_t)r * p.kv_stride;
-    const int pos = p.row_pos[r];
-    T* dst = cached_row<T>(p, p.row_seq[r], pos);
+    const int pos = p.row_pos[r], seq = p.row_seq[r];
+    float v[kAppendRegs];
     float ss = 0.f;
-    for (int i = lane; i < p.row.rank; i += 32) { const float v = src[i]; ss = fmaf(v, v, ss); }
+#pragma unroll
+    for (int j = 0; j < kAppendRegs; ++j) { const int i = lane + 32 * j; v[j] = i < p.row.rank ? src[i] : 0.f; }
+    T* dst = cached_row<T>(p, seq, pos);
+#pragma unroll
+    for (int j = 0; j < kAppendRegs; ++j) ss = fmaf(v[j], v[j], ss);
+    for (int i = lane + 32 * kAppendRegs; i < p.row.rank; i += 32) { const float x = src[i]; ss = fmaf(x, x, ss); }
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const float sc = 1.0f / sqrtf(ss / (float)p.row.rank + p.eps);
-    for (int i = lane; i < p.row.rp; i += 32)
+#pragma unroll
+    for (int j = 0; j < kAppendRegs; ++j) {
+        const int i = lane + 32 * j;
+        if (i < p.row.rp) lat_put(dst + i, i < p.row.rank ? v[j] * sc * (__bfloat162float(p.norm_w[i]) + p.weight_bias) : 0.f);
+    }
+    for (int i = lane + 32 * kAppendRegs; i < p.row.rp; i += 32)
         lat_put(dst + i, i < p.row.rank ? src[i] * sc * (__bfloat162float(p.norm_w[i]) + p.weight_bias) : 0.f);
     const float* rot = src + p.row.rank;
     auto at = [&](int i) { return rot[i]; };
     for (int i = lane; i < p.row.pitch - p.row.rp; i += 32) lat_put(dst + p.row.rp + i, i < p.row.rot ? rotated(p, at, pos, i) : 0.f);
 }
 
+// The same by a CTA of 256 threads: everything that does not depend on something else is requested at once.
+constexpr int kAppendThreads = 256;
+template <typename T>
+__device__ __forceinline__ void append_row_cta(const LatentParams& p, int r, float* red) {
+    const int tid = threadIdx.x, half = p.row.rp;
+    const float* src = p.kv + (size_t)r * p.kv_stride;
+    const int pos = p.row_pos[r], seq = p.row_seq[r];
+    float v[2], w[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int i = tid + kAppendThreads * j;
+        v[j] = i < p.row.rank ? src[i] : 0.f;
+        w[j] = i < p.row.rank ? __bfloat162float(p.norm_w[i]) + p.weight_bias : 0.f;
+    }
+    const float* rot = src + p.row.rank;
+    auto at = [&](int i) { return rot[i]; };
+    const int tail = p.row.pitch - p.row.rp;
+    const float turned = tid < p.row.rot ? rotated(p, at, pos, tid) : 0.f;
+    T* dst = cached_row<T>(p, seq, pos);
+    float ss = fmaf(v[0], v[0], v[1] * v[1]);
+    for (int i = tid + 2 * kAppendThreads; i < p.row.rank; i += kAppendThreads) { const float x = src[i]; ss = fmaf(x, x, ss); }
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kAppendThreads / 32; ++i) ss += red[i];
+    __syncthreads();
+    const float sc = 1.0f / sqrtf(ss / (float)p.row.rank + p.eps);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int i = tid + kAppendThreads * j;
+        if (i < half) lat_put(dst + i, v[j] * sc * w[j]);
+    }
+    for (int i = tid + 2 * kAppendThreads; i < half; i += kAppendThreads)
+        lat_put(dst + i, i < p.row.rank ? src[i] * sc * (__bfloat162float(p.norm_w[i]) + p.weight_bias) : 0.f);
+    if (tid < tail) lat_put(dst + half + tid, turned);
+    for (int i = tid + kAppendThreads; i < tail; i += kAppendThreads) lat_put(dst + half + i, i < p.row.rot ? rotated(p, at, pos, i) : 0.f);
+}
+
 // ---- rows one by one: queries -----------------------------------------------------------------------------------------
-// CTA (h < heads, group of kQueryRows rows): absorbed query of one head, qcat[row][h] = [W_uk^T q_plain | rotated part], fp32,
-// padding zero. CTA h == heads: the rows' own latents go to the cache.
-constexpr int kQueryRows = 4, kQueryThreads = 256;
+// CTA (h < heads, group of kQueryRows rows, 128 latent columns): absorbed query of one head, qcat[row][h] =
+// [W_uk^T q_plain | rotated part], fp32, padding zero (the CTA of the first columns adds rotated part and padding). Thread
+// (group g of 16, chunk of 8 columns): rows d = g, g + 16, ... of the head's key projection; the first batch of them is read
+// before the preceding kernel has finished. CTA h == heads: the rows' own latents go to the cache.
+constexpr int kQueryRows = 4, kQueryThreads = 256, kQueryChunks = 16, kQueryGroups = kQueryThreads / kQueryChunks, kQueryBatch = 8;
 template <typename T>
 __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const LatentParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) float query_smem[];
     const int tid = threadIdx.x, h = blockIdx.x, r0 = blockIdx.y * kQueryRows;
     const int nr = min(kQueryRows, p.n_rows - r0);
-    if (h < p.heads) {
-        // this head's rows of the key projection do not depend on the preceding kernel: bring them into L2
-        const char* w = reinterpret_cast<const char*>(p.uk + (size_t)h * p.dim * p.uk_ld);
-        const size_t bytes = (size_t)p.dim * p.uk_ld * 2;
-        for (size_t o = (size_t)tid * 128; o < bytes; o += (size_t)kQueryThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-    }
-    pdl_wait();
     if (h == p.heads) {
-        for (int i = tid >> 5; i < nr; i += kQueryThreads / 32) append_row<T>(p, batch_row(p, r0 + i), tid & 31);
+        static_assert(kQueryThreads == kAppendThreads, "a CTA appends a row");
+        pdl_wait();
+        for (int i = blockIdx.z; i < nr; i += gridDim.z) append_row_cta<T>(p, batch_row(p, r0 + i), query_smem);
         return;
     }
+    const int cc = tid % kQueryChunks, g = tid / kQueryChunks, chunk = blockIdx.z * kQueryChunks + cc;
+    const bool live = chunk < (p.uk_ld >> 3);
+    const __nv_bfloat16* w = p.uk + (size_t)h * p.dim * p.uk_ld + 8 * (live ? chunk : 0);
+    uint4 wv[kQueryBatch];
+    auto load = [&](int d0) {
+#pragma unroll
+        for (int u = 0; u < kQueryBatch; ++u) {
+            const int d = d0 + u * kQueryGroups;
+            wv[u] = live && d < p.dim ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)d * p.uk_ld)) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    load(g);
+    pdl_wait();
     const int per_head = p.dim + p.row.rot, qw = p.row.rp + p.row.rotp;
-    float* qs = query_smem;                              // [kQueryRows][per_head]
-    float* acc_s = query_smem + kQueryRows * per_head;   // [groups][kQueryRows][8] per chunk column
+    float* qs = query_smem;                                          // [kQueryRows][per_head]
+    float* acc_s = query_smem + (kQueryRows * per_head + 3) / 4 * 4; // [groups][kQueryRows][chunks * 8]
     for (int i = tid; i < nr * per_head; i += kQueryThreads) {
         const int rr = i / per_head, c = i - rr * per_head;
         qs[rr * per_head + c] = lat_get(static_cast<const T*>(p.q) + (size_t)batch_row(p, r0 + rr) * p.q_stride + (size_t)h * per_head + c);
     }
     __syncthreads();
-    // rotated part and padding
-    for (int i = tid; i < nr * (qw - p.row.rank); i += kQueryThreads) {
-        const int rr = i / (qw - p.row.rank), c = p.row.rank + i - rr * (qw - p.row.rank);
-        const int rc = c - p.row.rp;
-        const float* x = qs + rr * per_head + p.dim;
-        auto at = [&](int e) { return x[e]; };
-        p.qcat[((size_t)(r0 + rr) * p.heads + h) * qw + c] = rc >= 0 && rc < p.row.rot ? rotated(p, at, p.row_pos[batch_row(p, r0 + rr)], rc) : 0.f;
+    if (blockIdx.z == 0) {
+        for (int i = tid; i < nr * (qw - p.row.rank); i += kQueryThreads) {
+            const int rr = i / (qw - p.row.rank), c = p.row.rank + i - rr * (qw - p.row.rank);
+            const int rc = c - p.row.rp;
+            const float* x = qs + rr * per_head + p.dim;
+            auto at = [&](int e) { return x[e]; };
+            const float v = rc >= 0 && rc < p.row.rot ? rotated(p, at, p.row_pos[batch_row(p, r0 + rr)], rc) : 0.f;
+            store_query(p, r0 + rr, h, c, v);
+        }
     }
-    // absorbed part: 8 latent columns per thread, the dim rows dealt to the thread groups
-    const int chunks = p.uk_ld >> 3;
-    const int cols = min(chunks, kQueryThreads);                   // chunk columns per pass
-    const int groups = max(1, min(kQueryThreads / cols, 8)), g = tid / cols, cc = tid - g * cols;
-    for (int c0 = 0; c0 < chunks; c0 += cols) {
-        float acc[kQueryRows][8];
+    float acc[kQueryRows][8];
 #pragma unroll
-        for (int rr = 0; rr < kQueryRows; ++rr)
+    for (int rr = 0; rr < kQueryRows; ++rr)
 #pragma unroll
-            for (int e = 0; e < 8; ++e) acc[rr][e] = 0.f;
-        const int c = c0 + cc;
-        if (g < groups && c < chunks) {
-            const __nv_bfloat16* w = p.uk + (size_t)h * p.dim * p.uk_ld + 8 * c;
-#pragma unroll 8
-            for (int d = g; d < p.dim; d += groups) {
-                const uint4 v = __ldg(reinterpret_cast<const uint4*>(w + (size_t)d * p.uk_ld));
+        for (int e = 0; e < 8; ++e) acc[rr][e] = 0.f;
+    for (int d0 = g; d0 < p.dim; d0 += kQueryBatch * kQueryGroups) {
+        if (d0 != g) load(d0);
+#pragma unroll
+        for (int u = 0; u < kQueryBatch; ++u) {
+            const int d = d0 + u * kQueryGroups;
+            if (d < p.dim) {
+                const uint4 v = wv[u];
                 const float wf[8] = {lat_lo(v.x), lat_hi(v.x), lat_lo(v.y), lat_hi(v.y), lat_lo(v.z), lat_hi(v.z), lat_lo(v.w), lat_hi(v.w)};
 #pragma unroll
                 for (int rr = 0; rr < kQueryRows; ++rr) {
-                    const float x = rr < nr ? qs[rr * per_head + d] : 0.f;
+                    if (rr < nr) {
+                        const float x = qs[rr * per_head + d];
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) acc[rr][e] = fmaf(x, wf[e], acc[rr][e]);
+                        for (int e = 0; e < 8; ++e) acc[rr][e] = fmaf(x, wf[e], acc[rr][e]);
+                    }
                 }
             }
         }
-        if (g < groups) {
+    }
+    constexpr int COLS = kQueryChunks * 8;
+    for (int rr = 0; rr < kQueryRows; ++rr) {
+        float4* d = reinterpret_cast<float4*>(acc_s + (size_t)(g * kQueryRows + rr) * COLS + cc * 8);
 #pragma unroll
-            for (int rr = 0; rr < kQueryRows; ++rr)
+        for (int r = 0; r < kQueryRows; ++r)
+            if (r == rr) { d[0] = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]); d[1] = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]); }
+    }
+    __syncthreads();
+    for (int i = tid; i < nr * COLS; i += kQueryThreads) {
+        const int rr = i / COLS, col = i - rr * COLS, c = blockIdx.z * COLS + col;
+        float v = 0.f;
 #pragma unroll
-                for (int e = 0; e < 8; ++e) acc_s[((size_t)(g * kQueryRows + rr) * cols + cc) * 8 + e] = acc[rr][e];
-        }
-        __syncthreads();
-        for (int i = tid; i < nr * cols * 8; i += kQueryThreads) {
-            const int rr = i / (cols * 8), col = i - rr * cols * 8;
-            float v = 0.f;
-            for (int q = 0; q < groups; ++q) v += acc_s[(size_t)(q * kQueryRows + rr) * cols * 8 + col];
-            if (c0 * 8 + col < p.row.rank) p.qcat[((size_t)(r0 + rr) * p.heads + h) * qw + c0 * 8 + col] = v;
-        }
-        __syncthreads();
+        for (int q = 0; q < kQueryGroups; ++q) v += acc_s[(size_t)(q * kQueryRows + rr) * COLS + col];
+        if (c < p.row.rank) store_query(p, r0 + rr, h, c, v);
     }
 }
 size_t query_smem_bytes(const LatentLaunch& a) {
-    const int chunks = a.uk->ld / 8, cols = std::min(chunks, kQueryThreads), groups = std::max(1, std::min(kQueryThreads / cols, 8));
-    return ((size_t)kQueryRows * (a.dim + a.row.rot) + (size_t)groups * kQueryRows * cols * 8) * 4;
+    return ((size_t)(kQueryRows * (a.dim + a.row.rot) + 3) / 4 * 4 + (size_t)kQueryGroups * kQueryRows * kQueryChunks * 8) * 4;
 }
 
 // ---- rows one by one: attention on tensor cores (bf16 pool) -----------------------------------------------------------
@@ -224,16 +300,17 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
     }
     __syncthreads();
     pdl_wait();
-    const int r = batch_row(p, rl), pos = p.row_pos[r];
+    const int r = batch_row(p, rl), pos = p.row_pos[r], seq = p.row_seq[r];
+    const int32_t* table = p.page_table + (size_t)seq * p.pages_per_seq;
+    const int first_page = table[split];   // (within the table whatever the position: splits <= pages_per_seq)
     const int n_pages = pos / kPage + 1;
     if (split >= n_pages) return;
-    const int32_t* table = p.page_table + (size_t)p.row_seq[r] * p.pages_per_seq;
     const int mine = (n_pages - split + p.splits - 1) / p.splits;
     auto request = [&](int i) {   // thread 0: the i-th page of this CTA
         const unsigned bar = smem_u32(&full_bar[i & 1]);
         mbar_expect(bar, (unsigned)page_bytes);
         bulk_load(smem_u32(pages + (size_t)(i & 1) * page_bytes),
-                  static_cast<const unsigned char*>(p.pool) + (size_t)table[split + i * p.splits] * page_bytes, (unsigned)page_bytes, bar);
+                  static_cast<const unsigned char*>(p.pool) + (size_t)(i == 0 ? first_page : table[split + i * p.splits]) * page_bytes, (unsigned)page_bytes, bar);
     };
     if (tid == 0) { request(0); if (mine > 1) request(1); }
 
@@ -242,20 +319,15 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
     const int qw = p.row.rp + p.row.rotp, ksteps = qw >> 4;
     unsigned qh[KPW][4], ql[KPW][4];
     {
-        const float* q0 = p.qcat + ((size_t)rl * p.heads + min(h0 + g, p.heads - 1)) * qw;
-        const float* q1 = p.qcat + ((size_t)rl * p.heads + min(h0 + g + 8, p.heads - 1)) * qw;
+        // (heads past the last one hold whatever was there: their results are dropped)
+        const uint4* f = reinterpret_cast<const uint4*>(p.qcat) + (((size_t)rl * gridDim.y + blockIdx.y) * ksteps * 32 + lane) * 2;
 #pragma unroll
         for (int k = 0; k < KPW; ++k) {
             const int ks = kq * KPW + k;
-            float2 v[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                v[e] = make_float2(0.f, 0.f);
-                if (ks < ksteps) v[e] = __ldcg(reinterpret_cast<const float2*>(((e & 1) ? q1 : q0) + 16 * ks + 2 * t + ((e & 2) ? 8 : 0)));
-                const float a = lat_round(v[e].x), b = lat_round(v[e].y);
-                qh[k][e] = lat_pack(a, b);
-                ql[k][e] = lat_pack(v[e].x - a, v[e].y - b);
-            }
+            const uint4 zero = make_uint4(0, 0, 0, 0);
+            const uint4 hi = ks < ksteps ? __ldcg(f + (size_t)ks * 64) : zero, lo = ks < ksteps ? __ldcg(f + (size_t)ks * 64 + 1) : zero;
+            qh[k][0] = hi.x; qh[k][1] = hi.y; qh[k][2] = hi.z; qh[k][3] = hi.w;
+            ql[k][0] = lo.x; ql[k][1] = lo.y; ql[k][2] = lo.z; ql[k][3] = lo.w;
         }
     }
     float oacc[NPW][2][4];
@@ -365,7 +437,7 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
         if (tid == 0) for (int i = 0; i < 2 && i < mine; ++i) mbar_wait(&full_bar[i], 0u);
         return;
     }
-    const size_t pw = (size_t)p.row.rp + 2;
+    const size_t pw = (size_t)p.row.rp + kPartialTail;
     float* po = p.partial + ((size_t)rl * p.heads * p.splits + split) * pw;
 #pragma unroll
     for (int j = 0; j < NPW; ++j) {
@@ -419,7 +491,7 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) latent_simple_kernel(const 
     for (int w = 1; w < kSimpleWarps; ++w) top = fmaxf(top, ms[w]);
     float total = 0.f;
     for (int w = 0; w < kSimpleWarps; ++w) total += ls[w] * exp2f(ms[w] - top);
-    float* po = p.partial + ((size_t)rl * p.heads + h) * ((size_t)p.row.rp + 2);
+    float* po = p.partial + ((size_t)rl * p.heads + h) * ((size_t)p.row.rp + kPartialTail);
     for (int i = threadIdx.x; i < p.row.rp; i += blockDim.x) {
         float v = 0.f;
         for (int w = 0; w < kSimpleWarps; ++w) v += simple_smem[qw + (size_t)w * p.row.rp + i] * exp2f(ms[w] - top);
@@ -429,61 +501,114 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) latent_simple_kernel(const 
 }
 
 // ---- rows one by one: merge, value projection, gate --------------------------------------------------------------------
-constexpr int kOutThreads = 256, kLatMaxSplits = 296;
+constexpr int kOutThreads = 512, kLatMaxSplits = 296, kOutBatch = 16, kOutRows = 4;
 template <typename T>
 __global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const LatentParams p) {
-    extern __shared__ __align__(16) float out_smem[];   // [uv_ld]
+    extern __shared__ __align__(16) float out_smem[];   // [rp] merged, then [groups][rp] the thread groups' shares
     __shared__ float w_s[kLatMaxSplits];
     pdl_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, rl = blockIdx.y;
     const int per = (p.vdim + gridDim.z - 1) / gridDim.z, v0 = blockIdx.z * per, v1 = min(p.vdim, v0 + per);
-    {
-        const char* w = reinterpret_cast<const char*>(p.uv + ((size_t)h * p.vdim + v0) * p.uv_ld);
-        const size_t bytes = v1 > v0 ? (size_t)(v1 - v0) * p.uv_ld * 2 : 0;
-        for (size_t o = (size_t)tid * 128; o < bytes; o += (size_t)kOutThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-    }
+    // value projection rows v0 + warp, + 16, ... of this warp, their first 512 columns: not the preceding kernel's business
+    const int chunks = p.uv_ld >> 3;
+    uint4 wv[kOutRows][2];
+#pragma unroll
+    for (int j = 0; j < kOutRows; ++j)
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+            const int v = v0 + warp + j * (kOutThreads / 32), cq = lane + 32 * q;
+            wv[j][q] = v < v1 && cq < chunks ? __ldg(reinterpret_cast<const uint4*>(p.uv + ((size_t)h * p.vdim + v) * p.uv_ld + 8 * cq)) : make_uint4(0, 0, 0, 0);
+        }
     pdl_wait();
     const int r = batch_row(p, rl);
     const int used = min(p.splits, p.row_pos[r] / kPage + 1);
-    const size_t pw = (size_t)p.row.rp + 2;
+    const size_t pw = (size_t)p.row.rp + kPartialTail;
     const float* base = p.partial + ((size_t)rl * p.heads + h) * p.splits * pw;
+    // four columns per thread, the splits dealt to groups of threads; the first sums are requested before the weights are known
+    const int quads = p.row.rp >> 2, cols = min(quads, kOutThreads), groups = kOutThreads / cols, g = tid / cols, c = tid - g * cols;
+    float4 first[kOutBatch];
+#pragma unroll
+    for (int u = 0; u < kOutBatch; ++u) {
+        const int s = g + u * groups;
+        first[u] = g < groups && s < used ? __ldcg(reinterpret_cast<const float4*>(base + s * pw) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     if (warp == 0) {
+        float2 ml[(kLatMaxSplits + 31) / 32];
         float top = -INFINITY;
-        for (int s = lane; s < used; s += 32) top = fmaxf(top, __ldcg(base + s * pw + p.row.rp));
+#pragma unroll
+        for (int j = 0; j < (kLatMaxSplits + 31) / 32; ++j) {
+            const int s = lane + 32 * j;
+            ml[j] = s < used ? __ldcg(reinterpret_cast<const float2*>(base + s * pw + p.row.rp)) : make_float2(-INFINITY, 0.f);
+            top = fmaxf(top, ml[j].x);
+        }
         for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
         float total = 0.f;
-        for (int s = lane; s < used; s += 32) {
-            const float w = exp2f(__ldcg(base + s * pw + p.row.rp) - top);
-            w_s[s] = w;
-            total += w * __ldcg(base + s * pw + p.row.rp + 1);
-        }
+#pragma unroll
+        for (int j = 0; j < (kLatMaxSplits + 31) / 32; ++j) { ml[j].x = exp2f(ml[j].x - top); total = fmaf(ml[j].x, ml[j].y, total); }
         for (int o = 16; o > 0; o >>= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
         const float inv = 1.0f / total;
-        __syncwarp();
-        for (int s = lane; s < used; s += 32) w_s[s] *= inv;
+#pragma unroll
+        for (int j = 0; j < (kLatMaxSplits + 31) / 32; ++j) { const int s = lane + 32 * j; if (s < used) w_s[s] = ml[j].x * inv; }
     }
     __syncthreads();
-    for (int i = tid; i < p.uv_ld; i += kOutThreads) {
-        float v = 0.f;
-        if (i < p.row.rank) {
-#pragma unroll 8
-            for (int s = 0; s < used; ++s) v = fmaf(w_s[s], __ldcg(base + s * pw + i), v);
+    float* merged = out_smem;
+    float4* shares = reinterpret_cast<float4*>(out_smem + p.row.rp);
+    for (int c0 = 0; c0 < quads; c0 += cols) {
+        if (g < groups && c0 + c < quads) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int s0 = g; s0 < used; s0 += kOutBatch * groups) {
+                if (c0 > 0 || s0 != g) {
+#pragma unroll
+                    for (int u = 0; u < kOutBatch; ++u) {
+                        const int s = s0 + u * groups;
+                        first[u] = s < used ? __ldcg(reinterpret_cast<const float4*>(base + s * pw) + c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    }
+                }
+#pragma unroll
+                for (int u = 0; u < kOutBatch; ++u) {
+                    const int s = s0 + u * groups;
+                    if (s < used) {
+                        const float w = w_s[s];
+                        v.x = fmaf(w, first[u].x, v.x); v.y = fmaf(w, first[u].y, v.y); v.z = fmaf(w, first[u].z, v.z); v.w = fmaf(w, first[u].w, v.w);
+                    }
+                }
+            }
+            shares[g * quads + c0 + c] = v;
         }
-        out_smem[i] = v;
+    }
+    __syncthreads();
+    for (int i = tid; i < p.row.rp; i += kOutThreads) {
+        float v = 0.f;
+        for (int q = 0; q < groups; ++q) v += reinterpret_cast<const float*>(shares)[(size_t)q * p.row.rp + i];
+        merged[i] = v;
     }
     __syncthreads();
     const float gate = p.gate ? 1.0f / (1.0f + expf(-p.gate[(size_t)r * p.gate_stride + h])) : 1.0f;
-    for (int v = v0 + warp; v < v1; v += kOutThreads / 32) {
-        const __nv_bfloat16* w = p.uv + ((size_t)h * p.vdim + v) * p.uv_ld;
-        float acc = 0.f;
-        for (int c = lane; c < (p.uv_ld >> 3); c += 32) {
-            const uint4 x = __ldg(reinterpret_cast<const uint4*>(w + 8 * c));
-            const float4 a = *reinterpret_cast<const float4*>(out_smem + 8 * c), b = *reinterpret_cast<const float4*>(out_smem + 8 * c + 4);
-            acc = fmaf(lat_lo(x.x), a.x, acc); acc = fmaf(lat_hi(x.x), a.y, acc); acc = fmaf(lat_lo(x.y), a.z, acc); acc = fmaf(lat_hi(x.y), a.w, acc);
-            acc = fmaf(lat_lo(x.z), b.x, acc); acc = fmaf(lat_hi(x.z), b.y, acc); acc = fmaf(lat_lo(x.w), b.z, acc); acc = fmaf(lat_hi(x.w), b.w, acc);
-        }
+    auto dot = [&](const uint4& x, int cq) {
+        const float4 a = *reinterpret_cast<const float4*>(out_smem + 8 * cq), b = *reinterpret_cast<const float4*>(out_smem + 8 * cq + 4);
+        float acc = lat_lo(x.x) * a.x;
+        acc = fmaf(lat_hi(x.x), a.y, acc); acc = fmaf(lat_lo(x.y), a.z, acc); acc = fmaf(lat_hi(x.y), a.w, acc);
+        acc = fmaf(lat_lo(x.z), b.x, acc); acc = fmaf(lat_hi(x.z), b.y, acc); acc = fmaf(lat_lo(x.w), b.z, acc);
+        return fmaf(lat_hi(x.w), b.w, acc);
+    };
+    auto finish = [&](int v, float acc) {
         for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
         if (lane == 0) lat_put(static_cast<T*>(p.out) + (size_t)r * p.out_stride + (size_t)h * p.vdim + v, acc * gate);
+    };
+#pragma unroll
+    for (int j = 0; j < kOutRows; ++j) {
+        const int v = v0 + warp + j * (kOutThreads / 32);
+        if (v >= v1) break;   // uniform across the warp
+        float acc = 0.f;
+#pragma unroll
+        for (int q = 0; q < 2; ++q) if (lane + 32 * q < chunks) acc += dot(wv[j][q], lane + 32 * q);
+        for (int cq = lane + 64; cq < chunks; cq += 32) acc += dot(__ldg(reinterpret_cast<const uint4*>(p.uv + ((size_t)h * p.vdim + v) * p.uv_ld + 8 * cq)), cq);
+        finish(v, acc);
+    }
+    for (int v = v0 + warp + kOutRows * (kOutThreads / 32); v < v1; v += kOutThreads / 32) {
+        float acc = 0.f;
+        for (int cq = lane; cq < chunks; cq += 32) acc += dot(__ldg(reinterpret_cast<const uint4*>(p.uv + ((size_t)h * p.vdim + v) * p.uv_ld + 8 * cq)), cq);
+        finish(v, acc);
     }
 }
 
@@ -690,6 +815,8 @@ LatentParams latent_params(const LatentLaunch& a) {
     return p;
 }
 
+size_t out_smem_bytes(const LatentRow& r) { const int quads = r.rp / 4, cols = std::min(quads, kOutThreads); return (size_t)(1 + kOutThreads / cols) * r.rp * 4; }
+
 constexpr int kSplKpwSmall = 3, kSplNpwSmall = 2, kSplKpw = 9, kSplNpw = 4;
 bool split_small(const LatentRow& r) { return (r.rp + r.rotp) / 16 <= 4 * kSplKpwSmall && r.rp / 16 <= kSplWarps * kSplNpwSmall; }
 bool split_fits(const LatentRow& r) { return (r.rp + r.rotp) / 16 <= 4 * kSplKpw && r.rp / 16 <= kSplWarps * kSplNpw; }
@@ -703,9 +830,10 @@ int launch_short(const LatentLaunch& a, cudaStream_t s, int* launches) {
     p.n_rows = a.n_short; p.rows = a.short_rows; p.splits = a.splits;
     cudaError_t e;
     const bool mma = !a.f32 && split_fits(a.row);
+    p.frag = mma ? 1 : 0;
     if (!mma) p.splits = 1;
     if (!a.only_attention) {
-        const dim3 qg(a.heads + 1, (a.n_short + kQueryRows - 1) / kQueryRows);
+        const dim3 qg(a.heads + 1, (a.n_short + kQueryRows - 1) / kQueryRows, (a.uk->ld / 8 + kQueryChunks - 1) / kQueryChunks);
         e = launch_k(latent_query_kernel<T>, qg, dim3(kQueryThreads), query_smem_bytes(a), s, p);
         if (e != cudaSuccess) return cuda_fail(e, "latent query launch");
         *launches += 1;
@@ -720,8 +848,8 @@ int launch_short(const LatentLaunch& a, cudaStream_t s, int* launches) {
     if (e != cudaSuccess) return cuda_fail(e, "latent attention launch");
     *launches += 1;
     if (!a.only_attention) {
-        const int vs = std::max(1, std::min(148 / std::max(1, a.heads * a.n_short), (a.vdim + 15) / 16));
-        e = launch_k(latent_out_kernel<T>, dim3(a.heads, a.n_short, vs), dim3(kOutThreads), (size_t)a.uv->ld * 4, s, p);
+        const int vs = std::max(1, std::min(64 / std::max(1, a.heads * a.n_short), (a.vdim + 15) / 16));
+        e = launch_k(latent_out_kernel<T>, dim3(a.heads, a.n_short, vs), dim3(kOutThreads), out_smem_bytes(a.row), s, p);
         if (e != cudaSuccess) return cuda_fail(e, "latent output launch");
         *launches += 1;
     }
@@ -800,6 +928,8 @@ int latent_init() {
     SWLM_CUDA(cudaFuncSetAttribute(latent_simple_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSimpleMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    SWLM_CUDA(cudaFuncSetAttribute(latent_out_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
+    SWLM_CUDA(cudaFuncSetAttribute(latent_out_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
     SWLM_CUDA(cudaFuncSetAttribute(latent_prefill_kernel<4, 5>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_prefill_smem<4, 5>()));
     SWLM_CUDA(cudaFuncSetAttribute(latent_prefill_kernel<8, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_prefill_smem<8, 8>()));
     SWLM_CUDA(cudaFuncSetAttribute(latent_prefill_kernel<12, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_prefill_smem<12, 8>()));
@@ -811,8 +941,8 @@ int latent_pick_splits(int rows, int heads, int max_pages) {
     const int per_split = rows * ((heads + kSplHeads - 1) / kSplHeads);
     return std::max(1, std::min(std::min(148 / std::max(1, per_split), max_pages), kLatMaxSplits));
 }
-size_t latent_qcat_floats(const LatentRow& r, int heads) { return (size_t)heads * (r.rp + r.rotp); }
-size_t latent_partial_floats(const LatentRow& r, int heads) { return (size_t)heads * (r.rp + 2); }
+size_t latent_qcat_floats(const LatentRow& r, int heads) { return (size_t)(heads + 15) / 16 * 16 * (r.rp + r.rotp); }
+size_t latent_partial_floats(const LatentRow& r, int heads) { return (size_t)heads * (r.rp + kPartialTail); }
 size_t latent_expand_bytes(const LatentRow& r, int heads, int dim, int vdim, int total_ctx) { return expand_layout(r, heads, dim, vdim, total_ctx).total; }
 bool latent_expands(const LatentRow& r, int dim, int vdim, bool f32) {
     return !f32 && !((dim | vdim | r.rot | r.rank) & 7) && prefill_form(dim, r.rot, vdim) != PF_NONE;

@@ -1373,7 +1373,14 @@ int swlm_weights_add_dense_bf16(swlm_ctx* ctx, const char* name, int64_t rows, i
     auto old = ctx->dense.find(name);
     if (old != ctx->dense.end()) {
         SWLM_CUDA(cudaDeviceSynchronize());
+        // the same shape: new values in the old place, so that plans compiled against the tensor stay valid; another shape
+        // replaces it, and those plans must be rebuilt
+        if (old->second.rows == sl.rows && old->second.cols == cols && old->second.shard_kind == shard_kind) {
+            SWLM_CUDA(cudaMemcpy(old->second.data, data + (size_t)sl.row0 * cols, (size_t)sl.rows * cols * 2, cudaMemcpyHostToDevice));
+            return SWLM_OK;
+        }
         cudaFree(old->second.data);
+        ctx->bytes -= old->second.rows * old->second.cols * 2;
         ctx->dense.erase(old);
     }
     DenseTensor t;
@@ -1391,7 +1398,12 @@ int swlm_weights_add_dense_f32(swlm_ctx* ctx, const char* name, int64_t count, c
     auto old = ctx->densef.find(name);
     if (old != ctx->densef.end()) {
         SWLM_CUDA(cudaDeviceSynchronize());
+        if (old->second.count == count) {   // in place, as above
+            SWLM_CUDA(cudaMemcpy(old->second.data, data, (size_t)count * 4, cudaMemcpyHostToDevice));
+            return SWLM_OK;
+        }
         cudaFree(old->second.data);
+        ctx->bytes -= old->second.count * 4;
         ctx->densef.erase(old);
     }
     DenseF32 t;

@@ -198,6 +198,7 @@ int stream_compile(swlm_plan* plan) {
             if (!act_buf(plan, s.in_buf) || !stored_f32(plan, s.in2_buf) || !any_buf(s.in2_buf) || !act_buf(plan, s.out_buf) || s.out_buf == s.in_buf ||
                 (s.in3_buf != SWLM_BUF_NONE && (!any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf)))) { set_error("latent attention: q and the result in scratch 0..2, latent and gate in scratch 3 and 4"); return SWLM_ERR_INVALID; }
             if ((rc = find_vector(ctx, s.weight, s.n, &L.d1))) return rc;
+            if (s.n > 8192 || s.head_dim + s.key_dim > 4096) { set_error("latent attention: latent of %d, query of %d entries per head", s.n, s.head_dim + s.key_dim); return SWLM_ERR_UNSUPPORTED; }
             const Matrix *uk, *uv;
             if ((rc = find_matrix(ctx, s.weight2, s.heads * s.head_dim, s.n, &uk)) || (rc = find_matrix(ctx, s.weight3, s.heads * s.value_dim, s.n, &uv))) return rc;
             const Matrix* both;

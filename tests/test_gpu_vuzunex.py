@@ -198,7 +198,7 @@ def test_single_keys_at_page_and_tile_borders(pkg, load, dtype, name):
             return real(s)
 
         plain.causal_softmax = without_own
-        assert np.median(vc.row_errors(m.plain(tokens), want)[1:]) > 2.5 * limit
+        assert (vc.row_errors(m.plain(tokens), want)[1:] > 2.5 * limit).sum() > 10
     finally:
         plain.causal_softmax = real
 
