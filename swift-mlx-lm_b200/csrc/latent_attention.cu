@@ -13,11 +13,16 @@
 // Scores, softmax and sums are fp32. Where tensor cores take fp32 quantities (absorbed queries, softmax weights) these enter
 // as bf16 hi + lo pairs. The newest rows are read back from the cache like all others, so a row's result does not depend on
 // how a sequence was cut into batches.
+#include <cooperative_groups.h>
+
 #include <algorithm>
 #include <cstdlib>
+#include <utility>
 
 #include "swlm_internal.h"
 #include "tc_device.cuh"
+
+namespace cg = cooperative_groups;
 
 namespace swlm {
 namespace {
@@ -104,10 +109,10 @@ template <typename V>
 __device__ __forceinline__ float rotated(const LatentParams& p, const V& x, int pos, int i) {
     const int half = p.rot_dims >> 1;
     if (i >= p.rot_dims) return x(i);
+    const bool low = i < half;
     float c, s;
-    if (i < half) { angle(p, pos, i, c, s); return x(i) * c - x(i + half) * s; }
-    angle(p, pos, i - half, c, s);
-    return x(i) * c + x(i - half) * s;
+    angle(p, pos, low ? i : i - half, c, s);
+    return low ? x(i) * c - x(i + half) * s : x(i) * c + x(i - half) * s;
 }
 
 // The row a warp appends: norm of the latent, rotation of the shared key part, zeros in the padding.
@@ -179,17 +184,17 @@ __device__ __forceinline__ void append_row_cta(const LatentParams& p, int r, flo
 }
 
 // ---- rows one by one: queries -----------------------------------------------------------------------------------------
-// CTA (h < heads, group of kQueryRows rows, 128 latent columns): absorbed query of one head, qcat[row][h] =
+// CTA (h < heads, group of MR rows, 128 latent columns): absorbed query of one head, qcat[row][h] =
 // [W_uk^T q_plain | rotated part], fp32, padding zero (the CTA of the first columns adds rotated part and padding). Thread
 // (group g of 16, chunk of 8 columns): rows d = g, g + 16, ... of the head's key projection; the first batch of them is read
 // before the preceding kernel has finished. CTA h == heads: the rows' own latents go to the cache.
-constexpr int kQueryRows = 4, kQueryThreads = 256, kQueryChunks = 16, kQueryGroups = kQueryThreads / kQueryChunks, kQueryBatch = 8;
-template <typename T>
+constexpr int kQueryThreads = 256, kQueryChunks = 16, kQueryGroups = kQueryThreads / kQueryChunks, kQueryBatch = 8;
+template <typename T, int MR>
 __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const LatentParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) float query_smem[];
-    const int tid = threadIdx.x, h = blockIdx.x, r0 = blockIdx.y * kQueryRows;
-    const int nr = min(kQueryRows, p.n_rows - r0);
+    const int tid = threadIdx.x, h = blockIdx.x, r0 = blockIdx.y * MR;
+    const int nr = min(MR, p.n_rows - r0);
     if (h == p.heads) {
         static_assert(kQueryThreads == kAppendThreads, "a CTA appends a row");
         pdl_wait();
@@ -210,8 +215,8 @@ __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const Laten
     load(g);
     pdl_wait();
     const int per_head = p.dim + p.row.rot, qw = p.row.rp + p.row.rotp;
-    float* qs = query_smem;                                          // [kQueryRows][per_head]
-    float* acc_s = query_smem + (kQueryRows * per_head + 3) / 4 * 4; // [groups][kQueryRows][chunks * 8]
+    float* qs = query_smem;                                          // [MR][per_head]
+    float* acc_s = query_smem + (MR * per_head + 3) / 4 * 4; // [groups][MR][chunks * 8]
     for (int i = tid; i < nr * per_head; i += kQueryThreads) {
         const int rr = i / per_head, c = i - rr * per_head;
         qs[rr * per_head + c] = lat_get(static_cast<const T*>(p.q) + (size_t)batch_row(p, r0 + rr) * p.q_stride + (size_t)h * per_head + c);
@@ -227,9 +232,9 @@ __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const Laten
             store_query(p, r0 + rr, h, c, v);
         }
     }
-    float acc[kQueryRows][8];
+    float acc[MR][8];
 #pragma unroll
-    for (int rr = 0; rr < kQueryRows; ++rr)
+    for (int rr = 0; rr < MR; ++rr)
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[rr][e] = 0.f;
     for (int d0 = g; d0 < p.dim; d0 += kQueryBatch * kQueryGroups) {
@@ -241,7 +246,7 @@ __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const Laten
                 const uint4 v = wv[u];
                 const float wf[8] = {lat_lo(v.x), lat_hi(v.x), lat_lo(v.y), lat_hi(v.y), lat_lo(v.z), lat_hi(v.z), lat_lo(v.w), lat_hi(v.w)};
 #pragma unroll
-                for (int rr = 0; rr < kQueryRows; ++rr) {
+                for (int rr = 0; rr < MR; ++rr) {
                     if (rr < nr) {
                         const float x = qs[rr * per_head + d];
 #pragma unroll
@@ -252,23 +257,26 @@ __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const Laten
         }
     }
     constexpr int COLS = kQueryChunks * 8;
-    for (int rr = 0; rr < kQueryRows; ++rr) {
-        float4* d = reinterpret_cast<float4*>(acc_s + (size_t)(g * kQueryRows + rr) * COLS + cc * 8);
 #pragma unroll
-        for (int r = 0; r < kQueryRows; ++r)
-            if (r == rr) { d[0] = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]); d[1] = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]); }
+    for (int rr = 0; rr < MR; ++rr) {
+        float4* d = reinterpret_cast<float4*>(acc_s + (size_t)(g * MR + rr) * COLS + cc * 8);
+        d[0] = make_float4(acc[rr][0], acc[rr][1], acc[rr][2], acc[rr][3]);
+        d[1] = make_float4(acc[rr][4], acc[rr][5], acc[rr][6], acc[rr][7]);
     }
     __syncthreads();
     for (int i = tid; i < nr * COLS; i += kQueryThreads) {
         const int rr = i / COLS, col = i - rr * COLS, c = blockIdx.z * COLS + col;
         float v = 0.f;
 #pragma unroll
-        for (int q = 0; q < kQueryGroups; ++q) v += acc_s[(size_t)(q * kQueryRows + rr) * COLS + col];
+        for (int q = 0; q < kQueryGroups; ++q) v += acc_s[(size_t)(q * MR + rr) * COLS + col];
         if (c < p.row.rank) store_query(p, r0 + rr, h, c, v);
     }
 }
-size_t query_smem_bytes(const LatentLaunch& a) {
-    return ((size_t)(kQueryRows * (a.dim + a.row.rot) + 3) / 4 * 4 + (size_t)kQueryGroups * kQueryRows * kQueryChunks * 8) * 4;
+template <typename T, int MR>
+cudaError_t launch_query(const LatentLaunch& a, const LatentParams& p, cudaStream_t s) {
+    const size_t smem = ((size_t)(MR * (a.dim + a.row.rot) + 3) / 4 * 4 + (size_t)kQueryGroups * MR * kQueryChunks * 8) * 4;
+    const dim3 grid(a.heads + 1, (a.n_short + MR - 1) / MR, (a.uk->ld / 8 + kQueryChunks - 1) / kQueryChunks);
+    return launch_k(latent_query_kernel<T, MR>, grid, dim3(kQueryThreads), smem, s, p);
 }
 
 // ---- rows one by one: attention on tensor cores (bf16 pool) -----------------------------------------------------------
@@ -501,88 +509,77 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) latent_simple_kernel(const 
 }
 
 // ---- rows one by one: merge, value projection, gate --------------------------------------------------------------------
-constexpr int kOutThreads = 512, kLatMaxSplits = 296, kOutBatch = 16, kOutRows = 4;
+// A cluster of CTAs per (head, row): each merges its share of the latent columns over the splits and hands it to the others
+// through distributed shared memory, then multiplies its share of the head's value rows.
+constexpr int kOutThreads = 256, kOutWarps = kOutThreads / 32, kLatMaxSplits = 296, kOutBatch = 4, kOutRows = 2, kOutCluster = 8;
 template <typename T>
 __global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const LatentParams p) {
-    extern __shared__ __align__(16) float out_smem[];   // [rp] merged, then [groups][rp] the thread groups' shares
+    extern __shared__ __align__(16) float out_smem[];   // [rp] merged, then [groups][share] the thread groups' sums
     __shared__ float w_s[kLatMaxSplits];
+    const cg::cluster_group cluster = cg::this_cluster();
+    auto started = cluster.barrier_arrive();   // waited for before anything is written to another CTA's shared memory
     pdl_launch_dependents();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, rl = blockIdx.y;
-    const int per = (p.vdim + gridDim.z - 1) / gridDim.z, v0 = blockIdx.z * per, v1 = min(p.vdim, v0 + per);
-    // value projection rows v0 + warp, + 16, ... of this warp, their first 512 columns: not the preceding kernel's business
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, rl = blockIdx.y, z = blockIdx.z, nz = gridDim.z;
+    const int per = (p.vdim + nz - 1) / nz, v0 = z * per, v1 = min(p.vdim, v0 + per);
+    // value rows v0 + warp, + 8, ... of this warp, their first 512 columns: not the preceding kernel's business
     const int chunks = p.uv_ld >> 3;
+    const __nv_bfloat16* rows = p.uv + (size_t)h * p.vdim * p.uv_ld;
     uint4 wv[kOutRows][2];
 #pragma unroll
     for (int j = 0; j < kOutRows; ++j)
 #pragma unroll
         for (int q = 0; q < 2; ++q) {
-            const int v = v0 + warp + j * (kOutThreads / 32), cq = lane + 32 * q;
-            wv[j][q] = v < v1 && cq < chunks ? __ldg(reinterpret_cast<const uint4*>(p.uv + ((size_t)h * p.vdim + v) * p.uv_ld + 8 * cq)) : make_uint4(0, 0, 0, 0);
+            const int v = v0 + warp + j * kOutWarps, cq = lane + 32 * q;
+            wv[j][q] = v < v1 && cq < chunks ? __ldg(reinterpret_cast<const uint4*>(rows + (size_t)v * p.uv_ld) + cq) : make_uint4(0, 0, 0, 0);
         }
     pdl_wait();
     const int r = batch_row(p, rl);
     const int used = min(p.splits, p.row_pos[r] / kPage + 1);
     const size_t pw = (size_t)p.row.rp + kPartialTail;
     const float* base = p.partial + ((size_t)rl * p.heads + h) * p.splits * pw;
-    // four columns per thread, the splits dealt to groups of threads; the first sums are requested before the weights are known
-    const int quads = p.row.rp >> 2, cols = min(quads, kOutThreads), groups = kOutThreads / cols, g = tid / cols, c = tid - g * cols;
-    float4 first[kOutBatch];
-#pragma unroll
-    for (int u = 0; u < kOutBatch; ++u) {
-        const int s = g + u * groups;
-        first[u] = g < groups && s < used ? __ldcg(reinterpret_cast<const float4*>(base + s * pw) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
     if (warp == 0) {
-        float2 ml[(kLatMaxSplits + 31) / 32];
         float top = -INFINITY;
-#pragma unroll
-        for (int j = 0; j < (kLatMaxSplits + 31) / 32; ++j) {
-            const int s = lane + 32 * j;
-            ml[j] = s < used ? __ldcg(reinterpret_cast<const float2*>(base + s * pw + p.row.rp)) : make_float2(-INFINITY, 0.f);
-            top = fmaxf(top, ml[j].x);
-        }
+        for (int s = lane; s < used; s += 32) top = fmaxf(top, __ldcg(base + s * pw + p.row.rp));
         for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
         float total = 0.f;
-#pragma unroll
-        for (int j = 0; j < (kLatMaxSplits + 31) / 32; ++j) { ml[j].x = exp2f(ml[j].x - top); total = fmaf(ml[j].x, ml[j].y, total); }
+        for (int s = lane; s < used; s += 32) {
+            const float2 ml = __ldcg(reinterpret_cast<const float2*>(base + s * pw + p.row.rp));
+            const float w = exp2f(ml.x - top);
+            w_s[s] = w;
+            total = fmaf(w, ml.y, total);
+        }
         for (int o = 16; o > 0; o >>= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
         const float inv = 1.0f / total;
-#pragma unroll
-        for (int j = 0; j < (kLatMaxSplits + 31) / 32; ++j) { const int s = lane + 32 * j; if (s < used) w_s[s] = ml[j].x * inv; }
+        __syncwarp();
+        for (int s = lane; s < used; s += 32) w_s[s] *= inv;
     }
     __syncthreads();
-    float* merged = out_smem;
-    float4* shares = reinterpret_cast<float4*>(out_smem + p.row.rp);
-    for (int c0 = 0; c0 < quads; c0 += cols) {
-        if (g < groups && c0 + c < quads) {
+    // this CTA's latent columns, four per thread, the splits dealt to groups of threads
+    const int quads = p.row.rp >> 2, share = (quads + nz - 1) / nz, q0 = z * share, nq = max(0, min(share, quads - q0));
+    const int cols = min(share, kOutThreads), groups = kOutThreads / cols, g = tid / cols, c = tid - g * cols;
+    float4* sums = reinterpret_cast<float4*>(out_smem + p.row.rp);
+    for (int c0 = 0; c0 < nq; c0 += cols) {
+        if (g < groups && c0 + c < nq) {
+            const float* src = base + 4 * (q0 + c0 + c);
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int s0 = g; s0 < used; s0 += kOutBatch * groups) {
-                if (c0 > 0 || s0 != g) {
-#pragma unroll
-                    for (int u = 0; u < kOutBatch; ++u) {
-                        const int s = s0 + u * groups;
-                        first[u] = s < used ? __ldcg(reinterpret_cast<const float4*>(base + s * pw) + c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-                    }
-                }
-#pragma unroll
-                for (int u = 0; u < kOutBatch; ++u) {
-                    const int s = s0 + u * groups;
-                    if (s < used) {
-                        const float w = w_s[s];
-                        v.x = fmaf(w, first[u].x, v.x); v.y = fmaf(w, first[u].y, v.y); v.z = fmaf(w, first[u].z, v.z); v.w = fmaf(w, first[u].w, v.w);
-                    }
-                }
+#pragma unroll kOutBatch
+            for (int s = g; s < used; s += groups) {
+                const float4 x = __ldcg(reinterpret_cast<const float4*>(src + s * pw));
+                const float w = w_s[s];
+                v.x = fmaf(w, x.x, v.x); v.y = fmaf(w, x.y, v.y); v.z = fmaf(w, x.z, v.z); v.w = fmaf(w, x.w, v.w);
             }
-            shares[g * quads + c0 + c] = v;
+            sums[g * share + c0 + c] = v;
         }
     }
     __syncthreads();
-    for (int i = tid; i < p.row.rp; i += kOutThreads) {
+    cluster.barrier_wait(std::move(started));
+    for (int i = tid; i < nq * 4; i += kOutThreads) {
         float v = 0.f;
-        for (int q = 0; q < groups; ++q) v += reinterpret_cast<const float*>(shares)[(size_t)q * p.row.rp + i];
-        merged[i] = v;
+        for (int q = 0; q < groups; ++q) v += reinterpret_cast<const float*>(sums)[(size_t)q * share * 4 + i];
+        out_smem[q0 * 4 + i] = v;
+        for (int o = 1; o < nz; ++o) cluster.map_shared_rank(out_smem, (z + o) % nz)[q0 * 4 + i] = v;
     }
-    __syncthreads();
+    cluster.sync();
     const float gate = p.gate ? 1.0f / (1.0f + expf(-p.gate[(size_t)r * p.gate_stride + h])) : 1.0f;
     auto dot = [&](const uint4& x, int cq) {
         const float4 a = *reinterpret_cast<const float4*>(out_smem + 8 * cq), b = *reinterpret_cast<const float4*>(out_smem + 8 * cq + 4);
@@ -597,19 +594,43 @@ __global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const LatentPar
     };
 #pragma unroll
     for (int j = 0; j < kOutRows; ++j) {
-        const int v = v0 + warp + j * (kOutThreads / 32);
-        if (v >= v1) break;   // uniform across the warp
-        float acc = 0.f;
+        const int v = v0 + warp + j * kOutWarps;
+        if (v < v1) {   // uniform across the warp
+            float acc = 0.f;
 #pragma unroll
-        for (int q = 0; q < 2; ++q) if (lane + 32 * q < chunks) acc += dot(wv[j][q], lane + 32 * q);
-        for (int cq = lane + 64; cq < chunks; cq += 32) acc += dot(__ldg(reinterpret_cast<const uint4*>(p.uv + ((size_t)h * p.vdim + v) * p.uv_ld + 8 * cq)), cq);
-        finish(v, acc);
+            for (int q = 0; q < 2; ++q) if (lane + 32 * q < chunks) acc += dot(wv[j][q], lane + 32 * q);
+            for (int cq = lane + 64; cq < chunks; cq += 32) acc += dot(__ldg(reinterpret_cast<const uint4*>(rows + (size_t)v * p.uv_ld) + cq), cq);
+            finish(v, acc);
+        }
     }
-    for (int v = v0 + warp + kOutRows * (kOutThreads / 32); v < v1; v += kOutThreads / 32) {
+#pragma unroll 1
+    for (int v = v0 + warp + kOutRows * kOutWarps; v < v1; v += kOutWarps) {
         float acc = 0.f;
-        for (int cq = lane; cq < chunks; cq += 32) acc += dot(__ldg(reinterpret_cast<const uint4*>(p.uv + ((size_t)h * p.vdim + v) * p.uv_ld + 8 * cq)), cq);
+        for (int cq = lane; cq < chunks; cq += 32) acc += dot(__ldg(reinterpret_cast<const uint4*>(rows + (size_t)v * p.uv_ld) + cq), cq);
         finish(v, acc);
     }
+}
+// CTAs per (head, row): as many as the portable cluster size while the launch stays below four CTAs per SM
+int out_cluster(int heads, int rows, int vdim) {
+    int nz = kOutCluster;
+    while (nz > 1 && ((long long)heads * rows * nz > 4 * 148 || nz > vdim)) nz >>= 1;
+    return nz;
+}
+template <typename T>
+cudaError_t launch_out(const LatentLaunch& a, const LatentParams& p, cudaStream_t s) {
+    const int nz = out_cluster(a.heads, a.n_short, a.vdim);
+    const int share = (a.row.rp / 4 + nz - 1) / nz, cols = std::min(share, kOutThreads), groups = kOutThreads / cols;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.heads, a.n_short, nz); cfg.blockDim = dim3(kOutThreads); cfg.stream = s;
+    cfg.dynamicSmemBytes = ((size_t)a.row.rp + (size_t)groups * share * 4) * 4;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = 1; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = nz;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl_enabled() ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, latent_out_kernel<T>, p);
 }
 
 // ---- spans: append and rotate ------------------------------------------------------------------------------------------
@@ -815,8 +836,6 @@ LatentParams latent_params(const LatentLaunch& a) {
     return p;
 }
 
-size_t out_smem_bytes(const LatentRow& r) { const int quads = r.rp / 4, cols = std::min(quads, kOutThreads); return (size_t)(1 + kOutThreads / cols) * r.rp * 4; }
-
 constexpr int kSplKpwSmall = 3, kSplNpwSmall = 2, kSplKpw = 9, kSplNpw = 4;
 bool split_small(const LatentRow& r) { return (r.rp + r.rotp) / 16 <= 4 * kSplKpwSmall && r.rp / 16 <= kSplWarps * kSplNpwSmall; }
 bool split_fits(const LatentRow& r) { return (r.rp + r.rotp) / 16 <= 4 * kSplKpw && r.rp / 16 <= kSplWarps * kSplNpw; }
@@ -833,8 +852,7 @@ int launch_short(const LatentLaunch& a, cudaStream_t s, int* launches) {
     p.frag = mma ? 1 : 0;
     if (!mma) p.splits = 1;
     if (!a.only_attention) {
-        const dim3 qg(a.heads + 1, (a.n_short + kQueryRows - 1) / kQueryRows, (a.uk->ld / 8 + kQueryChunks - 1) / kQueryChunks);
-        e = launch_k(latent_query_kernel<T>, qg, dim3(kQueryThreads), query_smem_bytes(a), s, p);
+        e = a.n_short == 1 ? launch_query<T, 1>(a, p, s) : launch_query<T, 4>(a, p, s);
         if (e != cudaSuccess) return cuda_fail(e, "latent query launch");
         *launches += 1;
     }
@@ -848,8 +866,7 @@ int launch_short(const LatentLaunch& a, cudaStream_t s, int* launches) {
     if (e != cudaSuccess) return cuda_fail(e, "latent attention launch");
     *launches += 1;
     if (!a.only_attention) {
-        const int vs = std::max(1, std::min(64 / std::max(1, a.heads * a.n_short), (a.vdim + 15) / 16));
-        e = launch_k(latent_out_kernel<T>, dim3(a.heads, a.n_short, vs), dim3(kOutThreads), out_smem_bytes(a.row), s, p);
+        e = launch_out<T>(a, p, s);
         if (e != cudaSuccess) return cuda_fail(e, "latent output launch");
         *launches += 1;
     }
@@ -926,8 +943,10 @@ int latent_init() {
     SWLM_CUDA(cudaFuncSetAttribute(latent_split_kernel<kSplKpw, kSplNpw>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     SWLM_CUDA(cudaFuncSetAttribute(latent_simple_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSimpleMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(latent_simple_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSimpleMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<float, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    SWLM_CUDA(cudaFuncSetAttribute(latent_query_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     SWLM_CUDA(cudaFuncSetAttribute(latent_out_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
     SWLM_CUDA(cudaFuncSetAttribute(latent_out_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
     SWLM_CUDA(cudaFuncSetAttribute(latent_prefill_kernel<4, 5>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_prefill_smem<4, 5>()));
