@@ -74,7 +74,7 @@ __device__ __forceinline__ void get_x8(const __nv_bfloat16* p, float (&f)[8]) {
 
 // A warp takes groups of four weight rows (GATED: two of gate and the same two of up); WK warps share a group and cut K.
 template <typename T, int MR, int WK, bool GATED>
-__global__ void __launch_bounds__(kGemvThreads) bgemv_kernel(const GemvParams p) {
+__global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char gemv_raw[];
     __shared__ float red[kGemvWarps];
@@ -105,13 +105,74 @@ __global__ void __launch_bounds__(kGemvThreads) bgemv_kernel(const GemvParams p)
     };
     const int first_chunk = kw * 32 + lane;
     int group = blockIdx.x * per_cta + rg;
-    // the first weights do not depend on the preceding kernel
+    // the first weights (and a norm's) do not depend on the preceding kernel
     if (group < groups) load(group, first_chunk);
+    // a norm over at most 4096 entries keeps its row in registers: entries 4 tid + 1024 j
+    const bool norm_regs = p.norm.mode && p.k <= 16 * kGemvThreads && (p.k & 3) == 0;
+    uint2 nw[4], npw[4];
+    if (norm_regs) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = 4 * tid + 4 * kGemvThreads * j;
+            nw[j] = i < p.k ? __ldg(reinterpret_cast<const uint2*>(p.norm.w + i)) : make_uint2(0, 0);
+            npw[j] = i < p.k && p.norm.w_post ? __ldg(reinterpret_cast<const uint2*>(p.norm.w_post + i)) : make_uint2(0, 0);
+        }
+    }
     pdl_wait();
 
     // ---- activations to shared memory: plain rows, or the norm in front of the product (every CTA computes it; CTA 0 stores
     // the new residual) ----
-    if (p.norm.mode) {
+    if (norm_regs) {
+        for (int m = 0; m < MR; ++m) {
+            T* xr = xs + (size_t)m * p.ld;
+            const float* in = p.norm.in + (size_t)m * p.norm.in_stride;
+            const float* res = p.norm.res_in ? p.norm.res_in + (size_t)m * p.norm.res_stride : nullptr;
+            float h[4][4], rv[4][4];
+            float ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int i = 4 * tid + 4 * kGemvThreads * j;
+                const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 a = i < p.k ? __ldcg(reinterpret_cast<const float4*>(in + i)) : z, b = i < p.k && res ? __ldcg(reinterpret_cast<const float4*>(res + i)) : z;
+                h[j][0] = a.x; h[j][1] = a.y; h[j][2] = a.z; h[j][3] = a.w;
+                rv[j][0] = b.x; rv[j][1] = b.y; rv[j][2] = b.z; rv[j][3] = b.w;
+            }
+            if (p.norm.w_post) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) ss = fmaf(h[j][e], h[j][e], ss);
+                const float sc = 1.0f / sqrtf(cta_sum(ss, red) / (float)p.k + p.norm.eps);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float wf[4] = {b_lo(npw[j].x), b_hi(npw[j].x), b_lo(npw[j].y), b_hi(npw[j].y)};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) h[j][e] = h[j][e] * sc * (wf[e] + p.norm.weight_bias);
+                }
+            }
+            ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) { h[j][e] += rv[j][e]; ss = fmaf(h[j][e], h[j][e], ss); }
+            // (entries past k: zero input, zero residual)
+            const float sc = 1.0f / sqrtf(cta_sum(ss, red) / (float)p.k + p.norm.eps);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int i = 4 * tid + 4 * kGemvThreads * j;
+                const float wf[4] = {b_lo(nw[j].x), b_hi(nw[j].x), b_lo(nw[j].y), b_hi(nw[j].y)};
+                if (i < p.k) {
+                    if (p.norm.res_out && blockIdx.x == 0)
+                        *reinterpret_cast<float4*>(p.norm.res_out + (size_t)m * p.norm.res_stride + i) = make_float4(h[j][0], h[j][1], h[j][2], h[j][3]);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) put_x(xr + i + e, h[j][e] * sc * (wf[e] + p.norm.weight_bias));
+                } else if (i < p.ld) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) put_x(xr + i + e, 0.f);
+                }
+            }
+        }
+    } else if (p.norm.mode) {
         for (int m = 0; m < MR; ++m) {
             T* xr = xs + (size_t)m * p.ld;
             float* rowf = reinterpret_cast<float*>(gemv_raw + (size_t)MR * p.ld * sizeof(T));
@@ -448,11 +509,17 @@ int gemv_launch(const GemvParams& p, size_t smem, unsigned grid, cudaStream_t s)
 template <typename T, int MR>
 int gemv_pick(const GemvParams& p, bool gated, size_t smem, cudaStream_t s) {
     const int groups = (p.n + (gated ? 1 : 3)) / (gated ? 2 : 4);
-    // warps that share a group: enough for 16 warps per SM, as long as each still has a full round of loads
+    // warps that share a group: the fewest passes over the loop of 16-byte loads, a round of groups costing a little by itself
+    const int max_grid = 148 * (smem > 100 * 1024 ? 1 : 2), chunks = p.ld >> 3;
     int wk = 1;
-    while (wk < 8 && groups * wk < 148 * 16 && (p.ld >> 3) > 32 * wk * 2) wk *= 2;
+    float best = 0.f;
+    for (int q = 1; q <= 8; q *= 2) {
+        const int ctas = max_grid * (kGemvWarps / q), rounds = (groups + ctas - 1) / ctas, passes = (chunks + 32 * q * kGemvUnroll - 1) / (32 * q * kGemvUnroll);
+        const float cost = rounds * (passes + 0.3f);
+        if (q == 1 || cost < best) { best = cost; wk = q; }
+    }
     const int per_cta = kGemvWarps / wk;
-    const unsigned grid = (unsigned)std::min((groups + per_cta - 1) / per_cta, 148 * (smem > 100 * 1024 ? 1 : smem > 64 * 1024 ? 2 : 3));
+    const unsigned grid = (unsigned)std::min((groups + per_cta - 1) / per_cta, max_grid);
     if (gated) {
         switch (wk) {
         case 1: return gemv_launch<T, MR, 1, true>(p, smem, grid, s);

@@ -695,12 +695,12 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
     const int first_pos = span.pos0 + q0, last_pos = first_pos + nq - 1;
     const int n_tiles = last_pos / kPfKeys + 1;
     const int cd = p.dim >> 3, cr = p.row.rot >> 3, cv = p.vdim >> 3;
+    // 16-byte chunk tid, tid + 256, ... of a tile as (row, chunk of the row), without divisions in the loop
+    const int per_row = cd + cr + cv, r_first = tid / per_row, c_first = tid - r_first * per_row, r_step = kPfThreads / per_row, c_step = kPfThreads - r_step * per_row;
     auto load_tile = [&](int kt, int stage) {
         __nv_bfloat16* ks = kv_sm + stage * STAGE;
         __nv_bfloat16* vs = ks + kPfKeys * PK;
-        const int per_row = cd + cr + cv;
-        for (int i = tid; i < kPfKeys * per_row; i += kPfThreads) {
-            const int r = i / per_row, c = i - r * per_row;
+        for (int r = r_first, c = c_first; r < kPfKeys; r += r_step + (c + c_step >= per_row), c += c_step - (c + c_step >= per_row ? per_row : 0)) {
             const size_t row = span.ctx0 + min(kt * kPfKeys + r, last_pos);
             const __nv_bfloat16* src;
             __nv_bfloat16* dst;
