@@ -347,7 +347,8 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
     float m_run = -INFINITY, l_run = 0.f;
     const int n_ct = p.row.rp >> 4;
 
-    for (int i = 0; i < mine; ++i) {
+    int i = 0;
+    for (; i < mine; ++i) {
         if (!mbar_wait(&full_bar[i & 1], (unsigned)((i >> 1) & 1))) { atomicExch(p.status, 41); bad = 1; }
         const unsigned page = smem_u32(pages + (size_t)(i & 1) * page_bytes);
         float sacc[4][4];
@@ -441,8 +442,8 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
         if (tid == 0 && i + 2 < mine) request(i + 2);
     }
     if (bad) {
-        // leave only when the copies still requested have landed (bounded)
-        if (tid == 0) for (int i = 0; i < 2 && i < mine; ++i) mbar_wait(&full_bar[i], 0u);
+        // leave only when the copies that may still be under way have landed (bounded)
+        if (tid == 0) for (int k = i; k < i + 2 && k < mine; ++k) mbar_wait(&full_bar[k & 1], (unsigned)((k >> 1) & 1));
         return;
     }
     const size_t pw = (size_t)p.row.rp + kPartialTail;
