@@ -104,9 +104,34 @@ enum {
        The latent c is RMS-normed (`weight`, eps, weight_bias); rotate-half rotary positions act on the first rope_dim of
        the key_dim entries of q and of the shared key part. Cached per token: c and the rotated key part. Per head the
        plain key is weight2 [heads * head_dim][n] c, the value weight3 [heads * value_dim][n] c; score = (q . k over both
-       parts) * scale, softmax over all positions up to the token's own; out = sigmoid(gate) * value sum. */
-    SWLM_STEP_LATENT_ATTN = 16
+       parts) * scale, softmax over all positions up to the token's own; out = sigmoid(gate) * value sum.
+       window_left > 0: only the last window_left positions, the token's own among them. weight4 not empty: a sink, one
+       number per head whose exponential joins the softmax's denominator (no key, no value, not scaled). */
+    SWLM_STEP_LATENT_ATTN = 16,
+    /* Gated activation with limits: g = min(in, limit), u = clamp(in2, -limit, limit),
+       out = g * sigmoid(scale * g) * (u + 1). */
+    SWLM_STEP_CLAMPED_GLU = 17,
+    /* Gated delta rule with a state per sequence. in_buf = q | k | v before their convolutions (groups * key_dim, the same
+       again, heads * value_dim), in2_buf = step sizes before the sigmoid (heads), in3_buf = decay inputs (heads * k, k = 1 or
+       key_dim: one decay per head or per key channel), in4_buf = output gate before its activation (heads * value_dim),
+       out_buf = heads * value_dim (may be in4_buf). Head h reads q and k of group h / (heads / groups).
+       Every channel of q, k, v: causal convolution over conv_kernel tokens (weight, weight2, weight3: [channels][conv_kernel],
+       the last column meets the current token; zeros before the start), then SiLU. q and k per group: x / sqrt(sum(x^2) +
+       eps2), q also times scale. decay = exp(-exp(A_log) * softplus(in3 + dt_bias)), beta = sigmoid(in2);
+       S = decay * S; u = beta * (v - S^T k); S = S + k u^T; o = S^T q with S [key_dim][value_dim] fp32, zero at position 0.
+       out = o * rsqrt(mean(o^2) + eps) * weight4 * activation(in4); gate_act: one of SWLM_GATE_*.
+       weight5 = A_log [heads], weight6 = dt_bias [heads * k]. */
+    SWLM_STEP_GATED_DELTA = 18,
+    /* Routed feed-forward: in_buf = input (n values), in2_buf = router logits (experts), out_buf = n values in hidden.
+       s = sigmoid(logits); the experts form `groups` equal groups of neighbours, a group counts as the sum of its two largest
+       s, and only experts of the groups_keep best groups can be chosen; the `top` largest s among them are. Expert i is the
+       clamped gated feed-forward (CLAMPED_GLU with glu_alpha, limit) of the matrices <weight>i<weight2>, <weight>i<weight3>
+       [k][n] and <weight>i<weight4> [n][k]; its output is weighted with s / (sum of the chosen s + 1e-20) * scale. */
+    SWLM_STEP_ROUTED_MLP = 19,
+    /* logits = scale * tanh(logits / scale), in place */
+    SWLM_STEP_SOFTCAP = 20
 };
+enum { SWLM_GATE_SILU = 0, SWLM_GATE_SIGMOID = 1 };
 
 typedef struct swlm_step {
     int32_t kind;
@@ -145,6 +170,18 @@ typedef struct swlm_step {
     float   rope_original;
     float   rope_fast;
     float   rope_slow;
+    /* fp32-stream plans */
+    int32_t in_off;      /* PRODUCT: first column of the input in in_buf (a multiple of 8) */
+    int32_t out_off;     /* and of the result in out_buf, so that several results share a buffer */
+    int32_t experts;
+    int32_t top;
+    int32_t groups_keep;
+    int32_t gate_act;
+    float   limit;
+    float   glu_alpha;
+    float   eps2;
+    char    weight5[SWLM_NAME_MAX];
+    char    weight6[SWLM_NAME_MAX];
 } swlm_step;
 
 /* Sizes of the runtime buffer set; mirrors the inputs of
@@ -196,6 +233,7 @@ typedef struct swlm_buffers_desc {
     /* tokens the page pool of the latent rows holds over all sequences, rounded up to pages of 64;
        0 = max_batch * max_seq. Sequences take pages as they grow and give them back when they are reset. */
     int32_t kv_pool_tokens;
+    int32_t delta_layers;    /* number of SWLM_STEP_GATED_DELTA layers: fp32 state and convolution inputs per sequence */
 } swlm_buffers_desc;
 
 enum { SWLM_STREAM_BF16 = 0, SWLM_STREAM_F32 = 1, SWLM_STREAM_ALL_F32 = 2 };

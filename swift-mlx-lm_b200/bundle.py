@@ -16,6 +16,7 @@ import json
 import os
 from typing import Dict, Optional, Tuple
 
+from . import rirotar as _rirotar
 from . import staf as _staf
 from . import vuzunex as _vuzunex
 from .plan import DispatchPlanBuilder, ModelConfig
@@ -26,8 +27,11 @@ TRANSFORMER_MODEL_TYPES = ("llama", "qwen2", "qwen3", "mistral", "phi", "phi3", 
                            "deepseek", "yi", "baichuan", "chatglm")
 LFM2_MODEL_TYPES = ("lfm2",)
 
-# config.json `architecture` values of dense bf16 checkpoints: name -> (config decoder, plan builder)
-ARCHITECTURES = {_vuzunex.ARCHITECTURE: (_vuzunex.decode_config, _vuzunex.VuzunexPlanBuilder)}
+# config.json `architecture` values of dense bf16 checkpoints: name -> (decoder of the config and the tensors' shapes, plan builder)
+ARCHITECTURES = {
+    _vuzunex.ARCHITECTURE: (lambda config, shapes, **runtime: _vuzunex.decode_config(config, **runtime), _vuzunex.VuzunexPlanBuilder),
+    _rirotar.ARCHITECTURE: (_rirotar.decode_config, _rirotar.RirotarPlanBuilder),
+}
 
 # KVCachePolicy of InferencePolicy.default (Sources/MetalCompiler/InferencePolicy.swift:55-100)
 DEFAULT_MAXIMUM_SEQUENCE_LENGTH = 4096
@@ -189,16 +193,16 @@ def prepare_dense_bundle(directory: str, config: Optional[Dict] = None, **runtim
     if entry is None:
         raise BundleError(f"Unsupported architecture: {config.get('architecture')}")
     decode, make_builder = entry
-    try:
-        builder = make_builder(decode(config, **runtime))
-    except (KeyError, TypeError, ValueError) as e:
-        raise BundleError(f"{config['architecture']}: {e!r}") from e
     shards = sorted(glob.glob(os.path.join(directory, "*.safetensors")))
     if not shards:
         raise BundleError(f"{directory}: no safetensors shard")
     found = {}
     for path in shards:
         found.update(_staf.read_safetensors(path))
+    try:
+        builder = make_builder(decode(config, {name: tuple(shape) for name, (_dtype, shape, _data) in found.items()}, **runtime))
+    except (KeyError, TypeError, ValueError) as e:
+        raise BundleError(f"{config['architecture']}: {e!r}") from e
     weights = {}
     for name, _kind, shape, _shard in builder.tensors():
         if name not in found:

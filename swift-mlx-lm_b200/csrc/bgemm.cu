@@ -6,7 +6,8 @@
 //                    (with fp32 ones the product is a true fp32 product: a bf16 weight is exact in fp32).
 //   bgemm_tc_kernel  more rows, bf16 activations: tcgen05.mma with both operands staged by TMA (128-byte swizzle), two tiles
 //                    of 128 weight rows side by side in tensor memory, K cut across CTAs when there are few tiles. The two
-//                    tiles are 256 consecutive rows, or 128 rows of gate and the same rows of up.
+//                    tiles are 256 consecutive rows, or 128 rows of gate and the same rows of up. Grouped form: activation rows
+//                    sorted by expert, a device table names the expert and the rows of every tile.
 //   sgemm_kernel     more rows, fp32 activations: fp32 FMAs on 64 x 64 tiles.
 #include <algorithm>
 #include <cstdlib>
@@ -32,6 +33,7 @@ __device__ __forceinline__ void product_store(const ProductOut& o, int m, int ro
     for (int q = 1; q < kMaxProductSegs; ++q)
         if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; }
     const size_t at = (size_t)m * stride + (row - first);
+    if (o.softcap > 0.f) val = o.softcap * tanhf(val / o.softcap);
     if (f32) static_cast<float*>(y)[at] = val;
     else static_cast<__nv_bfloat16*>(y)[at] = __float2bfloat16_rn(val);
 }
@@ -44,7 +46,8 @@ constexpr size_t kGemvMaxSmem = 200 * 1024;
 
 struct GemvParams {
     const __nv_bfloat16* w; const __nv_bfloat16* w2;
-    int ld, n, k, m, act;
+    int ld, n, k, m;
+    GatedAct act;
     const void* x; int x_stride;
     StreamNorm norm;
     ProductOut out;
@@ -296,7 +299,8 @@ constexpr int kTcBlock = kTcWarps * 32;
 struct TcParams {
     int n, m, steps;                 // weight rows, activation rows, 64-column steps of K
     int split_steps;                 // steps per K range (gridDim.z ranges); == steps when K is not cut
-    int act;
+    GatedAct act;
+    const int4* tiles;               // grouped form: (expert, first row, rows, 0) of tile blockIdx.x; n = rows of one expert's matrix
     ProductOut out;
     float* part;                     // [range][gated ? 2 : 1][m][n] when K is cut
     int* status;
@@ -325,7 +329,15 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
     __shared__ unsigned tmem_base;
     __shared__ int failed;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int tok0 = blockIdx.x * BN;
+    int tok0 = blockIdx.x * BN, tok_end = p.m, wrow0 = 0;     // wrow0: first row of the expert's matrix
+    if (p.tiles) {
+        pdl_wait();   // (the table is the preceding kernel's)
+        const int4 tile = p.tiles[blockIdx.x];
+        if (tile.z == 0) { pdl_launch_dependents(); return; }
+        wrow0 = tile.x * p.n;
+        tok0 = tile.y;
+        tok_end = tile.y + tile.z;
+    }
     const int row0 = blockIdx.y * (GATED ? kTileRows : 2 * kTileRows);
     const int nt = !GATED && row0 + kTileRows >= p.n ? 1 : 2;                       // accumulators in use
     const int stage_bytes = nt * A_BYTES + B_BYTES;
@@ -356,8 +368,8 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
             auto weights = [&](int kt, int s) {
                 const unsigned bar = smem_u32(&full_bar[s]), dst = smem_u32(smem + s * STAGE);
                 mbar_expect(bar, (unsigned)stage_bytes);
-                tma_load_2d(dst, &wmap, (step0 + kt) * kTcK, row0, bar);
-                if (nt == 2) tma_load_2d(dst + A_BYTES, GATED ? &wmap2 : &wmap, (step0 + kt) * kTcK, GATED ? row0 : row0 + kTileRows, bar);
+                tma_load_2d(dst, &wmap, (step0 + kt) * kTcK, wrow0 + row0, bar);
+                if (nt == 2) tma_load_2d(dst + A_BYTES, GATED ? &wmap2 : &wmap, (step0 + kt) * kTcK, wrow0 + (GATED ? row0 : row0 + kTileRows), bar);
             };
             auto activations = [&](int kt, int s) {
                 tma_load_2d(smem_u32(smem + s * STAGE) + 2 * A_BYTES, &xmap, (step0 + kt) * kTcK, tok0, smem_u32(&full_bar[s]));
@@ -410,7 +422,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
                 const int row = row0 + (GATED ? 0 : t * kTileRows) + quarter * 32 + lane;
 #pragma unroll 1
                 for (int c0 = 0; c0 < BN; c0 += 16) {
-                    if (tok0 + c0 >= p.m) break;   // uniform across the warp
+                    if (tok0 + c0 >= tok_end) break;   // uniform across the warp
                     unsigned v[16], u[16];
                     const unsigned at = tmem + ((unsigned)(quarter * 32) << 16) + (unsigned)(t * BN + c0);
                     asm volatile(
@@ -429,7 +441,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
 #pragma unroll
                         for (int i = 0; i < 16; ++i) {
                             const int tok = tok0 + c0 + i;
-                            if (tok >= p.m) break;
+                            if (tok >= tok_end) break;
                             const float val = __uint_as_float(v[i]);
                             if (cut) p.part[(((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m + tok) * p.n + row] = val;
                             else product_store(p.out, tok, row, GATED ? gated_activation(val, __uint_as_float(u[i]), p.act) : val);
@@ -446,7 +458,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
 
 // Sum of the K ranges in order, then the store (GATED: activation(gate sum) * up sum).
 template <bool GATED>
-__global__ void __launch_bounds__(256) bgemm_sum_kernel(const float* part, int ranges, int m, int n, int act, const ProductOut out) {
+__global__ void __launch_bounds__(256) bgemm_sum_kernel(const float* part, int ranges, int m, int n, GatedAct act, const ProductOut out) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t total = (size_t)m * n;
@@ -587,7 +599,7 @@ template <int BN, int STAGES>
 int tc_launch(const ProductLaunch& a, const TcShape& t, cudaStream_t s) {
     const bool gated = a.w2 != nullptr;
     TcParams p{};
-    p.n = a.w->n; p.m = a.m; p.steps = (a.w->k + kTcK - 1) / kTcK; p.split_steps = t.split_steps; p.act = a.act; p.out = a.out; p.part = a.part; p.status = a.status;
+    p.n = a.experts ? a.w->n / a.experts : a.w->n; p.tiles = a.tiles; p.m = a.m; p.steps = (a.w->k + kTcK - 1) / kTcK; p.split_steps = t.split_steps; p.act = a.act; p.out = a.out; p.part = a.part; p.status = a.status;
     CUtensorMap xmap, wmap, wmap2;
     int rc = bf16_map(static_cast<const __nv_bfloat16*>(a.x), a.x_stride, a.m, a.w->k, BN, &xmap);
     if (!rc) rc = bf16_map(a.w->data, a.w->ld, a.w->n, a.w->k, kTileRows, &wmap);
@@ -605,6 +617,17 @@ int tc_launch(const ProductLaunch& a, const TcShape& t, cudaStream_t s) {
         if (e != cudaSuccess) return cuda_fail(e, "bgemm sum launch");
     }
     return SWLM_OK;
+}
+
+TcShape grouped_shape(const ProductLaunch& a) {
+    TcShape t;
+    const int n = a.w->n / a.experts, rows_n = a.w2 ? kTileRows : 2 * kTileRows;
+    t.bn = a.group_bn;
+    t.tiles_m = a.max_tiles;
+    t.tiles_n = (n + rows_n - 1) / rows_n;
+    t.ranges = 1;
+    t.split_steps = (a.w->k + kTcK - 1) / kTcK;
+    return t;
 }
 
 bool gemv_fits(int m, int k, bool x_f32, bool norm) {
@@ -631,7 +654,15 @@ size_t product_part_floats(int n, int k, int m, bool gated) {
     return t.ranges > 1 ? (size_t)t.ranges * (gated ? 2 : 1) * m * n : 0;
 }
 
+// tiles about as tall as an expert has rows on average
+int grouped_bn(int rows, int experts) {
+    const int avg = rows / std::max(1, experts);
+    return avg > 160 ? 256 : avg > 64 ? 128 : avg > 24 ? 64 : 32;
+}
+int grouped_max_tiles(int rows, int experts) { return std::min(rows, experts) + rows / grouped_bn(rows, experts); }
+
 int product_launch_count(const ProductLaunch& a) {
+    if (a.experts) return 1;
     if (gemv_fits(a.m, a.w->k, a.x_f32, a.norm.mode != 0) || a.x_f32) return 1;
     return tc_shape(a.w->n, a.w->k, a.m, a.w2 != nullptr).ranges > 1 ? 2 : 1;
 }
@@ -640,7 +671,8 @@ int launch_product(const ProductLaunch& a, cudaStream_t s) {
     if (a.m <= 0) return SWLM_OK;
     const bool gated = a.w2 != nullptr;
     if (gated && (a.w2->n != a.w->n || a.w2->k != a.w->k)) { set_error("gated product: the two matrices differ in shape"); return SWLM_ERR_INVALID; }
-    if (gemv_fits(a.m, a.w->k, a.x_f32, a.norm.mode != 0)) {
+    if (a.experts && (a.x_f32 || a.norm.mode || !a.tiles)) { set_error("a grouped product takes plain bf16 rows"); return SWLM_ERR_INVALID; }
+    if (!a.experts && gemv_fits(a.m, a.w->k, a.x_f32, a.norm.mode != 0)) {
         GemvParams p{};
         p.w = a.w->data; p.w2 = gated ? a.w2->data : nullptr; p.ld = a.w->ld; p.n = a.w->n; p.k = a.w->k; p.m = a.m; p.act = a.act;
         p.x = a.x; p.x_stride = a.x_stride; p.norm = a.norm; p.out = a.out;
@@ -655,7 +687,7 @@ int launch_product(const ProductLaunch& a, cudaStream_t s) {
         return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "sgemm launch");
     }
     if ((a.x_stride & 7) || (reinterpret_cast<uintptr_t>(a.x) & 15)) { set_error("dense product: activation rows must be 16-byte aligned"); return SWLM_ERR_INVALID; }
-    const TcShape t = tc_shape(a.w->n, a.w->k, a.m, gated);
+    const TcShape t = a.experts ? grouped_shape(a) : tc_shape(a.w->n, a.w->k, a.m, gated);
     if (t.ranges > 1 && (!a.part || a.part_floats < (size_t)t.ranges * (gated ? 2 : 1) * a.m * a.w->n)) { set_error("dense product: scratch too small"); return SWLM_ERR_INVALID; }
     switch (t.bn) {
     case 32: return tc_launch<32, 4>(a, t, s);

@@ -1,0 +1,545 @@
+// Gated delta rule over an fp32 state per sequence and head: short causal convolutions with SiLU in front of q, k and v, unit q
+// and k, one decay per head or per key channel, and a normed, gated read-out.
+//
+// Two ways through it, chosen per row of a batch:
+//   * a single token of a sequence (decode steps): delta_step_kernel does all of it in one launch, a cluster of CTAs per head
+//     that each own 32 columns of the state; state and convolution inputs are requested before the preceding kernel has
+//     finished.
+//   * portions: tokens are taken in blocks of kDeltaBlock. delta_prepare_kernel works out, for every block and head, what the
+//     recurrence needs of the block with the decays folded in; delta_scan_kernel walks the blocks with the state in registers;
+//     delta_gate_kernel norms and gates the rows.
+//
+// Inside a block, with S the state in front of it, G_t the product of the decays up to token t and D_ts the product of the
+// decays of tokens s + 1 .. t (all at most 1, nothing is divided):
+//   u_t = beta_t (v_t - S^T (G_t k_t)) - sum_{s < t} beta_t (k_s . D_ts k_t) u_s
+//   o_t = S^T (G_t q_t) + sum_{s <= t} (k_s . D_ts q_t) u_s
+//   S' = G_T S + sum_s (D_Ts k_s) u_s^T
+// The products of k and q with each other do not depend on the state's column: they are formed once per head. Everything is
+// fp32. Where a sequence is cut changes the blocks, and with them the order of sums, nothing else.
+#include <cooperative_groups.h>
+
+#include <algorithm>
+#include <utility>
+
+#include "swlm_internal.h"
+#include "tc_device.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace swlm {
+namespace {
+
+constexpr int TB = kDeltaBlock;
+constexpr int kScanCols = 16, kScanParts = 8, kScanThreads = kScanCols * kScanParts, kScanStages = 4;
+constexpr int kStepCols = 32, kStepWarps = 8, kStepThreads = kStepWarps * 32, kStepCluster = 8;
+constexpr int kPrepThreads = 128;
+
+struct DeltaParams {
+    DeltaShape sh;
+    int decay_dim, gate_act;
+    float eps, unit_eps, q_scale;
+    const void* qkv; int qkv_stride;
+    const float* beta; int beta_stride;
+    const float* decay; int decay_stride;
+    const void* gate; int gate_stride;
+    const __nv_bfloat16 *conv_q, *conv_k, *conv_v, *norm_w, *a_log, *dt_bias;
+    void* ring; float* state;
+    const int32_t* row_seq; const int32_t* row_pos;
+    void* out; int out_stride;
+    int n_single; const int32_t* single_rows;
+    const RowRun* runs; const int32_t* block_run;   // runs == null: every single row is a run of one token
+    float* rec; float* vrec; float* o;
+    int dp, rec_floats, vblocks;                    // padded key channels, floats per block and head, column blocks of the scan
+    int* status;
+};
+
+__device__ __forceinline__ float dl_get(const float* p) { return *p; }
+__device__ __forceinline__ float dl_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void dl_put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void dl_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return x * sigmoid(x); }
+__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float warp_sum(float v) {
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float gate_of(float x, int act) { return act == SWLM_GATE_SIGMOID ? sigmoid(x) : silu(x); }
+
+__device__ __forceinline__ RowRun run_of(const DeltaParams& p, int i) {
+    if (p.runs) return p.runs[i];
+    const int row = p.single_rows ? p.single_rows[i] : i;
+    return RowRun{row, 1, p.row_pos[row], p.row_seq[row], i};
+}
+// channel `ch` of q | k | v: its taps (q, k and v keep theirs in tensors of their own)
+__device__ __forceinline__ const __nv_bfloat16* taps_of(const DeltaParams& p, int ch) {
+    const int gk = p.sh.groups * p.sh.dim;
+    return ch < gk ? p.conv_q + (size_t)ch * p.sh.taps : ch < 2 * gk ? p.conv_k + (size_t)(ch - gk) * p.sh.taps : p.conv_v + (size_t)(ch - 2 * gk) * p.sh.taps;
+}
+// input of channel ch at token i of a run; i < 0: what earlier batches left
+template <typename T>
+__device__ __forceinline__ float conv_input(const DeltaParams& p, const RowRun& run, int ch, int i) {
+    if (i >= 0) return dl_get(static_cast<const T*>(p.qkv) + (size_t)(run.row0 + i) * p.qkv_stride + ch);
+    const int pos = run.pos0 + i;
+    if (pos < 0) return 0.f;
+    return dl_get(static_cast<const T*>(p.ring) + ((size_t)run.seq * p.sh.taps + pos % p.sh.taps) * p.sh.channels() + ch);
+}
+template <typename T>
+__device__ __forceinline__ float conv_silu(const DeltaParams& p, const RowRun& run, int ch, int i) {
+    const __nv_bfloat16* w = taps_of(p, ch);
+    float acc = 0.f;
+    for (int j = 0; j < p.sh.taps; ++j) acc = fmaf(__bfloat162float(w[j]), conv_input<T>(p, run, ch, i - (p.sh.taps - 1) + j), acc);
+    return silu(acc);
+}
+__device__ __forceinline__ float decay_of(const DeltaParams& p, int row, int h, int d, float rate) {
+    const int i = p.decay_dim == 1 ? h : h * p.decay_dim + d;
+    return expf(-rate * softplus(p.decay[(size_t)row * p.decay_stride + i] + __bfloat162float(p.dt_bias[i])));
+}
+
+// ---- portions: what a block needs of its tokens -----------------------------------------------------------------------
+// CTA (block, head). Record: [TB][dp] beta_t G_t k_t, [TB][dp] G_t q_t, [TB][dp] D_Ts k_s, [dp] G_T, then the coefficients
+// [TB][TB] of u_t and [TB][TB] of o_t. Values: [column block][TB][kScanCols] beta_t v_t. Tokens past the end of the run: k = q
+// = v = 0 and a decay of 1.
+template <typename T>
+__global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const DeltaParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float prep_smem[];
+    __shared__ float beta_s[TB], norm_s[2 * TB], red[kPrepThreads / 32][2 * TB * TB];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, blk = blockIdx.x, h = blockIdx.y;
+    const RowRun run = run_of(p, p.block_run ? p.block_run[blk] : blk);
+    const int t0 = (blk - run.blk0) * TB, nt = min(TB, run.count - t0);
+    const int dim = p.sh.dim, vdim = p.sh.vdim, grp = h / (p.sh.heads / p.sh.groups), gk = p.sh.groups * dim;
+    float* q = prep_smem;            // [TB][dim]
+    float* k = q + TB * dim;         // [TB][dim]
+    if (tid < TB) beta_s[tid] = tid < nt ? sigmoid(p.beta[(size_t)(run.row0 + t0 + tid) * p.beta_stride + h]) : 0.f;
+    __syncthreads();
+    for (int i = tid; i < 2 * dim; i += kPrepThreads) {
+        const int d = i < dim ? i : i - dim, ch = (i < dim ? 0 : gk) + grp * dim + d;
+        float* dst = i < dim ? q : k;
+#pragma unroll
+        for (int t = 0; t < TB; ++t) dst[t * dim + d] = t < nt ? conv_silu<T>(p, run, ch, t0 + t) : 0.f;
+    }
+    float* vr = p.vrec + (size_t)(blk * p.sh.heads + h) * p.vblocks * TB * kScanCols;
+    for (int c = tid; c < p.vblocks * kScanCols; c += kPrepThreads)
+#pragma unroll
+        for (int t = 0; t < TB; ++t)
+            vr[(c / kScanCols * TB + t) * kScanCols + c % kScanCols] = t < nt && c < vdim ? beta_s[t] * conv_silu<T>(p, run, 2 * gk + h * vdim + c, t0 + t) : 0.f;
+    __syncthreads();
+    for (int i = warp; i < 2 * TB; i += kPrepThreads / 32) {
+        const float* x = (i < TB ? q : k) + (i % TB) * dim;
+        float ss = 0.f;
+        for (int d = lane; d < dim; d += 32) ss = fmaf(x[d], x[d], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) norm_s[i] = (i < TB ? p.q_scale : 1.0f) / sqrtf(ss + p.unit_eps);
+    }
+    __syncthreads();
+    const float rate = expf(__bfloat162float(p.a_log[h]));
+    float* rec = p.rec + (size_t)(blk * p.sh.heads + h) * p.rec_floats;
+    float a[TB][TB], b[TB][TB];
+#pragma unroll
+    for (int t = 0; t < TB; ++t)
+#pragma unroll
+        for (int s = 0; s < TB; ++s) a[t][s] = b[t][s] = 0.f;
+    for (int d = tid; d < p.dp; d += kPrepThreads) {
+        float kv[TB], qv[TB], g[TB];
+#pragma unroll
+        for (int t = 0; t < TB; ++t) {
+            const bool live = d < dim && t < nt;
+            kv[t] = live ? k[t * dim + d] * norm_s[TB + t] : 0.f;
+            qv[t] = live ? q[t * dim + d] * norm_s[t] : 0.f;
+            g[t] = live ? decay_of(p, run.row0 + t0 + t, h, d, rate) : 1.f;
+        }
+        float gt = 1.f;
+#pragma unroll
+        for (int t = 0; t < TB; ++t) {
+            gt *= g[t];
+            rec[t * p.dp + d] = beta_s[t] * gt * kv[t];
+            rec[(TB + t) * p.dp + d] = gt * qv[t];
+        }
+        rec[3 * TB * p.dp + d] = gt;
+#pragma unroll
+        for (int s = 0; s < TB; ++s) {
+            float w = kv[s];
+            b[s][s] = fmaf(w, qv[s], b[s][s]);
+#pragma unroll
+            for (int t = s + 1; t < TB; ++t) {
+                w *= g[t];
+                a[t][s] = fmaf(w, kv[t], a[t][s]);
+                b[t][s] = fmaf(w, qv[t], b[t][s]);
+            }
+            rec[(2 * TB + s) * p.dp + d] = w;
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < TB; ++t)
+#pragma unroll
+        for (int s = 0; s <= t; ++s) {
+            const float y = warp_sum(b[t][s]);
+            const float x = s < t ? warp_sum(a[t][s]) : 0.f;
+            if (lane == 0) { red[warp][t * TB + s] = x; red[warp][TB * TB + t * TB + s] = y; }
+        }
+    __syncthreads();
+    if (tid < 2 * TB * TB) {
+        const int t = tid % (TB * TB) / TB, s = tid % TB;
+        float v = 0.f;
+        if (s <= t)
+            for (int w = 0; w < kPrepThreads / 32; ++w) v += red[w][tid];
+        rec[(3 * TB + 1) * p.dp + tid] = tid < TB * TB ? beta_s[t] * v : v;
+    }
+}
+
+// ---- portions: the recurrence -----------------------------------------------------------------------------------------
+// CTA (16 columns of the state, head, run). Eight lanes share a column: lane part j holds key channels 4 j + 32 i + (0 .. 3), so
+// that a 16-byte read of a record row by the parts of a warp is free of bank conflicts. Records come through a ring of bulk
+// copies. At the end the run's last inputs go to the convolution ring (all readers of the old ones have finished).
+template <typename T, int R>
+__global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaParams p) {
+    constexpr int DP = R * kScanParts, REC = (3 * TB + 1) * DP + 2 * TB * TB, VREC = TB * kScanCols, STAGE = REC + VREC;
+    extern __shared__ __align__(128) float scan_smem[];
+    __shared__ __align__(8) unsigned long long full_bar[kScanStages];
+    __shared__ int bad;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane & 7, lc = warp * 4 + (lane >> 3);
+    const int vb = blockIdx.x, h = blockIdx.y, col = vb * kScanCols + lc;
+    pdl_launch_dependents();
+    if (tid == 0) {
+        for (int s = 0; s < kScanStages; ++s) mbar_init(&full_bar[s], 1);
+        bad = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    pdl_wait();
+    const RowRun run = run_of(p, blockIdx.z);
+    const int nb = (run.count + TB - 1) / TB;
+    const bool live = col < p.sh.vdim;
+    auto request = [&](int b) {   // thread 0
+        const int s = b % kScanStages;
+        const unsigned bar = smem_u32(&full_bar[s]), dst = smem_u32(scan_smem + (size_t)s * STAGE);
+        const size_t at = (size_t)(run.blk0 + b) * p.sh.heads + h;
+        mbar_expect(bar, STAGE * 4);
+        bulk_load(dst, p.rec + at * REC, REC * 4, bar);
+        bulk_load(dst + REC * 4, p.vrec + (at * p.vblocks + vb) * VREC, VREC * 4, bar);
+    };
+    int issued = 0;
+    if (tid == 0) for (; issued < min(kScanStages, nb); ++issued) request(issued);
+    float* st = p.state + ((size_t)run.seq * p.sh.heads + h) * p.sh.dim * p.sh.vdim + col;
+    float S[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int d = part * 4 + 32 * (i >> 2) + (i & 3);
+        S[i] = live && run.pos0 > 0 && d < p.sh.dim ? st[(size_t)d * p.sh.vdim] : 0.f;
+    }
+    float* o_row = p.o + (size_t)run.row0 * p.sh.heads * p.sh.vdim + (size_t)h * p.sh.vdim + col;
+    const int o_stride = p.sh.heads * p.sh.vdim;
+    for (int b = 0; b < nb; ++b) {
+        const int s = b % kScanStages;
+        if (!mbar_wait(&full_bar[s], (unsigned)((b / kScanStages) & 1))) { atomicExch(p.status, 51); bad = 1; }
+        const float* rec = scan_smem + (size_t)s * STAGE;
+        const float4* r4 = reinterpret_cast<const float4*>(rec) + part;
+        float a[TB], q[TB];
+#pragma unroll
+        for (int t = 0; t < TB; ++t) a[t] = q[t] = 0.f;
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i)
+#pragma unroll
+            for (int t = 0; t < TB; ++t) {
+                const float4 kt = r4[(t * DP + 32 * i) / 4], qt = r4[((TB + t) * DP + 32 * i) / 4];
+                a[t] = fmaf(S[4 * i], kt.x, a[t]); a[t] = fmaf(S[4 * i + 1], kt.y, a[t]); a[t] = fmaf(S[4 * i + 2], kt.z, a[t]); a[t] = fmaf(S[4 * i + 3], kt.w, a[t]);
+                q[t] = fmaf(S[4 * i], qt.x, q[t]); q[t] = fmaf(S[4 * i + 1], qt.y, q[t]); q[t] = fmaf(S[4 * i + 2], qt.z, q[t]); q[t] = fmaf(S[4 * i + 3], qt.w, q[t]);
+            }
+#pragma unroll
+        for (int o = 1; o < kScanParts; o <<= 1)
+#pragma unroll
+            for (int t = 0; t < TB; ++t) {
+                a[t] += __shfl_xor_sync(0xffffffffu, a[t], o);
+                q[t] += __shfl_xor_sync(0xffffffffu, q[t], o);
+            }
+        const float* coef = rec + (3 * TB + 1) * DP;
+        const float* vv = rec + REC;
+        float u[TB];
+#pragma unroll
+        for (int t = 0; t < TB; ++t) {
+            u[t] = vv[t * kScanCols + lc] - a[t];
+#pragma unroll
+            for (int e = 0; e < t; ++e) u[t] = fmaf(-coef[t * TB + e], u[e], u[t]);
+        }
+#pragma unroll
+        for (int t = 0; t < TB; ++t)
+#pragma unroll
+            for (int e = 0; e <= t; ++e) q[t] = fmaf(coef[TB * TB + t * TB + e], u[e], q[t]);
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i) {
+            const float4 g = r4[(3 * TB * DP + 32 * i) / 4];
+            float x = S[4 * i] * g.x, y = S[4 * i + 1] * g.y, z = S[4 * i + 2] * g.z, w = S[4 * i + 3] * g.w;
+#pragma unroll
+            for (int t = 0; t < TB; ++t) {
+                const float4 kt = r4[((2 * TB + t) * DP + 32 * i) / 4];
+                x = fmaf(kt.x, u[t], x); y = fmaf(kt.y, u[t], y); z = fmaf(kt.z, u[t], z); w = fmaf(kt.w, u[t], w);
+            }
+            S[4 * i] = x; S[4 * i + 1] = y; S[4 * i + 2] = z; S[4 * i + 3] = w;
+        }
+#pragma unroll
+        for (int t = 0; t < TB; ++t)
+            if (part == t && live && b * TB + t < run.count) o_row[(size_t)(b * TB + t) * o_stride] = q[t];
+        __syncthreads();   // the stage is free
+        if (bad) break;    // uniform: written before the barrier by whoever gave up
+        if (tid == 0 && issued < nb) { request(issued); ++issued; }
+    }
+    if (bad) {   // leave only when the copies that may still be under way have landed (bounded)
+        if (tid == 0) for (int b = max(0, issued - kScanStages); b < issued; ++b) mbar_wait(&full_bar[b % kScanStages], (unsigned)((b / kScanStages) & 1));
+        return;
+    }
+    if (live) {
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+            const int d = part * 4 + 32 * (i >> 2) + (i & 3);
+            if (d < p.sh.dim) st[(size_t)d * p.sh.vdim] = S[i];
+        }
+    }
+    if (vb == 0) {
+        const int share = p.sh.heads / p.sh.groups, gk = p.sh.groups * p.sh.dim, ch_all = p.sh.channels();
+        const int n_qk = h % share == 0 ? p.sh.dim : 0, grp = h / share;
+        for (int back = 0; back < min(run.count, p.sh.taps); ++back) {
+            const int tok = run.count - 1 - back, slot = (run.pos0 + tok) % p.sh.taps;
+            const T* src = static_cast<const T*>(p.qkv) + (size_t)(run.row0 + tok) * p.qkv_stride;
+            T* dst = static_cast<T*>(p.ring) + ((size_t)run.seq * p.sh.taps + slot) * ch_all;
+            for (int i = tid; i < p.sh.vdim + 2 * n_qk; i += kScanThreads) {
+                const int ch = i < p.sh.vdim ? 2 * gk + h * p.sh.vdim + i : i < p.sh.vdim + n_qk ? grp * p.sh.dim + i - p.sh.vdim : gk + grp * p.sh.dim + i - p.sh.vdim - n_qk;
+                dst[ch] = src[ch];
+            }
+        }
+    }
+}
+
+// ---- portions: norm and gate ------------------------------------------------------------------------------------------
+// CTA (block, head), a warp per token.
+template <typename T>
+__global__ void __launch_bounds__(TB * 32) delta_gate_kernel(const DeltaParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, t = threadIdx.x >> 5, blk = blockIdx.x, h = blockIdx.y, vdim = p.sh.vdim;
+    const RowRun run = run_of(p, p.block_run ? p.block_run[blk] : blk);
+    const int i = (blk - run.blk0) * TB + t;
+    if (i >= run.count) return;
+    const int row = run.row0 + i;
+    const float* o = p.o + ((size_t)row * p.sh.heads + h) * vdim;
+    float ss = 0.f;
+    for (int c = lane; c < vdim; c += 32) ss = fmaf(o[c], o[c], ss);
+    const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + p.eps);
+    const T* gate = static_cast<const T*>(p.gate) + (size_t)row * p.gate_stride + (size_t)h * vdim;
+    T* out = static_cast<T*>(p.out) + (size_t)row * p.out_stride + (size_t)h * vdim;
+    for (int c = lane; c < vdim; c += 32) dl_put(out + c, o[c] * sc * __bfloat162float(p.norm_w[c]) * gate_of(dl_get(gate + c), p.gate_act));
+}
+
+// ---- single tokens ----------------------------------------------------------------------------------------------------
+// Cluster of CTAs per (head, row), 32 state columns each: warp w holds key channels w, w + 8, ... of the CTA's columns, lane =
+// column. Nothing of this layer's state is touched by the kernels in front of this one, so it is read ahead of them. The slot
+// of the convolution ring that is written (position % taps) is none of those that are read.
+template <typename T, int R>
+__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p) {
+    extern __shared__ __align__(16) float step_smem[];
+    __shared__ float part_a[kStepWarps][kStepCols], part_b[kStepWarps][kStepCols], scal[4], v_s[kStepCols], ssq[kStepCluster];
+    const cg::cluster_group cluster = cg::this_cluster();
+    auto started = cluster.barrier_arrive();   // waited for before anything is written to another CTA's shared memory
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, vb = blockIdx.x, h = blockIdx.y;
+    const int row = p.single_rows ? p.single_rows[blockIdx.z] : blockIdx.z, pos = p.row_pos[row], seq = p.row_seq[row];
+    const int dim = p.sh.dim, vdim = p.sh.vdim, taps = p.sh.taps, share = p.sh.heads / p.sh.groups, grp = h / share, gk = p.sh.groups * dim, ch_all = p.sh.channels();
+    const int col = vb * kStepCols + lane;
+    const bool live = col < vdim;
+    float* q = step_smem;        // [dim]
+    float* k = q + dim;          // [dim]
+    float* g = k + dim;          // [dim]
+    float* st = p.state + ((size_t)seq * p.sh.heads + h) * dim * vdim + col;
+    float S[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int d = warp + kStepWarps * i;
+        S[i] = live && pos > 0 && d < dim ? st[(size_t)d * vdim] : 0.f;
+    }
+    // channel tid + 256 j of q | k | this CTA's v: the past's share of the convolution
+    constexpr int CH = (2 * R * kStepWarps + kStepCols + kStepThreads - 1) / kStepThreads;
+    const T* ring = static_cast<const T*>(p.ring) + (size_t)seq * taps * ch_all;
+    float acc[CH], w_last[CH];
+    int chan[CH];
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+        const int i = tid + kStepThreads * j, vc = vb * kStepCols + i - 2 * dim;
+        chan[j] = i < dim ? grp * dim + i : i < 2 * dim ? gk + grp * dim + i - dim : i < 2 * dim + kStepCols && vc < vdim ? 2 * gk + h * vdim + vc : -1;
+        acc[j] = w_last[j] = 0.f;
+        if (chan[j] >= 0) {
+            const __nv_bfloat16* w = taps_of(p, chan[j]);
+            for (int e = 0; e + 1 < taps; ++e) {
+                const int at = pos - (taps - 1) + e;
+                if (at >= 0) acc[j] = fmaf(__bfloat162float(w[e]), dl_get(ring + (size_t)(at % taps) * ch_all + chan[j]), acc[j]);
+            }
+            w_last[j] = __bfloat162float(w[taps - 1]);
+        }
+    }
+    const float rate = expf(__bfloat162float(p.a_log[h]));
+    const float nw = live ? __bfloat162float(p.norm_w[col]) : 0.f;
+    pdl_wait();
+
+    const bool keeps_qk = vb == 0 && h % share == 0;
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+        const int i = tid + kStepThreads * j;
+        float y = 0.f;
+        if (chan[j] >= 0) {
+            const T x = static_cast<const T*>(p.qkv)[(size_t)row * p.qkv_stride + chan[j]];
+            y = silu(fmaf(w_last[j], dl_get(&x), acc[j]));
+            if (i >= 2 * dim || keeps_qk) const_cast<T*>(ring)[(size_t)(pos % taps) * ch_all + chan[j]] = x;
+        }
+        if (i < dim) q[i] = y;
+        else if (i < 2 * dim) k[i - dim] = y;
+        else if (i < 2 * dim + kStepCols) v_s[i - 2 * dim] = y;
+    }
+    if (p.decay_dim == 1) {
+        const float one = decay_of(p, row, h, 0, rate);
+        for (int d = tid; d < dim; d += kStepThreads) g[d] = one;
+    } else {
+        for (int d = tid; d < dim; d += kStepThreads) g[d] = decay_of(p, row, h, d, rate);
+    }
+    const float gate = live && warp == 0 ? gate_of(dl_get(static_cast<const T*>(p.gate) + (size_t)row * p.gate_stride + (size_t)h * vdim + col), p.gate_act) : 0.f;
+    const float beta = sigmoid(p.beta[(size_t)row * p.beta_stride + h]);
+    __syncthreads();
+    if (warp < 3) {
+        const float* x = warp == 1 ? k : q;
+        const float* y = warp == 0 ? q : k;
+        float ss = 0.f;
+        for (int d = lane; d < dim; d += 32) ss = fmaf(x[d], y[d], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) scal[warp] = ss;
+    }
+    __syncthreads();
+    const float qn = p.q_scale / sqrtf(scal[0] + p.unit_eps), kn = 1.0f / sqrtf(scal[1] + p.unit_eps);
+    float a = 0.f, b = 0.f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int d = warp + kStepWarps * i;
+        if (d < dim) {
+            S[i] *= g[d];
+            a = fmaf(S[i], k[d], a);
+            b = fmaf(S[i], q[d], b);
+        }
+    }
+    part_a[warp][lane] = a;
+    part_b[warp][lane] = b;
+    __syncthreads();
+    a = b = 0.f;
+#pragma unroll
+    for (int w = 0; w < kStepWarps; ++w) { a += part_a[w][lane]; b += part_b[w][lane]; }
+    const float u = beta * (v_s[lane] - a * kn), uk = u * kn;
+    const float o = live ? fmaf(scal[2] * qn, uk, b * qn) : 0.f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int d = warp + kStepWarps * i;
+        if (d < dim && live) st[(size_t)d * vdim] = fmaf(k[d], uk, S[i]);
+    }
+    const int nz = gridDim.x;
+    cluster.barrier_wait(std::move(started));
+    if (warp == 0) {
+        const float ss = warp_sum(o * o);
+        if (lane < nz) cluster.map_shared_rank(ssq, lane)[vb] = ss;
+    }
+    cluster.sync();
+    if (warp == 0 && live) {
+        float ss = 0.f;
+        for (int i = 0; i < nz; ++i) ss += ssq[i];
+        dl_put(static_cast<T*>(p.out) + (size_t)row * p.out_stride + (size_t)h * vdim + col, o / sqrtf(ss / (float)vdim + p.eps) * nw * gate);
+    }
+}
+
+// ---- launches ---------------------------------------------------------------------------------------------------------
+int scan_regs(int dim) { return dim <= 32 ? 4 : dim <= 64 ? 8 : dim <= 128 ? 16 : dim <= 256 ? 32 : dim <= 512 ? 64 : 0; }
+int rec_floats(int dim) { return (3 * TB + 1) * scan_regs(dim) * kScanParts + 2 * TB * TB; }
+int scan_vblocks(int vdim) { return (vdim + kScanCols - 1) / kScanCols; }
+size_t scan_smem_bytes(int dim) { return (size_t)kScanStages * (rec_floats(dim) + TB * kScanCols) * 4; }
+
+template <typename T, int R>
+int scan_launch(const DeltaParams& p, int runs, cudaStream_t s) {
+    static const cudaError_t attr = cudaFuncSetAttribute(delta_scan_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan_smem_bytes(R * kScanParts));
+    if (attr != cudaSuccess) return cuda_fail(attr, "delta scan attributes");
+    const cudaError_t e = launch_k(delta_scan_kernel<T, R>, dim3(p.vblocks, p.sh.heads, runs), dim3(kScanThreads), scan_smem_bytes(R * kScanParts), s, p);
+    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "delta scan launch");
+}
+template <typename T>
+int portions(const DeltaParams& p, int runs, int blocks, cudaStream_t s) {
+    cudaError_t e = launch_k(delta_prepare_kernel<T>, dim3(blocks, p.sh.heads), dim3(kPrepThreads), (size_t)2 * TB * p.sh.dim * 4, s, p);
+    if (e != cudaSuccess) return cuda_fail(e, "delta prepare launch");
+    int rc;
+    switch (scan_regs(p.sh.dim)) {
+    case 4: rc = scan_launch<T, 4>(p, runs, s); break;
+    case 8: rc = scan_launch<T, 8>(p, runs, s); break;
+    case 16: rc = scan_launch<T, 16>(p, runs, s); break;
+    case 32: rc = scan_launch<T, 32>(p, runs, s); break;
+    default: rc = scan_launch<T, 64>(p, runs, s); break;
+    }
+    if (rc) return rc;
+    e = launch_k(delta_gate_kernel<T>, dim3(blocks, p.sh.heads), dim3(TB * 32), 0, s, p);
+    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "delta gate launch");
+}
+template <typename T, int R>
+cudaError_t step_launch(const DeltaParams& p, cudaStream_t s) {
+    const int nz = (p.sh.vdim + kStepCols - 1) / kStepCols;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(nz, p.sh.heads, p.n_single); cfg.blockDim = dim3(kStepThreads); cfg.stream = s;
+    cfg.dynamicSmemBytes = (size_t)3 * p.sh.dim * 4;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = nz; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl_enabled() ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, R>, p);
+}
+template <typename T>
+int run(const DeltaLaunch& a, DeltaParams p, cudaStream_t s, int* launches) {
+    int rc;
+    if (a.n_single > 0) {
+        if (delta_step_fits(a.shape)) {
+            const int regs = (a.shape.dim + kStepWarps - 1) / kStepWarps;
+            const cudaError_t e = regs <= 8 ? step_launch<T, 8>(p, s) : regs <= 16 ? step_launch<T, 16>(p, s) : step_launch<T, 32>(p, s);
+            if (e != cudaSuccess) return cuda_fail(e, "delta step launch");
+            *launches += 1;
+        } else {
+            if ((rc = portions<T>(p, a.n_single, a.n_single, s))) return rc;
+            *launches += 3;
+        }
+    }
+    if (a.n_runs > 0) {
+        p.runs = a.runs;
+        p.block_run = a.block_run;
+        if ((rc = portions<T>(p, a.n_runs, a.n_blocks, s))) return rc;
+        *launches += 3;
+    }
+    return SWLM_OK;
+}
+
+}  // namespace
+
+bool delta_supported(const DeltaShape& s) {
+    return s.heads > 0 && s.groups > 0 && s.heads % s.groups == 0 && s.dim > 0 && s.vdim > 0 && s.taps > 0 && scan_regs(s.dim) > 0;
+}
+bool delta_step_fits(const DeltaShape& s) { return s.dim <= 32 * kStepWarps && s.vdim <= kStepCols * kStepCluster; }
+size_t delta_scratch_floats(const DeltaShape& s, int blocks, int rows) {
+    return (size_t)blocks * s.heads * (rec_floats(s.dim) + (size_t)scan_vblocks(s.vdim) * TB * kScanCols) + (size_t)rows * s.heads * s.vdim;
+}
+
+int launch_delta(const DeltaLaunch& a, cudaStream_t s, int* launches) {
+    DeltaParams p{};
+    p.sh = a.shape; p.decay_dim = a.decay_dim; p.gate_act = a.gate_act; p.eps = a.eps; p.unit_eps = a.unit_eps; p.q_scale = a.q_scale;
+    p.qkv = a.qkv; p.qkv_stride = a.qkv_stride; p.beta = a.beta; p.beta_stride = a.beta_stride; p.decay = a.decay; p.decay_stride = a.decay_stride;
+    p.gate = a.gate; p.gate_stride = a.gate_stride; p.conv_q = a.conv_q; p.conv_k = a.conv_k; p.conv_v = a.conv_v; p.norm_w = a.norm_w;
+    p.a_log = a.a_log; p.dt_bias = a.dt_bias; p.ring = a.ring; p.state = a.state; p.row_seq = a.row_seq; p.row_pos = a.row_pos;
+    p.out = a.out; p.out_stride = a.out_stride; p.n_single = a.n_single; p.single_rows = a.single_rows; p.status = a.status;
+    p.dp = scan_regs(a.shape.dim) * kScanParts; p.rec_floats = rec_floats(a.shape.dim); p.vblocks = scan_vblocks(a.shape.vdim);
+    const int blocks = std::max(a.n_blocks, a.n_single);
+    p.rec = a.scratch;
+    p.vrec = p.rec + (size_t)blocks * a.shape.heads * p.rec_floats;
+    p.o = p.vrec + (size_t)blocks * a.shape.heads * p.vblocks * TB * kScanCols;
+    return a.f32 ? run<float>(a, p, s, launches) : run<__nv_bfloat16>(a, p, s, launches);
+}
+
+}  // namespace swlm

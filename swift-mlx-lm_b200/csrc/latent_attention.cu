@@ -11,7 +11,8 @@
 //     attention over them with the gate in its epilogue.
 //
 // Scores, softmax and sums are fp32. Where tensor cores take fp32 quantities (absorbed queries, softmax weights) these enter
-// as bf16 hi + lo pairs. The newest rows are read back from the cache like all others, so a row's result does not depend on
+// as bf16 hi + lo pairs. With a sliding window only the pages it reaches into are touched; a sink joins the denominator when
+// the splits are merged, or at the end of a query tile. The newest rows are read back from the cache like all others, so a row's result does not depend on
 // how a sequence was cut into batches.
 #include <cooperative_groups.h>
 
@@ -57,6 +58,7 @@ struct LatentParams {
     LatentRow row;
     int heads, dim, vdim, rot_dims;
     float scale_log2, eps, weight_bias, magnitude;
+    int window; const __nv_bfloat16* sink;
     const float* inv_freq;
     void* q; int q_stride;
     const float* kv; int kv_stride;
@@ -91,6 +93,11 @@ __device__ __forceinline__ void store_query(const LatentParams& p, int rl, int h
     d[0] = hi;
     d[8] = __float2bfloat16_rn(v - __bfloat162float(hi));
 }
+
+// first position a row at `pos` sees
+__device__ __forceinline__ int first_seen(const LatentParams& p, int pos) { return p.window > 0 ? max(0, pos - p.window + 1) : 0; }
+// a head's sink as a score in base 2, -inf when there is none
+__device__ __forceinline__ float sink_log2(const LatentParams& p, int h) { return p.sink ? __bfloat162float(p.sink[h]) * kLog2e : -INFINITY; }
 
 __device__ __forceinline__ int batch_row(const LatentParams& p, int i) { return p.rows ? p.rows[i] : i; }
 template <typename T>
@@ -280,7 +287,7 @@ cudaError_t launch_query(const LatentLaunch& a, const LatentParams& p, cudaStrea
 }
 
 // ---- rows one by one: attention on tensor cores (bf16 pool) -----------------------------------------------------------
-// CTA (split, 16 heads, row): pages split, split + splits, ... of the row's sequence. A page is one bulk copy (rows pitched to
+// CTA (split, 16 heads, row): of the pages the row sees, number split, split + splits, ... A page is one bulk copy (rows pitched to
 // be free of bank conflicts), two pages in flight. Scores: warp (kq, tq) multiplies its quarter of the query columns, held in
 // registers as hi + lo fragments, with 32 of the page's 64 rows; the quarters are added in shared memory. Values: the same
 // page again, 16 latent columns per warp and step, softmax weights as hi + lo.
@@ -310,15 +317,16 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
     pdl_wait();
     const int r = batch_row(p, rl), pos = p.row_pos[r], seq = p.row_seq[r];
     const int32_t* table = p.page_table + (size_t)seq * p.pages_per_seq;
-    const int first_page = table[split];   // (within the table whatever the position: splits <= pages_per_seq)
-    const int n_pages = pos / kPage + 1;
+    const int seen0 = first_seen(p, pos), page0 = seen0 / kPage;
+    const int n_pages = pos / kPage + 1 - page0;
     if (split >= n_pages) return;
+    const int first_page = table[page0 + split];
     const int mine = (n_pages - split + p.splits - 1) / p.splits;
     auto request = [&](int i) {   // thread 0: the i-th page of this CTA
         const unsigned bar = smem_u32(&full_bar[i & 1]);
         mbar_expect(bar, (unsigned)page_bytes);
         bulk_load(smem_u32(pages + (size_t)(i & 1) * page_bytes),
-                  static_cast<const unsigned char*>(p.pool) + (size_t)(i == 0 ? first_page : table[split + i * p.splits]) * page_bytes, (unsigned)page_bytes, bar);
+                  static_cast<const unsigned char*>(p.pool) + (size_t)(i == 0 ? first_page : table[page0 + split + i * p.splits]) * page_bytes, (unsigned)page_bytes, bar);
     };
     if (tid == 0) { request(0); if (mine > 1) request(1); }
 
@@ -385,11 +393,11 @@ __global__ void __launch_bounds__(kSplThreads, 1) latent_split_kernel(const Late
                 const float4 v = *reinterpret_cast<const float4*>(s_sm + (q * kSplHeads + srow) * kSPitch + scol);
                 s4.x += v.x; s4.y += v.y; s4.z += v.z; s4.w += v.w;
             }
-            const int key0 = (split + i * p.splits) * kPage + scol;
+            const int key0 = (page0 + split + i * p.splits) * kPage + scol;
             float s[4] = {s4.x, s4.y, s4.z, s4.w};
             float mx = -INFINITY;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) { s[e] = key0 + e <= pos ? s[e] * p.scale_log2 : -INFINITY; mx = fmaxf(mx, s[e]); }
+            for (int e = 0; e < 4; ++e) { s[e] = key0 + e <= pos && key0 + e >= seen0 ? s[e] * p.scale_log2 : -INFINITY; mx = fmaxf(mx, s[e]); }
 #pragma unroll
             for (int o = 1; o < 16; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
             const float m_new = fmaxf(m_run, mx);       // every page holds at least one row that is seen
@@ -483,7 +491,7 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) latent_simple_kernel(const 
     for (int i = lane; i < p.row.rp; i += 32) acc[i] = 0.f;
     __syncthreads();
     float m = -INFINITY, l = 0.f;
-    for (int key = warp; key <= pos; key += kSimpleWarps) {
+    for (int key = first_seen(p, pos) + warp; key <= pos; key += kSimpleWarps) {
         const T* c = cached_row<T>(p, seq, key);
         float s = 0.f;
         for (int i = lane; i < qw; i += 32) s = fmaf(q[i], lat_get(c + i), s);
@@ -535,11 +543,12 @@ __global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const LatentPar
         }
     pdl_wait();
     const int r = batch_row(p, rl);
-    const int used = min(p.splits, p.row_pos[r] / kPage + 1);
+    const int pos = p.row_pos[r], used = min(p.splits, pos / kPage + 1 - first_seen(p, pos) / kPage);
+    const float sink = sink_log2(p, h);
     const size_t pw = (size_t)p.row.rp + kPartialTail;
     const float* base = p.partial + ((size_t)rl * p.heads + h) * p.splits * pw;
     if (warp == 0) {
-        float top = -INFINITY;
+        float top = sink;
         for (int s = lane; s < used; s += 32) top = fmaxf(top, __ldcg(base + s * pw + p.row.rp));
         for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
         float total = 0.f;
@@ -550,7 +559,7 @@ __global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const LatentPar
             total = fmaf(w, ml.y, total);
         }
         for (int o = 16; o > 0; o >>= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
-        const float inv = 1.0f / total;
+        const float inv = 1.0f / (total + exp2f(sink - top));
         __syncwarp();
         for (int s = lane; s < used; s += 32) w_s[s] *= inv;
     }
@@ -654,7 +663,7 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const LatentParams p
     }
 }
 
-// Cached rows of the spans, one after the other: latents [total_ctx][ctx_ld], rotated parts [total_ctx][rot_ld].
+// Cached rows of the spans (from position `lo` on), one after the other: latents [total_ctx][ctx_ld], rotated parts [total_ctx][rot_ld].
 __global__ void __launch_bounds__(128) latent_gather_kernel(const LatentParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -663,7 +672,7 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const LatentParams p
     int sp = 0;
     while (sp + 1 < p.n_spans && p.spans[sp + 1].ctx0 <= row) ++sp;
     const LatentSpan span = p.spans[sp];
-    const __nv_bfloat16* src = cached_row<__nv_bfloat16>(p, span.seq, row - span.ctx0);
+    const __nv_bfloat16* src = cached_row<__nv_bfloat16>(p, span.seq, span.lo + row - span.ctx0);
     for (int i = lane; i < p.ctx_ld / 8; i += 32) reinterpret_cast<uint4*>(p.ctx_latent + (size_t)row * p.ctx_ld)[i] = reinterpret_cast<const uint4*>(src)[i];
     for (int i = lane; i < p.rot_ld / 8; i += 32) reinterpret_cast<uint4*>(p.ctx_rot + (size_t)row * p.rot_ld)[i] = reinterpret_cast<const uint4*>(src + p.row.rp)[i];
 }
@@ -694,7 +703,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
     const LatentSpan span = p.spans[tile.x];
     const int q0 = tile.y * kLatentQueryTile, nq = min(kLatentQueryTile, span.count - q0);
     const int first_pos = span.pos0 + q0, last_pos = first_pos + nq - 1;
-    const int n_tiles = last_pos / kPfKeys + 1;
+    const int kt0 = first_seen(p, first_pos) / kPfKeys, n_tiles = last_pos / kPfKeys + 1;   // key tiles the first row sees from, and all
     const int cd = p.dim >> 3, cr = p.row.rot >> 3, cv = p.vdim >> 3;
     // 16-byte chunk tid, tid + 256, ... of a tile as (row, chunk of the row), without divisions in the loop
     const int per_row = cd + cr + cv, r_first = tid / per_row, c_first = tid - r_first * per_row, r_step = kPfThreads / per_row, c_step = kPfThreads - r_step * per_row;
@@ -702,7 +711,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
         __nv_bfloat16* ks = kv_sm + stage * STAGE;
         __nv_bfloat16* vs = ks + kPfKeys * PK;
         for (int r = r_first, c = c_first; r < kPfKeys; r += r_step + (c + c_step >= per_row), c += c_step - (c + c_step >= per_row ? per_row : 0)) {
-            const size_t row = span.ctx0 + min(kt * kPfKeys + r, last_pos);
+            const size_t row = span.ctx0 + min(kt * kPfKeys + r, last_pos) - span.lo;
             const __nv_bfloat16* src;
             __nv_bfloat16* dst;
             if (c < cd) { src = p.ctx_k + row * ((size_t)p.heads * p.dim) + (size_t)h * p.dim + 8 * c; dst = ks + r * PK + 8 * c; }
@@ -721,7 +730,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
         }
     }
-    load_tile(0, 0);   // one group with the query rows
+    load_tile(kt0, kt0 & 1);   // one group with the query rows
     unsigned qa[KQ][4];
     const int pos_a = first_pos + warp * 16 + g, pos_b = pos_a + 8;   // positions of this lane's two rows
     const int warp_first = first_pos + warp * 16, warp_last = min(warp_first + 15, last_pos);
@@ -730,16 +739,19 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
 #pragma unroll
     for (int j = 0; j < 2 * NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
 
-    for (int kt = 0; kt < n_tiles; ++kt) {
+    const int seen_a = first_seen(p, pos_a), seen_b = first_seen(p, pos_b), warp_seen = first_seen(p, warp_first);
+    const int full_from = p.window > 0 ? max(0, warp_last - p.window + 1) : 0;   // first position that no row of the warp has left behind
+
+    for (int kt = kt0; kt < n_tiles; ++kt) {
         if (kt + 1 < n_tiles) load_tile(kt + 1, (kt + 1) & 1);
         else asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
-        if (kt == 0) {
+        if (kt == kt0) {
 #pragma unroll
             for (int k = 0; k < KQ; ++k) lat_ldsm(qa[k], smem_u32(q_sm) + (unsigned)((warp * 16 + (lane & 15)) * PK + 16 * k + 8 * (lane >> 4)) * 2u);
         }
-        if (warp_first <= last_pos && kt * kPfKeys <= warp_last) {
+        if (warp_first <= last_pos && kt * kPfKeys <= warp_last && (kt + 1) * kPfKeys > warp_seen) {
             const unsigned kb = smem_u32(kv_sm + (kt & 1) * STAGE), vb = kb + (unsigned)(kPfKeys * PK) * 2u;
             float sacc[8][4];
 #pragma unroll
@@ -753,31 +765,33 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
                     lat_mma(sacc[2 * jp], qa[k], b[0], b[1]);
                     lat_mma(sacc[2 * jp + 1], qa[k], b[2], b[3]);
                 }
-            const bool edge = (kt + 1) * kPfKeys - 1 > warp_first;   // some row does not see the whole tile
+            const bool edge = (kt + 1) * kPfKeys - 1 > warp_first || kt * kPfKeys < full_from;   // some row does not see the whole tile
             float mx_a = -INFINITY, mx_b = -INFINITY;
 #pragma unroll
             for (int j = 0; j < 8; ++j)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = kt * kPfKeys + 8 * j + 2 * t + e;
-                    const float a = !edge || key <= pos_a ? sacc[j][e] * p.scale_log2 : -INFINITY;
-                    const float b = !edge || key <= pos_b ? sacc[j][2 + e] * p.scale_log2 : -INFINITY;
+                    const float a = !edge || (key <= pos_a && key >= seen_a) ? sacc[j][e] * p.scale_log2 : -INFINITY;
+                    const float b = !edge || (key <= pos_b && key >= seen_b) ? sacc[j][2 + e] * p.scale_log2 : -INFINITY;
                     sacc[j][e] = a; sacc[j][2 + e] = b;
                     mx_a = fmaxf(mx_a, a); mx_b = fmaxf(mx_b, b);
                 }
 #pragma unroll
             for (int o = 1; o < 4; o <<= 1) { mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, o)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, o)); }
             const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
-            // a row that sees nothing yet of its tiles (first rows of a warp in the warp's last tile never are: key 0 is seen by all)
-            const float ca = exp2f(m_a - mn_a), cb = exp2f(m_b - mn_b);
+            m_a = m_a == -INFINITY ? mn_a : m_a; m_b = m_b == -INFINITY ? mn_b : m_b;   // (nothing seen so far: sums are zero)
+            // a row whose window starts in a later tile sees nothing of this one: its weights must come out zero
+            const float ra = mn_a == -INFINITY ? 0.f : mn_a, rb = mn_b == -INFINITY ? 0.f : mn_b;
+            const float ca = mn_a == -INFINITY ? 1.f : exp2f(m_a - mn_a), cb = mn_b == -INFINITY ? 1.f : exp2f(m_b - mn_b);
             m_a = mn_a; m_b = mn_b;
             float sa = 0.f, sb = 0.f;
 #pragma unroll
             for (int j = 0; j < 8; ++j)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    sacc[j][e] = exp2f(sacc[j][e] - mn_a); sa += sacc[j][e];
-                    sacc[j][2 + e] = exp2f(sacc[j][2 + e] - mn_b); sb += sacc[j][2 + e];
+                    sacc[j][e] = exp2f(sacc[j][e] - ra); sa += sacc[j][e];
+                    sacc[j][2 + e] = exp2f(sacc[j][2 + e] - rb); sb += sacc[j][2 + e];
                 }
             l_a = l_a * ca + sa; l_b = l_b * cb + sb;
             if (__any_sync(0xffffffffu, ca != 1.0f || cb != 1.0f)) {
@@ -810,13 +824,16 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
     asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
     for (int o = 1; o < 4; o <<= 1) { l_a += __shfl_xor_sync(0xffffffffu, l_a, o); l_b += __shfl_xor_sync(0xffffffffu, l_b, o); }
+    const float sink = sink_log2(p, h);
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
         const int rr = warp * 16 + g + 8 * half;
         if (rr >= nq) continue;
         const int row = span.row0 + q0 + rr;
         const float gate = p.gate ? 1.0f / (1.0f + expf(-p.gate[(size_t)row * p.gate_stride + h])) : 1.0f;
-        const float f = gate / (half ? l_b : l_a);
+        // (every row sees its own key, so its maximum is finite)
+        const float m = half ? m_b : m_a, top = fmaxf(m, sink), own = exp2f(m - top);
+        const float f = gate * own / ((half ? l_b : l_a) * own + exp2f(sink - top));
         __nv_bfloat16* o = static_cast<__nv_bfloat16*>(p.out) + (size_t)row * p.out_stride + (size_t)h * p.vdim;
 #pragma unroll
         for (int j = 0; j < 2 * NV; ++j) {
@@ -829,6 +846,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
 LatentParams latent_params(const LatentLaunch& a) {
     LatentParams p{};
     p.row = a.row; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim; p.rot_dims = a.rot_dims;
+    p.window = a.window; p.sink = a.sink;
     p.scale_log2 = a.scale * kLog2e; p.eps = a.eps; p.weight_bias = a.weight_bias; p.magnitude = a.magnitude; p.inv_freq = a.inv_freq;
     p.q = a.q; p.q_stride = a.q_stride; p.kv = a.kv; p.kv_stride = a.kv_stride; p.gate = a.gate; p.gate_stride = a.gate_stride;
     p.norm_w = a.norm_w; p.uk = a.uk->data; p.uk_ld = a.uk->ld; p.uv = a.uv->data; p.uv_ld = a.uv->ld;
@@ -956,8 +974,9 @@ int latent_init() {
     return SWLM_OK;
 }
 
-// CTAs of the attention kernel fill the GPU once; no more splits than a sequence can have pages.
-int latent_pick_splits(int rows, int heads, int max_pages) {
+// CTAs of the attention kernel fill the GPU once; no more splits than a row can see pages.
+int latent_pick_splits(int rows, int heads, int max_pages, int window) {
+    if (window > 0) max_pages = std::min(max_pages, (window + kPage - 2) / kPage + 1);
     const int per_split = rows * ((heads + kSplHeads - 1) / kSplHeads);
     return std::max(1, std::min(std::min(148 / std::max(1, per_split), max_pages), kLatMaxSplits));
 }

@@ -1,0 +1,356 @@
+// Routed feed-forward: a router picks `top` of the experts for every row, the row's result is the weighted sum of theirs.
+//
+//   few rows (and fp32 plans)  routed_gate_kernel: every CTA works out its row's choice from the router's logits, then streams
+//                              gate and up rows of one chosen expert; routed_down_kernel: a warp per output runs through the
+//                              chosen experts' down rows one after the other, so the sum over experts needs no pass of its own.
+//   more rows (bf16)           routed_choose_kernel, routed_sort_kernel (rows sorted by expert, table of tiles), two grouped
+//                              tensor-core products, routed_sum_kernel.
+//
+// An expert's place among the candidates is the number of candidates before it (larger score, or equal score and lower index),
+// so the choice takes one pass without a sequence of maxima.
+#include <algorithm>
+
+#include "swlm_internal.h"
+
+namespace swlm {
+namespace {
+
+constexpr int kRtThreads = 256, kRtWarps = kRtThreads / 32;
+constexpr int kRtFewRows = 4;       // bf16 rows that go one by one
+
+struct RoutedParams {
+    RoutedShape sh;
+    float scale;
+    GatedAct act;
+    int m;
+    const void* x; int x_stride;
+    const float* z; int z_stride;
+    const __nv_bfloat16 *gate, *up, *down; int in_ld, mid_ld;   // row pitches of gate / up and of down
+    float* out; int out_stride;
+    int* sel; float* weight; int* rank;      // [rows][top]
+    unsigned* counts;                        // [experts]
+    void* mid; int mid_stride;               // [rows * top][mid_stride]
+    __nv_bfloat16* sorted; int sorted_stride;
+    float* y; int y_stride;
+    int4* tiles; int max_tiles, bn;
+};
+
+__device__ __forceinline__ float rt_get(const float* p) { return *p; }
+__device__ __forceinline__ float rt_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void rt_put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void rt_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float rt_lo(unsigned w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float rt_hi(unsigned w) { return __uint_as_float(w & 0xFFFF0000u); }
+__device__ __forceinline__ uint4 rt_stream(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ float rt_dot8(const uint4& w, const float* x, float acc) {
+    const float4 a = *reinterpret_cast<const float4*>(x), b = *reinterpret_cast<const float4*>(x + 4);
+    acc = fmaf(rt_lo(w.x), a.x, acc); acc = fmaf(rt_hi(w.x), a.y, acc); acc = fmaf(rt_lo(w.y), a.z, acc); acc = fmaf(rt_hi(w.y), a.w, acc);
+    acc = fmaf(rt_lo(w.z), b.x, acc); acc = fmaf(rt_hi(w.z), b.y, acc); acc = fmaf(rt_lo(w.w), b.z, acc); return fmaf(rt_hi(w.w), b.w, acc);
+}
+
+// The choice of one row by THREADS threads (a warp or the CTA). s: [experts] scores, gs: [groups] group scores, both shared;
+// sel / w: [top] in order of falling score.
+template <int THREADS>
+__device__ __forceinline__ void choose(const RoutedParams& p, const float* z, float* s, float* gs, int* sel, float* w, int tid) {
+    auto sync = [] { if (THREADS == 32) __syncwarp(); else __syncthreads(); };
+    const int E = p.sh.experts, G = p.sh.groups, per = E / G;
+    for (int i = tid; i < p.sh.top; i += THREADS) { sel[i] = i; w[i] = 0.f; }   // indices stay valid whatever the logits are
+    for (int e = tid; e < E; e += THREADS) s[e] = 1.0f / (1.0f + expf(-z[e]));
+    sync();
+    for (int g = tid; g < G; g += THREADS) {
+        float first = 0.f, second = 0.f;   // scores are positive
+        for (int e = g * per; e < (g + 1) * per; ++e) {
+            const float v = s[e];
+            second = fmaxf(second, fminf(first, v));
+            first = fmaxf(first, v);
+        }
+        gs[g] = first + second;
+    }
+    sync();
+    auto kept = [&](int g) {
+        int before = 0;
+        for (int o = 0; o < G; ++o) before += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+        return before < p.sh.keep;
+    };
+    if (p.sh.keep < G) {
+        // experts of the other groups leave the race (a score is never below zero)
+        for (int e = tid; e < E; e += THREADS) { const bool in = kept(e / per); if (!in) s[e] = -1.0f; }
+        sync();
+    }
+    for (int e = tid; e < E; e += THREADS) {
+        const float v = s[e];
+        int before = 0;
+        for (int o = 0; o < E; ++o) before += s[o] > v || (s[o] == v && o < e);
+        if (v >= 0.f && before < p.sh.top) { sel[before] = e; w[before] = v; }
+    }
+    sync();
+    float total = 0.f;
+    for (int i = 0; i < p.sh.top; ++i) total += w[i];
+    sync();
+    for (int i = tid; i < p.sh.top; i += THREADS) w[i] = w[i] / (total + 1e-20f) * p.scale;
+    sync();
+}
+
+// ---- few rows ---------------------------------------------------------------------------------------------------------
+// CTA (share of the expert's rows, slot of the choice, row).
+template <typename T>
+__global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float rt_smem[];
+    __shared__ int sel[kMaxTop];
+    __shared__ float weight[kMaxTop];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, slot = blockIdx.y, row = blockIdx.z;
+    float* x = rt_smem;                    // [in_ld]
+    float* s = x + p.in_ld;                // [experts], then [groups]
+    const T* src = static_cast<const T*>(p.x) + (size_t)row * p.x_stride;
+    for (int i = tid; i < p.in_ld; i += kRtThreads) x[i] = i < p.sh.width ? rt_get(src + i) : 0.f;
+    choose<kRtThreads>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.experts, sel, weight, tid);
+    if (blockIdx.x == 0 && slot == 0 && tid < p.sh.top) {
+        p.sel[row * p.sh.top + tid] = sel[tid];
+        p.weight[row * p.sh.top + tid] = weight[tid];
+    }
+    const size_t first = (size_t)sel[slot] * p.sh.ff;
+    const int chunks = p.in_ld >> 3;
+    T* mid = static_cast<T*>(p.mid) + (size_t)(row * p.sh.top + slot) * p.mid_stride;
+    constexpr int U = 4;
+    for (int f = blockIdx.x * kRtWarps + warp; f < p.sh.ff; f += gridDim.x * kRtWarps) {
+        const __nv_bfloat16* gr = p.gate + (first + f) * p.in_ld;
+        const __nv_bfloat16* ur = p.up + (first + f) * p.in_ld;
+        float g = 0.f, u = 0.f;
+        for (int c0 = lane; c0 < chunks; c0 += 32 * U) {
+            uint4 gv[U], uv[U];
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                const int c = c0 + 32 * j;
+                gv[j] = c < chunks ? rt_stream(gr + 8 * c) : make_uint4(0, 0, 0, 0);
+                uv[j] = c < chunks ? rt_stream(ur + 8 * c) : make_uint4(0, 0, 0, 0);
+            }
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                const int c = c0 + 32 * j;
+                if (c < chunks) { g = rt_dot8(gv[j], x + 8 * c, g); u = rt_dot8(uv[j], x + 8 * c, u); }
+            }
+        }
+        for (int o = 16; o > 0; o >>= 1) { g += __shfl_xor_sync(0xffffffffu, g, o); u += __shfl_xor_sync(0xffffffffu, u, o); }
+        if (lane == 0) rt_put(mid + f, gated_activation(g, u, p.act));
+    }
+}
+
+// CTA (share of the outputs, row): mid rows of all chosen experts, weighted, in shared memory; a warp per output.
+template <typename T>
+__global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float rt_smem[];   // [top][mid_ld]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, top = p.sh.top;
+    const int* sel = p.sel + row * top;
+    for (int t = 0; t < top; ++t) {
+        const T* mid = static_cast<const T*>(p.mid) + (size_t)(row * top + t) * p.mid_stride;
+        const float w = p.weight[row * top + t];
+        for (int i = tid; i < p.mid_ld; i += kRtThreads) rt_smem[t * p.mid_ld + i] = i < p.sh.ff ? rt_get(mid + i) * w : 0.f;
+    }
+    __syncthreads();
+    const int chunks = p.mid_ld >> 3, all = chunks * top;
+    constexpr int U = 8;
+    for (int n = blockIdx.x * kRtWarps + warp; n < p.sh.width; n += gridDim.x * kRtWarps) {
+        float acc = 0.f;
+        for (int c0 = lane; c0 < all; c0 += 32 * U) {
+            uint4 v[U];
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                const int i = c0 + 32 * j, t = i / chunks, c = i - t * chunks;
+                v[j] = i < all ? rt_stream(p.down + ((size_t)sel[t] * p.sh.width + n) * p.mid_ld + 8 * c) : make_uint4(0, 0, 0, 0);
+            }
+#pragma unroll
+            for (int j = 0; j < U; ++j)
+                if (c0 + 32 * j < all) acc = rt_dot8(v[j], rt_smem + 8 * (c0 + 32 * j), acc);
+        }
+        for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (lane == 0) p.out[(size_t)row * p.out_stride + n] = acc;
+    }
+}
+
+// ---- many rows --------------------------------------------------------------------------------------------------------
+// A warp per row; an expert's rows are numbered as they come.
+constexpr int kChooseWarps = 4;
+__global__ void __launch_bounds__(kChooseWarps * 32) routed_choose_kernel(const RoutedParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float rt_smem[];
+    __shared__ int sel[kChooseWarps][kMaxTop];
+    __shared__ float weight[kChooseWarps][kMaxTop];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, row = blockIdx.x * kChooseWarps + warp;
+    if (row >= p.m) return;
+    float* s = rt_smem + (size_t)warp * (p.sh.experts + p.sh.groups);
+    choose<32>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.experts, sel[warp], weight[warp], lane);
+    for (int t = lane; t < p.sh.top; t += 32) {
+        p.sel[row * p.sh.top + t] = sel[warp][t];
+        p.weight[row * p.sh.top + t] = weight[warp][t];
+        p.rank[row * p.sh.top + t] = (int)atomicAdd(p.counts + sel[warp][t], 1u);
+    }
+}
+
+// Every CTA works out where each expert's rows start; then a warp per (row, slot) copies the row to its place, which replaces
+// its rank. CTA 0 also writes the table of tiles.
+__global__ void __launch_bounds__(kRtThreads) routed_sort_kernel(const RoutedParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ int start[kMaxExperts], tile0[kMaxExperts], warp_rows[kRtWarps], warp_tiles[kRtWarps];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = p.sh.experts;
+    constexpr int PER = kMaxExperts / kRtThreads;   // experts per thread
+    int c[PER], rows = 0, tiles = 0;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int e = tid * PER + j;
+        c[j] = e < E ? (int)__ldcg(p.counts + e) : 0;
+        rows += c[j];
+        tiles += (c[j] + p.bn - 1) / p.bn;
+    }
+    int r = rows, t = tiles;
+    for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, r, o), b = __shfl_up_sync(0xffffffffu, t, o);
+        if (lane >= o) { r += a; t += b; }
+    }
+    if (lane == 31) { warp_rows[warp] = r; warp_tiles[warp] = t; }
+    __syncthreads();
+    for (int w = 0; w < warp; ++w) { r += warp_rows[w]; t += warp_tiles[w]; }
+    r -= rows; t -= tiles;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int e = tid * PER + j;
+        start[e] = r; tile0[e] = t;
+        r += c[j]; t += (c[j] + p.bn - 1) / p.bn;
+    }
+    __syncthreads();
+    if (blockIdx.x == 0) {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            const int e = tid * PER + j;
+            for (int i = 0; i * p.bn < c[j]; ++i) p.tiles[tile0[e] + i] = make_int4(e, start[e] + i * p.bn, min(p.bn, c[j] - i * p.bn), 0);
+        }
+        int used = 0;
+        for (int w = 0; w < kRtWarps; ++w) used += warp_tiles[w];
+        for (int i = used + tid; i < p.max_tiles; i += kRtThreads) p.tiles[i] = make_int4(0, 0, 0, 0);
+    }
+    const int chunks = p.sorted_stride >> 3, all = p.m * p.sh.top;
+    for (int a = blockIdx.x * kRtWarps + warp; a < all; a += gridDim.x * kRtWarps) {
+        const int at = start[p.sel[a]] + p.rank[a];
+        const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.x) + (size_t)(a / p.sh.top) * p.x_stride);
+        uint4* dst = reinterpret_cast<uint4*>(p.sorted + (size_t)at * p.sorted_stride);
+        for (int i = lane; i < chunks; i += 32) dst[i] = src[i];
+        __syncwarp();
+        if (lane == 0) p.rank[a] = at;
+    }
+}
+
+__global__ void __launch_bounds__(kRtThreads) routed_sum_kernel(const RoutedParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int row = blockIdx.y, i = (blockIdx.x * kRtThreads + threadIdx.x) * 4;
+    if (blockIdx.x == 0 && blockIdx.y == 0)
+        for (int e = threadIdx.x; e < p.sh.experts; e += kRtThreads) p.counts[e] = 0;
+    if (i >= p.sh.width) return;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int t = 0; t < p.sh.top; ++t) {
+        const float w = p.weight[row * p.sh.top + t];
+        const float4 y = *reinterpret_cast<const float4*>(p.y + (size_t)p.rank[row * p.sh.top + t] * p.y_stride + i);   // (rows are padded to 8)
+        v.x = fmaf(w, y.x, v.x); v.y = fmaf(w, y.y, v.y); v.z = fmaf(w, y.z, v.z); v.w = fmaf(w, y.w, v.w);
+    }
+    float* o = p.out + (size_t)row * p.out_stride + i;
+    const float r[4] = {v.x, v.y, v.z, v.w};
+    for (int j = 0; j < 4 && i + j < p.sh.width; ++j) o[j] = r[j];
+}
+
+// ---- launches ---------------------------------------------------------------------------------------------------------
+int up8(int v) { return (v + 7) / 8 * 8; }
+size_t up256(size_t v) { return (v + 255) / 256 * 256; }
+bool few(int m, bool f32) { return f32 || m <= kRtFewRows; }
+struct RoutedScratch { size_t sel, weight, rank, tiles, mid, sorted, y, total; };
+RoutedScratch layout(const RoutedShape& s, int m, bool f32) {
+    RoutedScratch l;
+    const size_t a = (size_t)m * s.top;
+    l.sel = 0;
+    l.weight = l.sel + up256(a * 4);
+    l.rank = l.weight + up256(a * 4);
+    l.tiles = l.rank + up256(a * 4);
+    l.mid = l.tiles + (few(m, f32) ? 0 : up256((size_t)grouped_max_tiles((int)a, s.experts) * 16));
+    l.sorted = l.mid + up256(a * up8(s.ff) * (f32 ? 4 : 2));
+    l.y = l.sorted + (few(m, f32) ? 0 : up256(a * up8(s.width) * 2));
+    l.total = l.y + (few(m, f32) ? 0 : up256(a * up8(s.width) * 4));
+    return l;
+}
+constexpr size_t kRtMaxSmem = 200 * 1024;
+size_t gate_smem(const RoutedShape& s) { return ((size_t)up8(s.width) + s.experts + s.groups) * 4; }
+size_t down_smem(const RoutedShape& s) { return (size_t)s.top * up8(s.ff) * 4; }
+
+template <typename T>
+int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
+    // about two CTAs per SM over the chosen experts of all rows
+    const int pairs = (p.sh.ff + kRtWarps - 1) / kRtWarps, gx = std::max(1, std::min(pairs, (4 * 148 + p.sh.top * p.m - 1) / (p.sh.top * p.m)));
+    cudaError_t e = launch_k(routed_gate_kernel<T>, dim3(gx, p.sh.top, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
+    if (e != cudaSuccess) return cuda_fail(e, "routed gate launch");
+    const int outs = (p.sh.width + kRtWarps - 1) / kRtWarps, dx = std::max(1, std::min(outs, (3 * 148 + p.m - 1) / p.m));
+    e = launch_k(routed_down_kernel<T>, dim3(dx, p.m), dim3(kRtThreads), down_smem(p.sh), s, p);
+    if (e != cudaSuccess) return cuda_fail(e, "routed down launch");
+    *launches += 2;
+    return SWLM_OK;
+}
+
+}  // namespace
+
+int routed_init() {
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    return SWLM_OK;
+}
+bool routed_supported(const RoutedShape& s) {
+    return s.experts > 0 && s.experts <= kMaxExperts && s.top > 0 && s.top <= kMaxTop && s.groups > 0 && s.experts % s.groups == 0 && s.keep > 0 &&
+           s.keep <= s.groups && s.top <= s.keep * (s.experts / s.groups) && s.width > 0 && s.ff > 0 && gate_smem(s) <= kRtMaxSmem && down_smem(s) <= kRtMaxSmem;
+}
+size_t routed_scratch_bytes(const RoutedShape& s, int m, bool f32) { return layout(s, m, f32).total; }
+
+int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches) {
+    if (a.m <= 0) return SWLM_OK;
+    const RoutedScratch l = layout(a.shape, a.m, a.f32);
+    RoutedParams p{};
+    p.sh = a.shape; p.scale = a.scale; p.act = a.act; p.m = a.m; p.x = a.x; p.x_stride = a.x_stride; p.z = a.z; p.z_stride = a.z_stride;
+    p.gate = a.gate->data; p.up = a.up->data; p.down = a.down->data; p.in_ld = a.gate->ld; p.mid_ld = a.down->ld; p.out = a.out; p.out_stride = a.out_stride;
+    p.sel = reinterpret_cast<int*>(a.scratch + l.sel); p.weight = reinterpret_cast<float*>(a.scratch + l.weight); p.rank = reinterpret_cast<int*>(a.scratch + l.rank);
+    p.counts = a.counts; p.mid = a.scratch + l.mid; p.mid_stride = up8(a.shape.ff);
+    if (few(a.m, a.f32)) return a.f32 ? few_rows<float>(p, s, launches) : few_rows<__nv_bfloat16>(p, s, launches);
+
+    const int all = a.m * a.shape.top, E = a.shape.experts;
+    p.sorted = reinterpret_cast<__nv_bfloat16*>(a.scratch + l.sorted); p.sorted_stride = up8(a.shape.width);
+    p.y = reinterpret_cast<float*>(a.scratch + l.y); p.y_stride = up8(a.shape.width);
+    p.tiles = reinterpret_cast<int4*>(a.scratch + l.tiles); p.bn = grouped_bn(all, E); p.max_tiles = grouped_max_tiles(all, E);
+    if ((a.x_stride & 7) || (reinterpret_cast<uintptr_t>(a.x) & 15)) { set_error("routed feed-forward: rows must be 16-byte aligned"); return SWLM_ERR_INVALID; }
+    cudaError_t e = launch_k(routed_choose_kernel, dim3((a.m + kChooseWarps - 1) / kChooseWarps), dim3(kChooseWarps * 32), (size_t)kChooseWarps * (E + a.shape.groups) * 4, s, p);
+    if (e != cudaSuccess) return cuda_fail(e, "routed choice launch");
+    e = launch_k(routed_sort_kernel, dim3(std::min((all + kRtWarps - 1) / kRtWarps, 4 * 148)), dim3(kRtThreads), 0, s, p);
+    if (e != cudaSuccess) return cuda_fail(e, "routed sort launch");
+    ProductLaunch g;
+    g.w = a.gate; g.w2 = a.up; g.act = a.act; g.m = all; g.x = p.sorted; g.x_stride = p.sorted_stride; g.status = a.status;
+    g.experts = E; g.tiles = p.tiles; g.max_tiles = p.max_tiles; g.group_bn = p.bn;
+    g.out.y[0] = p.mid; g.out.stride[0] = p.mid_stride;
+    for (int& end : g.out.end) end = a.shape.ff;
+    int rc = launch_product(g, s);
+    if (rc) return rc;
+    ProductLaunch d = g;
+    d.w = a.down; d.w2 = nullptr; d.x = p.mid; d.x_stride = p.mid_stride;
+    d.out.y[0] = p.y; d.out.stride[0] = p.y_stride; d.out.f32[0] = 1;
+    for (int& end : d.out.end) end = a.shape.width;
+    if ((rc = launch_product(d, s))) return rc;
+    e = launch_k(routed_sum_kernel, dim3((a.shape.width + kRtThreads * 4 - 1) / (kRtThreads * 4), a.m), dim3(kRtThreads), 0, s, p);
+    if (e != cudaSuccess) return cuda_fail(e, "routed sum launch");
+    *launches += 5;
+    return SWLM_OK;
+}
+
+}  // namespace swlm

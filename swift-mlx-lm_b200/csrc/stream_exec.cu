@@ -1,6 +1,7 @@
 // Executor of fp32-stream plans: step list -> launches, the paged pool of latent rows, and one row executor that runs decode
 // steps, prompt chunks and mixed batches alike. A batch is a list of rows, each with its token, sequence and position; the
-// only step that looks beyond its own row is latent attention, which finds the cached rows through the page table.
+// only steps that look beyond their own row are latent attention, which finds the cached rows through the page table, and
+// the gated delta rule, which carries a state per sequence.
 #include <cmath>
 #include <cstdio>
 #include <cstring>
@@ -100,7 +101,19 @@ bool is_norm(int kind) {
 }
 bool is_postnorm(int kind) { return kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_RMSNORM; }
 bool norm_stores(int kind) { return kind == SWLM_STEP_COPY_RMSNORM || kind == SWLM_STEP_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM; }
-bool reads(const swlm_step& s, int buf) { return s.in_buf == buf || (s.kind != SWLM_STEP_PRODUCT && !is_norm(s.kind) && (s.in2_buf == buf || s.in3_buf == buf)); }
+bool reads(const swlm_step& s, int buf) {
+    if (s.in_buf == buf) return true;
+    return s.kind != SWLM_STEP_PRODUCT && !is_norm(s.kind) && (s.in2_buf == buf || s.in3_buf == buf || s.in4_buf == buf);
+}
+bool is_glu(int kind) { return kind == SWLM_STEP_SWIGLU || kind == SWLM_STEP_GEGLU || kind == SWLM_STEP_CLAMPED_GLU; }
+GatedAct glu_of(const swlm_step& s) {
+    GatedAct a;
+    a.kind = s.kind == SWLM_STEP_GEGLU ? GATED_ACT_GELU_TANH : s.kind == SWLM_STEP_CLAMPED_GLU ? GATED_ACT_CLAMPED : GATED_ACT_SILU;
+    a.alpha = s.scale;
+    a.limit = s.limit;
+    return a;
+}
+const char* glu_name(int kind) { return kind == GATED_ACT_GELU_TANH ? "geglu" : kind == GATED_ACT_CLAMPED ? "clamped glu" : "swiglu"; }
 
 }  // namespace
 
@@ -113,6 +126,7 @@ int stream_compile(swlm_plan* plan) {
     int rc;
     auto widen = [&](int buf, int n) { plan->stream_width[buf] = std::max(plan->stream_width[buf], (n + 7) / 8 * 8); };
     plan->latent.assign(std::max(0, d.latent_layers), LatentLayer{});
+    plan->delta.assign(std::max(0, d.delta_layers), DeltaLayer{});
     widen(SWLM_BUF_HIDDEN, d.hidden);
     widen(SWLM_BUF_RESIDUAL, d.hidden);
     widen(SWLM_BUF_LOGITS, d.vocab);
@@ -143,17 +157,18 @@ int stream_compile(swlm_plan* plan) {
             L.kind = L_PRODUCT;
             if (!act_buf(plan, s.in_buf) || !any_buf(s.out_buf) || s.out_buf == s.in_buf || s.out_buf == SWLM_BUF_RESIDUAL) { set_error("product '%s': bad buffers", s.weight); return SWLM_ERR_INVALID; }
             if ((rc = find_matrix(ctx, s.weight, s.n, s.k, &L.m1))) return rc;
-            widen(s.in_buf, s.k);
-            widen(s.out_buf, s.n);
+            if (s.in_off < 0 || s.out_off < 0 || (s.in_off & 7) || (s.out_buf == SWLM_BUF_LOGITS && s.out_off)) { set_error("product '%s': input columns start at multiples of 8", s.weight); return SWLM_ERR_INVALID; }
+            widen(s.in_buf, s.in_off + s.k);
+            widen(s.out_buf, s.out_off + s.n);
             // gate, up, gated activation -> one launch
-            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && (st[i + 2].kind == SWLM_STEP_SWIGLU || st[i + 2].kind == SWLM_STEP_GEGLU) &&
+            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && is_glu(st[i + 2].kind) && !s.in_off && !s.out_off && !st[i + 1].in_off && !st[i + 1].out_off &&
                 st[i + 1].in_buf == s.in_buf && st[i + 1].k == s.k && st[i + 1].n == s.n && st[i + 2].in_buf == s.out_buf &&
                 st[i + 2].in2_buf == st[i + 1].out_buf && st[i + 2].n == s.n && act_buf(plan, st[i + 2].out_buf) && st[i + 2].out_buf != s.in_buf &&
                 act_buf(plan, s.out_buf) && act_buf(plan, st[i + 1].out_buf)) {
                 if ((rc = find_matrix(ctx, st[i + 1].weight, s.n, s.k, &L.m2))) return rc;
                 widen(st[i + 1].out_buf, s.n);
                 widen(st[i + 2].out_buf, s.n);
-                L.gated_act = st[i + 2].kind == SWLM_STEP_GEGLU ? GATED_ACT_GELU_TANH : GATED_ACT_SILU;
+                L.act = glu_of(st[i + 2]);
                 L.seg_buf[0] = st[i + 2].out_buf; L.seg_end[0] = s.n;
                 L.seg_buf[1] = s.out_buf; L.seg_buf[2] = st[i + 1].out_buf;   // where the halves go when they run apart
                 L.steps_covered = 3;
@@ -161,20 +176,28 @@ int stream_compile(swlm_plan* plan) {
                 break;
             }
             std::vector<std::string> names{s.weight};
-            L.seg_buf[0] = s.out_buf; L.seg_end[0] = s.n;
+            L.seg_buf[0] = s.out_buf; L.seg_off[0] = s.out_off; L.seg_end[0] = s.n;
             L.label = std::string("product ") + s.weight;
+            // the soft cap of the logits happens where they are stored
+            if (s.out_buf == SWLM_BUF_LOGITS && i + 1 < st.size() && st[i + 1].kind == SWLM_STEP_SOFTCAP && st[i + 1].scale > 0.f && st[i + 1].n == s.n) {
+                L.softcap = st[i + 1].scale;
+                L.steps_covered = 2;
+                L.label += " + softcap";
+                break;
+            }
             size_t j = i + 1;
-            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && st[j].in_buf == s.in_buf && st[j].k == s.k &&
-                   st[j].out_buf != s.in_buf && any_buf(st[j].out_buf) && st[j].out_buf != SWLM_BUF_LOGITS && s.out_buf != SWLM_BUF_LOGITS) {
+            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && st[j].in_buf == s.in_buf && st[j].in_off == s.in_off && st[j].k == s.k &&
+                   st[j].out_off >= 0 && st[j].out_buf != s.in_buf && any_buf(st[j].out_buf) && st[j].out_buf != SWLM_BUF_LOGITS && s.out_buf != SWLM_BUF_LOGITS) {
                 bool clash = false;
-                for (size_t q = i; q < j; ++q) clash |= st[q].out_buf == st[j].out_buf || !strcmp(st[q].weight, st[j].weight);
+                for (size_t q = i; q < j; ++q)
+                    clash |= (st[q].out_buf == st[j].out_buf && st[q].out_off < st[j].out_off + st[j].n && st[j].out_off < st[q].out_off + st[q].n) || !strcmp(st[q].weight, st[j].weight);
                 // a gate / up pair that starts here keeps its own launch
-                if (clash || (j + 2 < st.size() && (st[j + 2].kind == SWLM_STEP_SWIGLU || st[j + 2].kind == SWLM_STEP_GEGLU) && st[j + 2].in_buf == st[j].out_buf)) break;
+                if (clash || (j + 2 < st.size() && is_glu(st[j + 2].kind) && st[j + 2].in_buf == st[j].out_buf)) break;
                 const Matrix* m;
                 if ((rc = find_matrix(ctx, st[j].weight, st[j].n, st[j].k, &m))) return rc;
-                widen(st[j].out_buf, st[j].n);
+                widen(st[j].out_buf, st[j].out_off + st[j].n);
                 const int q = (int)names.size();
-                L.seg_buf[q] = st[j].out_buf; L.seg_end[q] = L.seg_end[q - 1] + st[j].n;
+                L.seg_buf[q] = st[j].out_buf; L.seg_off[q] = st[j].out_off; L.seg_end[q] = L.seg_end[q - 1] + st[j].n;
                 names.push_back(st[j].weight);
                 L.label += std::string(" ") + st[j].weight;
                 ++j;
@@ -184,12 +207,12 @@ int stream_compile(swlm_plan* plan) {
             if (L.n_seg > 1 && (rc = concat_matrices(ctx, names, &L.m1))) return rc;
             break;
         }
-        case SWLM_STEP_SWIGLU: case SWLM_STEP_GEGLU:
+        case SWLM_STEP_SWIGLU: case SWLM_STEP_GEGLU: case SWLM_STEP_CLAMPED_GLU:
             L.kind = L_SWIGLU;
-            L.gated_act = s.kind == SWLM_STEP_GEGLU ? GATED_ACT_GELU_TANH : GATED_ACT_SILU;
+            L.act = glu_of(s);
             if (!act_buf(plan, s.in_buf) || !act_buf(plan, s.in2_buf) || !act_buf(plan, s.out_buf) || s.n <= 0) { set_error("gated activation: bad buffers"); return SWLM_ERR_INVALID; }
             widen(s.in_buf, s.n); widen(s.in2_buf, s.n); widen(s.out_buf, s.n);
-            L.label = L.gated_act ? "geglu" : "swiglu";
+            L.label = glu_name(L.act.kind);
             break;
         case SWLM_STEP_LATENT_ATTN: {
             L.kind = L_LATENT;
@@ -206,6 +229,10 @@ int stream_compile(swlm_plan* plan) {
             if ((rc = concat_matrices(ctx, pair, &both))) return rc;
             L.m1 = uk; L.m2 = uv;
             if ((rc = stream_rope_table(plan, s, &L.rope_table))) return rc;
+            if (s.window_left < 0) { set_error("latent attention: window %d", s.window_left); return SWLM_ERR_INVALID; }
+            if (s.weight4[0] && (rc = find_vector(ctx, s.weight4, s.heads, &L.dv[0]))) return rc;
+            L.window_set = (int)(std::find(plan->windows.begin(), plan->windows.end(), s.window_left) - plan->windows.begin());
+            if (L.window_set == (int)plan->windows.size()) plan->windows.push_back(s.window_left);
             LatentLayer& ll = plan->latent[s.layer];
             if (ll.rank && (ll.rank != s.n || ll.rot != s.key_dim)) { set_error("latent layer %d is used with two row sizes", s.layer); return SWLM_ERR_INVALID; }
             ll.rank = s.n; ll.rot = s.key_dim; ll.row = latent_row(s.n, s.key_dim, plan->all_f32());
@@ -219,6 +246,56 @@ int stream_compile(swlm_plan* plan) {
             L.label = std::string("latent_attention ") + s.weight2;
             break;
         }
+        case SWLM_STEP_GATED_DELTA: {
+            L.kind = L_DELTA;
+            if (s.layer < 0 || s.layer >= d.delta_layers) { set_error("gated delta rule: layer %d has no state", s.layer); return SWLM_ERR_INVALID; }
+            DeltaShape shape;
+            shape.heads = s.heads; shape.groups = s.groups; shape.dim = s.key_dim; shape.vdim = s.value_dim; shape.taps = s.conv_kernel;
+            if (!delta_supported(shape) || (s.k != 1 && s.k != s.key_dim) || (s.gate_act != SWLM_GATE_SILU && s.gate_act != SWLM_GATE_SIGMOID)) { set_error("gated delta rule: %d heads over %d groups, %d x %d, %d taps, %d decays per head", s.heads, s.groups, s.key_dim, s.value_dim, s.conv_kernel, s.k); return SWLM_ERR_UNSUPPORTED; }
+            if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || !any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf) || s.in2_buf == s.in3_buf ||
+                !act_buf(plan, s.in4_buf) || !act_buf(plan, s.out_buf) || s.in4_buf == s.in_buf || s.out_buf == s.in_buf) { set_error("gated delta rule: q | k | v, gate and result in scratch 0..2, step sizes and decays in scratch 3 and 4"); return SWLM_ERR_INVALID; }
+            const char* names[6] = {s.weight, s.weight2, s.weight3, s.weight4, s.weight5, s.weight6};
+            const int counts[6] = {s.groups * s.key_dim * s.conv_kernel, s.groups * s.key_dim * s.conv_kernel, s.heads * s.value_dim * s.conv_kernel, s.value_dim, s.heads, s.heads * s.k};
+            for (int q = 0; q < 6; ++q) if ((rc = find_vector(ctx, names[q], counts[q], &L.dv[q]))) return rc;
+            DeltaLayer& dl = plan->delta[s.layer];
+            if (dl.shape.heads && memcmp(&dl.shape, &shape, sizeof(shape))) { set_error("gated-delta layer %d is used with two shapes", s.layer); return SWLM_ERR_INVALID; }
+            dl.shape = shape;
+            widen(s.in_buf, shape.channels());
+            widen(s.in2_buf, s.heads);
+            widen(s.in3_buf, s.heads * s.k);
+            widen(s.in4_buf, s.heads * s.value_dim);
+            widen(s.out_buf, s.heads * s.value_dim);
+            L.label = std::string("gated_delta ") + s.weight4;
+            break;
+        }
+        case SWLM_STEP_ROUTED_MLP: {
+            L.kind = L_ROUTED;
+            const RoutedShape shape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k};
+            if (!routed_supported(shape)) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k); return SWLM_ERR_UNSUPPORTED; }
+            if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || s.out_buf != SWLM_BUF_HIDDEN || s.n != d.hidden) { set_error("routed feed-forward: input in scratch 0..2, logits in scratch 3 or 4, result in hidden"); return SWLM_ERR_INVALID; }
+            const char* suffix[3] = {s.weight2, s.weight3, s.weight4};
+            const Matrix** into[3] = {&L.m1, &L.m2, &L.m3};
+            for (int q = 0; q < 3; ++q) {
+                std::vector<std::string> names;
+                for (int e = 0; e < s.experts; ++e) {
+                    names.push_back(std::string(s.weight) + std::to_string(e) + suffix[q]);
+                    const Matrix* m;
+                    if ((rc = find_matrix(ctx, names.back().c_str(), q < 2 ? s.k : s.n, q < 2 ? s.n : s.k, &m))) return rc;
+                }
+                if ((rc = concat_matrices(ctx, names, into[q]))) return rc;
+            }
+            L.act.kind = GATED_ACT_CLAMPED; L.act.alpha = s.glu_alpha; L.act.limit = s.limit;
+            widen(s.in_buf, s.n);
+            widen(s.in2_buf, s.experts);
+            widen(s.out_buf, s.n);
+            L.label = std::string("routed_mlp ") + s.weight;
+            break;
+        }
+        case SWLM_STEP_SOFTCAP:
+            L.kind = L_SOFTCAP;
+            if (s.in_buf != SWLM_BUF_LOGITS || s.n != d.vocab || !(s.scale > 0.f)) { set_error("soft cap: of the logits, by a positive number"); return SWLM_ERR_INVALID; }
+            L.label = "softcap";
+            break;
         case SWLM_STEP_ARGMAX:
             L.kind = L_ARGMAX;
             if (s.in_buf != SWLM_BUF_LOGITS || s.n != d.vocab) { set_error("argmax: reads the logits"); return SWLM_ERR_INVALID; }
@@ -233,13 +310,15 @@ int stream_compile(swlm_plan* plan) {
     }
     for (int l = 0; l < d.latent_layers; ++l)
         if (!plan->latent[l].rank && st.size() > 1) { set_error("latent layer %d has no step", l); return SWLM_ERR_INVALID; }
+    for (int l = 0; l < d.delta_layers; ++l)
+        if (!plan->delta[l].shape.heads && st.size() > 1) { set_error("gated-delta layer %d has no step", l); return SWLM_ERR_INVALID; }
 
     // A norm rides with the product behind it when that is its only reader: few rows compute it in the product's prologue,
     // more rows run it in front.
     for (size_t i = 0; i + 1 < plan->launches.size(); ++i) {
         const Launch A = plan->launches[i];
         Launch& B = plan->launches[i + 1];
-        if (A.kind != L_RMSNORM || B.kind != L_PRODUCT || B.st.in_buf != A.st.out_buf) continue;
+        if (A.kind != L_RMSNORM || B.kind != L_PRODUCT || B.st.in_buf != A.st.out_buf || B.st.in_off) continue;
         bool ok = true;
         for (size_t j = i + 2; j < plan->launches.size(); ++j) {
             const Launch& C = plan->launches[j];
@@ -351,6 +430,8 @@ int bufs_rows(swlm_state* s, StreamBufs* b, int rows, int wants) {
     return SWLM_OK;
 }
 
+RoutedShape routed_shape(const swlm_step& s) { return RoutedShape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k}; }
+
 size_t part_need(const swlm_plan* plan, int rows, int wants) {
     size_t need = 0;
     if (plan->all_f32()) return 0;
@@ -367,23 +448,33 @@ int bufs_scratch(swlm_state* s, StreamBufs* b, const RowBatch& r) {
     for (const Launch& L : plan->launches) {
         if (L.kind != L_LATENT || r.n_long == 0) continue;
         const LatentLayer& ll = plan->latent[L.st.layer];
-        expand = std::max(expand, latent_expand_bytes(ll.row, L.st.heads, L.st.head_dim, L.st.value_dim, r.total_ctx));
-        part = std::max(part, product_part_floats(L.st.heads * (L.st.head_dim + L.st.value_dim), ll.rank, r.total_ctx, false));
+        const int ctx = r.total_ctx[L.window_set];
+        expand = std::max(expand, latent_expand_bytes(ll.row, L.st.heads, L.st.head_dim, L.st.value_dim, ctx));
+        part = std::max(part, product_part_floats(L.st.heads * (L.st.head_dim + L.st.value_dim), ll.rank, ctx, false));
     }
     if ((rc = grow(&b->part, &b->part_cap, part, s->stream))) return rc;
     if ((rc = grow(&b->expand, &b->expand_cap, expand, s->stream))) return rc;
+    size_t delta = 0, routed = 0;
+    for (const Launch& L : plan->launches) {
+        if (L.kind == L_DELTA) {
+            const DeltaShape& sh = plan->delta[L.st.layer].shape;
+            if (r.n_runs || (r.n_single && !delta_step_fits(sh))) delta = std::max(delta, delta_scratch_floats(sh, std::max(r.n_blocks, r.n_single), r.rows));
+        } else if (L.kind == L_ROUTED) routed = std::max(routed, routed_scratch_bytes(routed_shape(L.st), r.rows, plan->all_f32()));
+    }
+    if ((rc = grow(&b->delta, &b->delta_cap, delta, s->stream))) return rc;
+    if ((rc = grow(&b->routed, &b->routed_cap, routed, s->stream))) return rc;
     if ((rc = grow(&b->qcat, &b->qcat_cap, (size_t)r.n_short * plan->latent_q_floats, s->stream))) return rc;
     size_t partial = 0;
     for (const Launch& L : plan->launches)
         if (L.kind == L_LATENT)
-            partial = std::max(partial, (size_t)r.n_short * latent_pick_splits(r.n_short, L.st.heads, r.splits_pages) * latent_partial_floats(plan->latent[L.st.layer].row, L.st.heads));
+            partial = std::max(partial, (size_t)r.n_short * latent_pick_splits(r.n_short, L.st.heads, r.splits_pages, L.st.window_left) * latent_partial_floats(plan->latent[L.st.layer].row, L.st.heads));
     return grow(&b->partial, &b->partial_cap, partial, s->stream);
 }
 
 void bufs_free(StreamBufs* b) {
     for (void* p : b->buf) cudaFree(p);
     cudaFree(b->res2); cudaFree(b->meta); cudaFree(b->argmax_out); cudaFree(b->qcat); cudaFree(b->partial); cudaFree(b->part);
-    cudaFree(b->expand); cudaFree(b->argmax_val); cudaFree(b->argmax_idx);
+    cudaFree(b->expand); cudaFree(b->delta); cudaFree(b->routed); cudaFree(b->argmax_val); cudaFree(b->argmax_idx);
     *b = StreamBufs{};
 }
 
@@ -431,8 +522,8 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             if (m == 0) break;
             const int32_t* idx = head ? r.wants_idx : nullptr;
             ProductLaunch a;
-            a.w = L.m1; a.w2 = L.m2; a.act = L.gated_act; a.m = m; a.x_f32 = f32;
-            a.x = b->buf[st.in_buf]; a.x_stride = s->width[st.in_buf];
+            a.w = L.m1; a.w2 = L.m2; a.act = L.act; a.m = m; a.x_f32 = f32;
+            a.x = static_cast<unsigned char*>(b->buf[st.in_buf]) + (size_t)st.in_off * stored_bytes(plan, st.in_buf); a.x_stride = s->width[st.in_buf];
             a.part = b->part; a.part_floats = b->part_cap; a.status = s->pf_status;
             if (head && idx && !L.norm.kind) { set_error("the output head must follow a norm that nothing else reads"); return SWLM_ERR_UNSUPPORTED; }
             if (L.norm.kind) {
@@ -444,8 +535,9 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
                     if (rc) return rc;
                 }
             }
-            auto segment = [&](int q, int buf, int end) {
-                a.out.y[q] = b->buf[buf]; a.out.stride[q] = s->width[buf]; a.out.f32[q] = stored_f32(plan, buf) ? 1 : 0; a.out.end[q] = end;
+            a.out.softcap = L.softcap;
+            auto segment = [&](int q, int buf, int off, int end) {
+                a.out.y[q] = static_cast<unsigned char*>(b->buf[buf]) + (size_t)off * stored_bytes(plan, buf); a.out.stride[q] = s->width[buf]; a.out.f32[q] = stored_f32(plan, buf) ? 1 : 0; a.out.end[q] = end;
             };
             if (L.m2 && !product_takes_gate(m, L.m1->k, f32)) {
                 // gate and up one after the other, then the activation
@@ -459,12 +551,12 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
                     s->launches += product_launch_count(c);
                 }
                 if (!rc) rc = launch_stream_gated(m, L.m1->n, b->buf[L.seg_buf[1]], s->width[L.seg_buf[1]], b->buf[L.seg_buf[2]], s->width[L.seg_buf[2]],
-                                                  b->buf[L.seg_buf[0]], s->width[L.seg_buf[0]], f32, L.gated_act, stream);
+                                                  b->buf[L.seg_buf[0]], s->width[L.seg_buf[0]], f32, L.act, stream);
                 s->launches += 1;
                 break;
             }
             a.out.count = L.n_seg;
-            for (int q = 0; q < L.n_seg; ++q) segment(q, L.seg_buf[q], L.seg_end[q]);
+            for (int q = 0; q < L.n_seg; ++q) segment(q, L.seg_buf[q], L.seg_off[q], L.seg_end[q]);
             for (int q = L.n_seg; q < kMaxProductSegs; ++q) a.out.end[q] = L.seg_end[L.n_seg - 1];
             rc = launch_product(a, stream);
             s->launches += product_launch_count(a);
@@ -472,15 +564,52 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
         }
         case L_SWIGLU:
             rc = launch_stream_gated(r.rows, st.n, b->buf[st.in_buf], s->width[st.in_buf], b->buf[st.in2_buf], s->width[st.in2_buf], b->buf[st.out_buf],
-                                     s->width[st.out_buf], f32, L.gated_act, stream);
+                                     s->width[st.out_buf], f32, L.act, stream);
             s->launches += 1;
             break;
+        case L_SOFTCAP:
+            rc = launch_stream_softcap(wants, st.n, static_cast<float*>(b->buf[SWLM_BUF_LOGITS]), s->width[SWLM_BUF_LOGITS], st.scale, stream);
+            s->launches += wants > 0 ? 1 : 0;
+            break;
+        case L_DELTA: {
+            DeltaLaunch a;
+            a.shape = plan->delta[st.layer].shape;
+            a.decay_dim = st.k; a.gate_act = st.gate_act; a.eps = st.eps; a.unit_eps = st.eps2; a.q_scale = st.scale; a.f32 = f32;
+            a.qkv = b->buf[st.in_buf]; a.qkv_stride = s->width[st.in_buf];
+            a.beta = static_cast<const float*>(b->buf[st.in2_buf]); a.beta_stride = s->width[st.in2_buf];
+            a.decay = static_cast<const float*>(b->buf[st.in3_buf]); a.decay_stride = s->width[st.in3_buf];
+            a.gate = b->buf[st.in4_buf]; a.gate_stride = s->width[st.in4_buf];
+            a.conv_q = L.dv[0]->data; a.conv_k = L.dv[1]->data; a.conv_v = L.dv[2]->data; a.norm_w = L.dv[3]->data; a.a_log = L.dv[4]->data; a.dt_bias = L.dv[5]->data;
+            a.ring = s->delta_ring[st.layer]; a.state = s->delta_state[st.layer];
+            a.row_seq = r.seq; a.row_pos = r.pos;
+            a.out = b->buf[st.out_buf]; a.out_stride = s->width[st.out_buf];
+            a.n_single = r.n_single; a.single_rows = r.single_rows; a.n_runs = r.n_runs; a.runs = r.runs; a.n_blocks = r.n_blocks; a.block_run = r.block_run;
+            a.scratch = b->delta; a.status = s->pf_status;
+            int n = 0;
+            rc = launch_delta(a, stream, &n);
+            s->launches += n;
+            break;
+        }
+        case L_ROUTED: {
+            RoutedLaunch a;
+            a.shape = routed_shape(st); a.scale = st.scale; a.act = L.act; a.m = r.rows; a.f32 = f32;
+            a.x = b->buf[st.in_buf]; a.x_stride = s->width[st.in_buf];
+            a.z = static_cast<const float*>(b->buf[st.in2_buf]); a.z_stride = s->width[st.in2_buf];
+            a.gate = L.m1; a.up = L.m2; a.down = L.m3;
+            a.out = static_cast<float*>(b->buf[st.out_buf]); a.out_stride = s->width[st.out_buf];
+            a.scratch = b->routed; a.counts = s->routed_counts; a.status = s->pf_status;
+            int n = 0;
+            rc = launch_routed(a, stream, &n);
+            s->launches += n;
+            break;
+        }
         case L_LATENT: {
             LatentLaunch a;
             const RopeTable& rope = plan->rope_tables[L.rope_table];
             a.row = plan->latent[st.layer].row;
             a.heads = st.heads; a.dim = st.head_dim; a.vdim = st.value_dim; a.rot_dims = st.rope_dim;
             a.scale = st.scale; a.eps = st.eps; a.weight_bias = st.weight_bias; a.magnitude = rope.magnitude; a.inv_freq = rope.inv_freq; a.f32 = f32;
+            a.window = st.window_left; a.sink = L.dv[0] ? L.dv[0]->data : nullptr;
             a.q = b->buf[st.in_buf]; a.q_stride = s->width[st.in_buf];
             a.kv = static_cast<const float*>(b->buf[st.in2_buf]); a.kv_stride = s->width[st.in2_buf];
             if (st.in3_buf != SWLM_BUF_NONE) { a.gate = static_cast<const float*>(b->buf[st.in3_buf]); a.gate_stride = s->width[st.in3_buf]; }
@@ -489,9 +618,10 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.pool = s->pool[st.layer]; a.page_table = s->page_table; a.pages_per_seq = s->pages_per_seq;
             a.row_seq = r.seq; a.row_pos = r.pos;
             a.out = b->buf[st.out_buf]; a.out_stride = s->width[st.out_buf];
-            a.n_short = r.n_short; a.short_rows = r.short_rows; a.splits = latent_pick_splits(r.n_short, st.heads, r.splits_pages);
+            a.n_short = r.n_short; a.short_rows = r.short_rows; a.splits = latent_pick_splits(r.n_short, st.heads, r.splits_pages, st.window_left);
             a.qcat = b->qcat; a.partial = b->partial;
-            a.n_long = r.n_long; a.long_rows = r.long_rows; a.n_spans = r.n_spans; a.spans = r.spans; a.n_tiles = r.n_tiles; a.tiles = r.tiles; a.total_ctx = r.total_ctx;
+            a.n_long = r.n_long; a.long_rows = r.long_rows; a.n_spans = r.n_spans; a.n_tiles = r.n_tiles; a.tiles = r.tiles;
+            if (r.n_spans) { a.spans = r.spans[L.window_set]; a.total_ctx = r.total_ctx[L.window_set]; }
             a.expand = b->expand; a.part = b->part; a.part_floats = b->part_cap; a.status = s->pf_status;
             a.only_attention = latent_kernel;
             int n = 0;
@@ -523,7 +653,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
 
 RowBatch identity_batch(const swlm_state* s) {
     RowBatch r;
-    r.rows = r.wants = r.n_short = s->plan->desc.max_batch;
+    r.rows = r.wants = r.n_short = r.n_single = s->plan->desc.max_batch;
     r.tok = s->token_in; r.seq = s->seq_identity; r.pos = s->position;
     r.splits_pages = s->pages_per_seq;
     r.advance = true;
@@ -534,7 +664,7 @@ RowBatch identity_batch(const swlm_state* s) {
 int decode_scratch(swlm_state* s) {
     for (int n = 1; n <= s->plan->desc.max_batch; ++n) {
         RowBatch r;
-        r.rows = r.wants = r.n_short = n;
+        r.rows = r.wants = r.n_short = r.n_single = n;
         r.splits_pages = s->pages_per_seq;
         const int rc = bufs_scratch(s, &s->dec, r);
         if (rc) return rc;
@@ -562,6 +692,20 @@ int stream_state_create(swlm_state* s) {
         // a page is read whole: rows nobody has written must hold finite numbers
         if (bytes) SWLM_CUDA(cudaMemset(p, 0, bytes));
     }
+    for (const DeltaLayer& l : plan->delta) {
+        float* st = nullptr;
+        unsigned char* ring = nullptr;
+        const size_t bytes = (size_t)d.max_batch * l.ring_elems() * elem;
+        if ((rc = dev_alloc(&st, (size_t)d.max_batch * l.state_elems()))) return rc;
+        s->delta_state.push_back(st);
+        if ((rc = dev_alloc(&ring, bytes))) return rc;
+        s->delta_ring.push_back(ring);
+        // (a sequence at position 0 starts from zeros whatever its slot holds; this is for positions that are set)
+        if (bytes) SWLM_CUDA(cudaMemset(ring, 0, bytes));
+        if (st) SWLM_CUDA(cudaMemset(st, 0, (size_t)d.max_batch * l.state_elems() * 4));
+    }
+    if ((rc = dev_alloc(&s->routed_counts, kMaxExperts))) return rc;
+    SWLM_CUDA(cudaMemset(s->routed_counts, 0, kMaxExperts * 4));
     s->seq_pages.assign(d.max_batch, {});
     s->page_table_host.assign((size_t)d.max_batch * s->pages_per_seq, 0);
     if ((rc = dev_alloc(&s->page_table, s->page_table_host.size()))) return rc;
@@ -590,6 +734,9 @@ void stream_drop_graphs(swlm_state* s) {
 void stream_state_free(swlm_state* s) {
     stream_drop_graphs(s);
     for (void* p : s->pool) cudaFree(p);
+    for (float* p : s->delta_state) cudaFree(p);
+    for (void* p : s->delta_ring) cudaFree(p);
+    cudaFree(s->routed_counts);
     cudaFree(s->page_table);
     cudaFree(s->seq_identity);
     bufs_free(&s->dec);
@@ -613,7 +760,9 @@ int stream_launches_per_step(const swlm_plan* plan) {
             else if (L.norm.kind) n += 1;
             if (L.m2 && !product_takes_gate(m, L.m1->k, a.x_f32)) { a.w2 = nullptr; n += 2 * product_launch_count(a) + 1; }
             else n += product_launch_count(a);
-        } else n += L.kind == L_LATENT ? 3 : L.kind == L_ARGMAX ? 2 : 1;
+        } else if (L.kind == L_DELTA) n += delta_step_fits(plan->delta[L.st.layer].shape) ? 1 : 3;
+        else if (L.kind == L_ROUTED) n += m <= 4 || plan->all_f32() ? 2 : 6;
+        else n += L.kind == L_LATENT ? 3 : L.kind == L_ARGMAX ? 2 : 1;
     }
     return n;
 }
@@ -651,7 +800,7 @@ int stage(swlm_state* s, StreamBufs* b, const std::vector<int32_t>& meta) {
 
 // spans of at least this many rows are attended over expanded keys and values
 constexpr int kSpanMinRows = 64;
-static_assert(sizeof(LatentSpan) == 20, "spans are staged as five words");
+static_assert(sizeof(LatentSpan) == 24 && sizeof(RowRun) == 20, "spans are staged as six words, runs as five");
 
 // Rows of `pieces` in one pass; `want_rows` get logits and tokens in b->buf[LOGITS] / b->argmax_out.
 int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<int32_t>& want_rows, StreamBufs** used, int only_kind = -1, int repeats = 1) {
@@ -678,7 +827,7 @@ int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<
     if (graph) {
         if ((rc = stage(s, b, meta))) return rc;
         r.tok = b->meta; r.seq = b->meta + rows; r.pos = b->meta + 2 * rows;
-        r.n_short = rows; r.splits_pages = s->pages_per_seq;
+        r.n_short = r.n_single = rows; r.splits_pages = s->pages_per_seq;
         auto it = s->row_graphs.find(rows);
         if (it == s->row_graphs.end()) {
             cudaGraph_t g = nullptr;
@@ -707,21 +856,26 @@ int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<
     bool expands = true;
     for (const Launch& L : plan->launches)
         if (L.kind == L_LATENT) expands &= latent_expands(plan->latent[L.st.layer].row, L.st.head_dim, L.st.value_dim, plan->all_f32());
-    std::vector<int32_t> shorts, longs;
+    std::vector<int32_t> shorts, longs, singles, block_run;
     std::vector<LatentSpan> spans;
+    std::vector<RowRun> runs;
     std::vector<std::pair<int, int2>> tiles;   // (context at the end of the tile, tile)
     int row0 = 0, short_longest = 0;
     for (const Piece& p : pieces) {
         if (expands && p.count >= kSpanMinRows) {
             const int sp = (int)spans.size();
-            spans.push_back(LatentSpan{row0, p.count, p.pos0, p.seq, r.total_ctx});
-            r.total_ctx += p.pos0 + p.count;
+            spans.push_back(LatentSpan{row0, p.count, p.pos0, p.seq, 0, 0});
             for (int i = 0; i < p.count; ++i) longs.push_back(row0 + i);
             for (int q = 0; q * kLatentQueryTile < p.count; ++q)
                 tiles.push_back({p.pos0 + std::min(p.count, (q + 1) * kLatentQueryTile), int2{sp, q}});
         } else {
             for (int i = 0; i < p.count; ++i) shorts.push_back(row0 + i);
             short_longest = std::max(short_longest, p.pos0 + p.count);
+        }
+        if (p.count == 1) singles.push_back(row0);
+        else {
+            runs.push_back(RowRun{row0, p.count, p.pos0, p.seq, (int)block_run.size()});
+            block_run.insert(block_run.end(), (p.count + kDeltaBlock - 1) / kDeltaBlock, (int)runs.size() - 1);
         }
         row0 += p.count;
     }
@@ -736,7 +890,25 @@ int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<
     const size_t o_tiles = meta.size();
     for (const auto& tl : tiles) { meta.push_back(tl.second.x); meta.push_back(tl.second.y); }
     const size_t o_spans = meta.size();
-    for (const LatentSpan& sp : spans) { const int32_t w[5] = {sp.row0, sp.count, sp.pos0, sp.seq, sp.ctx0}; meta.insert(meta.end(), w, w + 5); }
+    for (const int window : plan->windows) {
+        int ctx = 0;
+        for (const LatentSpan& sp : spans) {
+            const int lo = window > 0 ? std::max(0, sp.pos0 - window + 1) / SWLM_PAGE_TOKENS * SWLM_PAGE_TOKENS : 0;
+            const int32_t w[6] = {sp.row0, sp.count, sp.pos0, sp.seq, ctx, lo};
+            meta.insert(meta.end(), w, w + 6);
+            ctx += sp.pos0 + sp.count - lo;
+        }
+        r.total_ctx.push_back(ctx);
+    }
+    const size_t o_single = meta.size();
+    meta.insert(meta.end(), singles.begin(), singles.end());
+    const size_t o_runs = meta.size();
+    for (const RowRun& run : runs) { const int32_t w[5] = {run.row0, run.count, run.pos0, run.seq, run.blk0}; meta.insert(meta.end(), w, w + 5); }
+    const size_t o_blocks = meta.size();
+    meta.insert(meta.end(), block_run.begin(), block_run.end());
+    r.n_single = (int)singles.size();
+    r.n_runs = (int)runs.size();
+    r.n_blocks = (int)block_run.size();
     r.n_short = (int)shorts.size();
     r.n_long = (int)longs.size();
     r.n_spans = (int)spans.size();
@@ -747,7 +919,10 @@ int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<
     r.wants_idx = b->meta + o_want;
     r.short_rows = b->meta + o_short; r.long_rows = b->meta + o_long;
     r.tiles = reinterpret_cast<const int2*>(b->meta + o_tiles);
-    r.spans = reinterpret_cast<const LatentSpan*>(b->meta + o_spans);
+    for (size_t q = 0; q < plan->windows.size(); ++q) r.spans.push_back(reinterpret_cast<const LatentSpan*>(b->meta + o_spans + q * 6 * spans.size()));
+    r.single_rows = b->meta + o_single;
+    r.runs = reinterpret_cast<const RowRun*>(b->meta + o_runs);
+    r.block_run = b->meta + o_blocks;
     for (int i = 0; i < repeats && !rc; ++i) rc = enqueue_rows_stream(s, b, r, false, s->stream, only_kind);
     return rc;
 }
@@ -846,6 +1021,8 @@ int stream_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_i
         if (tmp.stream_width[i] > s->width[i]) { set_error("step: buffer %d is %d wide, the step needs %d", i, s->width[i], tmp.stream_width[i]); return done(SWLM_ERR_INVALID); }
     for (size_t l = 0; l < tmp.latent.size(); ++l)
         if (tmp.latent[l].rank && tmp.latent[l].row.pitch != s->plan->latent[l].row.pitch) { set_error("step: latent layer %zu has other rows", l); return done(SWLM_ERR_INVALID); }
+    for (size_t l = 0; l < tmp.delta.size(); ++l)
+        if (tmp.delta[l].shape.heads && memcmp(&tmp.delta[l].shape, &s->plan->delta[l].shape, sizeof(DeltaShape))) { set_error("step: gated-delta layer %zu has another shape", l); return done(SWLM_ERR_INVALID); }
     for (int b = 0; b < m; ++b)
         if ((rc = stream_reserve(s, b, s->pos_host[b] + 1))) return done(rc);
     if ((rc = stream_upload_pages(s))) return done(rc);

@@ -1,4 +1,4 @@
-// Row kernels of fp32-stream plans: embedding gather, sandwich norm, gated activation, argmax over fp32 logits. The residual
+// Row kernels of fp32-stream plans: embedding gather, norms, gated activation, soft cap of the logits. The residual
 // stream, the norms and the logits stay in fp32; results that feed a product are stored in the plan's activation type.
 #include "swlm_internal.h"
 
@@ -60,13 +60,22 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(int dim, const int32_
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) stream_gated_kernel(int n, const T* gate, int g_stride, const T* up, int u_stride, T* out, int o_stride, int act) {
+__global__ void __launch_bounds__(256) stream_gated_kernel(int n, const T* gate, int g_stride, const T* up, int u_stride, T* out, int o_stride, GatedAct act) {
     pdl_launch_dependents();
     pdl_wait();
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const size_t r = blockIdx.y;
     put(out + r * o_stride + i, gated_activation(get(gate + r * g_stride + i), get(up + r * u_stride + i), act));
+}
+
+__global__ void __launch_bounds__(256) stream_softcap_kernel(int n, float* x, int stride, float cap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    float* v = x + (size_t)blockIdx.y * stride + i;
+    *v = cap * tanhf(*v / cap);
 }
 
 }  // namespace
@@ -90,13 +99,19 @@ int launch_stream_embed(int m, int dim, const int32_t* tokens, int vocab, const 
     return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "stream embed launch");
 }
 
-int launch_stream_gated(int m, int n, const void* gate, int g_stride, const void* up, int u_stride, void* out, int o_stride, bool f32, int act, cudaStream_t s) {
+int launch_stream_gated(int m, int n, const void* gate, int g_stride, const void* up, int u_stride, void* out, int o_stride, bool f32, GatedAct act, cudaStream_t s) {
     cudaError_t e;
     const dim3 grid((n + 255) / 256, m);
     if (f32) e = launch_k(stream_gated_kernel<float>, grid, dim3(256), 0, s, n, static_cast<const float*>(gate), g_stride, static_cast<const float*>(up), u_stride, static_cast<float*>(out), o_stride, act);
     else e = launch_k(stream_gated_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, n, static_cast<const __nv_bfloat16*>(gate), g_stride,
                       static_cast<const __nv_bfloat16*>(up), u_stride, static_cast<__nv_bfloat16*>(out), o_stride, act);
     return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "gated activation launch");
+}
+
+int launch_stream_softcap(int m, int n, float* logits, int stride, float cap, cudaStream_t s) {
+    if (m <= 0) return SWLM_OK;
+    const cudaError_t e = launch_k(stream_softcap_kernel, dim3((n + 255) / 256, m), dim3(256), 0, s, n, logits, stride, cap);
+    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "soft cap launch");
 }
 
 }  // namespace swlm

@@ -106,7 +106,9 @@ int launch_repack(const RepackSrc* src, int n_src, int mode, int k, const Q4Tile
 int launch_untile_bf16(const Q4Tiled& t, __nv_bfloat16* out, cudaStream_t s);
 
 enum { QGEMV_EPI_STORE = 0, QGEMV_EPI_SWIGLU = 1 };   // SWIGLU: the gated-activation epilogue (SiLU or GELU, see gated_act)
-enum { GATED_ACT_SILU = 0, GATED_ACT_GELU_TANH = 1 };
+enum { GATED_ACT_SILU = 0, GATED_ACT_GELU_TANH = 1, GATED_ACT_CLAMPED = 2 };
+// Activation of a gated feed-forward. CLAMPED: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1).
+struct GatedAct { int kind = GATED_ACT_SILU; float alpha = 0.f, limit = 0.f; };
 #ifdef __CUDACC__
 // activation(gate) * up of the gated MLP (Generator/MetalSourceGenerator+NormAndElementwise.swift:176-208):
 // SiLU for SwiGLU, the tanh approximation of GELU for GEGLU.
@@ -114,6 +116,12 @@ __device__ __forceinline__ float gated_activation(float g, float up, int act) {
     const float a = act == GATED_ACT_GELU_TANH ? 0.5f * g * (1.0f + tanhf(0.7978845608f * (g + 0.044715f * g * g * g)))
                                                : g * (1.0f / (1.0f + expf(-g)));
     return a * up;
+}
+__device__ __forceinline__ float gated_activation(float g, float up, const GatedAct& act) {
+    if (act.kind != GATED_ACT_CLAMPED) return gated_activation(g, up, act.kind);
+    g = fminf(g, act.limit);
+    up = fminf(fmaxf(up, -act.limit), act.limit);
+    return g * (1.0f / (1.0f + expf(-act.alpha * g))) * (up + 1.0f);
 }
 #endif
 
@@ -336,15 +344,16 @@ struct Matrix {
     __nv_bfloat16* data = nullptr;
     bool view = false;   // rows of a concatenated matrix that owns the memory
 };
-constexpr int kMaxProductSegs = 4;
+constexpr int kMaxProductSegs = 8;
 
 // Where a product's rows go: rows [end[q-1], end[q]) to y[q], an fp32 or bf16 buffer [m][stride[q]].
 struct ProductOut {
     int count = 1;
-    int end[kMaxProductSegs] = {0, 0, 0, 0};
-    void* y[kMaxProductSegs] = {nullptr, nullptr, nullptr, nullptr};
-    int stride[kMaxProductSegs] = {0, 0, 0, 0};
-    int f32[kMaxProductSegs] = {0, 0, 0, 0};
+    int end[kMaxProductSegs] = {};
+    void* y[kMaxProductSegs] = {};
+    int stride[kMaxProductSegs] = {};
+    int f32[kMaxProductSegs] = {};
+    float softcap = 0.f;   // > 0: every value v becomes softcap * tanh(v / softcap)
 };
 
 // A norm step over the fp32 stream. mode = its step kind (0: none).
@@ -364,7 +373,9 @@ struct StreamNorm {
 int launch_stream_norm(const StreamNorm& a, int m, int dim, const int32_t* rows_idx, void* out, int out_stride, bool out_f32, cudaStream_t s);
 // out[r] = table[tok[r]] * scale, fp32
 int launch_stream_embed(int m, int dim, const int32_t* tokens, int vocab, const __nv_bfloat16* table, float scale, float* out, int out_stride, cudaStream_t s);
-int launch_stream_gated(int m, int n, const void* gate, int g_stride, const void* up, int u_stride, void* out, int o_stride, bool f32, int act, cudaStream_t s);
+int launch_stream_gated(int m, int n, const void* gate, int g_stride, const void* up, int u_stride, void* out, int o_stride, bool f32, GatedAct act, cudaStream_t s);
+// logits = cap * tanh(logits / cap), in place
+int launch_stream_softcap(int m, int n, float* logits, int stride, float cap, cudaStream_t s);
 // argmax over fp32 rows, any m (blocks of kMaxSequences rows); the advancing form of launch_argmax for m <= kMaxSequences
 int launch_argmax_f32(int m, int n, const float* logits, int stride, int32_t* token_out, int32_t* token_in_next, int32_t* ring,
                       int32_t* step_counter, int ring_cap, int32_t* position, int advance, float* scratch_val, int32_t* scratch_idx, cudaStream_t s);
@@ -372,16 +383,23 @@ int launch_argmax_f32(int m, int n, const float* logits, int stride, int32_t* to
 struct ProductLaunch {
     const Matrix* w = nullptr;
     const Matrix* w2 = nullptr;     // gated form: out = act(w x) * (w2 x), rows of both side by side
-    int act = GATED_ACT_SILU;
+    GatedAct act;
     int m = 0;
     const void* x = nullptr; int x_stride = 0; bool x_f32 = false;   // x_f32: activations fp32, true fp32 products
     StreamNorm norm;                // x = this norm's result (only when product_takes_norm)
     ProductOut out;
     float* part = nullptr; size_t part_floats = 0;   // split-K sums
     int* status = nullptr;          // device word set when a bounded wait expired
+    // Grouped form (bf16, tensor cores): w holds the rows of `experts` matrices one after the other, activation rows are sorted
+    // by expert, and tiles[i] = (expert, first row, rows, 0) names the rows of tile i (at most group_bn; 0 rows: nothing to do).
+    int experts = 0;
+    const int4* tiles = nullptr; int max_tiles = 0, group_bn = 0;
 };
 int bgemm_init();
 int launch_product(const ProductLaunch& a, cudaStream_t s);
+// rows per tile of a grouped product over `rows` activation rows, and the most tiles they can make
+int grouped_bn(int rows, int experts);
+int grouped_max_tiles(int rows, int experts);
 bool product_takes_norm(int m, int k);
 bool product_takes_gate(int m, int k, bool x_f32);
 int product_launch_count(const ProductLaunch& a);
@@ -394,12 +412,15 @@ struct LatentRow { int rank = 0, rot = 0, rp = 0, rotp = 0, pitch = 0; };
 LatentRow latent_row(int rank, int rot, bool f32);
 // Consecutive rows of one sequence inside a batch: rows row0 .. row0 + count - 1 at positions pos0 ..; ctx0 = first of the
 // pos0 + count gathered rows of this span.
-struct LatentSpan { int row0, count, pos0, seq, ctx0; };
+// With a sliding window the rows in front of `lo` (a multiple of the page size) are not gathered.
+struct LatentSpan { int row0, count, pos0, seq, ctx0, lo; };
 
 struct LatentLaunch {
     LatentRow row;
     int heads = 0, dim = 0, vdim = 0, rot_dims = 0;
     float scale = 1.f, eps = 0.f, weight_bias = 0.f, magnitude = 1.f;
+    int window = 0;                                        // > 0: a row sees its own and the window - 1 positions before it
+    const __nv_bfloat16* sink = nullptr;                   // [heads]: exp(sink) joins the denominator; null: none
     const float* inv_freq = nullptr;
     bool f32 = false;
     void* q = nullptr; int q_stride = 0;                   // [rows][heads * (dim + rot)]; rotated in place for span rows
@@ -424,7 +445,7 @@ struct LatentLaunch {
     bool only_attention = false;   // timing hook: the attention kernel alone
 };
 int latent_init();
-int latent_pick_splits(int rows, int heads, int max_pages);
+int latent_pick_splits(int rows, int heads, int max_pages, int window);
 size_t latent_qcat_floats(const LatentRow& r, int heads);              // per row
 size_t latent_partial_floats(const LatentRow& r, int heads);           // per row and split
 size_t latent_expand_bytes(const LatentRow& r, int heads, int dim, int vdim, int total_ctx);
@@ -433,5 +454,59 @@ bool latent_expands(const LatentRow& r, int dim, int vdim, bool f32);
 constexpr int kLatentQueryTile = 128;
 // launches (for the counters): short part 3, span part 4 or 5
 int launch_latent(const LatentLaunch& a, cudaStream_t s, int* launches);
+
+// ---- gated delta rule (delta_rule.cu) ----------------------------------------------------------------------------------
+// Consecutive rows of one sequence: rows row0 .. row0 + count - 1 of the batch at positions pos0 ..; walked in blocks of
+// kDeltaBlock tokens, blk0 = number of blocks of the runs before it.
+struct RowRun { int row0, count, pos0, seq, blk0; };
+constexpr int kDeltaBlock = 4;
+struct DeltaShape { int heads = 0, groups = 0, dim = 0, vdim = 0, taps = 0; __host__ __device__ int channels() const { return 2 * groups * dim + heads * vdim; } };
+struct DeltaLaunch {
+    DeltaShape shape;
+    int decay_dim = 1;                                     // decay inputs per head: 1 or dim
+    int gate_act = 0;                                      // SWLM_GATE_*
+    float eps = 0.f, unit_eps = 0.f, q_scale = 1.f;
+    bool f32 = false;
+    const void* qkv = nullptr; int qkv_stride = 0;
+    const float* beta = nullptr; int beta_stride = 0;
+    const float* decay = nullptr; int decay_stride = 0;
+    const void* gate = nullptr; int gate_stride = 0;
+    const __nv_bfloat16 *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr, *norm_w = nullptr, *a_log = nullptr, *dt_bias = nullptr;
+    void* ring = nullptr;                                  // [sequence][taps][channels]: inputs of the convolutions, slot = position % taps
+    float* state = nullptr;                                // [sequence][heads][dim][vdim]
+    const int32_t* row_seq = nullptr; const int32_t* row_pos = nullptr;
+    void* out = nullptr; int out_stride = 0;
+    int n_single = 0; const int32_t* single_rows = nullptr;   // rows that are one token of their sequence (null: rows 0 ..)
+    int n_runs = 0; const RowRun* runs = nullptr;             // longer portions
+    int n_blocks = 0; const int32_t* block_run = nullptr;     // the run of every block
+    float* scratch = nullptr;
+    int* status = nullptr;
+};
+int delta_init();
+bool delta_supported(const DeltaShape& s);
+bool delta_step_fits(const DeltaShape& s);                    // single tokens in one fused launch
+size_t delta_scratch_floats(const DeltaShape& s, int blocks, int rows);
+int launch_delta(const DeltaLaunch& a, cudaStream_t s, int* launches);
+
+// ---- routed feed-forward (routed_mlp.cu) -------------------------------------------------------------------------------
+struct RoutedShape { int experts = 0, top = 0, groups = 1, keep = 1, width = 0, ff = 0; };
+struct RoutedLaunch {
+    RoutedShape shape;
+    float scale = 1.f;
+    GatedAct act;
+    int m = 0; bool f32 = false;
+    const void* x = nullptr; int x_stride = 0;
+    const float* z = nullptr; int z_stride = 0;
+    const Matrix *gate = nullptr, *up = nullptr, *down = nullptr;   // the experts' rows one after the other
+    float* out = nullptr; int out_stride = 0;
+    unsigned char* scratch = nullptr;
+    unsigned* counts = nullptr;                            // [kMaxExperts], zero between launches
+    int* status = nullptr;
+};
+constexpr int kMaxExperts = 1024, kMaxTop = 64;
+int routed_init();
+bool routed_supported(const RoutedShape& s);
+size_t routed_scratch_bytes(const RoutedShape& s, int m, bool f32);
+int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches);
 
 }  // namespace swlm

@@ -22,7 +22,7 @@ inline int dev_alloc(T** p, size_t count, int64_t* total = nullptr) {
 
 
 enum LaunchKind { L_EMBED, L_RMSNORM, L_QGEMV, L_QK_NORM, L_ATTN, L_SWIGLU, L_CONV, L_ARGMAX, L_SSM,
-                  L_PRODUCT, L_LATENT };   // the last two: fp32-stream plans only
+                  L_PRODUCT, L_LATENT, L_DELTA, L_ROUTED, L_SOFTCAP };   // from L_PRODUCT on: fp32-stream plans only
 
 struct Launch {
     int kind = 0;
@@ -33,8 +33,9 @@ struct Launch {
     int epilogue = QGEMV_EPI_STORE;
     int gated_act = GATED_ACT_SILU;
     int n_seg = 1;
-    int seg_buf[kMaxProductSegs] = {-1, -1, -1, -1};
-    int seg_end[kMaxProductSegs] = {0, 0, 0, 0};
+    int seg_buf[kMaxProductSegs] = {-1, -1, -1, -1, -1, -1, -1, -1};
+    int seg_off[kMaxProductSegs] = {};     // first column in the buffer (fp32-stream plans)
+    int seg_end[kMaxProductSegs] = {};
     const DenseTensor* d1 = nullptr;
     const DenseTensor* d2 = nullptr;
     const Q4Raw* q_embed = nullptr;  // embedding step over a quantized table
@@ -53,6 +54,11 @@ struct Launch {
     // products of fp32-stream plans: one matrix (possibly the rows of several tensors), or gate and up
     const Matrix* m1 = nullptr;
     const Matrix* m2 = nullptr;
+    const Matrix* m3 = nullptr;               // routed feed-forward: the experts' down rows (m1, m2: gate, up)
+    GatedAct act;
+    float softcap = 0.f;                      // of the output head's logits
+    const DenseTensor* dv[6] = {};            // gated delta rule: taps of q, k, v, norm weight, A_log, dt_bias; latent attention: [0] sink
+    int window_set = 0;                       // latent attention: index into plan->windows
     const DenseTensor* norm_post = nullptr;   // norm steps: weight of the norm applied to the input before it is added
     int kv_prefetch_attn = -1;    // index of the attention launch whose K/V rows this product pulls into L2
 };
@@ -67,6 +73,13 @@ struct RopeTable {
 // One latent-attention layer's share of the page pool.
 struct LatentLayer { int rank = 0, rot = 0; LatentRow row{}; };
 
+// One gated-delta layer: per sequence an fp32 state and the last inputs of the convolutions.
+struct DeltaLayer {
+    DeltaShape shape;
+    size_t state_elems() const { return (size_t)shape.heads * shape.dim * shape.vdim; }
+    size_t ring_elems() const { return (size_t)shape.taps * shape.channels(); }
+};
+
 // Activation buffers and scratch of the row executor of fp32-stream plans. A state holds two sets: one sized for a decode
 // step (its pointers are captured in CUDA graphs and never change), one that grows with the largest batch of rows seen.
 struct StreamBufs {
@@ -79,6 +92,8 @@ struct StreamBufs {
     float* partial = nullptr; size_t partial_cap = 0;    // latent attention: partial results per split
     float* part = nullptr; size_t part_cap = 0;          // products: sums of K ranges
     unsigned char* expand = nullptr; size_t expand_cap = 0;
+    float* delta = nullptr; size_t delta_cap = 0;        // gated delta rule: records and read-outs of portions
+    unsigned char* routed = nullptr; size_t routed_cap = 0;
     float* argmax_val = nullptr; int32_t* argmax_idx = nullptr;
 };
 
@@ -89,7 +104,10 @@ struct RowBatch {
     int wants = 0; const int32_t* wants_idx = nullptr;              // rows that get logits; null: rows 0 .. wants - 1
     int n_short = 0; const int32_t* short_rows = nullptr; int splits_pages = 1;   // latent attention one by one; longest context in pages
     int n_long = 0; const int32_t* long_rows = nullptr;             // and in spans
-    int n_spans = 0; const LatentSpan* spans = nullptr; int n_tiles = 0; const int2* tiles = nullptr; int total_ctx = 0;
+    int n_spans = 0; int n_tiles = 0; const int2* tiles = nullptr;
+    std::vector<const LatentSpan*> spans; std::vector<int> total_ctx;   // per window of the plan: what is gathered depends on it
+    int n_single = 0; const int32_t* single_rows = nullptr;         // gated delta rule: single tokens (null: rows 0 .. n_single - 1)
+    int n_runs = 0; const RowRun* runs = nullptr; int n_blocks = 0; const int32_t* block_run = nullptr;   // and longer portions
     bool advance = false;                                           // decode step over all sequences: feed tokens back, advance positions
 };
 
@@ -137,6 +155,8 @@ struct swlm_plan {
     bool rows_groups_ready = false;
     // fp32-stream plans (desc.stream_dtype != 0)
     std::vector<LatentLayer> latent;      // by step.layer
+    std::vector<DeltaLayer> delta;        // by step.layer
+    std::vector<int> windows;             // distinct sliding windows of the latent layers
     int stream_width[SWLM_BUF_COUNT] = {};
     int latent_heads_max = 0, latent_q_floats = 0, latent_part_floats = 0;   // largest over the layers, per row / per row and split
     bool stream() const { return desc.stream_dtype != 0; }
@@ -192,6 +212,8 @@ struct swlm_state {
     // fp32-stream plans: paged pool of latent rows (one page list per sequence, the same page numbers in every layer's
     // pool), the page table on host and device, and the two activation sets
     std::vector<void*> pool; std::vector<size_t> pool_bytes;
+    std::vector<float*> delta_state; std::vector<void*> delta_ring;   // per gated-delta layer: [max_batch][state_elems], [max_batch][ring_elems]
+    unsigned* routed_counts = nullptr;                                // rows per expert, zero between launches
     int pool_pages = 0, pages_per_seq = 0;
     std::vector<int> free_pages;
     std::vector<std::vector<int>> seq_pages;

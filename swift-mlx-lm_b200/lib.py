@@ -53,6 +53,17 @@ class Step(C.Structure):
         ("rope_original", C.c_float),
         ("rope_fast", C.c_float),
         ("rope_slow", C.c_float),
+        ("in_off", C.c_int32),
+        ("out_off", C.c_int32),
+        ("experts", C.c_int32),
+        ("top", C.c_int32),
+        ("groups_keep", C.c_int32),
+        ("gate_act", C.c_int32),
+        ("limit", C.c_float),
+        ("glu_alpha", C.c_float),
+        ("eps2", C.c_float),
+        ("weight5", C.c_char * NAME_MAX),
+        ("weight6", C.c_char * NAME_MAX),
     ]
 
 
@@ -82,6 +93,7 @@ class BuffersDesc(C.Structure):
         ("stream_dtype", C.c_int32),
         ("latent_layers", C.c_int32),
         ("kv_pool_tokens", C.c_int32),
+        ("delta_layers", C.c_int32),
     ]
 
 

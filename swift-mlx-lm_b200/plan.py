@@ -36,6 +36,11 @@ STEP_PRODUCT = 13
 STEP_POSTNORM_RESADD_COPY_RMSNORM = 14
 STEP_POSTNORM_RESADD_RMSNORM = 15
 STEP_LATENT_ATTN = 16
+STEP_CLAMPED_GLU = 17
+STEP_GATED_DELTA = 18
+STEP_ROUTED_MLP = 19
+STEP_SOFTCAP = 20
+GATE_SILU, GATE_SIGMOID = 0, 1
 
 STREAM_BF16, STREAM_F32, STREAM_ALL_F32 = 0, 1, 2
 PAGE_TOKENS = 64
@@ -171,7 +176,7 @@ def _step(kind: int, **kw) -> Step:
     s.layer = -1
     s.in_buf = s.in2_buf = s.in3_buf = s.in4_buf = s.out_buf = -1
     for key, value in kw.items():
-        if key in ("weight", "weight2", "weight3", "weight4"):
+        if key.startswith("weight") and isinstance(value, str):
             value = value.encode()
         setattr(s, key, value)
     return s
