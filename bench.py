@@ -306,6 +306,7 @@ def run_op(args, pkg):
 
 VUZUNEX_SHAPES = {   # width, heads, feed-forward, layers: per-layer sizes of real models, fewer layers and a 32768-token vocabulary
     "1b": (2048, 16, 8192, 16), "8b": (4096, 32, 14336, 8)}
+BENCH_VOCAB = 32768
 
 
 def block_weights(builder, seed=3):
@@ -331,24 +332,9 @@ def block_weights(builder, seed=3):
     return out
 
 
-def run_vuzunex(args, pkg):
-    """Prompt and decode throughput of the Vuzunex design (dense bf16 weights, latent attention, fp32 stream) beside the Llama
-    recipe (4-bit weights, grouped-query attention) at equal width, heads, feed-forward, layers and vocabulary. One JSON line."""
+def stream_timer(stream):
+    """timed(fn, reps): milliseconds of one call on the device."""
     import torch
-
-    torch.cuda.set_device(0)
-    stream = torch.cuda.Stream()
-    torch.cuda.set_stream(stream)
-    width, heads, ff, layers = VUZUNEX_SHAPES[args.shape]
-    vocab, batch, ctx, P = 32768, args.batch, args.ctx, pkg.plan
-    dim, rot, vdim, rank = 128, 64, 128, 512
-    warm = max(3, args.warmup)
-    max_seq = ctx + 4 * (warm + args.steps) + 64
-    mixer = pkg.vuzunex.LatentAttention(heads, dim, rot, vdim, rank, (dim + rot) ** -0.5, 10000.0, rot, pkg.vuzunex.RotaryScaling(40.0, 4096.0, 32.0, 1.0))
-    vcfg = pkg.VuzunexConfig(vocab=vocab, width=width, layers=[pkg.vuzunex.Layer(mixer, ff, i) for i in range(layers)], max_seq=max_seq, max_batch=batch)
-    lcfg = pkg.ModelConfig("llama", width, ff, layers, heads, heads // 4, 128, vocab, max_seq=max_seq, max_batch=batch)
-    hbm, hbm_src = measured_peaks()
-    tensor, _ = measured_tensor_peak()
 
     def timed(fn, reps):
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
@@ -360,78 +346,235 @@ def run_vuzunex(args, pkg):
         torch.cuda.synchronize()
         return e0.elapsed_time(e1) / reps
 
-    def measure(builder, latent):
-        store = pkg.WeightStore(0)
-        model = pkg.load_model(store, builder, block_weights(builder))
-        model.set_stream(stream.cuda_stream)
-        prompt = np.random.default_rng(7).integers(0, vocab, size=(batch, ctx), dtype=np.int32)
-        seconds = []
-        for _ in range(4):
-            model.reset_state()
-            torch.cuda.synchronize()
-            t0 = time.perf_counter()
-            tok = model.prefill(prompt)
-            seconds.append(time.perf_counter() - t0)
-        sampler = ClockSampler(0)
-        sampler.start()
-        sampler.wait_first(3.0)
-        model.decode_n_async(tok, warm)
-        before = model.launches
-        step_ms = timed(lambda: model.decode_n_async(None, args.steps), 1) / args.steps
-        launches = model.launches - before
-        tok = model.read_tokens(args.steps)[-1]
+    return timed
+
+
+def serve_rates(model, prompt, args, timed):
+    """Prompt and decode throughput of a model through its public calls: prompt tokens from the host, decoding on the device and
+    token by token from the host."""
+    import torch
+
+    batch, ctx = prompt.shape
+    warm = max(3, args.warmup)
+    seconds = []
+    for _ in range(4):
+        model.reset_state()
         torch.cuda.synchronize()
         t0 = time.perf_counter()
-        for _ in range(args.steps):
-            tok = model.decode(tok)
-        e2e = batch * args.steps / (time.perf_counter() - t0)
-        clocks = sampler.stop()
-        out = {"prefill_tok_s": batch * ctx / min(seconds[1:]), "decode_tok_s": batch * 1e3 / step_ms, "ms_per_step": step_ms, "e2e_tok_s": e2e,
-               "launches_per_step": model.launches_per_step, "clocks": clocks, "gpu_launches": int(launches)}
-        pos = model.position
-        if batch <= 16 or latent:
-            kind = P.STEP_PRODUCT if latent else P.STEP_QGEMV
-            model.profile_kind(kind, 2)
-            ms = timed(lambda: model.profile_kind(kind, 1), 10)
-            weight_bytes = (vcfg.weight_elems() - layers * heads * (dim + vdim) * rank) * 2 if latent else lcfg.q4_weight_elems() * 0.5625
-            out["decode_products"] = {"ms": ms, "bytes": weight_bytes, "GBs": weight_bytes / ms / 1e6, "frac": weight_bytes / ms / 1e6 / hbm}
-            model.profile_kind(P.STEP_ATTN_DECODE, 2)
-            ms = timed(lambda: model.profile_kind(P.STEP_ATTN_DECODE, 1), 10)
-            kv = layers * batch * pos * (2 * (rank + rot) if latent else lcfg.kv_heads * 128 * 4)
-            out["decode_attention"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv, "GBs": kv / ms / 1e6, "frac": kv / ms / 1e6 / hbm}
-        if latent:
-            ms = timed(lambda: model.profile_kind(P.STEP_LATENT_ATTN, 1), 10)
-            small = layers * heads * (dim + vdim) * rank * 2
-            out["decode_latent_step"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv + small, "frac": (kv + small) / ms / 1e6 / hbm}
-            # one prompt chunk from position 0: products, and the attention kernel alone
-            n = min(ctx, 2048)
-            model.reset_state()
-            chunk = prompt[0, :n]
-            model.profile_batch(0, chunk, P.STEP_PRODUCT, 2)
-            ms = timed(lambda: model.profile_batch(0, chunk, P.STEP_PRODUCT, 5), 1) / 5
-            flops = 2.0 * n * (weight_bytes / 2 - vocab * width)
-            out["prefill_products"] = {"rows": n, "ms": ms, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
-            model.profile_batch(0, chunk, P.STEP_ATTN_DECODE, 2)
-            ms = timed(lambda: model.profile_batch(0, chunk, P.STEP_ATTN_DECODE, 5), 1) / 5
-            flops = layers * heads * n * (n + 1) / 2 * 2.0 * (dim + rot + vdim)
-            out["prefill_attention"] = {"rows": n, "us_per_layer": ms * 1e3 / layers, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
-            ms = timed(lambda: model.profile_batch(0, chunk, P.STEP_LATENT_ATTN, 5), 1) / 5
-            out["prefill_latent_step_us_per_layer"] = ms * 1e3 / layers
-        model.close()
-        store.close()
-        return out
+        tok = model.prefill(prompt)
+        seconds.append(time.perf_counter() - t0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.wait_first(3.0)
+    model.decode_n_async(tok, warm)
+    before = model.launches
+    step_ms = timed(lambda: model.decode_n_async(None, args.steps), 1) / args.steps
+    launches = model.launches - before
+    tok = model.read_tokens(args.steps)[-1]
+    torch.cuda.synchronize()
+    t0 = time.perf_counter()
+    for _ in range(args.steps):
+        tok = model.decode(tok)
+    e2e = batch * args.steps / (time.perf_counter() - t0)
+    clocks = sampler.stop()
+    return {"prefill_tok_s": batch * ctx / min(seconds[1:]), "decode_tok_s": batch * 1e3 / step_ms, "ms_per_step": step_ms, "e2e_tok_s": e2e,
+            "launches_per_step": model.launches_per_step, "clocks": clocks, "gpu_launches": int(launches)}
 
-    ours = measure(pkg.VuzunexPlanBuilder(vcfg), True)
-    closest = measure(pkg.DispatchPlanBuilder(lcfg), False)
-    print(json.dumps({
-        "metric": f"decode tok/s, Vuzunex {args.shape} layers bs{batch}", "value": ours["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
-        "warmup": warm, "ms_per_step": ours["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
-        "dtype": "bf16 weights and activations, fp32 stream and accumulation", "data": "synthetic (random-init weights of the named shape)",
-        "config": {"workload": f"{layers} layers, width {width}, {heads} heads (128 + 64 / 128, latent 512), feed-forward {ff}, vocabulary {vocab}, context {ctx}, batch {batch}",
-                   "l2": "weights larger than L2 are streamed per step", "peak_source": hbm_src},
-        "clocks": ours["clocks"], "gpu_launches": ours["gpu_launches"],
-        "e2e": {"value": ours["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 * batch, "d2h_bytes_per_step": 4 * batch},
-        "vuzunex": ours, "llama_q4_equal_size": closest}))
+
+def measure_vuzunex(pkg, vcfg, args, stream, timed):
+    """Rates and kernels of a Vuzunex model whose layers are alike."""
+    P, batch, ctx, layers, width = pkg.plan, args.batch, args.ctx, len(vcfg.layers), vcfg.width
+    m = vcfg.layers[0].mixer
+    hbm, _ = measured_peaks()
+    tensor, _ = measured_tensor_peak()
+    builder = pkg.VuzunexPlanBuilder(vcfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, block_weights(builder))
+    model.set_stream(stream.cuda_stream)
+    prompt = np.random.default_rng(7).integers(0, vcfg.vocab, size=(batch, ctx), dtype=np.int32)
+    out = serve_rates(model, prompt, args, timed)
+    pos = model.position
+
+    def kind_ms(kind):
+        model.profile_kind(kind, 2)
+        return timed(lambda: model.profile_kind(kind, 1), 10)
+
+    small = layers * m.heads * (m.dim + m.vdim) * m.kv_rank * 2
+    ms, weight_bytes = kind_ms(P.STEP_PRODUCT), vcfg.weight_elems() * 2 - small
+    out["decode_products"] = {"ms": ms, "bytes": weight_bytes, "GBs": weight_bytes / ms / 1e6, "frac": weight_bytes / ms / 1e6 / hbm}
+    ms, kv = kind_ms(P.STEP_ATTN_DECODE), layers * batch * pos * 2 * (m.kv_rank + m.rot_dim)
+    out["decode_attention"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv, "GBs": kv / ms / 1e6, "frac": kv / ms / 1e6 / hbm}
+    ms = kind_ms(P.STEP_LATENT_ATTN)
+    out["decode_latent_step"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv + small, "frac": (kv + small) / ms / 1e6 / hbm}
+    # one prompt chunk from position 0: products, and the attention kernel alone
+    n = min(ctx, 2048)
+    model.reset_state()
+    chunk = prompt[0, :n]
+
+    def chunk_ms(kind):
+        model.profile_batch(0, chunk, kind, 2)
+        return timed(lambda: model.profile_batch(0, chunk, kind, 5), 1) / 5
+
+    ms, flops = chunk_ms(P.STEP_PRODUCT), 2.0 * n * (weight_bytes / 2 - vcfg.vocab * width)
+    out["prefill_products"] = {"rows": n, "ms": ms, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
+    ms, flops = chunk_ms(P.STEP_ATTN_DECODE), layers * m.heads * n * (n + 1) / 2 * 2.0 * (m.dim + m.rot_dim + m.vdim)
+    out["prefill_attention"] = {"rows": n, "us_per_layer": ms * 1e3 / layers, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
+    out["prefill_latent_step_us_per_layer"] = chunk_ms(P.STEP_LATENT_ATTN) * 1e3 / layers
+    model.close()
+    store.close()
+    return out
+
+
+def vuzunex_config(pkg, args, layers, max_seq):
+    width, heads, ff, _ = VUZUNEX_SHAPES[args.shape]
+    mixer = pkg.vuzunex.LatentAttention(heads, 128, 64, 128, 512, 192 ** -0.5, 10000.0, 64, pkg.vuzunex.RotaryScaling(40.0, 4096.0, 32.0, 1.0))
+    return pkg.VuzunexConfig(vocab=BENCH_VOCAB, width=width, layers=[pkg.vuzunex.Layer(mixer, ff, i) for i in range(layers)], max_seq=max_seq, max_batch=args.batch)
+
+
+def design_line(args, name, ours, workload):
+    hbm_src = measured_peaks()[1]
+    return {"metric": f"decode tok/s, {name} {args.shape} layers bs{args.batch}", "value": ours["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+            "warmup": max(3, args.warmup), "ms_per_step": ours["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+            "dtype": "bf16 weights and activations, fp32 stream and accumulation", "data": "synthetic (random-init weights of the named shape)",
+            "config": {"workload": workload, "l2": "weights larger than L2 are streamed per step", "peak_source": hbm_src},
+            "clocks": ours["clocks"], "gpu_launches": ours["gpu_launches"],
+            "e2e": {"value": ours["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 * args.batch, "d2h_bytes_per_step": 4 * args.batch}}
+
+
+def bench_stream():
+    import torch
+
+    torch.cuda.set_device(0)
+    stream = torch.cuda.Stream()
+    torch.cuda.set_stream(stream)
+    return stream
+
+
+def run_vuzunex(args, pkg):
+    """Prompt and decode throughput of the Vuzunex design (dense bf16 weights, latent attention, fp32 stream) beside the Llama
+    recipe (4-bit weights, grouped-query attention) at equal width, heads, feed-forward, layers and vocabulary. One JSON line."""
+    stream = bench_stream()
+    timed = stream_timer(stream)
+    width, heads, ff, layers = VUZUNEX_SHAPES[args.shape]
+    batch, ctx, P = args.batch, args.ctx, pkg.plan
+    max_seq = ctx + 4 * (max(3, args.warmup) + args.steps) + 64
+    hbm, _ = measured_peaks()
+    ours = measure_vuzunex(pkg, vuzunex_config(pkg, args, layers, max_seq), args, stream, timed)
+    lcfg = pkg.ModelConfig("llama", width, ff, layers, heads, heads // 4, 128, BENCH_VOCAB, max_seq=max_seq, max_batch=batch)
+    builder = pkg.DispatchPlanBuilder(lcfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, block_weights(builder))
+    model.set_stream(stream.cuda_stream)
+    closest = serve_rates(model, np.random.default_rng(7).integers(0, BENCH_VOCAB, size=(batch, ctx), dtype=np.int32), args, timed)
+    if batch <= 16:
+        model.profile_kind(P.STEP_QGEMV, 2)
+        ms, weight_bytes = timed(lambda: model.profile_kind(P.STEP_QGEMV, 1), 10), lcfg.q4_weight_elems() * 0.5625
+        closest["decode_products"] = {"ms": ms, "bytes": weight_bytes, "GBs": weight_bytes / ms / 1e6, "frac": weight_bytes / ms / 1e6 / hbm}
+        model.profile_kind(P.STEP_ATTN_DECODE, 2)
+        ms, kv = timed(lambda: model.profile_kind(P.STEP_ATTN_DECODE, 1), 10), layers * batch * model.position * lcfg.kv_heads * 128 * 4
+        closest["decode_attention"] = {"us_per_layer": ms * 1e3 / layers, "bytes": kv, "GBs": kv / ms / 1e6, "frac": kv / ms / 1e6 / hbm}
+    model.close()
+    store.close()
+    workload = f"{layers} layers, width {width}, {heads} heads (128 + 64 / 128, latent 512), feed-forward {ff}, vocabulary {BENCH_VOCAB}, context {ctx}, batch {batch}"
+    print(json.dumps(dict(design_line(args, "Vuzunex", ours, workload), vuzunex=ours, llama_q4_equal_size=closest)))
+
+
+RIROTAR_SHAPES = {   # layers, experts, chosen experts, groups, kept groups: width, heads and active feed-forward are VUZUNEX_SHAPES's
+    "1b": (12, 64, 8, 8, 4), "8b": (8, 32, 8, 4, 2)}
+RIROTAR_WINDOW = 1024
+
+
+def run_rirotar(args, pkg):
+    """Prompt and decode throughput of the Rirotar design (three gated-delta layers to one latent-attention layer, routed
+    feed-forwards) beside Vuzunex (latent attention, dense feed-forwards of the active size) at equal width, heads, layers and
+    vocabulary, and its recurrence beside the DeltaNet recipe's. One JSON line."""
+    R, P = pkg.rirotar, pkg.plan
+    stream = bench_stream()
+    timed = stream_timer(stream)
+    width, heads, ff, _ = VUZUNEX_SHAPES[args.shape]
+    layers, experts, top, groups, keep = RIROTAR_SHAPES[args.shape]
+    batch, ctx = args.batch, args.ctx
+    max_seq = ctx + 4 * (max(3, args.warmup) + args.steps) + 64
+    hbm, _ = measured_peaks()
+    tensor, _ = measured_tensor_peak()
+    routed, dense = R.RoutedFF(ff // top, 7.0, experts, top, groups, keep, 2.5), R.DenseFF(ff, 7.0)
+    channel = R.GatedDelta(heads, heads, 128, 128, 4, True, 128, 128)
+    scalar = R.GatedDelta(heads, heads // 2, 128, 128, 4, False)
+    latent = R.WindowedLatentAttention(heads, 128, 128, 512, 128 ** -0.5, RIROTAR_WINDOW)
+    block = [R.Layer(channel, routed), R.Layer(scalar, routed), R.Layer(channel, routed), R.Layer(latent, dense)]
+    cfg = pkg.RirotarConfig(vocab=BENCH_VOCAB, width=width, layers=[block[i % 4] for i in range(layers)], logit_softcap=30.0, max_seq=max_seq, max_batch=batch)
+    n_routed, n_latent = 3 * layers // 4, layers // 4
+    n_delta = layers - n_latent
+    builder = pkg.RirotarPlanBuilder(cfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, block_weights(builder))
+    model.set_stream(stream.cuda_stream)
+    prompt = np.random.default_rng(7).integers(0, BENCH_VOCAB, size=(batch, ctx), dtype=np.int32)
+    ours = serve_rates(model, prompt, args, timed)
+
+    def kind_ms(kind):
+        model.profile_kind(kind, 2)
+        return timed(lambda: model.profile_kind(kind, 1), 10)
+
+    def hbm_entry(ms, nbytes, count):
+        return {"us_per_layer": ms * 1e3 / count, "bytes": nbytes, "GBs": nbytes / ms / 1e6, "frac": nbytes / ms / 1e6 / hbm}
+
+    product_bytes = cfg.product_elems() * 2
+    ours["decode_products"] = hbm_entry(kind_ms(P.STEP_PRODUCT), product_bytes, layers)
+    state_bytes = 2.0 * n_delta * batch * heads * 128 * 128 * 4
+    ours["decode_delta_step"] = hbm_entry(kind_ms(P.STEP_GATED_DELTA), state_bytes, n_delta)
+    # experts that `batch` rows of evenly spread choices reach
+    reached = experts * (1.0 - (1.0 - top / experts) ** batch)
+    expert_bytes = n_routed * reached * 3 * width * (ff // top) * 2
+    ours["decode_routed"] = hbm_entry(kind_ms(P.STEP_ROUTED_MLP), expert_bytes, n_routed)
+    small, kv = n_latent * heads * 256 * 512 * 2, n_latent * batch * min(model.position, RIROTAR_WINDOW) * 512 * 2
+    ours["decode_attention"] = hbm_entry(kind_ms(P.STEP_ATTN_DECODE), kv, n_latent)
+    ours["decode_latent_step"] = hbm_entry(kind_ms(P.STEP_LATENT_ATTN), small + kv, n_latent)
+    n = min(ctx, 2048)
+    model.reset_state()
+    chunk = prompt[0, :n]
+
+    def chunk_ms(kind):
+        model.profile_batch(0, chunk, kind, 2)
+        return timed(lambda: model.profile_batch(0, chunk, kind, 5), 1) / 5
+
+    def tensor_entry(ms, flops, count):
+        return {"rows": n, "us_per_layer": ms * 1e3 / count, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
+
+    ours["prefill_products"] = tensor_entry(chunk_ms(P.STEP_PRODUCT), 2.0 * n * (product_bytes / 2 - BENCH_VOCAB * width), layers)
+    ours["prefill_routed"] = tensor_entry(chunk_ms(P.STEP_ROUTED_MLP), n_routed * 2.0 * n * top * 3 * width * (ff // top), n_routed)
+    w = min(n, RIROTAR_WINDOW)
+    pairs = w * (w + 1) / 2 + (n - w) * w
+    ours["prefill_attention"] = tensor_entry(chunk_ms(P.STEP_ATTN_DECODE), n_latent * heads * pairs * 2.0 * 256, n_latent)
+    ours["prefill_latent_step_us_per_layer"] = chunk_ms(P.STEP_LATENT_ATTN) * 1e3 / n_latent
+    # per token and head: decay, two products with the state, one update
+    ours["prefill_delta"] = {"rows": n, "us_per_layer": chunk_ms(P.STEP_GATED_DELTA) * 1e3 / n_delta}
+    ours["prefill_delta"]["fp32_tflops"] = n * heads * 128 * 128 * 7.0 / ours["prefill_delta"]["us_per_layer"] / 1e6
+    model.close()
+    store.close()
+    closest = measure_vuzunex(pkg, vuzunex_config(pkg, args, layers, max_seq), args, stream, timed)
+    # the recurrence of the DeltaNet recipe at the same heads, in a model with little else (decode steps per layer)
+    dcfg = pkg.ModelConfig("deltanet", 512, 512, 5, 4, 2, 128, 4096, attention_layers=[4], max_seq=max_seq, max_batch=batch, ssm_heads=heads,
+                           ssm_groups=heads, ssm_key_dim=128, ssm_value_dim=128, ssm_conv_kernel=4)
+    builder = pkg.DispatchPlanBuilder(dcfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, pkg.synth_model_weights(builder, seed=3))
+    model.set_stream(stream.cuda_stream)
+    like = {}
+    if batch <= 16:
+        model.profile_kind(P.STEP_SSM_RECURRENCE, 2)
+        like["decode"] = hbm_entry(timed(lambda: model.profile_kind(P.STEP_SSM_RECURRENCE, 1), 10), 2.0 * 4 * batch * heads * 128 * 128 * 4, 4)
+    if batch == 1:
+        p = np.random.default_rng(8).integers(0, 4096, size=(1, n), dtype=np.int32)
+        model.set_prefill_chunk(n)
+        model.prefill(p)
+        model.reset_state()
+        like["prefill_us_per_layer_at_most"] = timed(lambda: model.prefill(p), 1) * 1e3 / 4
+    model.close()
+    store.close()
+    workload = (f"{layers} layers (channel delta, delta, channel delta, latent), width {width}, {heads} heads of 128 x 128, latent 512 over a window of {RIROTAR_WINDOW}, "
+                f"{top} of {experts} experts of {ff // top} (dense {ff} behind latent layers), vocabulary {BENCH_VOCAB}, context {ctx}, batch {batch}")
+    print(json.dumps(dict(design_line(args, "Rirotar", ours, workload), rirotar=ours, vuzunex_equal_size=closest, deltanet_recurrence_equal_heads=like)))
 
 
 def main():
@@ -449,9 +592,9 @@ def main():
     ap.add_argument("--prefill", choices=["real", "synthetic"], default="real",
                     help="how the KV cache gets its `ctx` tokens: by running the prompt, or random bf16 rows")
     ap.add_argument("--small", action="store_true")
-    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex"], default="llama",
-                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size")
-    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex: which layer sizes")
+    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex", "rirotar"], default="llama",
+                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size; rirotar: the gated-delta design beside Vuzunex of equal size")
+    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex, rirotar: which layer sizes")
     ap.add_argument("--batch", type=int, default=1, help="sequences decoded together (1..64), all at the same position")
     ap.add_argument("--kv", choices=["bf16", "q8", "rotor-q4", "rotor-q4-qjl16"], default="bf16",
                     help="KV cache elements: bf16, 8-bit groups of 32 (36-byte blocks), or the rotated 4-bit groups of 64 "
@@ -463,6 +606,9 @@ def main():
 
     if args.model == "vuzunex":
         run_vuzunex(args, pkg)
+        return
+    if args.model == "rirotar":
+        run_rirotar(args, pkg)
         return
     if args.model == "lfm2" and args.ctx == 4096:
         args.ctx = 2048   # the hybrid configuration's prompt length

@@ -26,16 +26,22 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
     return v;
 }
 
-__device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
+// Where the results of one weight row go: that of activation row m is m * stride bytes behind y.
+struct ProductRow { unsigned char* y; size_t stride; bool f32; };
+__device__ __forceinline__ ProductRow product_row(const ProductOut& o, int row) {
     void* y = o.y[0];
     int first = 0, stride = o.stride[0], f32 = o.f32[0];
 #pragma unroll
     for (int q = 1; q < kMaxProductSegs; ++q)
         if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; }
-    const size_t at = (size_t)m * stride + (row - first);
+    const int size = f32 ? 4 : 2;
+    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0};
+}
+__device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
+    const ProductRow r = product_row(o, row);
     if (o.softcap > 0.f) val = o.softcap * tanhf(val / o.softcap);
-    if (f32) static_cast<float*>(y)[at] = val;
-    else static_cast<__nv_bfloat16*>(y)[at] = __float2bfloat16_rn(val);
+    if (r.f32) *reinterpret_cast<float*>(r.y + m * r.stride) = val;
+    else *reinterpret_cast<__nv_bfloat16*>(r.y + m * r.stride) = __float2bfloat16_rn(val);
 }
 
 // ---- few rows ---------------------------------------------------------------------------------------------------------
@@ -293,7 +299,8 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
 // ---- many rows, bf16: tcgen05 -----------------------------------------------------------------------------------------
 constexpr int kTileRows = 128;       // weight rows of one accumulator = UMMA M
 constexpr int kTcK = 64;             // columns per stage = one 128-byte swizzle row
-constexpr int kTcWarps = 6;          // TMA, MMA, four epilogue warps
+constexpr int kTcEpilogueWarps = 8;
+constexpr int kTcWarps = 2 + kTcEpilogueWarps;   // TMA, MMA, epilogue
 constexpr int kTcBlock = kTcWarps * 32;
 
 struct TcParams {
@@ -316,6 +323,14 @@ __device__ __forceinline__ void umma_bf16(unsigned d_tmem, unsigned long long a_
         "setp.ne.b32 p, %4, 0;\n\t"
         "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
         ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
+}
+
+__device__ __forceinline__ void tmem_ld16(unsigned (&v)[16], unsigned at) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
+          "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+        : "r"(at) : "memory");
 }
 
 template <int BN, int STAGES, bool GATED>
@@ -409,7 +424,8 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
         }
         __syncwarp();
     } else {
-        // ---- epilogue: a warp reads the 32 accumulator lanes of its quarter (warp & 3), lane = weight row ----
+        // ---- epilogue: a warp reads the 32 accumulator lanes of its quarter (warp & 3), lane = weight row; the two warps of a
+        // quarter take turns with the activation rows ----
         pdl_wait();   // the outputs may still be read by the kernel before this one
         const bool ok = mbar_wait(&done_bar, 0u);
         if (!ok) { atomicExch(p.status, 33); }
@@ -420,31 +436,29 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
 #pragma unroll 1
             for (int t = 0; t < (GATED && !cut ? 1 : nt); ++t) {
                 const int row = row0 + (GATED ? 0 : t * kTileRows) + quarter * 32 + lane;
+                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true}
+                                           : product_row(p.out, row);
 #pragma unroll 1
-                for (int c0 = 0; c0 < BN; c0 += 16) {
+                for (int c0 = 16 * ((warp - 2) >> 2); c0 < BN; c0 += 16 * (kTcEpilogueWarps / 4)) {
                     if (tok0 + c0 >= tok_end) break;   // uniform across the warp
                     unsigned v[16], u[16];
                     const unsigned at = tmem + ((unsigned)(quarter * 32) << 16) + (unsigned)(t * BN + c0);
-                    asm volatile(
-                        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-                        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
-                          "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
-                        : "r"(at) : "memory");
-                    if (GATED && !cut)
-                        asm volatile(
-                            "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-                            : "=r"(u[0]), "=r"(u[1]), "=r"(u[2]), "=r"(u[3]), "=r"(u[4]), "=r"(u[5]), "=r"(u[6]), "=r"(u[7]),
-                              "=r"(u[8]), "=r"(u[9]), "=r"(u[10]), "=r"(u[11]), "=r"(u[12]), "=r"(u[13]), "=r"(u[14]), "=r"(u[15])
-                            : "r"(at + BN) : "memory");
+                    tmem_ld16(v, at);
+                    if (GATED && !cut) tmem_ld16(u, at + BN);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                     if (row < p.n) {
+                        const int count = tok_end - tok0 - c0;
+                        unsigned char* y = dst.y + (size_t)(tok0 + c0) * dst.stride;
 #pragma unroll
                         for (int i = 0; i < 16; ++i) {
-                            const int tok = tok0 + c0 + i;
-                            if (tok >= tok_end) break;
-                            const float val = __uint_as_float(v[i]);
-                            if (cut) p.part[(((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m + tok) * p.n + row] = val;
-                            else product_store(p.out, tok, row, GATED ? gated_activation(val, __uint_as_float(u[i]), p.act) : val);
+                            float val = __uint_as_float(v[i]);
+                            if (GATED && !cut) val = gated_activation(val, __uint_as_float(u[i]), p.act);
+                            if (p.out.softcap > 0.f && !cut) val = p.out.softcap * tanhf(val / p.out.softcap);
+                            if (i < count) {
+                                if (dst.f32) *reinterpret_cast<float*>(y) = val;
+                                else *reinterpret_cast<__nv_bfloat16*>(y) = __float2bfloat16_rn(val);
+                            }
+                            y += dst.stride;
                         }
                     }
                 }
@@ -611,7 +625,7 @@ int tc_launch(const ProductLaunch& a, const TcShape& t, cudaStream_t s) {
                           : launch_k(bgemm_tc_kernel<BN, STAGES, false>, grid, dim3(kTcBlock), tc_smem<BN, STAGES>(), s, p, xmap, wmap, wmap2);
     if (e != cudaSuccess) return cuda_fail(e, "bgemm launch");
     if (t.ranges > 1) {
-        const dim3 g((unsigned)((p.n + 255) / 256), (unsigned)std::min(p.m, 64));
+        const dim3 g((unsigned)((p.n + 255) / 256), (unsigned)std::min(p.m, std::max(64, 8 * 148 * 256 / p.n)));
         e = gated ? launch_k(bgemm_sum_kernel<true>, g, dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out)
                   : launch_k(bgemm_sum_kernel<false>, g, dim3(256), 0, s, (const float*)a.part, t.ranges, p.m, p.n, p.act, p.out);
         if (e != cudaSuccess) return cuda_fail(e, "bgemm sum launch");

@@ -11,7 +11,7 @@
 //
 // Inside a block, with S the state in front of it, G_t the product of the decays up to token t and D_ts the product of the
 // decays of tokens s + 1 .. t (all at most 1, nothing is divided):
-//   u_t = beta_t (v_t - S^T (G_t k_t)) - sum_{s < t} beta_t (k_s . D_ts k_t) u_s
+//   u_t = beta_t (v_t - S^T (G_t k_t)) - sum_{s < t} beta_t (k_s . D_ts k_t) u_s     (a triangular system)
 //   o_t = S^T (G_t q_t) + sum_{s <= t} (k_s . D_ts q_t) u_s
 //   S' = G_T S + sum_s (D_Ts k_s) u_s^T
 // The products of k and q with each other do not depend on the state's column: they are formed once per head. Everything is
@@ -30,7 +30,7 @@ namespace swlm {
 namespace {
 
 constexpr int TB = kDeltaBlock;
-constexpr int kScanCols = 16, kScanParts = 8, kScanThreads = kScanCols * kScanParts, kScanStages = 4;
+constexpr int kScanCols = 16, kScanWarpCols = 4, kScanThreads = kScanCols / kScanWarpCols * 32, kScanStages = 4;
 constexpr int kStepCols = 32, kStepWarps = 8, kStepThreads = kStepWarps * 32, kStepCluster = 8;
 constexpr int kPrepThreads = 128;
 
@@ -97,35 +97,93 @@ __device__ __forceinline__ float decay_of(const DeltaParams& p, int row, int h, 
 }
 
 // ---- portions: what a block needs of its tokens -----------------------------------------------------------------------
-// CTA (block, head). Record: [TB][dp] beta_t G_t k_t, [TB][dp] G_t q_t, [TB][dp] D_Ts k_s, [dp] G_T, then the coefficients
-// [TB][TB] of u_t and [TB][TB] of o_t. Values: [column block][TB][kScanCols] beta_t v_t. Tokens past the end of the run: k = q
-// = v = 0 and a decay of 1.
+// CTA (block, head). Record: [TB][dp] beta_t G_t k_t, [TB][dp] G_t q_t, [TB][dp] D_Ts k_s, [dp] G_T, then two [TB][TB] matrices
+// that turn w_s = beta_s v_s - S^T (beta_s G_s k_s) into u and into the block's own share of o: with A_ts = beta_t (k_s . D_ts k_t)
+// for s < t and B_ts = k_s . D_ts q_t for s <= t, u = (I + A)^-1 w and the share is B u. Values: [column block][TB][kScanCols]
+// beta_t v_t. Tokens past the end of the run: k = q = v = 0 and a decay of 1.
+constexpr int kPrepTaps = 4;   // convolutions of up to this many taps read every input once
+template <typename T>
+__device__ __forceinline__ void conv_block(const DeltaParams& p, const RowRun& run, int ch, int t0, int nt, float (&y)[TB]) {
+    if (p.sh.taps > kPrepTaps) {
+#pragma unroll
+        for (int t = 0; t < TB; ++t) y[t] = t < nt ? conv_silu<T>(p, run, ch, t0 + t) : 0.f;
+        return;
+    }
+    const __nv_bfloat16* w = taps_of(p, ch);
+    float wf[kPrepTaps], x[TB + kPrepTaps - 1];
+#pragma unroll
+    for (int j = 0; j < kPrepTaps; ++j) wf[j] = j < p.sh.taps ? __bfloat162float(w[p.sh.taps - 1 - j]) : 0.f;   // wf[j] meets the input j tokens back
+    const T* in = static_cast<const T*>(p.qkv) + (size_t)(run.row0 + t0) * p.qkv_stride + ch;
+    if (t0 >= kPrepTaps - 1) {
+#pragma unroll
+        for (int i = 0; i < TB + kPrepTaps - 1; ++i) {
+            const int at = i - (kPrepTaps - 1);
+            x[i] = at < nt ? dl_get(in + (ptrdiff_t)at * p.qkv_stride) : 0.f;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < TB + kPrepTaps - 1; ++i) {
+            const int at = i - (kPrepTaps - 1);
+            x[i] = at < nt && at > -p.sh.taps ? conv_input<T>(p, run, ch, t0 + at) : 0.f;
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < TB; ++t) {
+        float acc = 0.f;
+#pragma unroll
+        for (int j = kPrepTaps - 1; j >= 0; --j) acc = fmaf(wf[j], x[t + kPrepTaps - 1 - j], acc);
+        y[t] = t < nt ? silu(acc) : 0.f;
+    }
+}
+
+// Sums over the warp of 32 values a lane, value `lane` left in this lane: at every step half of the values go to the partner.
+__device__ __forceinline__ float warp_sums(float (&v)[32], int lane) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool upper = lane & o;
+#pragma unroll
+        for (int j = 0; j < o; ++j) {
+            const float give = upper ? v[j] : v[j + o], keep = upper ? v[j + o] : v[j];
+            v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+    return v[0];
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const DeltaParams p) {
-    pdl_launch_dependents();
+    static_assert(TB == 4, "the pair sums of a block fill the lanes of a warp");
     pdl_wait();
     extern __shared__ __align__(16) float prep_smem[];
-    __shared__ float beta_s[TB], norm_s[2 * TB], red[kPrepThreads / 32][2 * TB * TB];
+    __shared__ float beta_s[TB], decay_s[TB], norm_s[2 * TB], red[kPrepThreads / 32][2 * TB * TB], a_s[TB][TB], b_s[TB][TB], m_s[TB][TB];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, blk = blockIdx.x, h = blockIdx.y;
     const RowRun run = run_of(p, p.block_run ? p.block_run[blk] : blk);
     const int t0 = (blk - run.blk0) * TB, nt = min(TB, run.count - t0);
     const int dim = p.sh.dim, vdim = p.sh.vdim, grp = h / (p.sh.heads / p.sh.groups), gk = p.sh.groups * dim;
+    const float rate = expf(__bfloat162float(p.a_log[h]));
     float* q = prep_smem;            // [TB][dim]
     float* k = q + TB * dim;         // [TB][dim]
-    if (tid < TB) beta_s[tid] = tid < nt ? sigmoid(p.beta[(size_t)(run.row0 + t0 + tid) * p.beta_stride + h]) : 0.f;
-    __syncthreads();
+    if (tid < TB) {
+        const int row = run.row0 + t0 + tid;
+        beta_s[tid] = tid < nt ? sigmoid(p.beta[(size_t)row * p.beta_stride + h]) : 0.f;
+        if (p.decay_dim == 1) decay_s[tid] = tid < nt ? decay_of(p, row, h, 0, rate) : 1.f;
+    }
     for (int i = tid; i < 2 * dim; i += kPrepThreads) {
         const int d = i < dim ? i : i - dim, ch = (i < dim ? 0 : gk) + grp * dim + d;
         float* dst = i < dim ? q : k;
+        float y[TB];
+        conv_block<T>(p, run, ch, t0, nt, y);
 #pragma unroll
-        for (int t = 0; t < TB; ++t) dst[t * dim + d] = t < nt ? conv_silu<T>(p, run, ch, t0 + t) : 0.f;
+        for (int t = 0; t < TB; ++t) dst[t * dim + d] = y[t];
     }
-    float* vr = p.vrec + (size_t)(blk * p.sh.heads + h) * p.vblocks * TB * kScanCols;
-    for (int c = tid; c < p.vblocks * kScanCols; c += kPrepThreads)
-#pragma unroll
-        for (int t = 0; t < TB; ++t)
-            vr[(c / kScanCols * TB + t) * kScanCols + c % kScanCols] = t < nt && c < vdim ? beta_s[t] * conv_silu<T>(p, run, 2 * gk + h * vdim + c, t0 + t) : 0.f;
     __syncthreads();
+    float* vr = p.vrec + (size_t)(blk * p.sh.heads + h) * p.vblocks * TB * kScanCols;
+    for (int c = tid; c < p.vblocks * kScanCols; c += kPrepThreads) {
+        float y[TB] = {};
+        if (c < vdim) conv_block<T>(p, run, 2 * gk + h * vdim + c, t0, nt, y);
+#pragma unroll
+        for (int t = 0; t < TB; ++t) vr[(c / kScanCols * TB + t) * kScanCols + c % kScanCols] = beta_s[t] * y[t];
+    }
     for (int i = warp; i < 2 * TB; i += kPrepThreads / 32) {
         const float* x = (i < TB ? q : k) + (i % TB) * dim;
         float ss = 0.f;
@@ -134,13 +192,10 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Delta
         if (lane == 0) norm_s[i] = (i < TB ? p.q_scale : 1.0f) / sqrtf(ss + p.unit_eps);
     }
     __syncthreads();
-    const float rate = expf(__bfloat162float(p.a_log[h]));
     float* rec = p.rec + (size_t)(blk * p.sh.heads + h) * p.rec_floats;
-    float a[TB][TB], b[TB][TB];
+    float pairs[2 * TB * TB];   // A without beta, B
 #pragma unroll
-    for (int t = 0; t < TB; ++t)
-#pragma unroll
-        for (int s = 0; s < TB; ++s) a[t][s] = b[t][s] = 0.f;
+    for (int i = 0; i < 2 * TB * TB; ++i) pairs[i] = 0.f;
     for (int d = tid; d < p.dp; d += kPrepThreads) {
         float kv[TB], qv[TB], g[TB];
 #pragma unroll
@@ -148,7 +203,7 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Delta
             const bool live = d < dim && t < nt;
             kv[t] = live ? k[t * dim + d] * norm_s[TB + t] : 0.f;
             qv[t] = live ? q[t * dim + d] * norm_s[t] : 0.f;
-            g[t] = live ? decay_of(p, run.row0 + t0 + t, h, d, rate) : 1.f;
+            g[t] = !live ? 1.f : p.decay_dim == 1 ? decay_s[t] : decay_of(p, run.row0 + t0 + t, h, d, rate);
         }
         float gt = 1.f;
 #pragma unroll
@@ -161,47 +216,64 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Delta
 #pragma unroll
         for (int s = 0; s < TB; ++s) {
             float w = kv[s];
-            b[s][s] = fmaf(w, qv[s], b[s][s]);
+            pairs[TB * TB + s * TB + s] = fmaf(w, qv[s], pairs[TB * TB + s * TB + s]);
 #pragma unroll
             for (int t = s + 1; t < TB; ++t) {
                 w *= g[t];
-                a[t][s] = fmaf(w, kv[t], a[t][s]);
-                b[t][s] = fmaf(w, qv[t], b[t][s]);
+                pairs[t * TB + s] = fmaf(w, kv[t], pairs[t * TB + s]);
+                pairs[TB * TB + t * TB + s] = fmaf(w, qv[t], pairs[TB * TB + t * TB + s]);
             }
             rec[(2 * TB + s) * p.dp + d] = w;
         }
     }
-#pragma unroll
-    for (int t = 0; t < TB; ++t)
-#pragma unroll
-        for (int s = 0; s <= t; ++s) {
-            const float y = warp_sum(b[t][s]);
-            const float x = s < t ? warp_sum(a[t][s]) : 0.f;
-            if (lane == 0) { red[warp][t * TB + s] = x; red[warp][TB * TB + t * TB + s] = y; }
-        }
+    red[warp][lane] = warp_sums(pairs, lane);
     __syncthreads();
     if (tid < 2 * TB * TB) {
-        const int t = tid % (TB * TB) / TB, s = tid % TB;
         float v = 0.f;
-        if (s <= t)
-            for (int w = 0; w < kPrepThreads / 32; ++w) v += red[w][tid];
-        rec[(3 * TB + 1) * p.dp + tid] = tid < TB * TB ? beta_s[t] * v : v;
+#pragma unroll
+        for (int w = 0; w < kPrepThreads / 32; ++w) v += red[w][tid];
+        const int t = tid % (TB * TB) / TB, s = tid % TB;
+        if (tid < TB * TB) a_s[t][s] = beta_s[t] * v;
+        else b_s[t][s] = v;
+    }
+    __syncwarp();
+    if (tid < TB) {   // column tid of (I + A)^-1
+        float m[TB];
+#pragma unroll
+        for (int t = 0; t < TB; ++t) {
+            m[t] = t == tid ? 1.f : 0.f;
+#pragma unroll
+            for (int s = 0; s < t; ++s) m[t] = fmaf(-a_s[t][s], m[s], m[t]);
+            m_s[t][tid] = m[t];
+        }
+    }
+    __syncwarp();
+    if (tid < 2 * TB * TB) {
+        const int t = tid % (TB * TB) / TB, s = tid % TB;
+        float v = m_s[t][s];
+        if (tid >= TB * TB) {
+            v = 0.f;
+            for (int e = 0; e <= t; ++e) v = fmaf(b_s[t][e], m_s[e][s], v);
+        }
+        rec[(3 * TB + 1) * p.dp + tid] = v;
     }
 }
 
 // ---- portions: the recurrence -----------------------------------------------------------------------------------------
-// CTA (16 columns of the state, head, run). Eight lanes share a column: lane part j holds key channels 4 j + 32 i + (0 .. 3), so
-// that a 16-byte read of a record row by the parts of a warp is free of bank conflicts. Records come through a ring of bulk
-// copies. At the end the run's last inputs go to the convolution ring (all readers of the old ones have finished).
+// CTA (16 columns of the state, head, run): a warp holds four columns, a lane key channels 4 lane + 128 i + (0 .. 3) of them, so
+// that a record row is read once per four columns. The 32 products of a block with the state (w and o of four tokens and four
+// columns) are summed across the warp in 31 exchanges that leave one in each lane. Records come through a ring of bulk copies.
+// At the end the run's last inputs go to the convolution ring (all readers of the old ones have finished).
+// Launched without overlap: CTAs that move in while another kernel drains would crowd together on the SMs that drain first.
 template <typename T, int R>
 __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaParams p) {
-    constexpr int DP = R * kScanParts, REC = (3 * TB + 1) * DP + 2 * TB * TB, VREC = TB * kScanCols, STAGE = REC + VREC;
+    constexpr int DP = R * 32, REC = (3 * TB + 1) * DP + 2 * TB * TB, VREC = TB * kScanCols, STAGE = REC + VREC, WC = kScanWarpCols;
     extern __shared__ __align__(128) float scan_smem[];
     __shared__ __align__(8) unsigned long long full_bar[kScanStages];
+    __shared__ __align__(16) float u_s[kScanThreads / 32][TB * WC];
     __shared__ int bad;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane & 7, lc = warp * 4 + (lane >> 3);
-    const int vb = blockIdx.x, h = blockIdx.y, col = vb * kScanCols + lc;
-    pdl_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int vb = blockIdx.x, h = blockIdx.y, col0 = vb * kScanCols + warp * WC;
     if (tid == 0) {
         for (int s = 0; s < kScanStages; ++s) mbar_init(&full_bar[s], 1);
         bad = 0;
@@ -211,7 +283,6 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     pdl_wait();
     const RowRun run = run_of(p, blockIdx.z);
     const int nb = (run.count + TB - 1) / TB;
-    const bool live = col < p.sh.vdim;
     auto request = [&](int b) {   // thread 0
         const int s = b % kScanStages;
         const unsigned bar = smem_u32(&full_bar[s]), dst = smem_u32(scan_smem + (size_t)s * STAGE);
@@ -222,65 +293,67 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     };
     int issued = 0;
     if (tid == 0) for (; issued < min(kScanStages, nb); ++issued) request(issued);
-    float* st = p.state + ((size_t)run.seq * p.sh.heads + h) * p.sh.dim * p.sh.vdim + col;
-    float S[R];
+    float* st = p.state + ((size_t)run.seq * p.sh.heads + h) * p.sh.dim * p.sh.vdim + col0;
+    auto channel = [&](int i) { return lane * 4 + 128 * (i >> 2) + (i & 3); };
+    float S[WC][R];
 #pragma unroll
-    for (int i = 0; i < R; ++i) {
-        const int d = part * 4 + 32 * (i >> 2) + (i & 3);
-        S[i] = live && run.pos0 > 0 && d < p.sh.dim ? st[(size_t)d * p.sh.vdim] : 0.f;
-    }
-    float* o_row = p.o + (size_t)run.row0 * p.sh.heads * p.sh.vdim + (size_t)h * p.sh.vdim + col;
-    const int o_stride = p.sh.heads * p.sh.vdim;
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int c = 0; c < WC; ++c) S[c][i] = run.pos0 > 0 && channel(i) < p.sh.dim && col0 + c < p.sh.vdim ? st[(size_t)channel(i) * p.sh.vdim + c] : 0.f;
+    // after the sums lane = 16 * (0: w, 1: o) + 4 * token + column
+    const int tok = (lane >> 2) & 3, oc = col0 + (lane & 3);
+    float* o_at = p.o + ((size_t)(run.row0 + tok) * p.sh.heads + h) * p.sh.vdim + oc;
+    const size_t o_step = (size_t)TB * p.sh.heads * p.sh.vdim;
     for (int b = 0; b < nb; ++b) {
         const int s = b % kScanStages;
         if (!mbar_wait(&full_bar[s], (unsigned)((b / kScanStages) & 1))) { atomicExch(p.status, 51); bad = 1; }
         const float* rec = scan_smem + (size_t)s * STAGE;
-        const float4* r4 = reinterpret_cast<const float4*>(rec) + part;
-        float a[TB], q[TB];
+        const float4* r4 = reinterpret_cast<const float4*>(rec) + lane;
+        const float4 coef = *reinterpret_cast<const float4*>(rec + (3 * TB + 1) * DP + (lane >> 2) * TB);
+        const float vv = rec[REC + tok * kScanCols + warp * WC + (lane & 3)];
+        float x[2 * TB * WC];
 #pragma unroll
-        for (int t = 0; t < TB; ++t) a[t] = q[t] = 0.f;
+        for (int i = 0; i < 2 * TB * WC; ++i) x[i] = 0.f;
 #pragma unroll
         for (int i = 0; i < R / 4; ++i)
 #pragma unroll
-            for (int t = 0; t < TB; ++t) {
-                const float4 kt = r4[(t * DP + 32 * i) / 4], qt = r4[((TB + t) * DP + 32 * i) / 4];
-                a[t] = fmaf(S[4 * i], kt.x, a[t]); a[t] = fmaf(S[4 * i + 1], kt.y, a[t]); a[t] = fmaf(S[4 * i + 2], kt.z, a[t]); a[t] = fmaf(S[4 * i + 3], kt.w, a[t]);
-                q[t] = fmaf(S[4 * i], qt.x, q[t]); q[t] = fmaf(S[4 * i + 1], qt.y, q[t]); q[t] = fmaf(S[4 * i + 2], qt.z, q[t]); q[t] = fmaf(S[4 * i + 3], qt.w, q[t]);
+            for (int t = 0; t < 2 * TB; ++t) {
+                const float4 y = r4[(t * DP + 128 * i) / 4];
+#pragma unroll
+                for (int c = 0; c < WC; ++c) {
+                    float& acc = x[t * WC + c];
+                    acc = fmaf(S[c][4 * i], y.x, acc); acc = fmaf(S[c][4 * i + 1], y.y, acc); acc = fmaf(S[c][4 * i + 2], y.z, acc); acc = fmaf(S[c][4 * i + 3], y.w, acc);
+                }
             }
+        const float sum = warp_sums(x, lane);
+        const float w = vv - sum;                            // (of lanes 0 .. 15)
+        float r = lane < 16 ? 0.f : sum;
+        r = fmaf(coef.x, __shfl_sync(0xffffffffu, w, lane & 3), r);
+        r = fmaf(coef.y, __shfl_sync(0xffffffffu, w, 4 + (lane & 3)), r);
+        r = fmaf(coef.z, __shfl_sync(0xffffffffu, w, 8 + (lane & 3)), r);
+        r = fmaf(coef.w, __shfl_sync(0xffffffffu, w, 12 + (lane & 3)), r);
+        if (lane < 16) u_s[warp][lane] = r;
+        else if (oc < p.sh.vdim && b * TB + tok < run.count) o_at[b * o_step] = r;
+        __syncwarp();
+        float4 u[TB];
 #pragma unroll
-        for (int o = 1; o < kScanParts; o <<= 1)
-#pragma unroll
-            for (int t = 0; t < TB; ++t) {
-                a[t] += __shfl_xor_sync(0xffffffffu, a[t], o);
-                q[t] += __shfl_xor_sync(0xffffffffu, q[t], o);
-            }
-        const float* coef = rec + (3 * TB + 1) * DP;
-        const float* vv = rec + REC;
-        float u[TB];
-#pragma unroll
-        for (int t = 0; t < TB; ++t) {
-            u[t] = vv[t * kScanCols + lc] - a[t];
-#pragma unroll
-            for (int e = 0; e < t; ++e) u[t] = fmaf(-coef[t * TB + e], u[e], u[t]);
-        }
-#pragma unroll
-        for (int t = 0; t < TB; ++t)
-#pragma unroll
-            for (int e = 0; e <= t; ++e) q[t] = fmaf(coef[TB * TB + t * TB + e], u[e], q[t]);
+        for (int t = 0; t < TB; ++t) u[t] = *reinterpret_cast<const float4*>(&u_s[warp][t * WC]);
 #pragma unroll
         for (int i = 0; i < R / 4; ++i) {
-            const float4 g = r4[(3 * TB * DP + 32 * i) / 4];
-            float x = S[4 * i] * g.x, y = S[4 * i + 1] * g.y, z = S[4 * i + 2] * g.z, w = S[4 * i + 3] * g.w;
+            const float4 g = r4[(3 * TB * DP + 128 * i) / 4];
+#pragma unroll
+            for (int c = 0; c < WC; ++c) { S[c][4 * i] *= g.x; S[c][4 * i + 1] *= g.y; S[c][4 * i + 2] *= g.z; S[c][4 * i + 3] *= g.w; }
 #pragma unroll
             for (int t = 0; t < TB; ++t) {
-                const float4 kt = r4[((2 * TB + t) * DP + 32 * i) / 4];
-                x = fmaf(kt.x, u[t], x); y = fmaf(kt.y, u[t], y); z = fmaf(kt.z, u[t], z); w = fmaf(kt.w, u[t], w);
-            }
-            S[4 * i] = x; S[4 * i + 1] = y; S[4 * i + 2] = z; S[4 * i + 3] = w;
-        }
+                const float4 kt = r4[((2 * TB + t) * DP + 128 * i) / 4];
+                const float uc[WC] = {u[t].x, u[t].y, u[t].z, u[t].w};
 #pragma unroll
-        for (int t = 0; t < TB; ++t)
-            if (part == t && live && b * TB + t < run.count) o_row[(size_t)(b * TB + t) * o_stride] = q[t];
+                for (int c = 0; c < WC; ++c) {
+                    S[c][4 * i] = fmaf(kt.x, uc[c], S[c][4 * i]); S[c][4 * i + 1] = fmaf(kt.y, uc[c], S[c][4 * i + 1]);
+                    S[c][4 * i + 2] = fmaf(kt.z, uc[c], S[c][4 * i + 2]); S[c][4 * i + 3] = fmaf(kt.w, uc[c], S[c][4 * i + 3]);
+                }
+            }
+        }
         __syncthreads();   // the stage is free
         if (bad) break;    // uniform: written before the barrier by whoever gave up
         if (tid == 0 && issued < nb) { request(issued); ++issued; }
@@ -289,13 +362,11 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
         if (tid == 0) for (int b = max(0, issued - kScanStages); b < issued; ++b) mbar_wait(&full_bar[b % kScanStages], (unsigned)((b / kScanStages) & 1));
         return;
     }
-    if (live) {
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int d = part * 4 + 32 * (i >> 2) + (i & 3);
-            if (d < p.sh.dim) st[(size_t)d * p.sh.vdim] = S[i];
-        }
-    }
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int c = 0; c < WC; ++c)
+            if (channel(i) < p.sh.dim && col0 + c < p.sh.vdim) st[(size_t)channel(i) * p.sh.vdim + c] = S[c][i];
     if (vb == 0) {
         const int share = p.sh.heads / p.sh.groups, gk = p.sh.groups * p.sh.dim, ch_all = p.sh.channels();
         const int n_qk = h % share == 0 ? p.sh.dim : 0, grp = h / share;
@@ -451,16 +522,17 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
 }
 
 // ---- launches ---------------------------------------------------------------------------------------------------------
-int scan_regs(int dim) { return dim <= 32 ? 4 : dim <= 64 ? 8 : dim <= 128 ? 16 : dim <= 256 ? 32 : dim <= 512 ? 64 : 0; }
-int rec_floats(int dim) { return (3 * TB + 1) * scan_regs(dim) * kScanParts + 2 * TB * TB; }
+int scan_regs(int dim) { return dim <= 128 ? 4 : dim <= 256 ? 8 : dim <= 512 ? 16 : 0; }   // key channels per lane
+int rec_floats(int dim) { return (3 * TB + 1) * scan_regs(dim) * 32 + 2 * TB * TB; }
 int scan_vblocks(int vdim) { return (vdim + kScanCols - 1) / kScanCols; }
 size_t scan_smem_bytes(int dim) { return (size_t)kScanStages * (rec_floats(dim) + TB * kScanCols) * 4; }
 
 template <typename T, int R>
 int scan_launch(const DeltaParams& p, int runs, cudaStream_t s) {
-    static const cudaError_t attr = cudaFuncSetAttribute(delta_scan_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan_smem_bytes(R * kScanParts));
+    static const cudaError_t attr = cudaFuncSetAttribute(delta_scan_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan_smem_bytes(R * 32));
     if (attr != cudaSuccess) return cuda_fail(attr, "delta scan attributes");
-    const cudaError_t e = launch_k(delta_scan_kernel<T, R>, dim3(p.vblocks, p.sh.heads, runs), dim3(kScanThreads), scan_smem_bytes(R * kScanParts), s, p);
+    delta_scan_kernel<T, R><<<dim3(p.vblocks, p.sh.heads, runs), dim3(kScanThreads), scan_smem_bytes(R * 32), s>>>(p);
+    const cudaError_t e = cudaGetLastError();
     return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "delta scan launch");
 }
 template <typename T>
@@ -471,9 +543,7 @@ int portions(const DeltaParams& p, int runs, int blocks, cudaStream_t s) {
     switch (scan_regs(p.sh.dim)) {
     case 4: rc = scan_launch<T, 4>(p, runs, s); break;
     case 8: rc = scan_launch<T, 8>(p, runs, s); break;
-    case 16: rc = scan_launch<T, 16>(p, runs, s); break;
-    case 32: rc = scan_launch<T, 32>(p, runs, s); break;
-    default: rc = scan_launch<T, 64>(p, runs, s); break;
+    default: rc = scan_launch<T, 16>(p, runs, s); break;
     }
     if (rc) return rc;
     e = launch_k(delta_gate_kernel<T>, dim3(blocks, p.sh.heads), dim3(TB * 32), 0, s, p);
@@ -534,7 +604,7 @@ int launch_delta(const DeltaLaunch& a, cudaStream_t s, int* launches) {
     p.gate = a.gate; p.gate_stride = a.gate_stride; p.conv_q = a.conv_q; p.conv_k = a.conv_k; p.conv_v = a.conv_v; p.norm_w = a.norm_w;
     p.a_log = a.a_log; p.dt_bias = a.dt_bias; p.ring = a.ring; p.state = a.state; p.row_seq = a.row_seq; p.row_pos = a.row_pos;
     p.out = a.out; p.out_stride = a.out_stride; p.n_single = a.n_single; p.single_rows = a.single_rows; p.status = a.status;
-    p.dp = scan_regs(a.shape.dim) * kScanParts; p.rec_floats = rec_floats(a.shape.dim); p.vblocks = scan_vblocks(a.shape.vdim);
+    p.dp = scan_regs(a.shape.dim) * 32; p.rec_floats = rec_floats(a.shape.dim); p.vblocks = scan_vblocks(a.shape.vdim);
     const int blocks = std::max(a.n_blocks, a.n_single);
     p.rec = a.scratch;
     p.vrec = p.rec + (size_t)blocks * a.shape.heads * p.rec_floats;

@@ -2323,6 +2323,7 @@ static int profiled_launch_kind(int step_kind, int* kind) {
     switch (step_kind) {
     case SWLM_STEP_QGEMV: *kind = L_QGEMV; break;
     case SWLM_STEP_ATTN_DECODE: *kind = L_ATTN; break;   // of a latent step: its attention kernel alone
+    case SWLM_STEP_SSM_RECURRENCE: *kind = L_SSM; break;
     case SWLM_STEP_PRODUCT: *kind = L_PRODUCT; break;
     case SWLM_STEP_LATENT_ATTN: *kind = L_LATENT; break;
     case SWLM_STEP_GATED_DELTA: *kind = L_DELTA; break;
