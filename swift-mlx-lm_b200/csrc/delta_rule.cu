@@ -30,9 +30,12 @@ namespace swlm {
 namespace {
 
 constexpr int TB = kDeltaBlock;
-constexpr int kScanCols = 16, kScanWarpCols = 4, kScanThreads = kScanCols / kScanWarpCols * 32, kScanStages = 4;
+constexpr int kScanCols = 16, kScanWarpCols = 2, kScanThreads = kScanCols / kScanWarpCols * 32;
 constexpr int kStepCols = 32, kStepWarps = 8, kStepThreads = kStepWarps * 32, kStepCluster = 8;
 constexpr int kPrepThreads = 128;
+
+// copies in flight: a block is walked in a fraction of a copy's latency; two CTAs fit an SM at up to 256 key channels
+__host__ __device__ constexpr int scan_stages(int regs) { return regs <= 4 ? 14 : regs <= 8 ? 8 : 6; }
 
 struct DeltaParams {
     DeltaShape sh;
@@ -57,14 +60,42 @@ __device__ __forceinline__ float dl_get(const float* p) { return *p; }
 __device__ __forceinline__ float dl_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void dl_put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void dl_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
-__device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu(float x) { return x * sigmoid(x); }
-__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// With bf16 activations the hardware's approximations of exp, log and division are used (still fp32 numbers: their errors are a
+// few units in the last place); fp32 plans use the functions of full accuracy.
+template <typename T> struct Fn;
+template <> struct Fn<float> {
+    static __device__ __forceinline__ float exp(float x) { return expf(x); }
+    static __device__ __forceinline__ float log1p(float x) { return log1pf(x); }
+    static __device__ __forceinline__ float inv(float x) { return 1.0f / x; }
+};
+template <> struct Fn<__nv_bfloat16> {
+    static __device__ __forceinline__ float exp(float x) { return __expf(x); }
+    static __device__ __forceinline__ float log1p(float x) { return __logf(1.0f + x); }
+    static __device__ __forceinline__ float inv(float x) { return __fdividef(1.0f, x); }   // (1 + exp(..) above 2^126 comes out as 0, as it should)
+};
+template <typename T> __device__ __forceinline__ float sigmoid(float x) { return Fn<T>::inv(1.0f + Fn<T>::exp(-x)); }
+template <typename T> __device__ __forceinline__ float silu(float x) { return x * sigmoid<T>(x); }
+template <typename T> __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + Fn<T>::log1p(Fn<T>::exp(-fabsf(x))); }
 __device__ __forceinline__ float warp_sum(float v) {
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
 }
-__device__ __forceinline__ float gate_of(float x, int act) { return act == SWLM_GATE_SIGMOID ? sigmoid(x) : silu(x); }
+template <typename T> __device__ __forceinline__ float gate_of(float x, int act) { return act == SWLM_GATE_SIGMOID ? sigmoid<T>(x) : silu<T>(x); }
+// two fp32 numbers in one register pair: a * b + c and a * b on both
+typedef unsigned long long pair_t;
+__device__ __forceinline__ pair_t pair_of(float lo, float hi) { return (pair_t)__float_as_uint(lo) | ((pair_t)__float_as_uint(hi) << 32); }
+__device__ __forceinline__ float pair_lo(pair_t v) { return __uint_as_float((unsigned)v); }
+__device__ __forceinline__ float pair_hi(pair_t v) { return __uint_as_float((unsigned)(v >> 32)); }
+__device__ __forceinline__ pair_t pair_fma(pair_t a, pair_t b, pair_t c) {
+    pair_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ pair_t pair_mul(pair_t a, pair_t b) {
+    pair_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 
 __device__ __forceinline__ RowRun run_of(const DeltaParams& p, int i) {
     if (p.runs) return p.runs[i];
@@ -89,11 +120,12 @@ __device__ __forceinline__ float conv_silu(const DeltaParams& p, const RowRun& r
     const __nv_bfloat16* w = taps_of(p, ch);
     float acc = 0.f;
     for (int j = 0; j < p.sh.taps; ++j) acc = fmaf(__bfloat162float(w[j]), conv_input<T>(p, run, ch, i - (p.sh.taps - 1) + j), acc);
-    return silu(acc);
+    return silu<T>(acc);
 }
+template <typename T>
 __device__ __forceinline__ float decay_of(const DeltaParams& p, int row, int h, int d, float rate) {
     const int i = p.decay_dim == 1 ? h : h * p.decay_dim + d;
-    return expf(-rate * softplus(p.decay[(size_t)row * p.decay_stride + i] + __bfloat162float(p.dt_bias[i])));
+    return Fn<T>::exp(-rate * softplus<T>(p.decay[(size_t)row * p.decay_stride + i] + __bfloat162float(p.dt_bias[i])));
 }
 
 // ---- portions: what a block needs of its tokens -----------------------------------------------------------------------
@@ -132,22 +164,27 @@ __device__ __forceinline__ void conv_block(const DeltaParams& p, const RowRun& r
         float acc = 0.f;
 #pragma unroll
         for (int j = kPrepTaps - 1; j >= 0; --j) acc = fmaf(wf[j], x[t + kPrepTaps - 1 - j], acc);
-        y[t] = t < nt ? silu(acc) : 0.f;
+        y[t] = t < nt ? silu<T>(acc) : 0.f;
     }
 }
 
-// Sums over the warp of 32 values a lane, value `lane` left in this lane: at every step half of the values go to the partner.
-__device__ __forceinline__ float warp_sums(float (&v)[32], int lane) {
+// Sums over the warp of N values a lane (N a power of two up to 32); value lane * N / 32 is left in this lane. At every step half
+// of the values go to the partner.
+template <int N>
+__device__ __forceinline__ float warp_sums(float (&v)[N], int lane) {
+    int o = 16;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
+    for (int n = N / 2; n > 0; n >>= 1, o >>= 1) {
         const bool upper = lane & o;
 #pragma unroll
-        for (int j = 0; j < o; ++j) {
-            const float give = upper ? v[j] : v[j + o], keep = upper ? v[j + o] : v[j];
+        for (int j = 0; j < n; ++j) {
+            const float give = upper ? v[j] : v[j + n], keep = upper ? v[j + n] : v[j];
             v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
     }
-    return v[0];
+    float r = v[0];
+    for (; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+    return r;
 }
 
 template <typename T>
@@ -165,8 +202,8 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Delta
     float* k = q + TB * dim;         // [TB][dim]
     if (tid < TB) {
         const int row = run.row0 + t0 + tid;
-        beta_s[tid] = tid < nt ? sigmoid(p.beta[(size_t)row * p.beta_stride + h]) : 0.f;
-        if (p.decay_dim == 1) decay_s[tid] = tid < nt ? decay_of(p, row, h, 0, rate) : 1.f;
+        beta_s[tid] = tid < nt ? sigmoid<T>(p.beta[(size_t)row * p.beta_stride + h]) : 0.f;
+        if (p.decay_dim == 1) decay_s[tid] = tid < nt ? decay_of<T>(p, row, h, 0, rate) : 1.f;
     }
     for (int i = tid; i < 2 * dim; i += kPrepThreads) {
         const int d = i < dim ? i : i - dim, ch = (i < dim ? 0 : gk) + grp * dim + d;
@@ -203,7 +240,7 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Delta
             const bool live = d < dim && t < nt;
             kv[t] = live ? k[t * dim + d] * norm_s[TB + t] : 0.f;
             qv[t] = live ? q[t * dim + d] * norm_s[t] : 0.f;
-            g[t] = !live ? 1.f : p.decay_dim == 1 ? decay_s[t] : decay_of(p, run.row0 + t0 + t, h, d, rate);
+            g[t] = !live ? 1.f : p.decay_dim == 1 ? decay_s[t] : decay_of<T>(p, run.row0 + t0 + t, h, d, rate);
         }
         float gt = 1.f;
 #pragma unroll
@@ -260,17 +297,19 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Delta
 }
 
 // ---- portions: the recurrence -----------------------------------------------------------------------------------------
-// CTA (16 columns of the state, head, run): a warp holds four columns, a lane key channels 4 lane + 128 i + (0 .. 3) of them, so
-// that a record row is read once per four columns. The 32 products of a block with the state (w and o of four tokens and four
-// columns) are summed across the warp in 31 exchanges that leave one in each lane. Records come through a ring of bulk copies.
+// CTA (16 columns of the state, head, run): a warp holds two columns, a lane key channels 4 lane + 128 i + (0 .. 3) of them, so
+// that a record row is read once per two columns. The 16 products of a block with the state (w and o of four tokens and two
+// columns) are summed across the warp in 16 exchanges that leave one in each pair of lanes. Records come through a ring of bulk copies.
 // At the end the run's last inputs go to the convolution ring (all readers of the old ones have finished).
 // Launched without overlap: CTAs that move in while another kernel drains would crowd together on the SMs that drain first.
 template <typename T, int R>
 __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaParams p) {
     constexpr int DP = R * 32, REC = (3 * TB + 1) * DP + 2 * TB * TB, VREC = TB * kScanCols, STAGE = REC + VREC, WC = kScanWarpCols;
+    constexpr int kScanStages = scan_stages(R);
     extern __shared__ __align__(128) float scan_smem[];
     __shared__ __align__(8) unsigned long long full_bar[kScanStages];
     __shared__ __align__(16) float u_s[kScanThreads / 32][TB * WC];
+    static_assert(WC == 2, "lane = 16 * (0: w, 1: o) + 4 * token + 2 * column + copy");
     __shared__ int bad;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int vb = blockIdx.x, h = blockIdx.y, col0 = vb * kScanCols + warp * WC;
@@ -295,36 +334,39 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     if (tid == 0) for (; issued < min(kScanStages, nb); ++issued) request(issued);
     float* st = p.state + ((size_t)run.seq * p.sh.heads + h) * p.sh.dim * p.sh.vdim + col0;
     auto channel = [&](int i) { return lane * 4 + 128 * (i >> 2) + (i & 3); };
-    float S[WC][R];
+    pair_t S[WC][R / 2];
+    auto load = [&](int i, int c) { return run.pos0 > 0 && channel(i) < p.sh.dim && col0 + c < p.sh.vdim ? st[(size_t)channel(i) * p.sh.vdim + c] : 0.f; };
 #pragma unroll
-    for (int i = 0; i < R; ++i)
+    for (int i = 0; i < R; i += 2)
 #pragma unroll
-        for (int c = 0; c < WC; ++c) S[c][i] = run.pos0 > 0 && channel(i) < p.sh.dim && col0 + c < p.sh.vdim ? st[(size_t)channel(i) * p.sh.vdim + c] : 0.f;
-    // after the sums lane = 16 * (0: w, 1: o) + 4 * token + column
-    const int tok = (lane >> 2) & 3, oc = col0 + (lane & 3);
+        for (int c = 0; c < WC; ++c) S[c][i / 2] = pair_of(load(i, c), load(i + 1, c));
+    // after the sums lane = 16 * (0: w, 1: o) + 4 * token + 2 * column + copy
+    const int tok = (lane >> 2) & 3, lc = (lane >> 1) & 1, oc = col0 + lc;
     float* o_at = p.o + ((size_t)(run.row0 + tok) * p.sh.heads + h) * p.sh.vdim + oc;
     const size_t o_step = (size_t)TB * p.sh.heads * p.sh.vdim;
     for (int b = 0; b < nb; ++b) {
         const int s = b % kScanStages;
         if (!mbar_wait(&full_bar[s], (unsigned)((b / kScanStages) & 1))) { atomicExch(p.status, 51); bad = 1; }
         const float* rec = scan_smem + (size_t)s * STAGE;
-        const float4* r4 = reinterpret_cast<const float4*>(rec) + lane;
+        const ulonglong2* r2 = reinterpret_cast<const ulonglong2*>(rec) + lane;
         const float4 coef = *reinterpret_cast<const float4*>(rec + (3 * TB + 1) * DP + (lane >> 2) * TB);
-        const float vv = rec[REC + tok * kScanCols + warp * WC + (lane & 3)];
-        float x[2 * TB * WC];
-#pragma unroll
-        for (int i = 0; i < 2 * TB * WC; ++i) x[i] = 0.f;
+        const float vv = rec[REC + tok * kScanCols + warp * WC + lc];
+        pair_t acc[2 * TB * WC];
 #pragma unroll
         for (int i = 0; i < R / 4; ++i)
 #pragma unroll
             for (int t = 0; t < 2 * TB; ++t) {
-                const float4 y = r4[(t * DP + 128 * i) / 4];
+                const ulonglong2 y = r2[(t * DP + 128 * i) / 4];
 #pragma unroll
                 for (int c = 0; c < WC; ++c) {
-                    float& acc = x[t * WC + c];
-                    acc = fmaf(S[c][4 * i], y.x, acc); acc = fmaf(S[c][4 * i + 1], y.y, acc); acc = fmaf(S[c][4 * i + 2], y.z, acc); acc = fmaf(S[c][4 * i + 3], y.w, acc);
+                    pair_t& a = acc[t * WC + c];
+                    a = i == 0 ? pair_mul(S[c][0], y.x) : pair_fma(S[c][2 * i], y.x, a);
+                    a = pair_fma(S[c][2 * i + 1], y.y, a);
                 }
             }
+        float x[2 * TB * WC];
+#pragma unroll
+        for (int i = 0; i < 2 * TB * WC; ++i) x[i] = pair_lo(acc[i]) + pair_hi(acc[i]);
         const float sum = warp_sums(x, lane);
         const float w = vv - sum;                            // (of lanes 0 .. 15)
         float r = lane < 16 ? 0.f : sum;
@@ -332,25 +374,30 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
         r = fmaf(coef.y, __shfl_sync(0xffffffffu, w, 4 + (lane & 3)), r);
         r = fmaf(coef.z, __shfl_sync(0xffffffffu, w, 8 + (lane & 3)), r);
         r = fmaf(coef.w, __shfl_sync(0xffffffffu, w, 12 + (lane & 3)), r);
-        if (lane < 16) u_s[warp][lane] = r;
-        else if (oc < p.sh.vdim && b * TB + tok < run.count) o_at[b * o_step] = r;
+        if (!(lane & 1)) {
+            if (lane < 16) u_s[warp][lane >> 1] = r;
+            else if (oc < p.sh.vdim && b * TB + tok < run.count) o_at[b * o_step] = r;
+        }
         __syncwarp();
-        float4 u[TB];
+        float u[TB * WC];
 #pragma unroll
-        for (int t = 0; t < TB; ++t) u[t] = *reinterpret_cast<const float4*>(&u_s[warp][t * WC]);
+        for (int t = 0; t < TB * WC; t += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(&u_s[warp][t]);
+            u[t] = v.x; u[t + 1] = v.y; u[t + 2] = v.z; u[t + 3] = v.w;
+        }
 #pragma unroll
         for (int i = 0; i < R / 4; ++i) {
-            const float4 g = r4[(3 * TB * DP + 128 * i) / 4];
+            const ulonglong2 g = r2[(3 * TB * DP + 128 * i) / 4];
 #pragma unroll
-            for (int c = 0; c < WC; ++c) { S[c][4 * i] *= g.x; S[c][4 * i + 1] *= g.y; S[c][4 * i + 2] *= g.z; S[c][4 * i + 3] *= g.w; }
+            for (int c = 0; c < WC; ++c) { S[c][2 * i] = pair_mul(S[c][2 * i], g.x); S[c][2 * i + 1] = pair_mul(S[c][2 * i + 1], g.y); }
 #pragma unroll
             for (int t = 0; t < TB; ++t) {
-                const float4 kt = r4[((2 * TB + t) * DP + 128 * i) / 4];
-                const float uc[WC] = {u[t].x, u[t].y, u[t].z, u[t].w};
+                const ulonglong2 kt = r2[((2 * TB + t) * DP + 128 * i) / 4];
 #pragma unroll
                 for (int c = 0; c < WC; ++c) {
-                    S[c][4 * i] = fmaf(kt.x, uc[c], S[c][4 * i]); S[c][4 * i + 1] = fmaf(kt.y, uc[c], S[c][4 * i + 1]);
-                    S[c][4 * i + 2] = fmaf(kt.z, uc[c], S[c][4 * i + 2]); S[c][4 * i + 3] = fmaf(kt.w, uc[c], S[c][4 * i + 3]);
+                    const pair_t uu = pair_of(u[t * WC + c], u[t * WC + c]);
+                    S[c][2 * i] = pair_fma(kt.x, uu, S[c][2 * i]);
+                    S[c][2 * i + 1] = pair_fma(kt.y, uu, S[c][2 * i + 1]);
                 }
             }
         }
@@ -366,7 +413,7 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     for (int i = 0; i < R; ++i)
 #pragma unroll
         for (int c = 0; c < WC; ++c)
-            if (channel(i) < p.sh.dim && col0 + c < p.sh.vdim) st[(size_t)channel(i) * p.sh.vdim + c] = S[c][i];
+            if (channel(i) < p.sh.dim && col0 + c < p.sh.vdim) st[(size_t)channel(i) * p.sh.vdim + c] = i & 1 ? pair_hi(S[c][i / 2]) : pair_lo(S[c][i / 2]);
     if (vb == 0) {
         const int share = p.sh.heads / p.sh.groups, gk = p.sh.groups * p.sh.dim, ch_all = p.sh.channels();
         const int n_qk = h % share == 0 ? p.sh.dim : 0, grp = h / share;
@@ -399,7 +446,7 @@ __global__ void __launch_bounds__(TB * 32) delta_gate_kernel(const DeltaParams p
     const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + p.eps);
     const T* gate = static_cast<const T*>(p.gate) + (size_t)row * p.gate_stride + (size_t)h * vdim;
     T* out = static_cast<T*>(p.out) + (size_t)row * p.out_stride + (size_t)h * vdim;
-    for (int c = lane; c < vdim; c += 32) dl_put(out + c, o[c] * sc * __bfloat162float(p.norm_w[c]) * gate_of(dl_get(gate + c), p.gate_act));
+    for (int c = lane; c < vdim; c += 32) dl_put(out + c, o[c] * sc * __bfloat162float(p.norm_w[c]) * gate_of<T>(dl_get(gate + c), p.gate_act));
 }
 
 // ---- single tokens ----------------------------------------------------------------------------------------------------
@@ -407,7 +454,7 @@ __global__ void __launch_bounds__(TB * 32) delta_gate_kernel(const DeltaParams p
 // column. Nothing of this layer's state is touched by the kernels in front of this one, so it is read ahead of them. The slot
 // of the convolution ring that is written (position % taps) is none of those that are read.
 template <typename T, int R>
-__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(kStepThreads, R <= 16 ? 3 : 2) delta_step_kernel(const DeltaParams p) {
     extern __shared__ __align__(16) float step_smem[];
     __shared__ float part_a[kStepWarps][kStepCols], part_b[kStepWarps][kStepCols], scal[4], v_s[kStepCols], ssq[kStepCluster];
     const cg::cluster_group cluster = cg::this_cluster();
@@ -458,7 +505,7 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
         float y = 0.f;
         if (chan[j] >= 0) {
             const T x = static_cast<const T*>(p.qkv)[(size_t)row * p.qkv_stride + chan[j]];
-            y = silu(fmaf(w_last[j], dl_get(&x), acc[j]));
+            y = silu<T>(fmaf(w_last[j], dl_get(&x), acc[j]));
             if (i >= 2 * dim || keeps_qk) const_cast<T*>(ring)[(size_t)(pos % taps) * ch_all + chan[j]] = x;
         }
         if (i < dim) q[i] = y;
@@ -466,13 +513,13 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
         else if (i < 2 * dim + kStepCols) v_s[i - 2 * dim] = y;
     }
     if (p.decay_dim == 1) {
-        const float one = decay_of(p, row, h, 0, rate);
+        const float one = decay_of<T>(p, row, h, 0, rate);
         for (int d = tid; d < dim; d += kStepThreads) g[d] = one;
     } else {
-        for (int d = tid; d < dim; d += kStepThreads) g[d] = decay_of(p, row, h, d, rate);
+        for (int d = tid; d < dim; d += kStepThreads) g[d] = decay_of<T>(p, row, h, d, rate);
     }
-    const float gate = live && warp == 0 ? gate_of(dl_get(static_cast<const T*>(p.gate) + (size_t)row * p.gate_stride + (size_t)h * vdim + col), p.gate_act) : 0.f;
-    const float beta = sigmoid(p.beta[(size_t)row * p.beta_stride + h]);
+    const float gate = live && warp == 0 ? gate_of<T>(dl_get(static_cast<const T*>(p.gate) + (size_t)row * p.gate_stride + (size_t)h * vdim + col), p.gate_act) : 0.f;
+    const float beta = sigmoid<T>(p.beta[(size_t)row * p.beta_stride + h]);
     __syncthreads();
     if (warp < 3) {
         const float* x = warp == 1 ? k : q;
@@ -525,7 +572,7 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
 int scan_regs(int dim) { return dim <= 128 ? 4 : dim <= 256 ? 8 : dim <= 512 ? 16 : 0; }   // key channels per lane
 int rec_floats(int dim) { return (3 * TB + 1) * scan_regs(dim) * 32 + 2 * TB * TB; }
 int scan_vblocks(int vdim) { return (vdim + kScanCols - 1) / kScanCols; }
-size_t scan_smem_bytes(int dim) { return (size_t)kScanStages * (rec_floats(dim) + TB * kScanCols) * 4; }
+size_t scan_smem_bytes(int dim) { return (size_t)scan_stages(scan_regs(dim)) * (rec_floats(dim) + TB * kScanCols) * 4; }
 
 template <typename T, int R>
 int scan_launch(const DeltaParams& p, int runs, cudaStream_t s) {

@@ -141,37 +141,61 @@ __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedPar
     }
 }
 
-// CTA (share of the outputs, row): mid rows of all chosen experts, weighted, in shared memory; a warp per output.
+// CTA (share of the outputs, row): mid rows of all chosen experts, weighted, in shared memory; two warps per output, each with
+// half of the 16-byte chunks of the chosen experts' rows.
+constexpr int kDownUnroll = 8, kDownWarps = 2;
 template <typename T>
 __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedParams p) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) float rt_smem[];   // [top][mid_ld]
+    __shared__ float part[kRtWarps];
+    __shared__ int sel[kMaxTop];
+    __shared__ float weight[kMaxTop];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, top = p.sh.top;
-    const int* sel = p.sel + row * top;
+    if (tid < top) { sel[tid] = p.sel[row * top + tid]; weight[tid] = p.weight[row * top + tid]; }
+    __syncthreads();
+    const int chunks = p.mid_ld >> 3, all = chunks * top, half = warp % kDownWarps;
+    uint4 v[kDownUnroll];
+    auto load = [&](int n, int c0) {
+        int t = c0 / chunks, c = c0 - t * chunks;
+#pragma unroll
+        for (int j = 0; j < kDownUnroll; ++j) {
+            v[j] = t < top && n < p.sh.width ? rt_stream(p.down + ((size_t)sel[t] * p.sh.width + n) * p.mid_ld + 8 * c) : make_uint4(0, 0, 0, 0);
+            c += 32 * kDownWarps;
+            while (c >= chunks) { c -= chunks; ++t; }
+        }
+    };
+    const int first = half * 32 + lane;
+    int n = (blockIdx.x * kRtWarps + warp) / kDownWarps;
+    load(n, first);   // the first weights are on their way while the activations are gathered
     for (int t = 0; t < top; ++t) {
         const T* mid = static_cast<const T*>(p.mid) + (size_t)(row * top + t) * p.mid_stride;
-        const float w = p.weight[row * top + t];
+        const float w = weight[t];
         for (int i = tid; i < p.mid_ld; i += kRtThreads) rt_smem[t * p.mid_ld + i] = i < p.sh.ff ? rt_get(mid + i) * w : 0.f;
     }
     __syncthreads();
-    const int chunks = p.mid_ld >> 3, all = chunks * top;
-    constexpr int U = 8;
-    for (int n = blockIdx.x * kRtWarps + warp; n < p.sh.width; n += gridDim.x * kRtWarps) {
+    const int step = gridDim.x * kRtWarps / kDownWarps, rounds = (p.sh.width + step - 1) / step;
+    for (int it = 0; it < rounds; ++it, n += step) {
         float acc = 0.f;
-        for (int c0 = lane; c0 < all; c0 += 32 * U) {
-            uint4 v[U];
+        for (int c0 = first; c0 < all; c0 += 32 * kDownWarps * kDownUnroll) {
+            if (it > 0 || c0 != first) load(n, c0);
 #pragma unroll
-            for (int j = 0; j < U; ++j) {
-                const int i = c0 + 32 * j, t = i / chunks, c = i - t * chunks;
-                v[j] = i < all ? rt_stream(p.down + ((size_t)sel[t] * p.sh.width + n) * p.mid_ld + 8 * c) : make_uint4(0, 0, 0, 0);
+            for (int j = 0; j < kDownUnroll; ++j) {
+                const int i = c0 + 32 * kDownWarps * j;
+                if (i < all) acc = rt_dot8(v[j], rt_smem + 8 * i, acc);
             }
-#pragma unroll
-            for (int j = 0; j < U; ++j)
-                if (c0 + 32 * j < all) acc = rt_dot8(v[j], rt_smem + 8 * (c0 + 32 * j), acc);
         }
         for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-        if (lane == 0) p.out[(size_t)row * p.out_stride + n] = acc;
+        if (lane == 0) part[warp] = acc;
+        __syncthreads();
+        if (lane == 0 && half == 0 && n < p.sh.width) {
+            float total = 0.f;
+#pragma unroll
+            for (int w = 0; w < kDownWarps; ++w) total += part[warp + w];
+            p.out[(size_t)row * p.out_stride + n] = total;
+        }
+        __syncthreads();
     }
 }
 
@@ -294,7 +318,7 @@ int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
     const int pairs = (p.sh.ff + kRtWarps - 1) / kRtWarps, gx = std::max(1, std::min(pairs, (4 * 148 + p.sh.top * p.m - 1) / (p.sh.top * p.m)));
     cudaError_t e = launch_k(routed_gate_kernel<T>, dim3(gx, p.sh.top, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed gate launch");
-    const int outs = (p.sh.width + kRtWarps - 1) / kRtWarps, dx = std::max(1, std::min(outs, (3 * 148 + p.m - 1) / p.m));
+    const int outs = (p.sh.width * kDownWarps + kRtWarps - 1) / kRtWarps, dx = std::max(1, std::min(outs, (4 * 148 + p.m - 1) / p.m));
     e = launch_k(routed_down_kernel<T>, dim3(dx, p.m), dim3(kRtThreads), down_smem(p.sh), s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed down launch");
     *launches += 2;
