@@ -30,7 +30,7 @@ namespace swlm {
 namespace {
 
 constexpr int TB = kDeltaBlock;
-constexpr int kScanCols = 16, kScanWarpCols = 2, kScanThreads = kScanCols / kScanWarpCols * 32;
+constexpr int kScanCols = 16, kScanWarpCols = 2, kScanWarps = kScanCols / kScanWarpCols, kScanThreads = (kScanWarps + 1) * 32;   // the last warp requests the records
 constexpr int kStepCols = 32, kStepWarps = 8, kStepThreads = kStepWarps * 32, kStepCluster = 8;
 constexpr int kPrepThreads = 128;
 
@@ -307,31 +307,39 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     constexpr int DP = R * 32, REC = (3 * TB + 1) * DP + 2 * TB * TB, VREC = TB * kScanCols, STAGE = REC + VREC, WC = kScanWarpCols;
     constexpr int kScanStages = scan_stages(R);
     extern __shared__ __align__(128) float scan_smem[];
-    __shared__ __align__(8) unsigned long long full_bar[kScanStages];
-    __shared__ __align__(16) float u_s[kScanThreads / 32][TB * WC];
+    __shared__ __align__(8) unsigned long long full_bar[kScanStages], empty_bar[kScanStages];
+    __shared__ __align__(16) float u_s[kScanWarps][TB * WC];
     static_assert(WC == 2, "lane = 16 * (0: w, 1: o) + 4 * token + 2 * column + copy");
-    __shared__ int bad;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int vb = blockIdx.x, h = blockIdx.y, col0 = vb * kScanCols + warp * WC;
     if (tid == 0) {
-        for (int s = 0; s < kScanStages; ++s) mbar_init(&full_bar[s], 1);
-        bad = 0;
+        for (int s = 0; s < kScanStages; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], kScanWarps); }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
     pdl_wait();
     const RowRun run = run_of(p, blockIdx.z);
     const int nb = (run.count + TB - 1) / TB;
-    auto request = [&](int b) {   // thread 0
-        const int s = b % kScanStages;
+    auto request = [&](int b, int s) {
         const unsigned bar = smem_u32(&full_bar[s]), dst = smem_u32(scan_smem + (size_t)s * STAGE);
         const size_t at = (size_t)(run.blk0 + b) * p.sh.heads + h;
         mbar_expect(bar, STAGE * 4);
         bulk_load(dst, p.rec + at * REC, REC * 4, bar);
         bulk_load(dst + REC * 4, p.vrec + (at * p.vblocks + vb) * VREC, VREC * 4, bar);
     };
-    int issued = 0;
-    if (tid == 0) for (; issued < min(kScanStages, nb); ++issued) request(issued);
+    if (warp == kScanWarps) {
+        if (lane == 0) {
+            int b = 0;
+            for (int s = 0, round = 0; b < nb; ++b) {
+                if (round > 0 && !mbar_wait(&empty_bar[s], (unsigned)((round - 1) & 1))) { atomicExch(p.status, 52); break; }
+                request(b, s);
+                if (++s == kScanStages) { s = 0; ++round; }
+            }
+            // leave only when the copies that may still be under way have landed (bounded)
+            for (int q = max(0, b - kScanStages); q < b; ++q) mbar_wait(&full_bar[q % kScanStages], (unsigned)((q / kScanStages) & 1));
+        }
+        return;
+    }
     float* st = p.state + ((size_t)run.seq * p.sh.heads + h) * p.sh.dim * p.sh.vdim + col0;
     auto channel = [&](int i) { return lane * 4 + 128 * (i >> 2) + (i & 3); };
     pair_t S[WC][R / 2];
@@ -344,9 +352,8 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     const int tok = (lane >> 2) & 3, lc = (lane >> 1) & 1, oc = col0 + lc;
     float* o_at = p.o + ((size_t)(run.row0 + tok) * p.sh.heads + h) * p.sh.vdim + oc;
     const size_t o_step = (size_t)TB * p.sh.heads * p.sh.vdim;
-    for (int b = 0; b < nb; ++b) {
-        const int s = b % kScanStages;
-        if (!mbar_wait(&full_bar[s], (unsigned)((b / kScanStages) & 1))) { atomicExch(p.status, 51); bad = 1; }
+    for (int b = 0, s = 0, round = 0; b < nb; ++b) {
+        if (!mbar_wait(&full_bar[s], (unsigned)(round & 1))) { atomicExch(p.status, 51); return; }   // (uniform; the requesting warp sees the copies out)
         const float* rec = scan_smem + (size_t)s * STAGE;
         const ulonglong2* r2 = reinterpret_cast<const ulonglong2*>(rec) + lane;
         const float4 coef = *reinterpret_cast<const float4*>(rec + (3 * TB + 1) * DP + (lane >> 2) * TB);
@@ -401,13 +408,9 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
                 }
             }
         }
-        __syncthreads();   // the stage is free
-        if (bad) break;    // uniform: written before the barrier by whoever gave up
-        if (tid == 0 && issued < nb) { request(issued); ++issued; }
-    }
-    if (bad) {   // leave only when the copies that may still be under way have landed (bounded)
-        if (tid == 0) for (int b = max(0, issued - kScanStages); b < issued; ++b) mbar_wait(&full_bar[b % kScanStages], (unsigned)((b / kScanStages) & 1));
-        return;
+        __syncwarp();
+        if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&empty_bar[s])) : "memory");   // the stage is free
+        if (++s == kScanStages) { s = 0; ++round; }
     }
 #pragma unroll
     for (int i = 0; i < R; ++i)
@@ -421,7 +424,7 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
             const int tok = run.count - 1 - back, slot = (run.pos0 + tok) % p.sh.taps;
             const T* src = static_cast<const T*>(p.qkv) + (size_t)(run.row0 + tok) * p.qkv_stride;
             T* dst = static_cast<T*>(p.ring) + ((size_t)run.seq * p.sh.taps + slot) * ch_all;
-            for (int i = tid; i < p.sh.vdim + 2 * n_qk; i += kScanThreads) {
+            for (int i = tid; i < p.sh.vdim + 2 * n_qk; i += kScanWarps * 32) {
                 const int ch = i < p.sh.vdim ? 2 * gk + h * p.sh.vdim + i : i < p.sh.vdim + n_qk ? grp * p.sh.dim + i - p.sh.vdim : gk + grp * p.sh.dim + i - p.sh.vdim - n_qk;
                 dst[ch] = src[ch];
             }
