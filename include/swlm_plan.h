@@ -106,7 +106,7 @@ enum {
        plain key is weight2 [heads * head_dim][n] c, the value weight3 [heads * value_dim][n] c; score = (q . k over both
        parts) * scale, softmax over all positions up to the token's own; out = sigmoid(gate) * value sum.
        window_left > 0: only the last window_left positions, the token's own among them. weight4 not empty: a sink, one
-       number per head whose exponential joins the softmax's denominator (no key, no value, not scaled). */
+       number per head whose exponential is added to the softmax's denominator as it is. */
     SWLM_STEP_LATENT_ATTN = 16,
     /* Gated activation with limits: g = min(in, limit), u = clamp(in2, -limit, limit),
        out = g * sigmoid(scale * g) * (u + 1). */
