@@ -91,10 +91,13 @@ enum {
     SWLM_STEP_SSM_RECURRENCE = 12,
     /* ---- steps of fp32-stream plans (swlm_buffers_desc.stream_dtype != 0); no counterpart in the reference ----
        Such plans also use EMBED (times `scale` when it is not 0), the three norm steps, SWIGLU / GEGLU and ARGMAX. */
-    /* out[n] = sum_k W[n][k] in[k], W a dense bf16 matrix (swlm_weights_add_matrix_bf16), fp32 accumulation. */
+    /* out[n] = sum_k W[n][k] in[k], W a dense bf16 matrix (swlm_weights_add_matrix_bf16), fp32 accumulation.
+       weight2 not empty: a second matrix [n][k2] times the k2 columns that start at the next multiple of 8 behind the first
+       k ones is added (the two are kept side by side and run as one product). */
     SWLM_STEP_PRODUCT = 13,
     /* Sandwich norm: t = in * rsqrt(mean(in^2)+eps) * (weight + weight_bias); residual += t;
-       out = residual * rsqrt(mean(residual^2)+eps) * (weight2 + weight_bias). */
+       out = residual * rsqrt(mean(residual^2)+eps) * (weight2 + weight_bias).
+       weight3 not empty: an embedding table; the row of the token times `scale` is added to the residual with t. */
     SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM = 14,
     /* the same in front of the output head: the sum is not stored */
     SWLM_STEP_POSTNORM_RESADD_RMSNORM = 15,
@@ -102,7 +105,7 @@ enum {
        in2_buf = n latent entries followed by key_dim entries of the key part that all heads share, in3_buf = gate (heads,
        before the sigmoid; SWLM_BUF_NONE: no gate), out_buf = heads * value_dim.
        The latent c is RMS-normed (`weight`, eps, weight_bias); rotate-half rotary positions act on the first rope_dim of
-       the key_dim entries of q and of the shared key part. Cached per token: c and the rotated key part. Per head the
+       the key_dim entries of q and of the shared key part (rope_pairs 1: entries 2i and 2i + 1 form a pair instead). Cached per token: c and the rotated key part. Per head the
        plain key is weight2 [heads * head_dim][n] c, the value weight3 [heads * value_dim][n] c; score = (q . k over both
        parts) * scale, softmax over all positions up to the token's own; out = sigmoid(gate) * value sum.
        window_left > 0: only the last window_left positions, the token's own among them. weight4 not empty: a sink, one
@@ -126,12 +129,34 @@ enum {
        s = sigmoid(logits); the experts form `groups` equal groups of neighbours, a group counts as the sum of its two largest
        s, and only experts of the groups_keep best groups can be chosen; the `top` largest s among them are. Expert i is the
        clamped gated feed-forward (CLAMPED_GLU with glu_alpha, limit) of the matrices <weight>i<weight2>, <weight>i<weight3>
-       [k][n] and <weight>i<weight4> [n][k]; its output is weighted with s / (sum of the chosen s + 1e-20) * scale. */
+       [k][n] and <weight>i<weight4> [n][k]; its output is weighted with s / (sum of the chosen s + 1e-20) * scale.
+       score_act SWLM_SCORE_SOFTMAX: s = softmax(logits) over all experts. group_best 1: a group counts as its largest s.
+       raw_weights 1: an expert's output is weighted with s * scale. weight2 empty: expert i is <weight4>(gelu(<weight3> in))
+       with the exact (erf) GELU. weight5 not empty: a feed-forward weight6 [n][k2] (gelu(weight5 [k2][n] in)) that every
+       token takes, its output times sigmoid(in2[experts]) is added. */
     SWLM_STEP_ROUTED_MLP = 19,
     /* logits = scale * tanh(logits / scale), in place */
-    SWLM_STEP_SOFTCAP = 20
+    SWLM_STEP_SOFTCAP = 20,
+    /* Grouped-query attention over a paged cache. in_buf from column in_off on = q | k | v (heads * head_dim, kv_heads *
+       head_dim, kv_heads * value_dim), in3_buf = gate (heads, before the sigmoid; SWLM_BUF_NONE: none), out_buf from column
+       out_off on = heads * value_dim. Query head h reads key / value head h / (heads / kv_heads).
+       q and k per head: RMS norm with weight / weight2 [head_dim] (eps, weight_bias; empty: none), then rotary positions on
+       the first rope_dim entries (rope_pairs as in LATENT_ATTN). Cached per token: k after that, and v. score = (q . k) *
+       scale, softmax over the positions up to the token's own: window_left > 0: the last window_left of them; chunk > 0:
+       those of the token's own chunk of `chunk` positions, counted from position 0. sink_one 1: one is added to the softmax's
+       denominator. out = sigmoid(gate) * value sum * out_scale. */
+    SWLM_STEP_GROUPED_ATTN = 21,
+    /* Retention with a state per sequence. in_buf from column in_off on = q | k | v (heads * key_dim, the same again, heads *
+       value_dim), in4_buf from column in4_off on = output gate before its SiLU (heads * value_dim), out_buf from column
+       out_off on = heads * value_dim (may not be in_buf or in4_buf).
+       S = decay_h * S + (scale * k) v^T; o = S^T q with S [key_dim][value_dim] fp32, zero at position 0;
+       out = o * rsqrt(mean(o^2) + eps) * silu(gate) * out_scale. weight = decay [heads], an fp32 tensor.
+       `layer` indexes the same states as GATED_DELTA. */
+    SWLM_STEP_RETENTION = 22
 };
 enum { SWLM_GATE_SILU = 0, SWLM_GATE_SIGMOID = 1 };
+enum { SWLM_SCORE_SIGMOID = 0, SWLM_SCORE_SOFTMAX = 1 };
+enum { SWLM_ROPE_HALVES = 0, SWLM_ROPE_NEIGHBOURS = 1 };
 
 typedef struct swlm_step {
     int32_t kind;
@@ -171,7 +196,7 @@ typedef struct swlm_step {
     float   rope_fast;
     float   rope_slow;
     /* fp32-stream plans */
-    int32_t in_off;      /* PRODUCT: first column of the input in in_buf (a multiple of 8) */
+    int32_t in_off;      /* first column of the input in in_buf (a multiple of 8) */
     int32_t out_off;     /* and of the result in out_buf, so that several results share a buffer */
     int32_t experts;
     int32_t top;
@@ -182,6 +207,16 @@ typedef struct swlm_step {
     float   eps2;
     char    weight5[SWLM_NAME_MAX];
     char    weight6[SWLM_NAME_MAX];
+    int32_t rope_pairs;    /* SWLM_ROPE_* */
+    float   rope_divisor;  /* every rotary frequency is divided by it; 0 = 1 */
+    int32_t chunk;
+    int32_t sink_one;
+    int32_t k2;
+    int32_t in4_off;
+    float   out_scale;     /* GROUPED_ATTN, RETENTION */
+    int32_t score_act;     /* SWLM_SCORE_* */
+    int32_t group_best;    /* 0 = 2 */
+    int32_t raw_weights;
 } swlm_step;
 
 /* Sizes of the runtime buffer set; mirrors the inputs of
@@ -230,10 +265,12 @@ typedef struct swlm_buffers_desc {
        0 = the bf16 buffers of the reference. Buffer widths follow from the steps (slot_dim is not used). */
     int32_t stream_dtype;
     int32_t latent_layers;   /* number of latent-attention layers (page pools) */
-    /* tokens the page pool of the latent rows holds over all sequences, rounded up to pages of 64;
+    /* tokens the page pools of the cached rows hold over all sequences, rounded up to pages of 64;
        0 = max_batch * max_seq. Sequences take pages as they grow and give them back when they are reset. */
     int32_t kv_pool_tokens;
-    int32_t delta_layers;    /* number of SWLM_STEP_GATED_DELTA layers: fp32 state and convolution inputs per sequence */
+    int32_t delta_layers;    /* number of SWLM_STEP_GATED_DELTA and SWLM_STEP_RETENTION layers: fp32 state (and convolution
+                                inputs) per sequence */
+    int32_t grouped_layers;  /* number of SWLM_STEP_GROUPED_ATTN layers (page pools of keys and values) */
 } swlm_buffers_desc;
 
 enum { SWLM_STREAM_BF16 = 0, SWLM_STREAM_F32 = 1, SWLM_STREAM_ALL_F32 = 2 };

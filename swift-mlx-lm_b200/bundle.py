@@ -16,6 +16,7 @@ import json
 import os
 from typing import Dict, Optional, Tuple
 
+from . import kalevik as _kalevik
 from . import rirotar as _rirotar
 from . import staf as _staf
 from . import vuzunex as _vuzunex
@@ -31,6 +32,7 @@ LFM2_MODEL_TYPES = ("lfm2",)
 ARCHITECTURES = {
     _vuzunex.ARCHITECTURE: (lambda config, shapes, **runtime: _vuzunex.decode_config(config, **runtime), _vuzunex.VuzunexPlanBuilder),
     _rirotar.ARCHITECTURE: (_rirotar.decode_config, _rirotar.RirotarPlanBuilder),
+    _kalevik.ARCHITECTURE: (_kalevik.decode_config, _kalevik.KalevikPlanBuilder),
 }
 
 # KVCachePolicy of InferencePolicy.default (Sources/MetalCompiler/InferencePolicy.swift:55-100)

@@ -40,6 +40,7 @@ __device__ __forceinline__ ProductRow product_row(const ProductOut& o, int row) 
 __device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
     const ProductRow r = product_row(o, row);
     if (o.softcap > 0.f) val = o.softcap * tanhf(val / o.softcap);
+    if (o.gelu) val = gelu_erf(val);
     if (r.f32) *reinterpret_cast<float*>(r.y + m * r.stride) = val;
     else *reinterpret_cast<__nv_bfloat16*>(r.y + m * r.stride) = __float2bfloat16_rn(val);
 }
@@ -136,6 +137,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
             T* xr = xs + (size_t)m * p.ld;
             const float* in = p.norm.in + (size_t)m * p.norm.in_stride;
             const float* res = p.norm.res_in ? p.norm.res_in + (size_t)m * p.norm.res_stride : nullptr;
+            const __nv_bfloat16* joins = p.norm.table ? p.norm.table_row(m, p.k) : nullptr;
             float h[4][4], rv[4][4];
             float ss = 0.f;
 #pragma unroll
@@ -145,6 +147,11 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
                 const float4 a = i < p.k ? __ldcg(reinterpret_cast<const float4*>(in + i)) : z, b = i < p.k && res ? __ldcg(reinterpret_cast<const float4*>(res + i)) : z;
                 h[j][0] = a.x; h[j][1] = a.y; h[j][2] = a.z; h[j][3] = a.w;
                 rv[j][0] = b.x; rv[j][1] = b.y; rv[j][2] = b.z; rv[j][3] = b.w;
+                if (joins && i < p.k) {
+                    const uint2 v = __ldg(reinterpret_cast<const uint2*>(joins + i));
+                    rv[j][0] += b_lo(v.x) * p.norm.table_scale; rv[j][1] += b_hi(v.x) * p.norm.table_scale;
+                    rv[j][2] += b_lo(v.y) * p.norm.table_scale; rv[j][3] += b_hi(v.y) * p.norm.table_scale;
+                }
             }
             if (p.norm.w_post) {
 #pragma unroll
@@ -187,6 +194,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
             float* rowf = reinterpret_cast<float*>(gemv_raw + (size_t)MR * p.ld * sizeof(T));
             const float* in = p.norm.in + (size_t)m * p.norm.in_stride;
             const float* res = p.norm.res_in ? p.norm.res_in + (size_t)m * p.norm.res_stride : nullptr;
+            const __nv_bfloat16* joins = p.norm.table ? p.norm.table_row(m, p.k) : nullptr;
             float post_scale = 1.f;
             float ss = 0.f;
             for (int i = tid; i < p.k; i += kGemvThreads) { const float v = in[i]; rowf[i] = v; ss = fmaf(v, v, ss); }
@@ -196,6 +204,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
                 float h = rowf[i];
                 if (p.norm.w_post) h = h * post_scale * (__bfloat162float(p.norm.w_post[i]) + p.norm.weight_bias);
                 if (res) h += res[i];
+                if (joins) h += __bfloat162float(joins[i]) * p.norm.table_scale;
                 if (p.norm.res_out && blockIdx.x == 0) p.norm.res_out[(size_t)m * p.norm.res_stride + i] = h;
                 rowf[i] = h;
                 ss = fmaf(h, h, ss);
@@ -454,6 +463,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
                             float val = __uint_as_float(v[i]);
                             if (GATED && !cut) val = gated_activation(val, __uint_as_float(u[i]), p.act);
                             if (p.out.softcap > 0.f && !cut) val = p.out.softcap * tanhf(val / p.out.softcap);
+                            if (p.out.gelu && !cut) val = gelu_erf(val);
                             if (i < count) {
                                 if (dst.f32) *reinterpret_cast<float*>(y) = val;
                                 else *reinterpret_cast<__nv_bfloat16*>(y) = __float2bfloat16_rn(val);

@@ -1,0 +1,591 @@
+// Grouped-query attention of fp32-stream plans over a paged cache: norm of q and k per head, rotary positions, a softmax over the
+// positions a window or a chunk lets through with an optional constant in the denominator, and a gate per head.
+//
+// A page holds 64 tokens of every key / value head: per head 64 key rows, then 64 value rows, so that the keys and values of a
+// (page, head) pair are one contiguous piece of memory. grouped_append_kernel norms and rotates q in place and k and v into the
+// cache; then a batch's rows go one of two ways:
+//   * one by one (decode steps, short portions): grouped_decode_kernel, a cluster of CTAs per (row, key / value head) that deal the
+//     context out to their warps; every warp copies its keys and values by itself and keeps its own running softmax, the
+//     results are merged through shared memory and then through distributed shared memory.
+//   * in spans (prompt portions): grouped_prefill_kernel, a tiled attention of 128 queries by 64 keys.
+// Both multiply on tensor cores with fp32 sums; softmax weights enter as bf16 hi + lo pairs. grouped_simple_kernel (fp32 FMAs)
+// serves fp32 caches and head sizes beyond the others. The newest rows are read back from the cache like all others, so a row's
+// result does not depend on how a sequence was cut into batches.
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
+#include "swlm_internal.h"
+#include "tc_device.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace swlm {
+namespace {
+
+constexpr int kPage = SWLM_PAGE_TOKENS;
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float ga_get(const float* p) { return *p; }
+__device__ __forceinline__ float ga_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void ga_put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void ga_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ unsigned ga_pack(float a, float b) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const unsigned*>(&v);
+}
+__device__ __forceinline__ float ga_round(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
+__device__ __forceinline__ void ga_mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ga_ldsm(unsigned (&r)[4], unsigned addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ga_ldsm_trans(unsigned (&r)[4], unsigned addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+
+struct GroupedParams {
+    GroupedRow row;
+    int heads, share, rot_dims, rot_neighbours, window, chunk, sink_one;
+    float scale_log2, eps, weight_bias, magnitude, out_scale;
+    const float* inv_freq;
+    const __nv_bfloat16 *q_norm, *k_norm;
+    void* qkv; int qkv_stride;
+    const float* gate; int gate_stride;
+    void* pool;
+    const int32_t* page_table; int pages_per_seq;
+    const int32_t* row_seq; const int32_t* row_pos;
+    void* out; int out_stride;
+    int n_rows; const int32_t* rows;     // the rows of this launch; null: 0 .. n_rows - 1
+    const LatentSpan* spans; const int2* tiles;
+    int* status;
+};
+
+// first position a row at `pos` sees; never falls as pos grows
+__device__ __forceinline__ int ga_first_seen(const GroupedParams& p, int pos) {
+    const int w = p.window > 0 ? max(0, pos - p.window + 1) : 0, c = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+    return max(w, c);
+}
+__device__ __forceinline__ int ga_row(const GroupedParams& p, int i) { return p.rows ? p.rows[i] : i; }
+// keys of head g in the page of a position; its values lie kPage * pk entries behind
+template <typename T>
+__device__ __forceinline__ T* ga_block(const GroupedParams& p, int seq, int page_index, int g) {
+    const int page = p.page_table[(size_t)seq * p.pages_per_seq + page_index];
+    return static_cast<T*>(p.pool) + ((size_t)page * p.row.groups + g) * p.row.block;
+}
+__device__ __forceinline__ float ga_gate(const GroupedParams& p, int r, int h) {
+    return (p.gate ? 1.0f / (1.0f + expf(-p.gate[(size_t)r * p.gate_stride + h])) : 1.0f) * p.out_scale;
+}
+
+// ---- norm, rotation, append -------------------------------------------------------------------------------------------
+// CTA (row, eight vectors of the row): a warp per query, key or value vector.
+constexpr int kAppWarps = 8;
+template <typename T>
+__global__ void __launch_bounds__(kAppWarps * 32) grouped_append_kernel(const GroupedParams p) {
+    extern __shared__ __align__(16) float app_smem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, r = blockIdx.x, i = blockIdx.y * kAppWarps + warp;
+    const int G = p.row.groups, dim = p.row.dim, vdim = p.row.vdim;
+    if (i >= p.heads + 2 * G) return;
+    const int pos = p.row_pos[r], seq = p.row_seq[r];
+    T* base = static_cast<T*>(p.qkv) + (size_t)r * p.qkv_stride;
+    if (i >= p.heads + G) {
+        const int g = i - p.heads - G;
+        const T* src = base + (size_t)(p.heads + G) * dim + (size_t)g * vdim;
+        T* dst = ga_block<T>(p, seq, pos / kPage, g) + (size_t)kPage * p.row.pk + (size_t)(pos % kPage) * p.row.pv;
+        for (int c = lane; c < vdim; c += 32) dst[c] = src[c];
+        return;
+    }
+    float* x = app_smem + (size_t)warp * dim;
+    T* src = base + (size_t)i * dim;
+    float ss = 0.f;
+    for (int c = lane; c < dim; c += 32) { const float v = ga_get(src + c); x[c] = v; ss = fmaf(v, v, ss); }
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const __nv_bfloat16* w = i < p.heads ? p.q_norm : p.k_norm;
+    if (w) {
+        const float sc = 1.0f / sqrtf(ss / (float)dim + p.eps);
+        for (int c = lane; c < dim; c += 32) x[c] = x[c] * sc * (__bfloat162float(w[c]) + p.weight_bias);
+    }
+    __syncwarp();
+    T* dst = i < p.heads ? src : ga_block<T>(p, seq, pos / kPage, i - p.heads) + (size_t)(pos % kPage) * p.row.pk;
+    for (int c = lane; c < dim; c += 32) {
+        float v = x[c];
+        if (c < p.rot_dims) {
+            const RotaryEntry e = rotary_entry(c, p.rot_dims, p.rot_neighbours);
+            float cs, sn;
+            sincosf((float)pos * p.inv_freq[e.pair], &sn, &cs);
+            const float o = x[e.partner];
+            v = p.magnitude * (e.first ? v * cs - o * sn : v * cs + o * sn);
+        }
+        ga_put(dst + c, v);
+    }
+}
+
+// ---- rows one by one, fp32 FMAs ---------------------------------------------------------------------------------------
+// CTA (row, head), four warps that take the keys in turn.
+constexpr int kSimpleWarps = 4;
+template <typename T>
+__global__ void __launch_bounds__(kSimpleWarps * 32) grouped_simple_kernel(const GroupedParams p) {
+    extern __shared__ __align__(16) float simple_smem[];
+    __shared__ float ms[kSimpleWarps], ls[kSimpleWarps];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dim = p.row.dim, vdim = p.row.vdim, h = blockIdx.y, g = h / p.share;
+    const int r = ga_row(p, blockIdx.x), pos = p.row_pos[r], seq = p.row_seq[r];
+    float* q = simple_smem;                                     // [dim]
+    float* acc = simple_smem + dim + (size_t)warp * vdim;       // [warps][vdim]
+    const T* src = static_cast<const T*>(p.qkv) + (size_t)r * p.qkv_stride + (size_t)h * dim;
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) q[i] = ga_get(src + i);
+    for (int i = lane; i < vdim; i += 32) acc[i] = 0.f;
+    __syncthreads();
+    float m = -INFINITY, l = 0.f;
+    for (int key = ga_first_seen(p, pos) + warp; key <= pos; key += kSimpleWarps) {
+        const T* block = ga_block<T>(p, seq, key / kPage, g);
+        const T* k = block + (size_t)(key % kPage) * p.row.pk;
+        const T* v = block + (size_t)kPage * p.row.pk + (size_t)(key % kPage) * p.row.pv;
+        float s = 0.f;
+        for (int i = lane; i < dim; i += 32) s = fmaf(q[i], ga_get(k + i), s);
+        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        s *= p.scale_log2;
+        const float m_new = fmaxf(m, s), corr = exp2f(m - m_new), w = exp2f(s - m_new);
+        l = l * corr + w;
+        m = m_new;
+        for (int i = lane; i < vdim; i += 32) acc[i] = acc[i] * corr + w * ga_get(v + i);
+    }
+    if (lane == 0) { ms[warp] = m; ls[warp] = l; }
+    __syncthreads();
+    float top = p.sink_one ? 0.f : -INFINITY;
+    for (int w = 0; w < kSimpleWarps; ++w) top = fmaxf(top, ms[w]);
+    float total = p.sink_one ? exp2f(-top) : 0.f;
+    for (int w = 0; w < kSimpleWarps; ++w) total += ls[w] * exp2f(ms[w] - top);
+    const float f = ga_gate(p, r, h) / total;
+    T* out = static_cast<T*>(p.out) + (size_t)r * p.out_stride + (size_t)h * vdim;
+    for (int i = threadIdx.x; i < vdim; i += blockDim.x) {
+        float v = 0.f;
+        for (int w = 0; w < kSimpleWarps; ++w) v += simple_smem[dim + (size_t)w * vdim + i] * exp2f(ms[w] - top);
+        ga_put(out + i, v * f);
+    }
+}
+
+// ---- rows one by one, tensor cores ------------------------------------------------------------------------------------
+// Cluster of CTAs per (row, key / value head, 16 query heads of it): the context in units of UK keys, dealt out to all warps of the
+// cluster. A unit is two bulk copies (keys, values) into the warp's own stage.
+constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kDecHeads = 16, kDecCluster = 8;
+template <int KQ, int NV, int UK>   // 16-column steps of query / key and value rows, keys of a unit
+__global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const GroupedParams p) {
+    extern __shared__ __align__(128) unsigned char dec_smem[];
+    __shared__ __align__(8) unsigned long long bar[kDecWarps];
+    __shared__ float warp_m[kDecWarps][kDecHeads], warp_l[kDecWarps][kDecHeads], cta_m[kDecHeads], cta_l[kDecHeads];
+    const cg::cluster_group cluster = cg::this_cluster();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int nz = gridDim.x, rank = blockIdx.x, kv = blockIdx.y / ((p.share + kDecHeads - 1) / kDecHeads), tile = blockIdx.y % ((p.share + kDecHeads - 1) / kDecHeads);
+    const int h0 = kv * p.share + tile * kDecHeads, nh = min(kDecHeads, p.share - tile * kDecHeads);   // query heads of this CTA
+    pdl_launch_dependents();
+    if (tid < kDecWarps) mbar_init(&bar[tid], 1);
+    if (tid == 0) asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    __syncthreads();
+    pdl_wait();
+    const int r = ga_row(p, blockIdx.z), pos = p.row_pos[r], seq = p.row_seq[r];
+    const int seen0 = ga_first_seen(p, pos), unit0 = seen0 / UK, units = pos / UK + 1 - unit0;
+    const int pk = p.row.pk, pv = p.row.pv, k_bytes = UK * pk * 2, v_bytes = UK * pv * 2;
+    unsigned char* stage = dec_smem + (size_t)warp * (k_bytes + v_bytes);
+    const unsigned bar_at = smem_u32(&bar[warp]);
+    auto request = [&](int u) {   // lane 0
+        const int key0 = (unit0 + u) * UK;
+        const __nv_bfloat16* block = ga_block<__nv_bfloat16>(p, seq, key0 / kPage, kv);
+        mbar_expect(bar_at, (unsigned)(k_bytes + v_bytes));
+        bulk_load(smem_u32(stage), block + (size_t)(key0 % kPage) * pk, (unsigned)k_bytes, bar_at);
+        bulk_load(smem_u32(stage) + (unsigned)k_bytes, block + (size_t)kPage * pk + (size_t)(key0 % kPage) * pv, (unsigned)v_bytes, bar_at);
+    };
+    const int first = rank * kDecWarps + warp, step = nz * kDecWarps;
+    if (lane == 0 && first < units) request(first);
+    // query fragments: rows g and g + 8
+    const int ksteps = p.row.dp >> 4, n_vt = p.row.vp >> 4;
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)r * p.qkv_stride + (size_t)h0 * p.row.dim;
+    unsigned qa[KQ][4];
+#pragma unroll
+    for (int k = 0; k < KQ; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int hh = g + 8 * (e & 1), c = 16 * k + 8 * (e >> 1) + 2 * t;
+            qa[k][e] = hh < nh && c < p.row.dim ? __ldcg(reinterpret_cast<const unsigned*>(q + (size_t)hh * p.row.dim + c)) : 0u;
+        }
+    float oacc[2 * NV][4];
+#pragma unroll
+    for (int j = 0; j < 2 * NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
+    float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
+    const unsigned ks = smem_u32(stage), vs = ks + (unsigned)k_bytes;
+    unsigned phase = 0;
+    for (int u = first; u < units; u += step, phase ^= 1) {
+        if (!mbar_wait(&bar[warp], phase)) {
+            if (lane == 0) atomicExch(p.status, 61);
+            mbar_wait(&bar[warp], phase);   // leave the loop only when the copy has landed (bounded)
+            break;
+        }
+        float sacc[UK / 8][4];
+#pragma unroll
+        for (int j = 0; j < UK / 8; ++j) sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f;
+#pragma unroll
+        for (int k = 0; k < KQ; ++k)
+            if (k < ksteps) {
+#pragma unroll
+                for (int jp = 0; jp < UK / 16; ++jp) {
+                    unsigned b[4];
+                    ga_ldsm(b, ks + (unsigned)((jp * 16 + (lane & 7) + 8 * (lane >> 4)) * pk + 16 * k + 8 * ((lane >> 3) & 1)) * 2u);
+                    ga_mma(sacc[2 * jp], qa[k], b[0], b[1]);
+                    ga_mma(sacc[2 * jp + 1], qa[k], b[2], b[3]);
+                }
+            }
+        const int key0 = (unit0 + u) * UK;
+        float mx_a = -INFINITY, mx_b = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < UK / 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int key = key0 + 8 * j + 2 * t + e;
+                const bool seen = key <= pos && key >= seen0;
+                sacc[j][e] = seen ? sacc[j][e] * p.scale_log2 : -INFINITY;
+                sacc[j][2 + e] = seen ? sacc[j][2 + e] * p.scale_log2 : -INFINITY;
+                mx_a = fmaxf(mx_a, sacc[j][e]); mx_b = fmaxf(mx_b, sacc[j][2 + e]);
+            }
+#pragma unroll
+        for (int o = 1; o < 4; o <<= 1) { mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, o)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, o)); }
+        // (every unit holds at least one key that is seen, by all heads alike)
+        const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b), ca = exp2f(m_a - mn_a), cb = exp2f(m_b - mn_b);
+        m_a = mn_a; m_b = mn_b;
+        float sa = 0.f, sb = 0.f;
+#pragma unroll
+        for (int j = 0; j < UK / 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                sacc[j][e] = exp2f(sacc[j][e] - mn_a); sa += sacc[j][e];
+                sacc[j][2 + e] = exp2f(sacc[j][2 + e] - mn_b); sb += sacc[j][2 + e];
+            }
+        l_a = l_a * ca + sa; l_b = l_b * cb + sb;
+#pragma unroll
+        for (int j = 0; j < 2 * NV; ++j) { oacc[j][0] *= ca; oacc[j][1] *= ca; oacc[j][2] *= cb; oacc[j][3] *= cb; }
+#pragma unroll
+        for (int kk = 0; kk < UK / 16; ++kk) {
+            unsigned ah[4], al[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float x = sacc[2 * kk + (e >> 1)][(e & 1) * 2], y = sacc[2 * kk + (e >> 1)][(e & 1) * 2 + 1];
+                const float xh = ga_round(x), yh = ga_round(y);
+                ah[e] = ga_pack(xh, yh);
+                al[e] = ga_pack(x - xh, y - yh);
+            }
+#pragma unroll
+            for (int j = 0; j < NV; ++j)
+                if (j < n_vt) {
+                    unsigned b[4];
+                    ga_ldsm_trans(b, vs + (unsigned)((16 * kk + (lane & 7) + 8 * ((lane >> 3) & 1)) * pv + 16 * j + 8 * (lane >> 4)) * 2u);
+                    ga_mma(oacc[2 * j], ah, b[0], b[1]);
+                    ga_mma(oacc[2 * j], al, b[0], b[1]);
+                    ga_mma(oacc[2 * j + 1], ah, b[2], b[3]);
+                    ga_mma(oacc[2 * j + 1], al, b[2], b[3]);
+                }
+        }
+        __syncwarp();   // the stage is free
+        if (lane == 0 && u + step < units) request(u + step);
+    }
+#pragma unroll
+    for (int o = 1; o < 4; o <<= 1) { l_a += __shfl_xor_sync(0xffffffffu, l_a, o); l_b += __shfl_xor_sync(0xffffffffu, l_b, o); }
+    if (t == 0) { warp_m[warp][g] = m_a; warp_m[warp][g + 8] = m_b; warp_l[warp][g] = l_a; warp_l[warp][g + 8] = l_b; }
+    __syncthreads();
+    // the stages now hold the warps' sums: [warps][heads of this CTA][vp], behind them the CTA's own [heads][vp]
+    const int vp = p.row.vp;
+    float* sums = reinterpret_cast<float*>(dec_smem);
+    float* own = sums + (size_t)kDecWarps * nh * vp;
+#pragma unroll
+    for (int j = 0; j < 2 * NV; ++j) {
+        const int c = 8 * j + 2 * t;
+        if (c < vp) {
+            if (g < nh) *reinterpret_cast<float2*>(sums + ((size_t)warp * nh + g) * vp + c) = make_float2(oacc[j][0], oacc[j][1]);
+            if (g + 8 < nh) *reinterpret_cast<float2*>(sums + ((size_t)warp * nh + g + 8) * vp + c) = make_float2(oacc[j][2], oacc[j][3]);
+        }
+    }
+    if (tid < nh) {
+        float top = -INFINITY, total = 0.f;
+        for (int w = 0; w < kDecWarps; ++w) top = fmaxf(top, warp_m[w][tid]);
+        for (int w = 0; w < kDecWarps; ++w) {
+            const float f = warp_m[w][tid] == -INFINITY ? 0.f : exp2f(warp_m[w][tid] - top);
+            total += f * warp_l[w][tid];
+            warp_l[w][tid] = f;
+        }
+        cta_m[tid] = top;
+        cta_l[tid] = total;
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * vp; i += kDecThreads) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < kDecWarps; ++w) v = fmaf(warp_l[w][i / vp], sums[(size_t)w * nh * vp + i], v);
+        own[i] = v;
+    }
+    cluster.sync();
+    for (int i = rank * kDecThreads + tid; i < nh * p.row.vdim; i += nz * kDecThreads) {
+        const int hh = i / p.row.vdim, c = i - hh * p.row.vdim;
+        float top = p.sink_one ? 0.f : -INFINITY;
+        for (int z = 0; z < nz; ++z) top = fmaxf(top, cluster.map_shared_rank(cta_m, z)[hh]);
+        float total = p.sink_one ? exp2f(-top) : 0.f, v = 0.f;
+        for (int z = 0; z < nz; ++z) {
+            const float mz = cluster.map_shared_rank(cta_m, z)[hh], f = mz == -INFINITY ? 0.f : exp2f(mz - top);
+            total = fmaf(f, cluster.map_shared_rank(cta_l, z)[hh], total);
+            v = fmaf(f, cluster.map_shared_rank(own, z)[hh * vp + c], v);
+        }
+        static_cast<__nv_bfloat16*>(p.out)[(size_t)r * p.out_stride + (size_t)(h0 + hh) * p.row.vdim + c] = __float2bfloat16_rn(v / total * ga_gate(p, r, h0 + hh));
+    }
+    cluster.sync();   // nobody leaves while others still read
+}
+
+// ---- spans ------------------------------------------------------------------------------------------------------------
+// CTA (tile of 128 query rows of a span, head), 8 warps of 16 query rows; a key tile is a page, one bulk copy of keys and values.
+constexpr int kPfThreads = 256, kPfStages = 3;
+template <int KQ, int NV>
+__global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const GroupedParams p) {
+    extern __shared__ __align__(128) unsigned char pf_smem[];
+    __shared__ __align__(8) unsigned long long full_bar[kPfStages];
+    __shared__ int bad;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, h = blockIdx.y, kv = h / p.share;
+    const int pk = p.row.pk, pv = p.row.pv, stage_bytes = p.row.block * 2;
+    pdl_launch_dependents();
+    if (tid == 0) {
+        for (int s = 0; s < kPfStages; ++s) mbar_init(&full_bar[s], 1);
+        bad = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    pdl_wait();
+    const int2 tile = p.tiles[blockIdx.x];
+    const LatentSpan span = p.spans[tile.x];
+    const int q0 = tile.y * kLatentQueryTile, nq = min(kLatentQueryTile, span.count - q0);
+    const int first_pos = span.pos0 + q0, last_pos = first_pos + nq - 1;
+    const int kt0 = ga_first_seen(p, first_pos) / kPage, n_tiles = last_pos / kPage + 1 - kt0;
+    auto request = [&](int i) {   // thread 0: key tile kt0 + i
+        const unsigned at = smem_u32(&full_bar[i % kPfStages]);
+        mbar_expect(at, (unsigned)stage_bytes);
+        bulk_load(smem_u32(pf_smem) + (unsigned)(i % kPfStages * stage_bytes), ga_block<__nv_bfloat16>(p, span.seq, kt0 + i, kv), (unsigned)stage_bytes, at);
+    };
+    if (tid == 0) for (int i = 0; i < min(kPfStages, n_tiles); ++i) request(i);
+    unsigned qa[KQ][4];
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)(span.row0 + q0) * p.qkv_stride + (size_t)h * p.row.dim;
+#pragma unroll
+    for (int k = 0; k < KQ; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int rr = warp * 16 + g + 8 * (e & 1), c = 16 * k + 8 * (e >> 1) + 2 * t;
+            qa[k][e] = rr < nq && c < p.row.dim ? __ldcg(reinterpret_cast<const unsigned*>(q + (size_t)rr * p.qkv_stride + c)) : 0u;
+        }
+    const int pos_a = first_pos + warp * 16 + g, pos_b = pos_a + 8;
+    const int warp_first = first_pos + warp * 16, warp_last = min(warp_first + 15, last_pos);
+    const int seen_a = ga_first_seen(p, pos_a), seen_b = ga_first_seen(p, pos_b), warp_seen = ga_first_seen(p, warp_first), full_from = ga_first_seen(p, warp_last);
+    float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
+    float oacc[2 * NV][4];
+#pragma unroll
+    for (int j = 0; j < 2 * NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
+    const int ksteps = p.row.dp >> 4, n_vt = p.row.vp >> 4;
+    int i = 0;
+    for (; i < n_tiles; ++i) {
+        if (!mbar_wait(&full_bar[i % kPfStages], (unsigned)((i / kPfStages) & 1))) { atomicExch(p.status, 62); bad = 1; }
+        const int key0 = (kt0 + i) * kPage;
+        const unsigned kb = smem_u32(pf_smem) + (unsigned)(i % kPfStages * stage_bytes), vb = kb + (unsigned)(kPage * pk) * 2u;
+        if (warp_first <= last_pos && key0 <= warp_last && key0 + kPage > warp_seen) {
+            float sacc[8][4];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f;
+#pragma unroll
+            for (int k = 0; k < KQ; ++k)
+                if (k < ksteps) {
+#pragma unroll
+                    for (int jp = 0; jp < 4; ++jp) {
+                        unsigned b[4];
+                        ga_ldsm(b, kb + (unsigned)((jp * 16 + (lane & 7) + 8 * (lane >> 4)) * pk + 16 * k + 8 * ((lane >> 3) & 1)) * 2u);
+                        ga_mma(sacc[2 * jp], qa[k], b[0], b[1]);
+                        ga_mma(sacc[2 * jp + 1], qa[k], b[2], b[3]);
+                    }
+                }
+            const bool edge = key0 + kPage - 1 > warp_first || key0 < full_from;   // some row does not see the whole tile
+            float mx_a = -INFINITY, mx_b = -INFINITY;
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int key = key0 + 8 * j + 2 * t + e;
+                    const float a = !edge || (key <= pos_a && key >= seen_a) ? sacc[j][e] * p.scale_log2 : -INFINITY;
+                    const float b = !edge || (key <= pos_b && key >= seen_b) ? sacc[j][2 + e] * p.scale_log2 : -INFINITY;
+                    sacc[j][e] = a; sacc[j][2 + e] = b;
+                    mx_a = fmaxf(mx_a, a); mx_b = fmaxf(mx_b, b);
+                }
+#pragma unroll
+            for (int o = 1; o < 4; o <<= 1) { mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, o)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, o)); }
+            const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
+            // a row that sees nothing yet keeps a maximum of -inf, weights of zero and sums of zero
+            const float ra = mn_a == -INFINITY ? 0.f : mn_a, rb = mn_b == -INFINITY ? 0.f : mn_b;
+            const float ca = m_a == -INFINITY ? 1.f : exp2f(m_a - mn_a), cb = m_b == -INFINITY ? 1.f : exp2f(m_b - mn_b);
+            m_a = mn_a; m_b = mn_b;
+            float sa = 0.f, sb = 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    sacc[j][e] = exp2f(sacc[j][e] - ra); sa += sacc[j][e];
+                    sacc[j][2 + e] = exp2f(sacc[j][2 + e] - rb); sb += sacc[j][2 + e];
+                }
+            l_a = l_a * ca + sa; l_b = l_b * cb + sb;
+            if (__any_sync(0xffffffffu, ca != 1.0f || cb != 1.0f)) {
+#pragma unroll
+                for (int j = 0; j < 2 * NV; ++j) { oacc[j][0] *= ca; oacc[j][1] *= ca; oacc[j][2] *= cb; oacc[j][3] *= cb; }
+            }
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                unsigned ah[4], al[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float x = sacc[2 * kk + (e >> 1)][(e & 1) * 2], y = sacc[2 * kk + (e >> 1)][(e & 1) * 2 + 1];
+                    const float xh = ga_round(x), yh = ga_round(y);
+                    ah[e] = ga_pack(xh, yh);
+                    al[e] = ga_pack(x - xh, y - yh);
+                }
+#pragma unroll
+                for (int j = 0; j < NV; ++j)
+                    if (j < n_vt) {
+                        unsigned b[4];
+                        ga_ldsm_trans(b, vb + (unsigned)((16 * kk + (lane & 7) + 8 * ((lane >> 3) & 1)) * pv + 16 * j + 8 * (lane >> 4)) * 2u);
+                        ga_mma(oacc[2 * j], ah, b[0], b[1]);
+                        ga_mma(oacc[2 * j], al, b[0], b[1]);
+                        ga_mma(oacc[2 * j + 1], ah, b[2], b[3]);
+                        ga_mma(oacc[2 * j + 1], al, b[2], b[3]);
+                    }
+            }
+        }
+        __syncthreads();   // the stage is free
+        if (bad) break;    // uniform: written before the barrier by whoever gave up
+        if (tid == 0 && i + kPfStages < n_tiles) request(i + kPfStages);
+    }
+    if (bad) {
+        // leave only when the copies that may still be under way have landed (bounded)
+        if (tid == 0) for (int k = i; k < i + kPfStages && k < n_tiles; ++k) mbar_wait(&full_bar[k % kPfStages], (unsigned)((k / kPfStages) & 1));
+        return;
+    }
+#pragma unroll
+    for (int o = 1; o < 4; o <<= 1) { l_a += __shfl_xor_sync(0xffffffffu, l_a, o); l_b += __shfl_xor_sync(0xffffffffu, l_b, o); }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int rr = warp * 16 + g + 8 * half;
+        if (rr >= nq) continue;
+        const int row = span.row0 + q0 + rr;
+        // (every row sees its own key, so its maximum is finite)
+        const float m = half ? m_b : m_a, top = p.sink_one ? fmaxf(m, 0.f) : m, own = exp2f(m - top);
+        const float f = ga_gate(p, row, h) * own / ((half ? l_b : l_a) * own + (p.sink_one ? exp2f(-top) : 0.f));
+        __nv_bfloat16* o = static_cast<__nv_bfloat16*>(p.out) + (size_t)row * p.out_stride + (size_t)h * p.row.vdim;
+#pragma unroll
+        for (int j = 0; j < 2 * NV; ++j) {
+            const int c = 8 * j + 2 * t;
+            if (c < p.row.vdim) *reinterpret_cast<unsigned*>(o + c) = ga_pack(oacc[j][2 * half] * f, oacc[j][2 * half + 1] * f);
+        }
+    }
+}
+
+// ---- launches ---------------------------------------------------------------------------------------------------------
+enum { FORM_MEDIUM, FORM_LARGE, FORM_SIMPLE };
+// up to 128 entries per head: decode and prefill kernels; up to 256: the decode kernel for all rows; else fp32 FMAs
+int form_of(const GroupedRow& r, bool f32) {
+    if (f32 || ((r.dim | r.vdim) & 7)) return FORM_SIMPLE;
+    return r.dp <= 128 && r.vp <= 128 ? FORM_MEDIUM : r.dp <= 256 && r.vp <= 256 ? FORM_LARGE : FORM_SIMPLE;
+}
+constexpr size_t kGaMaxSmem = 200 * 1024;
+size_t decode_smem(const GroupedRow& r, int share, int unit) {
+    const size_t stages = (size_t)kDecWarps * unit * (r.pk + r.pv) * 2, sums = (size_t)(kDecWarps + 1) * std::min(share, kDecHeads) * r.vp * 4;
+    return std::max(stages, sums);
+}
+size_t simple_bytes(const GroupedRow& r) { return ((size_t)r.dim + (size_t)kSimpleWarps * r.vdim) * 4; }
+template <int KQ, int NV, int UK>
+cudaError_t decode_launch(const GroupedParams& p, int nz, cudaStream_t s) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(nz, p.row.groups * ((p.share + kDecHeads - 1) / kDecHeads), p.n_rows); cfg.blockDim = dim3(kDecThreads); cfg.stream = s;
+    cfg.dynamicSmemBytes = decode_smem(p.row, p.share, UK);
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = nz; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl_enabled() ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, grouped_decode_kernel<KQ, NV, UK>, p);
+}
+constexpr int kUnitMedium = 32, kUnitLarge = 16;
+// CTAs per cluster: enough warps for the longest context, about one CTA per SM over all rows
+int decode_cluster(const GroupedLaunch& a, int unit) {
+    int keys = a.max_pages * kPage;
+    if (a.window > 0) keys = std::min(keys, a.window);
+    if (a.chunk > 0) keys = std::min(keys, a.chunk);
+    const int units = (keys + unit - 2) / unit + 1, tiles = a.n_short * a.row.groups * ((a.heads / a.row.groups + kDecHeads - 1) / kDecHeads);
+    int nz = kDecCluster;
+    while (nz > 1 && ((nz >> 1) * kDecWarps >= units || (long long)tiles * nz > 148)) nz >>= 1;
+    return nz;
+}
+
+}  // namespace
+
+GroupedRow grouped_row(int groups, int dim, int vdim, bool f32) {
+    GroupedRow r;
+    r.groups = groups; r.dim = dim; r.vdim = vdim;
+    r.dp = (dim + 15) / 16 * 16; r.vp = (vdim + 15) / 16 * 16;
+    r.pk = r.dp + (f32 ? 0 : 8); r.pv = r.vp + (f32 ? 0 : 8);
+    r.block = kPage * (r.pk + r.pv);
+    return r;
+}
+bool grouped_supported(const GroupedRow& r) { return r.dim <= 4096 && simple_bytes(r) <= kGaMaxSmem; }
+bool grouped_spans(const GroupedRow& r, bool f32) { return form_of(r, f32) == FORM_MEDIUM; }
+
+int grouped_init() {
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_simple_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_simple_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<8, 8, kUnitMedium>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<16, 16, kUnitLarge>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_prefill_kernel<8, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    return SWLM_OK;
+}
+
+int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches) {
+    GroupedParams p{};
+    p.row = a.row; p.heads = a.heads; p.share = a.heads / a.row.groups; p.rot_dims = a.rot_dims; p.rot_neighbours = a.rot_neighbours;
+    p.window = a.window; p.chunk = a.chunk; p.sink_one = a.sink_one;
+    p.scale_log2 = a.scale * kLog2e; p.eps = a.eps; p.weight_bias = a.weight_bias; p.magnitude = a.magnitude; p.out_scale = a.out_scale; p.inv_freq = a.inv_freq;
+    p.q_norm = a.q_norm; p.k_norm = a.k_norm; p.qkv = a.qkv; p.qkv_stride = a.qkv_stride; p.gate = a.gate; p.gate_stride = a.gate_stride;
+    p.pool = a.pool; p.page_table = a.page_table; p.pages_per_seq = a.pages_per_seq; p.row_seq = a.row_seq; p.row_pos = a.row_pos;
+    p.out = a.out; p.out_stride = a.out_stride; p.spans = a.spans; p.tiles = a.tiles; p.status = a.status;
+    cudaError_t e;
+    if (!a.only_attention) {
+        const dim3 grid(a.n_rows, (a.heads + 2 * a.row.groups + kAppWarps - 1) / kAppWarps);
+        const size_t smem = (size_t)kAppWarps * a.row.dim * 4;
+        e = a.f32 ? launch_k(grouped_append_kernel<float>, grid, dim3(kAppWarps * 32), smem, s, p) : launch_k(grouped_append_kernel<__nv_bfloat16>, grid, dim3(kAppWarps * 32), smem, s, p);
+        if (e != cudaSuccess) return cuda_fail(e, "grouped append launch");
+        *launches += 1;
+    }
+    if (a.n_short > 0) {
+        p.n_rows = a.n_short; p.rows = a.short_rows;
+        switch (form_of(a.row, a.f32)) {
+        case FORM_MEDIUM: e = decode_launch<8, 8, kUnitMedium>(p, decode_cluster(a, kUnitMedium), s); break;
+        case FORM_LARGE: e = decode_launch<16, 16, kUnitLarge>(p, decode_cluster(a, kUnitLarge), s); break;
+        default:
+            e = a.f32 ? launch_k(grouped_simple_kernel<float>, dim3(a.n_short, a.heads), dim3(kSimpleWarps * 32), simple_bytes(a.row), s, p)
+                      : launch_k(grouped_simple_kernel<__nv_bfloat16>, dim3(a.n_short, a.heads), dim3(kSimpleWarps * 32), simple_bytes(a.row), s, p);
+        }
+        if (e != cudaSuccess) return cuda_fail(e, "grouped attention launch");
+        *launches += 1;
+    }
+    if (a.n_tiles > 0) {
+        e = launch_k(grouped_prefill_kernel<8, 8>, dim3(a.n_tiles, a.heads), dim3(kPfThreads), (size_t)kPfStages * a.row.block * 2, s, p);
+        if (e != cudaSuccess) return cuda_fail(e, "grouped prompt attention launch");
+        *launches += 1;
+    }
+    return SWLM_OK;
+}
+
+}  // namespace swlm

@@ -56,7 +56,7 @@ __device__ __forceinline__ void lat_ldsm_trans(unsigned (&r)[4], unsigned addr) 
 
 struct LatentParams {
     LatentRow row;
-    int heads, dim, vdim, rot_dims;
+    int heads, dim, vdim, rot_dims, rot_neighbours;
     float scale_log2, eps, weight_bias, magnitude;
     int window; const __nv_bfloat16* sink;
     const float* inv_freq;
@@ -111,15 +111,14 @@ __device__ __forceinline__ void angle(const LatentParams& p, int pos, int i, flo
     c *= p.magnitude;
     s *= p.magnitude;
 }
-// entry i of a rotated part x[0 .. rot) at position pos (rotate-half over the first rot_dims entries)
+// entry i of a rotated part x[0 .. rot) at position pos
 template <typename V>
 __device__ __forceinline__ float rotated(const LatentParams& p, const V& x, int pos, int i) {
-    const int half = p.rot_dims >> 1;
     if (i >= p.rot_dims) return x(i);
-    const bool low = i < half;
+    const RotaryEntry e = rotary_entry(i, p.rot_dims, p.rot_neighbours);
     float c, s;
-    angle(p, pos, low ? i : i - half, c, s);
-    return low ? x(i) * c - x(i + half) * s : x(i) * c + x(i - half) * s;
+    angle(p, pos, e.pair, c, s);
+    return e.first ? x(i) * c - x(e.partner) * s : x(i) * c + x(e.partner) * s;
 }
 
 // The row a warp appends: norm of the latent, rotation of the shared key part, zeros in the padding.
@@ -651,14 +650,15 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const LatentParams p
     if (warp == 0) { append_row<__nv_bfloat16>(p, r, lane); return; }
     const int half = p.rot_dims >> 1, per_head = p.dim + p.row.rot, pos = p.row_pos[r];
     __nv_bfloat16* q = static_cast<__nv_bfloat16*>(p.q) + (size_t)r * p.q_stride + p.dim;
+    const int step = rotary_step(p.rot_dims, p.rot_neighbours);
     for (int i = lane; i < half; i += 32) {
         float c, s;
         angle(p, pos, i, c, s);
         for (int h = warp - 1; h < p.heads; h += 3) {
-            __nv_bfloat16* x = q + (size_t)h * per_head;
-            const float u = __bfloat162float(x[i]), v = __bfloat162float(x[i + half]);
-            x[i] = __float2bfloat16_rn(u * c - v * s);
-            x[i + half] = __float2bfloat16_rn(v * c + u * s);
+            __nv_bfloat16* x = q + (size_t)h * per_head + rotary_first(i, p.rot_neighbours);
+            const float u = __bfloat162float(x[0]), v = __bfloat162float(x[step]);
+            x[0] = __float2bfloat16_rn(u * c - v * s);
+            x[step] = __float2bfloat16_rn(v * c + u * s);
         }
     }
 }
@@ -845,7 +845,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) latent_prefill_kernel(const Lat
 
 LatentParams latent_params(const LatentLaunch& a) {
     LatentParams p{};
-    p.row = a.row; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim; p.rot_dims = a.rot_dims;
+    p.row = a.row; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim; p.rot_dims = a.rot_dims; p.rot_neighbours = a.rot_neighbours;
     p.window = a.window; p.sink = a.sink;
     p.scale_log2 = a.scale * kLog2e; p.eps = a.eps; p.weight_bias = a.weight_bias; p.magnitude = a.magnitude; p.inv_freq = a.inv_freq;
     p.q = a.q; p.q_stride = a.q_stride; p.kv = a.kv; p.kv_stride = a.kv_stride; p.gate = a.gate; p.gate_stride = a.gate_stride;

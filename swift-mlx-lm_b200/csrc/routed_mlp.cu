@@ -1,10 +1,12 @@
-// Routed feed-forward: a router picks `top` of the experts for every row, the row's result is the weighted sum of theirs.
+// Routed feed-forward: a router picks `top` of the experts for every row, the row's result is the weighted sum of theirs; a
+// shared feed-forward that every row takes, weighted by a sigmoid, may join the sum.
 //
 //   few rows (and fp32 plans)  routed_gate_kernel: every CTA works out its row's choice from the router's logits, then streams
-//                              gate and up rows of one chosen expert; routed_down_kernel: a warp per output runs through the
-//                              chosen experts' down rows one after the other, so the sum over experts needs no pass of its own.
+//                              gate and up rows of one chosen expert (the shared feed-forward is one more slot of the choice);
+//                              routed_down_kernel: a warp per output runs through the chosen experts' down rows one after the
+//                              other, so the sum over experts needs no pass of its own.
 //   more rows (bf16)           routed_choose_kernel, routed_sort_kernel (rows sorted by expert, table of tiles), two grouped
-//                              tensor-core products, routed_sum_kernel.
+//                              tensor-core products, two plain ones for the shared feed-forward, routed_sum_kernel.
 //
 // An expert's place among the candidates is the number of candidates before it (larger score, or equal score and lower index),
 // so the choice takes one pass without a sequence of maxima.
@@ -22,10 +24,14 @@ struct RoutedParams {
     RoutedShape sh;
     float scale;
     GatedAct act;
+    int softmax, group_best, raw_weights;
     int m;
     const void* x; int x_stride;
     const float* z; int z_stride;
-    const __nv_bfloat16 *gate, *up, *down; int in_ld, mid_ld;   // row pitches of gate / up and of down
+    const __nv_bfloat16 *gate, *up, *down; int in_ld, mid_ld;   // row pitches of gate / up and of down; gate == null: GELU of up
+    const __nv_bfloat16 *shared_up, *shared_down; int shared_ld;
+    void* shared_mid; int shared_stride;     // [rows][shared_stride]
+    const float* shared_y; int shared_y_stride;
     float* out; int out_stride;
     int* sel; float* weight; int* rank;      // [rows][top]
     unsigned* counts;                        // [experts]
@@ -52,6 +58,8 @@ __device__ __forceinline__ float rt_dot8(const uint4& w, const float* x, float a
     acc = fmaf(rt_lo(w.z), b.x, acc); acc = fmaf(rt_hi(w.z), b.y, acc); acc = fmaf(rt_lo(w.w), b.z, acc); return fmaf(rt_hi(w.w), b.w, acc);
 }
 
+__device__ __forceinline__ float shared_weight(const RoutedParams& p, int row) { return 1.0f / (1.0f + expf(-p.z[(size_t)row * p.z_stride + p.sh.experts])); }
+
 // The choice of one row by THREADS threads (a warp or the CTA). s: [experts] scores, gs: [groups] group scores, both shared;
 // sel / w: [top] in order of falling score.
 template <int THREADS>
@@ -59,16 +67,25 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
     auto sync = [] { if (THREADS == 32) __syncwarp(); else __syncthreads(); };
     const int E = p.sh.experts, G = p.sh.groups, per = E / G;
     for (int i = tid; i < p.sh.top; i += THREADS) { sel[i] = i; w[i] = 0.f; }   // indices stay valid whatever the logits are
-    for (int e = tid; e < E; e += THREADS) s[e] = 1.0f / (1.0f + expf(-z[e]));
+    if (p.softmax) {   // every warp works out maximum and sum for itself
+        float top = -INFINITY, sum = 0.f;
+        for (int e = tid & 31; e < E; e += 32) top = fmaxf(top, z[e]);
+        for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+        for (int e = tid & 31; e < E; e += 32) sum += expf(z[e] - top);
+        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        for (int e = tid; e < E; e += THREADS) s[e] = expf(z[e] - top) / sum;
+    } else {
+        for (int e = tid; e < E; e += THREADS) s[e] = 1.0f / (1.0f + expf(-z[e]));
+    }
     sync();
     for (int g = tid; g < G; g += THREADS) {
-        float first = 0.f, second = 0.f;   // scores are positive
+        float first = 0.f, second = 0.f;   // scores are not negative
         for (int e = g * per; e < (g + 1) * per; ++e) {
             const float v = s[e];
             second = fmaxf(second, fminf(first, v));
             first = fmaxf(first, v);
         }
-        gs[g] = first + second;
+        gs[g] = p.group_best == 1 ? first : first + second;
     }
     sync();
     auto kept = [&](int g) {
@@ -91,13 +108,13 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
     float total = 0.f;
     for (int i = 0; i < p.sh.top; ++i) total += w[i];
     sync();
-    for (int i = tid; i < p.sh.top; i += THREADS) w[i] = w[i] / (total + 1e-20f) * p.scale;
+    for (int i = tid; i < p.sh.top; i += THREADS) w[i] = p.raw_weights ? w[i] * p.scale : w[i] / (total + 1e-20f) * p.scale;
     sync();
 }
 
 // ---- few rows ---------------------------------------------------------------------------------------------------------
-// CTA (share of the expert's rows, slot of the choice, row).
-template <typename T>
+// CTA (share of the expert's rows, slot of the choice, row); the slot behind the last one is the shared feed-forward.
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -114,56 +131,61 @@ __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedPar
         p.sel[row * p.sh.top + tid] = sel[tid];
         p.weight[row * p.sh.top + tid] = weight[tid];
     }
-    const size_t first = (size_t)sel[slot] * p.sh.ff;
+    const bool shared = slot == p.sh.top;
+    const int ff = shared ? p.sh.shared_ff : p.sh.ff;
+    const size_t first = shared ? 0 : (size_t)sel[slot] * p.sh.ff;
+    const __nv_bfloat16* up = shared ? p.shared_up : p.up;
     const int chunks = p.in_ld >> 3;
-    T* mid = static_cast<T*>(p.mid) + (size_t)(row * p.sh.top + slot) * p.mid_stride;
+    T* mid = shared ? static_cast<T*>(p.shared_mid) + (size_t)row * p.shared_stride : static_cast<T*>(p.mid) + (size_t)(row * p.sh.top + slot) * p.mid_stride;
     constexpr int U = 4;
-    for (int f = blockIdx.x * kRtWarps + warp; f < p.sh.ff; f += gridDim.x * kRtWarps) {
+    for (int f = blockIdx.x * kRtWarps + warp; f < ff; f += gridDim.x * kRtWarps) {
         const __nv_bfloat16* gr = p.gate + (first + f) * p.in_ld;
-        const __nv_bfloat16* ur = p.up + (first + f) * p.in_ld;
+        const __nv_bfloat16* ur = up + (first + f) * p.in_ld;
         float g = 0.f, u = 0.f;
         for (int c0 = lane; c0 < chunks; c0 += 32 * U) {
             uint4 gv[U], uv[U];
 #pragma unroll
             for (int j = 0; j < U; ++j) {
                 const int c = c0 + 32 * j;
-                gv[j] = c < chunks ? rt_stream(gr + 8 * c) : make_uint4(0, 0, 0, 0);
+                gv[j] = GATED && c < chunks ? rt_stream(gr + 8 * c) : make_uint4(0, 0, 0, 0);
                 uv[j] = c < chunks ? rt_stream(ur + 8 * c) : make_uint4(0, 0, 0, 0);
             }
 #pragma unroll
             for (int j = 0; j < U; ++j) {
                 const int c = c0 + 32 * j;
-                if (c < chunks) { g = rt_dot8(gv[j], x + 8 * c, g); u = rt_dot8(uv[j], x + 8 * c, u); }
+                if (c < chunks) { if (GATED) g = rt_dot8(gv[j], x + 8 * c, g); u = rt_dot8(uv[j], x + 8 * c, u); }
             }
         }
-        for (int o = 16; o > 0; o >>= 1) { g += __shfl_xor_sync(0xffffffffu, g, o); u += __shfl_xor_sync(0xffffffffu, u, o); }
-        if (lane == 0) rt_put(mid + f, gated_activation(g, u, p.act));
+        for (int o = 16; o > 0; o >>= 1) { if (GATED) g += __shfl_xor_sync(0xffffffffu, g, o); u += __shfl_xor_sync(0xffffffffu, u, o); }
+        if (lane == 0) rt_put(mid + f, GATED ? gated_activation(g, u, p.act) : gelu_erf(u));
     }
 }
 
 // CTA (share of the outputs, row): mid rows of all chosen experts, weighted, in shared memory; two warps per output, each with
-// half of the 16-byte chunks of the chosen experts' rows.
+// half of the 16-byte chunks of the chosen experts' rows, those of the shared feed-forward behind them.
 constexpr int kDownUnroll = 8, kDownWarps = 2;
 template <typename T>
 __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedParams p) {
     pdl_launch_dependents();
     pdl_wait();
-    extern __shared__ __align__(16) float rt_smem[];   // [top][mid_ld]
+    extern __shared__ __align__(16) float rt_smem[];   // [top][mid_ld], [shared_ld]
     __shared__ float part[kRtWarps];
     __shared__ int sel[kMaxTop];
     __shared__ float weight[kMaxTop];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, top = p.sh.top;
     if (tid < top) { sel[tid] = p.sel[row * top + tid]; weight[tid] = p.weight[row * top + tid]; }
     __syncthreads();
-    const int chunks = p.mid_ld >> 3, all = chunks * top, half = warp % kDownWarps;
+    const int chunks = p.mid_ld >> 3, routed = chunks * top, all = routed + (p.shared_ld >> 3), half = warp % kDownWarps;
     uint4 v[kDownUnroll];
     auto load = [&](int n, int c0) {
-        int t = c0 / chunks, c = c0 - t * chunks;
+        int t = min(c0 / chunks, top), c = c0 - t * chunks;
 #pragma unroll
         for (int j = 0; j < kDownUnroll; ++j) {
-            v[j] = t < top && n < p.sh.width ? rt_stream(p.down + ((size_t)sel[t] * p.sh.width + n) * p.mid_ld + 8 * c) : make_uint4(0, 0, 0, 0);
+            const bool live = n < p.sh.width && (t < top || c < all - routed);
+            const __nv_bfloat16* src = t < top ? p.down + ((size_t)sel[t] * p.sh.width + n) * p.mid_ld : p.shared_down + (size_t)n * p.shared_ld;
+            v[j] = live ? rt_stream(src + 8 * c) : make_uint4(0, 0, 0, 0);
             c += 32 * kDownWarps;
-            while (c >= chunks) { c -= chunks; ++t; }
+            while (t < top && c >= chunks) { c -= chunks; ++t; }
         }
     };
     const int first = half * 32 + lane;
@@ -173,6 +195,11 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
         const T* mid = static_cast<const T*>(p.mid) + (size_t)(row * top + t) * p.mid_stride;
         const float w = weight[t];
         for (int i = tid; i < p.mid_ld; i += kRtThreads) rt_smem[t * p.mid_ld + i] = i < p.sh.ff ? rt_get(mid + i) * w : 0.f;
+    }
+    if (p.shared_ld) {
+        const T* mid = static_cast<const T*>(p.shared_mid) + (size_t)row * p.shared_stride;
+        const float w = shared_weight(p, row);
+        for (int i = tid; i < p.shared_ld; i += kRtThreads) rt_smem[top * p.mid_ld + i] = i < p.sh.shared_ff ? rt_get(mid + i) * w : 0.f;
     }
     __syncthreads();
     const int step = gridDim.x * kRtWarps / kDownWarps, rounds = (p.sh.width + step - 1) / step;
@@ -285,6 +312,11 @@ __global__ void __launch_bounds__(kRtThreads) routed_sum_kernel(const RoutedPara
         const float4 y = *reinterpret_cast<const float4*>(p.y + (size_t)p.rank[row * p.sh.top + t] * p.y_stride + i);   // (rows are padded to 8)
         v.x = fmaf(w, y.x, v.x); v.y = fmaf(w, y.y, v.y); v.z = fmaf(w, y.z, v.z); v.w = fmaf(w, y.w, v.w);
     }
+    if (p.shared_y) {
+        const float w = shared_weight(p, row);
+        const float4 y = *reinterpret_cast<const float4*>(p.shared_y + (size_t)row * p.shared_y_stride + i);
+        v.x = fmaf(w, y.x, v.x); v.y = fmaf(w, y.y, v.y); v.z = fmaf(w, y.z, v.z); v.w = fmaf(w, y.w, v.w);
+    }
     float* o = p.out + (size_t)row * p.out_stride + i;
     const float r[4] = {v.x, v.y, v.z, v.w};
     for (int j = 0; j < 4 && i + j < p.sh.width; ++j) o[j] = r[j];
@@ -294,7 +326,7 @@ __global__ void __launch_bounds__(kRtThreads) routed_sum_kernel(const RoutedPara
 int up8(int v) { return (v + 7) / 8 * 8; }
 size_t up256(size_t v) { return (v + 255) / 256 * 256; }
 bool few(int m, bool f32) { return f32 || m <= kRtFewRows; }
-struct RoutedScratch { size_t sel, weight, rank, tiles, mid, sorted, y, total; };
+struct RoutedScratch { size_t sel, weight, rank, tiles, mid, sorted, y, shared_mid, shared_y, total; };
 RoutedScratch layout(const RoutedShape& s, int m, bool f32) {
     RoutedScratch l;
     const size_t a = (size_t)m * s.top;
@@ -305,18 +337,22 @@ RoutedScratch layout(const RoutedShape& s, int m, bool f32) {
     l.mid = l.tiles + (few(m, f32) ? 0 : up256((size_t)grouped_max_tiles((int)a, s.experts) * 16));
     l.sorted = l.mid + up256(a * up8(s.ff) * (f32 ? 4 : 2));
     l.y = l.sorted + (few(m, f32) ? 0 : up256(a * up8(s.width) * 2));
-    l.total = l.y + (few(m, f32) ? 0 : up256(a * up8(s.width) * 4));
+    l.shared_mid = l.y + (few(m, f32) ? 0 : up256(a * up8(s.width) * 4));
+    l.shared_y = l.shared_mid + up256((size_t)m * up8(s.shared_ff) * (f32 ? 4 : 2));
+    l.total = l.shared_y + (few(m, f32) || !s.shared_ff ? 0 : up256((size_t)m * up8(s.width) * 4));
     return l;
 }
 constexpr size_t kRtMaxSmem = 200 * 1024;
 size_t gate_smem(const RoutedShape& s) { return ((size_t)up8(s.width) + s.experts + s.groups) * 4; }
-size_t down_smem(const RoutedShape& s) { return (size_t)s.top * up8(s.ff) * 4; }
+size_t down_smem(const RoutedShape& s) { return ((size_t)s.top * up8(s.ff) + up8(s.shared_ff)) * 4; }
 
 template <typename T>
 int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
     // about two CTAs per SM over the chosen experts of all rows
-    const int pairs = (p.sh.ff + kRtWarps - 1) / kRtWarps, gx = std::max(1, std::min(pairs, (4 * 148 + p.sh.top * p.m - 1) / (p.sh.top * p.m)));
-    cudaError_t e = launch_k(routed_gate_kernel<T>, dim3(gx, p.sh.top, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
+    const int slots = p.sh.top + (p.sh.shared_ff ? 1 : 0);
+    const int pairs = (std::max(p.sh.ff, p.sh.shared_ff) + kRtWarps - 1) / kRtWarps, gx = std::max(1, std::min(pairs, (4 * 148 + slots * p.m - 1) / (slots * p.m)));
+    cudaError_t e = p.gate ? launch_k(routed_gate_kernel<T, true>, dim3(gx, slots, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p)
+                           : launch_k(routed_gate_kernel<T, false>, dim3(gx, slots, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed gate launch");
     const int outs = (p.sh.width * kDownWarps + kRtWarps - 1) / kRtWarps, dx = std::max(1, std::min(outs, (4 * 148 + p.m - 1) / p.m));
     e = launch_k(routed_down_kernel<T>, dim3(dx, p.m), dim3(kRtThreads), down_smem(p.sh), s, p);
@@ -328,15 +364,17 @@ int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
 }  // namespace
 
 int routed_init() {
-    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<float, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<float, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<__nv_bfloat16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<__nv_bfloat16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
     return SWLM_OK;
 }
 bool routed_supported(const RoutedShape& s) {
     return s.experts > 0 && s.experts <= kMaxExperts && s.top > 0 && s.top <= kMaxTop && s.groups > 0 && s.experts % s.groups == 0 && s.keep > 0 &&
-           s.keep <= s.groups && s.top <= s.keep * (s.experts / s.groups) && s.width > 0 && s.ff > 0 && gate_smem(s) <= kRtMaxSmem && down_smem(s) <= kRtMaxSmem;
+           s.keep <= s.groups && s.top <= s.keep * (s.experts / s.groups) && s.width > 0 && s.ff > 0 && s.shared_ff >= 0 && gate_smem(s) <= kRtMaxSmem && down_smem(s) <= kRtMaxSmem;
 }
 size_t routed_scratch_bytes(const RoutedShape& s, int m, bool f32) { return layout(s, m, f32).total; }
 
@@ -345,9 +383,13 @@ int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches) {
     const RoutedScratch l = layout(a.shape, a.m, a.f32);
     RoutedParams p{};
     p.sh = a.shape; p.scale = a.scale; p.act = a.act; p.m = a.m; p.x = a.x; p.x_stride = a.x_stride; p.z = a.z; p.z_stride = a.z_stride;
-    p.gate = a.gate->data; p.up = a.up->data; p.down = a.down->data; p.in_ld = a.gate->ld; p.mid_ld = a.down->ld; p.out = a.out; p.out_stride = a.out_stride;
+    p.softmax = a.softmax; p.group_best = a.group_best; p.raw_weights = a.raw_weights;
+    p.gate = a.gate ? a.gate->data : nullptr; p.up = a.up->data; p.down = a.down->data; p.in_ld = a.up->ld; p.mid_ld = a.down->ld; p.out = a.out; p.out_stride = a.out_stride;
     p.sel = reinterpret_cast<int*>(a.scratch + l.sel); p.weight = reinterpret_cast<float*>(a.scratch + l.weight); p.rank = reinterpret_cast<int*>(a.scratch + l.rank);
     p.counts = a.counts; p.mid = a.scratch + l.mid; p.mid_stride = up8(a.shape.ff);
+    const bool shared = a.shape.shared_ff > 0;
+    if (shared) { p.shared_up = a.shared_up->data; p.shared_down = a.shared_down->data; p.shared_ld = a.shared_down->ld; }
+    p.shared_mid = a.scratch + l.shared_mid; p.shared_stride = up8(a.shape.shared_ff);
     if (few(a.m, a.f32)) return a.f32 ? few_rows<float>(p, s, launches) : few_rows<__nv_bfloat16>(p, s, launches);
 
     const int all = a.m * a.shape.top, E = a.shape.experts;
@@ -360,17 +402,34 @@ int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches) {
     e = launch_k(routed_sort_kernel, dim3(std::min((all + kRtWarps - 1) / kRtWarps, 4 * 148)), dim3(kRtThreads), 0, s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed sort launch");
     ProductLaunch g;
-    g.w = a.gate; g.w2 = a.up; g.act = a.act; g.m = all; g.x = p.sorted; g.x_stride = p.sorted_stride; g.status = a.status;
+    if (a.gate) { g.w = a.gate; g.w2 = a.up; g.act = a.act; }
+    else { g.w = a.up; g.out.gelu = 1; }
+    g.m = all; g.x = p.sorted; g.x_stride = p.sorted_stride; g.status = a.status;
     g.experts = E; g.tiles = p.tiles; g.max_tiles = p.max_tiles; g.group_bn = p.bn;
     g.out.y[0] = p.mid; g.out.stride[0] = p.mid_stride;
     for (int& end : g.out.end) end = a.shape.ff;
     int rc = launch_product(g, s);
     if (rc) return rc;
     ProductLaunch d = g;
-    d.w = a.down; d.w2 = nullptr; d.x = p.mid; d.x_stride = p.mid_stride;
+    d.w = a.down; d.w2 = nullptr; d.out.gelu = 0; d.x = p.mid; d.x_stride = p.mid_stride;
     d.out.y[0] = p.y; d.out.stride[0] = p.y_stride; d.out.f32[0] = 1;
     for (int& end : d.out.end) end = a.shape.width;
     if ((rc = launch_product(d, s))) return rc;
+    if (shared) {
+        ProductLaunch u;
+        u.w = a.shared_up; u.m = a.m; u.x = a.x; u.x_stride = a.x_stride; u.part = a.part; u.part_floats = a.part_floats; u.status = a.status;
+        u.out.y[0] = p.shared_mid; u.out.stride[0] = p.shared_stride; u.out.gelu = 1;
+        for (int& end : u.out.end) end = a.shape.shared_ff;
+        if ((rc = launch_product(u, s))) return rc;
+        *launches += product_launch_count(u);
+        ProductLaunch w = u;
+        w.w = a.shared_down; w.x = p.shared_mid; w.x_stride = p.shared_stride;
+        p.shared_y = reinterpret_cast<const float*>(a.scratch + l.shared_y); p.shared_y_stride = up8(a.shape.width);
+        w.out.y[0] = a.scratch + l.shared_y; w.out.stride[0] = p.shared_y_stride; w.out.f32[0] = 1; w.out.gelu = 0;
+        for (int& end : w.out.end) end = a.shape.width;
+        if ((rc = launch_product(w, s))) return rc;
+        *launches += product_launch_count(w);
+    }
     e = launch_k(routed_sum_kernel, dim3((a.shape.width + kRtThreads * 4 - 1) / (kRtThreads * 4), a.m), dim3(kRtThreads), 0, s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed sum launch");
     *launches += 5;

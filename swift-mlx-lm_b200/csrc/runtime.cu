@@ -1293,6 +1293,8 @@ int swlm_ctx_create(int device_id, int tp_rank, int tp_size, swlm_ctx** out) {
     if (!rc) rc = bgemm_init();
     if (!rc) rc = latent_init();
     if (!rc) rc = routed_init();
+    if (!rc) rc = grouped_init();
+    if (!rc) rc = retention_init();
     if (rc) { cudaStreamDestroy(ctx->stream); delete ctx; return rc; }
     *out = ctx;
     return SWLM_OK;
@@ -1467,7 +1469,7 @@ int swlm_plan_build(swlm_ctx* ctx, const swlm_step* steps, int n_steps, const sw
     if (desc->max_batch < 1 || desc->max_batch > kMaxSequences) { set_error("max_batch %d outside 1..%d", desc->max_batch, kMaxSequences); return SWLM_ERR_INVALID; }
     if (desc->max_batch > kQGemvMaxRows && ctx->tp_size > 1) { set_error("more than %d sequences per step are not supported under tensor parallelism", kQGemvMaxRows); return SWLM_ERR_UNSUPPORTED; }
     const bool stream = desc->stream_dtype != 0;
-    if (stream && (desc->max_seq < 1 || desc->hidden < 1 || desc->vocab < 1 || desc->latent_layers < 0 || desc->delta_layers < 0 || desc->kv_pool_tokens < 0 || desc->kv_layers || desc->conv_layers || desc->ssm_layers)) {
+    if (stream && (desc->max_seq < 1 || desc->hidden < 1 || desc->vocab < 1 || desc->latent_layers < 0 || desc->delta_layers < 0 || desc->grouped_layers < 0 || desc->kv_pool_tokens < 0 || desc->kv_layers || desc->conv_layers || desc->ssm_layers)) {
         set_error("fp32-stream plan: bad sizes, or layers with bf16 state");
         return SWLM_ERR_INVALID;
     }
@@ -2328,6 +2330,8 @@ static int profiled_launch_kind(int step_kind, int* kind) {
     case SWLM_STEP_LATENT_ATTN: *kind = L_LATENT; break;
     case SWLM_STEP_GATED_DELTA: *kind = L_DELTA; break;
     case SWLM_STEP_ROUTED_MLP: *kind = L_ROUTED; break;
+    case SWLM_STEP_GROUPED_ATTN: *kind = L_GROUPED; break;
+    case SWLM_STEP_RETENTION: *kind = L_RETENTION; break;
     case SWLM_STEP_RESADD_COPY_RMSNORM: *kind = L_RMSNORM; break;
     default: set_error("profile: step kind %d has no per-kind loop", step_kind); return SWLM_ERR_UNSUPPORTED;
     }

@@ -1,7 +1,7 @@
 // Executor of fp32-stream plans: step list -> launches, the paged pool of latent rows, and one row executor that runs decode
 // steps, prompt chunks and mixed batches alike. A batch is a list of rows, each with its token, sequence and position; the
-// only steps that look beyond their own row are latent attention, which finds the cached rows through the page table, and
-// the gated delta rule, which carries a state per sequence.
+// only steps that look beyond their own row are latent and grouped attention, which find the cached rows through the page table,
+// and the gated delta rule and retention, which carry a state per sequence.
 #include <cmath>
 #include <cstdio>
 #include <cstring>
@@ -47,6 +47,7 @@ int concat_matrices(swlm_ctx* ctx, const std::vector<std::string>& names, const 
     size_t row = 0;
     for (const std::string& nm : names) {
         Matrix& m = ctx->matrices.at(nm);
+        if (m.ld != cat.ld) { set_error("matrix '%s' is already part of a product over side-by-side matrices", nm.c_str()); return SWLM_ERR_UNSUPPORTED; }
         SWLM_CUDA(cudaMemcpy(cat.data + row * cat.ld, m.data, (size_t)m.n * m.ld * 2, cudaMemcpyDeviceToDevice));
         if (!m.view) {
             // plans built earlier may hold the old address: their kernels are ordered before the free by the device
@@ -63,18 +64,47 @@ int concat_matrices(swlm_ctx* ctx, const std::vector<std::string>& names, const 
     return SWLM_OK;
 }
 
+// Two matrices side by side, the second from a multiple of 8 columns on; both become views of the result.
+int join_matrices(swlm_ctx* ctx, const char* left, const char* right, const Matrix** out) {
+    const std::string key = std::string(left) + "&" + right;
+    auto hit = ctx->matrix_cat.find(key);
+    if (hit != ctx->matrix_cat.end()) { *out = &hit->second; return SWLM_OK; }
+    Matrix* part[2] = {&ctx->matrices.at(left), &ctx->matrices.at(right)};
+    const int at[2] = {0, (part[0]->k + 7) / 8 * 8};
+    Matrix both;
+    both.n = part[0]->n; both.k = at[1] + part[1]->k; both.ld = (both.k + 7) / 8 * 8;
+    if (part[0]->view || part[1]->view || !strcmp(left, right)) { set_error("matrices '%s' and '%s' are already part of a concatenated matrix", left, right); return SWLM_ERR_UNSUPPORTED; }
+    const int rc = dev_alloc(&both.data, (size_t)both.n * both.ld, &ctx->bytes);
+    if (rc) return rc;
+    SWLM_CUDA(cudaMemset(both.data, 0, (size_t)both.n * both.ld * 2));
+    for (int i = 0; i < 2; ++i) {
+        Matrix& m = *part[i];
+        SWLM_CUDA(cudaMemcpy2D(both.data + at[i], (size_t)both.ld * 2, m.data, (size_t)m.ld * 2, (size_t)m.k * 2, m.n, cudaMemcpyDeviceToDevice));
+        SWLM_CUDA(cudaDeviceSynchronize());
+        cudaFree(m.data);
+        ctx->bytes -= (int64_t)m.n * m.ld * 2;
+        m.data = both.data + at[i];
+        m.ld = both.ld;
+        m.view = true;
+    }
+    ctx->matrix_cat[key] = both;
+    *out = &ctx->matrix_cat[key];
+    return SWLM_OK;
+}
+
 // Angle per position of every pair, interpolated by parts when the step says so, in double precision on the host.
 int stream_rope_table(swlm_plan* plan, const swlm_step& st, int* index) {
+    const float divisor = st.rope_divisor > 0.f ? st.rope_divisor : 1.f;
     for (size_t i = 0; i < plan->rope_tables.size(); ++i) {
         const RopeTable& t = plan->rope_tables[i];
-        if (t.rope_dim == st.rope_dim && t.base == st.rope_base && t.factor == st.rope_factor && t.original == st.rope_original &&
+        if (t.divisor == divisor && t.rope_dim == st.rope_dim && t.base == st.rope_base && t.factor == st.rope_factor && t.original == st.rope_original &&
             t.fast == st.rope_fast && t.slow == st.rope_slow) { *index = (int)i; return SWLM_OK; }
     }
     const int half = st.rope_dim / 2;
     std::vector<float> f(std::max(1, half));
     const double base = st.rope_base, dims = st.rope_dim;
     RopeTable t;
-    t.rope_dim = st.rope_dim; t.base = st.rope_base; t.factor = st.rope_factor; t.original = st.rope_original; t.fast = st.rope_fast; t.slow = st.rope_slow;
+    t.rope_dim = st.rope_dim; t.base = st.rope_base; t.factor = st.rope_factor; t.original = st.rope_original; t.fast = st.rope_fast; t.slow = st.rope_slow; t.divisor = divisor;
     double lo = 0, hi = 0;
     if (st.rope_factor > 0.f) {
         auto dim_of = [&](double turns) { return dims * std::log((double)st.rope_original / (2.0 * M_PI * turns)) / (2.0 * std::log(base)); };
@@ -85,7 +115,7 @@ int stream_rope_table(swlm_plan* plan, const swlm_step& st, int* index) {
     for (int i = 0; i < half; ++i) {
         const double plain = std::pow(base, -2.0 * i / dims);
         const double ramp = st.rope_factor > 0.f ? std::min(1.0, std::max(0.0, (i - lo) / std::max(hi - lo, 0.001))) : 0.0;
-        f[i] = (float)(ramp > 0.0 ? plain / st.rope_factor * ramp + plain * (1.0 - ramp) : plain);
+        f[i] = (float)((ramp > 0.0 ? plain / st.rope_factor * ramp + plain * (1.0 - ramp) : plain) / divisor);
     }
     int rc = dev_alloc(&t.inv_freq, f.size());
     if (rc) return rc;
@@ -113,6 +143,8 @@ GatedAct glu_of(const swlm_step& s) {
     a.limit = s.limit;
     return a;
 }
+RoutedShape routed_shape(const swlm_step& s) { return RoutedShape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k, s.weight5[0] ? s.k2 : 0}; }
+DeltaShape retention_shape(const swlm_step& s) { return DeltaShape{s.heads, s.heads, s.key_dim, s.value_dim, 0}; }
 const char* glu_name(int kind) { return kind == GATED_ACT_GELU_TANH ? "geglu" : kind == GATED_ACT_CLAMPED ? "clamped glu" : "swiglu"; }
 
 }  // namespace
@@ -125,7 +157,13 @@ int stream_compile(swlm_plan* plan) {
     if (d.stream_dtype < 0 || d.stream_dtype > SWLM_STREAM_ALL_F32) { set_error("stream_dtype %d", d.stream_dtype); return SWLM_ERR_INVALID; }
     int rc;
     auto widen = [&](int buf, int n) { plan->stream_width[buf] = std::max(plan->stream_width[buf], (n + 7) / 8 * 8); };
+    auto window_set = [&](int window) {
+        const int at = (int)(std::find(plan->windows.begin(), plan->windows.end(), window) - plan->windows.begin());
+        if (at == (int)plan->windows.size()) plan->windows.push_back(window);
+        return at;
+    };
     plan->latent.assign(std::max(0, d.latent_layers), LatentLayer{});
+    plan->grouped.assign(std::max(0, d.grouped_layers), GroupedLayer{});
     plan->delta.assign(std::max(0, d.delta_layers), DeltaLayer{});
     widen(SWLM_BUF_HIDDEN, d.hidden);
     widen(SWLM_BUF_RESIDUAL, d.hidden);
@@ -150,6 +188,12 @@ int stream_compile(swlm_plan* plan) {
             if (s.in_buf != SWLM_BUF_HIDDEN || !act_buf(plan, s.out_buf) || s.n != d.hidden) { set_error("norm '%s': reads hidden, writes scratch 0..2, width %d", s.weight, d.hidden); return SWLM_ERR_INVALID; }
             if ((rc = find_vector(ctx, is_postnorm(s.kind) ? s.weight2 : s.weight, s.n, &L.d1))) return rc;
             if (is_postnorm(s.kind) && (rc = find_vector(ctx, s.weight, s.n, &L.norm_post))) return rc;
+            if (is_postnorm(s.kind) && s.weight3[0]) {   // an embedding row joins
+                auto it = ctx->dense.find(s.weight3);
+                if (it == ctx->dense.end()) { set_error("embedding table '%s' missing", s.weight3); return SWLM_ERR_NOT_FOUND; }
+                if (it->second.cols != s.n || it->second.rows != d.vocab) { set_error("norm '%s': table '%s' is %lld x %lld", s.weight, s.weight3, (long long)it->second.rows, (long long)it->second.cols); return SWLM_ERR_INVALID; }
+                L.dv[0] = &it->second;
+            }
             widen(s.out_buf, s.n);
             L.label = std::string(is_postnorm(s.kind) ? "postnorm+rmsnorm " : "rmsnorm ") + (is_postnorm(s.kind) ? s.weight2 : s.weight);
             break;
@@ -157,11 +201,21 @@ int stream_compile(swlm_plan* plan) {
             L.kind = L_PRODUCT;
             if (!act_buf(plan, s.in_buf) || !any_buf(s.out_buf) || s.out_buf == s.in_buf || s.out_buf == SWLM_BUF_RESIDUAL) { set_error("product '%s': bad buffers", s.weight); return SWLM_ERR_INVALID; }
             if ((rc = find_matrix(ctx, s.weight, s.n, s.k, &L.m1))) return rc;
+            if (s.weight2[0]) {   // side by side with a second matrix
+                const Matrix* right;
+                if (s.k2 <= 0 || s.in_off < 0 || s.out_off < 0 || (s.in_off & 7)) { set_error("product '%s': bad columns", s.weight); return SWLM_ERR_INVALID; }
+                if ((rc = find_matrix(ctx, s.weight2, s.n, s.k2, &right)) || (rc = join_matrices(ctx, s.weight, s.weight2, &L.m1))) return rc;
+                widen(s.in_buf, s.in_off + L.m1->k);
+                widen(s.out_buf, s.out_off + s.n);
+                L.seg_buf[0] = s.out_buf; L.seg_off[0] = s.out_off; L.seg_end[0] = s.n;
+                L.label = std::string("product ") + s.weight + " & " + s.weight2;
+                break;
+            }
             if (s.in_off < 0 || s.out_off < 0 || (s.in_off & 7) || (s.out_buf == SWLM_BUF_LOGITS && s.out_off)) { set_error("product '%s': input columns start at multiples of 8", s.weight); return SWLM_ERR_INVALID; }
             widen(s.in_buf, s.in_off + s.k);
             widen(s.out_buf, s.out_off + s.n);
             // gate, up, gated activation -> one launch
-            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && is_glu(st[i + 2].kind) && !s.in_off && !s.out_off && !st[i + 1].in_off && !st[i + 1].out_off &&
+            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && !st[i + 1].weight2[0] && is_glu(st[i + 2].kind) && !s.in_off && !s.out_off && !st[i + 1].in_off && !st[i + 1].out_off &&
                 st[i + 1].in_buf == s.in_buf && st[i + 1].k == s.k && st[i + 1].n == s.n && st[i + 2].in_buf == s.out_buf &&
                 st[i + 2].in2_buf == st[i + 1].out_buf && st[i + 2].n == s.n && act_buf(plan, st[i + 2].out_buf) && st[i + 2].out_buf != s.in_buf &&
                 act_buf(plan, s.out_buf) && act_buf(plan, st[i + 1].out_buf)) {
@@ -186,7 +240,7 @@ int stream_compile(swlm_plan* plan) {
                 break;
             }
             size_t j = i + 1;
-            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && st[j].in_buf == s.in_buf && st[j].in_off == s.in_off && st[j].k == s.k &&
+            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && !st[j].weight2[0] && st[j].in_buf == s.in_buf && st[j].in_off == s.in_off && st[j].k == s.k &&
                    st[j].out_off >= 0 && st[j].out_buf != s.in_buf && any_buf(st[j].out_buf) && st[j].out_buf != SWLM_BUF_LOGITS && s.out_buf != SWLM_BUF_LOGITS) {
                 bool clash = false;
                 for (size_t q = i; q < j; ++q)
@@ -231,8 +285,7 @@ int stream_compile(swlm_plan* plan) {
             if ((rc = stream_rope_table(plan, s, &L.rope_table))) return rc;
             if (s.window_left < 0) { set_error("latent attention: window %d", s.window_left); return SWLM_ERR_INVALID; }
             if (s.weight4[0] && (rc = find_vector(ctx, s.weight4, s.heads, &L.dv[0]))) return rc;
-            L.window_set = (int)(std::find(plan->windows.begin(), plan->windows.end(), s.window_left) - plan->windows.begin());
-            if (L.window_set == (int)plan->windows.size()) plan->windows.push_back(s.window_left);
+            L.window_set = window_set(s.window_left);
             LatentLayer& ll = plan->latent[s.layer];
             if (ll.rank && (ll.rank != s.n || ll.rot != s.key_dim)) { set_error("latent layer %d is used with two row sizes", s.layer); return SWLM_ERR_INVALID; }
             ll.rank = s.n; ll.rot = s.key_dim; ll.row = latent_row(s.n, s.key_dim, plan->all_f32());
@@ -270,12 +323,14 @@ int stream_compile(swlm_plan* plan) {
         }
         case SWLM_STEP_ROUTED_MLP: {
             L.kind = L_ROUTED;
-            const RoutedShape shape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k};
-            if (!routed_supported(shape)) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k); return SWLM_ERR_UNSUPPORTED; }
+            const bool gated = s.weight2[0], shared = s.weight5[0];
+            const RoutedShape shape = routed_shape(s);
+            if (!routed_supported(shape) || (shared && s.k2 <= 0)) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d, shared %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k, s.k2); return SWLM_ERR_UNSUPPORTED; }
+            if (s.score_act < 0 || s.score_act > SWLM_SCORE_SOFTMAX || s.group_best < 0 || s.group_best > 2) { set_error("routed feed-forward: scores %d, group %d", s.score_act, s.group_best); return SWLM_ERR_UNSUPPORTED; }
             if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || s.out_buf != SWLM_BUF_HIDDEN || s.n != d.hidden) { set_error("routed feed-forward: input in scratch 0..2, logits in scratch 3 or 4, result in hidden"); return SWLM_ERR_INVALID; }
             const char* suffix[3] = {s.weight2, s.weight3, s.weight4};
             const Matrix** into[3] = {&L.m1, &L.m2, &L.m3};
-            for (int q = 0; q < 3; ++q) {
+            for (int q = gated ? 0 : 1; q < 3; ++q) {
                 std::vector<std::string> names;
                 for (int e = 0; e < s.experts; ++e) {
                     names.push_back(std::string(s.weight) + std::to_string(e) + suffix[q]);
@@ -284,11 +339,53 @@ int stream_compile(swlm_plan* plan) {
                 }
                 if ((rc = concat_matrices(ctx, names, into[q]))) return rc;
             }
+            if (shared && ((rc = find_matrix(ctx, s.weight5, s.k2, s.n, &L.m4)) || (rc = find_matrix(ctx, s.weight6, s.n, s.k2, &L.m5)))) return rc;
             L.act.kind = GATED_ACT_CLAMPED; L.act.alpha = s.glu_alpha; L.act.limit = s.limit;
             widen(s.in_buf, s.n);
-            widen(s.in2_buf, s.experts);
+            widen(s.in2_buf, s.experts + (shared ? 1 : 0));
             widen(s.out_buf, s.n);
             L.label = std::string("routed_mlp ") + s.weight;
+            break;
+        }
+        case SWLM_STEP_GROUPED_ATTN: {
+            L.kind = L_GROUPED;
+            if (s.layer < 0 || s.layer >= d.grouped_layers) { set_error("grouped attention: layer %d outside the pool", s.layer); return SWLM_ERR_INVALID; }
+            if (s.heads <= 0 || s.kv_heads <= 0 || s.heads % s.kv_heads || s.head_dim <= 0 || s.value_dim <= 0 || s.rope_dim < 0 || s.rope_dim > s.head_dim || (s.rope_dim & 1) ||
+                s.window_left < 0 || s.chunk < 0) { set_error("grouped attention: bad sizes"); return SWLM_ERR_INVALID; }
+            if (!act_buf(plan, s.in_buf) || !act_buf(plan, s.out_buf) || s.out_buf == s.in_buf || s.in_off < 0 || (s.in_off & 7) || s.out_off < 0 || (s.out_off & 7) ||
+                (s.in3_buf != SWLM_BUF_NONE && (!any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf)))) { set_error("grouped attention: q | k | v and the result in scratch 0..2 from columns that are multiples of 8, gate in scratch 3 or 4"); return SWLM_ERR_INVALID; }
+            if (s.weight[0] && (rc = find_vector(ctx, s.weight, s.head_dim, &L.dv[0]))) return rc;
+            if (s.weight2[0] && (rc = find_vector(ctx, s.weight2, s.head_dim, &L.dv[1]))) return rc;
+            const GroupedRow row = grouped_row(s.kv_heads, s.head_dim, s.value_dim, plan->all_f32());
+            if (!grouped_supported(row)) { set_error("grouped attention: heads of %d and %d", s.head_dim, s.value_dim); return SWLM_ERR_UNSUPPORTED; }
+            if ((rc = stream_rope_table(plan, s, &L.rope_table))) return rc;
+            L.window_set = window_set(s.window_left);
+            GroupedLayer& gl = plan->grouped[s.layer];
+            if (gl.row.groups && memcmp(&gl.row, &row, sizeof(row))) { set_error("grouped layer %d is used with two row sizes", s.layer); return SWLM_ERR_INVALID; }
+            gl.row = row;
+            widen(s.in_buf, s.in_off + (s.heads + s.kv_heads) * s.head_dim + s.kv_heads * s.value_dim);
+            if (s.in3_buf != SWLM_BUF_NONE) widen(s.in3_buf, s.heads);
+            widen(s.out_buf, s.out_off + s.heads * s.value_dim);
+            L.label = std::string("grouped_attention ") + s.weight;
+            break;
+        }
+        case SWLM_STEP_RETENTION: {
+            L.kind = L_RETENTION;
+            if (s.layer < 0 || s.layer >= d.delta_layers) { set_error("retention: layer %d has no state", s.layer); return SWLM_ERR_INVALID; }
+            if (!retention_supported(s.heads, s.key_dim, s.value_dim)) { set_error("retention: %d heads of %d x %d", s.heads, s.key_dim, s.value_dim); return SWLM_ERR_UNSUPPORTED; }
+            if (!act_buf(plan, s.in_buf) || !act_buf(plan, s.in4_buf) || !act_buf(plan, s.out_buf) || s.out_buf == s.in_buf || s.out_buf == s.in4_buf || s.in_off < 0 || s.in4_off < 0 || s.out_off < 0 ||
+                ((s.in_off | s.in4_off | s.out_off) & 7)) { set_error("retention: q | k | v, gate and result in scratch 0..2, from columns that are multiples of 8"); return SWLM_ERR_INVALID; }
+            auto decay = ctx->densef.find(s.weight);
+            if (decay == ctx->densef.end() || decay->second.count != s.heads) { set_error("retention: decays '%s' missing or not one per head", s.weight); return SWLM_ERR_NOT_FOUND; }
+            L.f1 = &decay->second;
+            DeltaLayer& dl = plan->delta[s.layer];
+            const DeltaShape shape = retention_shape(s);
+            if (dl.shape.heads && memcmp(&dl.shape, &shape, sizeof(shape))) { set_error("state %d is used with two shapes", s.layer); return SWLM_ERR_INVALID; }
+            dl.shape = shape;
+            widen(s.in_buf, s.in_off + s.heads * (2 * s.key_dim + s.value_dim));
+            widen(s.in4_buf, s.in4_off + s.heads * s.value_dim);
+            widen(s.out_buf, s.out_off + s.heads * s.value_dim);
+            L.label = std::string("retention ") + s.weight;
             break;
         }
         case SWLM_STEP_SOFTCAP:
@@ -310,8 +407,10 @@ int stream_compile(swlm_plan* plan) {
     }
     for (int l = 0; l < d.latent_layers; ++l)
         if (!plan->latent[l].rank && st.size() > 1) { set_error("latent layer %d has no step", l); return SWLM_ERR_INVALID; }
+    for (int l = 0; l < d.grouped_layers; ++l)
+        if (!plan->grouped[l].row.groups && st.size() > 1) { set_error("grouped layer %d has no step", l); return SWLM_ERR_INVALID; }
     for (int l = 0; l < d.delta_layers; ++l)
-        if (!plan->delta[l].shape.heads && st.size() > 1) { set_error("gated-delta layer %d has no step", l); return SWLM_ERR_INVALID; }
+        if (!plan->delta[l].shape.heads && st.size() > 1) { set_error("state %d has no step", l); return SWLM_ERR_INVALID; }
 
     // A norm rides with the product behind it when that is its only reader: few rows compute it in the product's prologue,
     // more rows run it in front.
@@ -328,7 +427,7 @@ int stream_compile(swlm_plan* plan) {
             if (writes) break;
         }
         if (!ok) continue;
-        B.norm = A.st; B.norm_w = A.d1; B.norm_post = A.norm_post;
+        B.norm = A.st; B.norm_w = A.d1; B.norm_post = A.norm_post; B.dv[0] = A.dv[0];
         B.label = A.label + " + " + B.label;
         B.steps_covered += 1;
         plan->launches.erase(plan->launches.begin() + i);
@@ -430,13 +529,12 @@ int bufs_rows(swlm_state* s, StreamBufs* b, int rows, int wants) {
     return SWLM_OK;
 }
 
-RoutedShape routed_shape(const swlm_step& s) { return RoutedShape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k}; }
-
 size_t part_need(const swlm_plan* plan, int rows, int wants) {
     size_t need = 0;
     if (plan->all_f32()) return 0;
     for (const Launch& L : plan->launches)
         if (L.kind == L_PRODUCT) need = std::max(need, product_part_floats(L.m1->n, L.m1->k, L.seg_buf[0] == SWLM_BUF_LOGITS ? wants : rows, L.m2 != nullptr));
+        else if (L.kind == L_ROUTED && L.m4) need = std::max(need, std::max(product_part_floats(L.m4->n, L.m4->k, rows, false), product_part_floats(L.m5->n, L.m5->k, rows, false)));
     return need;
 }
 
@@ -459,6 +557,8 @@ int bufs_scratch(swlm_state* s, StreamBufs* b, const RowBatch& r) {
         if (L.kind == L_DELTA) {
             const DeltaShape& sh = plan->delta[L.st.layer].shape;
             if (r.n_runs || (r.n_single && !delta_step_fits(sh))) delta = std::max(delta, delta_scratch_floats(sh, std::max(r.n_blocks, r.n_single), r.rows));
+        } else if (L.kind == L_RETENTION) {
+            if (r.n_runs || (r.n_single && !retention_step_fits(L.st.key_dim, L.st.value_dim))) delta = std::max(delta, (size_t)r.rows * L.st.heads * L.st.value_dim);
         } else if (L.kind == L_ROUTED) routed = std::max(routed, routed_scratch_bytes(routed_shape(L.st), r.rows, plan->all_f32()));
     }
     if ((rc = grow(&b->delta, &b->delta_cap, delta, s->stream))) return rc;
@@ -480,7 +580,8 @@ void bufs_free(StreamBufs* b) {
 
 float* residual(StreamBufs* b, int phys) { return phys ? b->res2 : static_cast<float*>(b->buf[SWLM_BUF_RESIDUAL]); }
 
-StreamNorm norm_of(swlm_state* s, StreamBufs* b, const swlm_step& st, const DenseTensor* w, const DenseTensor* post, int res_in, int res_out) {
+StreamNorm norm_of(swlm_state* s, StreamBufs* b, const RowBatch& r, const Launch& L, const swlm_step& st, const DenseTensor* w, int res_in, int res_out) {
+    const DenseTensor* post = L.norm_post;
     StreamNorm n;
     n.mode = st.kind;
     n.in = static_cast<const float*>(b->buf[st.in_buf]); n.in_stride = s->width[st.in_buf];
@@ -489,6 +590,7 @@ StreamNorm norm_of(swlm_state* s, StreamBufs* b, const swlm_step& st, const Dens
     if (norm_stores(st.kind)) n.res_out = residual(b, res_out);
     n.w = w->data; n.w_post = post ? post->data : nullptr;
     n.eps = st.eps; n.weight_bias = st.weight_bias;
+    if (L.dv[0]) { n.table = L.dv[0]->data; n.tokens = r.tok; n.vocab = s->plan->desc.vocab; n.table_scale = st.scale; }
     return n;
 }
 
@@ -501,11 +603,12 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
     const int wants = body_only ? 0 : r.wants;
     bool advanced = false;
     int rc = SWLM_OK;
+    auto column = [plan](StreamBufs* bufs, int buf, int off) -> void* { return static_cast<unsigned char*>(bufs->buf[buf]) + (size_t)off * stored_bytes(plan, buf); };
     s->last_bufs = b;
     s->last_res = plan->final_res;
     for (const Launch& L : plan->launches) {
         const swlm_step& st = L.st;
-        const bool latent_kernel = only_kind == L_ATTN && L.kind == L_LATENT;
+        const bool latent_kernel = only_kind == L_ATTN && (L.kind == L_LATENT || L.kind == L_GROUPED);
         if (only_kind >= 0 && L.kind != only_kind && !latent_kernel) continue;
         switch (L.kind) {
         case L_EMBED:
@@ -513,7 +616,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             s->launches += 1;
             break;
         case L_RMSNORM:
-            rc = launch_stream_norm(norm_of(s, b, st, L.d1, L.norm_post, L.res_in, L.res_out), r.rows, st.n, nullptr, b->buf[st.out_buf], s->width[st.out_buf], f32, stream);
+            rc = launch_stream_norm(norm_of(s, b, r, L, st, L.d1, L.res_in, L.res_out), r.rows, st.n, nullptr, b->buf[st.out_buf], s->width[st.out_buf], f32, stream);
             s->launches += 1;
             break;
         case L_PRODUCT: {
@@ -527,7 +630,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.part = b->part; a.part_floats = b->part_cap; a.status = s->pf_status;
             if (head && idx && !L.norm.kind) { set_error("the output head must follow a norm that nothing else reads"); return SWLM_ERR_UNSUPPORTED; }
             if (L.norm.kind) {
-                const StreamNorm n = norm_of(s, b, L.norm, L.norm_w, L.norm_post, L.res_in, L.res_out);
+                const StreamNorm n = norm_of(s, b, r, L, L.norm, L.norm_w, L.res_in, L.res_out);
                 if (!idx && product_takes_norm(m, L.m1->k)) a.norm = n;
                 else {
                     rc = launch_stream_norm(n, m, L.norm.n, idx, b->buf[st.in_buf], s->width[st.in_buf], f32, stream);
@@ -595,7 +698,9 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.shape = routed_shape(st); a.scale = st.scale; a.act = L.act; a.m = r.rows; a.f32 = f32;
             a.x = b->buf[st.in_buf]; a.x_stride = s->width[st.in_buf];
             a.z = static_cast<const float*>(b->buf[st.in2_buf]); a.z_stride = s->width[st.in2_buf];
-            a.gate = L.m1; a.up = L.m2; a.down = L.m3;
+            a.gate = L.m1; a.up = L.m2; a.down = L.m3; a.shared_up = L.m4; a.shared_down = L.m5;
+            a.softmax = st.score_act == SWLM_SCORE_SOFTMAX; a.group_best = st.group_best == 1 ? 1 : 2; a.raw_weights = st.raw_weights;
+            a.part = b->part; a.part_floats = b->part_cap;
             a.out = static_cast<float*>(b->buf[st.out_buf]); a.out_stride = s->width[st.out_buf];
             a.scratch = b->routed; a.counts = s->routed_counts; a.status = s->pf_status;
             int n = 0;
@@ -603,11 +708,46 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             s->launches += n;
             break;
         }
+        case L_GROUPED: {
+            GroupedLaunch a;
+            const RopeTable& rope = plan->rope_tables[L.rope_table];
+            a.row = plan->grouped[st.layer].row;
+            a.heads = st.heads; a.rot_dims = st.rope_dim; a.rot_neighbours = st.rope_pairs == SWLM_ROPE_NEIGHBOURS; a.window = st.window_left; a.chunk = st.chunk; a.sink_one = st.sink_one;
+            a.scale = st.scale; a.eps = st.eps; a.weight_bias = st.weight_bias; a.magnitude = rope.magnitude; a.inv_freq = rope.inv_freq; a.out_scale = st.out_scale; a.f32 = f32;
+            a.q_norm = L.dv[0] ? L.dv[0]->data : nullptr; a.k_norm = L.dv[1] ? L.dv[1]->data : nullptr;
+            a.qkv = column(b, st.in_buf, st.in_off); a.qkv_stride = s->width[st.in_buf];
+            if (st.in3_buf != SWLM_BUF_NONE) { a.gate = static_cast<const float*>(b->buf[st.in3_buf]); a.gate_stride = s->width[st.in3_buf]; }
+            a.pool = s->pool[plan->latent.size() + st.layer]; a.page_table = s->page_table; a.pages_per_seq = s->pages_per_seq;
+            a.row_seq = r.seq; a.row_pos = r.pos;
+            a.out = column(b, st.out_buf, st.out_off); a.out_stride = s->width[st.out_buf];
+            a.n_rows = r.rows; a.n_short = r.n_short; a.short_rows = r.short_rows; a.max_pages = r.splits_pages;
+            a.n_tiles = r.n_tiles; a.tiles = r.tiles; a.status = s->pf_status; a.only_attention = latent_kernel;
+            if (r.n_spans) a.spans = r.spans[L.window_set];
+            int n = 0;
+            rc = launch_grouped(a, stream, &n);
+            s->launches += n;
+            break;
+        }
+        case L_RETENTION: {
+            RetentionLaunch a;
+            a.heads = st.heads; a.dim = st.key_dim; a.vdim = st.value_dim; a.eps = st.eps; a.scale = st.scale; a.out_scale = st.out_scale; a.f32 = f32;
+            a.decay = L.f1->data;
+            a.qkv = column(b, st.in_buf, st.in_off); a.qkv_stride = s->width[st.in_buf];
+            a.gate = column(b, st.in4_buf, st.in4_off); a.gate_stride = s->width[st.in4_buf];
+            a.state = s->delta_state[st.layer]; a.row_seq = r.seq; a.row_pos = r.pos;
+            a.out = column(b, st.out_buf, st.out_off); a.out_stride = s->width[st.out_buf];
+            a.n_single = r.n_single; a.single_rows = r.single_rows; a.n_runs = r.n_runs; a.runs = r.runs; a.n_blocks = r.n_blocks; a.block_run = r.block_run;
+            a.scratch = b->delta;
+            int n = 0;
+            rc = launch_retention(a, stream, &n);
+            s->launches += n;
+            break;
+        }
         case L_LATENT: {
             LatentLaunch a;
             const RopeTable& rope = plan->rope_tables[L.rope_table];
             a.row = plan->latent[st.layer].row;
-            a.heads = st.heads; a.dim = st.head_dim; a.vdim = st.value_dim; a.rot_dims = st.rope_dim;
+            a.heads = st.heads; a.dim = st.head_dim; a.vdim = st.value_dim; a.rot_dims = st.rope_dim; a.rot_neighbours = st.rope_pairs == SWLM_ROPE_NEIGHBOURS;
             a.scale = st.scale; a.eps = st.eps; a.weight_bias = st.weight_bias; a.magnitude = rope.magnitude; a.inv_freq = rope.inv_freq; a.f32 = f32;
             a.window = st.window_left; a.sink = L.dv[0] ? L.dv[0]->data : nullptr;
             a.q = b->buf[st.in_buf]; a.q_stride = s->width[st.in_buf];
@@ -692,6 +832,14 @@ int stream_state_create(swlm_state* s) {
         // a page is read whole: rows nobody has written must hold finite numbers
         if (bytes) SWLM_CUDA(cudaMemset(p, 0, bytes));
     }
+    for (const GroupedLayer& l : plan->grouped) {
+        const size_t bytes = (size_t)s->pool_pages * l.row.groups * l.row.block * elem;
+        unsigned char* p = nullptr;
+        if ((rc = dev_alloc(&p, bytes))) return rc;
+        s->pool.push_back(p);
+        s->pool_bytes.push_back(bytes);
+        if (bytes) SWLM_CUDA(cudaMemset(p, 0, bytes));
+    }
     for (const DeltaLayer& l : plan->delta) {
         float* st = nullptr;
         unsigned char* ring = nullptr;
@@ -761,7 +909,13 @@ int stream_launches_per_step(const swlm_plan* plan) {
             if (L.m2 && !product_takes_gate(m, L.m1->k, a.x_f32)) { a.w2 = nullptr; n += 2 * product_launch_count(a) + 1; }
             else n += product_launch_count(a);
         } else if (L.kind == L_DELTA) n += delta_step_fits(plan->delta[L.st.layer].shape) ? 1 : 3;
-        else if (L.kind == L_ROUTED) n += m <= 4 || plan->all_f32() ? 2 : 6;
+        else if (L.kind == L_RETENTION) n += retention_step_fits(L.st.key_dim, L.st.value_dim) ? 1 : 2;
+        else if (L.kind == L_GROUPED) n += 2;
+        else if (L.kind == L_ROUTED) {
+            n += m <= 4 || plan->all_f32() ? 2 : 5;
+            if (L.m4 && m > 4 && !plan->all_f32())
+                for (const Matrix* w : {L.m4, L.m5}) { ProductLaunch a; a.w = w; a.m = m; n += product_launch_count(a); }
+        }
         else n += L.kind == L_LATENT ? 3 : L.kind == L_ARGMAX ? 2 : 1;
     }
     return n;
@@ -852,10 +1006,11 @@ int run_rows(swlm_state* s, const std::vector<Piece>& pieces, const std::vector<
         return SWLM_OK;
     }
 
-    // which pieces are attended in spans: every latent layer must allow it
+    // which pieces are attended in spans: every attention layer must allow it
     bool expands = true;
     for (const Launch& L : plan->launches)
         if (L.kind == L_LATENT) expands &= latent_expands(plan->latent[L.st.layer].row, L.st.head_dim, L.st.value_dim, plan->all_f32());
+        else if (L.kind == L_GROUPED) expands &= grouped_spans(plan->grouped[L.st.layer].row, plan->all_f32());
     std::vector<int32_t> shorts, longs, singles, block_run;
     std::vector<LatentSpan> spans;
     std::vector<RowRun> runs;
@@ -1021,6 +1176,8 @@ int stream_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_i
         if (tmp.stream_width[i] > s->width[i]) { set_error("step: buffer %d is %d wide, the step needs %d", i, s->width[i], tmp.stream_width[i]); return done(SWLM_ERR_INVALID); }
     for (size_t l = 0; l < tmp.latent.size(); ++l)
         if (tmp.latent[l].rank && tmp.latent[l].row.pitch != s->plan->latent[l].row.pitch) { set_error("step: latent layer %zu has other rows", l); return done(SWLM_ERR_INVALID); }
+    for (size_t l = 0; l < tmp.grouped.size(); ++l)
+        if (tmp.grouped[l].row.groups && memcmp(&tmp.grouped[l].row, &s->plan->grouped[l].row, sizeof(GroupedRow))) { set_error("step: grouped layer %zu has other rows", l); return done(SWLM_ERR_INVALID); }
     for (size_t l = 0; l < tmp.delta.size(); ++l)
         if (tmp.delta[l].shape.heads && memcmp(&tmp.delta[l].shape, &s->plan->delta[l].shape, sizeof(DeltaShape))) { set_error("step: gated-delta layer %zu has another shape", l); return done(SWLM_ERR_INVALID); }
     for (int b = 0; b < m; ++b)

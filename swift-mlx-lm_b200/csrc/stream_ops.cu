@@ -35,6 +35,7 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(StreamNorm a, int dim,
     const int r = rows_idx ? rows_idx[blockIdx.x] : blockIdx.x;
     const float* in = a.in + (size_t)r * a.in_stride;
     const bool post = a.w_post != nullptr, add = a.res_in != nullptr;
+    const __nv_bfloat16* joins = a.table ? a.table_row(r, dim) : nullptr;
     float post_scale = 1.f;
     if (post) {
         float ss = 0.f;
@@ -45,6 +46,7 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(StreamNorm a, int dim,
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
         float h = post ? row[i] * post_scale * (__bfloat162float(a.w_post[i]) + a.weight_bias) : in[i];
         if (add) h += a.res_in[(size_t)r * a.res_stride + i];
+        if (joins) h += __bfloat162float(joins[i]) * a.table_scale;
         if (a.res_out) a.res_out[(size_t)r * a.res_stride + i] = h;
         row[i] = h;
         ss = fmaf(h, h, ss);
@@ -71,6 +73,7 @@ __global__ void __launch_bounds__(256) stream_norm_quads_kernel(StreamNorm a, in
     pdl_wait();
     const int r = rows_idx ? rows_idx[blockIdx.x] : blockIdx.x;
     const float* in = a.in + (size_t)r * a.in_stride;
+    const __nv_bfloat16* joins = a.table ? a.table_row(r, dim) : nullptr;
     float h[kNormQuads][4], res[kNormQuads][4];
 #pragma unroll
     for (int j = 0; j < kNormQuads; ++j) {
@@ -80,6 +83,11 @@ __global__ void __launch_bounds__(256) stream_norm_quads_kernel(StreamNorm a, in
         const float4 y = i < dim && a.res_in ? *reinterpret_cast<const float4*>(a.res_in + (size_t)r * a.res_stride + i) : z;
         h[j][0] = x.x; h[j][1] = x.y; h[j][2] = x.z; h[j][3] = x.w;
         res[j][0] = y.x; res[j][1] = y.y; res[j][2] = y.z; res[j][3] = y.w;
+        if (joins && i < dim) {
+            const uint2 v = __ldg(reinterpret_cast<const uint2*>(joins + i));
+            res[j][0] += __uint_as_float(v.x << 16) * a.table_scale; res[j][1] += __uint_as_float(v.x & 0xFFFF0000u) * a.table_scale;
+            res[j][2] += __uint_as_float(v.y << 16) * a.table_scale; res[j][3] += __uint_as_float(v.y & 0xFFFF0000u) * a.table_scale;
+        }
     }
     auto weights = [&](const uint2& v, float (&f)[4]) {
         f[0] = __uint_as_float(v.x << 16) + a.weight_bias; f[1] = __uint_as_float(v.x & 0xFFFF0000u) + a.weight_bias;

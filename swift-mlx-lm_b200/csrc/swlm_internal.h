@@ -110,6 +110,8 @@ enum { GATED_ACT_SILU = 0, GATED_ACT_GELU_TANH = 1, GATED_ACT_CLAMPED = 2 };
 // Activation of a gated feed-forward. CLAMPED: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1).
 struct GatedAct { int kind = GATED_ACT_SILU; float alpha = 0.f, limit = 0.f; };
 #ifdef __CUDACC__
+// the exact GELU
+__device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.0f + erff(v * 0.70710678f)); }
 // activation(gate) * up of the gated MLP (Generator/MetalSourceGenerator+NormAndElementwise.swift:176-208):
 // SiLU for SwiGLU, the tanh approximation of GELU for GEGLU.
 __device__ __forceinline__ float gated_activation(float g, float up, int act) {
@@ -354,12 +356,13 @@ struct ProductOut {
     int stride[kMaxProductSegs] = {};
     int f32[kMaxProductSegs] = {};
     float softcap = 0.f;   // > 0: every value v becomes softcap * tanh(v / softcap)
+    int gelu = 0;          // every value v becomes v * (1 + erf(v / sqrt(2))) / 2
 };
 
 // A norm step over the fp32 stream. mode = its step kind (0: none).
 //   COPY_RMSNORM             h = in
 //   RESADD_*                 h = res_in + in
-//   POSTNORM_*               h = res_in + norm(in; w_post)
+//   POSTNORM_*               h = res_in + norm(in; w_post), and with a table + table[tokens[row]] * table_scale
 // res_out (unless null) = h; the result is norm(h; w).
 struct StreamNorm {
     int mode = 0;
@@ -368,6 +371,9 @@ struct StreamNorm {
     const __nv_bfloat16* w_post = nullptr;
     const __nv_bfloat16* w = nullptr;
     float eps = 0.f, weight_bias = 0.f;
+    const __nv_bfloat16* table = nullptr; const int32_t* tokens = nullptr; int vocab = 0; float table_scale = 0.f;
+    // row r's entry of the table
+    __device__ const __nv_bfloat16* table_row(int r, int dim) const { return table + (size_t)min(max(tokens[r], 0), vocab - 1) * dim; }
 };
 // rows_idx (may be null): output row r is computed from input row rows_idx[r].
 int launch_stream_norm(const StreamNorm& a, int m, int dim, const int32_t* rows_idx, void* out, int out_stride, bool out_f32, cudaStream_t s);
@@ -417,7 +423,7 @@ struct LatentSpan { int row0, count, pos0, seq, ctx0, lo; };
 
 struct LatentLaunch {
     LatentRow row;
-    int heads = 0, dim = 0, vdim = 0, rot_dims = 0;
+    int heads = 0, dim = 0, vdim = 0, rot_dims = 0, rot_neighbours = 0;
     float scale = 1.f, eps = 0.f, weight_bias = 0.f, magnitude = 1.f;
     int window = 0;                                        // > 0: a row sees its own and the window - 1 positions before it
     const __nv_bfloat16* sink = nullptr;                   // [heads]: exp(sink) joins the denominator; null: none
@@ -455,6 +461,20 @@ constexpr int kLatentQueryTile = 128;
 // launches (for the counters): short part 3, span part 4 or 5
 int launch_latent(const LatentLaunch& a, cudaStream_t s, int* launches);
 
+// ---- rotary positions --------------------------------------------------------------------------------------------------
+// Entry i of a vector whose first `dims` entries turn: the pair it belongs to, its partner, and whether it is the pair's first.
+struct RotaryEntry { int pair, partner; bool first; };
+#ifdef __CUDACC__
+__device__ __forceinline__ RotaryEntry rotary_entry(int i, int dims, int neighbours) {
+    if (neighbours) return RotaryEntry{i >> 1, i ^ 1, (i & 1) == 0};
+    const int half = dims >> 1;
+    return i < half ? RotaryEntry{i, i + half, true} : RotaryEntry{i - half, i - half, false};
+}
+// first entry of pair i, and the distance to the second
+__device__ __forceinline__ int rotary_first(int i, int neighbours) { return neighbours ? 2 * i : i; }
+__device__ __forceinline__ int rotary_step(int dims, int neighbours) { return neighbours ? 1 : dims >> 1; }
+#endif
+
 // ---- gated delta rule (delta_rule.cu) ----------------------------------------------------------------------------------
 // Consecutive rows of one sequence: rows row0 .. row0 + count - 1 of the batch at positions pos0 ..; walked in blocks of
 // kDeltaBlock tokens, blk0 = number of blocks of the runs before it.
@@ -488,19 +508,75 @@ bool delta_step_fits(const DeltaShape& s);                    // single tokens i
 size_t delta_scratch_floats(const DeltaShape& s, int blocks, int rows);
 int launch_delta(const DeltaLaunch& a, cudaStream_t s, int* launches);
 
+// ---- retention (retention.cu) -------------------------------------------------------------------------------------------
+struct RetentionLaunch {
+    int heads = 0, dim = 0, vdim = 0;
+    float eps = 0.f, scale = 1.f, out_scale = 1.f;
+    bool f32 = false;
+    const float* decay = nullptr;                          // [heads]
+    const void* qkv = nullptr; int qkv_stride = 0;
+    const void* gate = nullptr; int gate_stride = 0;
+    float* state = nullptr;                                // [sequence][heads][dim][vdim]
+    const int32_t* row_seq = nullptr; const int32_t* row_pos = nullptr;
+    void* out = nullptr; int out_stride = 0;
+    int n_single = 0; const int32_t* single_rows = nullptr;   // as DeltaLaunch
+    int n_runs = 0; const RowRun* runs = nullptr;
+    int n_blocks = 0; const int32_t* block_run = nullptr;
+    float* scratch = nullptr;                              // [row][heads][vdim]
+};
+int retention_init();
+bool retention_supported(int heads, int dim, int vdim);
+bool retention_step_fits(int dim, int vdim);
+int launch_retention(const RetentionLaunch& a, cudaStream_t s, int* launches);
+
+// ---- grouped-query attention over pages (grouped_attention.cu) -----------------------------------------------------------
+// A page holds, head after head, 64 key rows of `pk` entries and 64 value rows of `pv` (in bf16 pools odd multiples of 16 bytes,
+// see LatentRow); dp and vp are the sizes padded to 16, padding entries are zero. block: entries of a (page, head) pair.
+struct GroupedRow { int groups = 0, dim = 0, vdim = 0, dp = 0, vp = 0, pk = 0, pv = 0, block = 0; };
+GroupedRow grouped_row(int groups, int dim, int vdim, bool f32);
+struct GroupedLaunch {
+    GroupedRow row;
+    int heads = 0, rot_dims = 0, rot_neighbours = 0, window = 0, chunk = 0, sink_one = 0;
+    float scale = 1.f, eps = 0.f, weight_bias = 0.f, magnitude = 1.f, out_scale = 1.f;
+    const float* inv_freq = nullptr;
+    bool f32 = false;
+    const __nv_bfloat16 *q_norm = nullptr, *k_norm = nullptr;
+    void* qkv = nullptr; int qkv_stride = 0;               // q | k | v per row; q is normed and rotated in place
+    const float* gate = nullptr; int gate_stride = 0;
+    void* pool = nullptr;
+    const int32_t* page_table = nullptr; int pages_per_seq = 0;
+    const int32_t* row_seq = nullptr; const int32_t* row_pos = nullptr;
+    void* out = nullptr; int out_stride = 0;
+    int n_rows = 0;                                        // all rows of the batch
+    int n_short = 0; const int32_t* short_rows = nullptr; int max_pages = 1;   // attended one by one; longest context of theirs
+    const LatentSpan* spans = nullptr; int n_tiles = 0; const int2* tiles = nullptr;   // and in spans: tiles of kLatentQueryTile rows
+    int* status = nullptr;
+    bool only_attention = false;   // timing hook
+};
+int grouped_init();
+bool grouped_supported(const GroupedRow& r);
+// can rows of this layer be attended in spans?
+bool grouped_spans(const GroupedRow& r, bool f32);
+int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches);
+
 // ---- routed feed-forward (routed_mlp.cu) -------------------------------------------------------------------------------
-struct RoutedShape { int experts = 0, top = 0, groups = 1, keep = 1, width = 0, ff = 0; };
+// shared_ff > 0: inner size of the feed-forward that every row takes
+struct RoutedShape { int experts = 0, top = 0, groups = 1, keep = 1, width = 0, ff = 0, shared_ff = 0; };
 struct RoutedLaunch {
     RoutedShape shape;
     float scale = 1.f;
     GatedAct act;
+    int softmax = 0, group_best = 2, raw_weights = 0;      // scores, what a group counts as, whether weights are renormalised
     int m = 0; bool f32 = false;
     const void* x = nullptr; int x_stride = 0;
-    const float* z = nullptr; int z_stride = 0;
-    const Matrix *gate = nullptr, *up = nullptr, *down = nullptr;   // the experts' rows one after the other
+    const float* z = nullptr; int z_stride = 0;            // router logits; with a shared feed-forward its gate behind them
+    // the experts' rows one after the other; gate == null: an expert is down(gelu(up x))
+    const Matrix *gate = nullptr, *up = nullptr, *down = nullptr;
+    const Matrix *shared_up = nullptr, *shared_down = nullptr;
     float* out = nullptr; int out_stride = 0;
     unsigned char* scratch = nullptr;
     unsigned* counts = nullptr;                            // [kMaxExperts], zero between launches
+    float* part = nullptr; size_t part_floats = 0;         // split-K sums of the shared products
     int* status = nullptr;
 };
 constexpr int kMaxExperts = 1024, kMaxTop = 64;

@@ -22,7 +22,7 @@ inline int dev_alloc(T** p, size_t count, int64_t* total = nullptr) {
 
 
 enum LaunchKind { L_EMBED, L_RMSNORM, L_QGEMV, L_QK_NORM, L_ATTN, L_SWIGLU, L_CONV, L_ARGMAX, L_SSM,
-                  L_PRODUCT, L_LATENT, L_DELTA, L_ROUTED, L_SOFTCAP };   // from L_PRODUCT on: fp32-stream plans only
+                  L_PRODUCT, L_LATENT, L_DELTA, L_ROUTED, L_SOFTCAP, L_GROUPED, L_RETENTION };   // from L_PRODUCT on: fp32-stream plans only
 
 struct Launch {
     int kind = 0;
@@ -55,9 +55,10 @@ struct Launch {
     const Matrix* m1 = nullptr;
     const Matrix* m2 = nullptr;
     const Matrix* m3 = nullptr;               // routed feed-forward: the experts' down rows (m1, m2: gate, up)
+    const Matrix *m4 = nullptr, *m5 = nullptr;   // and the shared feed-forward's up and down
     GatedAct act;
     float softcap = 0.f;                      // of the output head's logits
-    const DenseTensor* dv[6] = {};            // gated delta rule: taps of q, k, v, norm weight, A_log, dt_bias; latent attention: [0] sink
+    const DenseTensor* dv[6] = {};            // gated delta rule: taps of q, k, v, norm weight, A_log, dt_bias; latent attention: [0] sink; norms: [0] table that joins
     int window_set = 0;                       // latent attention: index into plan->windows
     const DenseTensor* norm_post = nullptr;   // norm steps: weight of the norm applied to the input before it is added
     int kv_prefetch_attn = -1;    // index of the attention launch whose K/V rows this product pulls into L2
@@ -67,13 +68,16 @@ struct Launch {
 // multiplied by `magnitude`.
 struct RopeTable {
     int rope_dim; float base; float* inv_freq;
-    float factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f, magnitude = 1.f;
+    float factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f, magnitude = 1.f, divisor = 1.f;
 };
 
 // One latent-attention layer's share of the page pool.
 struct LatentLayer { int rank = 0, rot = 0; LatentRow row{}; };
 
-// One gated-delta layer: per sequence an fp32 state and the last inputs of the convolutions.
+// One grouped-attention layer's share of the page pool.
+struct GroupedLayer { GroupedRow row{}; };
+
+// One gated-delta or retention layer: per sequence an fp32 state and the last inputs of the convolutions (retention: no taps).
 struct DeltaLayer {
     DeltaShape shape;
     size_t state_elems() const { return (size_t)shape.heads * shape.dim * shape.vdim; }
@@ -155,8 +159,9 @@ struct swlm_plan {
     bool rows_groups_ready = false;
     // fp32-stream plans (desc.stream_dtype != 0)
     std::vector<LatentLayer> latent;      // by step.layer
+    std::vector<GroupedLayer> grouped;    // by step.layer
     std::vector<DeltaLayer> delta;        // by step.layer
-    std::vector<int> windows;             // distinct sliding windows of the latent layers
+    std::vector<int> windows;             // distinct sliding windows of the attention layers
     int stream_width[SWLM_BUF_COUNT] = {};
     int latent_heads_max = 0, latent_q_floats = 0, latent_part_floats = 0;   // largest over the layers, per row / per row and split
     bool stream() const { return desc.stream_dtype != 0; }
@@ -209,7 +214,7 @@ struct swlm_state {
     int* pf_status = nullptr;      // device word: a bounded wait of the tensor-core product expired
     int prefill_chunk = 2048;      // tokens per chunk; 0 = one token at a time through the decode graph
     int* tc_status = nullptr;      // pinned host word (mapped): a bounded wait of a kernel expired
-    // fp32-stream plans: paged pool of latent rows (one page list per sequence, the same page numbers in every layer's
+    // fp32-stream plans: paged pools, those of the latent layers first, then the grouped ones (one page list per sequence, the same page numbers in every layer's
     // pool), the page table on host and device, and the two activation sets
     std::vector<void*> pool; std::vector<size_t> pool_bytes;
     std::vector<float*> delta_state; std::vector<void*> delta_ring;   // per gated-delta layer: [max_batch][state_elems], [max_batch][ring_elems]

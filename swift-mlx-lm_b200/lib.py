@@ -64,6 +64,16 @@ class Step(C.Structure):
         ("eps2", C.c_float),
         ("weight5", C.c_char * NAME_MAX),
         ("weight6", C.c_char * NAME_MAX),
+        ("rope_pairs", C.c_int32),
+        ("rope_divisor", C.c_float),
+        ("chunk", C.c_int32),
+        ("sink_one", C.c_int32),
+        ("k2", C.c_int32),
+        ("in4_off", C.c_int32),
+        ("out_scale", C.c_float),
+        ("score_act", C.c_int32),
+        ("group_best", C.c_int32),
+        ("raw_weights", C.c_int32),
     ]
 
 
@@ -94,6 +104,7 @@ class BuffersDesc(C.Structure):
         ("latent_layers", C.c_int32),
         ("kv_pool_tokens", C.c_int32),
         ("delta_layers", C.c_int32),
+        ("grouped_layers", C.c_int32),
     ]
 
 

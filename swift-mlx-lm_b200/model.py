@@ -338,6 +338,9 @@ def upload_weights(store: WeightStore, builder, weights) -> None:
             store.add_matrix(name, entry)
         else:
             store.add_dense(name, entry, shard if kind == "conv" else 0)
+    if hasattr(builder, "constants"):   # fp32 tensors that the configuration gives
+        for name, values in builder.constants().items():
+            store.add_dense_f32(name, values)
 
 
 def load_model(store: WeightStore, builder, weights) -> InferenceModel:

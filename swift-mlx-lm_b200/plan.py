@@ -40,7 +40,11 @@ STEP_CLAMPED_GLU = 17
 STEP_GATED_DELTA = 18
 STEP_ROUTED_MLP = 19
 STEP_SOFTCAP = 20
+STEP_GROUPED_ATTN = 21
+STEP_RETENTION = 22
 GATE_SILU, GATE_SIGMOID = 0, 1
+SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
+ROPE_HALVES, ROPE_NEIGHBOURS = 0, 1
 
 STREAM_BF16, STREAM_F32, STREAM_ALL_F32 = 0, 1, 2
 PAGE_TOKENS = 64
