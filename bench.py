@@ -484,25 +484,45 @@ RIROTAR_SHAPES = {   # layers, experts, chosen experts, groups, kept groups: wid
 RIROTAR_WINDOW = 1024
 
 
-def run_rirotar(args, pkg):
-    """Prompt and decode throughput of the Rirotar design (three gated-delta layers to one latent-attention layer, routed
-    feed-forwards) beside Vuzunex (latent attention, dense feed-forwards of the active size) at equal width, heads, layers and
-    vocabulary, and its recurrence beside the DeltaNet recipe's. One JSON line."""
+class KindTimer:
+    """Times of one step kind of a model: in decode steps (`decode`), and over one prompt portion of `rows` tokens (`portion`)."""
+
+    def __init__(self, model, timed, chunk):
+        self.model, self.timed, self.chunk, self.rows = model, timed, chunk, len(chunk)
+        self.hbm, self.tensor = measured_peaks()[0], measured_tensor_peak()[0]
+
+    def decode(self, kind):
+        self.model.profile_kind(kind, 2)
+        return self.timed(lambda: self.model.profile_kind(kind, 1), 10)
+
+    def portion(self, kind):
+        self.model.profile_batch(0, self.chunk, kind, 2)
+        return self.timed(lambda: self.model.profile_batch(0, self.chunk, kind, 5), 1) / 5
+
+    def hbm_entry(self, ms, nbytes, count):
+        return {"us_per_layer": ms * 1e3 / count, "bytes": nbytes, "GBs": nbytes / ms / 1e6, "frac": nbytes / ms / 1e6 / self.hbm}
+
+    def tensor_entry(self, ms, flops, count):
+        return {"rows": self.rows, "us_per_layer": ms * 1e3 / count, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / self.tensor}
+
+
+def reached_experts(experts, top, batch):
+    """Experts that `batch` rows of evenly spread choices reach."""
+    return experts * (1.0 - (1.0 - top / experts) ** batch)
+
+
+def measure_rirotar(pkg, args, stream, timed):
+    """(rates and kernels of a Rirotar model of the shape, its configuration)."""
     R, P = pkg.rirotar, pkg.plan
-    stream = bench_stream()
-    timed = stream_timer(stream)
     width, heads, ff, _ = VUZUNEX_SHAPES[args.shape]
     layers, experts, top, groups, keep = RIROTAR_SHAPES[args.shape]
     batch, ctx = args.batch, args.ctx
-    max_seq = ctx + 4 * (max(3, args.warmup) + args.steps) + 64
-    hbm, _ = measured_peaks()
-    tensor, _ = measured_tensor_peak()
     routed, dense = R.RoutedFF(ff // top, 7.0, experts, top, groups, keep, 2.5), R.DenseFF(ff, 7.0)
     channel = R.GatedDelta(heads, heads, 128, 128, 4, True, 128, 128)
     scalar = R.GatedDelta(heads, heads // 2, 128, 128, 4, False)
     latent = R.WindowedLatentAttention(heads, 128, 128, 512, 128 ** -0.5, RIROTAR_WINDOW)
     block = [R.Layer(channel, routed), R.Layer(scalar, routed), R.Layer(channel, routed), R.Layer(latent, dense)]
-    cfg = pkg.RirotarConfig(vocab=BENCH_VOCAB, width=width, layers=[block[i % 4] for i in range(layers)], logit_softcap=30.0, max_seq=max_seq, max_batch=batch)
+    cfg = pkg.RirotarConfig(vocab=BENCH_VOCAB, width=width, layers=[block[i % 4] for i in range(layers)], logit_softcap=30.0, max_seq=bench_max_seq(args), max_batch=batch)
     n_routed, n_latent = 3 * layers // 4, layers // 4
     n_delta = layers - n_latent
     builder = pkg.RirotarPlanBuilder(cfg)
@@ -511,47 +531,45 @@ def run_rirotar(args, pkg):
     model.set_stream(stream.cuda_stream)
     prompt = np.random.default_rng(7).integers(0, BENCH_VOCAB, size=(batch, ctx), dtype=np.int32)
     ours = serve_rates(model, prompt, args, timed)
-
-    def kind_ms(kind):
-        model.profile_kind(kind, 2)
-        return timed(lambda: model.profile_kind(kind, 1), 10)
-
-    def hbm_entry(ms, nbytes, count):
-        return {"us_per_layer": ms * 1e3 / count, "bytes": nbytes, "GBs": nbytes / ms / 1e6, "frac": nbytes / ms / 1e6 / hbm}
-
-    product_bytes = cfg.product_elems() * 2
-    ours["decode_products"] = hbm_entry(kind_ms(P.STEP_PRODUCT), product_bytes, layers)
-    state_bytes = 2.0 * n_delta * batch * heads * 128 * 128 * 4
-    ours["decode_delta_step"] = hbm_entry(kind_ms(P.STEP_GATED_DELTA), state_bytes, n_delta)
-    # experts that `batch` rows of evenly spread choices reach
-    reached = experts * (1.0 - (1.0 - top / experts) ** batch)
-    expert_bytes = n_routed * reached * 3 * width * (ff // top) * 2
-    ours["decode_routed"] = hbm_entry(kind_ms(P.STEP_ROUTED_MLP), expert_bytes, n_routed)
-    small, kv = n_latent * heads * 256 * 512 * 2, n_latent * batch * min(model.position, RIROTAR_WINDOW) * 512 * 2
-    ours["decode_attention"] = hbm_entry(kind_ms(P.STEP_ATTN_DECODE), kv, n_latent)
-    ours["decode_latent_step"] = hbm_entry(kind_ms(P.STEP_LATENT_ATTN), small + kv, n_latent)
     n = min(ctx, 2048)
+    t = KindTimer(model, timed, prompt[0, :n])
+    product_bytes = cfg.product_elems() * 2
+    ours["decode_products"] = t.hbm_entry(t.decode(P.STEP_PRODUCT), product_bytes, layers)
+    ours["decode_delta_step"] = t.hbm_entry(t.decode(P.STEP_GATED_DELTA), 2.0 * n_delta * batch * heads * 128 * 128 * 4, n_delta)
+    ours["decode_routed"] = t.hbm_entry(t.decode(P.STEP_ROUTED_MLP), n_routed * reached_experts(experts, top, batch) * 3 * width * (ff // top) * 2, n_routed)
+    small, kv = n_latent * heads * 256 * 512 * 2, n_latent * batch * min(model.position, RIROTAR_WINDOW) * 512 * 2
+    ours["decode_attention"] = t.hbm_entry(t.decode(P.STEP_ATTN_DECODE), kv, n_latent)
+    ours["decode_latent_step"] = t.hbm_entry(t.decode(P.STEP_LATENT_ATTN), small + kv, n_latent)
     model.reset_state()
-    chunk = prompt[0, :n]
-
-    def chunk_ms(kind):
-        model.profile_batch(0, chunk, kind, 2)
-        return timed(lambda: model.profile_batch(0, chunk, kind, 5), 1) / 5
-
-    def tensor_entry(ms, flops, count):
-        return {"rows": n, "us_per_layer": ms * 1e3 / count, "tflops": flops / ms / 1e9, "frac": flops / ms / 1e9 / tensor}
-
-    ours["prefill_products"] = tensor_entry(chunk_ms(P.STEP_PRODUCT), 2.0 * n * (product_bytes / 2 - BENCH_VOCAB * width), layers)
-    ours["prefill_routed"] = tensor_entry(chunk_ms(P.STEP_ROUTED_MLP), n_routed * 2.0 * n * top * 3 * width * (ff // top), n_routed)
+    ours["prefill_products"] = t.tensor_entry(t.portion(P.STEP_PRODUCT), 2.0 * n * (product_bytes / 2 - BENCH_VOCAB * width), layers)
+    ours["prefill_routed"] = t.tensor_entry(t.portion(P.STEP_ROUTED_MLP), n_routed * 2.0 * n * top * 3 * width * (ff // top), n_routed)
     w = min(n, RIROTAR_WINDOW)
     pairs = w * (w + 1) / 2 + (n - w) * w
-    ours["prefill_attention"] = tensor_entry(chunk_ms(P.STEP_ATTN_DECODE), n_latent * heads * pairs * 2.0 * 256, n_latent)
-    ours["prefill_latent_step_us_per_layer"] = chunk_ms(P.STEP_LATENT_ATTN) * 1e3 / n_latent
+    ours["prefill_attention"] = t.tensor_entry(t.portion(P.STEP_ATTN_DECODE), n_latent * heads * pairs * 2.0 * 256, n_latent)
+    ours["prefill_latent_step_us_per_layer"] = t.portion(P.STEP_LATENT_ATTN) * 1e3 / n_latent
     # per token and head: decay, two products with the state, one update
-    ours["prefill_delta"] = {"rows": n, "us_per_layer": chunk_ms(P.STEP_GATED_DELTA) * 1e3 / n_delta}
-    ours["prefill_delta"]["fp32_tflops"] = n * heads * 128 * 128 * 7.0 / ours["prefill_delta"]["us_per_layer"] / 1e6
+    us = t.portion(P.STEP_GATED_DELTA) * 1e3 / n_delta
+    ours["prefill_delta"] = {"rows": n, "us_per_layer": us, "fp32_tflops": n * heads * 128 * 128 * 7.0 / us / 1e6}
     model.close()
     store.close()
+    return ours, cfg
+
+
+def bench_max_seq(args):
+    return args.ctx + 4 * (max(3, args.warmup) + args.steps) + 64
+
+
+def run_rirotar(args, pkg):
+    """Prompt and decode throughput of the Rirotar design (three gated-delta layers to one latent-attention layer, routed
+    feed-forwards) beside Vuzunex (latent attention, dense feed-forwards of the active size) at equal width, heads, layers and
+    vocabulary, and its recurrence beside the DeltaNet recipe's. One JSON line."""
+    P = pkg.plan
+    stream = bench_stream()
+    timed = stream_timer(stream)
+    width, heads, ff, _ = VUZUNEX_SHAPES[args.shape]
+    layers, experts, top, _, _ = RIROTAR_SHAPES[args.shape]
+    batch, ctx, max_seq = args.batch, args.ctx, bench_max_seq(args)
+    ours, _ = measure_rirotar(pkg, args, stream, timed)
     closest = measure_vuzunex(pkg, vuzunex_config(pkg, args, layers, max_seq), args, stream, timed)
     # the recurrence of the DeltaNet recipe at the same heads, in a model with little else (decode steps per layer)
     dcfg = pkg.ModelConfig("deltanet", 512, 512, 5, 4, 2, 128, 4096, attention_layers=[4], max_seq=max_seq, max_batch=batch, ssm_heads=heads,
@@ -563,8 +581,9 @@ def run_rirotar(args, pkg):
     like = {}
     if batch <= 16:
         model.profile_kind(P.STEP_SSM_RECURRENCE, 2)
-        like["decode"] = hbm_entry(timed(lambda: model.profile_kind(P.STEP_SSM_RECURRENCE, 1), 10), 2.0 * 4 * batch * heads * 128 * 128 * 4, 4)
+        like["decode"] = KindTimer(model, timed, []).hbm_entry(timed(lambda: model.profile_kind(P.STEP_SSM_RECURRENCE, 1), 10), 2.0 * 4 * batch * heads * 128 * 128 * 4, 4)
     if batch == 1:
+        n = min(ctx, 2048)
         p = np.random.default_rng(8).integers(0, 4096, size=(1, n), dtype=np.int32)
         model.set_prefill_chunk(n)
         model.prefill(p)
@@ -575,6 +594,79 @@ def run_rirotar(args, pkg):
     workload = (f"{layers} layers (channel delta, delta, channel delta, latent), width {width}, {heads} heads of 128 x 128, latent 512 over a window of {RIROTAR_WINDOW}, "
                 f"{top} of {experts} experts of {ff // top} (dense {ff} behind latent layers), vocabulary {BENCH_VOCAB}, context {ctx}, batch {batch}")
     print(json.dumps(dict(design_line(args, "Rirotar", ours, workload), rirotar=ours, vuzunex_equal_size=closest, deltanet_recurrence_equal_heads=like)))
+
+
+KALEVIK_SHAPES = {   # layers and the loop over some of them; experts and their choice are RIROTAR_SHAPES's
+    "1b": (9, (3, 6, 2)), "8b": (6, (2, 4, 2))}
+KALEVIK_CHUNK = 8192
+
+
+def run_kalevik(args, pkg):
+    """Prompt and decode throughput of the Kalevik design (latent-attention layers alternating with chunked grouped-query attention
+    beside retention, routed feed-forwards with a shared one, a loop) beside Rirotar at equal width, heads, layer runs, vocabulary
+    and active feed-forward, and its grouped-query attention beside the Llama recipe's at equal heads. One JSON line."""
+    K, P = pkg.kalevik, pkg.plan
+    stream = bench_stream()
+    timed = stream_timer(stream)
+    width, heads, ff, _ = VUZUNEX_SHAPES[args.shape]
+    layers, loop = KALEVIK_SHAPES[args.shape]
+    _, experts, top, groups, keep = RIROTAR_SHAPES[args.shape]
+    batch, ctx, kv_heads = args.batch, args.ctx, heads // 4
+    # two matrices per expert and a shared one of half the size: as many active entries as a gated feed-forward of `ff`
+    routed, dense = K.RoutedFF(ff // top, experts, top, groups, keep, ff // 2), K.DenseFF(ff)
+    latent = K.LatentAttention(heads, 128, 64, 128, 512, 192 ** -0.5, 500000.0, 64)
+    parallel = K.Parallel(K.ChunkedAttention(heads, kv_heads, 128, 128, 128 ** -0.5, KALEVIK_CHUNK, 500000.0, 64, 4.0),
+                          K.Retention(heads, 128, 128, tuple(1.0 - 2.0 ** (-5.0 - 7.0 * i / heads) for i in range(heads))), 0.7, 0.7)
+    cfg = K.KalevikConfig(vocab=BENCH_VOCAB, width=width, layers=[K.Layer(parallel if i % 2 else latent, routed if i else dense) for i in range(layers)], loop=loop,
+                          max_seq=bench_max_seq(args), max_batch=batch)
+    runs = [cfg.layers[i] for i, _ in cfg.runs()]
+    n_parallel = sum(isinstance(r.mixer, K.Parallel) for r in runs)
+    n_latent, n_routed = len(runs) - n_parallel, sum(isinstance(r.mlp, K.RoutedFF) for r in runs)
+    builder = pkg.KalevikPlanBuilder(cfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, block_weights(builder))
+    model.set_stream(stream.cuda_stream)
+    prompt = np.random.default_rng(7).integers(0, BENCH_VOCAB, size=(batch, ctx), dtype=np.int32)
+    ours = serve_rates(model, prompt, args, timed)
+    n = min(ctx, 2048)
+    t = KindTimer(model, timed, prompt[0, :n])
+    product_bytes = cfg.product_elems() * 2
+    ours["decode_products"] = t.hbm_entry(t.decode(P.STEP_PRODUCT), product_bytes, len(runs))
+    expert_bytes = n_routed * 2 * width * (reached_experts(experts, top, batch) * (ff // top) + ff // 2) * 2
+    ours["decode_routed"] = t.hbm_entry(t.decode(P.STEP_ROUTED_MLP), expert_bytes, n_routed)
+    seen = model.position % KALEVIK_CHUNK
+    ours["decode_grouped_step"] = t.hbm_entry(t.decode(P.STEP_GROUPED_ATTN), n_parallel * batch * seen * kv_heads * 256 * 2, n_parallel)
+    ours["decode_retention_step"] = t.hbm_entry(t.decode(P.STEP_RETENTION), 2.0 * n_parallel * batch * heads * 128 * 128 * 4, n_parallel)
+    latent_bytes = n_latent * (heads * 256 * 512 * 2 + batch * model.position * 576 * 2)
+    ours["decode_latent_step"] = t.hbm_entry(t.decode(P.STEP_LATENT_ATTN), latent_bytes, n_latent)
+    model.reset_state()
+    ours["prefill_products"] = t.tensor_entry(t.portion(P.STEP_PRODUCT), 2.0 * n * (product_bytes / 2 - BENCH_VOCAB * width), len(runs))
+    ours["prefill_routed"] = t.tensor_entry(t.portion(P.STEP_ROUTED_MLP), n_routed * 2.0 * n * 2 * width * (ff + ff // 2), n_routed)
+    ours["prefill_grouped_step"] = t.tensor_entry(t.portion(P.STEP_GROUPED_ATTN), n_parallel * heads * n * (n + 1) / 2 * 2.0 * 256, n_parallel)
+    ours["prefill_latent_step_us_per_layer"] = t.portion(P.STEP_LATENT_ATTN) * 1e3 / n_latent
+    us = t.portion(P.STEP_RETENTION) * 1e3 / n_parallel
+    moved = n * heads * 128 * 5 * 2   # q, k, v, gate and result
+    ours["prefill_retention"] = {"rows": n, "us_per_layer": us, "bytes": moved, "frac": moved / us / 1e3 / t.hbm, "fp32_tflops": n * heads * 128 * 128 * 5.0 / us / 1e6}
+    model.close()
+    store.close()
+    closest, rcfg = measure_rirotar(pkg, args, stream, timed)
+    assert len(rcfg.layers) == len(runs)
+    vuzunex = measure_vuzunex(pkg, vuzunex_config(pkg, args, 4, bench_max_seq(args)), args, stream, timed)
+    # grouped-query attention of the Llama recipe at the same heads, in a model with little else
+    like = {}
+    lcfg = pkg.ModelConfig("llama", 1024, 1024, 4, heads, kv_heads, 128, 4096, max_seq=bench_max_seq(args), max_batch=batch)
+    builder = pkg.DispatchPlanBuilder(lcfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, block_weights(builder))
+    model.set_stream(stream.cuda_stream)
+    model.prefill(np.random.default_rng(8).integers(0, 4096, size=(batch, ctx), dtype=np.int32))
+    like["decode_attention"] = t.hbm_entry(KindTimer(model, timed, []).decode(P.STEP_ATTN_DECODE), 4 * batch * model.position * kv_heads * 256 * 2, 4)
+    model.close()
+    store.close()
+    workload = (f"{layers} layers (latent and parallel in turn), layers {loop[0]} .. {loop[1] - 1} run {loop[2]} times, width {width}, {heads} heads, latent 512 + 64, "
+                f"{kv_heads} key / value heads of 128 in chunks of {KALEVIK_CHUNK}, retention of 128 x 128, {top} of {experts} experts of {ff // top} and a shared one of {ff // 2}, "
+                f"vocabulary {BENCH_VOCAB}, context {ctx}, batch {batch}")
+    print(json.dumps(dict(design_line(args, "Kalevik", ours, workload), kalevik=ours, rirotar_equal_size=closest, vuzunex_kernels=vuzunex, llama_attention_equal_heads=like)))
 
 
 def main():
@@ -592,9 +684,9 @@ def main():
     ap.add_argument("--prefill", choices=["real", "synthetic"], default="real",
                     help="how the KV cache gets its `ctx` tokens: by running the prompt, or random bf16 rows")
     ap.add_argument("--small", action="store_true")
-    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex", "rirotar"], default="llama",
-                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size; rirotar: the gated-delta design beside Vuzunex of equal size")
-    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex, rirotar: which layer sizes")
+    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex", "rirotar", "kalevik"], default="llama",
+                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size; rirotar: the gated-delta design beside Vuzunex of equal size; kalevik: the looped latent / retention design beside Rirotar of equal size")
+    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex, rirotar, kalevik: which layer sizes")
     ap.add_argument("--batch", type=int, default=1, help="sequences decoded together (1..64), all at the same position")
     ap.add_argument("--kv", choices=["bf16", "q8", "rotor-q4", "rotor-q4-qjl16"], default="bf16",
                     help="KV cache elements: bf16, 8-bit groups of 32 (36-byte blocks), or the rotated 4-bit groups of 64 "
@@ -609,6 +701,9 @@ def main():
         return
     if args.model == "rirotar":
         run_rirotar(args, pkg)
+        return
+    if args.model == "kalevik":
+        run_kalevik(args, pkg)
         return
     if args.model == "lfm2" and args.ctx == 4096:
         args.ctx = 2048   # the hybrid configuration's prompt length

@@ -132,7 +132,7 @@ enum {
        [k][n] and <weight>i<weight4> [n][k]; its output is weighted with s / (sum of the chosen s + 1e-20) * scale.
        score_act SWLM_SCORE_SOFTMAX: s = softmax(logits) over all experts. group_best 1: a group counts as its largest s.
        raw_weights 1: an expert's output is weighted with s * scale. weight2 empty: expert i is <weight4>(gelu(<weight3> in))
-       with the exact (erf) GELU. weight5 not empty: a feed-forward weight6 [n][k2] (gelu(weight5 [k2][n] in)) that every
+       with the exact (erf) GELU. weight5 not empty (only then): a feed-forward weight6 [n][k2] (gelu(weight5 [k2][n] in)) that every
        token takes, its output times sigmoid(in2[experts]) is added. */
     SWLM_STEP_ROUTED_MLP = 19,
     /* logits = scale * tanh(logits / scale), in place */

@@ -178,7 +178,7 @@ template <int KQ, int NV, int UK>   // 16-column steps of query / key and value 
 __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const GroupedParams p) {
     extern __shared__ __align__(128) unsigned char dec_smem[];
     __shared__ __align__(8) unsigned long long bar[kDecWarps];
-    __shared__ float warp_m[kDecWarps][kDecHeads], warp_l[kDecWarps][kDecHeads], cta_m[kDecHeads], cta_l[kDecHeads];
+    __shared__ float warp_m[kDecWarps][kDecHeads], warp_l[kDecWarps][kDecHeads], cta_m[kDecHeads], cta_l[kDecHeads], all_m[kDecCluster][kDecHeads], all_l[kDecCluster][kDecHeads];
     const cg::cluster_group cluster = cg::this_cluster();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int nz = gridDim.x, rank = blockIdx.x, kv = blockIdx.y / ((p.share + kDecHeads - 1) / kDecHeads), tile = blockIdx.y % ((p.share + kDecHeads - 1) / kDecHeads);
@@ -202,6 +202,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
     };
     const int first = rank * kDecWarps + warp, step = nz * kDecWarps;
     if (lane == 0 && first < units) request(first);
+    const float gate = tid < nh ? ga_gate(p, r, h0 + tid) : 0.f;
     // query fragments: rows g and g + 8
     const int ksteps = p.row.dp >> 4, n_vt = p.row.vp >> 4;
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)r * p.qkv_stride + (size_t)h0 * p.row.dim;
@@ -326,17 +327,32 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
         own[i] = v;
     }
     cluster.sync();
-    for (int i = rank * kDecThreads + tid; i < nh * p.row.vdim; i += nz * kDecThreads) {
-        const int hh = i / p.row.vdim, c = i - hh * p.row.vdim;
+    // every CTA's maximum and sum, then its share of every head's result
+    if (tid < nz * nh) {
+        const int z = tid / nh, hh = tid - z * nh;
+        all_m[z][hh] = cluster.map_shared_rank(cta_m, z)[hh];
+        all_l[z][hh] = cluster.map_shared_rank(cta_l, z)[hh];
+    }
+    __syncthreads();
+    if (tid < nh) {
         float top = p.sink_one ? 0.f : -INFINITY;
-        for (int z = 0; z < nz; ++z) top = fmaxf(top, cluster.map_shared_rank(cta_m, z)[hh]);
-        float total = p.sink_one ? exp2f(-top) : 0.f, v = 0.f;
+        for (int z = 0; z < nz; ++z) top = fmaxf(top, all_m[z][tid]);
+        float total = p.sink_one ? exp2f(-top) : 0.f;
         for (int z = 0; z < nz; ++z) {
-            const float mz = cluster.map_shared_rank(cta_m, z)[hh], f = mz == -INFINITY ? 0.f : exp2f(mz - top);
-            total = fmaf(f, cluster.map_shared_rank(cta_l, z)[hh], total);
-            v = fmaf(f, cluster.map_shared_rank(own, z)[hh * vp + c], v);
+            const float f = all_m[z][tid] == -INFINITY ? 0.f : exp2f(all_m[z][tid] - top);
+            total = fmaf(f, all_l[z][tid], total);
+            all_m[z][tid] = f;
         }
-        static_cast<__nv_bfloat16*>(p.out)[(size_t)r * p.out_stride + (size_t)(h0 + hh) * p.row.vdim + c] = __float2bfloat16_rn(v / total * ga_gate(p, r, h0 + hh));
+        const float f = gate / total;
+        for (int z = 0; z < kDecCluster; ++z) all_m[z][tid] = z < nz ? all_m[z][tid] * f : 0.f;
+    }
+    __syncthreads();
+    for (int i = rank * kDecThreads + tid; i < nh * vp; i += nz * kDecThreads) {
+        const int hh = i / vp, c = i - hh * vp;
+        float v = 0.f;
+#pragma unroll
+        for (int z = 0; z < kDecCluster; ++z) v = fmaf(all_m[z][hh], cluster.map_shared_rank(own, z < nz ? z : rank)[i], v);
+        if (c < p.row.vdim) static_cast<__nv_bfloat16*>(p.out)[(size_t)r * p.out_stride + (size_t)(h0 + hh) * p.row.vdim + c] = __float2bfloat16_rn(v);
     }
     cluster.sync();   // nobody leaves while others still read
 }

@@ -232,10 +232,11 @@ __global__ void __launch_bounds__(kRetThreads, 1) retention_chunk_kernel(const R
     const int cd = dim >> 3, cv = nv >> 3, per_row = 2 * cd + cv;
     const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)run.row0 * p.qkv_stride;
     const size_t k_at = (size_t)p.heads * dim + (size_t)h * dim, v_at = (size_t)2 * p.heads * dim + (size_t)h * vdim + c0;
+    // 16-byte piece tid, tid + 256, ... of a chunk as (row, piece of the row), without divisions in the loop
+    const int r_first = tid / per_row, c_first = tid - r_first * per_row, r_step = kRetThreads / per_row, c_step = kRetThreads - r_step * per_row;
     auto load = [&](int b) {
         const int st = b & 1, n = min(kRetChunk, run.count - b * kRetChunk);
-        for (int i = tid; i < kRetChunk * per_row; i += kRetThreads) {
-            const int r = i / per_row, c = i - r * per_row;
+        for (int r = r_first, c = c_first; r < kRetChunk; r += r_step + (c + c_step >= per_row), c += c_step - (c + c_step >= per_row ? per_row : 0)) {
             __nv_bfloat16* dst = c < cd ? qs + st * QK + r * PITCH + 8 * c : c < 2 * cd ? ks + st * QK + r * PITCH + 8 * (c - cd) : vs + st * VS + r * kRetVPitch + 8 * (c - 2 * cd);
             if (r < n) {
                 const __nv_bfloat16* src = base + (size_t)(b * kRetChunk + r) * p.qkv_stride + (c < cd ? (size_t)h * dim + 8 * c : c < 2 * cd ? k_at + 8 * (c - cd) : v_at + 8 * (c - 2 * cd));

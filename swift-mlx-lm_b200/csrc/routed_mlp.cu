@@ -1,8 +1,8 @@
 // Routed feed-forward: a router picks `top` of the experts for every row, the row's result is the weighted sum of theirs; a
 // shared feed-forward that every row takes, weighted by a sigmoid, may join the sum.
 //
-//   few rows (and fp32 plans)  routed_gate_kernel: every CTA works out its row's choice from the router's logits, then streams
-//                              gate and up rows of one chosen expert (the shared feed-forward is one more slot of the choice);
+//   few rows (and fp32 plans)  routed_gate_kernel: every CTA works out its row's choice from the router's logits, then its warps
+//                              stream gate and up rows of the chosen experts (and of the shared feed-forward);
 //                              routed_down_kernel: a warp per output runs through the chosen experts' down rows one after the
 //                              other, so the sum over experts needs no pass of its own.
 //   more rows (bf16)           routed_choose_kernel, routed_sort_kernel (rows sorted by expert, table of tiles), two grouped
@@ -45,6 +45,17 @@ __device__ __forceinline__ float rt_get(const float* p) { return *p; }
 __device__ __forceinline__ float rt_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void rt_put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void rt_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+// eight consecutive values, 16-byte aligned
+__device__ __forceinline__ void rt_get8(const float* p, float (&f)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void rt_get8(const __nv_bfloat16* p, float (&f)[8]) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const unsigned w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u); }
+}
 __device__ __forceinline__ float rt_lo(unsigned w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float rt_hi(unsigned w) { return __uint_as_float(w & 0xFFFF0000u); }
 __device__ __forceinline__ uint4 rt_stream(const void* p) {
@@ -113,51 +124,76 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
 }
 
 // ---- few rows ---------------------------------------------------------------------------------------------------------
-// CTA (share of the expert's rows, slot of the choice, row); the slot behind the last one is the shared feed-forward.
+// CTA (share of the work, row). A unit of work is one row of an expert's gate with the same row of its up, or without a gate two
+// rows of up; those of the shared feed-forward come first, because they are known before the choice.
+__host__ __device__ __forceinline__ int routed_units(int ff, bool gated) { return gated ? ff : (ff + 1) / 2; }
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedParams p) {
     pdl_launch_dependents();
-    pdl_wait();
     extern __shared__ __align__(16) float rt_smem[];
     __shared__ int sel[kMaxTop];
     __shared__ float weight[kMaxTop];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, slot = blockIdx.y, row = blockIdx.z;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y;
+    const int per = routed_units(p.sh.ff, GATED), shared = routed_units(p.sh.shared_ff, GATED), units = shared + p.sh.top * per;
+    const int chunks = p.in_ld >> 3;
+    constexpr int U = 4;
+    uint4 av[U], bv[U];
+    const __nv_bfloat16 *ar = nullptr, *br = nullptr;
+    int slot = 0, f = 0;
+    auto place = [&](int u) {   // rows of unit u
+        const bool mine = u >= shared;
+        slot = mine ? (u - shared) / per : p.sh.top;
+        f = mine ? u - shared - slot * per : u;
+        const __nv_bfloat16* up = mine ? p.up + (size_t)sel[slot] * p.sh.ff * p.in_ld : p.shared_up;
+        if (GATED) {
+            ar = up + (size_t)f * p.in_ld;
+            br = p.gate + ((size_t)sel[slot] * p.sh.ff + f) * p.in_ld;
+        } else {
+            f *= 2;
+            ar = up + (size_t)f * p.in_ld;
+            br = ar + (f + 1 < (mine ? p.sh.ff : p.sh.shared_ff) ? p.in_ld : 0);
+        }
+    };
+    auto load = [&](int c0) {
+#pragma unroll
+        for (int j = 0; j < U; ++j) {
+            const int c = c0 + 32 * j;
+            av[j] = c < chunks ? rt_stream(ar + 8 * c) : make_uint4(0, 0, 0, 0);
+            bv[j] = c < chunks ? rt_stream(br + 8 * c) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    const int first = blockIdx.x * kRtWarps + warp;
+    if (first < shared) { place(first); load(lane); }
+    pdl_wait();
     float* x = rt_smem;                    // [in_ld]
     float* s = x + p.in_ld;                // [experts], then [groups]
     const T* src = static_cast<const T*>(p.x) + (size_t)row * p.x_stride;
     for (int i = tid; i < p.in_ld; i += kRtThreads) x[i] = i < p.sh.width ? rt_get(src + i) : 0.f;
     choose<kRtThreads>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.experts, sel, weight, tid);
-    if (blockIdx.x == 0 && slot == 0 && tid < p.sh.top) {
+    if (blockIdx.x == 0 && tid < p.sh.top) {
         p.sel[row * p.sh.top + tid] = sel[tid];
         p.weight[row * p.sh.top + tid] = weight[tid];
     }
-    const bool shared = slot == p.sh.top;
-    const int ff = shared ? p.sh.shared_ff : p.sh.ff;
-    const size_t first = shared ? 0 : (size_t)sel[slot] * p.sh.ff;
-    const __nv_bfloat16* up = shared ? p.shared_up : p.up;
-    const int chunks = p.in_ld >> 3;
-    T* mid = shared ? static_cast<T*>(p.shared_mid) + (size_t)row * p.shared_stride : static_cast<T*>(p.mid) + (size_t)(row * p.sh.top + slot) * p.mid_stride;
-    constexpr int U = 4;
-    for (int f = blockIdx.x * kRtWarps + warp; f < ff; f += gridDim.x * kRtWarps) {
-        const __nv_bfloat16* gr = p.gate + (first + f) * p.in_ld;
-        const __nv_bfloat16* ur = up + (first + f) * p.in_ld;
-        float g = 0.f, u = 0.f;
+    for (int u = first; u < units; u += gridDim.x * kRtWarps) {
+        if (u != first || u >= shared) place(u);
+        float a = 0.f, b = 0.f;
         for (int c0 = lane; c0 < chunks; c0 += 32 * U) {
-            uint4 gv[U], uv[U];
+            if (c0 != lane || u != first || u >= shared) load(c0);
 #pragma unroll
             for (int j = 0; j < U; ++j) {
                 const int c = c0 + 32 * j;
-                gv[j] = GATED && c < chunks ? rt_stream(gr + 8 * c) : make_uint4(0, 0, 0, 0);
-                uv[j] = c < chunks ? rt_stream(ur + 8 * c) : make_uint4(0, 0, 0, 0);
-            }
-#pragma unroll
-            for (int j = 0; j < U; ++j) {
-                const int c = c0 + 32 * j;
-                if (c < chunks) { if (GATED) g = rt_dot8(gv[j], x + 8 * c, g); u = rt_dot8(uv[j], x + 8 * c, u); }
+                if (c < chunks) { a = rt_dot8(av[j], x + 8 * c, a); b = rt_dot8(bv[j], x + 8 * c, b); }
             }
         }
-        for (int o = 16; o > 0; o >>= 1) { if (GATED) g += __shfl_xor_sync(0xffffffffu, g, o); u += __shfl_xor_sync(0xffffffffu, u, o); }
-        if (lane == 0) rt_put(mid + f, GATED ? gated_activation(g, u, p.act) : gelu_erf(u));
+        for (int o = 16; o > 0; o >>= 1) { a += __shfl_xor_sync(0xffffffffu, a, o); b += __shfl_xor_sync(0xffffffffu, b, o); }
+        if (lane == 0) {
+            T* mid = slot == p.sh.top ? static_cast<T*>(p.shared_mid) + (size_t)row * p.shared_stride : static_cast<T*>(p.mid) + (size_t)(row * p.sh.top + slot) * p.mid_stride;
+            if (GATED) rt_put(mid + f, gated_activation(b, a, p.act));
+            else {
+                rt_put(mid + f, gelu_erf(a));
+                if (f + 1 < (slot == p.sh.top ? p.sh.shared_ff : p.sh.ff)) rt_put(mid + f + 1, gelu_erf(b));
+            }
+        }
     }
 }
 
@@ -191,15 +227,17 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
     const int first = half * 32 + lane;
     int n = (blockIdx.x * kRtWarps + warp) / kDownWarps;
     load(n, first);   // the first weights are on their way while the activations are gathered
-    for (int t = 0; t < top; ++t) {
-        const T* mid = static_cast<const T*>(p.mid) + (size_t)(row * top + t) * p.mid_stride;
-        const float w = weight[t];
-        for (int i = tid; i < p.mid_ld; i += kRtThreads) rt_smem[t * p.mid_ld + i] = i < p.sh.ff ? rt_get(mid + i) * w : 0.f;
-    }
-    if (p.shared_ld) {
-        const T* mid = static_cast<const T*>(p.shared_mid) + (size_t)row * p.shared_stride;
-        const float w = shared_weight(p, row);
-        for (int i = tid; i < p.shared_ld; i += kRtThreads) rt_smem[top * p.mid_ld + i] = i < p.sh.shared_ff ? rt_get(mid + i) * w : 0.f;
+    const float shared_w = p.shared_ld ? shared_weight(p, row) : 0.f;
+    for (int i = tid; i < all; i += kRtThreads) {   // eight activations each, times their weight; zeros in the padding
+        const int t = min(i / chunks, top), c = 8 * (i - t * chunks), ff = t < top ? p.sh.ff : p.sh.shared_ff;
+        const T* mid = t < top ? static_cast<const T*>(p.mid) + (size_t)(row * top + t) * p.mid_stride : static_cast<const T*>(p.shared_mid) + (size_t)row * p.shared_stride;
+        const float w = t < top ? weight[t] : shared_w;
+        float f[8];
+        rt_get8(mid + c, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = c + e < ff ? f[e] * w : 0.f;
+        *reinterpret_cast<float4*>(rt_smem + 8 * i) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(rt_smem + 8 * i + 4) = make_float4(f[4], f[5], f[6], f[7]);
     }
     __syncthreads();
     const int step = gridDim.x * kRtWarps / kDownWarps, rounds = (p.sh.width + step - 1) / step;
@@ -348,11 +386,12 @@ size_t down_smem(const RoutedShape& s) { return ((size_t)s.top * up8(s.ff) + up8
 
 template <typename T>
 int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
-    // about two CTAs per SM over the chosen experts of all rows
-    const int slots = p.sh.top + (p.sh.shared_ff ? 1 : 0);
-    const int pairs = (std::max(p.sh.ff, p.sh.shared_ff) + kRtWarps - 1) / kRtWarps, gx = std::max(1, std::min(pairs, (4 * 148 + slots * p.m - 1) / (slots * p.m)));
-    cudaError_t e = p.gate ? launch_k(routed_gate_kernel<T, true>, dim3(gx, slots, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p)
-                           : launch_k(routed_gate_kernel<T, false>, dim3(gx, slots, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
+    // up to four CTAs per SM, all with the same number of rounds
+    const bool gated = p.gate != nullptr;
+    const int units = p.sh.top * routed_units(p.sh.ff, gated) + routed_units(p.sh.shared_ff, gated);
+    const int most = std::max(1, (4 * 148 + p.m - 1) / p.m), rounds = (units + kRtWarps * most - 1) / (kRtWarps * most), gx = (units + kRtWarps * rounds - 1) / (kRtWarps * rounds);
+    cudaError_t e = gated ? launch_k(routed_gate_kernel<T, true>, dim3(gx, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p)
+                          : launch_k(routed_gate_kernel<T, false>, dim3(gx, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed gate launch");
     const int outs = (p.sh.width * kDownWarps + kRtWarps - 1) / kRtWarps, dx = std::max(1, std::min(outs, (4 * 148 + p.m - 1) / p.m));
     e = launch_k(routed_down_kernel<T>, dim3(dx, p.m), dim3(kRtThreads), down_smem(p.sh), s, p);

@@ -325,7 +325,7 @@ int stream_compile(swlm_plan* plan) {
             L.kind = L_ROUTED;
             const bool gated = s.weight2[0], shared = s.weight5[0];
             const RoutedShape shape = routed_shape(s);
-            if (!routed_supported(shape) || (shared && s.k2 <= 0)) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d, shared %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k, s.k2); return SWLM_ERR_UNSUPPORTED; }
+            if (!routed_supported(shape) || (shared && (s.k2 <= 0 || gated))) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d, shared %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k, s.k2); return SWLM_ERR_UNSUPPORTED; }
             if (s.score_act < 0 || s.score_act > SWLM_SCORE_SOFTMAX || s.group_best < 0 || s.group_best > 2) { set_error("routed feed-forward: scores %d, group %d", s.score_act, s.group_best); return SWLM_ERR_UNSUPPORTED; }
             if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || s.out_buf != SWLM_BUF_HIDDEN || s.n != d.hidden) { set_error("routed feed-forward: input in scratch 0..2, logits in scratch 3 or 4, result in hidden"); return SWLM_ERR_INVALID; }
             const char* suffix[3] = {s.weight2, s.weight3, s.weight4};
