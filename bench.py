@@ -614,8 +614,8 @@ def run_kalevik(args, pkg):
     batch, ctx, kv_heads = args.batch, args.ctx, heads // 4
     # two matrices per expert and a shared one of half the size: as many active entries as a gated feed-forward of `ff`
     routed, dense = K.RoutedFF(ff // top, experts, top, groups, keep, ff // 2), K.DenseFF(ff)
-    latent = K.LatentAttention(heads, 128, 64, 128, 512, 192 ** -0.5, 500000.0, 64)
-    parallel = K.Parallel(K.ChunkedAttention(heads, kv_heads, 128, 128, 128 ** -0.5, KALEVIK_CHUNK, 500000.0, 64, 4.0),
+    latent = K.LatentAttention(heads, 128, 64, 128, 512, 192 ** -0.5, 10000.0, 64)
+    parallel = K.Parallel(K.ChunkedAttention(heads, kv_heads, 128, 128, 128 ** -0.5, KALEVIK_CHUNK, 10000.0, 64, 8.0),
                           K.Retention(heads, 128, 128, tuple(1.0 - 2.0 ** (-5.0 - 7.0 * i / heads) for i in range(heads))), 0.7, 0.7)
     cfg = K.KalevikConfig(vocab=BENCH_VOCAB, width=width, layers=[K.Layer(parallel if i % 2 else latent, routed if i else dense) for i in range(layers)], loop=loop,
                           max_seq=bench_max_seq(args), max_batch=batch)
