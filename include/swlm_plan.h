@@ -92,6 +92,7 @@ enum {
     /* ---- steps of fp32-stream plans (swlm_buffers_desc.stream_dtype != 0); no counterpart in the reference ----
        Such plans also use EMBED (times `scale` when it is not 0), the three norm steps, SWIGLU / GEGLU and ARGMAX. */
     /* out[n] = sum_k W[n][k] in[k], W a dense bf16 matrix (swlm_weights_add_matrix_bf16), fp32 accumulation.
+       weight3 not empty: a bias [n] is added.
        weight2 not empty: a second matrix [n][k2] times the k2 columns that start at the next multiple of 8 behind the first
        k ones is added (the two are kept side by side and run as one product). */
     SWLM_STEP_PRODUCT = 13,
@@ -123,7 +124,7 @@ enum {
        eps2), q also times scale. decay = exp(-exp(A_log) * softplus(in3 + dt_bias)), beta = sigmoid(in2);
        S = decay * S; u = beta * (v - S^T k); S = S + k u^T; o = S^T q with S [key_dim][value_dim] fp32, zero at position 0.
        out = o * rsqrt(mean(o^2) + eps) * weight4 * activation(in4); gate_act: one of SWLM_GATE_*.
-       weight5 = A_log [heads], weight6 = dt_bias [heads * k]. */
+       weight5 = A_log [heads], weight6 = dt_bias [heads * k]. in2, in3 and in4 are read from columns in2_off, in3_off, in4_off on. */
     SWLM_STEP_GATED_DELTA = 18,
     /* Routed feed-forward: in_buf = input (n values), in2_buf = router logits (experts), out_buf = n values in hidden.
        s = sigmoid(logits); the experts form `groups` equal groups of neighbours, a group counts as the sum of its two largest
@@ -133,7 +134,10 @@ enum {
        score_act SWLM_SCORE_SOFTMAX: s = softmax(logits) over all experts. group_best 1: a group counts as its largest s.
        raw_weights 1: an expert's output is weighted with s * scale. weight2 empty: expert i is <weight4>(gelu(<weight3> in))
        with the exact (erf) GELU. weight5 not empty (only then): a feed-forward weight6 [n][k2] (gelu(weight5 [k2][n] in)) that every
-       token takes, its output times sigmoid(in2[experts]) is added. */
+       token takes, its output times sigmoid(in2[experts]) is added.
+       expert_act SWLM_EXPERT_SILU: gate and up are combined as silu(gate) * up. identity > 0: in2_buf holds experts + identity
+       logits; the last ones stand for experts without tensors whose output is the input (no groups then). weight7 not empty: a
+       vector [experts + identity] that is added to the scores for the choice only. */
     SWLM_STEP_ROUTED_MLP = 19,
     /* logits = scale * tanh(logits / scale), in place */
     SWLM_STEP_SOFTCAP = 20,
@@ -144,7 +148,11 @@ enum {
        the first rope_dim entries (rope_pairs as in LATENT_ATTN). Cached per token: k after that, and v. score = (q . k) *
        scale, softmax over the positions up to the token's own: window_left > 0: the last window_left of them; chunk > 0:
        those of the token's own chunk of `chunk` positions, counted from position 0. sink_one 1: one is added to the softmax's
-       denominator. out = sigmoid(gate) * value sum * out_scale. */
+       denominator. out = sigmoid(gate) * value sum * out_scale.
+       head_norm 1: q and k per head are divided by their root mean square (eps) without a weight. value_is_key 1: in_buf holds
+       q | k only and the values are the keys before their norm (value_dim = head_dim, no rotation); one row per token is cached.
+       temp_every > 0: q at position p is multiplied by 1 + temp_coef * ln((p + 1) div temp_every + 1). in4_buf from column
+       in4_off on (SWLM_BUF_NONE: none) = a gate per entry of the result, before its sigmoid, in the activation type. */
     SWLM_STEP_GROUPED_ATTN = 21,
     /* Retention with a state per sequence. in_buf from column in_off on = q | k | v (heads * key_dim, the same again, heads *
        value_dim), in4_buf from column in4_off on = output gate before its SiLU (heads * value_dim), out_buf from column
@@ -152,8 +160,25 @@ enum {
        S = decay_h * S + (scale * k) v^T; o = S^T q with S [key_dim][value_dim] fp32, zero at position 0;
        out = o * rsqrt(mean(o^2) + eps) * silu(gate) * out_scale. weight = decay [heads], an fp32 tensor.
        `layer` indexes the same states as GATED_DELTA. */
-    SWLM_STEP_RETENTION = 22
+    SWLM_STEP_RETENTION = 22,
+    /* ---- steps that act on the residual stream itself (sublayers that read the stream without a norm in front) ----
+       EMBED with out_buf = RESIDUAL starts such a stream; COPY_RMSNORM with in_buf = RESIDUAL norms it as it is.
+       Neighbours among the following steps run as one launch. */
+    /* t = in_buf (fp32), times sigmoid(in3_buf) (fp32; SWLM_BUF_NONE: no gate); residual += t * rsqrt(mean(t^2)+eps) * (weight + weight_bias) */
+    SWLM_STEP_GATED_POSTNORM_ADD = 23,
+    /* Depth-wise average: the stream is kept as result k - 1 of the pass (the embedding output is result 0), and becomes
+       sum over j < k of weight[j] * result j. */
+    SWLM_STEP_DEPTH_AVG = 24,
+    /* out_buf = h + conv(h), h the residual stream and conv a causal convolution over conv_kernel tokens per channel (weight
+       [n][conv_kernel], the last column meets the current token; zeros before the start). `layer` indexes the stream_convs
+       states that keep the last inputs of a sequence. */
+    SWLM_STEP_STREAM_CONV = 25,
+    /* out_buf = the residual stream, in the activation type */
+    SWLM_STEP_STREAM_COPY = 26,
+    /* out = gelu_tanh(in) * weight[token][in2_off ..], weight a table with a row per token of the vocabulary */
+    SWLM_STEP_TOKEN_GATE = 27
 };
+enum { SWLM_EXPERT_CLAMPED = 0, SWLM_EXPERT_SILU = 1 };
 enum { SWLM_GATE_SILU = 0, SWLM_GATE_SIGMOID = 1 };
 enum { SWLM_SCORE_SIGMOID = 0, SWLM_SCORE_SOFTMAX = 1 };
 enum { SWLM_ROPE_HALVES = 0, SWLM_ROPE_NEIGHBOURS = 1 };
@@ -217,6 +242,15 @@ typedef struct swlm_step {
     int32_t score_act;     /* SWLM_SCORE_* */
     int32_t group_best;    /* 0 = 2 */
     int32_t raw_weights;
+    int32_t in2_off;
+    int32_t in3_off;
+    int32_t value_is_key;  /* GROUPED_ATTN */
+    int32_t head_norm;
+    float   temp_coef;
+    int32_t temp_every;
+    int32_t identity;      /* ROUTED_MLP */
+    int32_t expert_act;    /* SWLM_EXPERT_* */
+    char    weight7[SWLM_NAME_MAX];
 } swlm_step;
 
 /* Sizes of the runtime buffer set; mirrors the inputs of
@@ -271,6 +305,8 @@ typedef struct swlm_buffers_desc {
     int32_t delta_layers;    /* number of SWLM_STEP_GATED_DELTA and SWLM_STEP_RETENTION layers: fp32 state (and convolution
                                 inputs) per sequence */
     int32_t grouped_layers;  /* number of SWLM_STEP_GROUPED_ATTN layers (page pools of keys and values) */
+    int32_t stream_convs;    /* number of SWLM_STEP_STREAM_CONV states */
+    int32_t depth_results;   /* results SWLM_STEP_DEPTH_AVG keeps (the embedding output among them); 0: none */
 } swlm_buffers_desc;
 
 enum { SWLM_STREAM_BF16 = 0, SWLM_STREAM_F32 = 1, SWLM_STREAM_ALL_F32 = 2 };

@@ -25,9 +25,10 @@ from .plan import (  # noqa: F401
     lfm2_like_config,
 )
 from .model import InferenceModel, WeightStore, bundle_tensors, load_model, load_model_from_staf, upload_weights  # noqa: F401
-from . import bundle, formats, kalevik, plan, rirotar, staf, tp, vuzunex  # noqa: F401
+from . import bundle, formats, kalevik, merudra, plan, rirotar, staf, tp, vuzunex  # noqa: F401
 from .bundle import load_bundle, prepare_bundle, prepare_dense_bundle  # noqa: F401
 from .kalevik import KalevikConfig, KalevikPlanBuilder  # noqa: F401
+from .merudra import MerudraConfig, MerudraPlanBuilder  # noqa: F401
 from .rirotar import RirotarConfig, RirotarPlanBuilder  # noqa: F401
 from .scheduler import BatchScheduler, Request, SequenceSlots  # noqa: F401
 from .vuzunex import VuzunexConfig, VuzunexPlanBuilder  # noqa: F401

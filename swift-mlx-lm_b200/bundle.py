@@ -17,6 +17,7 @@ import os
 from typing import Dict, Optional, Tuple
 
 from . import kalevik as _kalevik
+from . import merudra as _merudra
 from . import rirotar as _rirotar
 from . import staf as _staf
 from . import vuzunex as _vuzunex
@@ -33,6 +34,7 @@ ARCHITECTURES = {
     _vuzunex.ARCHITECTURE: (lambda config, shapes, **runtime: _vuzunex.decode_config(config, **runtime), _vuzunex.VuzunexPlanBuilder),
     _rirotar.ARCHITECTURE: (_rirotar.decode_config, _rirotar.RirotarPlanBuilder),
     _kalevik.ARCHITECTURE: (_kalevik.decode_config, _kalevik.KalevikPlanBuilder),
+    _merudra.ARCHITECTURE: (_merudra.decode_config, _merudra.MerudraPlanBuilder),
 }
 
 # KVCachePolicy of InferencePolicy.default (Sources/MetalCompiler/InferencePolicy.swift:55-100)

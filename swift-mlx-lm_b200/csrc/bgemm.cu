@@ -27,18 +27,21 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 }
 
 // Where the results of one weight row go: that of activation row m is m * stride bytes behind y.
-struct ProductRow { unsigned char* y; size_t stride; bool f32; };
+struct ProductRow { unsigned char* y; size_t stride; bool f32; float bias; };
 __device__ __forceinline__ ProductRow product_row(const ProductOut& o, int row) {
     void* y = o.y[0];
+    const __nv_bfloat16* bias = o.bias[0];
     int first = 0, stride = o.stride[0], f32 = o.f32[0];
 #pragma unroll
     for (int q = 1; q < kMaxProductSegs; ++q)
-        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; }
+        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; bias = o.bias[q]; }
     const int size = f32 ? 4 : 2;
-    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0};
+    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0,
+                      bias && row < o.end[o.count - 1] ? __bfloat162float(bias[row - first]) : 0.f};
 }
 __device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
     const ProductRow r = product_row(o, row);
+    val += r.bias;
     if (o.softcap > 0.f) val = o.softcap * tanhf(val / o.softcap);
     if (o.gelu) val = gelu_erf(val);
     if (r.f32) *reinterpret_cast<float*>(r.y + m * r.stride) = val;
@@ -56,6 +59,7 @@ struct GemvParams {
     int ld, n, k, m;
     GatedAct act;
     const void* x; int x_stride;
+    const void* x2; int x2_stride, split;        // rows from `split` on (a multiple of four) meet a second input
     StreamNorm norm;
     ProductOut out;
 };
@@ -218,6 +222,11 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
             const T* src = static_cast<const T*>(p.x) + (size_t)m * p.x_stride;
             for (int i = tid; i < p.ld; i += kGemvThreads) { T v = T(0.0f); if (i < p.k) v = src[i]; xs[(size_t)m * p.ld + i] = v; }
         }
+        if (p.x2)
+            for (int m = 0; m < MR; ++m) {
+                const T* src = static_cast<const T*>(p.x2) + (size_t)m * p.x2_stride;
+                for (int i = tid; i < p.ld; i += kGemvThreads) { T v = T(0.0f); if (i < p.k) v = src[i]; xs[(size_t)(MR + m) * p.ld + i] = v; }
+            }
     }
     __syncthreads();
 
@@ -229,6 +238,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
 #pragma unroll
             for (int m = 0; m < MR; ++m) acc[i][m] = 0.f;
         const bool live = group < groups;
+        const T* xg = xs + (p.x2 && group * ROWS >= p.split ? (size_t)MR * p.ld : 0);
         if (live) {
             for (int c0 = first_chunk; c0 < chunks; c0 += STEP * kGemvUnroll) {
                 if (it > 0 || c0 != first_chunk) load(group, c0);
@@ -246,7 +256,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
 #pragma unroll
                         for (int m = 0; m < MR; ++m) {
                             float xf[8];
-                            get_x8(xs + (size_t)m * p.ld + 8 * c, xf);
+                            get_x8(xg + (size_t)m * p.ld + 8 * c, xf);
 #pragma unroll
                             for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -445,7 +455,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
 #pragma unroll 1
             for (int t = 0; t < (GATED && !cut ? 1 : nt); ++t) {
                 const int row = row0 + (GATED ? 0 : t * kTileRows) + quarter * 32 + lane;
-                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true}
+                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true, 0.f}
                                            : product_row(p.out, row);
 #pragma unroll 1
                 for (int c0 = 16 * ((warp - 2) >> 2); c0 < BN; c0 += 16 * (kTcEpilogueWarps / 4)) {
@@ -462,6 +472,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
                         for (int i = 0; i < 16; ++i) {
                             float val = __uint_as_float(v[i]);
                             if (GATED && !cut) val = gated_activation(val, __uint_as_float(u[i]), p.act);
+                            val += dst.bias;
                             if (p.out.softcap > 0.f && !cut) val = p.out.softcap * tanhf(val / p.out.softcap);
                             if (p.out.gelu && !cut) val = gelu_erf(val);
                             if (i < count) {
@@ -672,6 +683,8 @@ bool product_takes_norm(int m, int k) { return m <= 2 && k <= 16384 && gemv_fits
 // gate and up in one launch: always, except as true fp32 products over many rows
 bool product_takes_gate(int m, int k, bool x_f32) { return !x_f32 || gemv_fits(m, k, true, false); }
 
+bool product_takes_two(int m, int k, int split, bool x_f32) { return m <= kGemvRows && !(split & 3) && gemv_smem(2 * m, (k + 7) / 8 * 8, x_f32, false) <= kGemvMaxSmem; }
+
 size_t product_part_floats(int n, int k, int m, bool gated) {
     if (gemv_fits(m, k, false, false)) return 0;
     const TcShape t = tc_shape(n, k, m, gated);
@@ -700,9 +713,12 @@ int launch_product(const ProductLaunch& a, cudaStream_t s) {
         GemvParams p{};
         p.w = a.w->data; p.w2 = gated ? a.w2->data : nullptr; p.ld = a.w->ld; p.n = a.w->n; p.k = a.w->k; p.m = a.m; p.act = a.act;
         p.x = a.x; p.x_stride = a.x_stride; p.norm = a.norm; p.out = a.out;
-        const size_t smem = gemv_smem(a.m, a.w->ld, a.x_f32, a.norm.mode != 0);
+        if (a.x2 && (gated || a.norm.mode || !product_takes_two(a.m, a.w->k, a.split, a.x_f32))) { set_error("two inputs of a product over %d rows run one after the other", a.m); return SWLM_ERR_INVALID; }
+        p.x2 = a.x2; p.x2_stride = a.x2_stride; p.split = a.split;
+        const size_t smem = gemv_smem(a.x2 ? 2 * a.m : a.m, a.w->ld, a.x_f32, a.norm.mode != 0);
         return a.x_f32 ? gemv_rows<float>(p, gated, smem, s) : gemv_rows<__nv_bfloat16>(p, gated, smem, s);
     }
+    if (a.x2) { set_error("two inputs of a product over %d rows run one after the other", a.m); return SWLM_ERR_INVALID; }
     if (a.norm.mode) { set_error("a norm in front of a product over %d rows runs on its own", a.m); return SWLM_ERR_INVALID; }
     if (a.x_f32) {
         if (gated) { set_error("gate and up of fp32 rows run one after the other"); return SWLM_ERR_INVALID; }

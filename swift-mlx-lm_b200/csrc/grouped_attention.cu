@@ -11,6 +11,9 @@
 // Both multiply on tensor cores with fp32 sums; softmax weights enter as bf16 hi + lo pairs. grouped_simple_kernel (fp32 FMAs)
 // serves fp32 caches and head sizes beyond the others. The newest rows are read back from the cache like all others, so a row's
 // result does not depend on how a sequence was cut into batches.
+//
+// Where the values are the keys before their norm, one row per token is kept and read as key and as value; the norm is a number
+// per row that scales the row's score.
 #include <cooperative_groups.h>
 
 #include <algorithm>
@@ -54,6 +57,8 @@ struct GroupedParams {
     const __nv_bfloat16 *q_norm, *k_norm;
     void* qkv; int qkv_stride;
     const float* gate; int gate_stride;
+    const void* entry_gate; int entry_gate_stride;
+    int head_norm, temp_every; float temp_coef;
     void* pool;
     const int32_t* page_table; int pages_per_seq;
     const int32_t* row_seq; const int32_t* row_pos;
@@ -69,11 +74,19 @@ __device__ __forceinline__ int ga_first_seen(const GroupedParams& p, int pos) {
     return max(w, c);
 }
 __device__ __forceinline__ int ga_row(const GroupedParams& p, int i) { return p.rows ? p.rows[i] : i; }
-// keys of head g in the page of a position; its values lie kPage * pk entries behind
+// keys of head g in the page of a position; ga_values: where its values lie, ga_factors: what turns shared rows into keys
 template <typename T>
 __device__ __forceinline__ T* ga_block(const GroupedParams& p, int seq, int page_index, int g) {
     const int page = p.page_table[(size_t)seq * p.pages_per_seq + page_index];
     return static_cast<T*>(p.pool) + ((size_t)page * p.row.groups + g) * p.row.block;
+}
+__device__ __forceinline__ int ga_values(const GroupedRow& r) { return r.shared ? 0 : kPage * r.pk; }
+template <typename T>
+__device__ __forceinline__ float* ga_factors(const GroupedParams& p, const T* block) { return reinterpret_cast<float*>(const_cast<T*>(block) + (size_t)kPage * p.row.pk); }
+// the gate of entry c of head h
+template <typename T>
+__device__ __forceinline__ float ga_entry_gate(const GroupedParams& p, int r, int h, int c) {
+    return 1.0f / (1.0f + expf(-ga_get(static_cast<const T*>(p.entry_gate) + (size_t)r * p.entry_gate_stride + (size_t)h * p.row.vdim + c)));
 }
 __device__ __forceinline__ float ga_gate(const GroupedParams& p, int r, int h) {
     return (p.gate ? 1.0f / (1.0f + expf(-p.gate[(size_t)r * p.gate_stride + h])) : 1.0f) * p.out_scale;
@@ -89,7 +102,7 @@ __global__ void __launch_bounds__(kAppWarps * 32) grouped_append_kernel(const Gr
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, r = blockIdx.x, i = blockIdx.y * kAppWarps + warp;
     const int G = p.row.groups, dim = p.row.dim, vdim = p.row.vdim;
-    if (i >= p.heads + 2 * G) return;
+    if (i >= p.heads + (p.row.shared ? G : 2 * G)) return;
     const int pos = p.row_pos[r], seq = p.row_seq[r];
     T* base = static_cast<T*>(p.qkv) + (size_t)r * p.qkv_stride;
     if (i >= p.heads + G) {
@@ -109,6 +122,12 @@ __global__ void __launch_bounds__(kAppWarps * 32) grouped_append_kernel(const Gr
         const float sc = 1.0f / sqrtf(ss / (float)dim + p.eps);
         for (int c = lane; c < dim; c += 32) x[c] = x[c] * sc * (__bfloat162float(w[c]) + p.weight_bias);
     }
+    float f = p.head_norm ? 1.0f / sqrtf(ss / (float)dim + p.eps) : 1.0f;
+    if (p.row.shared && i >= p.heads) {   // the row as it is; its norm becomes a factor of the scores
+        if (lane == 0) ga_factors(p, ga_block<T>(p, seq, pos / kPage, i - p.heads))[pos % kPage] = f;
+        f = 1.0f;
+    }
+    if (i < p.heads && p.temp_every > 0) f *= 1.0f + p.temp_coef * logf((float)((pos + 1) / p.temp_every) + 1.0f);
     __syncwarp();
     T* dst = i < p.heads ? src : ga_block<T>(p, seq, pos / kPage, i - p.heads) + (size_t)(pos % kPage) * p.row.pk;
     for (int c = lane; c < dim; c += 32) {
@@ -120,7 +139,7 @@ __global__ void __launch_bounds__(kAppWarps * 32) grouped_append_kernel(const Gr
             const float o = x[e.partner];
             v = p.magnitude * (e.first ? v * cs - o * sn : v * cs + o * sn);
         }
-        ga_put(dst + c, v);
+        ga_put(dst + c, v * f);
     }
 }
 
@@ -145,11 +164,12 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) grouped_simple_kernel(const
     for (int key = ga_first_seen(p, pos) + warp; key <= pos; key += kSimpleWarps) {
         const T* block = ga_block<T>(p, seq, key / kPage, g);
         const T* k = block + (size_t)(key % kPage) * p.row.pk;
-        const T* v = block + (size_t)kPage * p.row.pk + (size_t)(key % kPage) * p.row.pv;
+        const T* v = block + ga_values(p.row) + (size_t)(key % kPage) * p.row.pv;
         float s = 0.f;
         for (int i = lane; i < dim; i += 32) s = fmaf(q[i], ga_get(k + i), s);
         for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
         s *= p.scale_log2;
+        if (p.row.shared) s *= ga_factors(p, block)[key % kPage];
         const float m_new = fmaxf(m, s), corr = exp2f(m - m_new), w = exp2f(s - m_new);
         l = l * corr + w;
         m = m_new;
@@ -166,7 +186,7 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) grouped_simple_kernel(const
     for (int i = threadIdx.x; i < vdim; i += blockDim.x) {
         float v = 0.f;
         for (int w = 0; w < kSimpleWarps; ++w) v += simple_smem[dim + (size_t)w * vdim + i] * exp2f(ms[w] - top);
-        ga_put(out + i, v * f);
+        ga_put(out + i, v * f * (p.entry_gate ? ga_entry_gate<T>(p, r, h, i) : 1.0f));
     }
 }
 
@@ -190,7 +210,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
     pdl_wait();
     const int r = ga_row(p, blockIdx.z), pos = p.row_pos[r], seq = p.row_seq[r];
     const int seen0 = ga_first_seen(p, pos), unit0 = seen0 / UK, units = pos / UK + 1 - unit0;
-    const int pk = p.row.pk, pv = p.row.pv, k_bytes = UK * pk * 2, v_bytes = UK * pv * 2;
+    const int pk = p.row.pk, pv = p.row.pv, k_bytes = UK * pk * 2, v_bytes = p.row.shared ? UK * 4 : UK * pv * 2;   // (shared rows: their factors instead of values)
     unsigned char* stage = dec_smem + (size_t)warp * (k_bytes + v_bytes);
     const unsigned bar_at = smem_u32(&bar[warp]);
     auto request = [&](int u) {   // lane 0
@@ -198,7 +218,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
         const __nv_bfloat16* block = ga_block<__nv_bfloat16>(p, seq, key0 / kPage, kv);
         mbar_expect(bar_at, (unsigned)(k_bytes + v_bytes));
         bulk_load(smem_u32(stage), block + (size_t)(key0 % kPage) * pk, (unsigned)k_bytes, bar_at);
-        bulk_load(smem_u32(stage) + (unsigned)k_bytes, block + (size_t)kPage * pk + (size_t)(key0 % kPage) * pv, (unsigned)v_bytes, bar_at);
+        bulk_load(smem_u32(stage) + (unsigned)k_bytes, block + (size_t)kPage * pk + (size_t)(key0 % kPage) * (p.row.shared ? 2 : pv), (unsigned)v_bytes, bar_at);
     };
     const int first = rank * kDecWarps + warp, step = nz * kDecWarps;
     if (lane == 0 && first < units) request(first);
@@ -218,7 +238,8 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
 #pragma unroll
     for (int j = 0; j < 2 * NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-    const unsigned ks = smem_u32(stage), vs = ks + (unsigned)k_bytes;
+    const unsigned ks = smem_u32(stage), vs = p.row.shared ? ks : ks + (unsigned)k_bytes;
+    const float* factors = reinterpret_cast<const float*>(stage + k_bytes);
     unsigned phase = 0;
     for (int u = first; u < units; u += step, phase ^= 1) {
         if (!mbar_wait(&bar[warp], phase)) {
@@ -248,8 +269,9 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
             for (int e = 0; e < 2; ++e) {
                 const int key = key0 + 8 * j + 2 * t + e;
                 const bool seen = key <= pos && key >= seen0;
-                sacc[j][e] = seen ? sacc[j][e] * p.scale_log2 : -INFINITY;
-                sacc[j][2 + e] = seen ? sacc[j][2 + e] * p.scale_log2 : -INFINITY;
+                const float f = p.row.shared ? p.scale_log2 * factors[8 * j + 2 * t + e] : p.scale_log2;
+                sacc[j][e] = seen ? sacc[j][e] * f : -INFINITY;
+                sacc[j][2 + e] = seen ? sacc[j][2 + e] * f : -INFINITY;
                 mx_a = fmaxf(mx_a, sacc[j][e]); mx_b = fmaxf(mx_b, sacc[j][2 + e]);
             }
 #pragma unroll
@@ -352,6 +374,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
         float v = 0.f;
 #pragma unroll
         for (int z = 0; z < kDecCluster; ++z) v = fmaf(all_m[z][hh], cluster.map_shared_rank(own, z < nz ? z : rank)[i], v);
+        if (c < p.row.vdim && p.entry_gate) v *= ga_entry_gate<__nv_bfloat16>(p, r, h0 + hh, c);
         if (c < p.row.vdim) static_cast<__nv_bfloat16*>(p.out)[(size_t)r * p.out_stride + (size_t)(h0 + hh) * p.row.vdim + c] = __float2bfloat16_rn(v);
     }
     cluster.sync();   // nobody leaves while others still read
@@ -407,7 +430,8 @@ __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const Gr
     for (; i < n_tiles; ++i) {
         if (!mbar_wait(&full_bar[i % kPfStages], (unsigned)((i / kPfStages) & 1))) { atomicExch(p.status, 62); bad = 1; }
         const int key0 = (kt0 + i) * kPage;
-        const unsigned kb = smem_u32(pf_smem) + (unsigned)(i % kPfStages * stage_bytes), vb = kb + (unsigned)(kPage * pk) * 2u;
+        const unsigned kb = smem_u32(pf_smem) + (unsigned)(i % kPfStages * stage_bytes), vb = p.row.shared ? kb : kb + (unsigned)(kPage * pk) * 2u;
+        const float* factors = reinterpret_cast<const float*>(pf_smem + (size_t)(i % kPfStages) * stage_bytes + (size_t)kPage * pk * 2);
         if (warp_first <= last_pos && key0 <= warp_last && key0 + kPage > warp_seen) {
             float sacc[8][4];
 #pragma unroll
@@ -430,8 +454,9 @@ __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const Gr
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = key0 + 8 * j + 2 * t + e;
-                    const float a = !edge || (key <= pos_a && key >= seen_a) ? sacc[j][e] * p.scale_log2 : -INFINITY;
-                    const float b = !edge || (key <= pos_b && key >= seen_b) ? sacc[j][2 + e] * p.scale_log2 : -INFINITY;
+                    const float f = p.row.shared ? p.scale_log2 * factors[8 * j + 2 * t + e] : p.scale_log2;
+                    const float a = !edge || (key <= pos_a && key >= seen_a) ? sacc[j][e] * f : -INFINITY;
+                    const float b = !edge || (key <= pos_b && key >= seen_b) ? sacc[j][2 + e] * f : -INFINITY;
                     sacc[j][e] = a; sacc[j][2 + e] = b;
                     mx_a = fmaxf(mx_a, a); mx_b = fmaxf(mx_b, b);
                 }
@@ -500,7 +525,11 @@ __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const Gr
 #pragma unroll
         for (int j = 0; j < 2 * NV; ++j) {
             const int c = 8 * j + 2 * t;
-            if (c < p.row.vdim) *reinterpret_cast<unsigned*>(o + c) = ga_pack(oacc[j][2 * half] * f, oacc[j][2 * half + 1] * f);
+            if (c < p.row.vdim) {
+                float x = oacc[j][2 * half] * f, y = oacc[j][2 * half + 1] * f;
+                if (p.entry_gate) { x *= ga_entry_gate<__nv_bfloat16>(p, row, h, c); y *= ga_entry_gate<__nv_bfloat16>(p, row, h, c + 1); }
+                *reinterpret_cast<unsigned*>(o + c) = ga_pack(x, y);
+            }
         }
     }
 }
@@ -514,7 +543,7 @@ int form_of(const GroupedRow& r, bool f32) {
 }
 constexpr size_t kGaMaxSmem = 200 * 1024;
 size_t decode_smem(const GroupedRow& r, int share, int unit) {
-    const size_t stages = (size_t)kDecWarps * unit * (r.pk + r.pv) * 2, sums = (size_t)(kDecWarps + 1) * std::min(share, kDecHeads) * r.vp * 4;
+    const size_t stages = (size_t)kDecWarps * unit * (r.shared ? 2 * r.pk + 4 : 2 * (r.pk + r.pv)), sums = (size_t)(kDecWarps + 1) * std::min(share, kDecHeads) * r.vp * 4;
     return std::max(stages, sums);
 }
 size_t simple_bytes(const GroupedRow& r) { return ((size_t)r.dim + (size_t)kSimpleWarps * r.vdim) * 4; }
@@ -546,12 +575,12 @@ int decode_cluster(const GroupedLaunch& a, int unit) {
 
 }  // namespace
 
-GroupedRow grouped_row(int groups, int dim, int vdim, bool f32) {
+GroupedRow grouped_row(int groups, int dim, int vdim, bool f32, bool shared) {
     GroupedRow r;
-    r.groups = groups; r.dim = dim; r.vdim = vdim;
+    r.groups = groups; r.dim = dim; r.vdim = vdim; r.shared = shared;
     r.dp = (dim + 15) / 16 * 16; r.vp = (vdim + 15) / 16 * 16;
     r.pk = r.dp + (f32 ? 0 : 8); r.pv = r.vp + (f32 ? 0 : 8);
-    r.block = kPage * (r.pk + r.pv);
+    r.block = shared ? kPage * (r.pk + (f32 ? 1 : 2)) : kPage * (r.pk + r.pv);
     return r;
 }
 bool grouped_supported(const GroupedRow& r) { return r.dim <= 4096 && simple_bytes(r) <= kGaMaxSmem; }
@@ -573,12 +602,13 @@ int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches) {
     p.row = a.row; p.heads = a.heads; p.share = a.heads / a.row.groups; p.rot_dims = a.rot_dims; p.rot_neighbours = a.rot_neighbours;
     p.window = a.window; p.chunk = a.chunk; p.sink_one = a.sink_one;
     p.scale_log2 = a.scale * kLog2e; p.eps = a.eps; p.weight_bias = a.weight_bias; p.magnitude = a.magnitude; p.out_scale = a.out_scale; p.inv_freq = a.inv_freq;
+    p.head_norm = a.head_norm; p.temp_every = a.temp_every; p.temp_coef = a.temp_coef; p.entry_gate = a.entry_gate; p.entry_gate_stride = a.entry_gate_stride;
     p.q_norm = a.q_norm; p.k_norm = a.k_norm; p.qkv = a.qkv; p.qkv_stride = a.qkv_stride; p.gate = a.gate; p.gate_stride = a.gate_stride;
     p.pool = a.pool; p.page_table = a.page_table; p.pages_per_seq = a.pages_per_seq; p.row_seq = a.row_seq; p.row_pos = a.row_pos;
     p.out = a.out; p.out_stride = a.out_stride; p.spans = a.spans; p.tiles = a.tiles; p.status = a.status;
     cudaError_t e;
     if (!a.only_attention) {
-        const dim3 grid(a.n_rows, (a.heads + 2 * a.row.groups + kAppWarps - 1) / kAppWarps);
+        const dim3 grid(a.n_rows, (a.heads + (a.row.shared ? 1 : 2) * a.row.groups + kAppWarps - 1) / kAppWarps);
         const size_t smem = (size_t)kAppWarps * a.row.dim * 4;
         e = a.f32 ? launch_k(grouped_append_kernel<float>, grid, dim3(kAppWarps * 32), smem, s, p) : launch_k(grouped_append_kernel<__nv_bfloat16>, grid, dim3(kAppWarps * 32), smem, s, p);
         if (e != cudaSuccess) return cuda_fail(e, "grouped append launch");

@@ -25,6 +25,7 @@ struct RoutedParams {
     float scale;
     GatedAct act;
     int softmax, group_best, raw_weights;
+    const __nv_bfloat16* correction;
     int m;
     const void* x; int x_stride;
     const float* z; int z_stride;
@@ -71,12 +72,37 @@ __device__ __forceinline__ float rt_dot8(const uint4& w, const float* x, float a
 
 __device__ __forceinline__ float shared_weight(const RoutedParams& p, int row) { return 1.0f / (1.0f + expf(-p.z[(size_t)row * p.z_stride + p.sh.experts])); }
 
-// The choice of one row by THREADS threads (a warp or the CTA). s: [experts] scores, gs: [groups] group scores, both shared;
-// sel / w: [top] in order of falling score.
+// from the chosen scores to the weights
 template <int THREADS>
-__device__ __forceinline__ void choose(const RoutedParams& p, const float* z, float* s, float* gs, int* sel, float* w, int tid) {
+__device__ __forceinline__ void weigh(const RoutedParams& p, float* w, int tid) {
+    float total = 0.f;
+    for (int i = 0; i < p.sh.top; ++i) total += w[i];
+    if (THREADS == 32) __syncwarp(); else __syncthreads();
+    for (int i = tid; i < p.sh.top; i += THREADS) w[i] = p.raw_weights ? w[i] * p.scale : w[i] / (total + 1e-20f) * p.scale;
+}
+
+// Experts with tensors first, those that hand the input through behind them (one warp; top <= 64); returns the number of the first.
+__device__ __forceinline__ int real_first(const RoutedShape& sh, int* sel, float* w, int lane) {
+    if (!sh.identity) return sh.top;
+    const int a = lane < sh.top ? sel[lane] : 0, b = lane + 32 < sh.top ? sel[lane + 32] : 0;
+    const float wa = lane < sh.top ? w[lane] : 0.f, wb = lane + 32 < sh.top ? w[lane + 32] : 0.f;
+    const unsigned lower = (1u << lane) - 1u;
+    const unsigned la = __ballot_sync(0xffffffffu, lane < sh.top), lb = __ballot_sync(0xffffffffu, lane + 32 < sh.top);
+    const unsigned ra = __ballot_sync(0xffffffffu, lane < sh.top && a < sh.experts), rb = __ballot_sync(0xffffffffu, lane + 32 < sh.top && b < sh.experts);
+    const int real = __popc(ra) + __popc(rb);
+    __syncwarp();
+    if (lane < sh.top) { const int at = a < sh.experts ? __popc(ra & lower) : real + __popc(la & ~ra & lower); sel[at] = a; w[at] = wa; }
+    if (lane + 32 < sh.top) { const int at = b < sh.experts ? __popc(ra) + __popc(rb & lower) : real + __popc(la & ~ra) + __popc(lb & ~rb & lower); sel[at] = b; w[at] = wb; }
+    return real;
+}
+
+// The choice of one row by THREADS threads (a warp or the CTA). s: [experts] scores, gs: [groups] group scores, both shared;
+// sel / w: [top] in order of falling score. With a correction the choice looks at s + correction, kept in cs: [scored]; the weights
+// are the plain scores.
+template <int THREADS>
+__device__ __forceinline__ void choose(const RoutedParams& p, const float* z, float* s, float* gs, float* cs, int* sel, float* w, int tid) {
     auto sync = [] { if (THREADS == 32) __syncwarp(); else __syncthreads(); };
-    const int E = p.sh.experts, G = p.sh.groups, per = E / G;
+    const int E = p.sh.scored(), G = p.sh.groups, per = E / G;
     for (int i = tid; i < p.sh.top; i += THREADS) { sel[i] = i; w[i] = 0.f; }   // indices stay valid whatever the logits are
     if (p.softmax) {   // every warp works out maximum and sum for itself
         float top = -INFINITY, sum = 0.f;
@@ -89,6 +115,20 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
         for (int e = tid; e < E; e += THREADS) s[e] = 1.0f / (1.0f + expf(-z[e]));
     }
     sync();
+    if (p.correction) {
+        for (int e = tid; e < E; e += THREADS) cs[e] = s[e] + __bfloat162float(p.correction[e]);
+        sync();
+        for (int e = tid; e < E; e += THREADS) {
+            const float v = cs[e];
+            int before = 0;
+            for (int o = 0; o < E; ++o) before += cs[o] > v || (cs[o] == v && o < e);
+            if (before < p.sh.top) { sel[before] = e; w[before] = s[e]; }
+        }
+        sync();
+        weigh<THREADS>(p, w, tid);
+        sync();
+        return;
+    }
     for (int g = tid; g < G; g += THREADS) {
         float first = 0.f, second = 0.f;   // scores are not negative
         for (int e = g * per; e < (g + 1) * per; ++e) {
@@ -116,10 +156,7 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
         if (v >= 0.f && before < p.sh.top) { sel[before] = e; w[before] = v; }
     }
     sync();
-    float total = 0.f;
-    for (int i = 0; i < p.sh.top; ++i) total += w[i];
-    sync();
-    for (int i = tid; i < p.sh.top; i += THREADS) w[i] = p.raw_weights ? w[i] * p.scale : w[i] / (total + 1e-20f) * p.scale;
+    weigh<THREADS>(p, w, tid);
     sync();
 }
 
@@ -133,8 +170,9 @@ __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedPar
     extern __shared__ __align__(16) float rt_smem[];
     __shared__ int sel[kMaxTop];
     __shared__ float weight[kMaxTop];
+    __shared__ int real_s;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y;
-    const int per = routed_units(p.sh.ff, GATED), shared = routed_units(p.sh.shared_ff, GATED), units = shared + p.sh.top * per;
+    const int per = routed_units(p.sh.ff, GATED), shared = routed_units(p.sh.shared_ff, GATED);
     const int chunks = p.in_ld >> 3;
     constexpr int U = 4;
     uint4 av[U], bv[U];
@@ -166,10 +204,13 @@ __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedPar
     if (first < shared) { place(first); load(lane); }
     pdl_wait();
     float* x = rt_smem;                    // [in_ld]
-    float* s = x + p.in_ld;                // [experts], then [groups]
+    float* s = x + p.in_ld;                // [scored], then [groups], then [scored]
     const T* src = static_cast<const T*>(p.x) + (size_t)row * p.x_stride;
     for (int i = tid; i < p.in_ld; i += kRtThreads) x[i] = i < p.sh.width ? rt_get(src + i) : 0.f;
-    choose<kRtThreads>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.experts, sel, weight, tid);
+    choose<kRtThreads>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.scored(), s + p.sh.scored() + p.sh.groups, sel, weight, tid);
+    if (warp == 0) { const int n = real_first(p.sh, sel, weight, lane); if (lane == 0) real_s = n; }
+    __syncthreads();
+    const int units = shared + real_s * per;
     if (blockIdx.x == 0 && tid < p.sh.top) {
         p.sel[row * p.sh.top + tid] = sel[tid];
         p.weight[row * p.sh.top + tid] = weight[tid];
@@ -208,9 +249,14 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
     __shared__ float part[kRtWarps];
     __shared__ int sel[kMaxTop];
     __shared__ float weight[kMaxTop];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, top = p.sh.top;
-    if (tid < top) { sel[tid] = p.sel[row * top + tid]; weight[tid] = p.weight[row * top + tid]; }
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, all_top = p.sh.top;
+    if (tid < all_top) { sel[tid] = p.sel[row * all_top + tid]; weight[tid] = p.weight[row * all_top + tid]; }
     __syncthreads();
+    int top = all_top;         // experts with tensors come first
+    float through = 0.f;       // what the others hand through
+    if (p.sh.identity)
+        while (top > 0 && sel[top - 1] >= p.sh.experts) through += weight[--top];
+    const T* input = static_cast<const T*>(p.x) + (size_t)row * p.x_stride;
     const int chunks = p.mid_ld >> 3, routed = chunks * top, all = routed + (p.shared_ld >> 3), half = warp % kDownWarps;
     uint4 v[kDownUnroll];
     auto load = [&](int n, int c0) {
@@ -230,7 +276,7 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
     const float shared_w = p.shared_ld ? shared_weight(p, row) : 0.f;
     for (int i = tid; i < all; i += kRtThreads) {   // eight activations each, times their weight; zeros in the padding
         const int t = min(i / chunks, top), c = 8 * (i - t * chunks), ff = t < top ? p.sh.ff : p.sh.shared_ff;
-        const T* mid = t < top ? static_cast<const T*>(p.mid) + (size_t)(row * top + t) * p.mid_stride : static_cast<const T*>(p.shared_mid) + (size_t)row * p.shared_stride;
+        const T* mid = t < top ? static_cast<const T*>(p.mid) + (size_t)(row * all_top + t) * p.mid_stride : static_cast<const T*>(p.shared_mid) + (size_t)row * p.shared_stride;
         const float w = t < top ? weight[t] : shared_w;
         float f[8];
         rt_get8(mid + c, f);
@@ -258,6 +304,7 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
             float total = 0.f;
 #pragma unroll
             for (int w = 0; w < kDownWarps; ++w) total += part[warp + w];
+            if (p.sh.identity) total = fmaf(through, rt_get(input + n), total);
             p.out[(size_t)row * p.out_stride + n] = total;
         }
         __syncthreads();
@@ -275,12 +322,12 @@ __global__ void __launch_bounds__(kChooseWarps * 32) routed_choose_kernel(const 
     __shared__ float weight[kChooseWarps][kMaxTop];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, row = blockIdx.x * kChooseWarps + warp;
     if (row >= p.m) return;
-    float* s = rt_smem + (size_t)warp * (p.sh.experts + p.sh.groups);
-    choose<32>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.experts, sel[warp], weight[warp], lane);
+    float* s = rt_smem + (size_t)warp * (2 * p.sh.scored() + p.sh.groups);
+    choose<32>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.scored(), s + p.sh.scored() + p.sh.groups, sel[warp], weight[warp], lane);
     for (int t = lane; t < p.sh.top; t += 32) {
         p.sel[row * p.sh.top + t] = sel[warp][t];
         p.weight[row * p.sh.top + t] = weight[warp][t];
-        p.rank[row * p.sh.top + t] = (int)atomicAdd(p.counts + sel[warp][t], 1u);
+        p.rank[row * p.sh.top + t] = sel[warp][t] < p.sh.experts ? (int)atomicAdd(p.counts + sel[warp][t], 1u) : -1;
     }
 }
 
@@ -328,6 +375,7 @@ __global__ void __launch_bounds__(kRtThreads) routed_sort_kernel(const RoutedPar
     }
     const int chunks = p.sorted_stride >> 3, all = p.m * p.sh.top;
     for (int a = blockIdx.x * kRtWarps + warp; a < all; a += gridDim.x * kRtWarps) {
+        if (p.sel[a] >= p.sh.experts) continue;   // hands its input through
         const int at = start[p.sel[a]] + p.rank[a];
         const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.x) + (size_t)(a / p.sh.top) * p.x_stride);
         uint4* dst = reinterpret_cast<uint4*>(p.sorted + (size_t)at * p.sorted_stride);
@@ -347,7 +395,13 @@ __global__ void __launch_bounds__(kRtThreads) routed_sum_kernel(const RoutedPara
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int t = 0; t < p.sh.top; ++t) {
         const float w = p.weight[row * p.sh.top + t];
-        const float4 y = *reinterpret_cast<const float4*>(p.y + (size_t)p.rank[row * p.sh.top + t] * p.y_stride + i);   // (rows are padded to 8)
+        const int at = p.rank[row * p.sh.top + t];
+        float4 y;   // (rows are padded to 8)
+        if (at >= 0) y = *reinterpret_cast<const float4*>(p.y + (size_t)at * p.y_stride + i);
+        else {
+            const uint2 x = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.x) + (size_t)row * p.x_stride + i);
+            y = make_float4(rt_lo(x.x), rt_hi(x.x), rt_lo(x.y), rt_hi(x.y));
+        }
         v.x = fmaf(w, y.x, v.x); v.y = fmaf(w, y.y, v.y); v.z = fmaf(w, y.z, v.z); v.w = fmaf(w, y.w, v.w);
     }
     if (p.shared_y) {
@@ -381,7 +435,7 @@ RoutedScratch layout(const RoutedShape& s, int m, bool f32) {
     return l;
 }
 constexpr size_t kRtMaxSmem = 200 * 1024;
-size_t gate_smem(const RoutedShape& s) { return ((size_t)up8(s.width) + s.experts + s.groups) * 4; }
+size_t gate_smem(const RoutedShape& s) { return ((size_t)up8(s.width) + 2 * s.scored() + s.groups) * 4; }
 size_t down_smem(const RoutedShape& s) { return ((size_t)s.top * up8(s.ff) + up8(s.shared_ff)) * 4; }
 
 template <typename T>
@@ -412,8 +466,8 @@ int routed_init() {
     return SWLM_OK;
 }
 bool routed_supported(const RoutedShape& s) {
-    return s.experts > 0 && s.experts <= kMaxExperts && s.top > 0 && s.top <= kMaxTop && s.groups > 0 && s.experts % s.groups == 0 && s.keep > 0 &&
-           s.keep <= s.groups && s.top <= s.keep * (s.experts / s.groups) && s.width > 0 && s.ff > 0 && s.shared_ff >= 0 && gate_smem(s) <= kRtMaxSmem && down_smem(s) <= kRtMaxSmem;
+    return s.experts > 0 && s.identity >= 0 && s.scored() <= kMaxExperts && s.top > 0 && s.top <= kMaxTop && s.groups > 0 && s.scored() % s.groups == 0 && s.keep > 0 &&
+           s.keep <= s.groups && (!s.identity || s.groups == 1) && s.top <= s.keep * (s.scored() / s.groups) && s.width > 0 && s.ff > 0 && s.shared_ff >= 0 && gate_smem(s) <= kRtMaxSmem && down_smem(s) <= kRtMaxSmem;
 }
 size_t routed_scratch_bytes(const RoutedShape& s, int m, bool f32) { return layout(s, m, f32).total; }
 
@@ -422,6 +476,7 @@ int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches) {
     const RoutedScratch l = layout(a.shape, a.m, a.f32);
     RoutedParams p{};
     p.sh = a.shape; p.scale = a.scale; p.act = a.act; p.m = a.m; p.x = a.x; p.x_stride = a.x_stride; p.z = a.z; p.z_stride = a.z_stride;
+    p.correction = a.correction;
     p.softmax = a.softmax; p.group_best = a.group_best; p.raw_weights = a.raw_weights;
     p.gate = a.gate ? a.gate->data : nullptr; p.up = a.up->data; p.down = a.down->data; p.in_ld = a.up->ld; p.mid_ld = a.down->ld; p.out = a.out; p.out_stride = a.out_stride;
     p.sel = reinterpret_cast<int*>(a.scratch + l.sel); p.weight = reinterpret_cast<float*>(a.scratch + l.weight); p.rank = reinterpret_cast<int*>(a.scratch + l.rank);
@@ -436,7 +491,7 @@ int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches) {
     p.y = reinterpret_cast<float*>(a.scratch + l.y); p.y_stride = up8(a.shape.width);
     p.tiles = reinterpret_cast<int4*>(a.scratch + l.tiles); p.bn = grouped_bn(all, E); p.max_tiles = grouped_max_tiles(all, E);
     if ((a.x_stride & 7) || (reinterpret_cast<uintptr_t>(a.x) & 15)) { set_error("routed feed-forward: rows must be 16-byte aligned"); return SWLM_ERR_INVALID; }
-    cudaError_t e = launch_k(routed_choose_kernel, dim3((a.m + kChooseWarps - 1) / kChooseWarps), dim3(kChooseWarps * 32), (size_t)kChooseWarps * (E + a.shape.groups) * 4, s, p);
+    cudaError_t e = launch_k(routed_choose_kernel, dim3((a.m + kChooseWarps - 1) / kChooseWarps), dim3(kChooseWarps * 32), (size_t)kChooseWarps * (2 * a.shape.scored() + a.shape.groups) * 4, s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed choice launch");
     e = launch_k(routed_sort_kernel, dim3(std::min((all + kRtWarps - 1) / kRtWarps, 4 * 148)), dim3(kRtThreads), 0, s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed sort launch");

@@ -838,6 +838,7 @@ std::vector<Region> state_regions(swlm_state* s) {
         r.push_back({s->delta_state[l], (size_t)d.max_batch * dl.state_elems() * 4});
         r.push_back({s->delta_ring[l], (size_t)d.max_batch * dl.ring_elems() * (s->plan->all_f32() ? 4 : 2)});
     }
+    for (size_t l = 0; l < s->conv_state.size(); ++l) r.push_back({s->conv_state[l], (size_t)d.max_batch * std::max(0, s->plan->convs[l].taps - 1) * d.hidden * 4});
     for (int i = 0; i < SWLM_BUF_COUNT && !s->plan->stream(); ++i) r.push_back({s->buf[i], (size_t)d.max_batch * s->width[i] * 2});
     r.push_back({s->kcache, (size_t)d.kv_layers * s->kv_layer_elems * 2});
     r.push_back({s->vcache, (size_t)d.kv_layers * s->kv_layer_elems * 2});
@@ -1295,6 +1296,7 @@ int swlm_ctx_create(int device_id, int tp_rank, int tp_size, swlm_ctx** out) {
     if (!rc) rc = routed_init();
     if (!rc) rc = grouped_init();
     if (!rc) rc = retention_init();
+    if (!rc) rc = join_init();
     if (rc) { cudaStreamDestroy(ctx->stream); delete ctx; return rc; }
     *out = ctx;
     return SWLM_OK;
@@ -2332,6 +2334,7 @@ static int profiled_launch_kind(int step_kind, int* kind) {
     case SWLM_STEP_ROUTED_MLP: *kind = L_ROUTED; break;
     case SWLM_STEP_GROUPED_ATTN: *kind = L_GROUPED; break;
     case SWLM_STEP_RETENTION: *kind = L_RETENTION; break;
+    case SWLM_STEP_GATED_POSTNORM_ADD: case SWLM_STEP_DEPTH_AVG: case SWLM_STEP_STREAM_CONV: case SWLM_STEP_STREAM_COPY: *kind = L_JOIN; break;
     case SWLM_STEP_RESADD_COPY_RMSNORM: *kind = L_RMSNORM; break;
     default: set_error("profile: step kind %d has no per-kind loop", step_kind); return SWLM_ERR_UNSUPPORTED;
     }

@@ -1,7 +1,7 @@
 // Executor of fp32-stream plans: step list -> launches, the paged pool of latent rows, and one row executor that runs decode
 // steps, prompt chunks and mixed batches alike. A batch is a list of rows, each with its token, sequence and position; the
 // only steps that look beyond their own row are latent and grouped attention, which find the cached rows through the page table,
-// and the gated delta rule and retention, which carry a state per sequence.
+// and the gated delta rule, retention and convolutions over the stream, which carry a state per sequence.
 #include <cmath>
 #include <cstdio>
 #include <cstring>
@@ -130,9 +130,11 @@ bool is_norm(int kind) {
            kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_RMSNORM;
 }
 bool is_postnorm(int kind) { return kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_RMSNORM; }
-bool norm_stores(int kind) { return kind == SWLM_STEP_COPY_RMSNORM || kind == SWLM_STEP_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM; }
-bool reads(const swlm_step& s, int buf) {
-    if (s.in_buf == buf) return true;
+bool norm_stores(const swlm_step& s) { const int kind = s.kind; return (kind == SWLM_STEP_COPY_RMSNORM && s.in_buf != SWLM_BUF_RESIDUAL) || kind == SWLM_STEP_RESADD_COPY_RMSNORM || kind == SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM; }
+bool reads(const Launch& L, int buf) {
+    const swlm_step& s = L.st;
+    if (s.in_buf == buf || L.x2_buf == buf) return true;
+    if (L.kind == L_JOIN) return L.join.in_buf == buf || L.join.gate_buf == buf;
     return s.kind != SWLM_STEP_PRODUCT && !is_norm(s.kind) && (s.in2_buf == buf || s.in3_buf == buf || s.in4_buf == buf);
 }
 bool is_glu(int kind) { return kind == SWLM_STEP_SWIGLU || kind == SWLM_STEP_GEGLU || kind == SWLM_STEP_CLAMPED_GLU; }
@@ -143,9 +145,67 @@ GatedAct glu_of(const swlm_step& s) {
     a.limit = s.limit;
     return a;
 }
-RoutedShape routed_shape(const swlm_step& s) { return RoutedShape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k, s.weight5[0] ? s.k2 : 0}; }
+RoutedShape routed_shape(const swlm_step& s) { return RoutedShape{s.experts, s.top, s.groups, s.groups_keep, s.n, s.k, s.weight5[0] ? s.k2 : 0, s.identity}; }
+bool is_join(const swlm_step& s) {
+    return s.kind == SWLM_STEP_GATED_POSTNORM_ADD || s.kind == SWLM_STEP_DEPTH_AVG || s.kind == SWLM_STEP_STREAM_CONV || s.kind == SWLM_STEP_STREAM_COPY ||
+           (s.kind == SWLM_STEP_EMBED && s.out_buf == SWLM_BUF_RESIDUAL);
+}
 DeltaShape retention_shape(const swlm_step& s) { return DeltaShape{s.heads, s.heads, s.key_dim, s.value_dim, 0}; }
 const char* glu_name(int kind) { return kind == GATED_ACT_GELU_TANH ? "geglu" : kind == GATED_ACT_CLAMPED ? "clamped glu" : "swiglu"; }
+
+// One step over the stream into the parts of a launch; false: it has to be a launch of its own (the parts are in order).
+bool join_takes(const JoinParts& j, const swlm_step& s) {
+    const bool out = j.copy_buf >= 0 || j.conv_buf >= 0;
+    switch (s.kind) {
+    case SWLM_STEP_EMBED: return !j.changes() && !out;
+    case SWLM_STEP_GATED_POSTNORM_ADD: return !j.changes() && !out;
+    case SWLM_STEP_DEPTH_AVG: return !j.table && !j.avg && !out;
+    case SWLM_STEP_STREAM_CONV: return j.conv_buf < 0;
+    default: return j.copy_buf < 0;
+    }
+}
+
+int join_part(swlm_plan* plan, const swlm_step& s, JoinParts* j) {
+    swlm_ctx* ctx = plan->ctx;
+    const swlm_buffers_desc& d = plan->desc;
+    int rc;
+    if (s.n != d.hidden) { set_error("step over the stream: %d entries, the stream has %d", s.n, d.hidden); return SWLM_ERR_INVALID; }
+    switch (s.kind) {
+    case SWLM_STEP_EMBED: {
+        auto it = ctx->dense.find(s.weight);
+        if (it == ctx->dense.end()) { set_error("embedding table '%s' missing", s.weight); return SWLM_ERR_NOT_FOUND; }
+        if (it->second.cols != s.n || it->second.rows != d.vocab) { set_error("embedding '%s': table %lld x %lld for vocabulary %d, width %d", s.weight, (long long)it->second.rows, (long long)it->second.cols, d.vocab, d.hidden); return SWLM_ERR_INVALID; }
+        j->table = &it->second;
+        j->table_scale = s.scale != 0.f ? s.scale : 1.f;
+        if (d.depth_results > 0) j->store = 0;
+        return SWLM_OK;
+    }
+    case SWLM_STEP_GATED_POSTNORM_ADD:
+        if (s.in_buf != SWLM_BUF_HIDDEN || (s.in3_buf != SWLM_BUF_NONE && s.in3_buf != SWLM_BUF_SCRATCH3 && s.in3_buf != SWLM_BUF_SCRATCH4)) { set_error("gated norm '%s': reads hidden, gate in scratch 3 or 4", s.weight); return SWLM_ERR_INVALID; }
+        if ((rc = find_vector(ctx, s.weight, s.n, &j->w))) return rc;
+        j->adds = true; j->in_buf = s.in_buf; j->gate_buf = s.in3_buf; j->eps = s.eps; j->weight_bias = s.weight_bias;
+        return SWLM_OK;
+    case SWLM_STEP_DEPTH_AVG:
+        if (s.k < 1 || s.k > d.depth_results) { set_error("average over %d results, %d are kept", s.k, d.depth_results); return SWLM_ERR_INVALID; }
+        if ((rc = find_vector(ctx, s.weight, s.k, &j->avg_w))) return rc;
+        j->avg = s.k; j->store = s.k - 1;
+        return SWLM_OK;
+    case SWLM_STEP_STREAM_CONV: {
+        if (s.layer < 0 || s.layer >= d.stream_convs) { set_error("convolution over the stream: layer %d has no state", s.layer); return SWLM_ERR_INVALID; }
+        if (!act_buf(plan, s.out_buf) || !join_supported(s.n, s.conv_kernel) || s.conv_kernel < 1) { set_error("convolution over the stream: %d taps, result in scratch 0..2", s.conv_kernel); return SWLM_ERR_UNSUPPORTED; }
+        if ((rc = find_vector(ctx, s.weight, s.n * s.conv_kernel, &j->conv_w))) return rc;
+        StreamConv& c = plan->convs[s.layer];
+        if (c.taps && c.taps != s.conv_kernel) { set_error("convolution state %d is used with %d and %d taps", s.layer, c.taps, s.conv_kernel); return SWLM_ERR_INVALID; }
+        c.taps = s.conv_kernel;
+        j->conv = s.layer; j->conv_buf = s.out_buf;
+        return SWLM_OK;
+    }
+    default:
+        if (!act_buf(plan, s.out_buf)) { set_error("copy of the stream: into scratch 0..2"); return SWLM_ERR_INVALID; }
+        j->copy_buf = s.out_buf;
+        return SWLM_OK;
+    }
+}
 
 }  // namespace
 
@@ -165,6 +225,8 @@ int stream_compile(swlm_plan* plan) {
     plan->latent.assign(std::max(0, d.latent_layers), LatentLayer{});
     plan->grouped.assign(std::max(0, d.grouped_layers), GroupedLayer{});
     plan->delta.assign(std::max(0, d.delta_layers), DeltaLayer{});
+    plan->convs.assign(std::max(0, d.stream_convs), StreamConv{});
+    int unkept = -1;   // convolution whose state does not have its last inputs yet
     widen(SWLM_BUF_HIDDEN, d.hidden);
     widen(SWLM_BUF_RESIDUAL, d.hidden);
     widen(SWLM_BUF_LOGITS, d.vocab);
@@ -172,6 +234,26 @@ int stream_compile(swlm_plan* plan) {
         const swlm_step& s = st[i];
         Launch L;
         L.st = s;
+        if (is_join(s)) {
+            L.kind = L_JOIN;
+            L.label = "stream";
+            L.steps_covered = 0;
+            for (size_t j = i; j < st.size() && is_join(st[j]) && join_takes(L.join, st[j]); ++j) {
+                if ((rc = join_part(plan, st[j], &L.join))) return rc;
+                if (st[j].kind == SWLM_STEP_STREAM_CONV || st[j].kind == SWLM_STEP_STREAM_COPY) widen(st[j].out_buf, st[j].n);
+                if (st[j].in3_buf != SWLM_BUF_NONE) widen(st[j].in3_buf, st[j].n);
+                L.label += std::string(" + ") + (st[j].weight[0] ? st[j].weight : "copy");
+                L.steps_covered += 1;
+            }
+            if (L.join.changes() && unkept >= 0) { L.join.keep = unkept; unkept = -1; }
+            if (L.join.conv >= 0 && plan->convs[L.join.conv].taps > 1) {
+                if (unkept >= 0) { set_error("two convolutions over the stream without a change of it between them"); return SWLM_ERR_UNSUPPORTED; }
+                unkept = L.join.conv;
+            }
+            i += L.steps_covered;
+            plan->launches.push_back(L);
+            continue;
+        }
         switch (s.kind) {
         case SWLM_STEP_EMBED: {
             L.kind = L_EMBED;
@@ -185,7 +267,7 @@ int stream_compile(swlm_plan* plan) {
         case SWLM_STEP_COPY_RMSNORM: case SWLM_STEP_RESADD_COPY_RMSNORM: case SWLM_STEP_RESADD_RMSNORM:
         case SWLM_STEP_POSTNORM_RESADD_COPY_RMSNORM: case SWLM_STEP_POSTNORM_RESADD_RMSNORM:
             L.kind = L_RMSNORM;
-            if (s.in_buf != SWLM_BUF_HIDDEN || !act_buf(plan, s.out_buf) || s.n != d.hidden) { set_error("norm '%s': reads hidden, writes scratch 0..2, width %d", s.weight, d.hidden); return SWLM_ERR_INVALID; }
+            if ((s.in_buf != SWLM_BUF_HIDDEN && (s.in_buf != SWLM_BUF_RESIDUAL || s.kind != SWLM_STEP_COPY_RMSNORM)) || !act_buf(plan, s.out_buf) || s.n != d.hidden) { set_error("norm '%s': reads hidden, writes scratch 0..2, width %d", s.weight, d.hidden); return SWLM_ERR_INVALID; }
             if ((rc = find_vector(ctx, is_postnorm(s.kind) ? s.weight2 : s.weight, s.n, &L.d1))) return rc;
             if (is_postnorm(s.kind) && (rc = find_vector(ctx, s.weight, s.n, &L.norm_post))) return rc;
             if (is_postnorm(s.kind) && s.weight3[0]) {   // an embedding row joins
@@ -201,6 +283,7 @@ int stream_compile(swlm_plan* plan) {
             L.kind = L_PRODUCT;
             if (!act_buf(plan, s.in_buf) || !any_buf(s.out_buf) || s.out_buf == s.in_buf || s.out_buf == SWLM_BUF_RESIDUAL) { set_error("product '%s': bad buffers", s.weight); return SWLM_ERR_INVALID; }
             if ((rc = find_matrix(ctx, s.weight, s.n, s.k, &L.m1))) return rc;
+            if (s.weight3[0] && (rc = find_vector(ctx, s.weight3, s.n, &L.seg_bias[0]))) return rc;
             if (s.weight2[0]) {   // side by side with a second matrix
                 const Matrix* right;
                 if (s.k2 <= 0 || s.in_off < 0 || s.out_off < 0 || (s.in_off & 7)) { set_error("product '%s': bad columns", s.weight); return SWLM_ERR_INVALID; }
@@ -215,7 +298,7 @@ int stream_compile(swlm_plan* plan) {
             widen(s.in_buf, s.in_off + s.k);
             widen(s.out_buf, s.out_off + s.n);
             // gate, up, gated activation -> one launch
-            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && !st[i + 1].weight2[0] && is_glu(st[i + 2].kind) && !s.in_off && !s.out_off && !st[i + 1].in_off && !st[i + 1].out_off &&
+            if (i + 2 < st.size() && st[i + 1].kind == SWLM_STEP_PRODUCT && !st[i + 1].weight2[0] && !s.weight3[0] && !st[i + 1].weight3[0] && is_glu(st[i + 2].kind) && !s.in_off && !s.out_off && !st[i + 1].in_off && !st[i + 1].out_off &&
                 st[i + 1].in_buf == s.in_buf && st[i + 1].k == s.k && st[i + 1].n == s.n && st[i + 2].in_buf == s.out_buf &&
                 st[i + 2].in2_buf == st[i + 1].out_buf && st[i + 2].n == s.n && act_buf(plan, st[i + 2].out_buf) && st[i + 2].out_buf != s.in_buf &&
                 act_buf(plan, s.out_buf) && act_buf(plan, st[i + 1].out_buf)) {
@@ -240,17 +323,25 @@ int stream_compile(swlm_plan* plan) {
                 break;
             }
             size_t j = i + 1;
-            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && !st[j].weight2[0] && st[j].in_buf == s.in_buf && st[j].in_off == s.in_off && st[j].k == s.k &&
+            int rows = s.n;
+            while (j < st.size() && (int)names.size() < kMaxProductSegs && st[j].kind == SWLM_STEP_PRODUCT && !st[j].weight2[0] && st[j].k == s.k &&
                    st[j].out_off >= 0 && st[j].out_buf != s.in_buf && any_buf(st[j].out_buf) && st[j].out_buf != SWLM_BUF_LOGITS && s.out_buf != SWLM_BUF_LOGITS) {
+                // products of one input, and behind them of a second one (no result may go there)
+                const bool same = st[j].in_buf == s.in_buf && st[j].in_off == s.in_off && L.x2_buf < 0;
+                const bool second = act_buf(plan, st[j].in_buf) && st[j].in_buf != s.in_buf && !st[j].in_off && !s.in_off && (L.x2_buf < 0 || L.x2_buf == st[j].in_buf) && st[j].out_buf != st[j].in_buf;
+                if (!same && !second) break;
                 bool clash = false;
                 for (size_t q = i; q < j; ++q)
-                    clash |= (st[q].out_buf == st[j].out_buf && st[q].out_off < st[j].out_off + st[j].n && st[j].out_off < st[q].out_off + st[q].n) || !strcmp(st[q].weight, st[j].weight);
+                    clash |= (!same && st[q].out_buf == st[j].in_buf) || (st[q].out_buf == st[j].out_buf && st[q].out_off < st[j].out_off + st[j].n && st[j].out_off < st[q].out_off + st[q].n) || !strcmp(st[q].weight, st[j].weight);
                 // a gate / up pair that starts here keeps its own launch
                 if (clash || (j + 2 < st.size() && is_glu(st[j + 2].kind) && st[j + 2].in_buf == st[j].out_buf)) break;
                 const Matrix* m;
                 if ((rc = find_matrix(ctx, st[j].weight, st[j].n, st[j].k, &m))) return rc;
                 widen(st[j].out_buf, st[j].out_off + st[j].n);
                 const int q = (int)names.size();
+                if (st[j].weight3[0] && (rc = find_vector(ctx, st[j].weight3, st[j].n, &L.seg_bias[q]))) return rc;
+                if (!same && L.x2_buf < 0) { L.x2_buf = st[j].in_buf; L.first_segs = q; widen(st[j].in_buf, st[j].k); L.part[0].n = rows; }
+                rows += st[j].n;
                 L.seg_buf[q] = st[j].out_buf; L.seg_off[q] = st[j].out_off; L.seg_end[q] = L.seg_end[q - 1] + st[j].n;
                 names.push_back(st[j].weight);
                 L.label += std::string(" ") + st[j].weight;
@@ -259,6 +350,13 @@ int stream_compile(swlm_plan* plan) {
             L.n_seg = (int)names.size();
             L.steps_covered = L.n_seg;
             if (L.n_seg > 1 && (rc = concat_matrices(ctx, names, &L.m1))) return rc;
+            if (L.x2_buf >= 0) {
+                const int split = L.part[0].n;
+                L.part[0] = L.part[1] = *L.m1;
+                L.part[0].n = split;
+                L.part[1].n = rows - split;
+                L.part[1].data = L.m1->data + (size_t)split * L.m1->ld;
+            }
             break;
         }
         case SWLM_STEP_SWIGLU: case SWLM_STEP_GEGLU: case SWLM_STEP_CLAMPED_GLU:
@@ -305,8 +403,10 @@ int stream_compile(swlm_plan* plan) {
             DeltaShape shape;
             shape.heads = s.heads; shape.groups = s.groups; shape.dim = s.key_dim; shape.vdim = s.value_dim; shape.taps = s.conv_kernel;
             if (!delta_supported(shape) || (s.k != 1 && s.k != s.key_dim) || (s.gate_act != SWLM_GATE_SILU && s.gate_act != SWLM_GATE_SIGMOID)) { set_error("gated delta rule: %d heads over %d groups, %d x %d, %d taps, %d decays per head", s.heads, s.groups, s.key_dim, s.value_dim, s.conv_kernel, s.k); return SWLM_ERR_UNSUPPORTED; }
-            if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || !any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf) || s.in2_buf == s.in3_buf ||
-                !act_buf(plan, s.in4_buf) || !act_buf(plan, s.out_buf) || s.in4_buf == s.in_buf || s.out_buf == s.in_buf) { set_error("gated delta rule: q | k | v, gate and result in scratch 0..2, step sizes and decays in scratch 3 and 4"); return SWLM_ERR_INVALID; }
+            const bool same_scalars = s.in2_buf == s.in3_buf && s.in2_off < s.in3_off + s.heads * s.k && s.in3_off < s.in2_off + s.heads;
+            const bool same_rows = s.in4_buf == s.in_buf && s.in4_off < shape.channels();
+            if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || !any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf) || same_scalars || same_rows ||
+                s.in2_off < 0 || s.in3_off < 0 || s.in4_off < 0 || !act_buf(plan, s.in4_buf) || !act_buf(plan, s.out_buf) || s.out_buf == s.in_buf || (s.out_buf == s.in4_buf && s.in4_off)) { set_error("gated delta rule: q | k | v, gate and result in scratch 0..2, step sizes and decays in scratch 3 and 4"); return SWLM_ERR_INVALID; }
             const char* names[6] = {s.weight, s.weight2, s.weight3, s.weight4, s.weight5, s.weight6};
             const int counts[6] = {s.groups * s.key_dim * s.conv_kernel, s.groups * s.key_dim * s.conv_kernel, s.heads * s.value_dim * s.conv_kernel, s.value_dim, s.heads, s.heads * s.k};
             for (int q = 0; q < 6; ++q) if ((rc = find_vector(ctx, names[q], counts[q], &L.dv[q]))) return rc;
@@ -314,9 +414,9 @@ int stream_compile(swlm_plan* plan) {
             if (dl.shape.heads && memcmp(&dl.shape, &shape, sizeof(shape))) { set_error("gated-delta layer %d is used with two shapes", s.layer); return SWLM_ERR_INVALID; }
             dl.shape = shape;
             widen(s.in_buf, shape.channels());
-            widen(s.in2_buf, s.heads);
-            widen(s.in3_buf, s.heads * s.k);
-            widen(s.in4_buf, s.heads * s.value_dim);
+            widen(s.in2_buf, s.in2_off + s.heads);
+            widen(s.in3_buf, s.in3_off + s.heads * s.k);
+            widen(s.in4_buf, s.in4_off + s.heads * s.value_dim);
             widen(s.out_buf, s.heads * s.value_dim);
             L.label = std::string("gated_delta ") + s.weight4;
             break;
@@ -325,7 +425,7 @@ int stream_compile(swlm_plan* plan) {
             L.kind = L_ROUTED;
             const bool gated = s.weight2[0], shared = s.weight5[0];
             const RoutedShape shape = routed_shape(s);
-            if (!routed_supported(shape) || (shared && (s.k2 <= 0 || gated))) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d, shared %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k, s.k2); return SWLM_ERR_UNSUPPORTED; }
+            if (!routed_supported(shape) || (shared && (s.k2 <= 0 || gated || s.identity)) || s.expert_act < 0 || s.expert_act > SWLM_EXPERT_SILU) { set_error("routed feed-forward: %d of %d experts, %d of %d groups, %d x %d, shared %d", s.top, s.experts, s.groups_keep, s.groups, s.n, s.k, s.k2); return SWLM_ERR_UNSUPPORTED; }
             if (s.score_act < 0 || s.score_act > SWLM_SCORE_SOFTMAX || s.group_best < 0 || s.group_best > 2) { set_error("routed feed-forward: scores %d, group %d", s.score_act, s.group_best); return SWLM_ERR_UNSUPPORTED; }
             if (!act_buf(plan, s.in_buf) || !any_buf(s.in2_buf) || !stored_f32(plan, s.in2_buf) || s.out_buf != SWLM_BUF_HIDDEN || s.n != d.hidden) { set_error("routed feed-forward: input in scratch 0..2, logits in scratch 3 or 4, result in hidden"); return SWLM_ERR_INVALID; }
             const char* suffix[3] = {s.weight2, s.weight3, s.weight4};
@@ -340,9 +440,11 @@ int stream_compile(swlm_plan* plan) {
                 if ((rc = concat_matrices(ctx, names, into[q]))) return rc;
             }
             if (shared && ((rc = find_matrix(ctx, s.weight5, s.k2, s.n, &L.m4)) || (rc = find_matrix(ctx, s.weight6, s.n, s.k2, &L.m5)))) return rc;
-            L.act.kind = GATED_ACT_CLAMPED; L.act.alpha = s.glu_alpha; L.act.limit = s.limit;
+            if (s.weight7[0] && (rc = find_vector(ctx, s.weight7, shape.scored(), &L.dv[0]))) return rc;
+            if (L.dv[0] && s.groups != 1) { set_error("routed feed-forward: a correction goes with one group"); return SWLM_ERR_UNSUPPORTED; }
+            L.act.kind = s.expert_act == SWLM_EXPERT_SILU ? GATED_ACT_SILU : GATED_ACT_CLAMPED; L.act.alpha = s.glu_alpha; L.act.limit = s.limit;
             widen(s.in_buf, s.n);
-            widen(s.in2_buf, s.experts + (shared ? 1 : 0));
+            widen(s.in2_buf, shape.scored() + (shared ? 1 : 0));
             widen(s.out_buf, s.n);
             L.label = std::string("routed_mlp ") + s.weight;
             break;
@@ -356,14 +458,19 @@ int stream_compile(swlm_plan* plan) {
                 (s.in3_buf != SWLM_BUF_NONE && (!any_buf(s.in3_buf) || !stored_f32(plan, s.in3_buf)))) { set_error("grouped attention: q | k | v and the result in scratch 0..2 from columns that are multiples of 8, gate in scratch 3 or 4"); return SWLM_ERR_INVALID; }
             if (s.weight[0] && (rc = find_vector(ctx, s.weight, s.head_dim, &L.dv[0]))) return rc;
             if (s.weight2[0] && (rc = find_vector(ctx, s.weight2, s.head_dim, &L.dv[1]))) return rc;
-            const GroupedRow row = grouped_row(s.kv_heads, s.head_dim, s.value_dim, plan->all_f32());
+            if ((s.value_is_key && (s.value_dim != s.head_dim || s.rope_dim || s.weight[0] || s.weight2[0])) || (s.head_norm && (s.weight[0] || s.weight2[0])) || s.temp_every < 0) { set_error("grouped attention: values that are keys go without rotation and norm weights"); return SWLM_ERR_UNSUPPORTED; }
+            const bool entry_gate = s.in4_buf != SWLM_BUF_NONE;
+            const int kv_entries = s.kv_heads * (s.head_dim + (s.value_is_key ? 0 : s.value_dim));
+            if (entry_gate && (!act_buf(plan, s.in4_buf) || s.in4_buf == s.out_buf || s.in4_off < 0 || (s.in4_buf == s.in_buf && s.in4_off < s.in_off + s.heads * s.head_dim + kv_entries))) { set_error("grouped attention: gates of the entries in scratch 0..2, behind q | k | v"); return SWLM_ERR_INVALID; }
+            const GroupedRow row = grouped_row(s.kv_heads, s.head_dim, s.value_dim, plan->all_f32(), s.value_is_key);
             if (!grouped_supported(row)) { set_error("grouped attention: heads of %d and %d", s.head_dim, s.value_dim); return SWLM_ERR_UNSUPPORTED; }
             if ((rc = stream_rope_table(plan, s, &L.rope_table))) return rc;
             L.window_set = window_set(s.window_left);
             GroupedLayer& gl = plan->grouped[s.layer];
             if (gl.row.groups && memcmp(&gl.row, &row, sizeof(row))) { set_error("grouped layer %d is used with two row sizes", s.layer); return SWLM_ERR_INVALID; }
             gl.row = row;
-            widen(s.in_buf, s.in_off + (s.heads + s.kv_heads) * s.head_dim + s.kv_heads * s.value_dim);
+            widen(s.in_buf, s.in_off + s.heads * s.head_dim + kv_entries);
+            if (entry_gate) widen(s.in4_buf, s.in4_off + s.heads * s.value_dim);
             if (s.in3_buf != SWLM_BUF_NONE) widen(s.in3_buf, s.heads);
             widen(s.out_buf, s.out_off + s.heads * s.value_dim);
             L.label = std::string("grouped_attention ") + s.weight;
@@ -388,6 +495,16 @@ int stream_compile(swlm_plan* plan) {
             L.label = std::string("retention ") + s.weight;
             break;
         }
+        case SWLM_STEP_TOKEN_GATE: {
+            L.kind = L_TOKEN_GATE;
+            auto it = ctx->dense.find(s.weight);
+            if (it == ctx->dense.end()) { set_error("table '%s' missing", s.weight); return SWLM_ERR_NOT_FOUND; }
+            L.d1 = &it->second;
+            if (s.n <= 0 || !act_buf(plan, s.in_buf) || !act_buf(plan, s.out_buf) || s.in2_off < 0 || L.d1->rows != d.vocab || L.d1->cols < s.in2_off + s.n) { set_error("token gate '%s': columns %d .. %d of a table %lld x %lld", s.weight, s.in2_off, s.in2_off + s.n, (long long)L.d1->rows, (long long)L.d1->cols); return SWLM_ERR_INVALID; }
+            widen(s.in_buf, s.n); widen(s.out_buf, s.n);
+            L.label = std::string("token gate ") + s.weight;
+            break;
+        }
         case SWLM_STEP_SOFTCAP:
             L.kind = L_SOFTCAP;
             if (s.in_buf != SWLM_BUF_LOGITS || s.n != d.vocab || !(s.scale > 0.f)) { set_error("soft cap: of the logits, by a positive number"); return SWLM_ERR_INVALID; }
@@ -405,6 +522,17 @@ int stream_compile(swlm_plan* plan) {
         i += L.steps_covered;
         plan->launches.push_back(L);
     }
+    if (unkept >= 0) {   // nothing changes the stream any more: a launch that only keeps its rows
+        Launch L;
+        L.kind = L_JOIN;
+        L.join.keep = unkept;
+        L.st.in_buf = L.st.in2_buf = L.st.in3_buf = L.st.in4_buf = L.st.out_buf = SWLM_BUF_NONE;
+        L.label = "stream rows to their state";
+        L.steps_covered = 0;
+        plan->launches.push_back(L);
+    }
+    for (int l = 0; l < d.stream_convs; ++l)
+        if (!plan->convs[l].taps && st.size() > 1) { set_error("convolution %d has no step", l); return SWLM_ERR_INVALID; }
     for (int l = 0; l < d.latent_layers; ++l)
         if (!plan->latent[l].rank && st.size() > 1) { set_error("latent layer %d has no step", l); return SWLM_ERR_INVALID; }
     for (int l = 0; l < d.grouped_layers; ++l)
@@ -417,12 +545,12 @@ int stream_compile(swlm_plan* plan) {
     for (size_t i = 0; i + 1 < plan->launches.size(); ++i) {
         const Launch A = plan->launches[i];
         Launch& B = plan->launches[i + 1];
-        if (A.kind != L_RMSNORM || B.kind != L_PRODUCT || B.st.in_buf != A.st.out_buf || B.st.in_off) continue;
+        if (A.kind != L_RMSNORM || B.kind != L_PRODUCT || B.st.in_buf != A.st.out_buf || B.st.in_off || B.x2_buf >= 0) continue;
         bool ok = true;
         for (size_t j = i + 2; j < plan->launches.size(); ++j) {
             const Launch& C = plan->launches[j];
-            if (reads(C.st, A.st.out_buf)) { ok = false; break; }
-            bool writes = C.st.out_buf == A.st.out_buf;
+            if (reads(C, A.st.out_buf)) { ok = false; break; }
+            bool writes = C.kind == L_JOIN ? C.join.conv_buf == A.st.out_buf || C.join.copy_buf == A.st.out_buf : C.st.out_buf == A.st.out_buf;
             for (int q = 0; q < C.n_seg; ++q) writes |= C.seg_buf[q] == A.st.out_buf;
             if (writes) break;
         }
@@ -435,9 +563,9 @@ int stream_compile(swlm_plan* plan) {
     // the residual stream alternates between two buffers, so that a norm computed by every CTA of a product can be stored by one
     int cur = 0;
     for (Launch& L : plan->launches) {
-        const int kind = L.kind == L_RMSNORM ? L.st.kind : L.kind == L_PRODUCT ? L.norm.kind : 0;
+        const swlm_step* norm = L.kind == L_RMSNORM ? &L.st : L.kind == L_PRODUCT && L.norm.kind ? &L.norm : nullptr;
         L.res_in = L.res_out = cur;
-        if (is_norm(kind) && norm_stores(kind)) { L.res_out = 1 - cur; cur = 1 - cur; }
+        if ((norm && norm_stores(*norm)) || (L.kind == L_JOIN && L.join.changes())) { L.res_out = 1 - cur; cur = 1 - cur; }
     }
     plan->final_res = cur;
     return SWLM_OK;
@@ -509,6 +637,10 @@ int bufs_rows(swlm_state* s, StreamBufs* b, int rows, int wants) {
         cudaFree(b->res2);
         if ((rc = dev_alloc(&b->res2, (size_t)rows * s->width[SWLM_BUF_RESIDUAL]))) return rc;
         SWLM_CUDA(cudaMemsetAsync(b->res2, 0, (size_t)rows * s->width[SWLM_BUF_RESIDUAL] * 4, s->stream));
+        cudaFree(b->results);
+        const size_t results = (size_t)std::max(0, plan->desc.depth_results) * rows * s->width[SWLM_BUF_RESIDUAL];
+        if ((rc = dev_alloc(&b->results, results))) return rc;
+        if (results) SWLM_CUDA(cudaMemsetAsync(b->results, 0, results * 4, s->stream));
         b->rows = rows;
     }
     if (wants > b->wants) {
@@ -533,7 +665,8 @@ size_t part_need(const swlm_plan* plan, int rows, int wants) {
     size_t need = 0;
     if (plan->all_f32()) return 0;
     for (const Launch& L : plan->launches)
-        if (L.kind == L_PRODUCT) need = std::max(need, product_part_floats(L.m1->n, L.m1->k, L.seg_buf[0] == SWLM_BUF_LOGITS ? wants : rows, L.m2 != nullptr));
+        if (L.kind == L_PRODUCT && L.x2_buf >= 0) for (const Matrix& m : L.part) need = std::max(need, product_part_floats(m.n, m.k, rows, false));
+        else if (L.kind == L_PRODUCT) need = std::max(need, product_part_floats(L.m1->n, L.m1->k, L.seg_buf[0] == SWLM_BUF_LOGITS ? wants : rows, L.m2 != nullptr));
         else if (L.kind == L_ROUTED && L.m4) need = std::max(need, std::max(product_part_floats(L.m4->n, L.m4->k, rows, false), product_part_floats(L.m5->n, L.m5->k, rows, false)));
     return need;
 }
@@ -573,7 +706,7 @@ int bufs_scratch(swlm_state* s, StreamBufs* b, const RowBatch& r) {
 
 void bufs_free(StreamBufs* b) {
     for (void* p : b->buf) cudaFree(p);
-    cudaFree(b->res2); cudaFree(b->meta); cudaFree(b->argmax_out); cudaFree(b->qcat); cudaFree(b->partial); cudaFree(b->part);
+    cudaFree(b->res2); cudaFree(b->results); cudaFree(b->meta); cudaFree(b->argmax_out); cudaFree(b->qcat); cudaFree(b->partial); cudaFree(b->part);
     cudaFree(b->expand); cudaFree(b->delta); cudaFree(b->routed); cudaFree(b->argmax_val); cudaFree(b->argmax_idx);
     *b = StreamBufs{};
 }
@@ -584,13 +717,13 @@ StreamNorm norm_of(swlm_state* s, StreamBufs* b, const RowBatch& r, const Launch
     const DenseTensor* post = L.norm_post;
     StreamNorm n;
     n.mode = st.kind;
-    n.in = static_cast<const float*>(b->buf[st.in_buf]); n.in_stride = s->width[st.in_buf];
+    n.in = st.in_buf == SWLM_BUF_RESIDUAL ? residual(b, res_in) : static_cast<const float*>(b->buf[st.in_buf]); n.in_stride = s->width[st.in_buf];
     n.res_stride = s->width[SWLM_BUF_RESIDUAL];
     if (st.kind != SWLM_STEP_COPY_RMSNORM) n.res_in = residual(b, res_in);
-    if (norm_stores(st.kind)) n.res_out = residual(b, res_out);
+    if (norm_stores(st)) n.res_out = residual(b, res_out);
     n.w = w->data; n.w_post = post ? post->data : nullptr;
     n.eps = st.eps; n.weight_bias = st.weight_bias;
-    if (L.dv[0]) { n.table = L.dv[0]->data; n.tokens = r.tok; n.vocab = s->plan->desc.vocab; n.table_scale = st.scale; }
+    if (is_postnorm(st.kind) && L.dv[0]) { n.table = L.dv[0]->data; n.tokens = r.tok; n.vocab = s->plan->desc.vocab; n.table_scale = st.scale; }
     return n;
 }
 
@@ -640,6 +773,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             }
             a.out.softcap = L.softcap;
             auto segment = [&](int q, int buf, int off, int end) {
+                a.out.bias[q] = L.seg_bias[q] ? L.seg_bias[q]->data : nullptr;
                 a.out.y[q] = static_cast<unsigned char*>(b->buf[buf]) + (size_t)off * stored_bytes(plan, buf); a.out.stride[q] = s->width[buf]; a.out.f32[q] = stored_f32(plan, buf) ? 1 : 0; a.out.end[q] = end;
             };
             if (L.m2 && !product_takes_gate(m, L.m1->k, f32)) {
@@ -661,6 +795,26 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.out.count = L.n_seg;
             for (int q = 0; q < L.n_seg; ++q) segment(q, L.seg_buf[q], L.seg_off[q], L.seg_end[q]);
             for (int q = L.n_seg; q < kMaxProductSegs; ++q) a.out.end[q] = L.seg_end[L.n_seg - 1];
+            if (L.x2_buf >= 0) {
+                a.x2 = b->buf[L.x2_buf]; a.x2_stride = s->width[L.x2_buf]; a.split = L.part[0].n;
+                if (!product_takes_two(m, L.m1->k, a.split, f32)) {   // one input after the other
+                    for (int h = 0; h < 2 && !rc; ++h) {
+                        ProductLaunch c = a;
+                        c.w = &L.part[h]; c.x2 = nullptr;
+                        if (h) { c.x = a.x2; c.x_stride = a.x2_stride; }
+                        const int q0 = h ? L.first_segs : 0, q1 = h ? L.n_seg : L.first_segs;
+                        c.out.count = q1 - q0;
+                        for (int q = 0; q < kMaxProductSegs; ++q) {
+                            const int from = std::min(q0 + q, q1 - 1);
+                            c.out.y[q] = a.out.y[from]; c.out.stride[q] = a.out.stride[from]; c.out.f32[q] = a.out.f32[from]; c.out.bias[q] = a.out.bias[from];
+                            c.out.end[q] = a.out.end[from] - (h ? a.split : 0);
+                        }
+                        rc = launch_product(c, stream);
+                        s->launches += product_launch_count(c);
+                    }
+                    break;
+                }
+            }
             rc = launch_product(a, stream);
             s->launches += product_launch_count(a);
             break;
@@ -679,9 +833,9 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.shape = plan->delta[st.layer].shape;
             a.decay_dim = st.k; a.gate_act = st.gate_act; a.eps = st.eps; a.unit_eps = st.eps2; a.q_scale = st.scale; a.f32 = f32;
             a.qkv = b->buf[st.in_buf]; a.qkv_stride = s->width[st.in_buf];
-            a.beta = static_cast<const float*>(b->buf[st.in2_buf]); a.beta_stride = s->width[st.in2_buf];
-            a.decay = static_cast<const float*>(b->buf[st.in3_buf]); a.decay_stride = s->width[st.in3_buf];
-            a.gate = b->buf[st.in4_buf]; a.gate_stride = s->width[st.in4_buf];
+            a.beta = static_cast<const float*>(column(b, st.in2_buf, st.in2_off)); a.beta_stride = s->width[st.in2_buf];
+            a.decay = static_cast<const float*>(column(b, st.in3_buf, st.in3_off)); a.decay_stride = s->width[st.in3_buf];
+            a.gate = column(b, st.in4_buf, st.in4_off); a.gate_stride = s->width[st.in4_buf];
             a.conv_q = L.dv[0]->data; a.conv_k = L.dv[1]->data; a.conv_v = L.dv[2]->data; a.norm_w = L.dv[3]->data; a.a_log = L.dv[4]->data; a.dt_bias = L.dv[5]->data;
             a.ring = s->delta_ring[st.layer]; a.state = s->delta_state[st.layer];
             a.row_seq = r.seq; a.row_pos = r.pos;
@@ -700,7 +854,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.z = static_cast<const float*>(b->buf[st.in2_buf]); a.z_stride = s->width[st.in2_buf];
             a.gate = L.m1; a.up = L.m2; a.down = L.m3; a.shared_up = L.m4; a.shared_down = L.m5;
             a.softmax = st.score_act == SWLM_SCORE_SOFTMAX; a.group_best = st.group_best == 1 ? 1 : 2; a.raw_weights = st.raw_weights;
-            a.part = b->part; a.part_floats = b->part_cap;
+            a.part = b->part; a.part_floats = b->part_cap; a.correction = L.dv[0] ? L.dv[0]->data : nullptr;
             a.out = static_cast<float*>(b->buf[st.out_buf]); a.out_stride = s->width[st.out_buf];
             a.scratch = b->routed; a.counts = s->routed_counts; a.status = s->pf_status;
             int n = 0;
@@ -714,6 +868,8 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.row = plan->grouped[st.layer].row;
             a.heads = st.heads; a.rot_dims = st.rope_dim; a.rot_neighbours = st.rope_pairs == SWLM_ROPE_NEIGHBOURS; a.window = st.window_left; a.chunk = st.chunk; a.sink_one = st.sink_one;
             a.scale = st.scale; a.eps = st.eps; a.weight_bias = st.weight_bias; a.magnitude = rope.magnitude; a.inv_freq = rope.inv_freq; a.out_scale = st.out_scale; a.f32 = f32;
+            a.head_norm = st.head_norm; a.temp_every = st.temp_every; a.temp_coef = st.temp_coef;
+            if (st.in4_buf != SWLM_BUF_NONE) { a.entry_gate = column(b, st.in4_buf, st.in4_off); a.entry_gate_stride = s->width[st.in4_buf]; }
             a.q_norm = L.dv[0] ? L.dv[0]->data : nullptr; a.k_norm = L.dv[1] ? L.dv[1]->data : nullptr;
             a.qkv = column(b, st.in_buf, st.in_off); a.qkv_stride = s->width[st.in_buf];
             if (st.in3_buf != SWLM_BUF_NONE) { a.gate = static_cast<const float*>(b->buf[st.in3_buf]); a.gate_stride = s->width[st.in3_buf]; }
@@ -769,6 +925,30 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             s->launches += n;
             break;
         }
+        case L_JOIN: {
+            const JoinParts& j = L.join;
+            JoinLaunch a;
+            a.rows = r.rows; a.width = d.hidden; a.f32 = f32; a.singles = r.n_runs == 0;
+            a.row_seq = r.seq; a.row_pos = r.pos; a.tokens = r.tok;
+            a.res_stride = s->width[SWLM_BUF_RESIDUAL];
+            if (j.table) { a.table = j.table->data; a.vocab = d.vocab; a.table_scale = j.table_scale; }
+            else a.res_in = residual(b, L.res_in);
+            if (j.changes()) a.res_out = residual(b, L.res_out);
+            if (j.keep >= 0) { a.keep_ring = s->conv_state[j.keep]; a.keep_taps = plan->convs[j.keep].taps; }
+            if (j.adds) { a.in = static_cast<const float*>(b->buf[j.in_buf]); a.in_stride = s->width[j.in_buf]; a.w = j.w->data; a.eps = j.eps; a.weight_bias = j.weight_bias; }
+            if (j.adds && j.gate_buf >= 0) { a.gate = static_cast<const float*>(b->buf[j.gate_buf]); a.gate_stride = s->width[j.gate_buf]; }
+            a.results = b->results; a.result_step = (size_t)b->rows * a.res_stride; a.store = j.store;
+            if (j.avg) { a.avg_w = j.avg_w->data; a.avg = j.avg; }
+            if (j.conv >= 0) { a.conv_w = j.conv_w->data; a.conv_ring = s->conv_state[j.conv]; a.taps = plan->convs[j.conv].taps; a.conv_out = b->buf[j.conv_buf]; a.conv_stride = s->width[j.conv_buf]; }
+            if (j.copy_buf >= 0) { a.copy_out = b->buf[j.copy_buf]; a.copy_stride = s->width[j.copy_buf]; }
+            rc = launch_join(a, stream);
+            s->launches += 1;
+            break;
+        }
+        case L_TOKEN_GATE:
+            rc = launch_token_gate(r.rows, st.n, b->buf[st.in_buf], s->width[st.in_buf], r.tok, d.vocab, L.d1->data, (int)L.d1->cols, st.in2_off, b->buf[st.out_buf], s->width[st.out_buf], f32, stream);
+            s->launches += 1;
+            break;
         case L_ARGMAX:
             if (wants == 0) break;
             if (r.advance) {
@@ -852,6 +1032,13 @@ int stream_state_create(swlm_state* s) {
         if (bytes) SWLM_CUDA(cudaMemset(ring, 0, bytes));
         if (st) SWLM_CUDA(cudaMemset(st, 0, (size_t)d.max_batch * l.state_elems() * 4));
     }
+    for (const StreamConv& c : plan->convs) {   // (as above: a sequence at position 0 starts from zeros)
+        const size_t count = (size_t)d.max_batch * std::max(0, c.taps - 1) * d.hidden;
+        float* p = nullptr;
+        if ((rc = dev_alloc(&p, count))) return rc;
+        s->conv_state.push_back(p);
+        if (count) SWLM_CUDA(cudaMemset(p, 0, count * 4));
+    }
     if ((rc = dev_alloc(&s->routed_counts, kMaxExperts))) return rc;
     SWLM_CUDA(cudaMemset(s->routed_counts, 0, kMaxExperts * 4));
     s->seq_pages.assign(d.max_batch, {});
@@ -884,6 +1071,7 @@ void stream_state_free(swlm_state* s) {
     for (void* p : s->pool) cudaFree(p);
     for (float* p : s->delta_state) cudaFree(p);
     for (void* p : s->delta_ring) cudaFree(p);
+    for (float* p : s->conv_state) cudaFree(p);
     cudaFree(s->routed_counts);
     cudaFree(s->page_table);
     cudaFree(s->seq_identity);
@@ -907,6 +1095,8 @@ int stream_launches_per_step(const swlm_plan* plan) {
             if (fused) a.norm.mode = L.norm.kind;
             else if (L.norm.kind) n += 1;
             if (L.m2 && !product_takes_gate(m, L.m1->k, a.x_f32)) { a.w2 = nullptr; n += 2 * product_launch_count(a) + 1; }
+            else if (L.x2_buf >= 0 && !product_takes_two(m, L.m1->k, L.part[0].n, plan->all_f32()))
+                for (const Matrix& part : L.part) { a.w = &part; n += product_launch_count(a); }
             else n += product_launch_count(a);
         } else if (L.kind == L_DELTA) n += delta_step_fits(plan->delta[L.st.layer].shape) ? 1 : 3;
         else if (L.kind == L_RETENTION) n += retention_step_fits(L.st.key_dim, L.st.value_dim) ? 1 : 2;
@@ -1178,6 +1368,8 @@ int stream_run_step(swlm_state* s, const swlm_step* step, const int32_t* token_i
         if (tmp.latent[l].rank && tmp.latent[l].row.pitch != s->plan->latent[l].row.pitch) { set_error("step: latent layer %zu has other rows", l); return done(SWLM_ERR_INVALID); }
     for (size_t l = 0; l < tmp.grouped.size(); ++l)
         if (tmp.grouped[l].row.groups && memcmp(&tmp.grouped[l].row, &s->plan->grouped[l].row, sizeof(GroupedRow))) { set_error("step: grouped layer %zu has other rows", l); return done(SWLM_ERR_INVALID); }
+    for (size_t l = 0; l < tmp.convs.size(); ++l)
+        if (tmp.convs[l].taps && tmp.convs[l].taps != s->plan->convs[l].taps) { set_error("step: convolution %zu has other taps", l); return done(SWLM_ERR_INVALID); }
     for (size_t l = 0; l < tmp.delta.size(); ++l)
         if (tmp.delta[l].shape.heads && memcmp(&tmp.delta[l].shape, &s->plan->delta[l].shape, sizeof(DeltaShape))) { set_error("step: gated-delta layer %zu has another shape", l); return done(SWLM_ERR_INVALID); }
     for (int b = 0; b < m; ++b)

@@ -355,6 +355,7 @@ struct ProductOut {
     void* y[kMaxProductSegs] = {};
     int stride[kMaxProductSegs] = {};
     int f32[kMaxProductSegs] = {};
+    const __nv_bfloat16* bias[kMaxProductSegs] = {};   // added to the rows of a segment; null: none
     float softcap = 0.f;   // > 0: every value v becomes softcap * tanh(v / softcap)
     int gelu = 0;          // every value v becomes v * (1 + erf(v / sqrt(2))) / 2
 };
@@ -392,6 +393,7 @@ struct ProductLaunch {
     GatedAct act;
     int m = 0;
     const void* x = nullptr; int x_stride = 0; bool x_f32 = false;   // x_f32: activations fp32, true fp32 products
+    const void* x2 = nullptr; int x2_stride = 0, split = 0;   // weight rows from `split` on meet these activations (only when product_takes_two)
     StreamNorm norm;                // x = this norm's result (only when product_takes_norm)
     ProductOut out;
     float* part = nullptr; size_t part_floats = 0;   // split-K sums
@@ -408,6 +410,7 @@ int grouped_bn(int rows, int experts);
 int grouped_max_tiles(int rows, int experts);
 bool product_takes_norm(int m, int k);
 bool product_takes_gate(int m, int k, bool x_f32);
+bool product_takes_two(int m, int k, int split, bool x_f32);
 int product_launch_count(const ProductLaunch& a);
 size_t product_part_floats(int n, int k, int m, bool gated);
 
@@ -460,6 +463,35 @@ bool latent_expands(const LatentRow& r, int dim, int vdim, bool f32);
 constexpr int kLatentQueryTile = 128;
 // launches (for the counters): short part 3, span part 4 or 5
 int launch_latent(const LatentLaunch& a, cudaStream_t s, int* launches);
+
+// ---- the residual stream between sublayers (stream_join.cu) ------------------------------------------------------------
+// One launch over the rows of a batch; parts that are not set are left out:
+//   x = table[token] * table_scale, or res_in
+//   keep_ring: x of a portion's last rows goes to the state of the convolution that read it
+//   x += norm(in * sigmoid(gate); w)
+//   results[store] = x;  x = sum over j < avg of avg_w[j] * results[j] (x itself is the last of them)
+//   res_out = x, copy_out = x, conv_out = x + conv(x)
+struct JoinLaunch {
+    int rows = 0, width = 0; bool f32 = false;             // f32: copy_out and conv_out are fp32
+    bool singles = false;                                  // every row is the only one of its sequence
+    const int32_t *row_seq = nullptr, *row_pos = nullptr, *tokens = nullptr;
+    const __nv_bfloat16* table = nullptr; int vocab = 0; float table_scale = 1.f;
+    const float* res_in = nullptr; float* res_out = nullptr; int res_stride = 0;
+    const float* in = nullptr; int in_stride = 0;
+    const float* gate = nullptr; int gate_stride = 0;
+    const __nv_bfloat16* w = nullptr; float eps = 0.f, weight_bias = 0.f;
+    float* keep_ring = nullptr; int keep_taps = 0;         // [sequence][taps - 1][width], slot = position % (taps - 1)
+    float* results = nullptr; size_t result_step = 0; int store = -1;   // [result][row][res_stride]
+    const __nv_bfloat16* avg_w = nullptr; int avg = 0;
+    const __nv_bfloat16* conv_w = nullptr; const float* conv_ring = nullptr; int taps = 0; void* conv_out = nullptr; int conv_stride = 0;   // conv_w [width][taps]
+    void* copy_out = nullptr; int copy_stride = 0;
+};
+int join_init();
+bool join_supported(int width, int taps);
+int launch_join(const JoinLaunch& a, cudaStream_t s);
+// out = gelu_tanh(in) * table[token][col ..]
+int launch_token_gate(int m, int n, const void* in, int in_stride, const int32_t* tokens, int vocab, const __nv_bfloat16* table, int cols, int col, void* out,
+                      int out_stride, bool f32, cudaStream_t s);
 
 // ---- rotary positions --------------------------------------------------------------------------------------------------
 // Entry i of a vector whose first `dims` entries turn: the pair it belongs to, its partner, and whether it is the pair's first.
@@ -532,17 +564,21 @@ int launch_retention(const RetentionLaunch& a, cudaStream_t s, int* launches);
 // ---- grouped-query attention over pages (grouped_attention.cu) -----------------------------------------------------------
 // A page holds, head after head, 64 key rows of `pk` entries and 64 value rows of `pv` (in bf16 pools odd multiples of 16 bytes,
 // see LatentRow); dp and vp are the sizes padded to 16, padding entries are zero. block: entries of a (page, head) pair.
-struct GroupedRow { int groups = 0, dim = 0, vdim = 0, dp = 0, vp = 0, pk = 0, pv = 0, block = 0; };
-GroupedRow grouped_row(int groups, int dim, int vdim, bool f32);
+// shared: the values are the keys before their norm. One row per token is kept, and behind the 64 rows 64 fp32 numbers that turn
+// a row into its key.
+struct GroupedRow { int groups = 0, dim = 0, vdim = 0, dp = 0, vp = 0, pk = 0, pv = 0, block = 0, shared = 0; };
+GroupedRow grouped_row(int groups, int dim, int vdim, bool f32, bool shared);
 struct GroupedLaunch {
     GroupedRow row;
     int heads = 0, rot_dims = 0, rot_neighbours = 0, window = 0, chunk = 0, sink_one = 0;
     float scale = 1.f, eps = 0.f, weight_bias = 0.f, magnitude = 1.f, out_scale = 1.f;
+    int head_norm = 0, temp_every = 0; float temp_coef = 0.f;   // norm of q and k without weights; query temperature
     const float* inv_freq = nullptr;
     bool f32 = false;
     const __nv_bfloat16 *q_norm = nullptr, *k_norm = nullptr;
     void* qkv = nullptr; int qkv_stride = 0;               // q | k | v per row; q is normed and rotated in place
     const float* gate = nullptr; int gate_stride = 0;
+    const void* entry_gate = nullptr; int entry_gate_stride = 0;   // [rows][heads * vdim], in the activation type
     void* pool = nullptr;
     const int32_t* page_table = nullptr; int pages_per_seq = 0;
     const int32_t* row_seq = nullptr; const int32_t* row_pos = nullptr;
@@ -560,8 +596,9 @@ bool grouped_spans(const GroupedRow& r, bool f32);
 int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches);
 
 // ---- routed feed-forward (routed_mlp.cu) -------------------------------------------------------------------------------
-// shared_ff > 0: inner size of the feed-forward that every row takes
-struct RoutedShape { int experts = 0, top = 0, groups = 1, keep = 1, width = 0, ff = 0, shared_ff = 0; };
+// shared_ff > 0: inner size of the feed-forward that every row takes. The last `identity` of the experts + identity that are scored
+// hand their input through.
+struct RoutedShape { int experts = 0, top = 0, groups = 1, keep = 1, width = 0, ff = 0, shared_ff = 0, identity = 0; __host__ __device__ int scored() const { return experts + identity; } };
 struct RoutedLaunch {
     RoutedShape shape;
     float scale = 1.f;
@@ -573,6 +610,7 @@ struct RoutedLaunch {
     // the experts' rows one after the other; gate == null: an expert is down(gelu(up x))
     const Matrix *gate = nullptr, *up = nullptr, *down = nullptr;
     const Matrix *shared_up = nullptr, *shared_down = nullptr;
+    const __nv_bfloat16* correction = nullptr;             // [scored]: joins the scores for the choice only
     float* out = nullptr; int out_stride = 0;
     unsigned char* scratch = nullptr;
     unsigned* counts = nullptr;                            // [kMaxExperts], zero between launches

@@ -22,7 +22,18 @@ inline int dev_alloc(T** p, size_t count, int64_t* total = nullptr) {
 
 
 enum LaunchKind { L_EMBED, L_RMSNORM, L_QGEMV, L_QK_NORM, L_ATTN, L_SWIGLU, L_CONV, L_ARGMAX, L_SSM,
-                  L_PRODUCT, L_LATENT, L_DELTA, L_ROUTED, L_SOFTCAP, L_GROUPED, L_RETENTION };   // from L_PRODUCT on: fp32-stream plans only
+                  L_PRODUCT, L_LATENT, L_DELTA, L_ROUTED, L_SOFTCAP, L_GROUPED, L_RETENTION, L_JOIN, L_TOKEN_GATE };   // from L_PRODUCT on: fp32-stream plans only
+
+// What a launch over the residual stream does, in this order; parts that are not set are left out (see JoinLaunch).
+struct JoinParts {
+    const DenseTensor* table = nullptr; float table_scale = 1.f;               // starts the stream
+    int keep = -1;                                                             // convolution whose last inputs go to its state
+    bool adds = false; int in_buf = -1, gate_buf = -1; const DenseTensor* w = nullptr; float eps = 0.f, weight_bias = 0.f;
+    int store = -1; const DenseTensor* avg_w = nullptr; int avg = 0;           // results of the layers
+    int copy_buf = -1;
+    int conv = -1, conv_buf = -1; const DenseTensor* conv_w = nullptr;
+    bool changes() const { return table || adds || avg; }
+};
 
 struct Launch {
     int kind = 0;
@@ -58,6 +69,10 @@ struct Launch {
     const Matrix *m4 = nullptr, *m5 = nullptr;   // and the shared feed-forward's up and down
     GatedAct act;
     float softcap = 0.f;                      // of the output head's logits
+    const DenseTensor* seg_bias[kMaxProductSegs] = {};
+    Matrix part[2];                           // products of two inputs: the rows that meet the first and the second one
+    int x2_buf = -1, first_segs = 0;          // the second input, and how many results belong to the first
+    JoinParts join;
     const DenseTensor* dv[6] = {};            // gated delta rule: taps of q, k, v, norm weight, A_log, dt_bias; latent attention: [0] sink; norms: [0] table that joins
     int window_set = 0;                       // latent attention: index into plan->windows
     const DenseTensor* norm_post = nullptr;   // norm steps: weight of the norm applied to the input before it is added
@@ -76,6 +91,9 @@ struct LatentLayer { int rank = 0, rot = 0; LatentRow row{}; };
 
 // One grouped-attention layer's share of the page pool.
 struct GroupedLayer { GroupedRow row{}; };
+
+// One convolution over the stream: its last taps - 1 inputs per sequence, in fp32.
+struct StreamConv { int taps = 0; };
 
 // One gated-delta or retention layer: per sequence an fp32 state and the last inputs of the convolutions (retention: no taps).
 struct DeltaLayer {
@@ -99,6 +117,7 @@ struct StreamBufs {
     float* delta = nullptr; size_t delta_cap = 0;        // gated delta rule: records and read-outs of portions
     unsigned char* routed = nullptr; size_t routed_cap = 0;
     float* argmax_val = nullptr; int32_t* argmax_idx = nullptr;
+    float* results = nullptr;             // depth-wise average: [result][rows][width of RESIDUAL]
 };
 
 // One batch of rows for the row executor (device pointers).
@@ -161,6 +180,7 @@ struct swlm_plan {
     std::vector<LatentLayer> latent;      // by step.layer
     std::vector<GroupedLayer> grouped;    // by step.layer
     std::vector<DeltaLayer> delta;        // by step.layer
+    std::vector<StreamConv> convs;        // by step.layer
     std::vector<int> windows;             // distinct sliding windows of the attention layers
     int stream_width[SWLM_BUF_COUNT] = {};
     int latent_heads_max = 0, latent_q_floats = 0, latent_part_floats = 0;   // largest over the layers, per row / per row and split
@@ -218,6 +238,7 @@ struct swlm_state {
     // pool), the page table on host and device, and the two activation sets
     std::vector<void*> pool; std::vector<size_t> pool_bytes;
     std::vector<float*> delta_state; std::vector<void*> delta_ring;   // per gated-delta layer: [max_batch][state_elems], [max_batch][ring_elems]
+    std::vector<float*> conv_state;                                   // per convolution over the stream: [max_batch][taps - 1][hidden]
     unsigned* routed_counts = nullptr;                                // rows per expert, zero between launches
     int pool_pages = 0, pages_per_seq = 0;
     std::vector<int> free_pages;

@@ -74,6 +74,15 @@ class Step(C.Structure):
         ("score_act", C.c_int32),
         ("group_best", C.c_int32),
         ("raw_weights", C.c_int32),
+        ("in2_off", C.c_int32),
+        ("in3_off", C.c_int32),
+        ("value_is_key", C.c_int32),
+        ("head_norm", C.c_int32),
+        ("temp_coef", C.c_float),
+        ("temp_every", C.c_int32),
+        ("identity", C.c_int32),
+        ("expert_act", C.c_int32),
+        ("weight7", C.c_char * NAME_MAX),
     ]
 
 
@@ -105,6 +114,8 @@ class BuffersDesc(C.Structure):
         ("kv_pool_tokens", C.c_int32),
         ("delta_layers", C.c_int32),
         ("grouped_layers", C.c_int32),
+        ("stream_convs", C.c_int32),
+        ("depth_results", C.c_int32),
     ]
 
 

@@ -42,6 +42,12 @@ STEP_ROUTED_MLP = 19
 STEP_SOFTCAP = 20
 STEP_GROUPED_ATTN = 21
 STEP_RETENTION = 22
+STEP_GATED_POSTNORM_ADD = 23
+STEP_DEPTH_AVG = 24
+STEP_STREAM_CONV = 25
+STEP_STREAM_COPY = 26
+STEP_TOKEN_GATE = 27
+EXPERT_CLAMPED, EXPERT_SILU = 0, 1
 GATE_SILU, GATE_SIGMOID = 0, 1
 SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
 ROPE_HALVES, ROPE_NEIGHBOURS = 0, 1
