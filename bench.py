@@ -596,6 +596,22 @@ def run_rirotar(args, pkg):
     print(json.dumps(dict(design_line(args, "Rirotar", ours, workload), rirotar=ours, vuzunex_equal_size=closest, deltanet_recurrence_equal_heads=like)))
 
 
+def measure_llama_attention(pkg, args, stream, timed, heads, kv_heads):
+    """Grouped-query attention of the Llama recipe at the same heads, in a model with little else."""
+    P, batch = pkg.plan, args.batch
+    lcfg = pkg.ModelConfig("llama", 1024, 1024, 4, heads, kv_heads, 128, 4096, max_seq=bench_max_seq(args), max_batch=batch)
+    builder = pkg.DispatchPlanBuilder(lcfg)
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, block_weights(builder))
+    model.set_stream(stream.cuda_stream)
+    model.prefill(np.random.default_rng(8).integers(0, 4096, size=(batch, args.ctx), dtype=np.int32))
+    timer = KindTimer(model, timed, [])
+    like = {"decode_attention": timer.hbm_entry(timer.decode(P.STEP_ATTN_DECODE), 4 * batch * model.position * kv_heads * 256 * 2, 4)}
+    model.close()
+    store.close()
+    return like
+
+
 KALEVIK_SHAPES = {   # layers and the loop over some of them; experts and their choice are RIROTAR_SHAPES's
     "1b": (9, (3, 6, 2)), "8b": (6, (2, 4, 2))}
 KALEVIK_CHUNK = 8192
@@ -652,21 +668,79 @@ def run_kalevik(args, pkg):
     closest, rcfg = measure_rirotar(pkg, args, stream, timed)
     assert len(rcfg.layers) == len(runs)
     vuzunex = measure_vuzunex(pkg, vuzunex_config(pkg, args, 4, bench_max_seq(args)), args, stream, timed)
-    # grouped-query attention of the Llama recipe at the same heads, in a model with little else
-    like = {}
-    lcfg = pkg.ModelConfig("llama", 1024, 1024, 4, heads, kv_heads, 128, 4096, max_seq=bench_max_seq(args), max_batch=batch)
-    builder = pkg.DispatchPlanBuilder(lcfg)
-    store = pkg.WeightStore(0)
-    model = pkg.load_model(store, builder, block_weights(builder))
-    model.set_stream(stream.cuda_stream)
-    model.prefill(np.random.default_rng(8).integers(0, 4096, size=(batch, ctx), dtype=np.int32))
-    like["decode_attention"] = t.hbm_entry(KindTimer(model, timed, []).decode(P.STEP_ATTN_DECODE), 4 * batch * model.position * kv_heads * 256 * 2, 4)
-    model.close()
-    store.close()
+    like = measure_llama_attention(pkg, args, stream, timed, heads, kv_heads)
     workload = (f"{layers} layers (latent and parallel in turn), layers {loop[0]} .. {loop[1] - 1} run {loop[2]} times, width {width}, {heads} heads, latent 512 + 64, "
                 f"{kv_heads} key / value heads of 128 in chunks of {KALEVIK_CHUNK}, retention of 128 x 128, {top} of {experts} experts of {ff // top} and a shared one of {ff // 2}, "
                 f"vocabulary {BENCH_VOCAB}, context {ctx}, batch {batch}")
     print(json.dumps(dict(design_line(args, "Kalevik", ours, workload), kalevik=ours, rirotar_equal_size=closest, vuzunex_kernels=vuzunex, llama_attention_equal_heads=like)))
+
+
+MERUDRA_TAPS, MERUDRA_SIDE = 4, 256   # convolutions over the stream, entries per token and layer
+
+
+def merudra_stream_bytes(layers, n, width):
+    """Bytes that the launches over the stream move for n rows: what sublayers return, their gates, the stream, earlier results, and
+    what the next products read."""
+    per_entry = 2 + 4 + 4 + 2 + 2                                        # embedding -> stream, result 0, convolution, copy
+    for i in range(layers):
+        per_entry += (4 + 4 + 4) + 4 + 2 + 2                             # mixer: result, gate, stream -> stream, convolution, copy
+        per_entry += (4 + 4 + 4) + 4 + 2                                 # feed-forward: the same without a convolution
+        per_entry += (4 + 4 + 4 * (i + 1)) + 4 + 4 + (4 if i + 1 < layers else 0)   # token input, average -> result, stream, convolution, copy
+    return n * width * per_entry
+
+
+def run_merudra(args, pkg):
+    """Prompt and decode throughput of the Merudra design (two attention layers whose values are their keys to one gated-delta layer,
+    routed feed-forwards with identity experts, gated results, convolutions over the stream, token inputs, depth-wise averages) beside
+    Rirotar at equal width, heads, layers, vocabulary and active feed-forward, and its attention beside the Llama recipe's at equal
+    heads. One JSON line."""
+    M, P = pkg.merudra, pkg.plan
+    stream = bench_stream()
+    timed = stream_timer(stream)
+    width, heads, ff, _ = VUZUNEX_SHAPES[args.shape]
+    layers, experts, top, _, _ = RIROTAR_SHAPES[args.shape]
+    batch, ctx, kv_heads, identity = args.batch, args.ctx, heads // 4, experts // 8
+    routed = M.RoutedFF(ff // top, experts, identity, top)
+    attention, delta = M.KeyValueAttention(heads, kv_heads, 128, 128 ** -0.5, 0.5, 1024), M.GatedDelta(heads, heads // 2, 128, 128, 4)
+    cfg = pkg.MerudraConfig(vocab=BENCH_VOCAB, width=width, taps=MERUDRA_TAPS, side=MERUDRA_SIDE, layers=[M.Layer(delta if i % 3 == 2 else attention, routed) for i in range(layers)],
+                            max_seq=bench_max_seq(args), max_batch=batch)
+    n_delta = layers // 3
+    n_attention = layers - n_delta
+    builder = pkg.MerudraPlanBuilder(cfg)
+    weights = block_weights(builder)
+    for i in range(layers):   # averages that keep the stream alive, choices that the scores decide
+        weights[f"l{i}.dwa"] = np.where(np.arange(i + 2) == i + 1, 0x3F80, 0x3DCD).astype(np.uint16)   # 1.0, else 0.1
+        weights[f"l{i}.mlp.correction"][:] = 0
+    store = pkg.WeightStore(0)
+    model = pkg.load_model(store, builder, weights)
+    model.set_stream(stream.cuda_stream)
+    prompt = np.random.default_rng(7).integers(0, BENCH_VOCAB, size=(batch, ctx), dtype=np.int32)
+    ours = serve_rates(model, prompt, args, timed)
+    n = min(ctx, 2048)
+    t = KindTimer(model, timed, prompt[0, :n])
+    product_bytes = cfg.product_elems() * 2
+    chosen = top * experts / (experts + identity)   # with tensors, on average
+    ours["decode_products"] = t.hbm_entry(t.decode(P.STEP_PRODUCT), product_bytes, layers)
+    ours["decode_routed"] = t.hbm_entry(t.decode(P.STEP_ROUTED_MLP), layers * reached_experts(experts, chosen, batch) * 3 * width * (ff // top) * 2, layers)
+    # one row of 128 entries and a factor per token and key head
+    ours["decode_grouped_step"] = t.hbm_entry(t.decode(P.STEP_GROUPED_ATTN), n_attention * batch * model.position * kv_heads * (256 + 4), n_attention)
+    ours["decode_delta_step"] = t.hbm_entry(t.decode(P.STEP_GATED_DELTA), 2.0 * n_delta * batch * heads * 128 * 128 * 4, n_delta)
+    ours["decode_stream_us_per_layer"] = t.decode(P.STEP_GATED_POSTNORM_ADD) * 1e3 / layers
+    model.reset_state()
+    ours["prefill_products"] = t.tensor_entry(t.portion(P.STEP_PRODUCT), 2.0 * n * (product_bytes / 2 - BENCH_VOCAB * width), layers)
+    ours["prefill_routed"] = t.tensor_entry(t.portion(P.STEP_ROUTED_MLP), layers * 2.0 * n * chosen * 3 * width * (ff // top), layers)
+    ours["prefill_grouped_step"] = t.tensor_entry(t.portion(P.STEP_GROUPED_ATTN), n_attention * heads * n * (n + 1) / 2 * 2.0 * 256, n_attention)
+    us = t.portion(P.STEP_GATED_DELTA) * 1e3 / n_delta
+    ours["prefill_delta"] = {"rows": n, "us_per_layer": us, "fp32_tflops": n * heads * 128 * 128 * 7.0 / us / 1e6}
+    ours["prefill_stream"] = t.hbm_entry(t.portion(P.STEP_GATED_POSTNORM_ADD), merudra_stream_bytes(layers, n, width), layers)
+    model.close()
+    store.close()
+    closest, _ = measure_rirotar(pkg, args, stream, timed)
+    like = measure_llama_attention(pkg, args, stream, timed, heads, kv_heads)
+    vuzunex = measure_vuzunex(pkg, vuzunex_config(pkg, args, 4, bench_max_seq(args)), args, stream, timed)
+    workload = (f"{layers} layers (attention, attention, delta), width {width}, {heads} heads of 128 over {kv_heads} key heads, states of 128 x 128, {top} of {experts} + {identity} "
+                f"experts of {ff // top}, {MERUDRA_TAPS} taps over the stream, {MERUDRA_SIDE} entries per token and layer, vocabulary {BENCH_VOCAB}, context {ctx}, batch {batch}")
+    print(json.dumps(dict(design_line(args, "Merudra", ours, workload), merudra=ours, rirotar_equal_size=closest, vuzunex_kernels=vuzunex, llama_attention_equal_heads=like)))
 
 
 def main():
@@ -684,9 +758,9 @@ def main():
     ap.add_argument("--prefill", choices=["real", "synthetic"], default="real",
                     help="how the KV cache gets its `ctx` tokens: by running the prompt, or random bf16 rows")
     ap.add_argument("--small", action="store_true")
-    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex", "rirotar", "kalevik"], default="llama",
-                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size; rirotar: the gated-delta design beside Vuzunex of equal size; kalevik: the looped latent / retention design beside Rirotar of equal size")
-    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex, rirotar, kalevik: which layer sizes")
+    ap.add_argument("--model", choices=["llama", "lfm2", "vuzunex", "rirotar", "kalevik", "merudra"], default="llama",
+                    help="llama: Llama-3-8B shape; lfm2: the hybrid conv/attention shape; vuzunex: the latent-attention design beside a Llama of equal size; rirotar: the gated-delta design beside Vuzunex of equal size; kalevik: the looped latent / retention design beside Rirotar of equal size; merudra: the stream-reading attention / delta design beside Rirotar of equal size")
+    ap.add_argument("--shape", choices=sorted(VUZUNEX_SHAPES), default="1b", help="--model vuzunex, rirotar, kalevik, merudra: which layer sizes")
     ap.add_argument("--batch", type=int, default=1, help="sequences decoded together (1..64), all at the same position")
     ap.add_argument("--kv", choices=["bf16", "q8", "rotor-q4", "rotor-q4-qjl16"], default="bf16",
                     help="KV cache elements: bf16, 8-bit groups of 32 (36-byte blocks), or the rotated 4-bit groups of 64 "
@@ -704,6 +778,9 @@ def main():
         return
     if args.model == "kalevik":
         run_kalevik(args, pkg)
+        return
+    if args.model == "merudra":
+        run_merudra(args, pkg)
         return
     if args.model == "lfm2" and args.ctx == 4096:
         args.ctx = 2048   # the hybrid configuration's prompt length

@@ -1,0 +1,390 @@
+"""Merudra models on a GPU against the plain implementation: prompts, decoding, portions, mixed batches, pages, slots and states
+used again, keys at page borders, far keys and far writes to a state, the first tokens, long decoding, greedy generation through
+the scheduler and the command line tools."""
+import json
+
+import numpy as np
+import pytest
+
+import merudra_cases as mc
+import plain_merudra as plain
+from test_gpu_vuzunex import run_tool
+
+pytestmark = pytest.mark.gpu
+DTYPES = ["float32", "bfloat16"]
+
+
+class Loaded:
+    def __init__(self, pkg, cfg, dtype, seed=5, **runtime):
+        self.cfg, self.dtype = cfg, dtype
+        self.bits, self.weights = mc.random_weights(cfg, seed)
+        self.store = pkg.WeightStore(0)
+        self.builder = mc.builder_of(pkg, cfg, dtype, **runtime)
+        self.model = pkg.load_model(self.store, self.builder, self.bits)
+
+    def tokens(self, n, seed=0):
+        return np.random.default_rng(seed + 77).integers(0, self.cfg["vocab"], size=n).tolist()
+
+    def plain(self, tokens):
+        return plain.forward(self.cfg, self.weights, tokens)[0]
+
+    def portions(self, seq, tokens, sizes):
+        """Logits of every token, fed in portions of the given sizes (the last one repeated)."""
+        out, at, i = [], 0, 0
+        while at < len(tokens):
+            n = min(sizes[min(i, len(sizes) - 1)], len(tokens) - at)
+            out.append(self.model.run_batch([(seq, tokens[at:at + n], list(range(n)))])[0])
+            at, i = at + n, i + 1
+        return np.concatenate(out)
+
+    def agree(self, got, want, slack=1.0):
+        mc.agree(got, want, self.cfg, self.dtype, slack)
+
+    def close(self):
+        self.model.close()
+        self.store.close()
+
+
+@pytest.fixture
+def load(pkg):
+    made = []
+
+    def make(case, dtype, **kw):
+        made.append(Loaded(pkg, mc.cases()[case] if isinstance(case, str) else case, dtype, **kw))
+        return made[-1]
+
+    yield make
+    for m in made:
+        m.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", sorted(mc.cases()))
+def test_prompt_portions_and_decoding_agree_with_the_plain_model(load, dtype, name):
+    m = load(name, dtype)
+    tokens = m.tokens(150)
+    want = m.plain(tokens)
+    m.agree(m.portions(0, tokens, [150]), want)
+    m.model.reset_sequence(0)
+    m.agree(m.portions(0, tokens, [1]), want)
+    for seq, sizes in enumerate(([2], [64, 2, 63, 3, 65], [5, 64, 1, 80], [100, 1])):
+        if seq == 0:
+            m.model.reset_sequence(0)
+        m.agree(m.portions(seq, tokens, sizes), want)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["mid", "odd", "tiny"])
+def test_stream_after_every_layer(pkg, load, dtype, name):
+    m = load(name, dtype)
+    tokens = m.tokens(90)
+    _, after = plain.forward(m.cfg, m.weights, tokens)
+    for n in range(1, len(after) + 1):
+        model = pkg.InferenceModel(m.store, m.builder.decode_steps(layers=n), m.builder.config.buffers_desc(n))
+        for rows in (90, 3, 1):
+            model.run_batch([(0, tokens[:rows], list(range(rows)))])
+            got = model.read_buffer_f32(pkg.plan.BUF_RESIDUAL, rows, m.cfg["width"])
+            err = np.abs(got - after[n - 1][:rows]).max(axis=1) / np.abs(after[n - 1]).max()
+            # (in bf16 an expert with an all but equal score may be another: the bulk of the rows counts)
+            assert (err.max() if dtype == "float32" else np.quantile(err, 0.7)) <= (1e-5 if dtype == "float32" else 3e-2)
+            model.reset_sequence(0)
+        model.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["mid", "odd", "wide", "broad", "big", "state_only"])
+def test_mixed_batches_against_each_request_alone(load, dtype, name):
+    m = load(name, dtype, max_batch=4, max_seq=256)
+    requests = [m.tokens(n, seed=i) for i, n in enumerate((201, 1, 130, 67))]
+    cuts = [[70, 1, 1, 64, 65], [1], [1, 1, 66, 1, 61], [2, 3, 60, 1, 1]]
+    alone = []
+    for r in requests:
+        alone.append(m.portions(0, r, [len(r)]))
+        m.model.reset_sequence(0)
+    got, at = [[] for _ in requests], [0] * 4
+    for step in range(5):
+        entries = []
+        for i in (2, 0, 3, 1):   # not in the order of the slots
+            if step < len(cuts[i]) and at[i] < len(requests[i]):
+                n = cuts[i][step]
+                entries.append((i, requests[i][at[i]:at[i] + n], list(range(n))))
+                at[i] += n
+        logits, greedy = m.model.run_batch(entries)
+        assert greedy.tolist() == np.argmax(logits, axis=1).tolist()
+        row = 0
+        for i, part, _ in entries:
+            got[i].append(logits[row:row + len(part)])
+            row += len(part)
+    for i, r in enumerate(requests):
+        assert at[i] == len(r)
+        g = np.concatenate(got[i])
+        m.agree(g, m.plain(r))
+        m.agree(g, alone[i].astype(np.float64))
+    assert m.model.positions.tolist() == [201, 1, 130, 67]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_pages_slots_and_states_are_used_again(pkg, load, dtype):
+    m = load("mid", dtype, max_batch=3, max_seq=256, pool_tokens=5 * 64)
+    model = m.model
+    assert model.free_pages == 5
+    a, b, c = m.tokens(65, 1), m.tokens(130, 2), m.tokens(60, 3)
+    wa, wb, wc = m.plain(a), m.plain(b), m.plain(c)
+    m.agree(m.portions(0, a, [40, 1]), wa)
+    m.agree(m.portions(1, b, [128, 1]), wb)
+    assert model.free_pages == 0
+    with pytest.raises(pkg.SwlmError):   # no page left: refused, nothing changed
+        model.run_batch([(1, b[:1], [0]), (2, c, [0])])
+    assert model.free_pages == 0 and model.positions.tolist() == [65, 130, 0]
+    # slots whose states and pages other requests have used; a first token alone and a first portion
+    model.reset_sequence(0)
+    m.agree(m.portions(2, c, [7, 9]), wc)
+    m.agree(m.portions(0, c, [1]), wc)
+    model.reset_sequence(1)
+    model.reset_sequence(2)
+    m.agree(m.portions(1, c, [60]), wc)
+    model.reset_state()
+    for seq in (2, 0):
+        m.agree(m.portions(seq, b[:100], [64, 1]), wb[:100])
+    # a request that is left out of steps and goes on
+    model.reset_state()
+    first = m.portions(1, b[:50], [50])
+    m.portions(0, a, [30, 1])
+    m.agree(np.concatenate([first, m.portions(1, b[50:], [3, 1, 76])]), wb)
+    model.reset_state()
+    assert model.free_pages == 5
+    lg, _ = model.run_batch([(1, a, [64, 0, 64])])
+    m.agree(np.repeat(lg, 3, axis=0), np.repeat(wa[[64, 0, 64]], 3, axis=0))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads, kv, dim, every", [(4, 2, 32, 64), (3, 3, 24, 1), (6, 1, 13, 65), (2, 1, 136, 40), (2, 2, 264, 30)])
+def test_keys_at_page_borders_and_the_query_temperature(load, dtype, heads, kv, dim, every):
+    """Sharpened scores and little beside them: a row's result hangs on few keys and on its own temperature."""
+    def one(every=every, coef=1.5, sharpen=1.5):
+        return mc.config(256, 96, [mc.attention(heads, kv, dim, None, (coef, every), sharpen)], taps=2, side=8)
+
+    m = load(one(), dtype)
+    tokens = m.tokens(200, seed=9)
+    want = m.plain(tokens)
+    limit = {"float32": 5e-5, "bfloat16": 5e-2}[dtype]
+    for sizes in ([200], [64, 65, 1], [1], [127, 2, 1], [63, 66, 2], [every, every + 1, 2]):
+        err = mc.row_errors(m.portions(0, tokens, sizes), want)
+        assert err.max() <= limit, (sizes, int(err.argmax()), float(err.max()))
+        m.model.reset_sequence(0)
+    # the test itself: a step of the temperature one position off, or a key at a border that is left out, shows
+    shows = 10 * 5e-5
+    off = mc.row_errors(plain.forward(one(every=every + 1), m.weights, tokens)[0], want)
+    assert off[:every - 1].max(initial=0.0) < 1e-12 and (off[every - 1:] > shows).any()
+    full = plain.causal_softmax
+    for key in (0, 63, 64, 127, 128):
+        def without(scores):
+            s = scores.copy()
+            s[:, key + 1:, key] = -1e30
+            return full(s)
+
+        plain.causal_softmax = without
+        try:
+            err = mc.row_errors(m.plain(tokens), want)
+        finally:
+            plain.causal_softmax = full
+        assert err[:key + 1].max() < 1e-12 and (err[key + 1:] > shows).any(), key
+
+
+def quiet(w):
+    """Nothing around the mixer of layer 0 looks back or depends on the token."""
+    for name in ("canon1", "rg1", "rg1.b"):
+        w["l0." + name][:] = 0.0
+    return w
+
+
+def far_key_weights(weights):
+    """Token 298 asks for token 299: their embeddings lie along channels 1 and 0, which all others lack, and the query projection
+    makes of the one what the key projection makes of the other."""
+    w = quiet({k: v.copy() for k, v in weights.items()})
+    w["embed"][:, :2] = 0.0
+    for token, channel in ((298, 1), (299, 0)):
+        w["embed"][token] *= 0.1
+        w["embed"][token, channel] = 6.0
+    probe = 0.6 * np.sign(w["l0.mix.k"][:, 0])
+    w["l0.mix.k"][:, 0], w["l0.mix.k"][:, 1] = probe, 0.0
+    w["l0.mix.q"][:, 0], w["l0.mix.q"][:, 1] = 0.0, np.tile(probe, w["l0.mix.q"].shape[0] // probe.size)
+    w["l0.mix.q.b"][:] = w["l0.mix.k.b"][:] = 0.0
+    return w
+
+
+def far_write_weights(weights):
+    """Token 299 alone writes to the state, token 298 asks for what it wrote, and nothing is forgotten: q of 298 is k of 299
+    (opposite embeddings, opposite projections), and a component that all embeddings share keeps everyone else's step size at
+    zero."""
+    w = quiet({k: v.copy() for k, v in weights.items()})
+    w["embed"][:, 0] = 3.0
+    w["embed"][298] = -w["embed"][299]
+    h = w["embed"]
+    w["l0.mix.b"] = np.tile(20.0 * h[299] / (h[299] @ h[299]), (w["l0.mix.b"].shape[0], 1))
+    w["l0.mix.b"][:, 0] -= 10.0 / 3.0
+    w["l0.mix.q"] = -w["l0.mix.k"]
+    for t in "qk":
+        w[f"l0.mix.{t}.conv"][:, -1], w[f"l0.mix.{t}.conv"][:, :-1] = 1.0, 0.0
+    w["l0.mix.A_log"][:] = -9.0
+    w["l0.norm1"] *= 3.0
+    return w
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("kind", ["key", "shared key", "write"])
+def test_a_far_token_is_found_again(pkg, load, dtype, kind):
+    layer = mc.delta(2, 1, 64, 48, None, conv=2) if kind == "write" else mc.attention(4, 1 if kind == "shared key" else 4, 64, None, (0.1, 100), 8.0)
+    m = load(mc.config(300, 96, [layer], taps=3, side=4), dtype, max_seq=640)
+    w = (far_write_weights if kind == "write" else far_key_weights)(m.weights)
+    m.bits = {k: mc.to_bf16_bits(v) for k, v in w.items()}
+    m.weights = {k: mc.from_bf16_bits(v) for k, v in m.bits.items()}
+    pkg.upload_weights(m.store, m.builder, m.bits)
+    tokens = np.random.default_rng(3).integers(0, 298, size=600)
+    tokens[599] = 298
+    absent = m.plain(tokens)
+    for where in (0, 3, 250):
+        t = tokens.copy()
+        t[where] = 299
+        want = m.plain(t)
+        assert mc.row_errors(absent[599:], want[599:])[0] > 0.2
+        for sizes in ([600], [599, 1], [300, 298, 2], [3, 1]):
+            got = m.portions(0, t.tolist(), sizes)
+            assert mc.row_errors(got[599:], want[599:])[0] <= (1e-4 if dtype == "float32" else 5e-2), (where, sizes)
+            m.model.reset_sequence(0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("taps", [2, 3, 9])
+def test_convolutions_over_the_stream_across_portions(load, dtype, taps):
+    """Nothing but the convolutions looks back (one key of weight: attention with a first token of its own per row would do, so the
+    mixer is a delta rule that forgets at once); portions shorter than the convolution, down to one and two tokens."""
+    cfg = mc.config(200, 72, [mc.delta(1, 1, 8, 16, mc.routed(2, 1, 3, 24), conv=1), mc.delta(1, 1, 8, 16, None, conv=1)], taps=taps, side=8)
+    m = load(cfg, dtype)
+    for i in range(2):
+        m.weights[f"l{i}.mix.A_log"][:] = 3.0
+        m.weights[f"l{i}.mix.dt_bias"][:] = 4.0
+        for j in (1, 2) if i == 0 else (1,):
+            m.weights[f"l{i}.canon{j}"] *= 2.0
+    m.bits = {k: mc.to_bf16_bits(v) for k, v in m.weights.items()}
+    m.weights = {k: mc.from_bf16_bits(v) for k, v in m.bits.items()}
+    for name, bits in m.bits.items():
+        if name.endswith(("A_log", "dt_bias", "canon1", "canon2")):
+            m.store.add_dense(name, bits)
+    tokens = m.tokens(60, seed=4)
+    want = m.plain(tokens)
+    for sizes in ([60], [1], [2], [3], [1, 2, 1, 3, 1, 1, 2], [taps - 1, taps, taps + 1, 1], [17, 1, 1, 2]):
+        m.agree(m.portions(0, tokens, sizes), want, slack=2.0)
+        m.model.reset_sequence(0)
+    # the test itself: a lost tap shows
+    for name in ("l0.canon1", "l0.canon2", "l1.canon1"):
+        w = dict(m.weights, **{name: m.weights[name] * (np.arange(taps) > 0)})
+        assert np.median(mc.row_errors(plain.forward(cfg, w, tokens)[0][taps:], want[taps:])) > 0.1
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["odd", "tiny", "mid"])
+def test_first_tokens_of_a_sequence(load, dtype, name):
+    """Convolutions and portions that reach beyond the start."""
+    m = load(name, dtype)
+    for n in (1, 2, 3, 5, 6, 7):
+        tokens = m.tokens(n, seed=n)
+        want = m.plain(tokens)
+        for sizes in ([n], [1], [1, 2], [2, 1]):
+            got = m.portions(n % 4, tokens, sizes)
+            m.model.reset_sequence(n % 4)
+            if dtype == "float32":
+                m.agree(got, want)
+            else:
+                assert np.median(mc.row_errors(got, want)) <= 5e-2
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("batch", [1, 3, 9])
+def test_long_greedy_decoding_through_the_decode_graph(load, dtype, batch):
+    m = load("mid", dtype, max_batch=batch, max_seq=320)
+    prompt = np.array([m.tokens(5, seed=i) for i in range(batch)], dtype=np.int32)
+    first = m.model.prefill(prompt)
+    tokens = np.concatenate([first[None], m.model.decode_n(first, 290)])
+    assert m.model.positions.tolist() == [295] * batch
+    for b in range(min(batch, 3)):
+        seq = prompt[b].tolist() + tokens[:, b].tolist()
+        logits = m.plain(seq)[4:-1]
+        top = logits.max(axis=1)
+        chosen = logits[np.arange(291), tokens[:, b]]
+        # the device's choice is the plain model's, or as good within rounding
+        worse = (top - chosen) / logits.std()
+        if dtype == "float32":
+            assert worse.max() <= 1e-3 and (chosen == top).mean() >= 0.99
+        else:
+            assert np.quantile(worse, 0.95) <= 0.2 and (chosen == top).mean() >= 0.8
+    again = m.model.decode(tokens[-1])
+    lg = m.model.logits()
+    assert again.tolist() == np.argmax(lg, axis=1).tolist()
+    if dtype == "float32":
+        m.agree(lg[:1], m.plain(prompt[0].tolist() + tokens[:, 0].tolist())[-1:])
+
+
+def test_prompt_chunks_snapshot_and_reset(load):
+    m = load("mid", "float32", max_batch=2, max_seq=256)
+    model, tokens = m.model, m.tokens(180)
+    want = int(np.argmax(m.plain(tokens)[-1]))
+    model.set_prefill_chunk(70)
+    assert model.prefill_sequence(1, tokens) == want
+    snap = model.prompt_snapshot()
+    a = model.run_batch([(1, [want], [0])])[0]
+    model.reset_state()
+    assert model.free_pages == 8 and model.positions.tolist() == [0, 0]
+    model.run_batch([(1, tokens[:100], [])])   # other data on the pages and in the states
+    model.restore(snap)
+    assert model.positions.tolist() == [0, 180]
+    assert np.array_equal(a, model.run_batch([(1, [want], [0])])[0])
+    model.free_snapshot(snap)
+
+
+@pytest.mark.parametrize("name, budget", [("mid", 5), ("mid", 48), ("odd", 512), ("tiny", 7)])
+def test_greedy_generation_through_the_scheduler(pkg, load, name, budget):
+    m = load(name, "float32", max_batch=3, max_seq=256, pool_tokens=6 * 64)
+    sched = pkg.BatchScheduler(m.model, row_budget=budget)
+    requests = [pkg.Request(i, m.tokens(n, seed=20 + i), k) for i, (n, k) in enumerate([(3, 6), (100, 4), (64, 5), (1, 8), (30, 3)])]
+    for r in requests:
+        sched.submit(r)
+    sched.run()
+    assert m.model.free_pages == 6
+    for r in requests:
+        tokens, margins = plain.greedy(m.cfg, m.weights, r.prompt, r.max_new_tokens)
+        assert min(margins) > 1e-4   # no tie that rounding could turn
+        assert r.generated == tokens
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_trace_replay(pkg, tmp_path, dtype):
+    cfg = mc.cases()["mid"]
+    bits, w = mc.random_weights(cfg, 8)
+    mc.write_model(pkg, cfg, bits, str(tmp_path / "model"))
+    (tmp_path / "out").mkdir()
+    rng = np.random.default_rng(1)
+    a, b = (rng.integers(0, cfg["vocab"], size=n).tolist() for n in (90, 70))
+    places = list(range(20, 68))
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:80], "want": [3, 79]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": a[80:81], "want": []}, {"id": "b", "tokens": b[:2], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "b", "tokens": b[2:], "want": places}, {"id": "a", "tokens": a[81:], "want": [8]}], "end": ["a", "b"]},
+             {"step": 3, "entries": [{"id": "c", "tokens": b, "want": places}], "end": ["c"]}]
+    out = run_tool("trace_run", ["--model", str(tmp_path / "model"), "--dtype", dtype, "--out", str(tmp_path / "out"), "--max-tokens", "256"],
+                   input="".join(json.dumps(s) + "\n" for s in steps))
+    assert [x for x in out.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
+    pa, pb = plain.forward(cfg, w, a)[0], plain.forward(cfg, w, b)[0]
+    for step, want in ((2, np.concatenate([pb[22:70], pa[[89]]])), (3, pb[20:68])):
+        got = np.fromfile(tmp_path / "out" / f"{step}.f32", dtype="<f4").reshape(want.shape)
+        mc.agree(got, want, cfg, dtype, slack=1.5)
+    assert not (tmp_path / "out" / "1.f32").exists()
+
+
+def test_generate_tool(pkg, tmp_path):
+    cfg = mc.cases()["tiny"]
+    bits, w = mc.random_weights(cfg, 2)
+    mc.write_model(pkg, cfg, bits, str(tmp_path / "model"))
+    prompts = [[5, 6, 7], [1], [60, 2]]
+    args = ["--model", str(tmp_path / "model"), "--max-new", "6", "--dtype", "float32", "--batch", "2", "--max-seq", "64"]
+    out = run_tool("generate", args + [x for p in prompts for x in ("--prompt", ",".join(map(str, p)))])
+    assert [[int(t) for t in line.split(",")] for line in out.stdout.splitlines()] == [plain.greedy(cfg, w, p, 6)[0] for p in prompts]
