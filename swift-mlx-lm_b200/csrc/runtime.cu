@@ -1296,7 +1296,6 @@ int swlm_ctx_create(int device_id, int tp_rank, int tp_size, swlm_ctx** out) {
     if (!rc) rc = routed_init();
     if (!rc) rc = grouped_init();
     if (!rc) rc = retention_init();
-    if (!rc) rc = join_init();
     if (rc) { cudaStreamDestroy(ctx->stream); delete ctx; return rc; }
     *out = ctx;
     return SWLM_OK;

@@ -560,6 +560,25 @@ int stream_compile(swlm_plan* plan) {
         B.steps_covered += 1;
         plan->launches.erase(plan->launches.begin() + i);
     }
+    // A join that only hands the stream on to a token input, its two products, and the join behind them
+    for (size_t i = 0; i + 4 < plan->launches.size(); ++i) {
+        const Launch *q = &plan->launches[i], &A = q[0], &G = q[1], &T = q[2], &P = q[3], &B = q[4];
+        if (A.kind != L_JOIN || G.kind != L_PRODUCT || T.kind != L_TOKEN_GATE || P.kind != L_PRODUCT || B.kind != L_JOIN) continue;
+        const bool plain = G.n_seg == 1 && P.n_seg == 1 && !G.m2 && !P.m2 && !G.st.weight2[0] && !P.st.weight2[0] && !G.seg_bias[0] && !P.seg_bias[0] && !G.norm.kind && !P.norm.kind && !G.st.in_off && !P.st.in_off &&
+                           !G.st.out_off && !P.st.out_off;
+        const bool chain = A.join.adds && A.join.copy_buf >= 0 && A.join.conv < 0 && !A.join.avg && A.join.store < 0 && G.st.in_buf == A.join.copy_buf && T.st.in_buf == G.st.out_buf && T.st.n == G.st.n &&
+                           P.st.in_buf == T.st.out_buf && P.st.k == T.st.n && P.st.out_buf == SWLM_BUF_HIDDEN && P.st.n == d.hidden && G.st.k == d.hidden && B.join.adds && B.join.gate_buf < 0 && B.join.keep < 0;
+        bool again = false;   // does anything read the buffers that are not written then, before they are written again?
+        for (const int buf : {A.join.copy_buf, T.st.out_buf, (int)G.st.out_buf})
+            for (size_t j = i + 4; j < plan->launches.size(); ++j) {
+                const Launch& C = plan->launches[j];
+                if (j > i + 4 && reads(C, buf)) { again = true; break; }
+                bool writes = C.kind == L_JOIN ? C.join.conv_buf == buf || C.join.copy_buf == buf : C.st.out_buf == buf;
+                for (int s2 = 0; s2 < C.n_seg; ++s2) writes |= C.seg_buf[s2] == buf;
+                if (writes) break;
+            }
+        if (plain && chain && !again) plan->launches[i].fused = 4;
+    }
     // the residual stream alternates between two buffers, so that a norm computed by every CTA of a product can be stored by one
     int cur = 0;
     for (Launch& L : plan->launches) {
@@ -711,6 +730,14 @@ void bufs_free(StreamBufs* b) {
     *b = StreamBufs{};
 }
 
+TokenInput token_input(const Launch* L) {
+    TokenInput t;
+    t.n = L[1].st.n;
+    t.gate = L[1].m1->data; t.gate_ld = L[1].m1->ld; t.proj = L[3].m1->data; t.proj_ld = L[3].m1->ld;
+    t.table = L[2].d1->data; t.cols = (int)L[2].d1->cols; t.col = L[2].st.in2_off;
+    return t;
+}
+
 float* residual(StreamBufs* b, int phys) { return phys ? b->res2 : static_cast<float*>(b->buf[SWLM_BUF_RESIDUAL]); }
 
 StreamNorm norm_of(swlm_state* s, StreamBufs* b, const RowBatch& r, const Launch& L, const swlm_step& st, const DenseTensor* w, int res_in, int res_out) {
@@ -739,8 +766,37 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
     auto column = [plan](StreamBufs* bufs, int buf, int off) -> void* { return static_cast<unsigned char*>(bufs->buf[buf]) + (size_t)off * stored_bytes(plan, buf); };
     s->last_bufs = b;
     s->last_res = plan->final_res;
-    for (const Launch& L : plan->launches) {
+    auto join_of = [&](const Launch& L) {
+        const JoinParts& j = L.join;
+        JoinLaunch a;
+        a.rows = r.rows; a.width = d.hidden; a.f32 = f32; a.singles = r.n_runs == 0;
+        a.row_seq = r.seq; a.row_pos = r.pos; a.tokens = r.tok; a.vocab = d.vocab;
+        a.res_stride = s->width[SWLM_BUF_RESIDUAL];
+        if (j.table) { a.table = j.table->data; a.table_scale = j.table_scale; }
+        else a.res_in = residual(b, L.res_in);
+        if (j.changes()) a.res_out = residual(b, L.res_out);
+        if (j.keep >= 0) { a.keep_ring = s->conv_state[j.keep]; a.keep_taps = plan->convs[j.keep].taps; }
+        if (j.adds) { a.in = static_cast<const float*>(b->buf[j.in_buf]); a.in_stride = s->width[j.in_buf]; a.w = j.w->data; a.eps = j.eps; a.weight_bias = j.weight_bias; }
+        if (j.adds && j.gate_buf >= 0) { a.gate = static_cast<const float*>(b->buf[j.gate_buf]); a.gate_stride = s->width[j.gate_buf]; }
+        a.results = b->results; a.result_step = (size_t)b->rows * a.res_stride; a.store = j.store;
+        if (j.avg) { a.avg_w = j.avg_w->data; a.avg = j.avg; }
+        if (j.conv >= 0) { a.conv_w = j.conv_w->data; a.conv_ring = s->conv_state[j.conv]; a.taps = plan->convs[j.conv].taps; a.conv_out = b->buf[j.conv_buf]; a.conv_stride = s->width[j.conv_buf]; }
+        if (j.copy_buf >= 0) { a.copy_out = b->buf[j.copy_buf]; a.copy_stride = s->width[j.copy_buf]; }
+        return a;
+    };
+    for (size_t li = 0; li < plan->launches.size(); ++li) {
+        const Launch& L = plan->launches[li];
         const swlm_step& st = L.st;
+        if (L.fused && r.n_runs == 0) {
+            const TokenInput t = token_input(&L);
+            if (token_input_fits(t, r.rows, d.hidden)) {
+                li += L.fused;
+                if (only_kind >= 0 && only_kind != L_JOIN) continue;
+                if ((rc = launch_token_input(join_of(L), t, join_of(plan->launches[li]), stream))) return rc;
+                s->launches += 1;
+                continue;
+            }
+        }
         const bool latent_kernel = only_kind == L_ATTN && (L.kind == L_LATENT || L.kind == L_GROUPED);
         if (only_kind >= 0 && L.kind != only_kind && !latent_kernel) continue;
         switch (L.kind) {
@@ -926,23 +982,9 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             break;
         }
         case L_JOIN: {
-            const JoinParts& j = L.join;
-            JoinLaunch a;
-            a.rows = r.rows; a.width = d.hidden; a.f32 = f32; a.singles = r.n_runs == 0;
-            a.row_seq = r.seq; a.row_pos = r.pos; a.tokens = r.tok;
-            a.res_stride = s->width[SWLM_BUF_RESIDUAL];
-            if (j.table) { a.table = j.table->data; a.vocab = d.vocab; a.table_scale = j.table_scale; }
-            else a.res_in = residual(b, L.res_in);
-            if (j.changes()) a.res_out = residual(b, L.res_out);
-            if (j.keep >= 0) { a.keep_ring = s->conv_state[j.keep]; a.keep_taps = plan->convs[j.keep].taps; }
-            if (j.adds) { a.in = static_cast<const float*>(b->buf[j.in_buf]); a.in_stride = s->width[j.in_buf]; a.w = j.w->data; a.eps = j.eps; a.weight_bias = j.weight_bias; }
-            if (j.adds && j.gate_buf >= 0) { a.gate = static_cast<const float*>(b->buf[j.gate_buf]); a.gate_stride = s->width[j.gate_buf]; }
-            a.results = b->results; a.result_step = (size_t)b->rows * a.res_stride; a.store = j.store;
-            if (j.avg) { a.avg_w = j.avg_w->data; a.avg = j.avg; }
-            if (j.conv >= 0) { a.conv_w = j.conv_w->data; a.conv_ring = s->conv_state[j.conv]; a.taps = plan->convs[j.conv].taps; a.conv_out = b->buf[j.conv_buf]; a.conv_stride = s->width[j.conv_buf]; }
-            if (j.copy_buf >= 0) { a.copy_out = b->buf[j.copy_buf]; a.copy_stride = s->width[j.copy_buf]; }
-            rc = launch_join(a, stream);
-            s->launches += 1;
+            int n = 0;
+            rc = launch_join(join_of(L), stream, &n);
+            s->launches += n;
             break;
         }
         case L_TOKEN_GATE:
@@ -1087,7 +1129,9 @@ int stream_enqueue_step(swlm_state* s, bool body_only, cudaStream_t stream, int 
 int stream_launches_per_step(const swlm_plan* plan) {
     const int m = plan->desc.max_batch;
     int n = 0;
-    for (const Launch& L : plan->launches) {
+    for (size_t li = 0; li < plan->launches.size(); ++li) {
+        const Launch& L = plan->launches[li];
+        if (L.fused && token_input_fits(token_input(&L), m, plan->desc.hidden)) { n += 1; li += L.fused; continue; }
         if (L.kind == L_PRODUCT) {
             ProductLaunch a;
             a.w = L.m1; a.w2 = L.m2; a.m = m; a.x_f32 = plan->all_f32();

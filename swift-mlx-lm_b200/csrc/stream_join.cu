@@ -1,20 +1,30 @@
 // The residual stream between the sublayers of designs whose sublayers read the stream itself: what a sublayer returns is gated,
 // normed and added, results of layers are averaged over the depth, and the next sublayer gets the stream with a short causal
-// convolution over it. Everything that happens between two products is one launch over the batch's rows; all of it is fp32.
+// convolution over it. All of it is fp32.
 //
-// The convolution needs the stream at the tokens in front of a row. Inside a portion those are rows of the same launch, so a CTA
-// walks consecutive rows and keeps the last ones in shared memory; in front of its first row it works out as many rows of its
-// neighbour again as the convolution reaches back. In front of a portion they come from the state of the sequence. The state is
-// written by the launch that changes the stream next (it reads the same rows), so no CTA writes what another still reads.
+//   single tokens   stream_step_kernel: everything between two products in one launch, a cluster of CTAs per row that share its
+//                   columns; the norm's sum crosses the cluster through distributed shared memory. With a token input in between
+//                   (two small products with a gated table row between them, then a second norm) that is part of it: a CTA
+//                   multiplies its columns of the stream, the sums cross the cluster, and it works out its columns of the result.
+//   portions        stream_join_kernel (a CTA per row) and stream_conv_kernel (a thread walks a few rows of four channels).
+//
+// A convolution finds the tokens in front of a portion in the state of the sequence. The state is written by the launch that
+// changes the stream next (it reads the same rows), so nobody writes what others still read.
+#include <cooperative_groups.h>
+
 #include <algorithm>
+#include <utility>
 
 #include "swlm_internal.h"
+
+namespace cg = cooperative_groups;
 
 namespace swlm {
 namespace {
 
-constexpr int kJoinWarpsMax = 16;
-constexpr size_t kJoinMaxSmem = 200 * 1024;
+constexpr int kConvRows = 16, kConvThreads = 128;
+constexpr int kStepCluster = 8, kStepMaxRows = 16;   // rows beyond which the products of a token input run on their own
+constexpr int kSideThreads = 256, kSideRows = 16;    // weight rows of a warp whose loads are in flight together
 
 __device__ __forceinline__ void jn_put4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
 __device__ __forceinline__ void jn_put4(__nv_bfloat16* p, const float (&v)[4]) {
@@ -39,146 +49,329 @@ __device__ __forceinline__ void jn_weights4(const __nv_bfloat16* p, int i, int n
 }
 __device__ __forceinline__ float jn_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 
-// CTA: rows_per_cta consecutive rows. A thread keeps entries 4 (tid + NT j) .. + 3 of a row; the next row is requested while the
-// present one waits for its norm. Shared memory: [taps - 1][width] last rows of the stream, then [taps][width] weights in bf16
-// (a thread only ever touches its own columns of the rows).
+// sum over j < avg - 1 of avg_w[j] * results[j] at four entries of a row
+__device__ __forceinline__ void jn_results(const JoinLaunch& p, int r, int i, float (&sum)[4]) {
+    sum[0] = sum[1] = sum[2] = sum[3] = 0.f;
+    const float* at = p.results + (size_t)r * p.res_stride + i;
+#pragma unroll 8
+    for (int q = 0; q < p.avg - 1; ++q) {
+        float v[4];
+        jn_get4(at + q * p.result_step, v);
+        const float w = __bfloat162float(p.avg_w[q]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sum[e] = fmaf(w, v[e], sum[e]);
+    }
+}
+__device__ __forceinline__ void jn_average(const JoinLaunch& p, int r, int i, float (&h)[4]) {
+    float sum[4];
+    jn_results(p, r, i, sum);
+    const float w = __bfloat162float(p.avg_w[p.avg - 1]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h[e] = fmaf(w, h[e], sum[e]);
+}
+
+// ---- portions: gate, norm, sum, average -------------------------------------------------------------------------------
+// CTA per row; a thread keeps entries 4 (tid + NT j) .. + 3.
 template <typename T, int J, int NT>
-__global__ void __launch_bounds__(NT) stream_join_kernel(const JoinLaunch p, int rows_per_cta) {
-    extern __shared__ __align__(16) unsigned char join_smem[];
-    __shared__ float red[2][kJoinWarpsMax];
-    const int tid = threadIdx.x, width = p.width, pitch = (width + 3) / 4 * 4, past = max(0, p.taps - 1);
-    float* hist = reinterpret_cast<float*>(join_smem);
-    __nv_bfloat16* cw = reinterpret_cast<__nv_bfloat16*>(hist + (size_t)past * pitch);
+__global__ void __launch_bounds__(NT, 1024 / NT) stream_join_kernel(const JoinLaunch p) {
+    __shared__ float red[NT / 32];
+    const int tid = threadIdx.x, width = p.width, r = blockIdx.x;
     const bool whole = (width & 3) == 0;
     pdl_launch_dependents();
-    float nw[J][4];
+    pdl_wait();
+    const int seq = p.row_seq[r];
+    float h[J][4], t[J][4];
+    const __nv_bfloat16* row = p.table ? p.table + (size_t)min(max(p.tokens[r], 0), p.vocab - 1) * width : nullptr;
+    float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < J; ++j) {
         const int i = 4 * (tid + NT * j);
-        if (p.in) jn_weights4(p.w, i, width, whole, nw[j]);
+        h[j][0] = h[j][1] = h[j][2] = h[j][3] = t[j][0] = t[j][1] = t[j][2] = t[j][3] = 0.f;
+        if (i >= width) continue;
+        if (row) jn_weights4(row, i, width, whole, h[j]);
+        else jn_get4(p.res_in + (size_t)r * p.res_stride + i, h[j]);
+        if (p.in) jn_get4(p.in + (size_t)r * p.in_stride + i, t[j]);
+        float gate[4];
+        if (p.gate) jn_get4(p.gate + (size_t)r * p.gate_stride + i, gate);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) nw[j][e] += p.weight_bias;
-        if (p.conv_out)
-            for (int e = 0; e < 4; ++e)
-                for (int k = 0; k < p.taps; ++k)
-                    if (i + e < pitch) cw[(size_t)k * pitch + i + e] = i + e < width ? p.conv_w[(size_t)(i + e) * p.taps + k] : __float2bfloat16_rn(0.f);
+        for (int e = 0; e < 4; ++e) {
+            if (row) h[j][e] *= p.table_scale;
+            if (p.gate) t[j][e] *= jn_sigmoid(gate[e]);
+            if (i + e >= width) h[j][e] = t[j][e] = 0.f;
+            ss = fmaf(t[j][e], t[j][e], ss);
+        }
     }
-    pdl_wait();
-    const int r0 = blockIdx.x * rows_per_cta, r1 = min(r0 + rows_per_cta, p.rows);
-    int first = r0;   // rows in front of r0 that the convolution reaches
-    for (int n = 0; n < past && p.conv_out && first > 0 && p.row_seq[first - 1] == p.row_seq[r0]; ++n) --first;
-
-    float x[J][4], in[J][4], gate[J][4], sum[J][4];
-    auto request = [&](int r) {
-        const __nv_bfloat16* row = p.table ? p.table + (size_t)min(max(p.tokens[r], 0), p.vocab - 1) * width : nullptr;
+    if (p.keep_ring && !(r + p.keep_taps - 1 < p.rows && p.row_seq[r + p.keep_taps - 1] == seq)) {   // among the last of its portion
+        float* keep = p.keep_ring + ((size_t)seq * (p.keep_taps - 1) + p.row_pos[r] % (p.keep_taps - 1)) * width;
 #pragma unroll
-        for (int j = 0; j < J; ++j) {
-            const int i = 4 * (tid + NT * j);
-            if (i >= width) continue;
-            if (row) jn_weights4(row, i, width, whole, x[j]);
-            else jn_get4(p.res_in + (size_t)r * p.res_stride + i, x[j]);
-            if (p.in) jn_get4(p.in + (size_t)r * p.in_stride + i, in[j]);
-            if (p.gate) jn_get4(p.gate + (size_t)r * p.gate_stride + i, gate[j]);
-        }
-        if (p.avg) {
+        for (int j = 0; j < J; ++j)
 #pragma unroll
-            for (int j = 0; j < J; ++j) sum[j][0] = sum[j][1] = sum[j][2] = sum[j][3] = 0.f;
-#pragma unroll 4
-            for (int q = 0; q < p.avg - 1; ++q) {
-                const float w = __bfloat162float(p.avg_w[q]);
-                const float* result = p.results + q * p.result_step + (size_t)r * p.res_stride;
+            for (int e = 0; e < 4; ++e) { const int i = 4 * (tid + NT * j) + e; if (i < width) keep[i] = h[j][e]; }
+    }
+    float scale = 0.f;
+    if (p.in) {
+        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
+        __syncthreads();
+        float total = 0.f;
 #pragma unroll
-                for (int j = 0; j < J; ++j) {
-                    const int i = 4 * (tid + NT * j);
-                    if (i >= width) continue;
-                    float v[4];
-                    jn_get4(result + i, v);
+        for (int i = 0; i < NT / 32; ++i) total += red[i];
+        scale = 1.0f / sqrtf(total / (float)width + p.eps);
+    }
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) sum[j][e] = fmaf(w, v[e], sum[j][e]);
-                }
-            }
-        }
-    };
-    request(first);
-    const float own_w = p.avg ? __bfloat162float(p.avg_w[p.avg - 1]) : 1.f;
-    int slot = 0;   // of the row in hist
-    for (int r = first, turn = 0; r < r1; ++r, turn ^= 1) {
-        float h[J][4], t[J][4], before[J][4];
-        float ss = 0.f;
-#pragma unroll
-        for (int j = 0; j < J; ++j) {
-            const int i = 4 * (tid + NT * j);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const bool live = i + e < width;
-                h[j][e] = live ? x[j][e] * (p.table ? p.table_scale : 1.f) : 0.f;
-                t[j][e] = !live || !p.in ? 0.f : p.gate ? in[j][e] * jn_sigmoid(gate[j][e]) : in[j][e];
-                before[j][e] = p.avg ? sum[j][e] : 0.f;
-                ss = fmaf(t[j][e], t[j][e], ss);
-            }
-        }
-        const bool mine = r >= r0;
-        const int seq = p.row_seq[r], pos = p.row_pos[r];
-        if (p.keep_ring && mine && !(r + p.keep_taps - 1 < p.rows && p.row_seq[r + p.keep_taps - 1] == seq)) {
-            float* keep = p.keep_ring + ((size_t)seq * (p.keep_taps - 1) + pos % (p.keep_taps - 1)) * width;
-#pragma unroll
-            for (int j = 0; j < J; ++j)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) { const int i = 4 * (tid + NT * j) + e; if (i < width) keep[i] = h[j][e]; }
-        }
-        if (r + 1 < r1) request(r + 1);
+    for (int j = 0; j < J; ++j) {
+        const int i = 4 * (tid + NT * j);
+        if (i >= width) continue;
         if (p.in) {
-            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-            if ((tid & 31) == 0) red[turn][tid >> 5] = ss;
-            __syncthreads();
-            float total = 0.f;
+            float w[4];
+            jn_weights4(p.w, i, width, whole, w);
 #pragma unroll
-            for (int i = 0; i < NT / 32; ++i) total += red[turn][i];
-            const float scale = 1.0f / sqrtf(total / (float)width + p.eps);
-#pragma unroll
-            for (int j = 0; j < J; ++j)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) h[j][e] = fmaf(t[j][e] * scale, nw[j][e], h[j][e]);
+            for (int e = 0; e < 4; ++e) h[j][e] = fmaf(t[j][e] * scale, w[e] + p.weight_bias, h[j][e]);
         }
-        // a portion starts here: its past comes from the sequence's state
-        const bool starts = r == 0 || p.row_seq[r - 1] != seq;
-#pragma unroll
-        for (int j = 0; j < J; ++j) {
-            const int i = 4 * (tid + NT * j);
-            if (i >= width) continue;
-            if (p.store >= 0 && mine) jn_put4(p.results + p.store * p.result_step + (size_t)r * p.res_stride + i, h[j]);
-            if (p.avg) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) h[j][e] = fmaf(own_w, h[j][e], before[j][e]);
-            }
-            if (p.res_out && mine) jn_put4(p.res_out + (size_t)r * p.res_stride + i, h[j]);
-            if (p.copy_out && mine) jn_put4(static_cast<T*>(p.copy_out) + (size_t)r * p.copy_stride + i, h[j]);
-            if (!p.conv_out) continue;
-            if (starts)
-                for (int d = 1; d <= past; ++d) {
-                    const float* from = p.conv_ring + ((size_t)seq * past + (pos >= d ? (pos - d) % past : 0)) * width;
-                    float v[4];
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) v[e] = pos >= d && i + e < width ? from[i + e] : 0.f;
-                    jn_put4(hist + (size_t)(slot >= d ? slot - d : slot - d + past) * pitch + i, v);
-                }
-            float y[4];
-            const __nv_bfloat16* w = cw + i;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) y[e] = fmaf(__bfloat162float(w[(size_t)past * pitch + e]), h[j][e], h[j][e]);
-            for (int d = 1; d <= past; ++d) {
-                float v[4];
-                jn_get4(hist + (size_t)(slot >= d ? slot - d : slot - d + past) * pitch + i, v);
-#pragma unroll
-                for (int e = 0; e < 4; ++e) y[e] = fmaf(__bfloat162float(w[(size_t)(past - d) * pitch + e]), v[e], y[e]);
-            }
-            if (past) jn_put4(hist + (size_t)slot * pitch + i, h[j]);
-            if (mine) jn_put4(static_cast<T*>(p.conv_out) + (size_t)r * p.conv_stride + i, y);
-        }
-        if (++slot >= past) slot = 0;
+        if (p.store >= 0) jn_put4(p.results + p.store * p.result_step + (size_t)r * p.res_stride + i, h[j]);
+        if (p.avg) jn_average(p, r, i, h[j]);
+        if (p.res_out) jn_put4(p.res_out + (size_t)r * p.res_stride + i, h[j]);
+        if (p.copy_out) jn_put4(static_cast<T*>(p.copy_out) + (size_t)r * p.copy_stride + i, h[j]);
     }
 }
 
+// ---- portions: the convolution ----------------------------------------------------------------------------------------
+// CTA (128 quads of channels, kConvRows rows). `stream` are the rows the join left behind; TAPS 0: any number, rows read again.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kConvThreads) stream_conv_kernel(const JoinLaunch p, const float* stream) {
+    constexpr int PAST = TAPS > 1 ? TAPS - 1 : 1;
+    const int width = p.width, i = 4 * (blockIdx.x * kConvThreads + threadIdx.x), r0 = blockIdx.y * kConvRows, r1 = min(r0 + kConvRows, p.rows), past = p.taps - 1;
+    const bool live = i < width;
+    pdl_launch_dependents();
+    float w[TAPS > 0 ? TAPS : 1][4];
+    if (TAPS > 0 && live)
+#pragma unroll
+        for (int k = 0; k < (TAPS > 0 ? TAPS : 1); ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) w[k][e] = i + e < width ? __bfloat162float(p.conv_w[(size_t)(i + e) * TAPS + k]) : 0.f;
+    pdl_wait();
+    if (!live) return;
+    // the stream d tokens in front of row r
+    auto back = [&](int r, int d, float (&v)[4]) {
+        if (r - d >= 0 && p.row_seq[r - d] == p.row_seq[r]) { jn_get4(stream + (size_t)(r - d) * p.res_stride + i, v); return; }
+        const int at = p.row_pos[r] - d;
+        const float* from = p.conv_ring + ((size_t)p.row_seq[r] * past + (at >= 0 ? at % past : 0)) * width;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] = at >= 0 && i + e < width ? from[i + e] : 0.f;
+    };
+    float hist[PAST][4];   // hist[d - 1]: d tokens back
+    for (int r = r0; r < r1; ++r) {
+        float h[4], y[4];
+        jn_get4(stream + (size_t)r * p.res_stride + i, h);
+        if (TAPS > 0) {
+            if (TAPS > 1 && (r == r0 || p.row_seq[r - 1] != p.row_seq[r]))
+#pragma unroll
+                for (int d = 1; d <= PAST; ++d) back(r, d, hist[d - 1]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                y[e] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][e], h[e], h[e]);
+                if (TAPS > 1)
+#pragma unroll
+                    for (int d = 1; d <= PAST; ++d) y[e] = fmaf(w[TAPS > 1 ? TAPS - 1 - d : 0][e], hist[d - 1][e], y[e]);
+            }
+#pragma unroll
+            for (int d = PAST; d > 1; --d)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) hist[d - 1][e] = hist[d - 2][e];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) hist[0][e] = h[e];
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] = h[e];
+            for (int d = 0; d <= past; ++d) {
+                float v[4] = {h[0], h[1], h[2], h[3]};
+                if (d > 0) back(r, d, v);
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (i + e < width) y[e] = fmaf(__bfloat162float(p.conv_w[(size_t)(i + e) * p.taps + past - d]), v[e], y[e]);
+            }
+        }
+        jn_put4(static_cast<T*>(p.conv_out) + (size_t)r * p.conv_stride + i, y);
+    }
+}
+
+// ---- single tokens ----------------------------------------------------------------------------------------------------
+// Sums over the warp of 16 values a lane; the sum of value lane >> 1 is left in this lane.
+__device__ __forceinline__ float jn_sums16(float (&v)[16], int lane) {
+    int o = 16;
+#pragma unroll
+    for (int n = 8; n > 0; n >>= 1, o >>= 1) {
+        const bool upper = lane & o;
+#pragma unroll
+        for (int j = 0; j < n; ++j) {
+            const float give = upper ? v[j] : v[j + n], keep = upper ? v[j + n] : v[j];
+            v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+    return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+}
+// out[n] = W[n][0 .. 8 chunks) . x for n < rows, by the whole CTA; x and out in shared memory
+__device__ __forceinline__ void jn_rows(const __nv_bfloat16* w, int ld, int rows, int chunks, const float* x, float* out) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int n0 = warp * kSideRows; n0 < rows; n0 += kSideThreads / 32 * kSideRows) {
+        float acc[kSideRows];
+#pragma unroll
+        for (int q = 0; q < kSideRows; ++q) acc[q] = 0.f;
+        for (int c = lane; c < chunks; c += 32) {
+            uint4 v[kSideRows];
+#pragma unroll
+            for (int q = 0; q < kSideRows; ++q) v[q] = n0 + q < rows ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)(n0 + q) * ld) + c) : make_uint4(0, 0, 0, 0);
+            float f[8];
+            *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(x + 8 * c);
+            *reinterpret_cast<float4*>(f + 4) = *reinterpret_cast<const float4*>(x + 8 * c + 4);
+#pragma unroll
+            for (int q = 0; q < kSideRows; ++q) {
+                const unsigned b[4] = {v[q].x, v[q].y, v[q].z, v[q].w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    acc[q] = fmaf(__uint_as_float(b[e] << 16), f[2 * e], acc[q]);
+                    acc[q] = fmaf(__uint_as_float(b[e] & 0xFFFF0000u), f[2 * e + 1], acc[q]);
+                }
+            }
+        }
+        const float sum = jn_sums16(acc, lane);
+        if (!(lane & 1) && n0 + (lane >> 1) < rows) out[n0 + (lane >> 1)] = sum;
+    }
+}
+__device__ __forceinline__ float jn_rounded(float v, float) { return v; }
+__device__ __forceinline__ float jn_rounded(float v, __nv_bfloat16) { return __bfloat162float(__float2bfloat16_rn(v)); }
+
+// Cluster of CTAs per row, a thread per four columns. p: start, keep and first norm; f: what follows (SIDE: behind the token input,
+// whose result f's norm is for; else the same as p).
+template <typename T, bool SIDE, int NT>
+__global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, const TokenInput side, const JoinLaunch f) {
+    extern __shared__ __align__(16) float step_smem[];
+    __shared__ float red[NT / 32], ssq[2][kStepCluster];
+    const cg::cluster_group cluster = cg::this_cluster();
+    auto started = cluster.barrier_arrive();   // waited for before anything is written to another CTA's shared memory
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, nz = gridDim.x, rank = blockIdx.x, row = blockIdx.y, width = p.width;
+    const int chunks = (width + 7) / 8, share = (chunks + nz - 1) / nz, chunk0 = share * rank, own = max(0, min(share, chunks - chunk0));   // chunks of eight columns
+    const int i = 8 * chunk0 + 4 * tid;
+    const bool mine = 4 * tid < 8 * own, whole = (width & 3) == 0;
+    const int seq = p.row_seq[row], pos = p.row_pos[row], past = max(0, f.taps - 1);
+    // what does not depend on the kernels in front of this one: weights, and the convolution's past
+    float nw[4] = {}, fw[4] = {}, before[4] = {}, last[4] = {};
+    if (mine) {
+        if (p.in) jn_weights4(p.w, i, width, whole, nw);
+        if (SIDE) jn_weights4(f.w, i, width, whole, fw);
+        if (f.conv_out) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (i + e < width) {
+                    const __nv_bfloat16* w = f.conv_w + (size_t)(i + e) * f.taps;
+                    last[e] = __bfloat162float(w[past]);
+                    for (int d = 1; d <= past && d <= pos; ++d) before[e] = fmaf(__bfloat162float(w[past - d]), f.conv_ring[((size_t)seq * past + (pos - d) % past) * width + i + e], before[e]);
+                }
+        }
+    }
+    if (SIDE) {   // the token input's weights come closer
+        const int lines = (own + 7) / 8;   // of 128 bytes per row of this CTA's columns
+        for (int n = tid; n < side.n * lines; n += NT)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(side.gate + (size_t)(n / lines) * side.gate_ld + 8 * chunk0 + 64 * (n % lines)));
+        const int rows = min(8 * own, width - 8 * chunk0), all = (rows * side.proj_ld + 63) / 64;
+        for (int n = tid; n < all; n += NT) asm volatile("prefetch.global.L2 [%0];" ::"l"(side.proj + (size_t)8 * chunk0 * side.proj_ld + 64 * n));
+    }
+    pdl_wait();
+    float h[4] = {}, t[4] = {}, sum[4] = {};
+    if (mine) {
+        if (p.table) jn_weights4(p.table + (size_t)min(max(p.tokens[row], 0), p.vocab - 1) * width, i, width, whole, h);
+        else jn_get4(p.res_in + (size_t)row * p.res_stride + i, h);
+        if (p.in) jn_get4(p.in + (size_t)row * p.in_stride + i, t);
+        float gate[4];
+        if (p.gate) jn_get4(p.gate + (size_t)row * p.gate_stride + i, gate);
+        if (f.avg) jn_results(f, row, i, sum);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            if (p.table) h[e] *= p.table_scale;
+            if (p.gate) t[e] *= jn_sigmoid(gate[e]);
+            if (i + e >= width) h[e] = t[e] = 0.f;
+        }
+        if (p.keep_ring) {
+            float* keep = p.keep_ring + ((size_t)seq * (p.keep_taps - 1) + pos % (p.keep_taps - 1)) * width;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) if (i + e < width) keep[i + e] = h[e];
+        }
+    }
+    // 1 / root mean square over the row of what the threads hold; slot: 0 for the first norm, 1 for the second
+    auto over_rms = [&](const float (&v)[4], int slot, float eps) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss = fmaf(v[e], v[e], ss);
+        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
+        __syncthreads();
+        if (tid < nz) {
+            float total = 0.f;
+#pragma unroll
+            for (int q = 0; q < NT / 32; ++q) total += red[q];
+            cluster.map_shared_rank(ssq[slot], tid)[rank] = total;
+        }
+        cluster.sync();
+        float total = 0.f;
+        for (int q = 0; q < nz; ++q) total += ssq[slot][q];
+        return 1.0f / sqrtf(total / (float)width + eps);
+    };
+    cluster.barrier_wait(std::move(started));
+    if (p.in) {
+        const float scale = over_rms(t, 0, p.eps);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) h[e] = fmaf(t[e] * scale, nw[e] + p.weight_bias, h[e]);
+    }
+    if (SIDE) {
+        const int np = (side.n + 7) / 8 * 8;
+        float* xs = step_smem;             // [8 share] this CTA's columns of the stream, later of the result
+        float* part = xs + 8 * share;      // [np] this CTA's sums
+        float* all = part + np;            // [nz][np] everybody's
+        if (4 * tid < 8 * share)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) xs[4 * tid + e] = mine && i + e < width ? jn_rounded(h[e], T(0.f)) : 0.f;
+        __syncthreads();
+        jn_rows(side.gate + 8 * chunk0, side.gate_ld, side.n, own, xs, part);
+        __syncthreads();
+        for (int n = tid; n < side.n * nz; n += NT) cluster.map_shared_rank(all, n / side.n)[rank * np + n % side.n] = part[n % side.n];
+        cluster.sync();
+        const __nv_bfloat16* token = side.table + (size_t)min(max(p.tokens[row], 0), p.vocab - 1) * side.cols + side.col;
+        for (int n = tid; n < np; n += NT) {
+            float v = 0.f;
+            if (n < side.n) {
+                for (int q = 0; q < nz; ++q) v += all[q * np + n];
+                v = jn_rounded(gated_activation(jn_rounded(v, T(0.f)), __bfloat162float(token[n]), GATED_ACT_GELU_TANH), T(0.f));
+            }
+            part[n] = v;
+        }
+        __syncthreads();
+        jn_rows(side.proj + (size_t)8 * chunk0 * side.proj_ld, side.proj_ld, min(8 * own, width - 8 * chunk0), np / 8, part, xs);
+        __syncthreads();
+#pragma unroll
+        for (int e = 0; e < 4; ++e) t[e] = mine && i + e < width ? xs[4 * tid + e] : 0.f;
+        const float scale = over_rms(t, 1, f.eps);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) h[e] = fmaf(t[e] * scale, fw[e] + f.weight_bias, h[e]);
+    }
+    if (!mine) return;   // (nobody reaches into this CTA's shared memory any more)
+    if (f.store >= 0) jn_put4(f.results + f.store * f.result_step + (size_t)row * f.res_stride + i, h);
+    if (f.avg) {
+        const float w = __bfloat162float(f.avg_w[f.avg - 1]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) h[e] = fmaf(w, h[e], sum[e]);
+    }
+    if (f.res_out) jn_put4(f.res_out + (size_t)row * f.res_stride + i, h);
+    if (f.copy_out) jn_put4(static_cast<T*>(f.copy_out) + (size_t)row * f.copy_stride + i, h);
+    if (f.conv_out) {
+        float y[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] = h[e] + fmaf(last[e], h[e], before[e]);
+        jn_put4(static_cast<T*>(f.conv_out) + (size_t)row * f.conv_stride + i, y);
+    }
+}
+
+// ---- a gate out of a table --------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256) token_gate_kernel(int n, const T* in, int in_stride, const int32_t* tokens, int vocab, const __nv_bfloat16* table, int cols, int col,
                                                          T* out, int out_stride, int m) {
@@ -191,38 +384,75 @@ __global__ void __launch_bounds__(256) token_gate_kernel(int n, const T* in, int
     out[(size_t)r * out_stride + i] = (T)v;
 }
 
-size_t join_smem_bytes(int width, int taps) {
-    const size_t pitch = (width + 3) / 4 * 4;
-    return taps > 0 ? (size_t)(taps - 1) * pitch * 4 + (size_t)taps * pitch * 2 : 0;
-}
-
+// ---- launches ---------------------------------------------------------------------------------------------------------
 template <typename T, int J, int NT>
-int join_kernel(const JoinLaunch& a, int rows_per_cta, cudaStream_t s) {
-    static const cudaError_t attr = cudaFuncSetAttribute(stream_join_kernel<T, J, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kJoinMaxSmem);
-    if (attr != cudaSuccess) return cuda_fail(attr, "stream join attributes");
-    const cudaError_t e = launch_k(stream_join_kernel<T, J, NT>, dim3((a.rows + rows_per_cta - 1) / rows_per_cta), dim3(NT), join_smem_bytes(a.width, a.conv_out ? a.taps : 0), s, a, rows_per_cta);
-    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "stream join launch");
+cudaError_t join_launch(const JoinLaunch& a, cudaStream_t s) { return launch_k(stream_join_kernel<T, J, NT>, dim3(a.rows), dim3(NT), 0, s, a); }
+template <typename T, int TAPS>
+cudaError_t conv_launch(const JoinLaunch& a, cudaStream_t s) {
+    return launch_k(stream_conv_kernel<T, TAPS>, dim3((a.width + 4 * kConvThreads - 1) / (4 * kConvThreads), (a.rows + kConvRows - 1) / kConvRows), dim3(kConvThreads), 0, s, a,
+                    a.res_out ? (const float*)a.res_out : a.res_in);
 }
 template <typename T>
-int join_rows(const JoinLaunch& a, cudaStream_t s) {
-    // portions: a few rows per CTA, so that few are worked out twice
-    const int rows = a.singles || !a.conv_out || a.taps < 2 ? 1 : std::min(16, std::max(a.taps - 1, (a.rows + 3 * 148 - 1) / (3 * 148)));
-    if (a.width <= 4 * 128) return join_kernel<T, 1, 128>(a, rows, s);
-    if (a.width <= 4 * 256) return join_kernel<T, 1, 256>(a, rows, s);
-    if (a.width <= 4 * 512) return join_kernel<T, 2, 256>(a, rows, s);
-    if (a.width <= 4 * 1024) return join_kernel<T, 2, 512>(a, rows, s);
-    return join_kernel<T, 8, 512>(a, rows, s);
+int portions(const JoinLaunch& a, cudaStream_t s, int* launches) {
+    cudaError_t e = cudaSuccess;
+    if (a.res_out || a.copy_out || a.keep_ring) {
+        e = a.width <= 4 * 128 ? join_launch<T, 1, 128>(a, s) : a.width <= 4 * 256 ? join_launch<T, 1, 256>(a, s) : a.width <= 4 * 512 ? join_launch<T, 2, 256>(a, s)
+            : a.width <= 4 * 1024 ? join_launch<T, 2, 512>(a, s) : join_launch<T, 8, 512>(a, s);
+        *launches += 1;
+    }
+    if (e == cudaSuccess && a.conv_out) {
+        e = a.taps == 1 ? conv_launch<T, 1>(a, s) : a.taps == 2 ? conv_launch<T, 2>(a, s) : a.taps == 3 ? conv_launch<T, 3>(a, s) : a.taps == 4 ? conv_launch<T, 4>(a, s) : conv_launch<T, 0>(a, s);
+        *launches += 1;
+    }
+    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "stream join launch");
 }
+
+size_t side_smem(const TokenInput& t, int width, int nz) {
+    const size_t np = (t.n + 7) / 8 * 8, share = ((width + 7) / 8 + nz - 1) / nz;
+    return (8 * share + np * (nz + 1)) * 4;
+}
+template <typename T, bool SIDE, int NT>
+int step_launch(const JoinLaunch& p, const TokenInput& side, const JoinLaunch& f, int nz, cudaStream_t s) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(nz, p.rows); cfg.blockDim = dim3(NT); cfg.stream = s;
+    cfg.dynamicSmemBytes = SIDE ? side_smem(side, p.width, nz) : 0;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = nz; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl_enabled() ? 2 : 1;
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, stream_step_kernel<T, SIDE, NT>, p, side, f);
+    return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "stream step launch");
+}
+constexpr int kStepThreads = 128;
+constexpr size_t kSideMaxSmem = 40 * 1024;
+bool step_fits(int width) { return width <= 4 * kSideThreads * kStepCluster; }
 
 }  // namespace
 
-int join_init() { return SWLM_OK; }
-bool join_supported(int width, int taps) { return width > 0 && width <= 4 * 512 * 8 && taps >= 0 && join_smem_bytes(width, taps) <= kJoinMaxSmem; }
+bool join_supported(int width, int taps) { return width > 0 && width <= 4 * 512 * 8 && taps >= 0; }
 
-int launch_join(const JoinLaunch& a, cudaStream_t s) {
+int launch_join(const JoinLaunch& a, cudaStream_t s, int* launches) {
     if (a.rows <= 0) return SWLM_OK;
-    if (!join_supported(a.width, a.conv_out ? a.taps : 0)) { set_error("stream of %d entries with convolutions of %d taps", a.width, a.taps); return SWLM_ERR_UNSUPPORTED; }
-    return a.f32 ? join_rows<float>(a, s) : join_rows<__nv_bfloat16>(a, s);
+    if (!join_supported(a.width, a.taps)) { set_error("stream of %d entries with convolutions of %d taps", a.width, a.taps); return SWLM_ERR_UNSUPPORTED; }
+    if (a.singles && step_fits(a.width)) {
+        *launches += 1;
+        int nz = 1;
+        while (nz < kStepCluster && nz * 4 * kStepThreads < a.width) nz <<= 1;
+        const TokenInput none;
+        if (nz * 4 * kStepThreads >= a.width) return a.f32 ? step_launch<float, false, kStepThreads>(a, none, a, nz, s) : step_launch<__nv_bfloat16, false, kStepThreads>(a, none, a, nz, s);
+        return a.f32 ? step_launch<float, false, kSideThreads>(a, none, a, nz, s) : step_launch<__nv_bfloat16, false, kSideThreads>(a, none, a, nz, s);
+    }
+    return a.f32 ? portions<float>(a, s, launches) : portions<__nv_bfloat16>(a, s, launches);
+}
+
+bool token_input_fits(const TokenInput& t, int rows, int width) { return rows <= kStepMaxRows && step_fits(width) && side_smem(t, width, kStepCluster) <= kSideMaxSmem; }
+int launch_token_input(const JoinLaunch& first, const TokenInput& t, const JoinLaunch& last, cudaStream_t s) {
+    if (first.rows <= 0) return SWLM_OK;
+    if (!token_input_fits(t, first.rows, first.width)) { set_error("token input of %d entries into %d x %d", t.n, first.rows, first.width); return SWLM_ERR_UNSUPPORTED; }
+    return first.f32 ? step_launch<float, true, kSideThreads>(first, t, last, kStepCluster, s) : step_launch<__nv_bfloat16, true, kSideThreads>(first, t, last, kStepCluster, s);
 }
 
 int launch_token_gate(int m, int n, const void* in, int in_stride, const int32_t* tokens, int vocab, const __nv_bfloat16* table, int cols, int col, void* out,

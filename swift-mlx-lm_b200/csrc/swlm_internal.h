@@ -465,7 +465,7 @@ constexpr int kLatentQueryTile = 128;
 int launch_latent(const LatentLaunch& a, cudaStream_t s, int* launches);
 
 // ---- the residual stream between sublayers (stream_join.cu) ------------------------------------------------------------
-// One launch over the rows of a batch; parts that are not set are left out:
+// Parts that are not set are left out:
 //   x = table[token] * table_scale, or res_in
 //   keep_ring: x of a portion's last rows goes to the state of the convolution that read it
 //   x += norm(in * sigmoid(gate); w)
@@ -486,9 +486,17 @@ struct JoinLaunch {
     const __nv_bfloat16* conv_w = nullptr; const float* conv_ring = nullptr; int taps = 0; void* conv_out = nullptr; int conv_stride = 0;   // conv_w [width][taps]
     void* copy_out = nullptr; int copy_stride = 0;
 };
-int join_init();
 bool join_supported(int width, int taps);
-int launch_join(const JoinLaunch& a, cudaStream_t s);
+int launch_join(const JoinLaunch& a, cudaStream_t s, int* launches);
+// A token's own input to a layer, for single tokens: y = proj (gelu_tanh(gate x) * table[token][col ..]) between two joins that do
+// nothing else with what lies between them: `first` ends with x, `last` starts with it and adds norm(y).
+struct TokenInput {
+    int n = 0;
+    const __nv_bfloat16 *gate = nullptr, *proj = nullptr; int gate_ld = 0, proj_ld = 0;   // [n][width], [width][n]
+    const __nv_bfloat16* table = nullptr; int cols = 0, col = 0;
+};
+bool token_input_fits(const TokenInput& t, int rows, int width);
+int launch_token_input(const JoinLaunch& first, const TokenInput& t, const JoinLaunch& last, cudaStream_t s);
 // out = gelu_tanh(in) * table[token][col ..]
 int launch_token_gate(int m, int n, const void* in, int in_stride, const int32_t* tokens, int vocab, const __nv_bfloat16* table, int cols, int col, void* out,
                       int out_stride, bool f32, cudaStream_t s);

@@ -73,6 +73,7 @@ struct Launch {
     Matrix part[2];                           // products of two inputs: the rows that meet the first and the second one
     int x2_buf = -1, first_segs = 0;          // the second input, and how many results belong to the first
     JoinParts join;
+    int fused = 0;                            // single tokens: this many launches behind this one are part of it (a token input)
     const DenseTensor* dv[6] = {};            // gated delta rule: taps of q, k, v, norm weight, A_log, dt_bias; latent attention: [0] sink; norms: [0] table that joins
     int window_set = 0;                       // latent attention: index into plan->windows
     const DenseTensor* norm_post = nullptr;   // norm steps: weight of the norm applied to the input before it is added
