@@ -6,7 +6,9 @@
 // cache; then a batch's rows go one of two ways:
 //   * one by one (decode steps, short portions): grouped_decode_kernel, a cluster of CTAs per (row, key / value head) that deal the
 //     context out to their warps; every warp copies its keys and values by itself and keeps its own running softmax, the
-//     results are merged through shared memory and then through distributed shared memory.
+//     results are merged through shared memory and then through distributed shared memory. Where every row is a token of its own
+//     and nothing is rotated, the kernel norms and appends by itself: the cached rows in front of the token are requested before
+//     the preceding kernel has finished, the token's own key does not go through the cache.
 //   * in spans (prompt portions): grouped_prefill_kernel, a tiled attention of 128 queries by 64 keys.
 // Both multiply on tensor cores with fp32 sums; softmax weights enter as bf16 hi + lo pairs. grouped_simple_kernel (fp32 FMAs)
 // serves fp32 caches and head sizes beyond the others. The newest rows are read back from the cache like all others, so a row's
@@ -17,6 +19,7 @@
 #include <cooperative_groups.h>
 
 #include <algorithm>
+#include <utility>
 
 #include "swlm_internal.h"
 #include "tc_device.cuh"
@@ -87,6 +90,13 @@ __device__ __forceinline__ float* ga_factors(const GroupedParams& p, const T* bl
 template <typename T>
 __device__ __forceinline__ float ga_entry_gate(const GroupedParams& p, int r, int h, int c) {
     return 1.0f / (1.0f + expf(-ga_get(static_cast<const T*>(p.entry_gate) + (size_t)r * p.entry_gate_stride + (size_t)h * p.row.vdim + c)));
+}
+// a sigmoid by the hardware's approximations (an fp32 number, a few units in the last place off)
+__device__ __forceinline__ float ga_sigmoid(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+// two neighbours, bf16
+__device__ __forceinline__ float2 ga_entry_gates(const GroupedParams& p, int r, int h, int c) {
+    const unsigned v = __ldcg(reinterpret_cast<const unsigned*>(static_cast<const __nv_bfloat16*>(p.entry_gate) + (size_t)r * p.entry_gate_stride + (size_t)h * p.row.vdim + c));
+    return make_float2(ga_sigmoid(__uint_as_float(v << 16)), ga_sigmoid(__uint_as_float(v & 0xFFFF0000u)));
 }
 __device__ __forceinline__ float ga_gate(const GroupedParams& p, int r, int h) {
     return (p.gate ? 1.0f / (1.0f + expf(-p.gate[(size_t)r * p.gate_stride + h])) : 1.0f) * p.out_scale;
@@ -193,27 +203,34 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) grouped_simple_kernel(const
 // ---- rows one by one, tensor cores ------------------------------------------------------------------------------------
 // Cluster of CTAs per (row, key / value head, 16 query heads of it): the context in units of UK keys, dealt out to all warps of the
 // cluster. A unit is two bulk copies (keys, values) into the warp's own stage.
+constexpr int kDecStages = 2;   // units under way per warp, as far as shared memory goes
 constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kDecHeads = 16, kDecCluster = 8;
-template <int KQ, int NV, int UK>   // 16-column steps of query / key and value rows, keys of a unit
-__global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const GroupedParams p) {
+template <int KQ, int NV, int UK, bool APPENDS>   // 16-column steps of query / key and value rows, keys of a unit; norm and append in here
+__global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const GroupedParams p, int stages, int recv_at) {
     extern __shared__ __align__(128) unsigned char dec_smem[];
-    __shared__ __align__(8) unsigned long long bar[kDecWarps];
-    __shared__ float warp_m[kDecWarps][kDecHeads], warp_l[kDecWarps][kDecHeads], cta_m[kDecHeads], cta_l[kDecHeads], all_m[kDecCluster][kDecHeads], all_l[kDecCluster][kDecHeads];
+    __shared__ __align__(8) unsigned long long bar[kDecWarps][kDecStages];
+    constexpr int QP = 16 * KQ + 8;
+    __shared__ __align__(16) __nv_bfloat16 q_s[APPENDS ? kDecHeads * QP : 1], k_s[APPENDS ? 16 * KQ : 1], v_s[APPENDS ? 16 * NV : 1];
+    __shared__ float own_factor;
+    __shared__ float warp_m[kDecWarps][kDecHeads], warp_l[kDecWarps][kDecHeads], all_m[kDecCluster][kDecHeads], all_l[kDecCluster][kDecHeads];
     const cg::cluster_group cluster = cg::this_cluster();
+    auto started = cluster.barrier_arrive();   // waited for before anything is written to another CTA's shared memory
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int nz = gridDim.x, rank = blockIdx.x, kv = blockIdx.y / ((p.share + kDecHeads - 1) / kDecHeads), tile = blockIdx.y % ((p.share + kDecHeads - 1) / kDecHeads);
     const int h0 = kv * p.share + tile * kDecHeads, nh = min(kDecHeads, p.share - tile * kDecHeads);   // query heads of this CTA
     pdl_launch_dependents();
-    if (tid < kDecWarps) mbar_init(&bar[tid], 1);
+    if (tid < kDecWarps * kDecStages) mbar_init(&bar[0][0] + tid, 1);
     if (tid == 0) asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     __syncthreads();
-    pdl_wait();
+    if (!APPENDS) pdl_wait();   // (otherwise what is read first was there before this step)
     const int r = ga_row(p, blockIdx.z), pos = p.row_pos[r], seq = p.row_seq[r];
-    const int seen0 = ga_first_seen(p, pos), unit0 = seen0 / UK, units = pos / UK + 1 - unit0;
+    const int past_end = APPENDS ? pos : pos + 1;   // first position whose row is not read from the cache
+    const int seen0 = ga_first_seen(p, pos), unit0 = seen0 / UK, units = past_end > seen0 ? (past_end - 1) / UK + 1 - unit0 : 0;
     const int pk = p.row.pk, pv = p.row.pv, k_bytes = UK * pk * 2, v_bytes = p.row.shared ? UK * 4 : UK * pv * 2;   // (shared rows: their factors instead of values)
-    unsigned char* stage = dec_smem + (size_t)warp * (k_bytes + v_bytes);
-    const unsigned bar_at = smem_u32(&bar[warp]);
-    auto request = [&](int u) {   // lane 0
+    unsigned char* stage0 = dec_smem + (size_t)warp * stages * (k_bytes + v_bytes);
+    auto request = [&](int u, int st) {   // lane 0
+        const unsigned bar_at = smem_u32(&bar[warp][st]);
+        unsigned char* stage = stage0 + (size_t)st * (k_bytes + v_bytes);
         const int key0 = (unit0 + u) * UK;
         const __nv_bfloat16* block = ga_block<__nv_bfloat16>(p, seq, key0 / kPage, kv);
         mbar_expect(bar_at, (unsigned)(k_bytes + v_bytes));
@@ -221,44 +238,109 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
         bulk_load(smem_u32(stage) + (unsigned)k_bytes, block + (size_t)kPage * pk + (size_t)(key0 % kPage) * (p.row.shared ? 2 : pv), (unsigned)v_bytes, bar_at);
     };
     const int first = rank * kDecWarps + warp, step = nz * kDecWarps;
-    if (lane == 0 && first < units) request(first);
-    const float gate = tid < nh ? ga_gate(p, r, h0 + tid) : 0.f;
+    if (lane == 0) for (int st = 0; st < stages && first + st * step < units; ++st) request(first + st * step, st);
+    const bool keeps = APPENDS && rank == 0 && tile == 0;   // puts the token's row into the cache
+    __nv_bfloat16* own_block = keeps ? ga_block<__nv_bfloat16>(p, seq, pos / kPage, kv) : nullptr;
+    const float temperature = APPENDS && p.temp_every > 0 ? 1.0f + p.temp_coef * logf((float)((pos + 1) / p.temp_every) + 1.0f) : 1.0f;
+    if (APPENDS) pdl_wait();
+    const float gate = tid >> 3 < nh ? ga_gate(p, r, h0 + (tid >> 3)) : 0.f;   // of the head whose results this thread merges
     // query fragments: rows g and g + 8
     const int ksteps = p.row.dp >> 4, n_vt = p.row.vp >> 4;
-    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)r * p.qkv_stride + (size_t)h0 * p.row.dim;
+    const __nv_bfloat16* qkv = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)r * p.qkv_stride;
+    const __nv_bfloat16* q = qkv + (size_t)h0 * p.row.dim;
+    if (APPENDS) {
+        // a warp per vector: the queries of this CTA, then the key; the value is copied
+        const int dim = p.row.dim, vdim = p.row.vdim;
+        for (int i = warp; i <= nh; i += kDecWarps) {
+            const bool is_key = i == nh;
+            const __nv_bfloat16* src = is_key ? qkv + (size_t)(p.heads + kv) * dim : q + (size_t)i * dim;
+            __nv_bfloat16* dst = is_key ? k_s : q_s + (size_t)i * QP;
+            float x[KQ / 2];
+            float ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < KQ / 2; ++j) { const int c = lane + 32 * j; x[j] = c < dim ? ga_get(src + c) : 0.f; ss = fmaf(x[j], x[j], ss); }
+            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const __nv_bfloat16* w = is_key ? p.k_norm : p.q_norm;
+            float f = p.head_norm || w ? 1.0f / sqrtf(ss / (float)dim + p.eps) : 1.0f;
+            if (is_key && p.row.shared) {
+                if (lane == 0) own_factor = f;
+                f = 1.0f;
+            }
+            if (!is_key) f *= temperature;
+#pragma unroll
+            for (int j = 0; j < KQ / 2; ++j) {
+                const int c = lane + 32 * j;
+                if (c < 16 * KQ) ga_put(dst + c, c < dim ? x[j] * f * (w ? __bfloat162float(w[c]) + p.weight_bias : 1.0f) : 0.f);
+            }
+        }
+        const __nv_bfloat16* v = qkv + (size_t)(p.heads + p.row.groups) * dim + (size_t)kv * vdim;
+        if (!p.row.shared) for (int c = tid; c < 16 * NV; c += kDecThreads) v_s[c] = c < vdim ? v[c] : __float2bfloat16_rn(0.f);
+        __syncthreads();
+        if (keeps) {   // for the tokens to come
+            for (int c = tid; c < dim; c += kDecThreads) own_block[(size_t)(pos % kPage) * pk + c] = k_s[c];
+            if (p.row.shared) { if (tid == 0) ga_factors(p, own_block)[pos % kPage] = own_factor; }
+            else for (int c = tid; c < vdim; c += kDecThreads) own_block[(size_t)kPage * pk + (size_t)(pos % kPage) * pv + c] = v_s[c];
+        }
+    }
+    const __nv_bfloat16* own_v = APPENDS && p.row.shared ? k_s : v_s;
     unsigned qa[KQ][4];
 #pragma unroll
     for (int k = 0; k < KQ; ++k)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int hh = g + 8 * (e & 1), c = 16 * k + 8 * (e >> 1) + 2 * t;
-            qa[k][e] = hh < nh && c < p.row.dim ? __ldcg(reinterpret_cast<const unsigned*>(q + (size_t)hh * p.row.dim + c)) : 0u;
+            if (APPENDS) qa[k][e] = hh < nh ? *reinterpret_cast<const unsigned*>(q_s + (size_t)hh * QP + c) : 0u;
+            else qa[k][e] = hh < nh && c < p.row.dim ? __ldcg(reinterpret_cast<const unsigned*>(q + (size_t)hh * p.row.dim + c)) : 0u;
         }
     float oacc[2 * NV][4];
 #pragma unroll
     for (int j = 0; j < 2 * NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-    const unsigned ks = smem_u32(stage), vs = p.row.shared ? ks : ks + (unsigned)k_bytes;
-    const float* factors = reinterpret_cast<const float*>(stage + k_bytes);
+    if (APPENDS && rank == 0 && warp == 0) {   // the token's own key: the first column of a tile whose others are zero
+        float own[4] = {0.f, 0.f, 0.f, 0.f}, odd[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int k = 0; k < KQ; ++k) {
+            const unsigned b0 = g == 0 ? *reinterpret_cast<const unsigned*>(k_s + 16 * k + 2 * t) : 0u, b1 = g == 0 ? *reinterpret_cast<const unsigned*>(k_s + 16 * k + 8 + 2 * t) : 0u;
+            ga_mma(k & 1 ? odd : own, qa[k], b0, b1);
+        }
+        const float f = p.row.shared ? p.scale_log2 * own_factor : p.scale_log2;
+        m_a = f * __shfl_sync(0xffffffffu, own[0] + odd[0], lane & ~3);
+        m_b = f * __shfl_sync(0xffffffffu, own[2] + odd[2], lane & ~3);
+        l_a = l_b = t == 0 ? 1.f : 0.f;
+#pragma unroll
+        for (int j = 0; j < 2 * NV; ++j) {
+            oacc[j][0] = oacc[j][2] = __bfloat162float(own_v[8 * j + 2 * t]);
+            oacc[j][1] = oacc[j][3] = __bfloat162float(own_v[8 * j + 2 * t + 1]);
+        }
+    }
+    int at = 0;
     unsigned phase = 0;
-    for (int u = first; u < units; u += step, phase ^= 1) {
-        if (!mbar_wait(&bar[warp], phase)) {
+    for (int u = first; u < units; u += step) {
+        const unsigned ks = smem_u32(stage0) + (unsigned)(at * (k_bytes + v_bytes)), vs = p.row.shared ? ks : ks + (unsigned)k_bytes;
+        const float* factors = reinterpret_cast<const float*>(stage0 + (size_t)at * (k_bytes + v_bytes) + k_bytes);
+        if (!mbar_wait(&bar[warp][at], phase)) {
             if (lane == 0) atomicExch(p.status, 61);
-            mbar_wait(&bar[warp], phase);   // leave the loop only when the copy has landed (bounded)
+            // leave the loop only when the copies under way have landed (bounded)
+            for (int st = 0; st < stages && u + st * step < units; ++st) mbar_wait(&bar[warp][(at + st) % stages], phase ^ (unsigned)(at + st >= stages));
             break;
         }
         float sacc[UK / 8][4];
 #pragma unroll
         for (int j = 0; j < UK / 8; ++j) sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f;
+        unsigned kf[2][UK / 16][4];   // the next fragments are on their way while these multiply
+        auto keys = [&](int k) {
+#pragma unroll
+            for (int jp = 0; jp < UK / 16; ++jp) ga_ldsm(kf[k & 1][jp], ks + (unsigned)((jp * 16 + (lane & 7) + 8 * (lane >> 4)) * pk + 16 * k + 8 * ((lane >> 3) & 1)) * 2u);
+        };
+        keys(0);
 #pragma unroll
         for (int k = 0; k < KQ; ++k)
             if (k < ksteps) {
+                if (k + 1 < KQ && k + 1 < ksteps) keys(k + 1);
 #pragma unroll
                 for (int jp = 0; jp < UK / 16; ++jp) {
-                    unsigned b[4];
-                    ga_ldsm(b, ks + (unsigned)((jp * 16 + (lane & 7) + 8 * (lane >> 4)) * pk + 16 * k + 8 * ((lane >> 3) & 1)) * 2u);
-                    ga_mma(sacc[2 * jp], qa[k], b[0], b[1]);
-                    ga_mma(sacc[2 * jp + 1], qa[k], b[2], b[3]);
+                    ga_mma(sacc[2 * jp], qa[k], kf[k & 1][jp][0], kf[k & 1][jp][1]);
+                    ga_mma(sacc[2 * jp + 1], qa[k], kf[k & 1][jp][2], kf[k & 1][jp][3]);
                 }
             }
         const int key0 = (unit0 + u) * UK;
@@ -268,7 +350,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = key0 + 8 * j + 2 * t + e;
-                const bool seen = key <= pos && key >= seen0;
+                const bool seen = key < past_end && key >= seen0;
                 const float f = p.row.shared ? p.scale_log2 * factors[8 * j + 2 * t + e] : p.scale_log2;
                 sacc[j][e] = seen ? sacc[j][e] * f : -INFINITY;
                 sacc[j][2 + e] = seen ? sacc[j][2 + e] * f : -INFINITY;
@@ -300,28 +382,31 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
                 ah[e] = ga_pack(xh, yh);
                 al[e] = ga_pack(x - xh, y - yh);
             }
+            unsigned vf[2][4];
+            auto values = [&](int j) { ga_ldsm_trans(vf[j & 1], vs + (unsigned)((16 * kk + (lane & 7) + 8 * ((lane >> 3) & 1)) * pv + 16 * j + 8 * (lane >> 4)) * 2u); };
+            values(0);
 #pragma unroll
             for (int j = 0; j < NV; ++j)
                 if (j < n_vt) {
-                    unsigned b[4];
-                    ga_ldsm_trans(b, vs + (unsigned)((16 * kk + (lane & 7) + 8 * ((lane >> 3) & 1)) * pv + 16 * j + 8 * (lane >> 4)) * 2u);
-                    ga_mma(oacc[2 * j], ah, b[0], b[1]);
-                    ga_mma(oacc[2 * j], al, b[0], b[1]);
-                    ga_mma(oacc[2 * j + 1], ah, b[2], b[3]);
-                    ga_mma(oacc[2 * j + 1], al, b[2], b[3]);
+                    if (j + 1 < NV && j + 1 < n_vt) values(j + 1);
+                    ga_mma(oacc[2 * j], ah, vf[j & 1][0], vf[j & 1][1]);
+                    ga_mma(oacc[2 * j + 1], ah, vf[j & 1][2], vf[j & 1][3]);
+                    ga_mma(oacc[2 * j], al, vf[j & 1][0], vf[j & 1][1]);
+                    ga_mma(oacc[2 * j + 1], al, vf[j & 1][2], vf[j & 1][3]);
                 }
         }
         __syncwarp();   // the stage is free
-        if (lane == 0 && u + step < units) request(u + step);
+        if (lane == 0 && u + stages * step < units) request(u + stages * step, at);
+        if (++at == stages) { at = 0; phase ^= 1; }
     }
 #pragma unroll
     for (int o = 1; o < 4; o <<= 1) { l_a += __shfl_xor_sync(0xffffffffu, l_a, o); l_b += __shfl_xor_sync(0xffffffffu, l_b, o); }
     if (t == 0) { warp_m[warp][g] = m_a; warp_m[warp][g + 8] = m_b; warp_l[warp][g] = l_a; warp_l[warp][g + 8] = l_b; }
     __syncthreads();
-    // the stages now hold the warps' sums: [warps][heads of this CTA][vp], behind them the CTA's own [heads][vp]
-    const int vp = p.row.vp;
+    // the stages now hold the warps' sums: [warps][heads of this CTA][vp]
+    const int vp = p.row.vp, share = (nh * vp + nz - 1) / nz;   // entries of the result that a CTA of the cluster finishes
     float* sums = reinterpret_cast<float*>(dec_smem);
-    float* own = sums + (size_t)kDecWarps * nh * vp;
+    float* recv = reinterpret_cast<float*>(dec_smem + recv_at);   // [nz][share], written by the other CTAs
 #pragma unroll
     for (int j = 0; j < 2 * NV; ++j) {
         const int c = 8 * j + 2 * t;
@@ -330,60 +415,68 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
             if (g + 8 < nh) *reinterpret_cast<float2*>(sums + ((size_t)warp * nh + g + 8) * vp + c) = make_float2(oacc[j][2], oacc[j][3]);
         }
     }
-    if (tid < nh) {
-        float top = -INFINITY, total = 0.f;
-        for (int w = 0; w < kDecWarps; ++w) top = fmaxf(top, warp_m[w][tid]);
-        for (int w = 0; w < kDecWarps; ++w) {
-            const float f = warp_m[w][tid] == -INFINITY ? 0.f : exp2f(warp_m[w][tid] - top);
-            total += f * warp_l[w][tid];
-            warp_l[w][tid] = f;
+    // the gate of the first entry this thread finishes is on its way during the merge
+    const __nv_bfloat16* egate = static_cast<const __nv_bfloat16*>(p.entry_gate) + (size_t)r * p.entry_gate_stride + (size_t)h0 * p.row.vdim;
+    float entry = 1.f;
+    if (p.entry_gate && tid < share && rank * share + tid < nh * vp && (rank * share + tid) % vp < p.row.vdim)
+        entry = ga_sigmoid(__bfloat162float(egate[(size_t)((rank * share + tid) / vp) * p.row.vdim + (rank * share + tid) % vp]));
+    cluster.barrier_wait(std::move(started));
+    static_assert(kDecWarps == 8 && kDecCluster == 8, "eight lanes per head");
+    auto over8 = [](float& top, float& total, float m, float l) {   // maximum and rescaled sum over eight lanes; this lane's factor
+        top = m;
+#pragma unroll
+        for (int o = 1; o < 8; o <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+        const float f = m == -INFINITY ? 0.f : exp2f(m - top);
+        total = f * l;
+#pragma unroll
+        for (int o = 1; o < 8; o <<= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
+        return f;
+    };
+    const int eighth = tid & 7, of_head = tid >> 3;   // (16 heads: the first four warps)
+    if (warp < kDecHeads / 4) {
+        float top, total;
+        const float f = over8(top, total, warp_m[eighth][of_head], warp_l[eighth][of_head]);
+        warp_l[eighth][of_head] = f;
+        if (eighth < nz) {
+            cluster.map_shared_rank(all_m[rank], eighth)[of_head] = top;
+            cluster.map_shared_rank(all_l[rank], eighth)[of_head] = total;
         }
-        cta_m[tid] = top;
-        cta_l[tid] = total;
     }
     __syncthreads();
     for (int i = tid; i < nh * vp; i += kDecThreads) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < kDecWarps; ++w) v = fmaf(warp_l[w][i / vp], sums[(size_t)w * nh * vp + i], v);
-        own[i] = v;
+        const int z = i / share;
+        cluster.map_shared_rank(recv, z)[rank * share + i - z * share] = v;
     }
-    cluster.sync();
-    // every CTA's maximum and sum, then its share of every head's result
-    if (tid < nz * nh) {
-        const int z = tid / nh, hh = tid - z * nh;
-        all_m[z][hh] = cluster.map_shared_rank(cta_m, z)[hh];
-        all_l[z][hh] = cluster.map_shared_rank(cta_l, z)[hh];
-    }
-    __syncthreads();
-    if (tid < nh) {
-        float top = p.sink_one ? 0.f : -INFINITY;
-        for (int z = 0; z < nz; ++z) top = fmaxf(top, all_m[z][tid]);
-        float total = p.sink_one ? exp2f(-top) : 0.f;
-        for (int z = 0; z < nz; ++z) {
-            const float f = all_m[z][tid] == -INFINITY ? 0.f : exp2f(all_m[z][tid] - top);
-            total = fmaf(f, all_l[z][tid], total);
-            all_m[z][tid] = f;
+    cluster.sync();   // (nobody reaches into another CTA's shared memory behind this)
+    if (warp < kDecHeads / 4) {
+        const bool there = eighth < nz;
+        float top, total;
+        float f = over8(top, total, there ? all_m[eighth][of_head] : -INFINITY, there ? all_l[eighth][of_head] : 0.f);
+        if (p.sink_one) {   // one joins the sum
+            const float scale = top > 0.f ? 1.f : exp2f(top);
+            f *= scale;
+            total = total * scale + exp2f(-fmaxf(top, 0.f));
         }
-        const float f = gate / total;
-        for (int z = 0; z < kDecCluster; ++z) all_m[z][tid] = z < nz ? all_m[z][tid] * f : 0.f;
+        all_m[eighth][of_head] = f * gate / total;
     }
     __syncthreads();
-    for (int i = rank * kDecThreads + tid; i < nh * vp; i += nz * kDecThreads) {
-        const int hh = i / vp, c = i - hh * vp;
+    for (int q = tid; q < share && rank * share + q < nh * vp; q += kDecThreads) {
+        const int i = rank * share + q, hh = i / vp, c = i - hh * vp;
+        if (c >= p.row.vdim) continue;
         float v = 0.f;
-#pragma unroll
-        for (int z = 0; z < kDecCluster; ++z) v = fmaf(all_m[z][hh], cluster.map_shared_rank(own, z < nz ? z : rank)[i], v);
-        if (c < p.row.vdim && p.entry_gate) v *= ga_entry_gate<__nv_bfloat16>(p, r, h0 + hh, c);
-        if (c < p.row.vdim) static_cast<__nv_bfloat16*>(p.out)[(size_t)r * p.out_stride + (size_t)(h0 + hh) * p.row.vdim + c] = __float2bfloat16_rn(v);
+        for (int z = 0; z < nz; ++z) v = fmaf(all_m[z][hh], recv[z * share + q], v);
+        if (p.entry_gate) v *= q == tid ? entry : ga_sigmoid(__bfloat162float(egate[(size_t)hh * p.row.vdim + c]));
+        static_cast<__nv_bfloat16*>(p.out)[(size_t)r * p.out_stride + (size_t)(h0 + hh) * p.row.vdim + c] = __float2bfloat16_rn(v);
     }
-    cluster.sync();   // nobody leaves while others still read
 }
 
 // ---- spans ------------------------------------------------------------------------------------------------------------
 // CTA (tile of 128 query rows of a span, head), 8 warps of 16 query rows; a key tile is a page, one bulk copy of keys and values.
 constexpr int kPfThreads = 256, kPfStages = 3;
-template <int KQ, int NV>
+template <int KQ, int NV, bool SHARED>
 __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const GroupedParams p) {
     extern __shared__ __align__(128) unsigned char pf_smem[];
     __shared__ __align__(8) unsigned long long full_bar[kPfStages];
@@ -430,7 +523,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const Gr
     for (; i < n_tiles; ++i) {
         if (!mbar_wait(&full_bar[i % kPfStages], (unsigned)((i / kPfStages) & 1))) { atomicExch(p.status, 62); bad = 1; }
         const int key0 = (kt0 + i) * kPage;
-        const unsigned kb = smem_u32(pf_smem) + (unsigned)(i % kPfStages * stage_bytes), vb = p.row.shared ? kb : kb + (unsigned)(kPage * pk) * 2u;
+        const unsigned kb = smem_u32(pf_smem) + (unsigned)(i % kPfStages * stage_bytes), vb = SHARED ? kb : kb + (unsigned)(kPage * pk) * 2u;
         const float* factors = reinterpret_cast<const float*>(pf_smem + (size_t)(i % kPfStages) * stage_bytes + (size_t)kPage * pk * 2);
         if (warp_first <= last_pos && key0 <= warp_last && key0 + kPage > warp_seen) {
             float sacc[8][4];
@@ -450,16 +543,19 @@ __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const Gr
             const bool edge = key0 + kPage - 1 > warp_first || key0 < full_from;   // some row does not see the whole tile
             float mx_a = -INFINITY, mx_b = -INFINITY;
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
+            for (int j = 0; j < 8; ++j) {
+                float2 ff = make_float2(p.scale_log2, p.scale_log2);
+                if (SHARED) { const float2 v = *reinterpret_cast<const float2*>(factors + 8 * j + 2 * t); ff.x *= v.x; ff.y *= v.y; }
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = key0 + 8 * j + 2 * t + e;
-                    const float f = p.row.shared ? p.scale_log2 * factors[8 * j + 2 * t + e] : p.scale_log2;
+                    const float f = e ? ff.y : ff.x;
                     const float a = !edge || (key <= pos_a && key >= seen_a) ? sacc[j][e] * f : -INFINITY;
                     const float b = !edge || (key <= pos_b && key >= seen_b) ? sacc[j][2 + e] * f : -INFINITY;
                     sacc[j][e] = a; sacc[j][2 + e] = b;
                     mx_a = fmaxf(mx_a, a); mx_b = fmaxf(mx_b, b);
                 }
+            }
 #pragma unroll
             for (int o = 1; o < 4; o <<= 1) { mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, o)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, o)); }
             const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
@@ -527,7 +623,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) grouped_prefill_kernel(const Gr
             const int c = 8 * j + 2 * t;
             if (c < p.row.vdim) {
                 float x = oacc[j][2 * half] * f, y = oacc[j][2 * half + 1] * f;
-                if (p.entry_gate) { x *= ga_entry_gate<__nv_bfloat16>(p, row, h, c); y *= ga_entry_gate<__nv_bfloat16>(p, row, h, c + 1); }
+                if (p.entry_gate) { const float2 s = ga_entry_gates(p, row, h, c); x *= s.x; y *= s.y; }
                 *reinterpret_cast<unsigned*>(o + c) = ga_pack(x, y);
             }
         }
@@ -541,17 +637,24 @@ int form_of(const GroupedRow& r, bool f32) {
     if (f32 || ((r.dim | r.vdim) & 7)) return FORM_SIMPLE;
     return r.dp <= 128 && r.vp <= 128 ? FORM_MEDIUM : r.dp <= 256 && r.vp <= 256 ? FORM_LARGE : FORM_SIMPLE;
 }
-constexpr size_t kGaMaxSmem = 200 * 1024;
-size_t decode_smem(const GroupedRow& r, int share, int unit) {
-    const size_t stages = (size_t)kDecWarps * unit * (r.shared ? 2 * r.pk + 4 : 2 * (r.pk + r.pv)), sums = (size_t)(kDecWarps + 1) * std::min(share, kDecHeads) * r.vp * 4;
-    return std::max(stages, sums);
+constexpr size_t kGaMaxSmem = 200 * 1024, kDecSmem = 160 * 1024;
+// stages, then sums in their place
+size_t decode_recv_at(const GroupedRow& r, int share, int unit, int stage_count) {
+    const size_t stages = (size_t)stage_count * kDecWarps * unit * (r.shared ? 2 * r.pk + 4 : 2 * (r.pk + r.pv)), sums = (size_t)kDecWarps * std::min(share, kDecHeads) * r.vp * 4;
+    return (std::max(stages, sums) + 15) / 16 * 16;
+}
+// and what the other CTAs of the cluster send
+size_t decode_smem(const GroupedRow& r, int share, int unit, int stage_count) {
+    return decode_recv_at(r, share, unit, stage_count) + ((size_t)std::min(share, kDecHeads) * r.vp + kDecCluster) * 4;
 }
 size_t simple_bytes(const GroupedRow& r) { return ((size_t)r.dim + (size_t)kSimpleWarps * r.vdim) * 4; }
-template <int KQ, int NV, int UK>
+template <int KQ, int NV, int UK, bool APPENDS>
 cudaError_t decode_launch(const GroupedParams& p, int nz, cudaStream_t s) {
+    int stages = kDecStages;
+    while (stages > 1 && decode_smem(p.row, p.share, UK, stages) > kDecSmem) --stages;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(nz, p.row.groups * ((p.share + kDecHeads - 1) / kDecHeads), p.n_rows); cfg.blockDim = dim3(kDecThreads); cfg.stream = s;
-    cfg.dynamicSmemBytes = decode_smem(p.row, p.share, UK);
+    cfg.dynamicSmemBytes = decode_smem(p.row, p.share, UK, stages);
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeClusterDimension;
     attr[0].val.clusterDim.x = nz; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
@@ -559,7 +662,7 @@ cudaError_t decode_launch(const GroupedParams& p, int nz, cudaStream_t s) {
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = pdl_enabled() ? 2 : 1;
-    return cudaLaunchKernelEx(&cfg, grouped_decode_kernel<KQ, NV, UK>, p);
+    return cudaLaunchKernelEx(&cfg, grouped_decode_kernel<KQ, NV, UK, APPENDS>, p, stages, (int)decode_recv_at(p.row, p.share, UK, stages));
 }
 constexpr int kUnitMedium = 32, kUnitLarge = 16;
 // CTAs per cluster: enough warps for the longest context, about one CTA per SM over all rows
@@ -584,6 +687,7 @@ GroupedRow grouped_row(int groups, int dim, int vdim, bool f32, bool shared) {
     return r;
 }
 bool grouped_supported(const GroupedRow& r) { return r.dim <= 4096 && simple_bytes(r) <= kGaMaxSmem; }
+bool grouped_appends(const GroupedRow& r, bool f32, int rot_dims) { return form_of(r, f32) != FORM_SIMPLE && rot_dims == 0; }
 bool grouped_spans(const GroupedRow& r, bool f32) { return form_of(r, f32) == FORM_MEDIUM; }
 
 int grouped_init() {
@@ -591,9 +695,12 @@ int grouped_init() {
     SWLM_CUDA(cudaFuncSetAttribute(grouped_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(grouped_simple_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(grouped_simple_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<8, 8, kUnitMedium>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<16, 16, kUnitLarge>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_prefill_kernel<8, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<8, 8, kUnitMedium, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<16, 16, kUnitLarge, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<8, 8, kUnitMedium, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<16, 16, kUnitLarge, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_prefill_kernel<8, 8, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(grouped_prefill_kernel<8, 8, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     return SWLM_OK;
 }
 
@@ -607,7 +714,8 @@ int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches) {
     p.pool = a.pool; p.page_table = a.page_table; p.pages_per_seq = a.pages_per_seq; p.row_seq = a.row_seq; p.row_pos = a.row_pos;
     p.out = a.out; p.out_stride = a.out_stride; p.spans = a.spans; p.tiles = a.tiles; p.status = a.status;
     cudaError_t e;
-    if (!a.only_attention) {
+    const bool appends = grouped_appends(a.row, a.f32, a.rot_dims) && a.singles && a.n_short == a.n_rows && !a.only_attention;
+    if (!a.only_attention && !appends) {
         const dim3 grid(a.n_rows, (a.heads + (a.row.shared ? 1 : 2) * a.row.groups + kAppWarps - 1) / kAppWarps);
         const size_t smem = (size_t)kAppWarps * a.row.dim * 4;
         e = a.f32 ? launch_k(grouped_append_kernel<float>, grid, dim3(kAppWarps * 32), smem, s, p) : launch_k(grouped_append_kernel<__nv_bfloat16>, grid, dim3(kAppWarps * 32), smem, s, p);
@@ -617,8 +725,8 @@ int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches) {
     if (a.n_short > 0) {
         p.n_rows = a.n_short; p.rows = a.short_rows;
         switch (form_of(a.row, a.f32)) {
-        case FORM_MEDIUM: e = decode_launch<8, 8, kUnitMedium>(p, decode_cluster(a, kUnitMedium), s); break;
-        case FORM_LARGE: e = decode_launch<16, 16, kUnitLarge>(p, decode_cluster(a, kUnitLarge), s); break;
+        case FORM_MEDIUM: e = appends ? decode_launch<8, 8, kUnitMedium, true>(p, decode_cluster(a, kUnitMedium), s) : decode_launch<8, 8, kUnitMedium, false>(p, decode_cluster(a, kUnitMedium), s); break;
+        case FORM_LARGE: e = appends ? decode_launch<16, 16, kUnitLarge, true>(p, decode_cluster(a, kUnitLarge), s) : decode_launch<16, 16, kUnitLarge, false>(p, decode_cluster(a, kUnitLarge), s); break;
         default:
             e = a.f32 ? launch_k(grouped_simple_kernel<float>, dim3(a.n_short, a.heads), dim3(kSimpleWarps * 32), simple_bytes(a.row), s, p)
                       : launch_k(grouped_simple_kernel<__nv_bfloat16>, dim3(a.n_short, a.heads), dim3(kSimpleWarps * 32), simple_bytes(a.row), s, p);
@@ -627,7 +735,9 @@ int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches) {
         *launches += 1;
     }
     if (a.n_tiles > 0) {
-        e = launch_k(grouped_prefill_kernel<8, 8>, dim3(a.n_tiles, a.heads), dim3(kPfThreads), (size_t)kPfStages * a.row.block * 2, s, p);
+        const dim3 grid(a.n_tiles, a.heads);
+        const size_t smem = (size_t)kPfStages * a.row.block * 2;
+        e = a.row.shared ? launch_k(grouped_prefill_kernel<8, 8, true>, grid, dim3(kPfThreads), smem, s, p) : launch_k(grouped_prefill_kernel<8, 8, false>, grid, dim3(kPfThreads), smem, s, p);
         if (e != cudaSuccess) return cuda_fail(e, "grouped prompt attention launch");
         *launches += 1;
     }

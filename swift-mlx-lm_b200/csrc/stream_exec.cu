@@ -933,7 +933,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.row_seq = r.seq; a.row_pos = r.pos;
             a.out = column(b, st.out_buf, st.out_off); a.out_stride = s->width[st.out_buf];
             a.n_rows = r.rows; a.n_short = r.n_short; a.short_rows = r.short_rows; a.max_pages = r.splits_pages;
-            a.n_tiles = r.n_tiles; a.tiles = r.tiles; a.status = s->pf_status; a.only_attention = latent_kernel;
+            a.n_tiles = r.n_tiles; a.tiles = r.tiles; a.status = s->pf_status; a.only_attention = latent_kernel; a.singles = r.n_runs == 0;
             if (r.n_spans) a.spans = r.spans[L.window_set];
             int n = 0;
             rc = launch_grouped(a, stream, &n);
@@ -1144,7 +1144,7 @@ int stream_launches_per_step(const swlm_plan* plan) {
             else n += product_launch_count(a);
         } else if (L.kind == L_DELTA) n += delta_step_fits(plan->delta[L.st.layer].shape) ? 1 : 3;
         else if (L.kind == L_RETENTION) n += retention_step_fits(L.st.key_dim, L.st.value_dim) ? 1 : 2;
-        else if (L.kind == L_GROUPED) n += 2;
+        else if (L.kind == L_GROUPED) n += grouped_appends(plan->grouped[L.st.layer].row, plan->all_f32(), L.st.rope_dim) ? 1 : 2;
         else if (L.kind == L_ROUTED) {
             n += m <= 4 || plan->all_f32() ? 2 : 5;
             if (L.m4 && m > 4 && !plan->all_f32())

@@ -595,10 +595,13 @@ struct GroupedLaunch {
     int n_short = 0; const int32_t* short_rows = nullptr; int max_pages = 1;   // attended one by one; longest context of theirs
     const LatentSpan* spans = nullptr; int n_tiles = 0; const int2* tiles = nullptr;   // and in spans: tiles of kLatentQueryTile rows
     int* status = nullptr;
+    bool singles = false;          // every row is the only one of its sequence
     bool only_attention = false;   // timing hook
 };
 int grouped_init();
 bool grouped_supported(const GroupedRow& r);
+// do batches of single tokens take one launch (norm and append in the attention kernel)?
+bool grouped_appends(const GroupedRow& r, bool f32, int rot_dims);
 // can rows of this layer be attended in spans?
 bool grouped_spans(const GroupedRow& r, bool f32);
 int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches);
