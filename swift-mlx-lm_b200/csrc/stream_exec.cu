@@ -788,7 +788,8 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
         const Launch& L = plan->launches[li];
         const swlm_step& st = L.st;
         if (L.fused && r.n_runs == 0) {
-            const TokenInput t = token_input(&L);
+            TokenInput t = token_input(&L);
+            t.status = s->pf_status;
             if (token_input_fits(t, r.rows, d.hidden)) {
                 li += L.fused;
                 if (only_kind >= 0 && only_kind != L_JOIN) continue;

@@ -6,6 +6,7 @@
 //                   columns; the norm's sum crosses the cluster through distributed shared memory. With a token input in between
 //                   (two small products with a gated table row between them, then a second norm) that is part of it: a CTA
 //                   multiplies its columns of the stream, the sums cross the cluster, and it works out its columns of the result.
+//                   Its weights come to shared memory before the preceding kernel has finished, as far as they fit.
 //   portions        stream_join_kernel (a CTA per row) and stream_conv_kernel (a thread walks a few rows of four channels).
 //
 // A convolution finds the tokens in front of a portion in the state of the sequence. The state is written by the launch that
@@ -16,6 +17,7 @@
 #include <utility>
 
 #include "swlm_internal.h"
+#include "tc_device.cuh"
 
 namespace cg = cooperative_groups;
 
@@ -23,8 +25,10 @@ namespace swlm {
 namespace {
 
 constexpr int kConvRows = 16, kConvThreads = 128;
-constexpr int kStepCluster = 8, kStepMaxRows = 16;   // rows beyond which the products of a token input run on their own
-constexpr int kSideThreads = 256, kSideRows = 16;    // weight rows of a warp whose loads are in flight together
+constexpr int kStepCluster = 8;
+constexpr int kSideThreads = 256, kSideCluster = 16, kSideMaxRows = 8;   // rows beyond which the products of a token input run on their own
+constexpr int kStepResults = 128;   // earlier results whose weights are kept at hand
+constexpr size_t kSideSmem = 160 * 1024;
 
 __device__ __forceinline__ void jn_put4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
 __device__ __forceinline__ void jn_put4(__nv_bfloat16* p, const float (&v)[4]) {
@@ -49,22 +53,23 @@ __device__ __forceinline__ void jn_weights4(const __nv_bfloat16* p, int i, int n
 }
 __device__ __forceinline__ float jn_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 
-// sum over j < avg - 1 of avg_w[j] * results[j] at four entries of a row
-__device__ __forceinline__ void jn_results(const JoinLaunch& p, int r, int i, float (&sum)[4]) {
+// sum over j < avg - 1 of weight(j) * results[j] at four entries of a row
+template <typename W>
+__device__ __forceinline__ void jn_results(const JoinLaunch& p, W weight, int r, int i, float (&sum)[4]) {
     sum[0] = sum[1] = sum[2] = sum[3] = 0.f;
     const float* at = p.results + (size_t)r * p.res_stride + i;
 #pragma unroll 8
     for (int q = 0; q < p.avg - 1; ++q) {
         float v[4];
         jn_get4(at + q * p.result_step, v);
-        const float w = __bfloat162float(p.avg_w[q]);
+        const float w = weight(q);
 #pragma unroll
         for (int e = 0; e < 4; ++e) sum[e] = fmaf(w, v[e], sum[e]);
     }
 }
 __device__ __forceinline__ void jn_average(const JoinLaunch& p, int r, int i, float (&h)[4]) {
     float sum[4];
-    jn_results(p, r, i, sum);
+    jn_results(p, [&](int q) { return __bfloat162float(p.avg_w[q]); }, r, i, sum);
     const float w = __bfloat162float(p.avg_w[p.avg - 1]);
 #pragma unroll
     for (int e = 0; e < 4; ++e) h[e] = fmaf(w, h[e], sum[e]);
@@ -196,11 +201,12 @@ __global__ void __launch_bounds__(kConvThreads) stream_conv_kernel(const JoinLau
 }
 
 // ---- single tokens ----------------------------------------------------------------------------------------------------
-// Sums over the warp of 16 values a lane; the sum of value lane >> 1 is left in this lane.
-__device__ __forceinline__ float jn_sums16(float (&v)[16], int lane) {
-    int o = 16;
+// Sums over LANES neighbouring lanes of V values each; the sum of value (lane % LANES) * V / LANES is left in this lane.
+template <int LANES, int V>
+__device__ __forceinline__ float jn_sums(float (&v)[V], int lane) {
+    int o = LANES / 2;
 #pragma unroll
-    for (int n = 8; n > 0; n >>= 1, o >>= 1) {
+    for (int n = V / 2; n > 0; n >>= 1, o >>= 1) {
         const bool upper = lane & o;
 #pragma unroll
         for (int j = 0; j < n; ++j) {
@@ -208,24 +214,28 @@ __device__ __forceinline__ float jn_sums16(float (&v)[16], int lane) {
             v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
     }
-    return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+    float r = v[0];
+    for (; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+    return r;
 }
-// out[n] = W[n][0 .. 8 chunks) . x for n < rows, by the whole CTA; x and out in shared memory
-__device__ __forceinline__ void jn_rows(const __nv_bfloat16* w, int ld, int rows, int chunks, const float* x, float* out) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int n0 = warp * kSideRows; n0 < rows; n0 += kSideThreads / 32 * kSideRows) {
-        float acc[kSideRows];
+// out[n] = W[n][0 .. 8 chunks) . x for n < rows, by the whole CTA, LANES lanes to a row; x and out in shared memory, W anywhere
+template <int LANES, int V>
+__device__ __forceinline__ void jn_rows_by(const __nv_bfloat16* w, int ld, int rows, int chunks, const float* x, float* out) {
+    constexpr int PER = 32 / LANES;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, part = lane / LANES, l = lane % LANES;
+    for (int n0 = warp * V * PER; n0 < rows; n0 += kSideThreads / 32 * V * PER) {
+        float acc[V];
 #pragma unroll
-        for (int q = 0; q < kSideRows; ++q) acc[q] = 0.f;
-        for (int c = lane; c < chunks; c += 32) {
-            uint4 v[kSideRows];
+        for (int q = 0; q < V; ++q) acc[q] = 0.f;
+        for (int c = l; c < chunks; c += LANES) {
+            uint4 v[V];
 #pragma unroll
-            for (int q = 0; q < kSideRows; ++q) v[q] = n0 + q < rows ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)(n0 + q) * ld) + c) : make_uint4(0, 0, 0, 0);
+            for (int q = 0; q < V; ++q) v[q] = n0 + q * PER + part < rows ? *(reinterpret_cast<const uint4*>(w + (size_t)(n0 + q * PER + part) * ld) + c) : make_uint4(0, 0, 0, 0);
             float f[8];
             *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(x + 8 * c);
             *reinterpret_cast<float4*>(f + 4) = *reinterpret_cast<const float4*>(x + 8 * c + 4);
 #pragma unroll
-            for (int q = 0; q < kSideRows; ++q) {
+            for (int q = 0; q < V; ++q) {
                 const unsigned b[4] = {v[q].x, v[q].y, v[q].z, v[q].w};
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
@@ -234,9 +244,15 @@ __device__ __forceinline__ void jn_rows(const __nv_bfloat16* w, int ld, int rows
                 }
             }
         }
-        const float sum = jn_sums16(acc, lane);
-        if (!(lane & 1) && n0 + (lane >> 1) < rows) out[n0 + (lane >> 1)] = sum;
+        const float sum = jn_sums<LANES, V>(acc, lane);
+        const int n = n0 + l * V / LANES * PER + part;
+        if (l % (LANES / V) == 0 && n < rows) out[n] = sum;
     }
+}
+__device__ __forceinline__ void jn_rows(const __nv_bfloat16* w, int ld, int rows, int chunks, const float* x, float* out) {
+    if (chunks > 16) jn_rows_by<32, 16>(w, ld, rows, chunks, x, out);
+    else if (chunks > 8) jn_rows_by<16, 16>(w, ld, rows, chunks, x, out);
+    else jn_rows_by<8, 8>(w, ld, rows, chunks, x, out);
 }
 __device__ __forceinline__ float jn_rounded(float v, float) { return v; }
 __device__ __forceinline__ float jn_rounded(float v, __nv_bfloat16) { return __bfloat162float(__float2bfloat16_rn(v)); }
@@ -245,17 +261,42 @@ __device__ __forceinline__ float jn_rounded(float v, __nv_bfloat16) { return __b
 // whose result f's norm is for; else the same as p).
 template <typename T, bool SIDE, int NT>
 __global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, const TokenInput side, const JoinLaunch f) {
-    extern __shared__ __align__(16) float step_smem[];
-    __shared__ float red[NT / 32], ssq[2][kStepCluster];
+    extern __shared__ __align__(128) float step_smem[];
+    __shared__ float red[NT / 32], ssq[2][SIDE ? kSideCluster : kStepCluster], avg_s[kStepResults];
+    __shared__ __align__(8) unsigned long long landed[2];
     const cg::cluster_group cluster = cg::this_cluster();
     auto started = cluster.barrier_arrive();   // waited for before anything is written to another CTA's shared memory
     pdl_launch_dependents();
     const int tid = threadIdx.x, nz = gridDim.x, rank = blockIdx.x, row = blockIdx.y, width = p.width;
     const int chunks = (width + 7) / 8, share = (chunks + nz - 1) / nz, chunk0 = share * rank, own = max(0, min(share, chunks - chunk0));   // chunks of eight columns
+    // shared memory of a token input: this CTA's columns of the stream, later of the result; its sums; everybody's; its columns of the
+    // first matrix; its rows of the second
+    const int np = (side.n + 7) / 8 * 8, own_rows = max(0, min(8 * own, width - 8 * chunk0));
+    float* xs = step_smem;
+    float* part = xs + 8 * share;
+    float* all = part + np;
+    __nv_bfloat16* gate_s = reinterpret_cast<__nv_bfloat16*>(all + (size_t)nz * np);
+    __nv_bfloat16* proj_s = gate_s + (side.gate_here ? (size_t)side.n * 8 * share : 0);
+    if (SIDE && (side.gate_here || side.proj_here)) {
+        if (tid == 0) {
+            mbar_init(&landed[0], 1);
+            mbar_init(&landed[1], 1);
+            asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+            mbar_expect(smem_u32(&landed[0]), side.gate_here ? (unsigned)(side.n * own * 16) : 0u);
+            mbar_expect(smem_u32(&landed[1]), side.proj_here ? (unsigned)(own_rows * np * 2) : 0u);
+        }
+        __syncthreads();
+        if (side.gate_here && own > 0)
+            for (int n = tid; n < side.n; n += NT) bulk_load(smem_u32(gate_s + (size_t)n * 8 * share), side.gate + (size_t)n * side.gate_ld + 8 * chunk0, own * 16, smem_u32(&landed[0]));
+        if (side.proj_here)
+            for (int n = 16 * tid; n < own_rows; n += 16 * NT)
+                bulk_load(smem_u32(proj_s + (size_t)n * np), side.proj + (size_t)(8 * chunk0 + n) * side.proj_ld, (unsigned)(min(16, own_rows - n) * np * 2), smem_u32(&landed[1]));
+    }
     const int i = 8 * chunk0 + 4 * tid;
     const bool mine = 4 * tid < 8 * own, whole = (width & 3) == 0;
     const int seq = p.row_seq[row], pos = p.row_pos[row], past = max(0, f.taps - 1);
     // what does not depend on the kernels in front of this one: weights, and the convolution's past
+    for (int q = tid; q < min(f.avg, kStepResults); q += NT) avg_s[q] = __bfloat162float(f.avg_w[q]);
     float nw[4] = {}, fw[4] = {}, before[4] = {}, last[4] = {};
     if (mine) {
         if (p.in) jn_weights4(p.w, i, width, whole, nw);
@@ -270,13 +311,14 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, con
                 }
         }
     }
-    if (SIDE) {   // the token input's weights come closer
+    if (SIDE && !side.gate_here) {   // the other weights come closer
         const int lines = (own + 7) / 8;   // of 128 bytes per row of this CTA's columns
         for (int n = tid; n < side.n * lines; n += NT)
             asm volatile("prefetch.global.L2 [%0];" ::"l"(side.gate + (size_t)(n / lines) * side.gate_ld + 8 * chunk0 + 64 * (n % lines)));
-        const int rows = min(8 * own, width - 8 * chunk0), all = (rows * side.proj_ld + 63) / 64;
-        for (int n = tid; n < all; n += NT) asm volatile("prefetch.global.L2 [%0];" ::"l"(side.proj + (size_t)8 * chunk0 * side.proj_ld + 64 * n));
     }
+    if (SIDE && !side.proj_here)
+        for (int n = tid; n < (own_rows * side.proj_ld + 63) / 64; n += NT) asm volatile("prefetch.global.L2 [%0];" ::"l"(side.proj + (size_t)8 * chunk0 * side.proj_ld + 64 * n));
+    __syncthreads();   // (avg_s)
     pdl_wait();
     float h[4] = {}, t[4] = {}, sum[4] = {};
     if (mine) {
@@ -285,7 +327,7 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, con
         if (p.in) jn_get4(p.in + (size_t)row * p.in_stride + i, t);
         float gate[4];
         if (p.gate) jn_get4(p.gate + (size_t)row * p.gate_stride + i, gate);
-        if (f.avg) jn_results(f, row, i, sum);
+        if (f.avg) jn_results(f, [&](int q) { return q < kStepResults ? avg_s[q] : __bfloat162float(f.avg_w[q]); }, row, i, sum);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             if (p.table) h[e] *= p.table_scale;
@@ -317,6 +359,11 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, con
         for (int q = 0; q < nz; ++q) total += ssq[slot][q];
         return 1.0f / sqrtf(total / (float)width + eps);
     };
+    auto wait = [&](int which) {   // for the weights in shared memory; never leave with a copy under way (bounded)
+        if (mbar_wait(&landed[which], 0u)) return;
+        if (tid == 0) atomicExch(side.status, 71);
+        mbar_wait(&landed[which], 0u);
+    };
     cluster.barrier_wait(std::move(started));
     if (p.in) {
         const float scale = over_rms(t, 0, p.eps);
@@ -324,15 +371,14 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, con
         for (int e = 0; e < 4; ++e) h[e] = fmaf(t[e] * scale, nw[e] + p.weight_bias, h[e]);
     }
     if (SIDE) {
-        const int np = (side.n + 7) / 8 * 8;
-        float* xs = step_smem;             // [8 share] this CTA's columns of the stream, later of the result
-        float* part = xs + 8 * share;      // [np] this CTA's sums
-        float* all = part + np;            // [nz][np] everybody's
         if (4 * tid < 8 * share)
 #pragma unroll
             for (int e = 0; e < 4; ++e) xs[4 * tid + e] = mine && i + e < width ? jn_rounded(h[e], T(0.f)) : 0.f;
         __syncthreads();
-        jn_rows(side.gate + 8 * chunk0, side.gate_ld, side.n, own, xs, part);
+        if (side.gate_here) {
+            wait(0);
+            jn_rows(gate_s, 8 * share, side.n, own, xs, part);
+        } else jn_rows(side.gate + 8 * chunk0, side.gate_ld, side.n, own, xs, part);
         __syncthreads();
         for (int n = tid; n < side.n * nz; n += NT) cluster.map_shared_rank(all, n / side.n)[rank * np + n % side.n] = part[n % side.n];
         cluster.sync();
@@ -346,7 +392,10 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const JoinLaunch p, con
             part[n] = v;
         }
         __syncthreads();
-        jn_rows(side.proj + (size_t)8 * chunk0 * side.proj_ld, side.proj_ld, min(8 * own, width - 8 * chunk0), np / 8, part, xs);
+        if (side.proj_here) {
+            wait(1);
+            jn_rows(proj_s, np, own_rows, np / 8, part, xs);
+        } else jn_rows(side.proj + (size_t)8 * chunk0 * side.proj_ld, side.proj_ld, own_rows, np / 8, part, xs);
         __syncthreads();
 #pragma unroll
         for (int e = 0; e < 4; ++e) t[e] = mine && i + e < width ? xs[4 * tid + e] : 0.f;
@@ -409,7 +458,7 @@ int portions(const JoinLaunch& a, cudaStream_t s, int* launches) {
 
 size_t side_smem(const TokenInput& t, int width, int nz) {
     const size_t np = (t.n + 7) / 8 * 8, share = ((width + 7) / 8 + nz - 1) / nz;
-    return (8 * share + np * (nz + 1)) * 4;
+    return (8 * share + np * (nz + 1)) * 4 + (t.gate_here ? (size_t)t.n * share * 16 : 0) + (t.proj_here ? 8 * share * np * 2 : 0);
 }
 template <typename T, bool SIDE, int NT>
 int step_launch(const JoinLaunch& p, const TokenInput& side, const JoinLaunch& f, int nz, cudaStream_t s) {
@@ -427,8 +476,37 @@ int step_launch(const JoinLaunch& p, const TokenInput& side, const JoinLaunch& f
     return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "stream step launch");
 }
 constexpr int kStepThreads = 128;
-constexpr size_t kSideMaxSmem = 40 * 1024;
 bool step_fits(int width) { return width <= 4 * kSideThreads * kStepCluster; }
+
+// What of the weights fits shared memory, and the size of the cluster: as many CTAs as the GPU runs together, so that most does.
+TokenInput side_shape(TokenInput t, int width, int nz) {
+    t.gate_here = 1;
+    if (side_smem(t, width, nz) > kSideSmem) t.gate_here = 0;
+    t.proj_here = t.proj_ld == (t.n + 7) / 8 * 8;
+    if (side_smem(t, width, nz) > kSideSmem) t.proj_here = 0;
+    return t;
+}
+template <typename T>
+int side_launch(const JoinLaunch& first, const TokenInput& t, const JoinLaunch& last, cudaStream_t s) {
+    const auto kernel = stream_step_kernel<T, true, kSideThreads>;
+    static const cudaError_t attr = [&] {
+        const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSideSmem);
+        return e != cudaSuccess ? e : cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    }();
+    if (attr != cudaSuccess) return cuda_fail(attr, "stream step attributes");
+    static const int largest = [&] {   // are clusters of 16 CTAs with all of the shared memory possible here?
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = dim3(kSideCluster); cfg.blockDim = dim3(kSideThreads); cfg.dynamicSmemBytes = kSideSmem;
+        cudaLaunchAttribute cluster[1];
+        cluster[0].id = cudaLaunchAttributeClusterDimension;
+        cluster[0].val.clusterDim.x = kSideCluster; cluster[0].val.clusterDim.y = 1; cluster[0].val.clusterDim.z = 1;
+        cfg.attrs = cluster;
+        cfg.numAttrs = 1;
+        int n = 0;
+        return cudaOccupancyMaxActiveClusters(&n, kernel, &cfg) == cudaSuccess && n > 0 ? kSideCluster : kStepCluster;
+    }();
+    return step_launch<T, true, kSideThreads>(first, side_shape(t, first.width, largest), last, largest, s);
+}
 
 }  // namespace
 
@@ -448,11 +526,15 @@ int launch_join(const JoinLaunch& a, cudaStream_t s, int* launches) {
     return a.f32 ? portions<float>(a, s, launches) : portions<__nv_bfloat16>(a, s, launches);
 }
 
-bool token_input_fits(const TokenInput& t, int rows, int width) { return rows <= kStepMaxRows && step_fits(width) && side_smem(t, width, kStepCluster) <= kSideMaxSmem; }
+bool token_input_fits(const TokenInput& t, int rows, int width) {
+    TokenInput none = t;
+    none.gate_here = none.proj_here = 0;
+    return rows <= kSideMaxRows && step_fits(width) && side_smem(none, width, kSideCluster) <= kSideSmem && side_smem(none, width, kStepCluster) <= kSideSmem;
+}
 int launch_token_input(const JoinLaunch& first, const TokenInput& t, const JoinLaunch& last, cudaStream_t s) {
     if (first.rows <= 0) return SWLM_OK;
     if (!token_input_fits(t, first.rows, first.width)) { set_error("token input of %d entries into %d x %d", t.n, first.rows, first.width); return SWLM_ERR_UNSUPPORTED; }
-    return first.f32 ? step_launch<float, true, kSideThreads>(first, t, last, kStepCluster, s) : step_launch<__nv_bfloat16, true, kSideThreads>(first, t, last, kStepCluster, s);
+    return first.f32 ? side_launch<float>(first, t, last, s) : side_launch<__nv_bfloat16>(first, t, last, s);
 }
 
 int launch_token_gate(int m, int n, const void* in, int in_stride, const int32_t* tokens, int vocab, const __nv_bfloat16* table, int cols, int col, void* out,

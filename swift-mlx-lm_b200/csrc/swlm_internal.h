@@ -494,6 +494,8 @@ struct TokenInput {
     int n = 0;
     const __nv_bfloat16 *gate = nullptr, *proj = nullptr; int gate_ld = 0, proj_ld = 0;   // [n][width], [width][n]
     const __nv_bfloat16* table = nullptr; int cols = 0, col = 0;
+    int* status = nullptr;
+    int gate_here = 0, proj_here = 0;                      // (decided at the launch) which weights are held in shared memory
 };
 bool token_input_fits(const TokenInput& t, int rows, int width);
 int launch_token_input(const JoinLaunch& first, const TokenInput& t, const JoinLaunch& last, cudaStream_t s);
