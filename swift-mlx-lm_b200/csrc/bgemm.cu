@@ -324,6 +324,7 @@ constexpr int kTcBlock = kTcWarps * 32;
 
 struct TcParams {
     int n, m, steps;                 // weight rows, activation rows, 64-column steps of K
+    int split;                       // weight rows from here on (a multiple of 256) meet the activations of wmap2's place
     int split_steps;                 // steps per K range (gridDim.z ranges); == steps when K is not cut
     GatedAct act;
     const int4* tiles;               // grouped form: (expert, first row, rows, 0) of tile blockIdx.x; n = rows of one expert's matrix
@@ -406,7 +407,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
                 if (nt == 2) tma_load_2d(dst + A_BYTES, GATED ? &wmap2 : &wmap, (step0 + kt) * kTcK, wrow0 + (GATED ? row0 : row0 + kTileRows), bar);
             };
             auto activations = [&](int kt, int s) {
-                tma_load_2d(smem_u32(smem + s * STAGE) + 2 * A_BYTES, &xmap, (step0 + kt) * kTcK, tok0, smem_u32(&full_bar[s]));
+                tma_load_2d(smem_u32(smem + s * STAGE) + 2 * A_BYTES, !GATED && row0 >= p.split ? &wmap2 : &xmap, (step0 + kt) * kTcK, tok0, smem_u32(&full_bar[s]));
             };
             for (int kt = 0; kt < ahead; ++kt) weights(kt, kt);
             pdl_wait();
@@ -639,6 +640,8 @@ int tc_launch(const ProductLaunch& a, const TcShape& t, cudaStream_t s) {
     int rc = bf16_map(static_cast<const __nv_bfloat16*>(a.x), a.x_stride, a.m, a.w->k, BN, &xmap);
     if (!rc) rc = bf16_map(a.w->data, a.w->ld, a.w->n, a.w->k, kTileRows, &wmap);
     wmap2 = wmap;
+    p.split = a.x2 ? a.split : p.n;
+    if (!rc && a.x2) rc = bf16_map(static_cast<const __nv_bfloat16*>(a.x2), a.x2_stride, a.m, a.w->k, BN, &wmap2);
     if (!rc && gated) rc = bf16_map(a.w2->data, a.w2->ld, a.w2->n, a.w2->k, kTileRows, &wmap2);
     if (rc) return rc;
     const dim3 grid((unsigned)t.tiles_m, (unsigned)t.tiles_n, (unsigned)t.ranges);
@@ -683,7 +686,10 @@ bool product_takes_norm(int m, int k) { return m <= 2 && k <= 16384 && gemv_fits
 // gate and up in one launch: always, except as true fp32 products over many rows
 bool product_takes_gate(int m, int k, bool x_f32) { return !x_f32 || gemv_fits(m, k, true, false); }
 
-bool product_takes_two(int m, int k, int split, bool x_f32) { return m <= kGemvRows && !(split & 3) && gemv_smem(2 * m, (k + 7) / 8 * 8, x_f32, false) <= kGemvMaxSmem; }
+bool product_takes_two(int m, int k, int split, bool x_f32) {
+    if (gemv_fits(m, k, x_f32, false)) return !(split & 3) && gemv_smem(2 * m, (k + 7) / 8 * 8, x_f32, false) <= kGemvMaxSmem;
+    return !x_f32 && split % (2 * kTileRows) == 0;   // no tile has rows of both
+}
 
 size_t product_part_floats(int n, int k, int m, bool gated) {
     if (gemv_fits(m, k, false, false)) return 0;
@@ -718,7 +724,7 @@ int launch_product(const ProductLaunch& a, cudaStream_t s) {
         const size_t smem = gemv_smem(a.x2 ? 2 * a.m : a.m, a.w->ld, a.x_f32, a.norm.mode != 0);
         return a.x_f32 ? gemv_rows<float>(p, gated, smem, s) : gemv_rows<__nv_bfloat16>(p, gated, smem, s);
     }
-    if (a.x2) { set_error("two inputs of a product over %d rows run one after the other", a.m); return SWLM_ERR_INVALID; }
+    if (a.x2 && (gated || a.experts || !product_takes_two(a.m, a.w->k, a.split, a.x_f32))) { set_error("two inputs of a product over %d rows run one after the other", a.m); return SWLM_ERR_INVALID; }
     if (a.norm.mode) { set_error("a norm in front of a product over %d rows runs on its own", a.m); return SWLM_ERR_INVALID; }
     if (a.x_f32) {
         if (gated) { set_error("gate and up of fp32 rows run one after the other"); return SWLM_ERR_INVALID; }
@@ -726,7 +732,7 @@ int launch_product(const ProductLaunch& a, cudaStream_t s) {
                                        a.w->ld, a.w->n, a.w->k, a.m, static_cast<const float*>(a.x), a.x_stride, a.out);
         return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "sgemm launch");
     }
-    if ((a.x_stride & 7) || (reinterpret_cast<uintptr_t>(a.x) & 15)) { set_error("dense product: activation rows must be 16-byte aligned"); return SWLM_ERR_INVALID; }
+    if (((a.x_stride | a.x2_stride) & 7) || ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.x2)) & 15)) { set_error("dense product: activation rows must be 16-byte aligned"); return SWLM_ERR_INVALID; }
     const TcShape t = a.experts ? grouped_shape(a) : tc_shape(a.w->n, a.w->k, a.m, gated);
     if (t.ranges > 1 && (!a.part || a.part_floats < (size_t)t.ranges * (gated ? 2 : 1) * a.m * a.w->n)) { set_error("dense product: scratch too small"); return SWLM_ERR_INVALID; }
     switch (t.bn) {

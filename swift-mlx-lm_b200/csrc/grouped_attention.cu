@@ -48,6 +48,12 @@ __device__ __forceinline__ void ga_mma(float (&d)[4], const unsigned (&a)[4], un
 __device__ __forceinline__ void ga_ldsm(unsigned (&r)[4], unsigned addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
+// lane (g, t) gives entries 2t and 2t + 1 of row g of an 8 x 8 matrix and gets those of row g of its transpose
+__device__ __forceinline__ unsigned ga_transpose(unsigned v) {
+    unsigned r;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+    return r;
+}
 __device__ __forceinline__ void ga_ldsm_trans(unsigned (&r)[4], unsigned addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
@@ -201,10 +207,11 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) grouped_simple_kernel(const
 }
 
 // ---- rows one by one, tensor cores ------------------------------------------------------------------------------------
-// Cluster of CTAs per (row, key / value head, 16 query heads of it): the context in units of UK keys, dealt out to all warps of the
-// cluster. A unit is two bulk copies (keys, values) into the warp's own stage.
+// Cluster of CTAs per (row, key / value head, eight query heads of it): the context in units of UK keys, dealt out to all warps of the
+// cluster. A unit is two bulk copies (keys, values) into a stage of the warp's own. Keys (and entries of the values) are the rows of the
+// multiplications, the few heads their columns.
 constexpr int kDecStages = 2;   // units under way per warp, as far as shared memory goes
-constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kDecHeads = 16, kDecCluster = 8;
+constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kDecHeads = 8, kDecCluster = 16;
 template <int KQ, int NV, int UK, bool APPENDS>   // 16-column steps of query / key and value rows, keys of a unit; norm and append in here
 __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const GroupedParams p, int stages, int recv_at) {
     extern __shared__ __align__(128) unsigned char dec_smem[];
@@ -243,8 +250,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
     __nv_bfloat16* own_block = keeps ? ga_block<__nv_bfloat16>(p, seq, pos / kPage, kv) : nullptr;
     const float temperature = APPENDS && p.temp_every > 0 ? 1.0f + p.temp_coef * logf((float)((pos + 1) / p.temp_every) + 1.0f) : 1.0f;
     if (APPENDS) pdl_wait();
-    const float gate = tid >> 3 < nh ? ga_gate(p, r, h0 + (tid >> 3)) : 0.f;   // of the head whose results this thread merges
-    // query fragments: rows g and g + 8
+    const float gate = tid >> 4 < nh ? ga_gate(p, r, h0 + (tid >> 4)) : 0.f;   // of the head whose results this thread merges
     const int ksteps = p.row.dp >> 4, n_vt = p.row.vp >> 4;
     const __nv_bfloat16* qkv = static_cast<const __nv_bfloat16*>(p.qkv) + (size_t)r * p.qkv_stride;
     const __nv_bfloat16* q = qkv + (size_t)h0 * p.row.dim;
@@ -283,36 +289,46 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
         }
     }
     const __nv_bfloat16* own_v = APPENDS && p.row.shared ? k_s : v_s;
-    unsigned qa[KQ][4];
+    // A column is a head. Up to four heads fill the columns twice: the first four carry the high parts of the softmax weights, the
+    // others the low parts.
+    const bool twice = nh <= kDecHeads / 2;
+    const int hq = twice ? g & 3 : g;          // the head of column g
+    unsigned qb[KQ][2];
 #pragma unroll
     for (int k = 0; k < KQ; ++k)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int hh = g + 8 * (e & 1), c = 16 * k + 8 * (e >> 1) + 2 * t;
-            if (APPENDS) qa[k][e] = hh < nh ? *reinterpret_cast<const unsigned*>(q_s + (size_t)hh * QP + c) : 0u;
-            else qa[k][e] = hh < nh && c < p.row.dim ? __ldcg(reinterpret_cast<const unsigned*>(q + (size_t)hh * p.row.dim + c)) : 0u;
+        for (int e = 0; e < 2; ++e) {
+            const int c = 16 * k + 8 * e + 2 * t;
+            if (APPENDS) qb[k][e] = hq < nh ? *reinterpret_cast<const unsigned*>(q_s + (size_t)hq * QP + c) : 0u;
+            else qb[k][e] = hq < nh && c < p.row.dim ? __ldcg(reinterpret_cast<const unsigned*>(q + (size_t)hq * p.row.dim + c)) : 0u;
         }
-    float oacc[2 * NV][4];
+    // lane (g, t): rows g and g + 8 of every tile (keys, or entries of the values), columns 2t and 2t + 1
+    float oacc[NV][4];
 #pragma unroll
-    for (int j = 0; j < 2 * NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
-    float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-    if (APPENDS && rank == 0 && warp == 0) {   // the token's own key: the first column of a tile whose others are zero
+    for (int j = 0; j < NV; ++j) oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    if (APPENDS && rank == 0 && warp == 0) {   // the token's own key: the first row of a tile whose others are zero
         float own[4] = {0.f, 0.f, 0.f, 0.f}, odd[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int k = 0; k < KQ; ++k) {
-            const unsigned b0 = g == 0 ? *reinterpret_cast<const unsigned*>(k_s + 16 * k + 2 * t) : 0u, b1 = g == 0 ? *reinterpret_cast<const unsigned*>(k_s + 16 * k + 8 + 2 * t) : 0u;
-            ga_mma(k & 1 ? odd : own, qa[k], b0, b1);
+            const unsigned ka[4] = {g == 0 ? *reinterpret_cast<const unsigned*>(k_s + 16 * k + 2 * t) : 0u, 0u, g == 0 ? *reinterpret_cast<const unsigned*>(k_s + 16 * k + 8 + 2 * t) : 0u, 0u};
+            ga_mma(k & 1 ? odd : own, ka, qb[k][0], qb[k][1]);
         }
         const float f = p.row.shared ? p.scale_log2 * own_factor : p.scale_log2;
-        m_a = f * __shfl_sync(0xffffffffu, own[0] + odd[0], lane & ~3);
-        m_b = f * __shfl_sync(0xffffffffu, own[2] + odd[2], lane & ~3);
-        l_a = l_b = t == 0 ? 1.f : 0.f;
 #pragma unroll
-        for (int j = 0; j < 2 * NV; ++j) {
-            oacc[j][0] = oacc[j][2] = __bfloat162float(own_v[8 * j + 2 * t]);
-            oacc[j][1] = oacc[j][3] = __bfloat162float(own_v[8 * j + 2 * t + 1]);
+        for (int e = 0; e < 2; ++e) {
+            m[e] = f * __shfl_sync(0xffffffffu, own[e] + odd[e], t);
+            l[e] = g == 0 ? 1.f : 0.f;
+        }
+        if (!twice || t < 2) {
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                oacc[j][0] = oacc[j][1] = __bfloat162float(own_v[16 * j + g]);
+                oacc[j][2] = oacc[j][3] = __bfloat162float(own_v[16 * j + 8 + g]);
+            }
         }
     }
+    constexpr int MT = UK / 16;
     int at = 0;
     unsigned phase = 0;
     for (int u = first; u < units; u += step) {
@@ -324,13 +340,13 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
             for (int st = 0; st < stages && u + st * step < units; ++st) mbar_wait(&bar[warp][(at + st) % stages], phase ^ (unsigned)(at + st >= stages));
             break;
         }
-        float sacc[UK / 8][4];
+        float sacc[MT][4];
 #pragma unroll
-        for (int j = 0; j < UK / 8; ++j) sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f;
-        unsigned kf[2][UK / 16][4];   // the next fragments are on their way while these multiply
+        for (int i = 0; i < MT; ++i) sacc[i][0] = sacc[i][1] = sacc[i][2] = sacc[i][3] = 0.f;
+        unsigned kf[2][MT][4];   // the next fragments are on their way while these multiply
         auto keys = [&](int k) {
 #pragma unroll
-            for (int jp = 0; jp < UK / 16; ++jp) ga_ldsm(kf[k & 1][jp], ks + (unsigned)((jp * 16 + (lane & 7) + 8 * (lane >> 4)) * pk + 16 * k + 8 * ((lane >> 3) & 1)) * 2u);
+            for (int i = 0; i < MT; ++i) ga_ldsm(kf[k & 1][i], ks + (unsigned)((16 * i + (lane & 15)) * pk + 16 * k + 8 * (lane >> 4)) * 2u);
         };
         keys(0);
 #pragma unroll
@@ -338,61 +354,58 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
             if (k < ksteps) {
                 if (k + 1 < KQ && k + 1 < ksteps) keys(k + 1);
 #pragma unroll
-                for (int jp = 0; jp < UK / 16; ++jp) {
-                    ga_mma(sacc[2 * jp], qa[k], kf[k & 1][jp][0], kf[k & 1][jp][1]);
-                    ga_mma(sacc[2 * jp + 1], qa[k], kf[k & 1][jp][2], kf[k & 1][jp][3]);
-                }
+                for (int i = 0; i < MT; ++i) ga_mma(sacc[i], kf[k & 1][i], qb[k][0], qb[k][1]);
             }
         const int key0 = (unit0 + u) * UK;
-        float mx_a = -INFINITY, mx_b = -INFINITY;
+        float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-        for (int j = 0; j < UK / 8; ++j)
+        for (int i = 0; i < MT; ++i)
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int key = key0 + 8 * j + 2 * t + e;
+            for (int half = 0; half < 2; ++half) {
+                const int at_key = 16 * i + 8 * half + g, key = key0 + at_key;
                 const bool seen = key < past_end && key >= seen0;
-                const float f = p.row.shared ? p.scale_log2 * factors[8 * j + 2 * t + e] : p.scale_log2;
-                sacc[j][e] = seen ? sacc[j][e] * f : -INFINITY;
-                sacc[j][2 + e] = seen ? sacc[j][2 + e] * f : -INFINITY;
-                mx_a = fmaxf(mx_a, sacc[j][e]); mx_b = fmaxf(mx_b, sacc[j][2 + e]);
+                const float f = p.row.shared ? p.scale_log2 * factors[at_key] : p.scale_log2;
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    float& v = sacc[i][2 * half + e];
+                    v = seen ? v * f : -INFINITY;
+                    mx[e] = fmaxf(mx[e], v);
+                }
             }
 #pragma unroll
-        for (int o = 1; o < 4; o <<= 1) { mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, o)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, o)); }
+        for (int o = 4; o < 32; o <<= 1) { mx[0] = fmaxf(mx[0], __shfl_xor_sync(0xffffffffu, mx[0], o)); mx[1] = fmaxf(mx[1], __shfl_xor_sync(0xffffffffu, mx[1], o)); }
         // (every unit holds at least one key that is seen, by all heads alike)
-        const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b), ca = exp2f(m_a - mn_a), cb = exp2f(m_b - mn_b);
-        m_a = mn_a; m_b = mn_b;
-        float sa = 0.f, sb = 0.f;
+        float corr[2];
 #pragma unroll
-        for (int j = 0; j < UK / 8; ++j)
+        for (int e = 0; e < 2; ++e) {
+            const float next = fmaxf(m[e], mx[e]);
+            corr[e] = exp2f(m[e] - next);
+            m[e] = next;
+            l[e] *= corr[e];
+        }
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                sacc[j][e] = exp2f(sacc[j][e] - mn_a); sa += sacc[j][e];
-                sacc[j][2 + e] = exp2f(sacc[j][2 + e] - mn_b); sb += sacc[j][2 + e];
-            }
-        l_a = l_a * ca + sa; l_b = l_b * cb + sb;
+        for (int j = 0; j < NV; ++j) { oacc[j][0] *= corr[0]; oacc[j][1] *= corr[1]; oacc[j][2] *= corr[0]; oacc[j][3] *= corr[1]; }
 #pragma unroll
-        for (int j = 0; j < 2 * NV; ++j) { oacc[j][0] *= ca; oacc[j][1] *= ca; oacc[j][2] *= cb; oacc[j][3] *= cb; }
+        for (int i = 0; i < MT; ++i) {
+            unsigned hi[2], lo[2];   // weights of keys 2t, 2t + 1 (and + 8) for head g, after the transposition
 #pragma unroll
-        for (int kk = 0; kk < UK / 16; ++kk) {
-            unsigned ah[4], al[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float x = sacc[2 * kk + (e >> 1)][(e & 1) * 2], y = sacc[2 * kk + (e >> 1)][(e & 1) * 2 + 1];
+            for (int half = 0; half < 2; ++half) {
+                const float x = exp2f(sacc[i][2 * half] - m[0]), y = exp2f(sacc[i][2 * half + 1] - m[1]);
+                l[0] += x; l[1] += y;
                 const float xh = ga_round(x), yh = ga_round(y);
-                ah[e] = ga_pack(xh, yh);
-                al[e] = ga_pack(x - xh, y - yh);
+                const unsigned high = ga_pack(xh, yh), low = ga_pack(x - xh, y - yh);
+                hi[half] = ga_transpose(twice && t >= 2 ? low : high);
+                lo[half] = ga_transpose(low);
             }
             unsigned vf[2][4];
-            auto values = [&](int j) { ga_ldsm_trans(vf[j & 1], vs + (unsigned)((16 * kk + (lane & 7) + 8 * ((lane >> 3) & 1)) * pv + 16 * j + 8 * (lane >> 4)) * 2u); };
+            auto values = [&](int j) { ga_ldsm_trans(vf[j & 1], vs + (unsigned)((16 * i + (lane & 7) + 8 * (lane >> 4)) * pv + 16 * j + 8 * ((lane >> 3) & 1)) * 2u); };
             values(0);
 #pragma unroll
             for (int j = 0; j < NV; ++j)
                 if (j < n_vt) {
                     if (j + 1 < NV && j + 1 < n_vt) values(j + 1);
-                    ga_mma(oacc[2 * j], ah, vf[j & 1][0], vf[j & 1][1]);
-                    ga_mma(oacc[2 * j + 1], ah, vf[j & 1][2], vf[j & 1][3]);
-                    ga_mma(oacc[2 * j], al, vf[j & 1][0], vf[j & 1][1]);
-                    ga_mma(oacc[2 * j + 1], al, vf[j & 1][2], vf[j & 1][3]);
+                    ga_mma(oacc[j], vf[j & 1], hi[0], hi[1]);
+                    if (!twice) ga_mma(oacc[j], vf[j & 1], lo[0], lo[1]);
                 }
         }
         __syncwarp();   // the stage is free
@@ -400,67 +413,77 @@ __global__ void __launch_bounds__(kDecThreads, 1) grouped_decode_kernel(const Gr
         if (++at == stages) { at = 0; phase ^= 1; }
     }
 #pragma unroll
-    for (int o = 1; o < 4; o <<= 1) { l_a += __shfl_xor_sync(0xffffffffu, l_a, o); l_b += __shfl_xor_sync(0xffffffffu, l_b, o); }
-    if (t == 0) { warp_m[warp][g] = m_a; warp_m[warp][g + 8] = m_b; warp_l[warp][g] = l_a; warp_l[warp][g + 8] = l_b; }
+    for (int o = 4; o < 32; o <<= 1) { l[0] += __shfl_xor_sync(0xffffffffu, l[0], o); l[1] += __shfl_xor_sync(0xffffffffu, l[1], o); }
+    if (twice) {   // high and low parts
+#pragma unroll
+        for (int j = 0; j < NV; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) oacc[j][e] += __shfl_xor_sync(0xffffffffu, oacc[j][e], 2);
+    }
+    if (g == 0) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) { warp_m[warp][2 * t + e] = m[e]; warp_l[warp][2 * t + e] = l[e]; }
+    }
     __syncthreads();
-    // the stages now hold the warps' sums: [warps][heads of this CTA][vp]
-    const int vp = p.row.vp, share = (nh * vp + nz - 1) / nz;   // entries of the result that a CTA of the cluster finishes
+    // the stages now hold the warps' sums: [warps][heads of this CTA][pitch]
+    const int vp = p.row.vp, pitch = vp + 4, share = (nh * vp + nz - 1) / nz;   // share: entries of the result that a CTA of the cluster finishes
     float* sums = reinterpret_cast<float*>(dec_smem);
     float* recv = reinterpret_cast<float*>(dec_smem + recv_at);   // [nz][share], written by the other CTAs
 #pragma unroll
-    for (int j = 0; j < 2 * NV; ++j) {
-        const int c = 8 * j + 2 * t;
-        if (c < vp) {
-            if (g < nh) *reinterpret_cast<float2*>(sums + ((size_t)warp * nh + g) * vp + c) = make_float2(oacc[j][0], oacc[j][1]);
-            if (g + 8 < nh) *reinterpret_cast<float2*>(sums + ((size_t)warp * nh + g + 8) * vp + c) = make_float2(oacc[j][2], oacc[j][3]);
+    for (int e = 0; e < 2; ++e)
+        if (2 * t + e < nh) {
+            float* row = sums + ((size_t)warp * nh + 2 * t + e) * pitch + g;
+#pragma unroll
+            for (int j = 0; j < NV; ++j)
+                if (j < n_vt) { row[16 * j] = oacc[j][e]; row[16 * j + 8] = oacc[j][2 + e]; }
         }
-    }
     // the gate of the first entry this thread finishes is on its way during the merge
     const __nv_bfloat16* egate = static_cast<const __nv_bfloat16*>(p.entry_gate) + (size_t)r * p.entry_gate_stride + (size_t)h0 * p.row.vdim;
     float entry = 1.f;
     if (p.entry_gate && tid < share && rank * share + tid < nh * vp && (rank * share + tid) % vp < p.row.vdim)
         entry = ga_sigmoid(__bfloat162float(egate[(size_t)((rank * share + tid) / vp) * p.row.vdim + (rank * share + tid) % vp]));
     cluster.barrier_wait(std::move(started));
-    static_assert(kDecWarps == 8 && kDecCluster == 8, "eight lanes per head");
-    auto over8 = [](float& top, float& total, float m, float l) {   // maximum and rescaled sum over eight lanes; this lane's factor
-        top = m;
+    static_assert(kDecWarps <= 16 && kDecCluster == 16 && kDecHeads * 16 <= kDecThreads, "sixteen lanes per head");
+    auto merge = [](float& top, float& total, float mine, float sum) {   // maximum and rescaled sum over sixteen lanes; this lane's factor
+        top = mine;
 #pragma unroll
-        for (int o = 1; o < 8; o <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
-        const float f = m == -INFINITY ? 0.f : exp2f(m - top);
-        total = f * l;
+        for (int o = 1; o < 16; o <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+        const float f = mine == -INFINITY ? 0.f : exp2f(mine - top);
+        total = f * sum;
 #pragma unroll
-        for (int o = 1; o < 8; o <<= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
+        for (int o = 1; o < 16; o <<= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
         return f;
     };
-    const int eighth = tid & 7, of_head = tid >> 3;   // (16 heads: the first four warps)
-    if (warp < kDecHeads / 4) {
+    const int part = tid & 15, of_head = tid >> 4;   // (the first warps, two heads each)
+    if (warp < kDecHeads / 2) {
+        const bool there = part < kDecWarps;
         float top, total;
-        const float f = over8(top, total, warp_m[eighth][of_head], warp_l[eighth][of_head]);
-        warp_l[eighth][of_head] = f;
-        if (eighth < nz) {
-            cluster.map_shared_rank(all_m[rank], eighth)[of_head] = top;
-            cluster.map_shared_rank(all_l[rank], eighth)[of_head] = total;
+        const float f = merge(top, total, there ? warp_m[part][of_head] : -INFINITY, there ? warp_l[part][of_head] : 0.f);
+        if (there) warp_l[part][of_head] = f;
+        if (part < nz) {
+            cluster.map_shared_rank(all_m[rank], part)[of_head] = top;
+            cluster.map_shared_rank(all_l[rank], part)[of_head] = total;
         }
     }
     __syncthreads();
     for (int i = tid; i < nh * vp; i += kDecThreads) {
+        const int hh = i / vp, z = i / share;
         float v = 0.f;
 #pragma unroll
-        for (int w = 0; w < kDecWarps; ++w) v = fmaf(warp_l[w][i / vp], sums[(size_t)w * nh * vp + i], v);
-        const int z = i / share;
+        for (int w = 0; w < kDecWarps; ++w) v = fmaf(warp_l[w][hh], sums[((size_t)w * nh + hh) * pitch + i - hh * vp], v);
         cluster.map_shared_rank(recv, z)[rank * share + i - z * share] = v;
     }
     cluster.sync();   // (nobody reaches into another CTA's shared memory behind this)
-    if (warp < kDecHeads / 4) {
-        const bool there = eighth < nz;
+    if (warp < kDecHeads / 2) {
+        const bool there = part < nz;
         float top, total;
-        float f = over8(top, total, there ? all_m[eighth][of_head] : -INFINITY, there ? all_l[eighth][of_head] : 0.f);
+        float f = merge(top, total, there ? all_m[part][of_head] : -INFINITY, there ? all_l[part][of_head] : 0.f);
         if (p.sink_one) {   // one joins the sum
             const float scale = top > 0.f ? 1.f : exp2f(top);
             f *= scale;
             total = total * scale + exp2f(-fmaxf(top, 0.f));
         }
-        all_m[eighth][of_head] = f * gate / total;
+        all_m[part][of_head] = f * gate / total;
     }
     __syncthreads();
     for (int q = tid; q < share && rank * share + q < nh * vp; q += kDecThreads) {
@@ -640,7 +663,7 @@ int form_of(const GroupedRow& r, bool f32) {
 constexpr size_t kGaMaxSmem = 200 * 1024, kDecSmem = 160 * 1024;
 // stages, then sums in their place
 size_t decode_recv_at(const GroupedRow& r, int share, int unit, int stage_count) {
-    const size_t stages = (size_t)stage_count * kDecWarps * unit * (r.shared ? 2 * r.pk + 4 : 2 * (r.pk + r.pv)), sums = (size_t)kDecWarps * std::min(share, kDecHeads) * r.vp * 4;
+    const size_t stages = (size_t)stage_count * kDecWarps * unit * (r.shared ? 2 * r.pk + 4 : 2 * (r.pk + r.pv)), sums = (size_t)kDecWarps * std::min(share, kDecHeads) * (r.vp + 4) * 4;
     return (std::max(stages, sums) + 15) / 16 * 16;
 }
 // and what the other CTAs of the cluster send
@@ -648,8 +671,35 @@ size_t decode_smem(const GroupedRow& r, int share, int unit, int stage_count) {
     return decode_recv_at(r, share, unit, stage_count) + ((size_t)std::min(share, kDecHeads) * r.vp + kDecCluster) * 4;
 }
 size_t simple_bytes(const GroupedRow& r) { return ((size_t)r.dim + (size_t)kSimpleWarps * r.vdim) * 4; }
+constexpr int kUnitMedium = 32, kUnitLarge = 16;
+// CTAs per cluster: enough warps for the longest context, about one CTA per SM over all rows; the largest clusters only when all of them
+// run at once with room to spare (`clusters`: how many fit an empty GPU)
+int decode_cluster(const GroupedLaunch& a, int unit, int clusters) {
+    int keys = a.max_pages * kPage;
+    if (a.window > 0) keys = std::min(keys, a.window);
+    if (a.chunk > 0) keys = std::min(keys, a.chunk);
+    const int units = (keys + unit - 2) / unit + 1, tiles = a.n_short * a.row.groups * ((a.heads / a.row.groups + kDecHeads - 1) / kDecHeads);
+    int nz = 2 * tiles <= clusters + 1 ? kDecCluster : kDecCluster / 2;
+    while (nz > 1 && ((nz >> 1) * kDecWarps >= units || (long long)tiles * nz > 148)) nz >>= 1;
+    return nz;
+}
+// how many of the largest clusters of a kernel the GPU runs at once
+template <typename K>
+int largest_clusters(K kernel) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(kDecCluster); cfg.blockDim = dim3(kDecThreads); cfg.dynamicSmemBytes = kDecSmem;
+    cudaLaunchAttribute cluster[1];
+    cluster[0].id = cudaLaunchAttributeClusterDimension;
+    cluster[0].val.clusterDim.x = kDecCluster; cluster[0].val.clusterDim.y = 1; cluster[0].val.clusterDim.z = 1;
+    cfg.attrs = cluster;
+    cfg.numAttrs = 1;
+    int n = 0;
+    return cudaOccupancyMaxActiveClusters(&n, kernel, &cfg) == cudaSuccess ? n : 0;
+}
 template <int KQ, int NV, int UK, bool APPENDS>
-cudaError_t decode_launch(const GroupedParams& p, int nz, cudaStream_t s) {
+cudaError_t decode_launch(const GroupedParams& p, const GroupedLaunch& a, cudaStream_t s) {
+    static const int clusters = largest_clusters(grouped_decode_kernel<KQ, NV, UK, APPENDS>);
+    const int nz = decode_cluster(a, UK, clusters);
     int stages = kDecStages;
     while (stages > 1 && decode_smem(p.row, p.share, UK, stages) > kDecSmem) --stages;
     cudaLaunchConfig_t cfg = {};
@@ -664,16 +714,11 @@ cudaError_t decode_launch(const GroupedParams& p, int nz, cudaStream_t s) {
     cfg.numAttrs = pdl_enabled() ? 2 : 1;
     return cudaLaunchKernelEx(&cfg, grouped_decode_kernel<KQ, NV, UK, APPENDS>, p, stages, (int)decode_recv_at(p.row, p.share, UK, stages));
 }
-constexpr int kUnitMedium = 32, kUnitLarge = 16;
-// CTAs per cluster: enough warps for the longest context, about one CTA per SM over all rows
-int decode_cluster(const GroupedLaunch& a, int unit) {
-    int keys = a.max_pages * kPage;
-    if (a.window > 0) keys = std::min(keys, a.window);
-    if (a.chunk > 0) keys = std::min(keys, a.chunk);
-    const int units = (keys + unit - 2) / unit + 1, tiles = a.n_short * a.row.groups * ((a.heads / a.row.groups + kDecHeads - 1) / kDecHeads);
-    int nz = kDecCluster;
-    while (nz > 1 && ((nz >> 1) * kDecWarps >= units || (long long)tiles * nz > 148)) nz >>= 1;
-    return nz;
+template <typename K>
+int decode_attr(K kernel) {
+    SWLM_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+    return SWLM_OK;
 }
 
 }  // namespace
@@ -695,10 +740,9 @@ int grouped_init() {
     SWLM_CUDA(cudaFuncSetAttribute(grouped_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(grouped_simple_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(grouped_simple_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<8, 8, kUnitMedium, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<16, 16, kUnitLarge, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<8, 8, kUnitMedium, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(grouped_decode_kernel<16, 16, kUnitLarge, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
+    int rc;
+    if ((rc = decode_attr(grouped_decode_kernel<8, 8, kUnitMedium, false>)) || (rc = decode_attr(grouped_decode_kernel<8, 8, kUnitMedium, true>)) ||
+        (rc = decode_attr(grouped_decode_kernel<16, 16, kUnitLarge, false>)) || (rc = decode_attr(grouped_decode_kernel<16, 16, kUnitLarge, true>))) return rc;
     SWLM_CUDA(cudaFuncSetAttribute(grouped_prefill_kernel<8, 8, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     SWLM_CUDA(cudaFuncSetAttribute(grouped_prefill_kernel<8, 8, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGaMaxSmem));
     return SWLM_OK;
@@ -725,8 +769,8 @@ int launch_grouped(const GroupedLaunch& a, cudaStream_t s, int* launches) {
     if (a.n_short > 0) {
         p.n_rows = a.n_short; p.rows = a.short_rows;
         switch (form_of(a.row, a.f32)) {
-        case FORM_MEDIUM: e = appends ? decode_launch<8, 8, kUnitMedium, true>(p, decode_cluster(a, kUnitMedium), s) : decode_launch<8, 8, kUnitMedium, false>(p, decode_cluster(a, kUnitMedium), s); break;
-        case FORM_LARGE: e = appends ? decode_launch<16, 16, kUnitLarge, true>(p, decode_cluster(a, kUnitLarge), s) : decode_launch<16, 16, kUnitLarge, false>(p, decode_cluster(a, kUnitLarge), s); break;
+        case FORM_MEDIUM: e = appends ? decode_launch<8, 8, kUnitMedium, true>(p, a, s) : decode_launch<8, 8, kUnitMedium, false>(p, a, s); break;
+        case FORM_LARGE: e = appends ? decode_launch<16, 16, kUnitLarge, true>(p, a, s) : decode_launch<16, 16, kUnitLarge, false>(p, a, s); break;
         default:
             e = a.f32 ? launch_k(grouped_simple_kernel<float>, dim3(a.n_short, a.heads), dim3(kSimpleWarps * 32), simple_bytes(a.row), s, p)
                       : launch_k(grouped_simple_kernel<__nv_bfloat16>, dim3(a.n_short, a.heads), dim3(kSimpleWarps * 32), simple_bytes(a.row), s, p);

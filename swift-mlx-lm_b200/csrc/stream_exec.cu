@@ -684,7 +684,7 @@ size_t part_need(const swlm_plan* plan, int rows, int wants) {
     size_t need = 0;
     if (plan->all_f32()) return 0;
     for (const Launch& L : plan->launches)
-        if (L.kind == L_PRODUCT && L.x2_buf >= 0) for (const Matrix& m : L.part) need = std::max(need, product_part_floats(m.n, m.k, rows, false));
+        if (L.kind == L_PRODUCT && L.x2_buf >= 0) for (const Matrix* m : {L.m1, &L.part[0], &L.part[1]}) need = std::max(need, product_part_floats(m->n, m->k, rows, false));
         else if (L.kind == L_PRODUCT) need = std::max(need, product_part_floats(L.m1->n, L.m1->k, L.seg_buf[0] == SWLM_BUF_LOGITS ? wants : rows, L.m2 != nullptr));
         else if (L.kind == L_ROUTED && L.m4) need = std::max(need, std::max(product_part_floats(L.m4->n, L.m4->k, rows, false), product_part_floats(L.m5->n, L.m5->k, rows, false)));
     return need;

@@ -26,7 +26,7 @@ namespace {
 
 constexpr int kConvRows = 16, kConvThreads = 128;
 constexpr int kStepCluster = 8;
-constexpr int kSideThreads = 256, kSideCluster = 16, kSideMaxRows = 8;   // rows beyond which the products of a token input run on their own
+constexpr int kSideThreads = 256, kSideCluster = 16, kSideMaxRows = 16;   // rows beyond which the products of a token input run on their own
 constexpr int kStepResults = 128;   // earlier results whose weights are kept at hand
 constexpr size_t kSideSmem = 160 * 1024;
 
@@ -505,6 +505,8 @@ int side_launch(const JoinLaunch& first, const TokenInput& t, const JoinLaunch& 
         int n = 0;
         return cudaOccupancyMaxActiveClusters(&n, kernel, &cfg) == cudaSuccess && n > 0 ? kSideCluster : kStepCluster;
     }();
+    // (many rows: smaller clusters that read the weights where they are, so that all run at once)
+    if (first.rows * largest > 148) return step_launch<T, true, kSideThreads>(first, t, last, kStepCluster, s);
     return step_launch<T, true, kSideThreads>(first, side_shape(t, first.width, largest), last, largest, s);
 }
 

@@ -203,6 +203,7 @@ class MerudraPlanBuilder:
         for i, layer in enumerate(c.layers[:layers]):
             p, m, mlp = f"l{i}.", layer.mixer, layer.mlp
             enter(p + "canon1")
+            product(p + "rg1", BUF_S0, BUF_S3, w, w, bias=True)   # (one product with what the mixer projects, of another input)
             if isinstance(m, KeyValueAttention):
                 self._attention(steps, product, p, m, counts[KeyValueAttention])
             else:
@@ -211,8 +212,8 @@ class MerudraPlanBuilder:
             leave(p + "norm1", BUF_S3)
             if mlp is not None:
                 enter(p + "canon2")
-                product(p + "mlp.router", BUF_S1, BUF_S4, mlp.experts + mlp.identity, w)
                 product(p + "rg2", BUF_S0, BUF_S3, w, w, bias=True)
+                product(p + "mlp.router", BUF_S1, BUF_S4, mlp.experts + mlp.identity, w)
                 steps.append(_step(STEP_ROUTED_MLP, in_buf=BUF_S1, in2_buf=BUF_S4, out_buf=BUF_HIDDEN, n=w, k=mlp.ff, experts=mlp.experts, identity=mlp.identity,
                                    top=mlp.top, groups=1, groups_keep=1, scale=1.0, score_act=SCORE_SOFTMAX, group_best=1, raw_weights=1,
                                    expert_act=EXPERT_SILU, weight=p + "mlp.e", weight2=".gate", weight3=".up", weight4=".down", weight7=p + "mlp.correction"))
@@ -229,13 +230,12 @@ class MerudraPlanBuilder:
         return steps
 
     def _attention(self, steps: List[Step], product, p: str, m: KeyValueAttention, index: int) -> None:
-        """q | k | gate side by side; the stream's gate is one product with them, of another input."""
+        """q | k | gate side by side."""
         w, x, qa, ka = self.config.width, p + "mix.", m.heads * m.dim, m.kv_heads * m.dim
         gate_at = _up8(qa + ka)
         product(x + "q", BUF_S1, BUF_S2, qa, w, bias=True)
         product(x + "k", BUF_S1, BUF_S2, ka, w, dst_off=qa, bias=True)
         product(x + "g", BUF_S1, BUF_S2, qa, w, dst_off=gate_at)
-        product(p + "rg1", BUF_S0, BUF_S3, w, w, bias=True)
         steps.append(_step(STEP_GROUPED_ATTN, layer=index, in_buf=BUF_S2, in4_buf=BUF_S2, in4_off=gate_at, out_buf=BUF_S0, heads=m.heads, kv_heads=m.kv_heads,
                            head_dim=m.dim, value_dim=m.dim, value_is_key=1, head_norm=1, scale=m.scale, eps=self.config.norm_eps, temp_coef=m.temp_coef,
                            temp_every=m.temp_every, out_scale=1.0, rope_base=1.0))
@@ -251,7 +251,6 @@ class MerudraPlanBuilder:
         product(x + "g", BUF_S1, BUF_S2, hv, w, dst_off=gate_at)
         product(x + "b", BUF_S1, BUF_S4, m.heads, w)
         product(x + "a", BUF_S1, BUF_S4, m.heads, w, dst_off=decay_at)
-        product(p + "rg1", BUF_S0, BUF_S3, w, w, bias=True)
         steps.append(_step(STEP_GATED_DELTA, layer=index, in_buf=BUF_S2, in2_buf=BUF_S4, in3_buf=BUF_S4, in3_off=decay_at, in4_buf=BUF_S2, in4_off=gate_at,
                            out_buf=BUF_S0, k=1, heads=m.heads, groups=m.kv_heads, key_dim=m.dim, value_dim=m.vdim, conv_kernel=m.conv, eps=self.config.norm_eps,
                            eps2=UNIT_EPS, scale=m.dim ** -0.5, gate_act=GATE_SILU, weight=x + "q.conv", weight2=x + "k.conv", weight3=x + "v.conv",
