@@ -20,7 +20,7 @@ def store(pkg):
 # ---- products with biases and of two inputs ------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("rows", [1, 2, 4, 5, 40, 130])
-@pytest.mark.parametrize("k, first, second", [(64, (24, 8), (40,)), (133, (37, 13, 5), (21, 8)), (520, (300, 4), (520, 3)), (72, (6,), (72,))])
+@pytest.mark.parametrize("k, first, second", [(64, (24, 8), (40,)), (133, (37, 13, 5), (21, 8)), (520, (300, 4), (520, 3)), (72, (6,), (72,)), (136, (256,), (72, 13)), (200, (500, 12), (264,))])
 def test_products_of_two_inputs_with_biases(pkg, store, dtype, rows, k, first, second):
     """Results of both inputs side by side in one buffer, every other one with a bias; the second input starts at rows that are a
     multiple of four, and at others."""
