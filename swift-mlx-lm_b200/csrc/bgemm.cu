@@ -27,21 +27,29 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 }
 
 // Where the results of one weight row go: that of activation row m is m * stride bytes behind y.
-struct ProductRow { unsigned char* y; size_t stride; bool f32; float bias; };
+struct ProductRow { unsigned char* y; size_t stride; bool f32; };
 __device__ __forceinline__ ProductRow product_row(const ProductOut& o, int row) {
     void* y = o.y[0];
-    const __nv_bfloat16* bias = o.bias[0];
     int first = 0, stride = o.stride[0], f32 = o.f32[0];
 #pragma unroll
     for (int q = 1; q < kMaxProductSegs; ++q)
-        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; bias = o.bias[q]; }
+        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; }
     const int size = f32 ? 4 : 2;
-    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0,
-                      bias && row < o.end[o.count - 1] ? __bfloat162float(bias[row - first]) : 0.f};
+    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0};
 }
+// what is added to the results of a weight row (only when biased)
+__device__ __forceinline__ float product_bias(const ProductOut& o, int row) {
+    const __nv_bfloat16* bias = o.bias[0];
+    int first = 0;
+#pragma unroll
+    for (int q = 1; q < kMaxProductSegs; ++q)
+        if (q < o.count && row >= o.end[q - 1]) { bias = o.bias[q]; first = o.end[q - 1]; }
+    return bias ? __bfloat162float(bias[row - first]) : 0.f;
+}
+template <bool BIASED>
 __device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
     const ProductRow r = product_row(o, row);
-    val += r.bias;
+    if (BIASED && o.biased) val += product_bias(o, row);
     if (o.softcap > 0.f) val = o.softcap * tanhf(val / o.softcap);
     if (o.gelu) val = gelu_erf(val);
     if (r.f32) *reinterpret_cast<float*>(r.y + m * r.stride) = val;
@@ -86,8 +94,9 @@ __device__ __forceinline__ void get_x8(const __nv_bfloat16* p, float (&f)[8]) {
     f[0] = b_lo(v.x); f[1] = b_hi(v.x); f[2] = b_lo(v.y); f[3] = b_hi(v.y); f[4] = b_lo(v.z); f[5] = b_hi(v.z); f[6] = b_lo(v.w); f[7] = b_hi(v.w);
 }
 
-// A warp takes groups of four weight rows (GATED: two of gate and the same two of up); WK warps share a group and cut K.
-template <typename T, int MR, int WK, bool GATED>
+// A warp takes groups of four weight rows (GATED: two of gate and the same two of up); WK warps share a group and cut K. MORE: biases
+// and a second input are possible (others do without that code: its instructions have to be fetched, too).
+template <typename T, int MR, int WK, bool GATED, bool MORE>
 __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char gemv_raw[];
@@ -222,7 +231,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
             const T* src = static_cast<const T*>(p.x) + (size_t)m * p.x_stride;
             for (int i = tid; i < p.ld; i += kGemvThreads) { T v = T(0.0f); if (i < p.k) v = src[i]; xs[(size_t)m * p.ld + i] = v; }
         }
-        if (p.x2)
+        if (MORE && p.x2)
             for (int m = 0; m < MR; ++m) {
                 const T* src = static_cast<const T*>(p.x2) + (size_t)m * p.x2_stride;
                 for (int i = tid; i < p.ld; i += kGemvThreads) { T v = T(0.0f); if (i < p.k) v = src[i]; xs[(size_t)(MR + m) * p.ld + i] = v; }
@@ -238,7 +247,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
 #pragma unroll
             for (int m = 0; m < MR; ++m) acc[i][m] = 0.f;
         const bool live = group < groups;
-        const T* xg = xs + (p.x2 && group * ROWS >= p.split ? (size_t)MR * p.ld : 0);
+        const T* xg = xs + (MORE && p.x2 && group * ROWS >= p.split ? (size_t)MR * p.ld : 0);
         if (live) {
             for (int c0 = first_chunk; c0 < chunks; c0 += STEP * kGemvUnroll) {
                 if (it > 0 || c0 != first_chunk) load(group, c0);
@@ -300,13 +309,13 @@ __global__ void __launch_bounds__(kGemvThreads, 2) bgemv_kernel(const GemvParams
 #pragma unroll
                     for (int i = 0; i < 2; ++i) {
                         const int row = group * 2 + i;
-                        if (lane == i * MR + m && row < p.n) product_store(p.out, m, row, gated_activation(acc[i][m], acc[2 + i][m], p.act));
+                        if (lane == i * MR + m && row < p.n) product_store<false>(p.out, m, row, gated_activation(acc[i][m], acc[2 + i][m], p.act));
                     }
                 } else {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const int row = group * 4 + i;
-                        if (lane == i * MR + m && row < p.n) product_store(p.out, m, row, acc[i][m]);
+                        if (lane == i * MR + m && row < p.n) product_store<MORE>(p.out, m, row, acc[i][m]);
                     }
                 }
             }
@@ -456,8 +465,9 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
 #pragma unroll 1
             for (int t = 0; t < (GATED && !cut ? 1 : nt); ++t) {
                 const int row = row0 + (GATED ? 0 : t * kTileRows) + quarter * 32 + lane;
-                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true, 0.f}
+                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true}
                                            : product_row(p.out, row);
+                const float bias = !cut && p.out.biased && row < p.n ? product_bias(p.out, row) : 0.f;
 #pragma unroll 1
                 for (int c0 = 16 * ((warp - 2) >> 2); c0 < BN; c0 += 16 * (kTcEpilogueWarps / 4)) {
                     if (tok0 + c0 >= tok_end) break;   // uniform across the warp
@@ -473,7 +483,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
                         for (int i = 0; i < 16; ++i) {
                             float val = __uint_as_float(v[i]);
                             if (GATED && !cut) val = gated_activation(val, __uint_as_float(u[i]), p.act);
-                            val += dst.bias;
+                            val += bias;
                             if (p.out.softcap > 0.f && !cut) val = p.out.softcap * tanhf(val / p.out.softcap);
                             if (p.out.gelu && !cut) val = gelu_erf(val);
                             if (i < count) {
@@ -509,7 +519,7 @@ __global__ void __launch_bounds__(256) bgemm_sum_kernel(const float* part, int r
             a += __ldcg(base + i);
             if (GATED) b += __ldcg(base + total + i);
         }
-        product_store(out, t, r, GATED ? gated_activation(a, b, act) : a);
+        product_store<!GATED>(out, t, r, GATED ? gated_activation(a, b, act) : a);
     }
 }
 
@@ -542,16 +552,16 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const __nv_bfloat16* w, int 
     for (int i = 0; i < 4; ++i)
         for (int j = 0; j < 4; ++j) {
             const int mm = m0 + ty * 4 + i, nn = n0 + tx * 4 + j;
-            if (mm < m && nn < n) product_store(out, mm, nn, acc[i][j]);
+            if (mm < m && nn < n) product_store<true>(out, mm, nn, acc[i][j]);
         }
 }
 
 // ---- launches ---------------------------------------------------------------------------------------------------------
-template <typename T, int MR, int WK, bool GATED>
+template <typename T, int MR, int WK, bool GATED, bool MORE = false>
 int gemv_launch(const GemvParams& p, size_t smem, unsigned grid, cudaStream_t s) {
-    static const cudaError_t attr = cudaFuncSetAttribute(bgemv_kernel<T, MR, WK, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGemvMaxSmem);
+    static const cudaError_t attr = cudaFuncSetAttribute(bgemv_kernel<T, MR, WK, GATED, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kGemvMaxSmem);
     if (attr != cudaSuccess) return cuda_fail(attr, "bgemv attributes");
-    const cudaError_t e = launch_k(bgemv_kernel<T, MR, WK, GATED>, dim3(grid), dim3(kGemvThreads), smem, s, p);
+    const cudaError_t e = launch_k(bgemv_kernel<T, MR, WK, GATED, MORE>, dim3(grid), dim3(kGemvThreads), smem, s, p);
     return e == cudaSuccess ? SWLM_OK : cuda_fail(e, "bgemv launch");
 }
 template <typename T, int MR>
@@ -574,6 +584,14 @@ int gemv_pick(const GemvParams& p, bool gated, size_t smem, cudaStream_t s) {
         case 2: return gemv_launch<T, MR, 2, true>(p, smem, grid, s);
         case 4: return gemv_launch<T, MR, 4, true>(p, smem, grid, s);
         default: return gemv_launch<T, MR, 8, true>(p, smem, grid, s);
+        }
+    }
+    if (p.x2 || p.out.biased) {
+        switch (wk) {
+        case 1: return gemv_launch<T, MR, 1, false, true>(p, smem, grid, s);
+        case 2: return gemv_launch<T, MR, 2, false, true>(p, smem, grid, s);
+        case 4: return gemv_launch<T, MR, 4, false, true>(p, smem, grid, s);
+        default: return gemv_launch<T, MR, 8, false, true>(p, smem, grid, s);
         }
     }
     switch (wk) {

@@ -83,7 +83,6 @@ __device__ __forceinline__ void weigh(const RoutedParams& p, float* w, int tid) 
 
 // Experts with tensors first, those that hand the input through behind them (one warp; top <= 64); returns the number of the first.
 __device__ __forceinline__ int real_first(const RoutedShape& sh, int* sel, float* w, int lane) {
-    if (!sh.identity) return sh.top;
     const int a = lane < sh.top ? sel[lane] : 0, b = lane + 32 < sh.top ? sel[lane + 32] : 0;
     const float wa = lane < sh.top ? w[lane] : 0.f, wb = lane + 32 < sh.top ? w[lane + 32] : 0.f;
     const unsigned lower = (1u << lane) - 1u;
@@ -98,11 +97,11 @@ __device__ __forceinline__ int real_first(const RoutedShape& sh, int* sel, float
 
 // The choice of one row by THREADS threads (a warp or the CTA). s: [experts] scores, gs: [groups] group scores, both shared;
 // sel / w: [top] in order of falling score. With a correction the choice looks at s + correction, kept in cs: [scored]; the weights
-// are the plain scores.
-template <int THREADS>
+// are the plain scores. MORE: corrections and identity experts are possible (others do without that code).
+template <int THREADS, bool MORE>
 __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, float* s, float* gs, float* cs, int* sel, float* w, int tid) {
     auto sync = [] { if (THREADS == 32) __syncwarp(); else __syncthreads(); };
-    const int E = p.sh.scored(), G = p.sh.groups, per = E / G;
+    const int E = MORE ? p.sh.scored() : p.sh.experts, G = p.sh.groups, per = E / G;
     for (int i = tid; i < p.sh.top; i += THREADS) { sel[i] = i; w[i] = 0.f; }   // indices stay valid whatever the logits are
     if (p.softmax) {   // every warp works out maximum and sum for itself
         float top = -INFINITY, sum = 0.f;
@@ -115,7 +114,7 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
         for (int e = tid; e < E; e += THREADS) s[e] = 1.0f / (1.0f + expf(-z[e]));
     }
     sync();
-    if (p.correction) {
+    if (MORE && p.correction) {
         for (int e = tid; e < E; e += THREADS) cs[e] = s[e] + __bfloat162float(p.correction[e]);
         sync();
         for (int e = tid; e < E; e += THREADS) {
@@ -164,7 +163,7 @@ __device__ __forceinline__ void choose(const RoutedParams& p, const float* z, fl
 // CTA (share of the work, row). A unit of work is one row of an expert's gate with the same row of its up, or without a gate two
 // rows of up; those of the shared feed-forward come first, because they are known before the choice.
 __host__ __device__ __forceinline__ int routed_units(int ff, bool gated) { return gated ? ff : (ff + 1) / 2; }
-template <typename T, bool GATED>
+template <typename T, bool GATED, bool MORE>
 __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedParams p) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) float rt_smem[];
@@ -207,10 +206,14 @@ __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedPar
     float* s = x + p.in_ld;                // [scored], then [groups], then [scored]
     const T* src = static_cast<const T*>(p.x) + (size_t)row * p.x_stride;
     for (int i = tid; i < p.in_ld; i += kRtThreads) x[i] = i < p.sh.width ? rt_get(src + i) : 0.f;
-    choose<kRtThreads>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.scored(), s + p.sh.scored() + p.sh.groups, sel, weight, tid);
-    if (warp == 0) { const int n = real_first(p.sh, sel, weight, lane); if (lane == 0) real_s = n; }
-    __syncthreads();
-    const int units = shared + real_s * per;
+    choose<kRtThreads, MORE>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.scored(), s + p.sh.scored() + p.sh.groups, sel, weight, tid);
+    int real = p.sh.top;
+    if (MORE && p.sh.identity) {
+        if (warp == 0) { const int n = real_first(p.sh, sel, weight, lane); if (lane == 0) real_s = n; }
+        __syncthreads();
+        real = real_s;
+    }
+    const int units = shared + real * per;
     if (blockIdx.x == 0 && tid < p.sh.top) {
         p.sel[row * p.sh.top + tid] = sel[tid];
         p.weight[row * p.sh.top + tid] = weight[tid];
@@ -241,7 +244,7 @@ __global__ void __launch_bounds__(kRtThreads) routed_gate_kernel(const RoutedPar
 // CTA (share of the outputs, row): mid rows of all chosen experts, weighted, in shared memory; two warps per output, each with
 // half of the 16-byte chunks of the chosen experts' rows, those of the shared feed-forward behind them.
 constexpr int kDownUnroll = 8, kDownWarps = 2;
-template <typename T>
+template <typename T, bool MORE>
 __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -253,8 +256,8 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
     if (tid < all_top) { sel[tid] = p.sel[row * all_top + tid]; weight[tid] = p.weight[row * all_top + tid]; }
     __syncthreads();
     int top = all_top;         // experts with tensors come first
-    float through = 0.f;       // what the others hand through
-    if (p.sh.identity)
+    float through = 0.f;       // weight of the others
+    if (MORE && p.sh.identity)
         while (top > 0 && sel[top - 1] >= p.sh.experts) through += weight[--top];
     const T* input = static_cast<const T*>(p.x) + (size_t)row * p.x_stride;
     const int chunks = p.mid_ld >> 3, routed = chunks * top, all = routed + (p.shared_ld >> 3), half = warp % kDownWarps;
@@ -304,7 +307,7 @@ __global__ void __launch_bounds__(kRtThreads) routed_down_kernel(const RoutedPar
             float total = 0.f;
 #pragma unroll
             for (int w = 0; w < kDownWarps; ++w) total += part[warp + w];
-            if (p.sh.identity) total = fmaf(through, rt_get(input + n), total);
+            if (MORE && p.sh.identity) total = fmaf(through, rt_get(input + n), total);
             p.out[(size_t)row * p.out_stride + n] = total;
         }
         __syncthreads();
@@ -323,7 +326,7 @@ __global__ void __launch_bounds__(kChooseWarps * 32) routed_choose_kernel(const 
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, row = blockIdx.x * kChooseWarps + warp;
     if (row >= p.m) return;
     float* s = rt_smem + (size_t)warp * (2 * p.sh.scored() + p.sh.groups);
-    choose<32>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.scored(), s + p.sh.scored() + p.sh.groups, sel[warp], weight[warp], lane);
+    choose<32, true>(p, p.z + (size_t)row * p.z_stride, s, s + p.sh.scored(), s + p.sh.scored() + p.sh.groups, sel[warp], weight[warp], lane);
     for (int t = lane; t < p.sh.top; t += 32) {
         p.sel[row * p.sh.top + t] = sel[warp][t];
         p.weight[row * p.sh.top + t] = weight[warp][t];
@@ -438,17 +441,17 @@ constexpr size_t kRtMaxSmem = 200 * 1024;
 size_t gate_smem(const RoutedShape& s) { return ((size_t)up8(s.width) + 2 * s.scored() + s.groups) * 4; }
 size_t down_smem(const RoutedShape& s) { return ((size_t)s.top * up8(s.ff) + up8(s.shared_ff)) * 4; }
 
-template <typename T>
+template <typename T, bool MORE>
 int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
     // up to four CTAs per SM, all with the same number of rounds
     const bool gated = p.gate != nullptr;
     const int units = p.sh.top * routed_units(p.sh.ff, gated) + routed_units(p.sh.shared_ff, gated);
     const int most = std::max(1, (4 * 148 + p.m - 1) / p.m), rounds = (units + kRtWarps * most - 1) / (kRtWarps * most), gx = (units + kRtWarps * rounds - 1) / (kRtWarps * rounds);
-    cudaError_t e = gated ? launch_k(routed_gate_kernel<T, true>, dim3(gx, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p)
-                          : launch_k(routed_gate_kernel<T, false>, dim3(gx, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
+    cudaError_t e = gated ? launch_k(routed_gate_kernel<T, true, MORE>, dim3(gx, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p)
+                          : launch_k(routed_gate_kernel<T, false, MORE>, dim3(gx, p.m), dim3(kRtThreads), gate_smem(p.sh), s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed gate launch");
     const int outs = (p.sh.width * kDownWarps + kRtWarps - 1) / kRtWarps, dx = std::max(1, std::min(outs, (4 * 148 + p.m - 1) / p.m));
-    e = launch_k(routed_down_kernel<T>, dim3(dx, p.m), dim3(kRtThreads), down_smem(p.sh), s, p);
+    e = launch_k(routed_down_kernel<T, MORE>, dim3(dx, p.m), dim3(kRtThreads), down_smem(p.sh), s, p);
     if (e != cudaSuccess) return cuda_fail(e, "routed down launch");
     *launches += 2;
     return SWLM_OK;
@@ -456,13 +459,16 @@ int few_rows(const RoutedParams& p, cudaStream_t s, int* launches) {
 
 }  // namespace
 
+template <typename T, bool MORE>
+static int few_attr() {
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<T, true, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<T, false, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<T, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    return SWLM_OK;
+}
 int routed_init() {
-    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<float, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<float, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<__nv_bfloat16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(routed_gate_kernel<__nv_bfloat16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
-    SWLM_CUDA(cudaFuncSetAttribute(routed_down_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kRtMaxSmem));
+    int rc;
+    if ((rc = few_attr<float, false>()) || (rc = few_attr<float, true>()) || (rc = few_attr<__nv_bfloat16, false>()) || (rc = few_attr<__nv_bfloat16, true>())) return rc;
     return SWLM_OK;
 }
 bool routed_supported(const RoutedShape& s) {
@@ -484,7 +490,10 @@ int launch_routed(const RoutedLaunch& a, cudaStream_t s, int* launches) {
     const bool shared = a.shape.shared_ff > 0;
     if (shared) { p.shared_up = a.shared_up->data; p.shared_down = a.shared_down->data; p.shared_ld = a.shared_down->ld; }
     p.shared_mid = a.scratch + l.shared_mid; p.shared_stride = up8(a.shape.shared_ff);
-    if (few(a.m, a.f32)) return a.f32 ? few_rows<float>(p, s, launches) : few_rows<__nv_bfloat16>(p, s, launches);
+    if (few(a.m, a.f32)) {
+        if (p.correction || a.shape.identity) return a.f32 ? few_rows<float, true>(p, s, launches) : few_rows<__nv_bfloat16, true>(p, s, launches);
+        return a.f32 ? few_rows<float, false>(p, s, launches) : few_rows<__nv_bfloat16, false>(p, s, launches);
+    }
 
     const int all = a.m * a.shape.top, E = a.shape.experts;
     p.sorted = reinterpret_cast<__nv_bfloat16*>(a.scratch + l.sorted); p.sorted_stride = up8(a.shape.width);

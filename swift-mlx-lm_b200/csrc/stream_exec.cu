@@ -831,6 +831,7 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
             a.out.softcap = L.softcap;
             auto segment = [&](int q, int buf, int off, int end) {
                 a.out.bias[q] = L.seg_bias[q] ? L.seg_bias[q]->data : nullptr;
+                a.out.biased |= L.seg_bias[q] != nullptr;
                 a.out.y[q] = static_cast<unsigned char*>(b->buf[buf]) + (size_t)off * stored_bytes(plan, buf); a.out.stride[q] = s->width[buf]; a.out.f32[q] = stored_f32(plan, buf) ? 1 : 0; a.out.end[q] = end;
             };
             if (L.m2 && !product_takes_gate(m, L.m1->k, f32)) {
