@@ -27,29 +27,23 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 }
 
 // Where the results of one weight row go: that of activation row m is m * stride bytes behind y.
-struct ProductRow { unsigned char* y; size_t stride; bool f32; };
+struct ProductRow { unsigned char* y; size_t stride; bool f32; float bias; };
+template <bool BIASED>
 __device__ __forceinline__ ProductRow product_row(const ProductOut& o, int row) {
     void* y = o.y[0];
+    const __nv_bfloat16* bias = BIASED ? o.bias[0] : nullptr;
     int first = 0, stride = o.stride[0], f32 = o.f32[0];
 #pragma unroll
     for (int q = 1; q < kMaxProductSegs; ++q)
-        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; }
+        if (q < o.count && row >= o.end[q - 1]) { y = o.y[q]; first = o.end[q - 1]; stride = o.stride[q]; f32 = o.f32[q]; if (BIASED) bias = o.bias[q]; }
     const int size = f32 ? 4 : 2;
-    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0};
-}
-// what is added to the results of a weight row (only when biased)
-__device__ __forceinline__ float product_bias(const ProductOut& o, int row) {
-    const __nv_bfloat16* bias = o.bias[0];
-    int first = 0;
-#pragma unroll
-    for (int q = 1; q < kMaxProductSegs; ++q)
-        if (q < o.count && row >= o.end[q - 1]) { bias = o.bias[q]; first = o.end[q - 1]; }
-    return bias ? __bfloat162float(bias[row - first]) : 0.f;
+    return ProductRow{static_cast<unsigned char*>(y) + (ptrdiff_t)(row - first) * size, (size_t)stride * size, f32 != 0,
+                      BIASED && bias && row < o.end[o.count - 1] ? __bfloat162float(bias[row - first]) : 0.f};
 }
 template <bool BIASED>
 __device__ __forceinline__ void product_store(const ProductOut& o, int m, int row, float val) {
-    const ProductRow r = product_row(o, row);
-    if (BIASED && o.biased) val += product_bias(o, row);
+    const ProductRow r = product_row<BIASED>(o, row);
+    if (BIASED) val += r.bias;
     if (o.softcap > 0.f) val = o.softcap * tanhf(val / o.softcap);
     if (o.gelu) val = gelu_erf(val);
     if (r.f32) *reinterpret_cast<float*>(r.y + m * r.stride) = val;
@@ -465,9 +459,8 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
 #pragma unroll 1
             for (int t = 0; t < (GATED && !cut ? 1 : nt); ++t) {
                 const int row = row0 + (GATED ? 0 : t * kTileRows) + quarter * 32 + lane;
-                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true}
-                                           : product_row(p.out, row);
-                const float bias = !cut && p.out.biased && row < p.n ? product_bias(p.out, row) : 0.f;
+                const ProductRow dst = cut ? ProductRow{reinterpret_cast<unsigned char*>(p.part + ((size_t)blockIdx.z * (GATED ? 2 : 1) + (GATED ? t : 0)) * p.m * p.n + row), (size_t)p.n * 4, true, 0.f}
+                                           : product_row<true>(p.out, row);
 #pragma unroll 1
                 for (int c0 = 16 * ((warp - 2) >> 2); c0 < BN; c0 += 16 * (kTcEpilogueWarps / 4)) {
                     if (tok0 + c0 >= tok_end) break;   // uniform across the warp
@@ -483,7 +476,7 @@ __global__ void __launch_bounds__(kTcBlock) bgemm_tc_kernel(const TcParams p, co
                         for (int i = 0; i < 16; ++i) {
                             float val = __uint_as_float(v[i]);
                             if (GATED && !cut) val = gated_activation(val, __uint_as_float(u[i]), p.act);
-                            val += bias;
+                            val += dst.bias;
                             if (p.out.softcap > 0.f && !cut) val = p.out.softcap * tanhf(val / p.out.softcap);
                             if (p.out.gelu && !cut) val = gelu_erf(val);
                             if (i < count) {

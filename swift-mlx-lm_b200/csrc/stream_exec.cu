@@ -225,6 +225,7 @@ int stream_compile(swlm_plan* plan) {
     plan->latent.assign(std::max(0, d.latent_layers), LatentLayer{});
     plan->grouped.assign(std::max(0, d.grouped_layers), GroupedLayer{});
     plan->delta.assign(std::max(0, d.delta_layers), DeltaLayer{});
+    for (const swlm_step& s : st) plan->biased |= s.kind == SWLM_STEP_PRODUCT && s.weight3[0];
     plan->convs.assign(std::max(0, d.stream_convs), StreamConv{});
     int unkept = -1;   // convolution whose state does not have its last inputs yet
     widen(SWLM_BUF_HIDDEN, d.hidden);
@@ -829,9 +830,9 @@ int enqueue_rows_stream(swlm_state* s, StreamBufs* b, const RowBatch& r, bool bo
                 }
             }
             a.out.softcap = L.softcap;
+            a.out.biased = plan->biased;   // (one form of the kernel for all products of the plan: the fewer instructions, the sooner they are fetched)
             auto segment = [&](int q, int buf, int off, int end) {
                 a.out.bias[q] = L.seg_bias[q] ? L.seg_bias[q]->data : nullptr;
-                a.out.biased |= L.seg_bias[q] != nullptr;
                 a.out.y[q] = static_cast<unsigned char*>(b->buf[buf]) + (size_t)off * stored_bytes(plan, buf); a.out.stride[q] = s->width[buf]; a.out.f32[q] = stored_f32(plan, buf) ? 1 : 0; a.out.end[q] = end;
             };
             if (L.m2 && !product_takes_gate(m, L.m1->k, f32)) {

@@ -355,8 +355,8 @@ struct ProductOut {
     void* y[kMaxProductSegs] = {};
     int stride[kMaxProductSegs] = {};
     int f32[kMaxProductSegs] = {};
-    const __nv_bfloat16* bias[kMaxProductSegs] = {};   // added to the rows of a segment (null: none) when `biased`
-    int biased = 0;
+    const __nv_bfloat16* bias[kMaxProductSegs] = {};   // added to the rows of a segment; null: none
+    int biased = 0;        // are there any?
     float softcap = 0.f;   // > 0: every value v becomes softcap * tanh(v / softcap)
     int gelu = 0;          // every value v becomes v * (1 + erf(v / sqrt(2))) / 2
 };

@@ -182,6 +182,7 @@ struct swlm_plan {
     std::vector<GroupedLayer> grouped;    // by step.layer
     std::vector<DeltaLayer> delta;        // by step.layer
     std::vector<StreamConv> convs;        // by step.layer
+    bool biased = false;                  // do products have biases?
     std::vector<int> windows;             // distinct sliding windows of the attention layers
     int stream_width[SWLM_BUF_COUNT] = {};
     int latent_heads_max = 0, latent_q_floats = 0, latent_part_floats = 0;   // largest over the layers, per row / per row and split
