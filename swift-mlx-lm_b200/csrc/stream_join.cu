@@ -24,7 +24,7 @@ namespace cg = cooperative_groups;
 namespace swlm {
 namespace {
 
-constexpr int kConvRows = 16, kConvThreads = 128;
+constexpr int kConvRows = 8, kConvThreads = 128;
 constexpr int kStepCluster = 8;
 constexpr int kSideThreads = 256, kSideCluster = 16, kSideMaxRows = 16;   // rows beyond which the products of a token input run on their own
 constexpr int kStepResults = 128;   // earlier results whose weights are kept at hand
@@ -164,6 +164,23 @@ __global__ void __launch_bounds__(kConvThreads) stream_conv_kernel(const JoinLau
 #pragma unroll
         for (int e = 0; e < 4; ++e) v[e] = at >= 0 && i + e < width ? from[i + e] : 0.f;
     };
+    if (TAPS > 0 && r1 - r0 == kConvRows && r0 >= past && p.row_seq[r0 - past] == p.row_seq[r1 - 1]) {   // all rows of one portion: requested at once
+        float h[kConvRows + (TAPS > 1 ? TAPS - 1 : 0)][4];
+#pragma unroll
+        for (int n = 0; n < kConvRows + TAPS - 1; ++n) jn_get4(stream + (size_t)(r0 - past + n) * p.res_stride + i, h[n]);
+#pragma unroll
+        for (int n = 0; n < kConvRows; ++n) {
+            float y[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                y[e] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][e], h[n + TAPS - 1][e], h[n + TAPS - 1][e]);
+#pragma unroll
+                for (int d = 1; d < TAPS; ++d) y[e] = fmaf(w[TAPS - 1 - d][e], h[n + TAPS - 1 - d][e], y[e]);
+            }
+            jn_put4(static_cast<T*>(p.conv_out) + (size_t)(r0 + n) * p.conv_stride + i, y);
+        }
+        return;
+    }
     float hist[PAST][4];   // hist[d - 1]: d tokens back
     for (int r = r0; r < r1; ++r) {
         float h[4], y[4];
