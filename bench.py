@@ -720,7 +720,9 @@ def run_merudra(args, pkg):
     t = KindTimer(model, timed, prompt[0, :n])
     product_bytes = cfg.product_elems() * 2
     chosen = top * experts / (experts + identity)   # with tensors, on average
-    ours["decode_products"] = t.hbm_entry(t.decode(P.STEP_PRODUCT), product_bytes, layers)
+    # (up to 16 sequences the matrices of the token inputs belong to the launches over the stream)
+    side_bytes = layers * 2 * width * MERUDRA_SIDE * 2 if batch <= 16 else 0
+    ours["decode_products"] = t.hbm_entry(t.decode(P.STEP_PRODUCT), product_bytes - side_bytes, layers)
     ours["decode_routed"] = t.hbm_entry(t.decode(P.STEP_ROUTED_MLP), layers * reached_experts(experts, chosen, batch) * 3 * width * (ff // top) * 2, layers)
     # one row of 128 entries and a factor per token and key head
     ours["decode_grouped_step"] = t.hbm_entry(t.decode(P.STEP_GROUPED_ATTN), n_attention * batch * model.position * kv_heads * (256 + 4), n_attention)

@@ -257,8 +257,8 @@ def test_a_far_token_is_found_again(pkg, load, dtype, kind):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("taps", [2, 3, 9])
 def test_convolutions_over_the_stream_across_portions(load, dtype, taps):
-    """Nothing but the convolutions looks back (one key of weight: attention with a first token of its own per row would do, so the
-    mixer is a delta rule that forgets at once); portions shorter than the convolution, down to one and two tokens."""
+    """Nothing but the convolutions looks back (the mixer is a delta rule that forgets at once); portions shorter than the convolution,
+    down to one and two tokens."""
     cfg = mc.config(200, 72, [mc.delta(1, 1, 8, 16, mc.routed(2, 1, 3, 24), conv=1), mc.delta(1, 1, 8, 16, None, conv=1)], taps=taps, side=8)
     m = load(cfg, dtype)
     for i in range(2):
